@@ -25,22 +25,32 @@ class KvCacheConfig:
     kv_heads: int
     head_dim: int
     block_size: int = 16
-    dtype: str = "bf16"             # bf16 | fp8
+    dtype: str = "bf16"             # bf16 | fp8 | fp32
     v_head_dim: Optional[int] = None
     has_v: bool = True              # False for MLA latent caches
     high_precision_layers: tuple = ()   # cache layers kept in bf16 although dtype is fp8
+    layer_dims: Optional[tuple] = None  # per cache layer (kv_heads, K row, V row) when layers differ
 
     @property
     def elem_bytes(self) -> int:
-        return 1 if self.dtype == "fp8" else 2
+        return {"fp8": 1, "fp32": 4}.get(self.dtype, 2)
+
+    def dims(self, i: int) -> tuple:
+        """(kv heads, K row, V row) of cache layer i."""
+        if self.layer_dims:
+            return tuple(self.layer_dims[i])
+        return self.kv_heads, self.head_dim, self.v_head_dim or self.head_dim
 
     def layer_dtype(self, i: int) -> str:
         return "bf16" if (self.dtype == "fp8" and i in self.high_precision_layers) else self.dtype
 
     def block_bytes(self) -> int:
         """Bytes one block occupies across all layers (K and V)."""
-        per_elem = self.block_size * self.kv_heads * (self.head_dim + ((self.v_head_dim or self.head_dim) if self.has_v else 0))
-        return sum(per_elem * (1 if self.layer_dtype(i) == "fp8" else 2) for i in range(self.num_layers))
+        n = 0
+        for i in range(self.num_layers):
+            h, dk, dv = self.dims(i)
+            n += self.block_size * h * (dk + (dv if self.has_v else 0)) * {"fp8": 1, "fp32": 4}.get(self.layer_dtype(i), 2)
+        return n
 
     def blocks_for_budget(self, nbytes: int) -> int:
         return max(0, nbytes // max(1, self.block_bytes()))
@@ -96,7 +106,7 @@ class BlockAllocator:
 
 
 class PagedKvCache:
-    """Device pools + allocator. ``k[i]`` / ``v[i]`` index by *cache layer* (the i-th layer
+    """Device pools + allocator (layers may have their own head counts and sizes). ``k[i]`` / ``v[i]`` index by *cache layer* (the i-th layer
     that owns a pool), see ``layer_map``."""
 
     def __init__(self, cfg: KvCacheConfig, num_blocks: int, device="cpu", poison: bool = False):
@@ -105,13 +115,13 @@ class PagedKvCache:
         self.device = torch.device(device)
         from . import make_allocator
         self.allocator = make_allocator(num_blocks)
-        shape_k = (num_blocks, cfg.block_size, cfg.kv_heads, cfg.head_dim)
-        shape_v = (num_blocks, cfg.block_size, cfg.kv_heads, cfg.v_head_dim or cfg.head_dim)
         fill = torch.full if poison else None
         self.k: List[torch.Tensor] = []
         self.v: List[Optional[torch.Tensor]] = []
         for li in range(cfg.num_layers):
-            dt = torch.uint8 if cfg.layer_dtype(li) == "fp8" else torch.bfloat16
+            dt = {"fp8": torch.uint8, "fp32": torch.float32}.get(cfg.layer_dtype(li), torch.bfloat16)
+            heads, dk, dv = cfg.dims(li)
+            shape_k, shape_v = (num_blocks, cfg.block_size, heads, dk), (num_blocks, cfg.block_size, heads, dv)
             if poison:
                 # new blocks start as 0xFF bytes (NaN in bf16 / e4m3) so a read of a never
                 # written slot shows up in the output (kv_poison in the reference)

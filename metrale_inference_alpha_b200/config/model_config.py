@@ -10,20 +10,23 @@ Role of the reference's ``crates/config`` (``ModelConfig`` and the per-family pa
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 from typing import List, Optional
 
-WEIGHT_FORMATS = ("bf16", "nvfp4", "fp8_block", "fp8_row")
-KV_DTYPES = ("bf16", "fp8")
-LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda")
+WEIGHT_FORMATS = ("bf16", "nvfp4", "fp8_block", "fp8_row", "fp32")
+KV_DTYPES = ("bf16", "fp8", "fp32")
+LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning")
+KV_KINDS = ("attention", "mla", "parallel")                       # kinds that own a KV pool
+STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning")   # kinds that own a recurrent state
 FFN_KINDS = ("dense", "moe", "none")
 
 
 @dataclass
 class ModelConfig:
     name: str = "model"
-    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla
+    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix
     vocab_size: int = 4096
     hidden_size: int = 256
     num_layers: int = 2
@@ -58,6 +61,10 @@ class ModelConfig:
     residual_multiplier: float = 1.0    # Granite: a block's output is scaled by this before it joins the stream
     logits_divisor: float = 1.0         # Granite: logits are divided by this
     tie_embeddings: bool = False
+    # fabulix: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
+    layer_specs: List[dict] = field(default_factory=list)
+    token_side_dim: int = 0             # width of a layer's slice of the token side embedding (0 = none)
+    glu_alpha: float = 1.702            # sigmoid slope of the clamped GLU
     # per-layer structure
     layer_types: List[str] = field(default_factory=list)   # mixer per layer
     ffn_types: List[str] = field(default_factory=list)     # ffn per layer
@@ -158,7 +165,23 @@ class ModelConfig:
         return self.mamba_inner + 2 * self.mamba_groups * self.mamba_state
 
     def attention_layers(self) -> List[int]:
-        return [i for i, t in enumerate(self.layer_types) if t in ("attention", "mla")]
+        return [i for i, t in enumerate(self.layer_types) if t in KV_KINDS]
+
+    @property
+    def act_fmt(self) -> str:
+        """Activation type of models with a 32-bit residual stream: bf16, or fp32 when served in 32-bit."""
+        return "fp32" if self.weight_format == "fp32" else "bf16"
+
+    def kv_layer_dims(self) -> List[tuple]:
+        """(kv heads, K row, V row) of every KV pool of a model whose layers have their own head sizes; the
+        rows are padded to what the attention kernels tile."""
+        from ..ops.mixers import padded_head_dims
+        out = []
+        for t, sp in zip(self.layer_types, self.layer_specs):
+            if t == "parallel":
+                m = sp["mixer"]["left"]
+                out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
+        return out
 
     def kv_bytes_per_token(self) -> int:
         e = 1 if self.kv_dtype == "fp8" else 2
@@ -168,11 +191,15 @@ class ModelConfig:
                 n += 2 * self.num_kv_heads * self.head_dim * e
             elif t == "mla":
                 n += (self.kv_lora_rank + self.qk_rope_dim) * e
+        n += sum(h * (dk + dv) * (4 if self.kv_dtype == "fp32" else 2) for h, dk, dv in self.kv_layer_dims())
         return n + self.mtp_layers * 2 * self.num_kv_heads * self.head_dim * e * (self.arch != "deepseek_mla")
 
     def param_count(self) -> int:
         """Approximate parameter count (linear layers + embeddings)."""
         h = self.hidden_size
+        if self.arch == "fabulix":
+            from ..weights.fabulix import tensor_shapes
+            return sum(math.prod(s) for s, _ in tensor_shapes(self).values())
         n = self.vocab_size * h * (1 if self.tie_embeddings else 2)
         for lt, ft in zip(self.layer_types, self.ffn_types):
             if lt == "attention":
@@ -325,8 +352,49 @@ def tiny_kimi_linear(**kw) -> ModelConfig:
     return qwen_hybrid_moe_35b(**base)
 
 
+def fabulix(num_layers: int = 4, width: int = 256, heads: int = 4, kv_heads: int = 2, dim: int = 64, vdim: int = 64, rot_dims: int = 32,
+            rot_base: float = 10000.0, right_heads: int = 4, right_dim: int = 64, lin_heads: int = 4, lin_dim: int = 64, lin_vdim: int = 64,
+            ff: int = 512, limit: float = 3.0, side_dim: int = 16, vocab: int = 1024, period: int = 3, eps: float = 1e-5, **kw) -> ModelConfig:
+    """Fabulix decoder of uniform layers: every `period`-th layer is a lightning mixer, the others run sink
+    attention and RWKV-style time mixing side by side; clamped-GLU feed-forward, Dynamic-Tanh norms before
+    and after every sublayer, a token side input per layer, tied embeddings."""
+    layers = []
+    for i in range(num_layers):
+        if i % period == period - 1:
+            m = {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim,
+                 "decay": [1.0 - 2.0 ** -(1.0 + 6.0 * (h + 1) / lin_heads) for h in range(lin_heads)]}
+            layers.append({"type": "lightning", "mixer": m, "mlp": {"kind": "dense", "ff": ff, "limit": limit}})
+        else:
+            left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                    "rot": {"base": rot_base, "dims": rot_dims}}
+            layers.append({"type": "parallel", "mlp": {"kind": "dense", "ff": ff, "limit": limit},
+                           "mixer": {"left": left, "right": {"heads": right_heads, "dim": right_dim},
+                                     "left_scale": 0.7, "right_scale": 0.7}})
+    cfg = {"architecture": "Fabulix", "vocab": vocab, "width": width, "embedding": {"scale": float(width) ** 0.5},
+           "norm": {"eps": eps}, "layers": layers}
+    if side_dim:
+        cfg["token_side"] = {"dim": side_dim}
+    return from_fabulix_config(cfg, name=kw.pop("name", "fabulix")).scaled(**kw)
+
+
+def tiny_fabulix(**kw) -> ModelConfig:
+    """Four-layer Fabulix (tests, smoke runs)."""
+    return fabulix(**{"name": "tiny-fabulix", **kw})
+
+
+def fabulix_3b(**kw) -> ModelConfig:
+    """Fabulix with the layer sizes of a ~3B model: width 2560, 20 query / 4 key-value heads of 128, 20
+    time-mixing heads of 128, lightning layers of 20 heads of 128, feed-forward 6912, 24 layers."""
+    base = dict(name="fabulix-3b", num_layers=24, width=2560, heads=20, kv_heads=4, dim=128, vdim=128, rot_dims=128, right_heads=20,
+                right_dim=128, lin_heads=20, lin_dim=128, lin_vdim=128, ff=6912, side_dim=128, vocab=65536)
+    base.update(kw)
+    return fabulix(**base)
+
+
 PRESETS = {
     "tiny-dense": tiny_dense,
+    "tiny-fabulix": tiny_fabulix,
+    "fabulix-3b": fabulix_3b,
     "tiny-kimi-linear": tiny_kimi_linear,
     "tiny-dense-hc": tiny_dense_hc,
     "tiny-hybrid-moe": tiny_hybrid_moe,
@@ -383,8 +451,38 @@ def detect_weight_format(qc: Optional[dict]) -> str:
     raise ValueError(f"unsupported quant_method {method!r}")
 
 
+def from_fabulix_config(cfg: dict, name: str = "model") -> ModelConfig:
+    """A Fabulix ``config.json``: sizes and constants are given per layer and kept per layer. Mixer types and
+    feed-forward kinds this engine does not know are refused."""
+    types, ffns, specs = [], [], []
+    for i, L in enumerate(cfg["layers"]):
+        t, m, mlp = L["type"], L["mixer"], L.get("mlp")
+        if t not in ("parallel", "lightning"):
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+        if mlp is not None and mlp.get("kind") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        if t == "parallel":
+            a = m["left"]
+            if a["heads"] % a["kv_heads"] or a["rot"]["dims"] % 2 or a["rot"]["dims"] > a["dim"]:
+                raise ValueError(f"layer {i}: attention heads, key/value heads or rotary size do not fit together")
+        elif len(m["decay"]) != m["heads"]:
+            raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+        types.append(t)
+        ffns.append("none" if mlp is None else "dense")
+        specs.append({"mixer": m, "mlp": mlp})
+    att = next((s["mixer"]["left"] for t, s in zip(types, specs) if t == "parallel"), {"heads": 1, "kv_heads": 1, "dim": 64})
+    return ModelConfig(
+        name=name, arch="fabulix", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(types), layer_types=types,
+        ffn_types=ffns, layer_specs=specs, num_heads=att["heads"], num_kv_heads=att["kv_heads"], head_dim=att["dim"], rotary_dim=-1,
+        rms_eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), tie_embeddings=True,
+        intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"]), default=0),
+        token_side_dim=int((cfg.get("token_side") or {}).get("dim", 0)), max_position=131072)
+
+
 def from_hf_config(cfg: dict, name: str = "model") -> ModelConfig:
     """Map a HF ``config.json`` dict (text stack) to ModelConfig; refuses unknown model types."""
+    if cfg.get("architecture") == "Fabulix":
+        return from_fabulix_config(cfg, name)
     outer = cfg
     if "text_config" in cfg:
         inner = dict(cfg["text_config"])

@@ -44,6 +44,12 @@ def state_shapes(cfg: ModelConfig, w: ModelW):
             m = lw.mixer
             C = m.heads * cfg.mamba_head_dim + 2 * m.groups * cfg.mamba_state
             out.append(((C, cfg.conv_kernel - 1), (m.heads, cfg.mamba_head_dim, cfg.mamba_state)))
+        elif lw.kind == "parallel":                # the token shift's window is the previous token's mixer input
+            m = lw.mixer.right
+            out.append(((cfg.hidden_size,), (m.heads, m.dim, m.dim)))
+        elif lw.kind == "lightning":
+            m = lw.mixer
+            out.append(((0,), (m.heads, m.dim, m.vdim)))
     return out
 
 
@@ -53,6 +59,9 @@ def kv_config(cfg: ModelConfig, w: ModelW, block_size: int, mtp: bool = False) -
         return KvCacheConfig(1 if mtp else len(cfg.attention_layers()), 1, cfg.kv_lora_rank + cfg.qk_rope_dim,
                              block_size, cfg.kv_dtype if cfg.kv_dtype == "bf16" else "bf16",
                              v_head_dim=cfg.index_head_dim if cfg.index_topk > 0 else None, has_v=cfg.index_topk > 0)
+    if cfg.arch == "fabulix":
+        dims = tuple(cfg.kv_layer_dims()) or ((1, 16, 16),)      # a model without attention keeps a token-sized pool
+        return KvCacheConfig(len(dims), dims[0][0], dims[0][1], block_size, cfg.kv_dtype, layer_dims=dims)
     kvh = cfg.num_kv_heads
     for lw in ([w.mtp.layer] if (mtp and w.mtp) else w.layers):
         if lw.kind == "attention":

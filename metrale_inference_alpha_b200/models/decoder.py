@@ -17,11 +17,13 @@ from typing import List, Optional, Tuple
 import torch
 
 from .. import ops
-from ..config.model_config import ModelConfig
+from ..config.model_config import KV_KINDS, STATE_KINDS, ModelConfig
 from ..engine.batch import ForwardBatch
 from ..ops import ACT_FOR_WEIGHT, Act
 from ..ops import reference as ref
+from ..ops import mixers
 from ..weights.loader import AttnW, FfnW, LayerW, ModelW
+from .stream import ResidualStream
 
 
 class LayerCaches:
@@ -32,10 +34,10 @@ class LayerCaches:
         self.kv_index, self.state_index = {}, {}
         a = s = 0
         for i, t in enumerate(cfg.layer_types):
-            if t in ("attention", "mla"):
+            if t in KV_KINDS:
                 self.kv_index[i] = a
                 a += 1
-            else:
+            if t in STATE_KINDS:
                 self.state_index[i] = s
                 s += 1
 
@@ -84,14 +86,27 @@ class Decoder:
         self.kv_cal = None                 # cache.fp8_calibration.Fp8KvCalibration while FP8 KV scales are being calibrated
         self.lora = None                   # lora.LoraManager when adapters are served
         self.calib = None                  # dict while calibrating static activation scales (engine/runner.py)
+        self._rotary = {}                  # (rotated dims, base) -> cos / sin tables of layers with their own rotation
         self.side_head = None              # speculative.dflash.DflashDrafter: sees chosen layers' hidden states of every forward
 
     # ------------------------------------------------------------------ helpers
+    def rotary(self, dims: int, base: float):
+        """cos / sin [max_position, dims / 2] of a layer that names its own rotated size and base."""
+        if dims <= 0:
+            return None, None
+        key = (dims, float(base))
+        if key not in self._rotary:
+            self._rotary[key] = ref.rope_tables(self.cfg.max_position, dims, base, device=self.device)
+        return self._rotary[key]
+
     def _norm_act(self, x, w, fmt: str, also_bf16: bool = False, res_only: bool = False) -> Act:
         """RMSNorm(x) encoded for the GEMM that consumes it. When x is a pending cross-rank sum
         the norm kernel performs the sum (+ residual) itself; afterwards ``self.res(x)`` is the
         summed stream. `res_only`: the caller uses that stream only as the residual of the next
         row-parallel projection, so each rank may keep just its own row share."""
+        if isinstance(w, mixers.DytNorm):
+            s = x if isinstance(x, ResidualStream) else ResidualStream(x, self.cfg.act_fmt)
+            return mixers.act_of(s.norm(w), s.fmt)
         if hasattr(x, "resolve"):
             if w is None:
                 x = x.resolve()
@@ -222,6 +237,8 @@ class Decoder:
             hb = (torch.nn.functional.gelu(gu[:, :inter].float(), approximate="tanh") * gu[:, inter:].float()
                   ).to(torch.bfloat16)
             h = self._as_act(hb, fmt_d)
+        elif w.clamp_glu is not None:
+            h = mixers.act_of(ops.linear(a, w.gate_up, clamp_glu=w.clamp_glu), fmt_d)
         elif w.interleaved:
             static = w.down_in_scale if (fmt_d == "nvfp4" and self.calib is None) else 0.0
             if static > 0.0 and lora is None:
@@ -248,6 +265,9 @@ class Decoder:
         if lw.ffn_kind == "none":
             return x
         if lw.ffn_kind == "dense":
+            if isinstance(x, ResidualStream):            # the output joins through its post-norm in the next norm's kernel
+                y = self.dense_ffn(self._norm_act(x, lw.ln2, ACT_FOR_WEIGHT[lw.ffn.gate_up.fmt]), lw.ffn, None)
+                return x.add(y, lw.post_ffn)
             plain = lw.post_ffn is None and self.cfg.residual_multiplier == 1.0
             a = self._norm_act(x, lw.ln2, ACT_FOR_WEIGHT[lw.ffn.gate_up.fmt], res_only=plain)
             x = self.res(x)
@@ -294,10 +314,22 @@ class Decoder:
             kv = kv or caches.kv
             j = caches.kv_index[i] if kv_idx is None else kv_idx
             x = mla_block(self, x, lw, batch, kv, j)
-        return self.ffn_block(x, lw, batch, i)
+        elif lw.kind == "parallel":
+            from .parallel_mix import parallel_block
+            x = parallel_block(self, x, lw, batch, caches.kv, caches.kv_index[i], caches.state, caches.state_index[i])
+        elif lw.kind == "lightning":
+            from .parallel_mix import lightning_block
+            x = lightning_block(self, x, lw, batch, caches.state, caches.state_index[i])
+        x = self.ffn_block(x, lw, batch, i)
+        if lw.side is not None:
+            from .parallel_mix import token_side
+            x = token_side(self, x, lw.side, batch)
+        return x
 
     # ------------------------------------------------------------------ full forward
     def embed(self, token_ids: torch.Tensor) -> torch.Tensor:
+        if self.cfg.arch == "fabulix":             # 32-bit residual stream
+            return ResidualStream(mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale), self.cfg.act_fmt)
         x = ops.embed(token_ids, self.w.embed)
         if self.cfg.embed_scale != 1.0:
             x = x * torch.tensor(self.cfg.embed_scale, dtype=torch.bfloat16).to(x.dtype)
@@ -352,7 +384,7 @@ class Decoder:
 
     def logits(self, hidden_rows, final_norm=None, out_f32: bool = False, gather: bool = True) -> torch.Tensor:
         """Final norm + (vocab-parallel) lm_head on the selected rows."""
-        a = self._norm_act(hidden_rows, self.w.final_norm if final_norm is None else final_norm, "bf16")
+        a = self._norm_act(hidden_rows, self.w.final_norm if final_norm is None else final_norm, ACT_FOR_WEIGHT[self.w.lm_head.fmt])
         lg = ops.linear(a, self.w.lm_head, out_f32=out_f32)
         if self.cfg.logits_divisor != 1.0:
             lg = (lg.float() / self.cfg.logits_divisor).to(lg.dtype)

@@ -103,7 +103,10 @@ def commit_recurrent(cfg, pool, stash, commit_batch) -> None:
     sequence (0 = leave the sequence's state as it was)."""
     for sidx, (kind, lw, x_in, conv_out, gate) in stash.layers.items():
         w = lw.mixer
-        if kind == "gdn":
+        if kind in ("parallel", "lightning"):
+            from .parallel_mix import commit
+            commit(kind, lw, x_in, conv_out, gate, pool, sidx, commit_batch)
+        elif kind == "gdn":
             kd, vd, kh, vh = cfg.gdn_k_dim, cfg.gdn_v_dim, w.k_heads, w.v_heads
             rops.causal_conv1d(x_in, 2 * kh * kd + vh * vd, w.conv_w, None, pool.conv[sidx], commit_batch,
                                activation=True, write_out=False)

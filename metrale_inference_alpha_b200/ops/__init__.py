@@ -20,7 +20,7 @@ import torch
 from . import _native, reference as ref
 
 KIND = {"bf16": 0, "fp8_row": 1, "nvfp4": 2, "fp8_block": 3}
-NATIVE_ACT_FOR_WEIGHT = {"bf16": "bf16", "fp8_row": "fp8_row", "fp8_block": "fp8_g128", "nvfp4": "nvfp4"}
+NATIVE_ACT_FOR_WEIGHT = {"bf16": "bf16", "fp8_row": "fp8_row", "fp8_block": "fp8_g128", "nvfp4": "nvfp4", "fp32": "fp32"}
 # the activation encoding each weight format is fed with; `set_activation_precision` rewrites it in place
 ACT_FOR_WEIGHT = dict(NATIVE_ACT_FOR_WEIGHT)
 IN_COPY, IN_RMSNORM, IN_SILU_MUL, IN_RELU2, IN_SIGMOID_GATE, IN_GATED_RMSNORM = range(6)
@@ -33,6 +33,7 @@ GEMM_ONE_TILE_PER_CTA, GEMM_DECODE_TILE_ORDER, GEMM_PERSISTENT_PREFILL, GEMM_DSM
 # measure 1.5x faster there; METRALE_PERSISTENT_PREFILL=0 keeps one tile per CTA)
 _PERSIST_PREFILL = GEMM_PERSISTENT_PREFILL if os.environ.get("METRALE_PERSISTENT_PREFILL", "1") != "0" else 0
 GEMM_GROUPED_ONE_CTA = 512
+EPI_CLAMP_GLU, EPI_SILU_COLS, EPI_NEG_EXP = 2, 3, 4      # csrc/epilogue.cuh
 _GROUPED_CTAS = GEMM_GROUPED_ONE_CTA if os.environ.get("METRALE_GROUPED_CTAS", "2") == "1" else 0
 
 
@@ -105,6 +106,7 @@ class QuantWeight:
     fp8_row    u8   [N, K]         fp32 [N]
     fp8_block  u8   [N, K]         fp32 [ceil(N/128), ceil(K/128)]
     nvfp4      u8   [N, K/2]       u8 e4m3 [N, K/16] (+ tiled copy on CUDA), gscale fp32
+    fp32       fp32 [N, K]         -  (models served in true 32-bit: CUDA-core GEMM)
     """
     fmt: str
     N: int
@@ -120,7 +122,7 @@ class QuantWeight:
     def dequant(self) -> torch.Tensor:
         if self._deq is not None:
             return self._deq
-        if self.fmt == "bf16":
+        if self.fmt in ("bf16", "fp32"):
             d = self.data.float()
         elif self.fmt == "fp8_row":
             d = ref.from_e4m3(self.data) * self.scale.float()[:, None]
@@ -175,6 +177,8 @@ def make_weight(w: torch.Tensor, fmt: str) -> QuantWeight:
     N, K = w.shape
     if fmt == "bf16":
         return QuantWeight("bf16", N, K, w.to(torch.bfloat16).contiguous())
+    if fmt == "fp32":
+        return QuantWeight("fp32", N, K, w.float().contiguous())
     if fmt == "fp8_row":
         q, s = ref.quantize_fp8_rowwise(w)
         return QuantWeight("fp8_row", N, K, q, s)
@@ -342,6 +346,8 @@ def encode_act_ref(y: torch.Tensor, fmt: str, static_scale: float = 0.0) -> Act:
     M, K = y.shape
     if fmt == "bf16":
         d = ref.bf16_round(y)
+    elif fmt == "fp32":
+        d = y.float()
     elif fmt == "fp8_row":
         q, s = ref.quantize_fp8_rowwise(y)
         d = ref.from_e4m3(q) * s[:, None]
@@ -366,7 +372,7 @@ def set_activation_precision(mode: str) -> None:
     outliers that 4- or 8-bit rows cannot hold. Process-wide. Expert GEMMs keep the native format."""
     assert mode in ("native", "a16"), mode
     for k, v in NATIVE_ACT_FOR_WEIGHT.items():
-        ACT_FOR_WEIGHT[k] = v if mode == "native" else "bf16"
+        ACT_FOR_WEIGHT[k] = v if mode == "native" or k == "fp32" else "bf16"
 
 
 _A16_GEMV_MAX_M = 32           # up to this many rows: passes of the streaming kernel, 8 rows each
@@ -418,10 +424,39 @@ def _linear_a16(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool,
     return out
 
 
+def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual):
+    if clamp_glu is not None:
+        alpha, limit = clamp_glu
+        g, u = y[:, 0::2].clamp(max=limit), y[:, 1::2].clamp(-limit, limit)
+        y = g * torch.sigmoid(alpha * g) * (u + 1.0)
+    elif swiglu:
+        y = torch.nn.functional.silu(y[:, 0::2]) * y[:, 1::2]
+    elif silu_cols > 0:
+        y = torch.cat([torch.nn.functional.silu(y[:, :silu_cols]), y[:, silu_cols:]], 1)
+    return y if residual is None else y + residual.float()
+
+
+def _linear_simt(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool, out, clamp_glu, silu_cols: int):
+    """CUDA-core GEMM (csrc/gemm_simt.cu); on CPU its fp64-accumulated restatement."""
+    assert not swiglu and residual is None, "the CUDA-core GEMM has no SwiGLU or residual epilogue"
+    f32 = out_f32 or w.fmt == "fp32"
+    if not act.data.is_cuda:
+        y = _linear_epilogue_ref((act.data.double() @ w.dequant64().t()).float(), False, clamp_glu, silu_cols, None)
+        y = y if f32 else y.to(torch.bfloat16)
+        return y if out is None else out.copy_(y)
+    from .mixers import gemm_simt
+    if out is None:
+        out = torch.empty(act.M, w.N // 2 if clamp_glu else w.N, dtype=torch.float32 if f32 else torch.bfloat16, device=act.data.device)
+    if clamp_glu is not None:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_CLAMP_GLU, epi_a=clamp_glu[0], epi_b=clamp_glu[1])
+    return gemm_simt(act.data, w.data, out, epilogue=EPI_SILU_COLS if silu_cols else 0, epi_n=silu_cols)
+
+
 def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
            swiglu: bool = False, out_f32: bool = False, out: Optional[torch.Tensor] = None,
            force_tn: int = 0, force_splits: int = 0, one_tile_per_cta: bool = False, decode_tile_order: bool = False,
-           dsmem_splitk: bool = False, grouped=None, no_cluster: bool = False, quant_out: float = 0.0):
+           dsmem_splitk: bool = False, grouped=None, no_cluster: bool = False, quant_out: float = 0.0,
+           clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0):
     """out[m, n] = sum_k act[m, k] * w[n, k] (+ residual); with `swiglu`, w holds gate/up rows
     interleaved (2j, 2j+1) and the result is silu(gate) * up of width N/2. `quant_out` > 0 (with
     `swiglu`): return the result as an NVFP4 `Act` quantised with that calibrated global scale --
@@ -429,8 +464,13 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     `one_tile_per_cta` keeps the shape off the persistent kernel and `decode_tile_order` keeps
     prefill-sized GEMMs on the decode launch order; `dsmem_splitk` makes a split-K cluster exchange
     its partial tiles over distributed shared memory instead of the L2-resident workspace (all
-    three for A/B comparisons and tests)."""
+    three for A/B comparisons and tests). `clamp_glu` = (alpha, limit): like `swiglu` with the gate
+    g = min(gate, limit) and u = clamp(up, -limit, limit), result g * sigmoid(alpha g) * (u + 1).
+    `silu_cols`: SiLU on the first that many output columns. An fp32 weight gives fp32 outputs."""
     assert act.K == w.K, (act.K, w.K)
+    if w.fmt == "fp32" or (act.data.is_cuda and w.fmt == "bf16" and w.K % 8):
+        # true 32-bit, or bf16 rows that are not whole 16-byte vectors (no tensor map can describe them)
+        return _linear_simt(act, w, residual, swiglu, out_f32, out, clamp_glu, silu_cols)
     a16 = act.fmt == "bf16" and w.fmt != "bf16"
     assert a16 or act.fmt == NATIVE_ACT_FOR_WEIGHT[w.fmt], (act.fmt, w.fmt)
     M, N = act.M, w.N
@@ -451,14 +491,11 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         # (fp32 BLAS picks different blockings for different M, and a random-weight test model has
         # near-ties everywhere), so that batch-invariance tests on the CPU path are exact
         y = (act.data.double() @ w.dequant64().t()).float()
-        if swiglu:
-            y = torch.nn.functional.silu(y[:, 0::2]) * y[:, 1::2]
-        if residual is not None:
-            y = y + residual.float()
+        y = _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual)
         return y if out_f32 else y.to(torch.bfloat16)
     L = _native.lib()
     rt = runtime(act.data.device)
-    n_out = N // 2 if swiglu else N
+    n_out = N // 2 if (swiglu or clamp_glu) else N
     if grouped is not None:
         n_out = grouped[3] // 2 if swiglu else grouped[3]
     if out is None and quant_out <= 0.0:
@@ -482,6 +519,10 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         a.w_scale = _ptr(w.row_gscale)
         a.alpha = w.gscale
     a.epilogue, a.out_f32 = int(swiglu), int(out_f32)
+    if clamp_glu is not None:
+        a.epilogue, a.epi_a, a.epi_b = EPI_CLAMP_GLU, clamp_glu[0], clamp_glu[1]
+    elif silu_cols > 0:
+        a.epilogue, a.epi_n = EPI_SILU_COLS, silu_cols
     a.ws, a.ws_bytes, a.status = _ptr(rt.ws), rt.ws_bytes, _ptr(rt.status)
     a.force_tn, a.force_splits, a.sm_count = force_tn, force_splits, rt.sm_count
     a.flags = (_PERSIST_PREFILL | _GROUPED_CTAS | (GEMM_ONE_TILE_PER_CTA if one_tile_per_cta else 0)
@@ -530,7 +571,7 @@ def concat_weights(ws) -> QuantWeight:
     assert all(w.fmt == fmt and w.K == K for w in ws)
     data = torch.cat([w.data for w in ws], 0)
     N = sum(w.N for w in ws)
-    if fmt == "bf16":
+    if fmt in ("bf16", "fp32"):
         return QuantWeight(fmt, N, K, data)
     if fmt == "fp8_block":
         assert all(w.N % 128 == 0 for w in ws[:-1]), "block-scaled parts must be 128-row aligned"

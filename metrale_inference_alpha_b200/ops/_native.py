@@ -29,6 +29,7 @@ class GemmArgs(C.Structure):
         ("outq", c_void_p), ("ldq", c_int), ("outq_sf", c_void_p), ("outq_sf_k64", c_int), ("outq_gs", c_float),
         ("tile_expert", c_void_p), ("tile_row0", c_void_p), ("tile_nrows", c_void_p),
         ("n_per_expert", c_int), ("max_tiles", c_int),
+        ("epi_a", c_float), ("epi_b", c_float), ("epi_n", c_int),
     ]
 
 
@@ -53,6 +54,7 @@ class AttnTcArgs(C.Structure):
         ("out", c_void_p), ("status", c_void_p), ("num_blocks", c_ll),
         ("max_blocks", c_int), ("num_seqs", c_int), ("max_q_len", c_int), ("Hq", c_int), ("Hkv", c_int), ("D", c_int),
         ("block_size", c_int), ("cache_fp8", c_int), ("scale", c_float), ("v_mn", c_int),
+        ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
     ]
 
 
@@ -92,6 +94,7 @@ class AttnArgs(C.Structure):
         ("ws", c_void_p), ("ws_bytes", c_size_t), ("total_rows", c_int),
         ("part_tokens", c_int), ("window", c_int), ("force_mode", c_int), ("status", c_void_p),
         ("outq", c_void_p), ("ldq", c_int), ("outq_sf", c_void_p), ("outq_sf_k64", c_int), ("outq_gs", c_float),
+        ("DV", c_int), ("dv", c_int), ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
     ]
 
 

@@ -25,6 +25,7 @@
 // reshape_and_cache.cu, rope.cu, paged_decode_attn{,_fp8,_bf16_gqa,_fp8_gqa}.cu
 // (+ split-K reduce), prefill_paged_compute.cuh and attn_prefill_paged{,_fp8,_batched}.cu.
 #include "common.cuh"
+#include <type_traits>
 
 namespace {
 
@@ -251,6 +252,12 @@ struct AttnParams {
   uint8_t* outq_sf;
   int outq_sf_k64;
   float outq_gs;
+  // output layout and softmax variants
+  long long out_ld;         // elements between consecutive tokens' output rows
+  int dv;                   // value columns stored per head (<= the DV tile; the cache rows' padding is dropped)
+  float out_scale;          // multiplies the normalised output
+  int sink;                 // one is added to the softmax denominator (a key of score 0 without a value)
+  int split_p;              // the weights enter the product with V as two bf16 terms (16 mantissa bits)
 };
 
 // Final store of four consecutive dims (c4 * 4 ..) of output row `orow` = token * Hq + head. In the
@@ -275,9 +282,24 @@ __device__ __forceinline__ void store_out4(const AttnParams& p, size_t orow, int
     }
     return;
   }
-  __nv_bfloat16* dst = p.out + orow * D + c4 * 4;
-  *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a, b);
-  *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(c, d);
+  const size_t m = orow / p.Hq;
+  __nv_bfloat16* dst = p.out + m * p.out_ld + (orow - m * p.Hq) * p.dv + c4 * 4;
+  const float os = p.out_scale;
+  if (p.dv == D) {
+    *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a * os, b * os);
+    *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(c * os, d * os);
+    return;
+  }
+  const float v[4] = {a, b, c, d};
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (c4 * 4 + i < p.dv) dst[i] = __float2bfloat16(v[i] * os);
+}
+
+// the second bf16 term of two fp32 weights: w - bf16(w)
+__device__ __forceinline__ uint32_t pack_rest(float a, float b) {
+  const __nv_bfloat162 r = __floats2bfloat162_rn(a - __bfloat162float(__float2bfloat16(a)), b - __bfloat162float(__float2bfloat16(b)));
+  return *reinterpret_cast<const uint32_t*>(&r);
 }
 
 // Stage a [64 x D] tile of cache rows for one kv head into shared memory.
@@ -388,23 +410,51 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <int D, bool FP8, int MT>
+template <int DK, int DV, bool FP8, int MT>
 struct SplitKvCfg {
-  static constexpr int kRowB = FP8 ? D : 2 * D;                // bytes per cached row in smem
-  static constexpr int kTileB = 64 * kRowB;                    // one K (or V) tile
+  static constexpr int kRowK = FP8 ? DK : 2 * DK;              // bytes per cached row in smem
+  static constexpr int kRowV = FP8 ? DV : 2 * DV;
+  static constexpr int kTileK = 64 * kRowK, kTileV = 64 * kRowV;
   static constexpr int kStages = 3;
-  static constexpr int kPipeB = kStages * 2 * kTileB;
-  static constexpr int kMergeB = 4 * MT * 16 * 2 * 4 + 4 * MT * 16 * D * 4;
+  static constexpr int kStageB = kTileK + kTileV;
+  static constexpr int kPipeB = kStages * kStageB;
+  static constexpr int kMergeB = 4 * MT * 16 * 2 * 4 + 4 * MT * 16 * DV * 4;
   static constexpr int kSmem = kPipeB > kMergeB ? kPipeB : kMergeB;
 };
 
-template <int D, bool FP8, int MT>
-__global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_splitkv_kernel(const AttnParams p) {
-  using C = SplitKvCfg<D, FP8, MT>;
+// Global -> shared copies of one 64-token tile of a cache whose rows are ROWB bytes.
+template <int ROWB>
+struct TileCopy {
+  static constexpr int kChunks = ROWB / 16;                    // 16-byte chunks per row
+  static constexpr int kCopies = (64 * kChunks) / 128;
+  // When the rows a thread copies are a whole number of cache blocks apart, everything but the
+  // block id is the same for every tile: one shared-memory read and one multiply-add per copy.
+  static constexpr int kStep = (kChunks <= 128 && 128 % kChunks == 0) ? 128 / kChunks : 0;   // rows between copies
+  const uint8_t* cache;
+  size_t row_pitch, gbase, blk_pitch;
+  uint32_t soff0;
+  int r0, bsel0, bstep;
+  bool lin;
+  __device__ __forceinline__ TileCopy(const void* c, int Hkv, int kvh, int bs, int bs_shift, bool fast_blocks, int tid) {
+    cache = reinterpret_cast<const uint8_t*>(c);
+    row_pitch = (size_t)Hkv * ROWB;                            // bytes between consecutive tokens
+    lin = fast_blocks && kStep > 0 && (kStep % bs) == 0 && kCopies <= 8;
+    r0 = tid / kChunks;
+    const int c0 = tid % kChunks;
+    soff0 = raw_off<ROWB>(r0, c0);                             // kStep % 8 == 0: the swizzle term is fixed
+    gbase = (size_t)(r0 & (bs - 1)) * row_pitch + (size_t)kvh * ROWB + (size_t)c0 * 16;
+    blk_pitch = (size_t)bs * row_pitch;
+    bsel0 = r0 >> bs_shift;
+    bstep = kStep >> bs_shift;
+  }
+};
+
+template <int DK, int DV, bool FP8, int MT>
+__global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 : 1) attn_splitkv_kernel(const AttnParams p) {
+  using C = SplitKvCfg<DK, DV, FP8, MT>;
   constexpr bool F16 = FP8;
   constexpr int kTile = 64;
-  constexpr int kRowB = C::kRowB, kTileB = C::kTileB, kStages = C::kStages;
-  constexpr int kChunks = kRowB / 16;                          // 16-byte chunks per row
+  constexpr int kRowK = C::kRowK, kRowV = C::kRowV, kTileK = C::kTileK, kStages = C::kStages;
   extern __shared__ __align__(128) uint8_t smem_attn[];
   const uint32_t sbase = mb::smem_u32(smem_attn);
   const int kvh = blockIdx.x, seq = blockIdx.y, part = blockIdx.z;
@@ -447,42 +497,27 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
     }
   }
   __syncthreads();
-  // per-thread constants of the copy pattern: chunk i of a tile is row r_i, 16-byte column c_i
-  constexpr int kCopies = (64 * kChunks) / 128;
-  const size_t row_pitch = (size_t)p.Hkv * kRowB;              // bytes between consecutive tokens
-  // When the rows a thread copies are a whole number of cache blocks apart, everything but the
-  // block id is the same for every tile: one shared-memory read and one multiply-add per copy.
-  constexpr int kStep = (kChunks <= 128 && 128 % kChunks == 0) ? 128 / kChunks : 0;   // rows between copies
-  const bool lin = fast_blocks && kStep > 0 && (kStep % bs) == 0 && kCopies <= 8;
-  const int r0 = tid / kChunks, c0 = tid % kChunks;
-  const uint32_t soff0 = raw_off<kRowB>(r0, c0);               // kStep % 8 == 0: the swizzle term is fixed
-  const size_t gbase = (size_t)(r0 & (bs - 1)) * row_pitch + (size_t)kvh * kRowB + (size_t)c0 * 16;
-  const size_t blk_pitch = (size_t)bs * row_pitch;
-  const int bsel0 = r0 >> bs_shift, bstep = kStep >> bs_shift;
-  auto issue_tile = [&](int it) {
-    const int stage = it % kStages;
-    const uint32_t sK = sbase + stage * 2 * kTileB, sV = sK + kTileB;
-    const int tok0 = tok_begin + it * kTile;
-    const int blk0 = (tok0 - tok_begin) >> bs_shift;
-    if (lin) {
+  const TileCopy<kRowK> ck(p.k_cache, p.Hkv, kvh, bs, bs_shift, fast_blocks, tid);
+  const TileCopy<kRowV> cv(p.v_cache, p.Hkv, kvh, bs, bs_shift, fast_blocks, tid);
+  auto issue_lin = [&](auto& cp, int tok0, int blk0, uint32_t dst, int rowb) {
+    using CP = std::remove_reference_t<decltype(cp)>;
 #pragma unroll
-      for (int i = 0; i < kCopies; ++i) {
-        const bool valid = tok0 + r0 + i * kStep < tok_end;
-        const int blk = valid ? s_blk[blk0 + bsel0 + i * bstep] : 0;
-        const size_t off = (size_t)blk * blk_pitch + gbase;
-        const int sz = valid ? 16 : 0;
-        const uint32_t so = soff0 + (uint32_t)(i * kStep * kRowB);
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + so),
-                     "l"(reinterpret_cast<const uint8_t*>(p.k_cache) + off), "r"(sz) : "memory");
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + so),
-                     "l"(reinterpret_cast<const uint8_t*>(p.v_cache) + off), "r"(sz) : "memory");
-      }
-      return;
+    for (int i = 0; i < CP::kCopies; ++i) {
+      const bool valid = tok0 + cp.r0 + i * CP::kStep < tok_end;
+      const int blk = valid ? s_blk[blk0 + cp.bsel0 + i * cp.bstep] : 0;
+      const size_t off = (size_t)blk * cp.blk_pitch + cp.gbase;
+      const int sz = valid ? 16 : 0;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + cp.soff0 + (uint32_t)(i * CP::kStep * rowb)),
+                   "l"(cp.cache + off), "r"(sz) : "memory");
     }
+  };
+  auto issue_any = [&](auto& cp, int tok0, int blk0, uint32_t dst, auto rowb) {
+    using CP = std::remove_reference_t<decltype(cp)>;
+    constexpr int kRow = decltype(rowb)::value;
 #pragma unroll
-    for (int i = 0; i < kCopies; ++i) {
+    for (int i = 0; i < CP::kCopies; ++i) {
       const int idx = tid + i * 128;
-      const int r = idx / kChunks, c = idx % kChunks;          // compile-time divisors
+      const int r = idx / CP::kChunks, c = idx % CP::kChunks;  // compile-time divisors
       const int tok = tok0 + r;
       int sz = 0;
       size_t off = 0;
@@ -496,14 +531,20 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
           within = tok % bs;
           if (blk < 0 || blk >= p.num_blocks) blk = 0;
         }
-        off = ((size_t)blk * bs + within) * row_pitch + (size_t)kvh * kRowB + (size_t)c * 16;
+        off = ((size_t)blk * bs + within) * cp.row_pitch + (size_t)kvh * kRow + (size_t)c * 16;
         sz = 16;
       }
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + raw_off<kRowB>(r, c)),
-                   "l"(reinterpret_cast<const uint8_t*>(p.k_cache) + off), "r"(sz) : "memory");
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + raw_off<kRowB>(r, c)),
-                   "l"(reinterpret_cast<const uint8_t*>(p.v_cache) + off), "r"(sz) : "memory");
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + raw_off<kRow>(r, c)), "l"(cp.cache + off), "r"(sz) : "memory");
     }
+  };
+  auto issue_tile = [&](int it) {
+    const uint32_t sK = sbase + (it % kStages) * C::kStageB, sV = sK + kTileK;
+    const int tok0 = tok_begin + it * kTile;
+    const int blk0 = (tok0 - tok_begin) >> bs_shift;
+    if (ck.lin) issue_lin(ck, tok0, blk0, sK, kRowK);
+    else issue_any(ck, tok0, blk0, sK, std::integral_constant<int, kRowK>{});
+    if (cv.lin) issue_lin(cv, tok0, blk0, sV, kRowV);
+    else issue_any(cv, tok0, blk0, sV, std::integral_constant<int, kRowV>{});
   };
 
   // prologue: fill the pipeline, then load the Q fragments while the copies fly
@@ -513,7 +554,7 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
 
-  uint32_t qf[MT][D / 16][4];
+  uint32_t qf[MT][DK / 16][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
@@ -522,10 +563,10 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       const __nv_bfloat16* qrow = nullptr;
       if (r < R) {
         const int tq = r / G, hh = r - tq * G;
-        qrow = p.q + ((size_t)(qs + tq) * p.Hq + kvh * G + hh) * D;
+        qrow = p.q + ((size_t)(qs + tq) * p.Hq + kvh * G + hh) * DK;
       }
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         uint32_t lo = 0, hi = 0;
         if (qrow) {
           if constexpr (FP8) {
@@ -546,14 +587,14 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
   }
 
   // O accumulators: o_acc[mt][n][4]; for an e4m3 cache n = 2 * (16-dim group) + parity
-  float o_acc[MT][D / 8][4];
+  float o_acc[MT][DV / 8][4];
   float m_run[MT][2], l_run[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
     m_run[mt][0] = m_run[mt][1] = -INFINITY;
     l_run[mt][0] = l_run[mt][1] = 0.f;
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n)
+    for (int n = 0; n < DV / 8; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) o_acc[mt][n][i] = 0.f;
   }
@@ -580,7 +621,7 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
     if (it + kStages - 1 < ntiles) issue_tile(it + kStages - 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
     const int stage = it % kStages;
-    const uint32_t kT = sbase + stage * 2 * kTileB, vT = kT + kTileB;
+    const uint32_t kT = sbase + stage * C::kStageB, vT = kT + kTileK;
     const int tok0 = tok_begin + it * kTile + warp * 16;
     if (tok0 >= tok_end) continue;
     float s[MT][2][4];
@@ -592,11 +633,11 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
         for (int i = 0; i < 4; ++i) s[mt][n][i] = 0.f;
     if constexpr (FP8) {
 #pragma unroll
-      for (int kg = 0; kg < D / 32; ++kg) {              // 32 dims = 2 k steps per ldmatrix.x4
+      for (int kg = 0; kg < DK / 32; ++kg) {              // 32 dims = 2 k steps per ldmatrix.x4
         uint32_t r[4];
         // matrices: (tok 0-7, bytes lo) (tok 0-7, bytes hi) (tok 8-15, lo) (tok 8-15, hi)
         const int row = warp * 16 + (lane & 7) + ((lane >> 4) << 3);
-        ldsm4(r, kT + raw_off<kRowB>(row, kg * 2 + ((lane >> 3) & 1)));
+        ldsm4(r, kT + raw_off<kRowK>(row, kg * 2 + ((lane >> 3) & 1)));
 #pragma unroll
         for (int h = 0; h < 2; ++h) {                     // k step 2 kg + h
           const uint32_t b00 = e4m3_lo16(r[h]), b01 = e4m3_hi16(r[h]);
@@ -610,10 +651,10 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       }
     } else {
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         uint32_t b[4];
         const int row = warp * 16 + (lane & 7) + ((lane >> 4) << 3);
-        ldsm4(b, kT + raw_off<kRowB>(row, ks * 2 + ((lane >> 3) & 1)));
+        ldsm4(b, kT + raw_off<kRowK>(row, ks * 2 + ((lane >> 3) & 1)));
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma16816<false>(s[mt][0], qf[mt][ks], b[0], b[1]);
@@ -624,7 +665,7 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
     // online softmax over this warp's 16 tokens; the mask code only runs for tiles that
     // touch a causal limit, the end of the range or a sliding window
     const bool need_mask = (tok0 + 16 > min_limit) || (tok0 + 16 > tok_end) || (p.window > 0);
-    uint32_t pa[MT][4];
+    uint32_t pa[MT][4], pr[MT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
@@ -671,7 +712,7 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
         m_run[mt][hr] = m_new;
         if (alpha != 1.f) {
 #pragma unroll
-          for (int n = 0; n < D / 8; ++n) {
+          for (int n = 0; n < DV / 8; ++n) {
             o_acc[mt][n][hr * 2] *= alpha;
             o_acc[mt][n][hr * 2 + 1] *= alpha;
           }
@@ -681,15 +722,23 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       pa[mt][1] = pack2<F16>(s[mt][0][2], s[mt][0][3]);
       pa[mt][2] = pack2<F16>(s[mt][1][0], s[mt][1][1]);
       pa[mt][3] = pack2<F16>(s[mt][1][2], s[mt][1][3]);
+      if constexpr (!FP8) {
+        if (p.split_p) {
+          pr[mt][0] = pack_rest(s[mt][0][0], s[mt][0][1]);
+          pr[mt][1] = pack_rest(s[mt][0][2], s[mt][0][3]);
+          pr[mt][2] = pack_rest(s[mt][1][0], s[mt][1][1]);
+          pr[mt][3] = pack_rest(s[mt][1][2], s[mt][1][3]);
+        }
+      }
     }
     // O += P V
     if constexpr (FP8) {
 #pragma unroll
-      for (int d2 = 0; d2 < D / 32; ++d2) {               // two 16-dim groups per ldmatrix.x4.trans
+      for (int d2 = 0; d2 < DV / 32; ++d2) {               // two 16-dim groups per ldmatrix.x4.trans
         uint32_t r[4];
         // matrices: (tok 0-7, grp 2 d2) (tok 8-15, grp 2 d2) (tok 0-7, grp 2 d2 + 1) (tok 8-15, ...)
         const int row = warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-        ldsm4t(r, vT + raw_off<kRowB>(row, d2 * 2 + (lane >> 4)));
+        ldsm4t(r, vT + raw_off<kRowV>(row, d2 * 2 + (lane >> 4)));
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
           const int dg = d2 * 2 + h;
@@ -704,14 +753,18 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       }
     } else {
 #pragma unroll
-      for (int n2 = 0; n2 < D / 16; ++n2) {
+      for (int n2 = 0; n2 < DV / 16; ++n2) {
         uint32_t b[4];
         const int row = warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-        ldsm4t(b, vT + raw_off<kRowB>(row, n2 * 2 + (lane >> 4)));
+        ldsm4t(b, vT + raw_off<kRowV>(row, n2 * 2 + (lane >> 4)));
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma16816<false>(o_acc[mt][n2 * 2], pa[mt], b[0], b[1]);
           mma16816<false>(o_acc[mt][n2 * 2 + 1], pa[mt], b[2], b[3]);
+          if (p.split_p) {
+            mma16816<false>(o_acc[mt][n2 * 2], pr[mt], b[0], b[1]);
+            mma16816<false>(o_acc[mt][n2 * 2 + 1], pr[mt], b[2], b[3]);
+          }
         }
       }
     }
@@ -735,10 +788,10 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
         s_ml[(warp * MT * 16 + r) * 2] = m_run[mt][hr];
         s_ml[(warp * MT * 16 + r) * 2 + 1] = l;
       }
-      float* orow = s_o + ((size_t)(warp * MT * 16 + r)) * D;
+      float* orow = s_o + ((size_t)(warp * MT * 16 + r)) * DV;
       if constexpr (FP8) {
 #pragma unroll
-        for (int dg = 0; dg < D / 16; ++dg) {
+        for (int dg = 0; dg < DV / 16; ++dg) {
           // even tile cols (2t, 2t+1) -> dims 4t, 4t+2 ; odd tile -> dims 4t+1, 4t+3
           float4 v4;
           v4.x = o_acc[mt][dg * 2][hr * 2];
@@ -749,15 +802,15 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
         }
       } else {
 #pragma unroll
-        for (int n = 0; n < D / 8; ++n) {
+        for (int n = 0; n < DV / 8; ++n) {
           orow[n * 8 + t * 2] = o_acc[mt][n][hr * 2];
           orow[n * 8 + t * 2 + 1] = o_acc[mt][n][hr * 2 + 1];
         }
       }
     }
   __syncthreads();
-  for (int idx = tid; idx < R * (D / 4); idx += 128) {
-    const int r = idx / (D / 4), c4 = idx - r * (D / 4);
+  for (int idx = tid; idx < R * (DV / 4); idx += 128) {
+    const int r = idx / (DV / 4), c4 = idx - r * (DV / 4);
     float mw[4], lw[4];
     float mx = -INFINITY;
 #pragma unroll
@@ -766,13 +819,15 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       lw[w] = s_ml[(w * MT * 16 + r) * 2 + 1];
       mx = fmaxf(mx, mw[w]);
     }
-    float l = 0.f;
+    const bool sink_here = p.sink && nparts == 1;
+    if (sink_here) mx = fmaxf(mx, 0.f);
+    float l = sink_here ? exp2f(-mx) : 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float f = mw[w] == -INFINITY ? 0.f : exp2f(mw[w] - mx);
       l += lw[w] * f;
-      const float4 ov = *reinterpret_cast<const float4*>(s_o + ((size_t)(w * MT * 16 + r)) * D + c4 * 4);
+      const float4 ov = *reinterpret_cast<const float4*>(s_o + ((size_t)(w * MT * 16 + r)) * DV + c4 * 4);
       acc.x += ov.x * f; acc.y += ov.y * f; acc.z += ov.z * f; acc.w += ov.w * f;
     }
     const float inv = l > 0.f ? vmul / l : 0.f;
@@ -780,9 +835,9 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
     const int tq = r / G, hh = r - tq * G;
     const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
     if (nparts == 1) {
-      store_out4<D>(p, orow, c4, acc.x, acc.y, acc.z, acc.w);
+      store_out4<DV>(p, orow, c4, acc.x, acc.y, acc.z, acc.w);
     } else {
-      *reinterpret_cast<float4*>(p.part_o + (orow * p.parts + part) * D + c4 * 4) = acc;
+      *reinterpret_cast<float4*>(p.part_o + (orow * p.parts + part) * DV + c4 * 4) = acc;
       if (c4 == 0) {
         p.part_ml[(orow * p.parts + part) * 2] = mx;          // log2-domain max
         p.part_ml[(orow * p.parts + part) * 2 + 1] = l;
@@ -803,13 +858,14 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  for (int idx = tid; idx < R * (D / 4); idx += 128) {
-    const int r = idx / (D / 4), c4 = idx - r * (D / 4);
+  for (int idx = tid; idx < R * (DV / 4); idx += 128) {
+    const int r = idx / (DV / 4), c4 = idx - r * (DV / 4);
     const int tq = r / G, hh = r - tq * G;
     const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
     float mx = -INFINITY;
     for (int s2 = 0; s2 < nparts; ++s2) mx = fmaxf(mx, __ldcg(&p.part_ml[(orow * p.parts + s2) * 2]));
-    float denom = 0.f;
+    if (p.sink) mx = fmaxf(mx, 0.f);
+    float denom = p.sink ? exp2f(-mx) : 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s2 = 0; s2 < nparts; ++s2) {
       const float m = __ldcg(&p.part_ml[(orow * p.parts + s2) * 2]);
@@ -817,26 +873,26 @@ __global__ void __launch_bounds__(128, (D <= 128 && MT == 1) ? 4 : 1) attn_split
       if (m == -INFINITY || l <= 0.f) continue;
       const float wgt = l * exp2f(m - mx);
       denom += wgt;
-      const float4 ov = __ldcg(reinterpret_cast<const float4*>(p.part_o + (orow * p.parts + s2) * D + c4 * 4));
+      const float4 ov = __ldcg(reinterpret_cast<const float4*>(p.part_o + (orow * p.parts + s2) * DV + c4 * 4));
       acc.x += ov.x * wgt; acc.y += ov.y * wgt; acc.z += ov.z * wgt; acc.w += ov.w * wgt;
     }
     const float inv = denom > 0.f ? 1.f / denom : 0.f;
-    store_out4<D>(p, orow, c4, acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
+    store_out4<DV>(p, orow, c4, acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
   }
 }
 
 // ------------------------------------------------------------------ split-Q (prefill) kernel
 // grid (ceil(max_q_len / 64), Hq, num_seqs), 128 threads; warp w owns query rows 16w..16w+15.
-template <int D, bool FP8>
+template <int DK, int DV, bool FP8>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   constexpr bool F16 = FP8;
   constexpr int kTile = 64;
-  constexpr int kTileBytes = kTile * D * 2;
+  constexpr int kTileBytesK = kTile * DK * 2, kTileBytesV = kTile * DV * 2;
   extern __shared__ __align__(128) uint8_t smem_attn[];
   const uint32_t sbase = mb::smem_u32(smem_attn);
   const uint32_t sQ = sbase;
-  const uint32_t sK = sbase + kTileBytes;
-  const uint32_t sV = sK + 2 * kTileBytes;
+  const uint32_t sK = sbase + kTileBytesK;
+  const uint32_t sV = sK + 2 * kTileBytesK;
   const int qt = blockIdx.x, head = blockIdx.y, seq = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int G = p.Hq / p.Hkv, kvh = head / G;
@@ -852,11 +908,11 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   if (p.window > 0) tok_begin = max(0, past + q0 + 1 - p.window);
   tok_begin &= ~63;
 
-  for (int idx = tid; idx < 64 * (D / 8); idx += 128) {
-    const int r = idx / (D / 8), c = idx - r * (D / 8);
+  for (int idx = tid; idx < 64 * (DK / 8); idx += 128) {
+    const int r = idx / (DK / 8), c = idx - r * (DK / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
     if (q0 + r < qlen) {
-      v = *reinterpret_cast<const uint4*>(p.q + ((size_t)(qs + q0 + r) * p.Hq + head) * D + c * 8);
+      v = *reinterpret_cast<const uint4*>(p.q + ((size_t)(qs + q0 + r) * p.Hq + head) * DK + c * 8);
       if constexpr (F16) {
         const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&v);
         uint4 o;
@@ -869,35 +925,36 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
         v = o;
       }
     }
-    asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(sQ + tile_off<D>(r, c)), "r"(v.x),
+    asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(sQ + tile_off<DK>(r, c)), "r"(v.x),
                  "r"(v.y), "r"(v.z), "r"(v.w));
   }
 
-  float o_acc[D / 8][4];
+  float o_acc[DV / 8][4];
 #pragma unroll
-  for (int n = 0; n < D / 8; ++n)
+  for (int n = 0; n < DV / 8; ++n)
 #pragma unroll
     for (int i = 0; i < 4; ++i) o_acc[n][i] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const float kmul = FP8 ? (*p.k_scale) * 256.f : 1.f;
   const float sc_log2 = p.scale * kmul * 1.44269504088896f;
 
-  TileLoader<D, FP8> ldK, ldV;
+  TileLoader<DK, FP8> ldK;
+  TileLoader<DV, FP8> ldV;
   const int ntiles = (tok_end - tok_begin + kTile - 1) / kTile;
   ldK.fetch(p, p.k_cache, bt, kvh, tok_begin, tok_end, tid, sK);
   ldV.fetch(p, p.v_cache, bt, kvh, tok_begin, tok_end, tid, sV);
   for (int it = 0; it < ntiles; ++it) {
     const int buf = it & 1;
-    ldK.commit(sK + buf * kTileBytes, tid);
-    ldV.commit(sV + buf * kTileBytes, tid);
+    ldK.commit(sK + buf * kTileBytesK, tid);
+    ldV.commit(sV + buf * kTileBytesV, tid);
     __syncthreads();
     if (it + 1 < ntiles) {
       ldK.fetch(p, p.k_cache, bt, kvh, tok_begin + (it + 1) * kTile, tok_end, tid,
-                sK + (buf ^ 1) * kTileBytes);
+                sK + (buf ^ 1) * kTileBytesK);
       ldV.fetch(p, p.v_cache, bt, kvh, tok_begin + (it + 1) * kTile, tok_end, tid,
-                sV + (buf ^ 1) * kTileBytes);
+                sV + (buf ^ 1) * kTileBytesV);
     }
-    const uint32_t kT = sK + buf * kTileBytes, vT = sV + buf * kTileBytes;
+    const uint32_t kT = sK + buf * kTileBytesK, vT = sV + buf * kTileBytesV;
     const int tile_tok0 = tok_begin + it * kTile;
     // S[16 x 64] for this warp
     float s[8][4];
@@ -906,14 +963,14 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) s[n][i] = 0.f;
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks) {
+    for (int ks = 0; ks < DK / 16; ++ks) {
       uint32_t a[4];
-      ldsm4(a, sQ + tile_off<D>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+      ldsm4(a, sQ + tile_off<DK>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
 #pragma unroll
       for (int nb = 0; nb < 4; ++nb) {
         uint32_t b[4];
         const int row = nb * 16 + (lane & 7) + ((lane >> 4) << 3);
-        ldsm4(b, kT + tile_off<D>(row, ks * 2 + ((lane >> 3) & 1)));
+        ldsm4(b, kT + tile_off<DK>(row, ks * 2 + ((lane >> 3) & 1)));
         mma16816<F16>(s[nb * 2], a, b[0], b[1]);
         mma16816<F16>(s[nb * 2 + 1], a, b[2], b[3]);
       }
@@ -953,7 +1010,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
       m_run[hr] = m_new;
     }
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n) {
+    for (int n = 0; n < DV / 8; ++n) {
       o_acc[n][0] *= alpha[0]; o_acc[n][1] *= alpha[0];
       o_acc[n][2] *= alpha[1]; o_acc[n][3] *= alpha[1];
     }
@@ -964,13 +1021,28 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
       pa[1] = pack2<F16>(s[kb * 2][2], s[kb * 2][3]);
       pa[2] = pack2<F16>(s[kb * 2 + 1][0], s[kb * 2 + 1][1]);
       pa[3] = pack2<F16>(s[kb * 2 + 1][2], s[kb * 2 + 1][3]);
+      uint32_t pr[4];
+      if constexpr (!FP8) {
+        if (p.split_p) {
+          pr[0] = pack_rest(s[kb * 2][0], s[kb * 2][1]);
+          pr[1] = pack_rest(s[kb * 2][2], s[kb * 2][3]);
+          pr[2] = pack_rest(s[kb * 2 + 1][0], s[kb * 2 + 1][1]);
+          pr[3] = pack_rest(s[kb * 2 + 1][2], s[kb * 2 + 1][3]);
+        }
+      }
 #pragma unroll
-      for (int n2 = 0; n2 < D / 16; ++n2) {
+      for (int n2 = 0; n2 < DV / 16; ++n2) {
         uint32_t b[4];
         const int row = kb * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-        ldsm4t(b, vT + tile_off<D>(row, n2 * 2 + (lane >> 4)));
+        ldsm4t(b, vT + tile_off<DV>(row, n2 * 2 + (lane >> 4)));
         mma16816<F16>(o_acc[n2 * 2], pa, b[0], b[1]);
         mma16816<F16>(o_acc[n2 * 2 + 1], pa, b[2], b[3]);
+        if constexpr (!FP8) {
+          if (p.split_p) {
+            mma16816<false>(o_acc[n2 * 2], pr, b[0], b[1]);
+            mma16816<false>(o_acc[n2 * 2 + 1], pr, b[2], b[3]);
+          }
+        }
       }
     }
     __syncthreads();
@@ -983,19 +1055,29 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
     l += __shfl_xor_sync(0xffffffffu, l, 2);
     const int qr = q0 + warp * 16 + (lane >> 2) + hr * 8;
     if (qr >= qlen) continue;
-    const float inv = l > 0.f ? vmul / l : 0.f;
-    __nv_bfloat16* dst = p.out + ((size_t)(qs + qr) * p.Hq + head) * D + (lane & 3) * 2;
+    // the sink's share of the denominator, at this row's running maximum (every row has seen a key)
+    if (p.sink) l += exp2f(-m_run[hr]);
+    const float inv = (l > 0.f ? vmul / l : 0.f) * p.out_scale;
+    __nv_bfloat16* dst = p.out + (size_t)(qs + qr) * p.out_ld + (size_t)head * p.dv + (lane & 3) * 2;
+    if (p.dv == DV) {
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n)
-      *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) =
-          __floats2bfloat162_rn(o_acc[n][hr * 2] * inv, o_acc[n][hr * 2 + 1] * inv);
+      for (int n = 0; n < DV / 8; ++n)
+        *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) =
+            __floats2bfloat162_rn(o_acc[n][hr * 2] * inv, o_acc[n][hr * 2 + 1] * inv);
+    } else {
+#pragma unroll
+      for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          if (n * 8 + (lane & 3) * 2 + i < p.dv) dst[n * 8 + i] = __float2bfloat16(o_acc[n][hr * 2 + i] * inv);
+    }
   }
 }
 
-template <int D, bool FP8, int MT>
+template <int DK, int DV, bool FP8, int MT>
 int launch_splitkv(const AttnParams& p, int num_seqs, cudaStream_t stream) {
-  constexpr int smem = SplitKvCfg<D, FP8, MT>::kSmem;
-  auto kern = attn_splitkv_kernel<D, FP8, MT>;
+  constexpr int smem = SplitKvCfg<DK, DV, FP8, MT>::kSmem;
+  auto kern = attn_splitkv_kernel<DK, DV, FP8, MT>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -1004,10 +1086,10 @@ int launch_splitkv(const AttnParams& p, int num_seqs, cudaStream_t stream) {
   }
   return (int)mb::launch_kernel(kern, dim3(p.Hkv, num_seqs, p.parts), dim3(128), smem, stream, p);
 }
-template <int D, bool FP8>
+template <int DK, int DV, bool FP8>
 int launch_prefill(const AttnParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
-  constexpr int smem = 5 * 64 * D * 2;
-  auto kern = attn_prefill_kernel<D, FP8>;
+  constexpr int smem = (3 * DK + 2 * DV) * 64 * 2;
+  auto kern = attn_prefill_kernel<DK, DV, FP8>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -1017,12 +1099,12 @@ int launch_prefill(const AttnParams& p, int num_seqs, int max_q_len, cudaStream_
   return (int)mb::launch_kernel(kern, dim3((max_q_len + 63) / 64, p.Hq, num_seqs), dim3(128), smem, stream, p);
 }
 
-template <int D, bool FP8>
+template <int DK, int DV, bool FP8>
 int dispatch_mt(int mt, const AttnParams& p, int num_seqs, cudaStream_t stream) {
-  if (mt == 1) return launch_splitkv<D, FP8, 1>(p, num_seqs, stream);
+  if (mt == 1) return launch_splitkv<DK, DV, FP8, 1>(p, num_seqs, stream);
   // two m16 row tiles keep 2 * D / 2 accumulator registers per thread: fits up to D = 128
-  if constexpr (D <= 128) {
-    if (mt == 2) return launch_splitkv<D, FP8, 2>(p, num_seqs, stream);
+  if constexpr (DK <= 128 && DV <= 128) {
+    if (mt == 2) return launch_splitkv<DK, DV, FP8, 2>(p, num_seqs, stream);
   }
   return MB_ERR_UNSUPPORTED;
 }
@@ -1117,6 +1199,12 @@ struct MbAttnArgs {
   void* outq_sf;
   int outq_sf_k64;
   float outq_gs;
+  // separate value head size and softmax variants (all zero = values as wide as keys, plain softmax)
+  int DV;                  // padded value row of the cache (0 = D); bf16 caches
+  int dv;                  // value columns stored per head (0 = DV)
+  long long out_ld;        // elements between output rows (0 = Hq * dv)
+  float out_scale;         // 0 = 1
+  int sink, split_p;
 };
 
 // workspace bytes for the split-KV path
@@ -1140,6 +1228,14 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
   p.scale = a->scale; p.k_scale = a->k_scale; p.v_scale = a->v_scale;
   p.out = reinterpret_cast<__nv_bfloat16*>(a->out);
   p.window = a->window; p.status = a->status;
+  const int DV = a->DV > 0 ? a->DV : a->D;
+  p.dv = a->dv > 0 ? a->dv : DV;
+  p.out_ld = a->out_ld > 0 ? a->out_ld : (long long)a->Hq * p.dv;
+  p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.f;
+  p.sink = a->sink; p.split_p = a->split_p;
+  if (p.dv > DV || p.out_ld < (long long)a->Hq * p.dv) return MB_ERR_BAD_ARG;
+  if (p.dv == DV && (p.out_ld % 2 || (reinterpret_cast<uintptr_t>(a->out) & 3))) return MB_ERR_BAD_ARG;   // paired stores
+  if ((DV != a->D || p.sink || p.split_p || p.dv != DV) && (a->cache_fp8 || a->outq || a->window)) return MB_ERR_UNSUPPORTED;
   const int G = a->Hq / a->Hkv;
   const int rows = G * a->max_q_len;
   int mode = a->force_mode;
@@ -1160,31 +1256,35 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
     if (p.parts < 1) p.parts = 1;
     if (p.parts > 1) {
       const size_t cnt_bytes = ((size_t)a->num_seqs * a->Hkv * sizeof(uint32_t) + 255) & ~size_t(255);
-      const size_t need = cnt_bytes + (size_t)a->total_rows * a->Hq * p.parts * (a->D + 2) * sizeof(float);
+      const size_t need = cnt_bytes + (size_t)a->total_rows * a->Hq * p.parts * (DV + 2) * sizeof(float);
       if (!a->ws || a->ws_bytes < need || cnt_bytes > kAttnCntBytes) return MB_ERR_TOO_LARGE;
       // counters sit in the first kAttnCntBytes of the workspace (zero-initialised by the
       // owner once; every launch leaves them at zero again)
       p.part_cnt = reinterpret_cast<uint32_t*>(a->ws);
       p.part_o = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(a->ws) + kAttnCntBytes);
-      p.part_ml = p.part_o + (size_t)a->total_rows * a->Hq * p.parts * a->D;
+      p.part_ml = p.part_o + (size_t)a->total_rows * a->Hq * p.parts * DV;
     }
     int rc;
-    if (a->D == 128) rc = fp8 ? dispatch_mt<128, true>(mt, p, a->num_seqs, stream)
-                              : dispatch_mt<128, false>(mt, p, a->num_seqs, stream);
-    else if (a->D == 64) rc = fp8 ? dispatch_mt<64, true>(mt, p, a->num_seqs, stream)
-                                  : dispatch_mt<64, false>(mt, p, a->num_seqs, stream);
-    else if (a->D == 256) rc = fp8 ? dispatch_mt<256, true>(mt, p, a->num_seqs, stream)
-                                   : dispatch_mt<256, false>(mt, p, a->num_seqs, stream);
+    if (a->D == 128 && DV == 128) rc = fp8 ? dispatch_mt<128, 128, true>(mt, p, a->num_seqs, stream)
+                                           : dispatch_mt<128, 128, false>(mt, p, a->num_seqs, stream);
+    else if (a->D == 64 && DV == 64) rc = fp8 ? dispatch_mt<64, 64, true>(mt, p, a->num_seqs, stream)
+                                              : dispatch_mt<64, 64, false>(mt, p, a->num_seqs, stream);
+    else if (a->D == 256 && DV == 256) rc = fp8 ? dispatch_mt<256, 256, true>(mt, p, a->num_seqs, stream)
+                                                : dispatch_mt<256, 256, false>(mt, p, a->num_seqs, stream);
+    else if (a->D == 64 && DV == 128) rc = dispatch_mt<64, 128, false>(mt, p, a->num_seqs, stream);
+    else if (a->D == 128 && DV == 64) rc = dispatch_mt<128, 64, false>(mt, p, a->num_seqs, stream);
     else return MB_ERR_UNSUPPORTED;
     return rc;                    // partitions are merged inside the kernel by the last arriver
   }
   p.parts = 1;
-  if (a->D == 128) return fp8 ? launch_prefill<128, true>(p, a->num_seqs, a->max_q_len, stream)
-                              : launch_prefill<128, false>(p, a->num_seqs, a->max_q_len, stream);
-  if (a->D == 64) return fp8 ? launch_prefill<64, true>(p, a->num_seqs, a->max_q_len, stream)
-                             : launch_prefill<64, false>(p, a->num_seqs, a->max_q_len, stream);
-  if (a->D == 256) return fp8 ? launch_prefill<256, true>(p, a->num_seqs, a->max_q_len, stream)
-                              : launch_prefill<256, false>(p, a->num_seqs, a->max_q_len, stream);
+  if (a->D == 128 && DV == 128) return fp8 ? launch_prefill<128, 128, true>(p, a->num_seqs, a->max_q_len, stream)
+                                           : launch_prefill<128, 128, false>(p, a->num_seqs, a->max_q_len, stream);
+  if (a->D == 64 && DV == 64) return fp8 ? launch_prefill<64, 64, true>(p, a->num_seqs, a->max_q_len, stream)
+                                         : launch_prefill<64, 64, false>(p, a->num_seqs, a->max_q_len, stream);
+  if (a->D == 256 && DV == 256) return fp8 ? launch_prefill<256, 256, true>(p, a->num_seqs, a->max_q_len, stream)
+                                           : launch_prefill<256, 256, false>(p, a->num_seqs, a->max_q_len, stream);
+  if (a->D == 64 && DV == 128) return launch_prefill<64, 128, false>(p, a->num_seqs, a->max_q_len, stream);
+  if (a->D == 128 && DV == 64) return launch_prefill<128, 64, false>(p, a->num_seqs, a->max_q_len, stream);
   return MB_ERR_UNSUPPORTED;
 }
 

@@ -20,6 +20,10 @@
 // softmax overlap the other's tensor work. Every wait on an mbarrier is bounded and reports
 // through the status word; TMEM is freed on every path.
 //
+// Softmax variants: a sink (one added to the denominator), and SPLIT, in which the weights enter the
+// product with V as two bf16 terms (hi + rest: 16 mantissa bits), for models whose attention weights are
+// 32-bit quantities; the output may be a column range of a wider matrix and takes a constant factor.
+//
 // Serves q_len >= 128 chunks with head_dim 128, bf16 or e4m3 caches, no sliding window; other
 // shapes stay on the mma.sync kernels in attention.cu, which are also the oracle in the tests.
 // Reference behaviour covered: the prefill paged-attention family
@@ -46,7 +50,10 @@ struct TcParams {
   float scale;
   const float* k_scale;
   const float* v_scale;
-  __nv_bfloat16* out;            // [rows, Hq, D]
+  __nv_bfloat16* out;            // [rows, out_ld]: head h at columns h * D
+  long long out_ld;
+  float out_scale;
+  int sink;
   uint32_t* status;
 };
 
@@ -80,7 +87,7 @@ __device__ __forceinline__ uint4 widen8(uint2 v) {
 
 // kD = head dim (128 or 256; 256 needs the MN-major V path). kNH = 64-dim blocks per row; a staging
 // thread owns one token and the blocks sub, sub + 2, ... (sub = tid / 64).
-template <int kD, bool FP8, bool VMN>
+template <int kD, bool FP8, bool VMN, bool SPLIT>
 __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel(const TcParams p) {
   static_assert(kD == 128 || (kD == 256 && VMN), "head dim 256 stages V as stored");
   constexpr int kNH = kD / 64, kNHT = kNH / 2;
@@ -91,6 +98,7 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   uint8_t* sK = sQ + kNH * kQ * 128;        // kNH blocks x [64 rows x 128 B]
   uint8_t* sV = sK + kNH * kT * 128;        // as stored: kNH blocks x [64 tokens x 128 B]; transposed: [kD dims x 128 B]
   uint8_t* sP = sV + kD * 128;              // [128 rows x 128 B (64 tokens)]
+  uint8_t* sR = sP + kQ * 128;              // SPLIT: what bf16 rounding took off P
   __shared__ uint64_t bar_s, bar_o;
   __shared__ uint32_t s_tmem;
   const int qt = blockIdx.x, head = blockIdx.y, seq = blockIdx.z;
@@ -127,7 +135,7 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   const uint32_t t_row = tmem + ((uint32_t)(warp * 32) << 16);   // this warp's 32 TMEM lanes
   constexpr uint32_t kIdescS = mb::umma_idesc(1, 1, kQ, kT);
   constexpr uint32_t kIdescO = mb::umma_idesc(1, 1, kQ, kD, 0, VMN ? 1 : 0);
-  const uint32_t aQ = mb::smem_u32(sQ), aK = mb::smem_u32(sK), aV = mb::smem_u32(sV), aP = mb::smem_u32(sP);
+  const uint32_t aQ = mb::smem_u32(sQ), aK = mb::smem_u32(sK), aV = mb::smem_u32(sV), aP = mb::smem_u32(sP), aR = mb::smem_u32(sR);
 
   const int qi = q0 + tid;
   const bool row_ok = qi < qlen;
@@ -275,16 +283,23 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
       float rs = 0.f;
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
-        uint4 pk;
+        uint4 pk, rk;
         uint32_t* pw = reinterpret_cast<uint32_t*>(&pk);
+        uint32_t* rw = reinterpret_cast<uint32_t*>(&rk);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float a = ex2(sv[c * 8 + 2 * i] - m_use), b = ex2(sv[c * 8 + 2 * i + 1] - m_use);
           const __nv_bfloat162 pb = __floats2bfloat162_rn(a, b);
           rs += a + b;
           pw[i] = *reinterpret_cast<const uint32_t*>(&pb);
+          if constexpr (SPLIT) {
+            const float2 f = __bfloat1622float2(pb);
+            const __nv_bfloat162 rb = __floats2bfloat162_rn(a - f.x, b - f.y);
+            rw[i] = *reinterpret_cast<const uint32_t*>(&rb);
+          }
         }
         *reinterpret_cast<uint4*>(sP + sw_off(tid, c)) = pk;
+        if constexpr (SPLIT) *reinterpret_cast<uint4*>(sR + sw_off(tid, c)) = rk;
       }
       l_run = l_run * alpha + rs;
     }
@@ -297,11 +312,12 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
     if (tid == 0) {
       mb::tc_fence_after();
 #pragma unroll
-      for (int s = 0; s < 4; ++s)
-        mb::umma_f16(tmem + 64, mb::umma_desc_sw128(aP + s * 32),
-                     VMN ? mb::umma_desc_sw128_mn(aV + s * 2048, kT * 128, 1024)   // 16 tokens = two 8-row groups on
-                         : mb::umma_desc_sw128(aV + s * 32),
-                     kIdescO, (j | s) != 0);
+      for (int s = 0; s < 4; ++s) {
+        const uint64_t dv = VMN ? mb::umma_desc_sw128_mn(aV + s * 2048, kT * 128, 1024)   // 16 tokens = two 8-row groups on
+                                : mb::umma_desc_sw128(aV + s * 32);
+        mb::umma_f16(tmem + 64, mb::umma_desc_sw128(aP + s * 32), dv, kIdescO, (j | s) != 0);
+        if constexpr (SPLIT) mb::umma_f16(tmem + 64, mb::umma_desc_sw128(aR + s * 32), dv, kIdescO, 1);
+      }
       mb::tc_commit(&bar_o);
     }
   }
@@ -311,8 +327,9 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   }
   if (ok) {                                               // uniform: tcgen05.ld is a whole-warp instruction
     const float vmul = FP8 ? (*p.v_scale) * 256.f : 1.f;
-    const float inv = l_run > 0.f ? vmul / l_run : 0.f;
-    uint4* dst = reinterpret_cast<uint4*>(p.out + ((size_t)(qs + (row_ok ? qi : 0)) * p.Hq + head) * kD);
+    if (p.sink) l_run += ex2(-m_run);                     // the sink's weight at this row's running maximum
+    const float inv = (l_run > 0.f ? vmul / l_run : 0.f) * p.out_scale;
+    uint4* dst = reinterpret_cast<uint4*>(p.out + (size_t)(qs + (row_ok ? qi : 0)) * p.out_ld + (size_t)head * kD);
 #pragma unroll
     for (int c = 0; c < kD / 16; ++c) {
       float ov[16];
@@ -330,6 +347,18 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   mb::tc_fence_before();
   __syncthreads();
   if (warp == 0) mb::tmem_dealloc(tmem, kTmemCols);
+}
+
+template <int kD, bool FP8, bool VMN, bool SPLIT>
+int launch_tc(const TcParams& p, dim3 grid, size_t smem, cudaStream_t stream) {
+  auto kern = attn_prefill_tc_kernel<kD, FP8, VMN, SPLIT>;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  return (int)mb::launch_kernel(kern, grid, dim3(128), smem, stream, p);
 }
 
 }  // namespace
@@ -350,6 +379,9 @@ struct MbAttnTcArgs {
   int max_blocks, num_seqs, max_q_len, Hq, Hkv, D, block_size, cache_fp8;
   float scale;
   int v_mn;      // 1: V staged as stored and read as an MN-major operand (no transposition)
+  long long out_ld;    // elements between output rows (0 = Hq * D)
+  float out_scale;     // 0 = 1
+  int sink, split_p;
 };
 
 // Causal paged attention for prefill chunks (head dim 128). Returns 0, MB_ERR_* or a CUDA error.
@@ -364,28 +396,22 @@ extern "C" int mb_attn_prefill_tc(const MbAttnTcArgs* a, cudaStream_t stream) {
   p.Hq = a->Hq; p.Hkv = a->Hkv; p.block_size = a->block_size; p.num_blocks = a->num_blocks;
   p.scale = a->scale; p.k_scale = a->k_scale; p.v_scale = a->v_scale;
   p.out = (__nv_bfloat16*)a->out; p.status = a->status;
-  const size_t smem = (size_t)(a->D / 64) * (kQ + 2 * kT) * 128 + kQ * 128 + 1024;
-  static bool configured = false;
-  if (!configured) {
-    const int s128 = 2 * (kQ + 2 * kT) * 128 + kQ * 128 + 1024, s256 = 4 * (kQ + 2 * kT) * 128 + kQ * 128 + 1024;
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, s128);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, s128);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, s128);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, s128);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<256, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, s256);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<256, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, s256);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
-  }
+  p.out_ld = a->out_ld > 0 ? a->out_ld : (long long)a->Hq * a->D;
+  p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.f;
+  p.sink = a->sink;
+  if (p.out_ld % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15)) return MB_ERR_BAD_ARG;      // 16-byte stores
+  if (a->split_p && a->cache_fp8) return MB_ERR_UNSUPPORTED;
+  const size_t smem = (size_t)(a->D / 64) * (kQ + 2 * kT) * 128 + (a->split_p ? 2 : 1) * kQ * 128 + 1024;
   const dim3 grid((a->max_q_len + kQ - 1) / kQ, a->Hq, a->num_seqs);
   if (a->D == 256) {
-    if (a->cache_fp8) return (int)mb::launch_kernel(attn_prefill_tc_kernel<256, true, true>, grid, dim3(128), smem, stream, p);
-    return (int)mb::launch_kernel(attn_prefill_tc_kernel<256, false, true>, grid, dim3(128), smem, stream, p);
+    if (a->cache_fp8) return launch_tc<256, true, true, false>(p, grid, smem, stream);
+    return a->split_p ? launch_tc<256, false, true, true>(p, grid, smem, stream) : launch_tc<256, false, true, false>(p, grid, smem, stream);
   }
   if (a->v_mn) {
-    if (a->cache_fp8) return (int)mb::launch_kernel(attn_prefill_tc_kernel<128, true, true>, grid, dim3(128), smem, stream, p);
-    return (int)mb::launch_kernel(attn_prefill_tc_kernel<128, false, true>, grid, dim3(128), smem, stream, p);
+    if (a->cache_fp8) return launch_tc<128, true, true, false>(p, grid, smem, stream);
+    return a->split_p ? launch_tc<128, false, true, true>(p, grid, smem, stream) : launch_tc<128, false, true, false>(p, grid, smem, stream);
   }
-  if (a->cache_fp8) return (int)mb::launch_kernel(attn_prefill_tc_kernel<128, true, false>, grid, dim3(128), smem, stream, p);
-  return (int)mb::launch_kernel(attn_prefill_tc_kernel<128, false, false>, grid, dim3(128), smem, stream, p);
+  if (a->split_p) return MB_ERR_UNSUPPORTED;
+  if (a->cache_fp8) return launch_tc<128, true, false, false>(p, grid, smem, stream);
+  return launch_tc<128, false, false, false>(p, grid, smem, stream);
 }

@@ -1,0 +1,18 @@
+// GEMM epilogue numbering and the elementwise functions the two GEMM families share.
+#pragma once
+#include "common.cuh"
+
+namespace mb {
+
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_NEG_EXP = 4 };
+
+__device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+
+// g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(alpha g) (u + 1)
+__device__ __forceinline__ float clamp_glu(float gate, float up, float alpha, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g * sigmoid_exact(alpha * g) * (u + 1.f);
+}
+
+}  // namespace mb

@@ -44,6 +44,9 @@ struct MbGemmArgs {
   const int* tile_row0;
   const int* tile_nrows;
   int n_per_expert, max_tiles;
+  // epilogue parameters: 2 = clamped GLU (epi_a sigmoid slope, epi_b limit), 3 = SiLU on columns below epi_n
+  float epi_a, epi_b;
+  int epi_n;
 };
 
 extern "C" int mb_gemm(const MbGemmArgs* args, cudaStream_t stream);

@@ -33,6 +33,7 @@
 // w8a16_gemm*,w8a8_gemv,fp8_gemm_t_blockscaled}.cu and the W4A4 path of
 // kernels/gb10/qwen3.6-27b/nvfp4/nvfp4_mmq.cu (compiled out for sm_100a there).
 #include "common.cuh"
+#include "epilogue.cuh"
 #include "gemm_args.h"
 #include <mutex>
 #include "tensormap.h"
@@ -41,7 +42,10 @@
 namespace {
 
 enum { KIND_BF16 = 0, KIND_FP8 = 1, KIND_NVFP4 = 2, KIND_FP8_BLOCK = 3 };
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1 };
+using mb::EPI_CLAMP_GLU;
+using mb::EPI_PLAIN;
+using mb::EPI_SILU_COLS;
+using mb::EPI_SWIGLU;
 
 struct GemmParams {
   int M, N, K, ldo;
@@ -58,6 +62,8 @@ struct GemmParams {
   uint32_t* cnt;
   int splits, kb_per_split, num_kb;
   int epilogue, out_f32;
+  float epi_a, epi_b;     // EPI_CLAMP_GLU: sigmoid slope and clamp limit
+  int epi_n;              // EPI_SILU_COLS: SiLU on output columns below this
   uint32_t* status;
   // grouped (MoE) mode: blockIdx.y indexes a tile work-list; W is [experts * n_per_expert, K]
   const int* tile_expert;
@@ -309,7 +315,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
     float* s_tile = reinterpret_cast<float*>(smem);
     bool ok = true;
-    const bool swiglu = p.epilogue == EPI_SWIGLU;
+    const bool swiglu = p.epilogue == EPI_SWIGLU || p.epilogue == EPI_CLAMP_GLU;   // paired (gate, up) columns
+    const bool clamp_glu = p.epilogue == EPI_CLAMP_GLU;
     mb::pdl_wait();                                        // first global access of these warps follows
     // per-token scales of this tile, staged while the main loop runs
     for (int j = et; j < TN; j += 128) {
@@ -435,12 +442,21 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         const int m = m0 + mr;
         const float as = s_ascale[mr];
         float y[8];
-        if (swiglu) {
+        if (clamp_glu) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            y[i] = mb::clamp_glu(x[2 * i] * wcol[2 * i] * as, x[2 * i + 1] * wcol[2 * i + 1] * as, p.epi_a, p.epi_b);
+        } else if (swiglu) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = mb::silu(x[2 * i] * wcol[2 * i] * as) * (x[2 * i + 1] * wcol[2 * i + 1] * as);
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = x[i] * wcol[i] * as;
+          if (p.epilogue == EPI_SILU_COLS) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              if (n_out0 + i < p.epi_n) y[i] = mb::silu(y[i]);
+          }
         }
         const size_t o = (size_t)m * p.ldo + n_out0;
         if (vec_ok) {
@@ -771,7 +787,8 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
     const int lane = threadIdx.x & 31;
     const int et = threadIdx.x - 64;
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
-    const bool swiglu = p.epilogue == EPI_SWIGLU;
+    const bool swiglu = p.epilogue == EPI_SWIGLU || p.epilogue == EPI_CLAMP_GLU;   // paired (gate, up) columns
+    const bool clamp_glu = p.epilogue == EPI_CLAMP_GLU;
     mb::pdl_wait();
     const int f = q * 32 + lane;                          // weight row of this thread inside a tile
     const float outq_inv6gs = p.outq ? 1.f / (6.f * p.outq_gs) : 0.f;
@@ -820,7 +837,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             const float x0 = v[j] * (wsc * as.x), x1 = v[j + 1] * (wsc * as.y);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
             const float gate = odd ? other : x0, up = odd ? x1 : other;
-            const float y = mb::silu(gate) * up;
+            const float y = clamp_glu ? mb::clamp_glu(gate, up, p.epi_a, p.epi_b) : mb::silu(gate) * up;
             const int ml = m0 + (odd ? 1 : 0);                 // row inside the tile
             const int m = m_base + ml;
             if (p.outq) {
@@ -856,6 +873,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             const int ml = c * 16 + j;
             if (ml < m_valid && n < p.N) {
               float y = v[j] * wsc * asc[ml];
+              if (p.epilogue == EPI_SILU_COLS && n < p.epi_n) y = mb::silu(y);
               const size_t o = (size_t)(m_base + ml) * p.ldo + n;
               if (p.residual) y += __bfloat162float(p.residual[o]);
               if (p.out_f32) reinterpret_cast<float*>(p.out)[o] = y;
@@ -960,7 +978,8 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   if (row_bytes % 16) return MB_ERR_BAD_ARG;           // TMA global stride rule
   if (kind == KIND_NVFP4 && (!a->sfa || !a->sfb)) return MB_ERR_BAD_ARG;
   if (kind == KIND_FP8_BLOCK && (!a->w_scale || !a->a_scale)) return MB_ERR_BAD_ARG;
-  if (a->epilogue == EPI_SWIGLU && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
+  if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
+  if (a->epilogue == EPI_SILU_COLS && a->residual) return MB_ERR_BAD_ARG;
   const int num_kb = (a->K + kelems - 1) / kelems;
   if (kind == KIND_NVFP4 && a->sf_k64 < num_kb * 4) return MB_ERR_BAD_ARG;
 
@@ -1018,6 +1037,7 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   p.sf_k64 = a->sf_k64;
   p.splits = splits; p.kb_per_split = kb_per; p.num_kb = num_kb;
   p.epilogue = a->epilogue; p.out_f32 = a->out_f32;
+  p.epi_a = a->epi_a; p.epi_b = a->epi_b; p.epi_n = a->epi_n;
   p.status = a->status;
 #ifdef MB_GEMM_TIMING_EXPERIMENTS
   p.dbg = a->flags & 47;

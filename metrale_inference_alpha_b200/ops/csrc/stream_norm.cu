@@ -1,0 +1,522 @@
+// Row kernels of models with a 32-bit residual stream and Dynamic-Tanh norms.
+//
+//   stream_norm   one pass over the stream between two sublayers: the previous sublayer's output y joins
+//                 the fp32 stream x through its post-norm (Dynamic Tanh, or RMS with a plain weight), and
+//                 the next sublayer's input is produced from the new value (Dynamic Tanh, or the value as
+//                 it is). Dynamic Tanh needs no statistics, so both norms and the add are one elementwise
+//                 pass; only the RMS add reduces a row. With `mu` set the consumer is a token-shift mixer:
+//                 five mixes h + (h_prev - h) mu_s are written next to h, where h_prev is the previous
+//                 token's h: recomputed from the previous row (elementwise), or read from the sequence's
+//                 carried state on the first row of its portion (zero at position 0). The CTA of a
+//                 sequence's first row also advances that state to its last row's h: it is the only
+//                 reader of the old value, so no other CTA can see a half-updated state.
+//   shift_commit  state := h of the last accepted row (write-on-accept after speculative verification)
+//   gated_norm    RMS over groups of channels x weight x act(gate) x scale, act = SiLU or sigmoid; the
+//                 output may be a column range of a wider matrix
+//   side_gate     gelu_tanh(z) * e, e gathered from a per-layer slice of a second embedding table
+//   embed_scaled  fp32 embedding rows times a constant
+//   rope_dims     rotate-half positions on q and k with separate query/key and value head sizes, scattered
+//                 into a paged cache whose rows are padded (with zeros) to the attention kernel's tile
+// T is the activation type: bf16, or fp32 for models served in 32-bit.
+#include "common.cuh"
+#include "epilogue.cuh"
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+
+template <typename T>
+__device__ __forceinline__ float ldv(const T* p) {
+  if constexpr (sizeof(T) == 2) return __bfloat162float(*p);
+  else return *p;
+}
+template <typename T>
+__device__ __forceinline__ void stv(T* p, float v) {
+  if constexpr (sizeof(T) == 2) *p = __float2bfloat16(v);
+  else *p = v;
+}
+// VEC consecutive elements <-> floats (VEC is 1 or 4; 4 needs the natural vector alignment)
+template <int VEC, typename T>
+__device__ __forceinline__ void ldn(const T* p, float* o) {
+  if constexpr (VEC == 1) {
+    o[0] = ldv(p);
+  } else if constexpr (sizeof(T) == 2) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+  } else {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+  }
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void stn(T* p, const float* o) {
+  if constexpr (VEC == 1) {
+    stv(p, o[0]);
+  } else if constexpr (sizeof(T) == 2) {
+    uint2 v;
+    *reinterpret_cast<__nv_bfloat162*>(&v.x) = __floats2bfloat162_rn(o[0], o[1]);
+    *reinterpret_cast<__nv_bfloat162*>(&v.y) = __floats2bfloat162_rn(o[2], o[3]);
+    *reinterpret_cast<uint2*>(p) = v;
+  } else {
+    *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]);
+  }
+}
+
+struct DytW {
+  float alpha;
+  const bf16* w;
+  const bf16* b;
+};
+
+enum { ADD_NONE = 0, ADD_DYT = 1, ADD_RMS = 2 };
+enum { OUT_NONE = 0, OUT_DYT = 1, OUT_RAW = 2 };
+
+struct StreamParams {
+  int T, W;
+  const float* x;
+  const void* y;
+  int add_mode, out_mode;
+  DytW post, pre;            // ADD_RMS uses post.w and eps
+  float eps;
+  float* x_out;
+  void* out;                 // [T, W]
+  float* h32;                // optional fp32 copy of the produced rows
+  const bf16* mu;            // [5, W] or null
+  void* mixes;               // [5, T, W]
+  float* state;              // [slots, W]
+  const int* q_start;
+  const int* q_len;
+  const int* positions;
+  const int* slots;
+  int num_seqs, num_slots, write_state;
+  uint32_t* status;
+};
+
+template <int VEC, typename T>
+__global__ void __launch_bounds__(256) stream_norm_kernel(const StreamParams p) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, W = p.W;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const T* y = reinterpret_cast<const T*>(p.y);
+  auto row_inv = [&](int row) -> float {
+    if (p.add_mode != ADD_RMS) return 1.f;
+    float ss = 0.f;
+    for (int k = tid * VEC; k < W; k += nt * VEC) {
+      float v[VEC];
+      ldn<VEC>(y + (size_t)row * W + k, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+    }
+    return rsqrtf(mb::block_sum(ss, red) / (float)W + p.eps);
+  };
+  // the stream after the pending add, elements k .. k + VEC - 1 of `row`
+  auto value = [&](int row, int k, float inv, float* o) {
+    ldn<VEC>(p.x + (size_t)row * W + k, o);
+    if (p.add_mode == ADD_NONE) return;
+    float v[VEC], w[VEC], b[VEC];
+    ldn<VEC>(y + (size_t)row * W + k, v);
+    ldn<VEC>(p.post.w + k, w);
+    if (p.add_mode == ADD_DYT) {
+      ldn<VEC>(p.post.b + k, b);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] += fmaf(tanhf(p.post.alpha * v[i]), w[i], b[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] += v[i] * inv * w[i];
+    }
+  };
+  auto normed = [&](int k, const float* x, float* o) {
+    if (p.out_mode == OUT_RAW) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] = x[i];
+      return;
+    }
+    float w[VEC], b[VEC];
+    ldn<VEC>(p.pre.w + k, w);
+    ldn<VEC>(p.pre.b + k, b);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) o[i] = fmaf(tanhf(p.pre.alpha * x[i]), w[i], b[i]);
+  };
+
+  // token shift: which sequence this row belongs to, and where its previous token's h comes from
+  int prev = -1, last = -1;          // rows; prev = -1: from the state, or zero
+  const float* st = nullptr;
+  float* st_out = nullptr;
+  if (p.mu) {
+    int lo = 0, hi = p.num_seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.q_start[mid] <= t) lo = mid;
+      else hi = mid - 1;
+    }
+    const int r0 = p.q_start[lo], n = p.q_len[lo];
+    if (t < r0 || t >= r0 + n) return;
+    if (t > r0) {
+      prev = t - 1;
+    } else {
+      const int slot = p.slots[lo];
+      if (slot < 0 || slot >= p.num_slots) {
+        if (p.status && tid == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+      } else {
+        if (p.positions[t] != 0) st = p.state + (size_t)slot * W;
+        if (p.write_state) { st_out = p.state + (size_t)slot * W; last = r0 + n - 1; }
+      }
+    }
+  }
+  const float inv = row_inv(t);
+  const float inv_prev = prev >= 0 ? row_inv(prev) : 1.f;
+  const float inv_last = (st_out && last != t) ? row_inv(last) : inv;
+  for (int k = tid * VEC; k < W; k += nt * VEC) {
+    float x[VEC], h[VEC];
+    value(t, k, inv, x);
+    if (p.x_out) stn<VEC>(p.x_out + (size_t)t * W + k, x);
+    if (p.out_mode == OUT_NONE) continue;
+    normed(k, x, h);
+    if (p.out) stn<VEC>(reinterpret_cast<T*>(p.out) + (size_t)t * W + k, h);
+    if (p.h32) stn<VEC>(p.h32 + (size_t)t * W + k, h);
+    if (!p.mu) continue;
+    float hp[VEC];
+    if (prev >= 0) {
+      float xp[VEC];
+      value(prev, k, inv_prev, xp);
+      normed(k, xp, hp);
+    } else if (st) {
+      ldn<VEC>(st + k, hp);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) hp[i] = 0.f;
+    }
+#pragma unroll
+    for (int s = 0; s < 5; ++s) {
+      float m[VEC], o[VEC];
+      ldn<VEC>(p.mu + (size_t)s * W + k, m);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] = fmaf(hp[i] - h[i], m[i], h[i]);
+      stn<VEC>(reinterpret_cast<T*>(p.mixes) + ((size_t)s * p.T + t) * W + k, o);
+    }
+    if (st_out) {
+      if (last != t) {
+        float xl[VEC], hl[VEC];
+        value(last, k, inv_last, xl);
+        normed(k, xl, hl);
+        stn<VEC>(st_out + k, hl);
+      } else {
+        stn<VEC>(st_out + k, h);
+      }
+    }
+  }
+}
+
+__global__ void __launch_bounds__(256) shift_commit_kernel(const float* h32, int W, float* state, const int* q_start, const int* q_len,
+                                                           const int* slots, int num_slots, uint32_t* status) {
+  const int s = blockIdx.x, n = q_len[s];
+  if (n <= 0) return;
+  const int slot = slots[s];
+  if (slot < 0 || slot >= num_slots) {
+    if (status && threadIdx.x == 0) atomicCAS(status, 0u, MB_ST_BOUNDS);
+    return;
+  }
+  const float* src = h32 + (size_t)(q_start[s] + n - 1) * W;
+  for (int k = threadIdx.x; k < W; k += blockDim.x) state[(size_t)slot * W + k] = src[k];
+}
+
+// ------------------------------------------------------------------ gated group RMS
+struct GatedParams {
+  int T, K, group;
+  const float* x;
+  const bf16* w;
+  const void* gate;
+  long long gate_ld;
+  int sigmoid_gate;        // 0: SiLU
+  float eps, scale;
+  void* out;
+  long long out_ld;
+};
+
+template <int VEC, typename T>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedParams p) {
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const float* x = p.x + (size_t)t * p.K;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + (size_t)t * p.gate_ld;
+  T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.out_ld;
+  auto emit = [&](int k, float inv) {
+    float v[VEC], w[VEC], g[VEC], o[VEC];
+    ldn<VEC>(x + k, v);
+    ldn<VEC>(p.w + k, w);
+    ldn<VEC>(gate + k, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      const float a = p.sigmoid_gate ? mb::sigmoid_exact(g[i]) : mb::silu_exact(g[i]);
+      o[i] = v[i] * inv * w[i] * a * p.scale;
+    }
+    stn<VEC>(out + k, o);
+  };
+  auto sumsq = [&](int k) {
+    float v[VEC], ss = 0.f;
+    ldn<VEC>(x + k, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+    return ss;
+  };
+  if (p.group >= p.K) {
+    float ss = 0.f;
+    for (int k = tid * VEC; k < p.K; k += nt * VEC) ss += sumsq(k);
+    const float inv = rsqrtf(mb::block_sum(ss, red) / (float)p.K + p.eps);
+    for (int k = tid * VEC; k < p.K; k += nt * VEC) emit(k, inv);
+    return;
+  }
+  const int warp = tid >> 5, lane = tid & 31, nw = nt >> 5;
+  for (int g0 = warp * p.group; g0 < p.K; g0 += nw * p.group) {
+    float ss = 0.f;
+    for (int k = lane * VEC; k < p.group; k += 32 * VEC) ss += sumsq(g0 + k);
+    const float inv = rsqrtf(mb::warp_sum(ss) / (float)p.group + p.eps);
+    for (int k = lane * VEC; k < p.group; k += 32 * VEC) emit(g0 + k, inv);
+  }
+}
+
+// ------------------------------------------------------------------ token side input
+template <typename T>
+__global__ void __launch_bounds__(128) side_gate_kernel(const float* z, const int* tokens, const bf16* table, long long table_ld, int off,
+                                                        int dim, int rows, int num_rows, T* out, uint32_t* status) {
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (long long)rows * dim) return;
+  const int t = (int)(i / dim), c = (int)(i - (long long)t * dim);
+  const int tok = tokens[t];
+  float e = 0.f;
+  if (tok < 0 || tok >= num_rows) {
+    if (status) atomicCAS(status, 0u, MB_ST_BOUNDS);
+  } else {
+    e = __bfloat162float(table[(size_t)tok * table_ld + off + c]);
+  }
+  const float v = z[i];
+  const float g = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));   // sqrt(2 / pi)
+  stv(out + i, g * e);
+}
+
+__global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, const bf16* table, float* out, int W, int vocab, float scale,
+                                                           uint32_t* status) {
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const int t = blockIdx.x, tok = tokens[t];
+  const bool ok = tok >= 0 && tok < vocab;
+  if (!ok && status && threadIdx.x == 0) atomicCAS(status, 0u, MB_ST_BOUNDS);
+  for (int k = threadIdx.x; k < W; k += blockDim.x)
+    out[(size_t)t * W + k] = ok ? __bfloat162float(table[(size_t)tok * W + k]) * scale : 0.f;
+}
+
+// ------------------------------------------------------------------ rotary + cache write, separate head sizes
+struct RopeDimsParams {
+  int M, Hq, Hkv, dk, dv, rot, dkp, dvp;    // dkp / dvp: padded row lengths of q_out / K and of V
+  const void* qkv;
+  long long qkv_ld;
+  const int* positions;
+  const long long* slots;
+  const float* cos_tab;
+  const float* sin_tab;
+  int max_pos;
+  void* q_out;
+  void* k_cache;
+  void* v_cache;
+  long long num_slots;
+  uint32_t* status;
+};
+
+// grid (tokens, y): the y CTAs of a token share its q | k | v output elements
+template <int VEC, typename T>
+__global__ void __launch_bounds__(256) rope_dims_kernel(const RopeDimsParams p) {
+  const int m = blockIdx.x;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)m * p.qkv_ld;
+  int pos = p.positions[m];
+  if (pos < 0 || (p.rot > 0 && pos >= p.max_pos)) {
+    if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+    pos = 0;
+  }
+  long long slot = p.slots[m];
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+    slot = -1;
+  }
+  const int half = p.rot / 2;
+  const float* cs = p.cos_tab + (size_t)pos * half;
+  const float* sn = p.sin_tab + (size_t)pos * half;
+  const int nq = p.Hq * p.dkp, nk = p.Hkv * p.dkp, nv = p.Hkv * p.dvp;
+  for (int e = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; e < nq + nk + nv; e += gridDim.y * blockDim.x * VEC) {
+    float o[VEC];
+    if (e < nq + nk) {
+      const bool is_q = e < nq;
+      const int i = is_q ? e : e - nq;
+      const int h = i / p.dkp, d = i - h * p.dkp;
+      const T* row = src + (is_q ? 0 : p.Hq * p.dk) + h * p.dk;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+      if (d < p.dk) {
+        ldn<VEC>(row + d, o);
+        if (d < p.rot) {                       // VEC divides rot / 2: the whole vector is on one side
+          float q[VEC];
+          const bool first = d < half;
+          ldn<VEC>(row + (first ? d + half : d - half), q);
+          const int a = first ? d : d - half;
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) {
+            const float c = cs[a + j], s = sn[a + j];
+            o[j] = first ? o[j] * c - q[j] * s : o[j] * c + q[j] * s;
+          }
+        }
+      }
+      if (is_q) stn<VEC>(reinterpret_cast<T*>(p.q_out) + (size_t)m * nq + i, o);
+      else if (slot >= 0) stn<VEC>(reinterpret_cast<T*>(p.k_cache) + (size_t)slot * nk + i, o);
+    } else if (slot >= 0) {
+      const int i = e - nq - nk;
+      const int h = i / p.dvp, d = i - h * p.dvp;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+      if (d < p.dv) ldn<VEC>(src + (size_t)(p.Hq + p.Hkv) * p.dk + h * p.dv + d, o);
+      stn<VEC>(reinterpret_cast<T*>(p.v_cache) + (size_t)slot * nv + i, o);
+    }
+  }
+}
+
+}  // namespace
+
+struct MbStreamNormArgs {
+  int T, W, f32, add_mode, out_mode;
+  const float* x;
+  const void* y;
+  float post_alpha;
+  const void* post_w;
+  const void* post_b;
+  float pre_alpha;
+  const void* pre_w;
+  const void* pre_b;
+  float eps;
+  float* x_out;
+  void* out;
+  float* h32;
+  const void* mu;
+  void* mixes;
+  float* state;
+  const int* q_start;
+  const int* q_len;
+  const int* positions;
+  const int* slots;
+  int num_seqs, num_slots, write_state;
+  uint32_t* status;
+};
+
+struct MbGatedNormArgs {
+  int T, K, group, f32;
+  const float* x;
+  const void* w;
+  const void* gate;
+  long long gate_ld;
+  int sigmoid_gate;
+  float eps, scale;
+  void* out;
+  long long out_ld;
+};
+
+struct MbRopeDimsArgs {
+  int M, Hq, Hkv, dk, dv, rot, dkp, dvp, f32;
+  const void* qkv;
+  long long qkv_ld;
+  const int* positions;
+  const long long* slots;
+  const float* cos_tab;
+  const float* sin_tab;
+  int max_pos;
+  void* q_out;
+  void* k_cache;
+  void* v_cache;
+  long long num_slots;
+  uint32_t* status;
+};
+
+namespace {
+bool al(const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) % n) == 0; }
+int row_threads(int W, int vec) {
+  int n = 32;
+  while (n < 256 && n * vec < W) n <<= 1;
+  return n;
+}
+}  // namespace
+
+extern "C" {
+
+int mb_stream_norm(const MbStreamNormArgs* a, cudaStream_t stream) {
+  if (!a || a->T <= 0 || a->W <= 0 || !a->x) return MB_ERR_BAD_ARG;
+  if (a->add_mode != ADD_NONE && (!a->y || !a->post_w || (a->add_mode == ADD_DYT && !a->post_b))) return MB_ERR_BAD_ARG;
+  if (a->out_mode == OUT_DYT && (!a->pre_w || !a->pre_b)) return MB_ERR_BAD_ARG;
+  if (a->mu && (!a->mixes || !a->state || !a->q_start || !a->q_len || !a->positions || !a->slots || a->num_seqs <= 0 || a->out_mode != OUT_DYT ||
+                a->x_out == a->x))
+    return MB_ERR_BAD_ARG;
+  StreamParams p{};
+  p.T = a->T; p.W = a->W; p.x = a->x; p.y = a->y; p.add_mode = a->add_mode; p.out_mode = a->out_mode;
+  p.post = DytW{a->post_alpha, (const bf16*)a->post_w, (const bf16*)a->post_b};
+  p.pre = DytW{a->pre_alpha, (const bf16*)a->pre_w, (const bf16*)a->pre_b};
+  p.eps = a->eps; p.x_out = a->x_out; p.out = a->out; p.h32 = a->h32;
+  p.mu = (const bf16*)a->mu; p.mixes = a->mixes; p.state = a->state;
+  p.q_start = a->q_start; p.q_len = a->q_len; p.positions = a->positions; p.slots = a->slots;
+  p.num_seqs = a->num_seqs; p.num_slots = a->num_slots; p.write_state = a->write_state; p.status = a->status;
+  const bool v4 = a->W % 4 == 0 && al(a->x, 16) && al(a->y, 16) && al(a->x_out, 16) && al(a->out, 16) && al(a->h32, 16) && al(a->mixes, 16) &&
+                  al(a->state, 16) && al(a->post_w, 8) && al(a->post_b, 8) && al(a->pre_w, 8) && al(a->pre_b, 8) && al(a->mu, 8);
+  const dim3 g(a->T), b(row_threads(a->W, v4 ? 4 : 1));
+  if (a->f32) return (int)(v4 ? mb::launch_kernel(stream_norm_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(stream_norm_kernel<1, float>, g, b, 0, stream, p));
+  return (int)(v4 ? mb::launch_kernel(stream_norm_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(stream_norm_kernel<1, bf16>, g, b, 0, stream, p));
+}
+
+int mb_shift_commit(const float* h32, int W, float* state, const int* q_start, const int* q_len, const int* slots, int num_seqs, int num_slots,
+                    uint32_t* status, cudaStream_t stream) {
+  if (!h32 || !state || W <= 0 || num_seqs <= 0) return MB_ERR_BAD_ARG;
+  return (int)mb::launch_kernel(shift_commit_kernel, dim3(num_seqs), dim3(256), 0, stream, h32, W, state, q_start, q_len, slots, num_slots, status);
+}
+
+int mb_gated_norm(const MbGatedNormArgs* a, cudaStream_t stream) {
+  if (!a || a->T <= 0 || a->K <= 0 || a->group <= 0 || a->K % a->group || !a->x || !a->w || !a->gate || !a->out) return MB_ERR_BAD_ARG;
+  GatedParams p{a->T, a->K, a->group, a->x, (const bf16*)a->w, a->gate, a->gate_ld, a->sigmoid_gate, a->eps, a->scale, a->out, a->out_ld};
+  const size_t es = a->f32 ? 4 : 2;
+  const bool v4 = a->group % 4 == 0 && a->gate_ld % 4 == 0 && a->out_ld % 4 == 0 && al(a->x, 16) && al(a->w, 8) && al(a->gate, 4 * es) && al(a->out, 4 * es);
+  const dim3 g(a->T), b(row_threads(a->K, v4 ? 4 : 1));
+  if (a->f32) return (int)(v4 ? mb::launch_kernel(gated_norm_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(gated_norm_kernel<1, float>, g, b, 0, stream, p));
+  return (int)(v4 ? mb::launch_kernel(gated_norm_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(gated_norm_kernel<1, bf16>, g, b, 0, stream, p));
+}
+
+int mb_side_gate(const float* z, const int* tokens, const void* table, long long table_ld, int off, int dim, int rows, int num_rows, void* out,
+                 int f32, uint32_t* status, cudaStream_t stream) {
+  if (!z || !tokens || !table || !out || rows <= 0 || dim <= 0 || off < 0 || off + dim > table_ld) return MB_ERR_BAD_ARG;
+  const dim3 g((unsigned)(((long long)rows * dim + 127) / 128));
+  if (f32) return (int)mb::launch_kernel(side_gate_kernel<float>, g, dim3(128), 0, stream, z, tokens, (const bf16*)table, table_ld, off, dim, rows, num_rows, (float*)out, status);
+  return (int)mb::launch_kernel(side_gate_kernel<bf16>, g, dim3(128), 0, stream, z, tokens, (const bf16*)table, table_ld, off, dim, rows, num_rows, (bf16*)out, status);
+}
+
+int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, uint32_t* status, cudaStream_t stream) {
+  if (!tokens || !table || !out || M <= 0 || W <= 0) return MB_ERR_BAD_ARG;
+  return (int)mb::launch_kernel(embed_scaled_kernel, dim3(M), dim3(256), 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status);
+}
+
+int mb_rope_dims(const MbRopeDimsArgs* a, cudaStream_t stream) {
+  if (!a || a->M <= 0 || !a->qkv || !a->positions || !a->slots || !a->q_out || !a->k_cache || !a->v_cache) return MB_ERR_BAD_ARG;
+  if (a->dk <= 0 || a->dv <= 0 || a->dk > a->dkp || a->dv > a->dvp || a->rot < 0 || a->rot > a->dk || a->rot % 2) return MB_ERR_UNSUPPORTED;
+  if (a->rot > 0 && (!a->cos_tab || !a->sin_tab)) return MB_ERR_BAD_ARG;
+  RopeDimsParams p{a->M, a->Hq, a->Hkv, a->dk, a->dv, a->rot, a->dkp, a->dvp, a->qkv, a->qkv_ld, a->positions, a->slots, a->cos_tab,
+                   a->sin_tab, a->max_pos, a->q_out, a->k_cache, a->v_cache, a->num_slots, a->status};
+  const bool v4 = a->dk % 4 == 0 && a->dv % 4 == 0 && a->rot % 8 == 0 && a->dkp % 4 == 0 && a->dvp % 4 == 0 && a->qkv_ld % 4 == 0 &&
+                  al(a->qkv, 16) && al(a->q_out, 16) && al(a->k_cache, 16) && al(a->v_cache, 16);
+  const int total = (a->Hq + a->Hkv) * a->dkp + a->Hkv * a->dvp;
+  const int vec = v4 ? 4 : 1;
+  const int want = (total + 256 * vec - 1) / (256 * vec);
+  const dim3 g(a->M, a->M >= 2048 ? 1 : (want < 8 ? want : 8)), b(256);
+  if (a->f32) return (int)(v4 ? mb::launch_kernel(rope_dims_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(rope_dims_kernel<1, float>, g, b, 0, stream, p));
+  return (int)(v4 ? mb::launch_kernel(rope_dims_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(rope_dims_kernel<1, bf16>, g, b, 0, stream, p));
+}
+
+}  // extern "C"

@@ -1,0 +1,486 @@
+"""Ops of models with a 32-bit residual stream: Dynamic-Tanh norms fused around the stream, token-shift
+mixes, attention with separate query/key and value head sizes and a softmax sink, decaying linear
+attention (per-head or per-channel decay), gated group norms and the token side input.
+
+CUDA tensors run the kernels in ``csrc/{stream_norm,attention,attention_tc,attention_simt,linear_attn,
+linear_chunked,gemm_simt}.cu``; CPU tensors run the restatements below, which compute the same quantities
+in fp32 and round where the kernels round. The activation type is bf16, or fp32 for models served in
+32-bit (``Act.fmt`` "bf16" / "fp32").
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import Optional, Tuple
+
+import torch
+
+from . import Act, _count, _native, _ptr, _stream, runtime
+from . import reference as ref
+
+ADD = {None: 0, "dyt": 1, "rms": 2}
+DTYPE = {"bf16": torch.bfloat16, "fp32": torch.float32}
+
+
+@dataclass
+class DytNorm:
+    """tanh(alpha x) w + b."""
+    alpha: float
+    w: torch.Tensor        # bf16 [W]
+    b: torch.Tensor        # bf16 [W]
+
+
+@dataclass
+class RmsNorm:
+    """x / sqrt(mean(x^2) + eps) * w."""
+    w: torch.Tensor        # bf16 [W]
+    eps: float
+
+
+def act_of(t: torch.Tensor, fmt: str) -> Act:
+    """`t` (already of the activation type) as a GEMM operand; on CPU operands are kept in fp32."""
+    d = t if t.is_cuda else t.float()
+    return Act(fmt, t.shape[0], t.shape[1], d, bf16=t if fmt == "bf16" else None)
+
+
+def _f32(fmt: str) -> int:
+    return int(fmt == "fp32")
+
+
+# ----------------------------------------------------------------------------- stream norm
+class _StreamNormArgs(C.Structure):
+    _fields_ = [("T", C.c_int), ("W", C.c_int), ("f32", C.c_int), ("add_mode", C.c_int), ("out_mode", C.c_int),
+                ("x", C.c_void_p), ("y", C.c_void_p), ("post_alpha", C.c_float), ("post_w", C.c_void_p), ("post_b", C.c_void_p),
+                ("pre_alpha", C.c_float), ("pre_w", C.c_void_p), ("pre_b", C.c_void_p), ("eps", C.c_float),
+                ("x_out", C.c_void_p), ("out", C.c_void_p), ("h32", C.c_void_p), ("mu", C.c_void_p), ("mixes", C.c_void_p),
+                ("state", C.c_void_p), ("q_start", C.c_void_p), ("q_len", C.c_void_p), ("positions", C.c_void_p),
+                ("slots", C.c_void_p), ("num_seqs", C.c_int), ("num_slots", C.c_int), ("write_state", C.c_int),
+                ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_stream_norm", [C.POINTER(_StreamNormArgs), C.c_void_p])
+_native.register_optional("mb_shift_commit", [C.c_void_p, C.c_int] + [C.c_void_p] * 4 + [C.c_int, C.c_int, C.c_void_p, C.c_void_p])
+
+
+def dyt_ref(x: torch.Tensor, n: DytNorm) -> torch.Tensor:
+    return torch.tanh(n.alpha * x.float()) * n.w.float() + n.b.float()
+
+
+def stream_norm(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, post=None, pre: Optional[DytNorm] = None,
+                raw: bool = False, want_x: bool = True, mu: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
+                batch=None, write_state: bool = True, want_h32: bool = False):
+    """x [T, W] fp32. With ``y`` (activation type) and ``post`` (DytNorm | RmsNorm): x' = x + post(y), else
+    x' = x. Output h = pre(x'), or x' itself with ``raw``, or none. With ``mu`` [5, W] (and ``state``
+    [slots, W] fp32, ``batch``): the five token-shift mixes of h, and the state advanced to each sequence's
+    last row. Returns (x', h, mixes [5, T, W] or None, h in fp32 or None); x' is x itself when nothing is added."""
+    T, W = x.shape
+    out_dt = DTYPE[fmt]
+    if not x.is_cuda:
+        x1 = x
+        if y is not None:
+            add = dyt_ref(y, post) if isinstance(post, DytNorm) else \
+                y.float() * torch.rsqrt(y.float().pow(2).mean(-1, keepdim=True) + post.eps) * post.w.float()
+            x1 = x + add
+        if pre is None and not raw:
+            return x1, None, None, None
+        h = x1 if raw else dyt_ref(x1, pre)
+        mixes = None
+        if mu is not None:
+            prev = torch.zeros_like(h)
+            qs, ql, sl = batch.q_start.tolist(), batch.q_len.tolist(), batch.state_slots.tolist()
+            for s, n in enumerate(ql):
+                if n <= 0:
+                    continue
+                r = qs[s]
+                if int(batch.positions[r]) != 0:
+                    prev[r] = state[sl[s]]
+                prev[r + 1:r + n] = h[r:r + n - 1]
+            mixes = (h[None] + (prev - h)[None] * mu.float()[:, None, :]).to(out_dt)
+            if write_state:
+                for s, n in enumerate(ql):
+                    if n > 0:
+                        state[sl[s]] = h[qs[s] + n - 1]
+        return x1, h.to(out_dt), mixes, (h if want_h32 else None)
+    dev = x.device
+    a = _StreamNormArgs()
+    a.T, a.W, a.f32 = T, W, _f32(fmt)
+    a.x = _ptr(x)
+    x1 = x
+    if y is not None:
+        assert y.dtype == out_dt and y.is_contiguous()
+        a.y, a.post_w = _ptr(y), _ptr(post.w)
+        if isinstance(post, DytNorm):
+            a.add_mode, a.post_alpha, a.post_b = 1, post.alpha, _ptr(post.b)
+        else:
+            a.add_mode, a.eps = 2, post.eps
+        if want_x:
+            x1 = torch.empty_like(x)
+            a.x_out = _ptr(x1)
+    h = mixes = h32 = None
+    if pre is not None or raw:
+        h = torch.empty(T, W, dtype=out_dt, device=dev)
+        a.out, a.out_mode = _ptr(h), 2 if raw else 1
+        if pre is not None:
+            a.pre_alpha, a.pre_w, a.pre_b = pre.alpha, _ptr(pre.w), _ptr(pre.b)
+        if want_h32:
+            h32 = torch.empty(T, W, dtype=torch.float32, device=dev)
+            a.h32 = _ptr(h32)
+    if mu is not None:
+        mixes = torch.empty(5, T, W, dtype=out_dt, device=dev)
+        a.mu, a.mixes, a.state = _ptr(mu), _ptr(mixes), _ptr(state)
+        a.q_start, a.q_len, a.positions, a.slots = (_ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.positions),
+                                                    _ptr(batch.state_slots))
+        a.num_seqs, a.num_slots, a.write_state = batch.q_len.numel(), state.shape[0], int(write_state)
+    a.status = _ptr(runtime(dev).status)
+    _native.check(_native.lib().mb_stream_norm(C.byref(a), _stream()), f"stream_norm[T={T} W={W}]")
+    _count()
+    return x1, h, mixes, h32
+
+
+def shift_commit(h32: torch.Tensor, state: torch.Tensor, batch) -> None:
+    """state[slot] := h of each sequence's last row in ``batch`` (sequences of zero rows keep theirs)."""
+    if not h32.is_cuda:
+        for s, n in enumerate(batch.q_len.tolist()):
+            if n > 0:
+                state[int(batch.state_slots[s])] = h32[int(batch.q_start[s]) + n - 1]
+        return
+    rc = _native.lib().mb_shift_commit(_ptr(h32), h32.shape[1], _ptr(state), _ptr(batch.q_start), _ptr(batch.q_len),
+                                       _ptr(batch.state_slots), batch.q_len.numel(), state.shape[0],
+                                       _ptr(runtime(h32.device).status), _stream())
+    _native.check(rc, "shift_commit")
+    _count()
+
+
+# ----------------------------------------------------------------------------- projections of the token-shift mixes
+def grouped_ok(width: int, rows: int, fmt: str) -> bool:
+    """Whether the r, k, v, g projections can be one grouped tcgen05 GEMM: whole 128-row weight tiles each."""
+    return fmt == "bf16" and rows % 128 == 0 and width % 8 == 0
+
+
+_GROUP_LISTS: dict = {}          # never evicted: captured graphs hold the lists' addresses (a few KB per row count)
+_GROUPED_MAX_ROWS = 256          # above this, one full-width GEMM per projection fills the GPU by itself
+
+
+def _group_list(T: int, groups: int, device):
+    """Work list of a grouped GEMM whose group s owns rows [s T, (s + 1) T): (expert, first row, rows) per tile."""
+    tn = 16
+    while tn < T and tn < 64:
+        tn <<= 1
+    key = (T, groups, str(device))
+    if key not in _GROUP_LISTS:
+        tiles = [(s, s * T + r, min(tn, T - r)) for s in range(groups) for r in range(0, T, tn)]
+        cols = [torch.tensor(c, dtype=torch.int32).to(device) for c in zip(*tiles)]
+        _GROUP_LISTS[key] = (*cols, len(tiles))
+    e, r0, nr, n = _GROUP_LISTS[key]
+    return e, r0, nr, n, tn
+
+
+def mix_projections(mixes: torch.Tensor, w, fmt: str):
+    """r, k, v, g [T, H D] from the first four token-shift mixes, each through its own matrix."""
+    from . import linear
+    _, T, W = mixes.shape
+    if w.rkvg_stack is None or not mixes.is_cuda:
+        return tuple(linear(act_of(mixes[s], fmt), w.rkvg[s]) for s in range(4))
+    n = w.rkvg_stack.N // 4
+    if T > _GROUPED_MAX_ROWS:
+        from . import QuantWeight
+        if not w.rkvg:
+            w.rkvg = [QuantWeight(fmt, n, W, w.rkvg_stack.data[s * n:(s + 1) * n]) for s in range(4)]
+        return tuple(linear(act_of(mixes[s], fmt), w.rkvg[s]) for s in range(4))
+    e, r0, nr, tiles, tn = _group_list(T, 4, mixes.device)
+    y = linear(act_of(mixes[:4].reshape(4 * T, W), fmt), w.rkvg_stack, grouped=(e, r0, nr, n, tiles, tn))
+    return tuple(y[s * T:(s + 1) * T] for s in range(4))
+
+
+# ----------------------------------------------------------------------------- gated norm
+class _GatedNormArgs(C.Structure):
+    _fields_ = [("T", C.c_int), ("K", C.c_int), ("group", C.c_int), ("f32", C.c_int), ("x", C.c_void_p), ("w", C.c_void_p),
+                ("gate", C.c_void_p), ("gate_ld", C.c_longlong), ("sigmoid_gate", C.c_int), ("eps", C.c_float),
+                ("scale", C.c_float), ("out", C.c_void_p), ("out_ld", C.c_longlong)]
+
+
+_native.register_optional("mb_gated_norm", [C.POINTER(_GatedNormArgs), C.c_void_p])
+
+
+def gated_norm(x: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, fmt: str, *, group: int, gate_act: str, eps: float,
+               scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """scale * act(gate) * w * x / rms(x over groups of `group` channels). x [T, K] fp32; ``gate`` [T, K] may
+    be a column range; ``gate_act`` "silu" | "sigmoid"; ``out`` may be a column range of a wider matrix."""
+    T, K = x.shape
+    if out is None:
+        out = torch.empty(T, K, dtype=DTYPE[fmt], device=x.device)
+    if not x.is_cuda:
+        g = x.view(T, K // group, group)
+        n = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, K)
+        z = gate.float()
+        act = torch.sigmoid(z) if gate_act == "sigmoid" else torch.nn.functional.silu(z)
+        out.copy_(n * w.float() * act * scale)
+        return out
+    assert x.is_contiguous() and gate.stride(1) == 1 and out.stride(1) == 1 and gate.dtype == out.dtype == DTYPE[fmt]
+    a = _GatedNormArgs(T, K, group, _f32(fmt), _ptr(x), _ptr(w), _ptr(gate), gate.stride(0), int(gate_act == "sigmoid"),
+                       float(eps), float(scale), _ptr(out), out.stride(0))
+    _native.check(_native.lib().mb_gated_norm(C.byref(a), _stream()), f"gated_norm[T={T} K={K}]")
+    _count()
+    return out
+
+
+# ----------------------------------------------------------------------------- embedding, token side input
+_native.register_optional("mb_embed_scaled", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_void_p,
+                                              C.c_void_p])
+_native.register_optional("mb_side_gate", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_longlong] + [C.c_int] * 4 +
+                          [C.c_void_p, C.c_int, C.c_void_p, C.c_void_p])
+
+
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+    """fp32 [T, W] = table[ids] * scale."""
+    if not table.is_cuda:
+        return table[ids.long()].float() * scale
+    M, W = ids.numel(), table.shape[1]
+    out = torch.empty(M, W, dtype=torch.float32, device=table.device)
+    rc = _native.lib().mb_embed_scaled(_ptr(ids), _ptr(table), _ptr(out), M, W, table.shape[0], float(scale),
+                                       _ptr(runtime(table.device).status), _stream())
+    _native.check(rc, "embed_scaled")
+    _count()
+    return out
+
+
+def side_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, off: int, fmt: str) -> torch.Tensor:
+    """gelu_tanh(z) * table[ids, off : off + dim]; z [T, dim] fp32."""
+    T, dim = z.shape
+    if not z.is_cuda:
+        e = table[ids.long(), off:off + dim].float()
+        return (torch.nn.functional.gelu(z, approximate="tanh") * e).to(DTYPE[fmt])
+    out = torch.empty(T, dim, dtype=DTYPE[fmt], device=z.device)
+    rc = _native.lib().mb_side_gate(_ptr(z), _ptr(ids), _ptr(table), table.stride(0), off, dim, T, table.shape[0], _ptr(out),
+                                    _f32(fmt), _ptr(runtime(z.device).status), _stream())
+    _native.check(rc, "side_gate")
+    _count()
+    return out
+
+
+# ----------------------------------------------------------------------------- attention with its own head sizes
+class _RopeDimsArgs(C.Structure):
+    _fields_ = [("M", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("rot", C.c_int),
+                ("dkp", C.c_int), ("dvp", C.c_int), ("f32", C.c_int), ("qkv", C.c_void_p), ("qkv_ld", C.c_longlong),
+                ("positions", C.c_void_p), ("slots", C.c_void_p), ("cos_tab", C.c_void_p), ("sin_tab", C.c_void_p),
+                ("max_pos", C.c_int), ("q_out", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p),
+                ("num_slots", C.c_longlong), ("status", C.c_void_p)]
+
+
+class _SimtAttnArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("block_table", C.c_void_p),
+                ("max_blocks", C.c_int), ("q_start", C.c_void_p), ("q_len", C.c_void_p), ("ctx_len", C.c_void_p),
+                ("total_rows", C.c_int), ("num_seqs", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("dk", C.c_int),
+                ("dv", C.c_int), ("dkp", C.c_int), ("dvp", C.c_int), ("block_size", C.c_int), ("num_blocks", C.c_longlong),
+                ("scale", C.c_float), ("out_scale", C.c_float), ("sink", C.c_int), ("f32", C.c_int), ("out", C.c_void_p),
+                ("out_ld", C.c_longlong), ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_rope_dims", [C.POINTER(_RopeDimsArgs), C.c_void_p])
+_native.register_optional("mb_attn_simt", [C.POINTER(_SimtAttnArgs), C.c_void_p])
+
+
+def padded_head_dims(dk: int, dv: int, fmt: str) -> Tuple[int, int]:
+    """Row lengths of the K and V pools: the tensor-core kernels' tiles (64 or 128 each, or 256 both) for bf16
+    caches, the head sizes themselves where only the fp32 kernel serves the shape."""
+    if fmt != "bf16" or max(dk, dv) > 256:
+        return dk, dv
+    if max(dk, dv) > 128:
+        return 256, 256
+    tile = lambda d: 64 if d <= 64 else 128
+    return tile(dk), tile(dv)
+
+
+def rope_dims(qkv: torch.Tensor, *, Hq: int, Hkv: int, dk: int, dv: int, positions, slots, k_cache, v_cache, cos, sin,
+              fmt: str) -> torch.Tensor:
+    """qkv [T, Hq dk | Hkv dk | Hkv dv]: rotate the first 2 * cos.shape[1] dimensions of every q and k head
+    (rotate-half pairing) and scatter k, v into caches [blocks, block, Hkv, padded]. Returns q [T, Hq, padded dk]."""
+    M = qkv.shape[0]
+    dkp, dvp = k_cache.shape[3], v_cache.shape[3]
+    rot = 2 * cos.shape[1] if cos is not None else 0
+    if not qkv.is_cuda:
+        x = qkv.float()
+        q = x[:, :Hq * dk].view(M, Hq, dk)
+        k = x[:, Hq * dk:(Hq + Hkv) * dk].view(M, Hkv, dk)
+        v = x[:, (Hq + Hkv) * dk:].reshape(M, Hkv, dv)
+        if rot:
+            q, k = ref.apply_rope_neox(q, positions, cos, sin), ref.apply_rope_neox(k, positions, cos, sin)
+        pad = torch.nn.functional.pad
+        ok = slots >= 0
+        idx = slots[ok].long()
+        k_cache.view(-1, Hkv, dkp)[idx] = pad(k, (0, dkp - dk))[ok].to(k_cache.dtype)
+        v_cache.view(-1, Hkv, dvp)[idx] = pad(v, (0, dvp - dv))[ok].to(v_cache.dtype)
+        return pad(q, (0, dkp - dk)).to(DTYPE[fmt])
+    assert qkv.dtype == k_cache.dtype == v_cache.dtype == DTYPE[fmt]
+    q_out = torch.empty(M, Hq, dkp, dtype=DTYPE[fmt], device=qkv.device)
+    a = _RopeDimsArgs(M, Hq, Hkv, dk, dv, rot, dkp, dvp, _f32(fmt), _ptr(qkv), qkv.stride(0), _ptr(positions), _ptr(slots),
+                      _ptr(cos) if rot else None, _ptr(sin) if rot else None, cos.shape[0] if rot else 0, _ptr(q_out),
+                      _ptr(k_cache), _ptr(v_cache), k_cache.shape[0] * k_cache.shape[1], _ptr(runtime(qkv.device).status))
+    _native.check(_native.lib().mb_rope_dims(C.byref(a), _stream()), f"rope_dims[T={M}]")
+    _count()
+    return q_out
+
+
+def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int, scale: float, sink: bool, fmt: str,
+                   out: torch.Tensor, out_scale: float = 1.0, kernel: str = "auto") -> torch.Tensor:
+    """Causal paged attention of q [T, Hq, padded dk] into ``out`` [T, Hq * dv] (may be a column range), times
+    ``out_scale``. ``sink``: one is added to the softmax denominator. The softmax weights keep 32-bit
+    precision: they enter the product with V as two bf16 terms. ``kernel``: auto | simt | mma | tc (tests)."""
+    T, Hq, dkp = q.shape
+    nb, bs, Hkv, _ = k_cache.shape
+    dvp = v_cache.shape[3]
+    if not q.is_cuda:
+        qs, ql, cl = batch.q_start.tolist(), batch.q_len.tolist(), batch.ctx_len.tolist()
+        G = Hq // Hkv
+        for s, n in enumerate(ql):
+            if n <= 0:
+                continue
+            ctx = cl[s]
+            blocks = batch.block_table[s, :(ctx + bs - 1) // bs].long()
+            k = k_cache[blocks].reshape(-1, Hkv, dkp)[:ctx, :, :dk].float().repeat_interleave(G, 1)
+            v = v_cache[blocks].reshape(-1, Hkv, dvp)[:ctx, :, :dv].float().repeat_interleave(G, 1)
+            sc = torch.einsum("ihd,jhd->hij", q[qs[s]:qs[s] + n, :, :dk].double(), k.double()) * scale
+            i = torch.arange(ctx - n, ctx)[:, None]
+            sc.masked_fill_(torch.arange(ctx)[None, :] > i, float("-inf"))
+            m = sc.amax(-1, keepdim=True)
+            if sink:
+                m = m.clamp(min=0.0)
+            e = torch.exp(sc - m)
+            den = e.sum(-1, keepdim=True) + (torch.exp(-m) if sink else 0.0)
+            o = torch.einsum("hij,jhd->ihd", e / den, v.double()) * out_scale
+            out[qs[s]:qs[s] + n] = o.reshape(n, Hq * dv).to(out.dtype)
+        return out
+    L, rt = _native.lib(), runtime(q.device)
+    S, mq = batch.q_len.numel(), int(batch.max_q_len)
+    assert out.stride(1) == 1 and out.dtype == DTYPE[fmt]
+    G = Hq // Hkv
+    tiles_ok = fmt == "bf16" and dkp in (64, 128, 256) and dvp in (64, 128, 256) and (dkp == dvp or max(dkp, dvp) <= 128) \
+        and (dv != dvp or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0))
+    if kernel == "auto":
+        kernel = "mma" if tiles_ok else "simt"
+        if tiles_ok and tc_serves(dkp, dvp, dv, out) and mq >= 128:
+            kernel = "tc"
+        elif kernel == "mma" and dkp == 256 and 16 < G * mq <= 32:
+            kernel = "simt"                          # between the two row-tile limits of the 256-wide tiles
+    if kernel == "simt":
+        a = _SimtAttnArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_table), batch.block_table.stride(0),
+                          _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len), T, S, Hq, Hkv, dk, dv, dkp, dvp, bs, nb,
+                          float(scale), float(out_scale), int(sink), _f32(fmt), _ptr(out), out.stride(0), _ptr(rt.status))
+        _native.check(L.mb_attn_simt(C.byref(a), _stream()), f"attn_simt[T={T}]")
+        _count()
+        return out
+    if kernel == "tc":
+        t = _native.AttnTcArgs()
+        t.q, t.k_cache, t.v_cache, t.block_table = _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_table)
+        t.q_start, t.q_len, t.ctx_len = _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len)
+        t.out, t.status, t.num_blocks, t.max_blocks, t.num_seqs, t.max_q_len = _ptr(out), _ptr(rt.status), nb, \
+            batch.block_table.stride(0), S, mq
+        t.Hq, t.Hkv, t.D, t.block_size, t.scale, t.v_mn = Hq, Hkv, dkp, bs, float(scale), 1
+        t.out_ld, t.out_scale, t.sink, t.split_p = out.stride(0), float(out_scale), int(sink), 1
+        _native.check(L.mb_attn_prefill_tc(C.byref(t), _stream()), "attn_prefill_tc")
+        _count()
+        return out
+    from . import _ATTN_PART_TOKENS
+    a = _native.AttnArgs()
+    a.q, a.k_cache, a.v_cache = _ptr(q), _ptr(k_cache), _ptr(v_cache)
+    a.block_table, a.max_blocks = _ptr(batch.block_table), batch.block_table.stride(0)
+    a.q_start, a.q_len, a.ctx_len = _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len)
+    a.num_seqs, a.max_q_len, a.max_ctx = S, mq, int(batch.max_ctx)
+    a.Hq, a.Hkv, a.D, a.block_size, a.num_blocks, a.scale = Hq, Hkv, dkp, bs, nb, float(scale)
+    a.out, a.total_rows, a.part_tokens, a.status = _ptr(out), T, _ATTN_PART_TOKENS, _ptr(rt.status)
+    a.DV, a.dv, a.out_ld, a.out_scale, a.sink, a.split_p = dvp, dv, out.stride(0), float(out_scale), int(sink), 1
+    if G * mq <= 32:
+        rt.ensure_attn_ws(L.mb_attn_ws_bytes(T, Hq, dvp, int(batch.max_ctx), _ATTN_PART_TOKENS))
+    a.ws, a.ws_bytes = _ptr(rt.attn_ws), rt.attn_ws.numel()
+    _native.check(L.mb_paged_attention(C.byref(a), _stream()), f"attention_dims[T={T}]")
+    _count()
+    return out
+
+
+def tc_serves(dkp: int, dvp: int, dv: int, out: torch.Tensor) -> bool:
+    """Shapes of the tcgen05 prefill kernel: equal 128- or 256-wide tiles stored whole in 16-byte vectors."""
+    from . import _ATTN_TC
+    return _ATTN_TC and dkp == dvp == dv and dkp in (128, 256) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+
+
+# ----------------------------------------------------------------------------- decaying linear attention
+class _LinearAttnArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("q_ld", C.c_longlong), ("k_ld", C.c_longlong),
+                ("v_ld", C.c_longlong), ("H", C.c_int), ("DK", C.c_int), ("DV", C.c_int), ("f32", C.c_int), ("log_w", C.c_void_p),
+                ("decay", C.c_void_p), ("u", C.c_void_p), ("state", C.c_void_p), ("out", C.c_void_p), ("q_start", C.c_void_p),
+                ("q_len", C.c_void_p), ("positions", C.c_void_p), ("slots", C.c_void_p), ("num_seqs", C.c_int),
+                ("num_slots", C.c_int), ("write_state", C.c_int), ("write_out", C.c_int), ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_linear_attn", [C.POINTER(_LinearAttnArgs), C.c_void_p])
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, *, heads: int, dk: int, dv: int,
+                     fmt: str, log_w: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None,
+                     u: Optional[torch.Tensor] = None, write_state: bool = True, write_out: bool = True,
+                     kernel: str = "auto") -> Optional[torch.Tensor]:
+    """Per head S_t = diag(w_t) S_(t-1) + k_t v_t^T over a ragged batch; w_t = ``decay`` [H], or exp(``log_w``
+    [T, H dk]). Output q_t^T S_t, or with ``u`` [H, dk] q_t^T (S_(t-1) + diag(u) k_t v_t^T). q, k, v [T, *]
+    may be column ranges; state [slots, H, dk, dv] fp32. Returns fp32 [T, H dv]."""
+    T, H = q.shape[0], heads
+    if not q.is_cuda:
+        out = torch.zeros(T, H * dv, dtype=torch.float32)
+        qs, ql, sl = batch.q_start.tolist(), batch.q_len.tolist(), batch.state_slots.tolist()
+        qf, kf, vf = q.float().view(T, H, dk), k.float().view(T, H, dk), v.float().view(T, H, dv)
+        w = torch.exp(log_w).view(T, H, dk) if log_w is not None else decay.float()[None, :, None].expand(T, H, dk)
+        for s, n in enumerate(ql):
+            if n <= 0:
+                continue
+            S = torch.zeros(H, dk, dv) if int(batch.positions[qs[s]]) == 0 else state[sl[s]].clone()
+            for t in range(qs[s], qs[s] + n):
+                kv = kf[t][:, :, None] * vf[t][:, None, :]
+                if u is not None:
+                    out[t] = ((S + u[:, :, None] * kv) * qf[t][:, :, None]).sum(1).reshape(-1)
+                S = w[t][:, :, None] * S + kv
+                if u is None:
+                    out[t] = (S * qf[t][:, :, None]).sum(1).reshape(-1)
+            if write_state:
+                state[sl[s]] = S
+        return out if write_out else None
+    assert q.dtype == k.dtype == v.dtype == DTYPE[fmt] and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    dev = q.device
+    out = torch.empty(T, H * dv, dtype=torch.float32, device=dev) if write_out else None
+    a = _LinearAttnArgs(_ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), H, dk, dv, _f32(fmt), _ptr(log_w),
+                        _ptr(decay), _ptr(u), _ptr(state), _ptr(out), _ptr(batch.q_start), _ptr(batch.q_len),
+                        _ptr(batch.positions), _ptr(batch.state_slots), batch.q_len.numel(), state.shape[0], int(write_state),
+                        int(write_out), _ptr(runtime(dev).status))
+    _native.check(_native.lib().mb_linear_attn(C.byref(a), _stream()), f"linear_attn[T={T} H={H}]")
+    _count()
+    return out
+
+
+# ----------------------------------------------------------------------------- CUDA-core GEMM
+class _SimtGemmArgs(C.Structure):
+    _fields_ = [("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("x_bf16", C.c_int), ("w_bf16", C.c_int), ("out_bf16", C.c_int),
+                ("X", C.c_void_p), ("ldx", C.c_longlong), ("W", C.c_void_p), ("ldw", C.c_longlong), ("out", C.c_void_p),
+                ("ldo", C.c_longlong), ("a_op", C.c_int), ("epilogue", C.c_int), ("bias", C.c_void_p), ("epi_a", C.c_float),
+                ("epi_b", C.c_float), ("epi_n", C.c_int)]
+
+
+_native.register_optional("mb_gemm_simt", [C.POINTER(_SimtGemmArgs), C.c_void_p])
+
+
+def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, tanh_in: bool = False, epilogue: int = 0, bias=None,
+              epi_a: float = 0.0, epi_b: float = 0.0, epi_n: int = 0) -> torch.Tensor:
+    M, K = x.shape
+    N = w.shape[0]
+    assert x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
+    bf = torch.bfloat16
+    a = _SimtGemmArgs(M, N, K, int(x.dtype == bf), int(w.dtype == bf), int(out.dtype == bf), _ptr(x), x.stride(0), _ptr(w),
+                      w.stride(0), _ptr(out), out.stride(0), int(tanh_in), epilogue, _ptr(bias), float(epi_a), float(epi_b), epi_n)
+    _native.check(_native.lib().mb_gemm_simt(C.byref(a), _stream()), f"gemm_simt[M={M} N={N} K={K}]")
+    _count()
+    return out
+
+
+def log_decay(z: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor) -> torch.Tensor:
+    """-exp(tanh(z) w2^T + w0) in fp32: the logarithm of the decay exp(-exp(.)). z [T, rank] fp32."""
+    if not z.is_cuda:
+        return -torch.exp((torch.tanh(z).double() @ w2.double().t()).float() + w0)
+    out = torch.empty(z.shape[0], w2.shape[0], dtype=torch.float32, device=z.device)
+    return gemm_simt(z, w2, out, tanh_in=True, epilogue=4, bias=w0)

@@ -116,6 +116,7 @@ class FfnW:
     down: QuantWeight = None
     interleaved: bool = False        # True -> the GEMM epilogue applies SwiGLU
     down_in_scale: float = 0.0       # NVFP4: calibrated global scale of down's input (0 = per-token dynamic)
+    clamp_glu: Optional[tuple] = None   # (alpha, limit): clamped GLU instead of SwiGLU (rows interleaved)
 
 
 @dataclass
@@ -195,6 +196,63 @@ class MlaW:
 
 
 @dataclass
+class SinkAttnW:
+    """Attention with its own query/key and value head sizes, partial rotary positions and a softmax sink."""
+    qkv: QuantWeight = None
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    scale: float = 1.0
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+
+
+@dataclass
+class TimeMixW:
+    """RWKV-style time mixing: token-shift mixes, per-channel data-dependent decay, bonus, gated group norm."""
+    mu: torch.Tensor = None              # bf16 [5, W]: r, k, v, g, w
+    rkvg: List[QuantWeight] = field(default_factory=list)
+    w1: QuantWeight = None               # hidden -> rank
+    w2: torch.Tensor = None              # [H D, rank], as stored
+    w0: torch.Tensor = None              # fp32 [H D]
+    u: torch.Tensor = None               # fp32 [H, D]
+    norm: torch.Tensor = None            # bf16 [H D]
+    heads: int = 0
+    dim: int = 0
+    rkvg_stack: Optional[QuantWeight] = None   # r | k | v | g stacked for the grouped GEMM (None: one GEMM each)
+
+
+@dataclass
+class ParallelW:
+    """Two mixers on the same input; their output projections are one GEMM over [left | right]."""
+    left: SinkAttnW = None
+    right: TimeMixW = None
+    o: QuantWeight = None                # [W, left width + right width]
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass
+class LightningW:
+    qkvg: QuantWeight = None
+    o: QuantWeight = None
+    norm: torch.Tensor = None            # bf16 [H vdim]
+    decay: torch.Tensor = None           # fp32 [H]
+    heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+
+
+@dataclass
+class TokenSideW:
+    gate: QuantWeight = None             # width -> dim
+    proj: QuantWeight = None             # dim -> width
+    norm: object = None                  # ops.mixers.RmsNorm
+    offset: int = 0                      # this layer's first column of ModelW.side_embed
+
+
+@dataclass
 class LayerW:
     kind: str = "attention"
     ffn_kind: str = "dense"
@@ -206,6 +264,7 @@ class LayerW:
     ffn: object = None
     hc_attn: Optional[tuple] = None              # hyper-connection site in front of the mixer: (fn bf16, scale fp32 [3], base fp32)
     hc_ffn: Optional[tuple] = None               # ... and in front of the feed-forward block
+    side: Optional[TokenSideW] = None            # per-layer token side input, after the feed-forward block
 
 
 @dataclass
@@ -226,6 +285,7 @@ class ModelW:
     mtp: Optional[MtpW] = None
     vocab_lo: int = 0
     vocab_hi: int = 0
+    side_embed: Optional[torch.Tensor] = None      # bf16 [V, layers * side dim]
 
     def nbytes(self) -> int:
         n = 0
@@ -389,6 +449,9 @@ class Loader:
         c = self.cfg
         if c.arch == "nemotron_h":
             return loader_ext.load_nemotron(self)
+        if c.arch == "fabulix":
+            from .fabulix import load_fabulix
+            return load_fabulix(self)
         m = ModelW()
         m.embed = self.vec("model.embed_tokens.weight")
         m.final_norm = self.vec("model.norm.weight")

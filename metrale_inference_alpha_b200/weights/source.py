@@ -158,6 +158,11 @@ class SyntheticSource(TensorSource):
         c = self.cfg
         if c.arch == "nemotron_h":
             return self._describe_nemotron()
+        if c.arch == "fabulix":
+            from .fabulix import tensor_shapes
+            for name, (shape, kind) in tensor_shapes(c).items():
+                self._vec(name, shape, kind)
+            return
         self._lin("model.embed_tokens", c.vocab_size, c.hidden_size, quant=False)
         if not c.tie_embeddings:
             self._lin("lm_head", c.vocab_size, c.hidden_size, quant=False)
@@ -362,6 +367,12 @@ class SyntheticSource(TensorSource):
                 return self._rand(name, shape, 0.1).float()
             if kind == "small":
                 return self._rand(name, shape, 0.02).to(torch.bfloat16)
+            if kind == "linear":                             # unit-gain rows, for networks without statistics in their norms
+                return self._rand(name, shape, shape[-1] ** -0.5).to(torch.bfloat16)
+            if kind == "alpha":
+                return (0.5 + self._rand(name, (1,), 0.05).reshape(())).to(torch.bfloat16)
+            if kind == "mix":
+                return (0.5 + self._rand(name, shape, 0.2)).to(torch.bfloat16)
         prefix, suffix = self._split(name)
         if prefix is None or not self.has(name):
             raise KeyError(name)
