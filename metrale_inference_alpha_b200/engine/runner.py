@@ -12,7 +12,7 @@ from __future__ import annotations
 import contextlib
 import gc
 import time
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Dict, List, Optional, Tuple
 
 import numpy as np
@@ -287,7 +287,10 @@ class ModelRunner:
             barr = np.asarray(blocks, dtype=np.int64)
             slots[row:row + n] = barr[pp // bs] * bs + pp % bs
             qs[s], ql[s], ctx[s], state[s] = row, n, p0 + n, it.seq.state_slot
-            if it.sample:
+            if it.want is not None:
+                lrows[nl:nl + len(it.want)] = row + np.asarray(it.want, dtype=np.int64)
+                nl += len(it.want)
+            elif it.sample:
                 k = it.verify if logits_all_verify else 0
                 lrows[nl:nl + k + 1] = np.arange(row + n - 1 - k, row + n)
                 nl += k + 1
@@ -596,6 +599,28 @@ class ModelRunner:
         self.last_hidden = hidden
         return rung
 
+    def _logits_graph(self, plan: StepPlan) -> torch.Tensor:
+        """fp32 logits [rung, vocab] of a one-token-per-sequence step, replayed from the rung's graph (captured
+        on first use like ``_decode_graph``'s, ending at the logits instead of a selected token)."""
+        rung = self._rung(len(plan.items))
+        key = ("logits", rung)
+        if key not in self.graphs:
+            null = self._stage(StepPlan("decode", []), pad_seqs=rung)
+            null.max_ctx, null.max_q_len = self.sched.max_model_len, 1
+            self.decoder.forward(null, self.caches, out_f32=True)
+            torch.cuda.synchronize(self.device)
+            g = torch.cuda.CUDAGraph()
+            count0 = ops.launch_count
+            with _capture(g):
+                logits = self.decoder.forward(null, self.caches, out_f32=True)[0]
+            self.graphs[key] = (g, ops.launch_count - count0, logits)
+        self._stage(StepPlan("decode", [replace(it, want=[0]) for it in plan.items]), pad_seqs=rung)
+        g, launches, logits = self.graphs[key]
+        g.replay()
+        ops.launch_count += launches
+        self.graph_replays += 1
+        return logits
+
     def _verify_graph(self, plan: StepPlan, K: int) -> None:
         """Replay (capturing on first use) the CUDA graph of a speculative verify step in which
         every sequence feeds K drafts: one forward over rung x (K + 1) rows, argmax of every row
@@ -740,6 +765,26 @@ class ModelRunner:
             r += k
         return StepResult(toks, lpo if lps else None, hidden=self.last_hidden,
                           device_ms=(time.perf_counter() - t0) * 1e3)
+
+    def execute_fed(self, plan: StepPlan) -> Optional[torch.Tensor]:
+        """One step of fed sequences: fp32 logits (on the host) of every item's wanted rows, in item order, or
+        None when nothing is wanted. All items run as one batch; a step of single tokens takes the decode graphs."""
+        rows = [(i, w) for i, it in enumerate(plan.items) for w in it.want]
+        if self.graphs_ready() and all(len(it.tokens) == 1 and it.start_pos > 0 for it in plan.items):
+            logits = self._logits_graph(plan)
+            out = logits[[i for i, _ in rows]] if rows else None
+        elif rows:
+            out = self.decoder.forward(self._stage_with_adapters(plan), self.caches, out_f32=True)[0]
+        else:
+            self.decoder.backbone(self._stage_with_adapters(plan), self.caches)
+            out = None
+        self.tp.end_forward()
+        self._post_status()
+        out = None if out is None else out.float().cpu()
+        if self.device.type == "cuda":
+            torch.cuda.current_stream(self.device).synchronize()
+        self._check_status()
+        return out
 
     def _execute_host_logits(self, plan: StepPlan, t0: float) -> StepResult:
         """Full-logits path: penalties, logit bias, grammar masks, top-n-sigma, top log-probs."""

@@ -19,6 +19,7 @@ from collections import deque
 from typing import Callable, Deque, Dict, List, Optional
 
 from ..cache import BlockAllocator, NoFreeBlocks, RadixTree
+from ..sampling.params import SamplingParams
 from .policy import SchedulerConfig, make_policy
 from .types import (FinishReason, Request, RequestOutput, SeqStatus, SeqStep, Sequence, StepPlan,
                     StepResult)
@@ -179,6 +180,45 @@ class SchedulerCore:
         if self.pool is not None and seq.state_slot:
             self.pool.free(seq.state_slot)
             seq.state_slot = 0
+
+    # ------------------------------------------------------------------ fed sequences
+    # A caller that brings every token itself (trace replay, scoring) gets its cache blocks and state slot from
+    # the same pools and lists as a served request; it decides which tokens run in which step.
+    def open_fed(self, request_id: str) -> Sequence:
+        """Admit an empty sequence whose tokens will be fed with ``feed``."""
+        if self.num_active >= self.cfg.max_num_seqs:
+            raise RuntimeError(f"more than {self.cfg.max_num_seqs} live sequences")
+        if request_id in self._by_req and not self._by_req[request_id].is_finished():
+            raise ValueError(f"request {request_id!r} is live")
+        seq = Sequence(Request(request_id, [], SamplingParams()), next(self._ids))
+        if self.pool is not None:
+            seq.state_slot = self.pool.alloc()
+        seq.status = SeqStatus.PREFILL
+        self.prefilling.append(seq)
+        self._by_req[request_id] = seq
+        self.stats["admitted"] += 1
+        return seq
+
+    def feed(self, seq: Sequence, tokens: List[int], want: List[int]) -> SeqStep:
+        """The next tokens of a fed sequence as one step item; ``fed`` marks them computed afterwards."""
+        if not tokens or len(seq.tokens) + len(tokens) > self.cfg.max_model_len:
+            raise ValueError(f"{len(seq.tokens)} + {len(tokens)} tokens: outside 1..{self.cfg.max_model_len}")
+        start = len(seq.tokens)
+        self._ensure_blocks(seq, start + len(tokens))
+        seq.tokens = seq.tokens + list(tokens)
+        return SeqStep(seq, list(tokens), start, sample=False, want=list(want))
+
+    def fed(self, plan: StepPlan) -> None:
+        self.stats["steps"] += 1
+        for it in plan.items:
+            it.seq.num_computed = len(it.seq.tokens)
+            self.stats["prefill_tokens"] += len(it.tokens)
+
+    def close_fed(self, seq: Sequence) -> None:
+        """Give back what the sequence holds."""
+        self._finish(seq, FinishReason.STOP, publish=False)
+        self._finished_now.remove(seq)
+        self._by_req.pop(seq.req.request_id, None)
 
     # ------------------------------------------------------------------ planning
     def plan(self) -> Optional[StepPlan]:

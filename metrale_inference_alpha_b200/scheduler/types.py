@@ -98,6 +98,7 @@ class SeqStep:
     start_pos: int
     sample: bool = True          # produce a token from the last row
     verify: int = 0              # number of trailing draft tokens (rows that need logits)
+    want: Optional[List[int]] = None   # fed sequences: the rows (places among `tokens`) whose logits are asked for
 
 
 @dataclass

@@ -147,6 +147,9 @@ def build_parser() -> argparse.ArgumentParser:
     ml.add_argument("--cache-dir", default=None)
     ml.add_argument("--json", action="store_true")
 
+    from ..engine import replay
+    replay.add_arguments(sub.add_parser("replay", help="feed a trace of token ids through a model (steps on standard input) and write logits"))
+
     d = sub.add_parser("doctor", help="report device, driver and library state")
     d.add_argument("--json", action="store_true")
 
@@ -444,6 +447,9 @@ def main(argv: Optional[List[str]] = None) -> int:
             for r in rows:
                 print(f"{r['repo']:50s} {(r['revision'] or '-')[:12]:12s} {r['bytes'] / 2**30:8.2f} GiB  "
                       f"{'ok' if r['complete'] else 'incomplete'}")
+    elif ns.cmd == "replay":
+        from ..engine.replay import run
+        return run(ns)
     elif ns.cmd == "doctor":
         rep = doctor()
         print(json.dumps(rep, indent=None if ns.json else 2))

@@ -50,7 +50,7 @@ def test_activation_precision_switch_and_engine_runs_a16_on_cpu():
     try:
         eng = LLMEngine(EngineArgs(model="tiny-dense", device="cpu", max_num_seqs=2, max_model_len=128,
                                    activation_precision="a16"))
-        assert set(ops.ACT_FOR_WEIGHT.values()) == {"bf16"}
+        assert {v for k, v in ops.ACT_FOR_WEIGHT.items() if k != "fp32"} == {"bf16"}      # 32-bit models keep 32-bit activations
         out = eng.generate([[5, 6, 7, 8]], SamplingParams(max_tokens=6))[0].output_ids
         assert len(out) == 6
     finally:
