@@ -412,7 +412,46 @@ class _LinearAttnArgs(C.Structure):
                 ("num_slots", C.c_int), ("write_state", C.c_int), ("write_out", C.c_int), ("status", C.c_void_p)]
 
 
+class _LinearChunkedArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("q_ld", C.c_longlong), ("k_ld", C.c_longlong),
+                ("v_ld", C.c_longlong), ("H", C.c_int), ("DK", C.c_int), ("DV", C.c_int), ("total_rows", C.c_int), ("log_w", C.c_void_p),
+                ("decay", C.c_void_p), ("u", C.c_void_p), ("state", C.c_void_p), ("out", C.c_void_p), ("ws", C.c_void_p),
+                ("ws_bytes", C.c_size_t), ("q_start", C.c_void_p), ("q_len", C.c_void_p), ("positions", C.c_void_p),
+                ("slots", C.c_void_p), ("num_seqs", C.c_int), ("num_slots", C.c_int), ("max_q_len", C.c_int),
+                ("write_state", C.c_int), ("status", C.c_void_p)]
+
+
 _native.register_optional("mb_linear_attn", [C.POINTER(_LinearAttnArgs), C.c_void_p])
+_native.register_optional("mb_linear_chunked", [C.POINTER(_LinearChunkedArgs), C.c_void_p])
+_CHUNK_MIN_TOKENS = 48           # portions at least this long take the chunked kernels
+_CHUNK_WS_MAX = 4 << 30
+_chunk_ws: dict = {}
+
+
+def _linear_chunked(q, k, v, state, batch, H, dk, dv, log_w, decay, u, write_state):
+    """Chunked kernels (csrc/linear_chunked.cu); None for shapes, layouts or sizes they do not take."""
+    if dk not in (64, 128) or dv not in (64, 128) or q.dtype != torch.bfloat16 or (log_w is None) != (u is None):
+        return None
+    if any(t.data_ptr() % 16 or t.stride(0) % 8 for t in (q, k, v)):
+        return None
+    L, dev, T, S = _native.lib(), q.device, q.shape[0], batch.q_len.numel()
+    L.mb_linear_chunked_ws_bytes.restype, L.mb_linear_chunked_ws_bytes.argtypes = C.c_size_t, [C.c_int] * 5
+    need = int(L.mb_linear_chunked_ws_bytes(T, S, H, dk, dv))
+    if need > _CHUNK_WS_MAX:
+        return None
+    ws = _chunk_ws.get(dev)
+    if ws is None or ws.numel() < need:
+        if torch.cuda.is_current_stream_capturing():
+            return None
+        ws = _chunk_ws[dev] = torch.empty(int(need * 1.25), dtype=torch.uint8, device=dev)
+    out = torch.empty(T, H * dv, dtype=torch.float32, device=dev)
+    a = _LinearChunkedArgs(_ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), H, dk, dv, T, _ptr(log_w), _ptr(decay),
+                           _ptr(u), _ptr(state), _ptr(out), _ptr(ws), ws.numel(), _ptr(batch.q_start), _ptr(batch.q_len),
+                           _ptr(batch.positions), _ptr(batch.state_slots), S, state.shape[0], int(batch.max_q_len), int(write_state),
+                           _ptr(runtime(dev).status))
+    _native.check(L.mb_linear_chunked(C.byref(a), _stream()), f"linear_chunked[T={T} H={H}]")
+    _count(3)
+    return out
 
 
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, *, heads: int, dk: int, dv: int,
@@ -421,7 +460,8 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
                      kernel: str = "auto") -> Optional[torch.Tensor]:
     """Per head S_t = diag(w_t) S_(t-1) + k_t v_t^T over a ragged batch; w_t = ``decay`` [H], or exp(``log_w``
     [T, H dk]). Output q_t^T S_t, or with ``u`` [H, dk] q_t^T (S_(t-1) + diag(u) k_t v_t^T). q, k, v [T, *]
-    may be column ranges; state [slots, H, dk, dv] fp32. Returns fp32 [T, H dv]."""
+    may be column ranges; state [slots, H, dk, dv] fp32. Returns fp32 [T, H dv]. ``kernel``: auto | seq |
+    chunked (tests)."""
     T, H = q.shape[0], heads
     if not q.is_cuda:
         out = torch.zeros(T, H * dv, dtype=torch.float32)
@@ -444,6 +484,11 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
         return out if write_out else None
     assert q.dtype == k.dtype == v.dtype == DTYPE[fmt] and q.stride(1) == k.stride(1) == v.stride(1) == 1
     dev = q.device
+    if kernel == "chunked" or (kernel == "auto" and write_out and int(batch.max_q_len) >= _CHUNK_MIN_TOKENS):
+        out = _linear_chunked(q, k, v, state, batch, H, dk, dv, log_w, decay, u, write_state)
+        if out is not None:
+            return out
+        assert kernel == "auto", "the chunked kernels do not take this shape"
     out = torch.empty(T, H * dv, dtype=torch.float32, device=dev) if write_out else None
     a = _LinearAttnArgs(_ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), H, dk, dv, _f32(fmt), _ptr(log_w),
                         _ptr(decay), _ptr(u), _ptr(state), _ptr(out), _ptr(batch.q_start), _ptr(batch.q_len),

@@ -284,6 +284,41 @@ def test_linear_attention(device, fmt, dims, mode):
         close(state2[[1, 2, 3][s]], S, 2e-4)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dims", [(2, 64, 64), (3, 64, 128), (2, 128, 64), (5, 128, 128)])
+@pytest.mark.parametrize("mode", ["head", "channel+bonus"])
+def test_chunked_linear_attention(dims, mode):
+    """Chunk edges in every position, ragged batches, a state handed from chunk to chunk and portion to portion,
+    strong decays, keys that stand out just before and after chunk and sub-block edges."""
+    H, dk, dv = dims
+    lens = (333, 64, 65, 1, 16, 200)
+    qkv = [[b16(gen(n, H, d, seed=10 * i + n)) for i, d in enumerate((dk, dk, dv))] for n in lens]
+    q, k, v = qkv[0]
+    for i, j in ((64, 63), (63, 62), (128, 127), (129, 64), (80, 79), (79, 64), (17, 15), (332, 63), (331, 331), (200, 0)):
+        k[j] *= 6
+        q[i] = k[j]
+    decay = log_w = u = None
+    if mode == "head":
+        decay = torch.tensor([0.9995, 0.5, 0.97, 0.0, 1.0][:H])
+        ws = [decay.view(1, H, 1).expand(n, H, dk) for n in lens]
+    else:
+        log_w = [-torch.exp(gen(n, H, dk, seed=77 + n, std=2.0, mean=-3.0)).clamp(max=200.0) for n in lens]
+        for lw in log_w:
+            lw[..., 0], lw[..., 1] = -1e-4, -90.0
+            lw[30:90, :, 2] = -25.0
+        u = gen(H, dk, seed=5)
+        ws = [torch.exp(lw.double()) for lw in log_w]
+    cuts = [(100, 64, 65, 1, 0, 0), (64, 0, 0, 0, 16, 63), (1, 0, 0, 0, 0, 0), (168, 0, 0, 0, 0, 137)]
+    slots = [3, 1, 2, 6, 5, 4]
+    outs, state = run_linear("cuda", "bf16", qkv, log_w, decay, u, dims, cuts, slots, kernel="chunked")
+    for s, n in enumerate(lens):
+        want, S = plain_linear(*qkv[s], ws[s], u)
+        err = (outs[s].double() - want).abs().amax(2) / want.abs().amax(2).clamp(min=0.02 * float(want.abs().max()))
+        assert float(err.max()) < 3e-4, (s, float(err.max()), int(err.amax(1).argmax()))
+        close(state[slots[s]], S, 1e-4)
+    ops.check_status("cuda")
+
+
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("fmt", DTYPES)
 @pytest.mark.parametrize("group,act", [(24, "silu"), (72, "sigmoid"), (9, "silu")])
