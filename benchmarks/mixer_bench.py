@@ -135,7 +135,8 @@ def kernels(W=2560, H=20, G=4, D=128, FF=6912, R=64, side=128):
              lambda: ops.linear(act, w4), gb, gf)
         z, w2, w0 = rnd(T, R, dtype=torch.float32), rnd(HD, R, std=0.1), torch.zeros(HD, device=DEV)
         zb, w2q = mx.act_of(rnd(T, R), "bf16"), QuantWeight("bf16", HD, R, w2)
-        pair(shape, "log decay (32-bit low-rank)", lambda: mx.log_decay(z, w2, w0), T * HD * 4 + T * R * 4 + HD * R * 2, 0, "low-rank decay GEMM, bf16",
+        w2t = QuantWeight("bf16", HD, 2 * R, torch.cat([w2, w2], 1))
+        pair(shape, "log decay (32-bit low-rank)", lambda: mx.log_decay(z, w2, w0, w2t), T * HD * 4 + T * R * 4 + HD * R * 2, 0, "low-rank decay GEMM, bf16",
              lambda: ops.linear(zb, w2q, out_f32=True), T * HD * 4 + T * R * 2 + HD * R * 2, 0)
         ids, tab, zz = torch.randint(0, 60000, (T,), dtype=torch.int32, device=DEV), rnd(60000, side * 4), rnd(T, side, dtype=torch.float32)
         et = rnd(60000, W)

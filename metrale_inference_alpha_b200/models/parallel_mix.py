@@ -34,12 +34,11 @@ def parallel_block(dec, x, lw, batch, kv, j: int, pool, sidx: int):
                       out_scale=w.left_scale)
     # ---- right: time mixing
     r, k, v, g = mx.mix_projections(mixes, R, fmt)
-    log_w = mx.log_decay(ops.linear(mx.act_of(mixes[4], fmt), R.w1, out_f32=True), R.w2, R.w0)
-    core = mx.linear_attention(r, k, v, pool.ssm[sidx], batch, heads=R.heads, dk=R.dim, dv=R.dim, fmt=fmt, log_w=log_w, u=R.u,
-                               write_state=ws)
+    log_w = mx.log_decay(ops.linear(mx.act_of(mixes[4], fmt), R.w1, out_f32=True), R.w2, R.w0, R.w2_twice)
+    mx.linear_attention(r, k, v, pool.ssm[sidx], batch, heads=R.heads, dk=R.dim, dv=R.dim, fmt=fmt, log_w=log_w, u=R.u, write_state=ws,
+                        norm=dict(w=R.norm, gate=g, gate_act="silu", eps=c.rms_eps, scale=w.right_scale, out=cat[:, nl:]))
     if stash is not None:
         stash.layers[sidx] = ("parallel", lw, h32, (r, k, v), log_w)
-    mx.gated_norm(core, R.norm, g, fmt, group=R.dim, gate_act="silu", eps=c.rms_eps, scale=w.right_scale, out=cat[:, nl:])
     return x.add(ops.linear(mx.act_of(cat, fmt), w.o), lw.post_attn)
 
 

@@ -456,7 +456,7 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
            swiglu: bool = False, out_f32: bool = False, out: Optional[torch.Tensor] = None,
            force_tn: int = 0, force_splits: int = 0, one_tile_per_cta: bool = False, decode_tile_order: bool = False,
            dsmem_splitk: bool = False, grouped=None, no_cluster: bool = False, quant_out: float = 0.0,
-           clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0):
+           clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0, neg_exp_bias=None):
     """out[m, n] = sum_k act[m, k] * w[n, k] (+ residual); with `swiglu`, w holds gate/up rows
     interleaved (2j, 2j+1) and the result is silu(gate) * up of width N/2. `quant_out` > 0 (with
     `swiglu`): return the result as an NVFP4 `Act` quantised with that calibrated global scale --
@@ -466,7 +466,7 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     its partial tiles over distributed shared memory instead of the L2-resident workspace (all
     three for A/B comparisons and tests). `clamp_glu` = (alpha, limit): like `swiglu` with the gate
     g = min(gate, limit) and u = clamp(up, -limit, limit), result g * sigmoid(alpha g) * (u + 1).
-    `silu_cols`: SiLU on the first that many output columns. An fp32 weight gives fp32 outputs."""
+    `silu_cols`: SiLU on the first that many output columns. `neg_exp_bias` (CUDA, bf16): -exp(y + bias). An fp32 weight gives fp32 outputs."""
     assert act.K == w.K, (act.K, w.K)
     if w.fmt == "fp32" or (act.data.is_cuda and w.fmt == "bf16" and w.K % 8):
         # true 32-bit, or bf16 rows that are not whole 16-byte vectors (no tensor map can describe them)
@@ -523,6 +523,8 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         a.epilogue, a.epi_a, a.epi_b = EPI_CLAMP_GLU, clamp_glu[0], clamp_glu[1]
     elif silu_cols > 0:
         a.epilogue, a.epi_n = EPI_SILU_COLS, silu_cols
+    elif neg_exp_bias is not None:
+        a.epilogue, a.epi_bias = EPI_NEG_EXP, _ptr(neg_exp_bias)
     a.ws, a.ws_bytes, a.status = _ptr(rt.ws), rt.ws_bytes, _ptr(rt.status)
     a.force_tn, a.force_splits, a.sm_count = force_tn, force_splits, rt.sm_count
     a.flags = (_PERSIST_PREFILL | _GROUPED_CTAS | (GEMM_ONE_TILE_PER_CTA if one_tile_per_cta else 0)

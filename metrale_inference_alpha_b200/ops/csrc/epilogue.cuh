@@ -14,5 +14,10 @@ __device__ __forceinline__ float clamp_glu(float gate, float up, float alpha, fl
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   return g * sigmoid_exact(alpha * g) * (u + 1.f);
 }
+// the same with the approximate exponential and divide (a few ulp), for outputs that are rounded to bf16
+__device__ __forceinline__ float clamp_glu_fast(float gate, float up, float alpha, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return __fdividef(g * (u + 1.f), 1.f + __expf(-alpha * g));
+}
 
 }  // namespace mb

@@ -44,9 +44,11 @@ struct MbGemmArgs {
   const int* tile_row0;
   const int* tile_nrows;
   int n_per_expert, max_tiles;
-  // epilogue parameters: 2 = clamped GLU (epi_a sigmoid slope, epi_b limit), 3 = SiLU on columns below epi_n
+  // epilogue parameters: 2 = clamped GLU (epi_a sigmoid slope, epi_b limit), 3 = SiLU on columns below epi_n,
+  // 4 = -exp(y + epi_bias[n]) (3 and 4: bf16 operands)
   float epi_a, epi_b;
   int epi_n;
+  const float* epi_bias;
 };
 
 extern "C" int mb_gemm(const MbGemmArgs* args, cudaStream_t stream);

@@ -43,6 +43,7 @@ namespace {
 
 enum { KIND_BF16 = 0, KIND_FP8 = 1, KIND_NVFP4 = 2, KIND_FP8_BLOCK = 3 };
 using mb::EPI_CLAMP_GLU;
+using mb::EPI_NEG_EXP;
 using mb::EPI_PLAIN;
 using mb::EPI_SILU_COLS;
 using mb::EPI_SWIGLU;
@@ -64,6 +65,7 @@ struct GemmParams {
   int epilogue, out_f32;
   float epi_a, epi_b;     // EPI_CLAMP_GLU: sigmoid slope and clamp limit
   int epi_n;              // EPI_SILU_COLS: SiLU on output columns below this
+  const float* epi_bias;  // EPI_NEG_EXP: -exp(y + bias[n])
   uint32_t* status;
   // grouped (MoE) mode: blockIdx.y indexes a tile work-list; W is [experts * n_per_expert, K]
   const int* tile_expert;
@@ -445,7 +447,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         if (clamp_glu) {
 #pragma unroll
           for (int i = 0; i < 8; ++i)
-            y[i] = mb::clamp_glu(x[2 * i] * wcol[2 * i] * as, x[2 * i + 1] * wcol[2 * i + 1] * as, p.epi_a, p.epi_b);
+            y[i] = mb::clamp_glu_fast(x[2 * i] * wcol[2 * i] * as, x[2 * i + 1] * wcol[2 * i + 1] * as, p.epi_a, p.epi_b);
         } else if (swiglu) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = mb::silu(x[2 * i] * wcol[2 * i] * as) * (x[2 * i + 1] * wcol[2 * i + 1] * as);
@@ -456,6 +458,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
             for (int i = 0; i < 8; ++i)
               if (n_out0 + i < p.epi_n) y[i] = mb::silu(y[i]);
+          } else if (p.epilogue == EPI_NEG_EXP) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              if (n_out0 + i < n_out_limit) y[i] = -expf(y[i] + p.epi_bias[n_out0 + i]);
           }
         }
         const size_t o = (size_t)m * p.ldo + n_out0;
@@ -837,7 +843,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             const float x0 = v[j] * (wsc * as.x), x1 = v[j + 1] * (wsc * as.y);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
             const float gate = odd ? other : x0, up = odd ? x1 : other;
-            const float y = clamp_glu ? mb::clamp_glu(gate, up, p.epi_a, p.epi_b) : mb::silu(gate) * up;
+            const float y = clamp_glu ? mb::clamp_glu_fast(gate, up, p.epi_a, p.epi_b) : mb::silu(gate) * up;
             const int ml = m0 + (odd ? 1 : 0);                 // row inside the tile
             const int m = m_base + ml;
             if (p.outq) {
@@ -868,12 +874,21 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             }
           }
         } else {
+          if (p.epilogue == EPI_SILU_COLS) {
+            if (n < p.epi_n) {                                 // bf16 operands only: the scales below are 1
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = mb::silu(v[j] * wsc * asc[c * 16 + j]);
+            }
+          } else if (p.epilogue == EPI_NEG_EXP) {
+            const float bias = n < p.N ? p.epi_bias[n] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = -expf(v[j] * wsc * asc[c * 16 + j] + bias);
+          }
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int ml = c * 16 + j;
             if (ml < m_valid && n < p.N) {
               float y = v[j] * wsc * asc[ml];
-              if (p.epilogue == EPI_SILU_COLS && n < p.epi_n) y = mb::silu(y);
               const size_t o = (size_t)(m_base + ml) * p.ldo + n;
               if (p.residual) y += __bfloat162float(p.residual[o]);
               if (p.out_f32) reinterpret_cast<float*>(p.out)[o] = y;
@@ -979,7 +994,8 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   if (kind == KIND_NVFP4 && (!a->sfa || !a->sfb)) return MB_ERR_BAD_ARG;
   if (kind == KIND_FP8_BLOCK && (!a->w_scale || !a->a_scale)) return MB_ERR_BAD_ARG;
   if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
-  if (a->epilogue == EPI_SILU_COLS && a->residual) return MB_ERR_BAD_ARG;
+  if ((a->epilogue == EPI_SILU_COLS || a->epilogue == EPI_NEG_EXP) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
+  if (a->epilogue == EPI_NEG_EXP && !a->epi_bias) return MB_ERR_BAD_ARG;
   const int num_kb = (a->K + kelems - 1) / kelems;
   if (kind == KIND_NVFP4 && a->sf_k64 < num_kb * 4) return MB_ERR_BAD_ARG;
 
@@ -1037,7 +1053,7 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   p.sf_k64 = a->sf_k64;
   p.splits = splits; p.kb_per_split = kb_per; p.num_kb = num_kb;
   p.epilogue = a->epilogue; p.out_f32 = a->out_f32;
-  p.epi_a = a->epi_a; p.epi_b = a->epi_b; p.epi_n = a->epi_n;
+  p.epi_a = a->epi_a; p.epi_b = a->epi_b; p.epi_n = a->epi_n; p.epi_bias = a->epi_bias;
   p.status = a->status;
 #ifdef MB_GEMM_TIMING_EXPERIMENTS
   p.dbg = a->flags & 47;

@@ -13,7 +13,12 @@
 // key rows sit in one 64-bit register pair, so the update runs on the packed fp32 FMA. Producer warps load
 // and convert the next 16 tokens into the other half of a double buffer meanwhile (and compute each token's
 // bonus coefficient sum_i q_i u_i k_i), so the recurrence never waits on global memory.
+//
+// Steps of one token per sequence take linear_decode_kernel instead: one CTA per (sequence, head) streams the
+// state once, 16 rows of 16-byte vectors in flight per thread, and can finish the head's output itself (RMS over
+// the head, weight, gate, scale), so decode needs no separate norm launch.
 #include "common.cuh"
+#include "epilogue.cuh"
 
 namespace {
 
@@ -267,6 +272,118 @@ __global__ void __launch_bounds__(32 * (kNW + kPW)) linear_attn_kernel(const Lin
   }
 }
 
+// ------------------------------------------------------------------ one token per sequence
+struct DecodeNorm {
+  const bf16* w;                   // [H * DV] or null: no norm, fp32 output
+  const void* gate;
+  long long gate_ld;
+  int sigmoid_gate;
+  float eps, scale;
+  void* out;                       // row stride out_ld
+  long long out_ld;
+};
+
+constexpr int kDecRows = 16;       // state rows in flight per thread
+
+// QV threads cover the DV / 4 column vectors of a row; 256 / QV rows are in work side by side
+template <typename T, int QV, bool CH, bool BONUS>
+__global__ void __launch_bounds__(256, 2) linear_decode_kernel(const LinParams p, const DecodeNorm nm) {
+  constexpr int RG = 256 / QV;
+  __shared__ float sq[256], sk[256], sw[CH ? 256 : 1], so[RG * QV * 4], red[32];
+  const int hd = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  if (p.q_len[seq] <= 0) return;
+  const size_t t = (size_t)p.q_start[seq];
+  const int slot = p.slots[seq];
+  if (slot < 0 || slot >= p.num_slots) {
+    if (p.status && tid == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+    return;
+  }
+  const bool fresh = p.positions[t] == 0;
+  const int DK = p.DK, DV = p.DV, c4 = (tid % QV) * 4, rg = tid / QV;
+  const bool col_ok = c4 < DV;
+  float* st = p.state + ((size_t)slot * p.H + hd) * DK * DV + c4;
+  float4 s[kDecRows];
+  auto load = [&](int r0) {
+#pragma unroll
+    for (int i = 0; i < kDecRows; ++i) {
+      const int r = r0 + rg + i * RG;
+      s[i] = (!fresh && col_ok && r < DK) ? *reinterpret_cast<const float4*>(st + (size_t)r * DV) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  load(0);
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (col_ok) {
+    const size_t b = t * p.v_ld + (size_t)hd * DV + c4;
+    v = make_float4(ldx<T>(p.v, b), ldx<T>(p.v, b + 1), ldx<T>(p.v, b + 2), ldx<T>(p.v, b + 3));
+  }
+  float bonus = 0.f;
+  if (tid < DK) {
+    const float qv = ldx<T>(p.q, t * p.q_ld + (size_t)hd * DK + tid), kv = ldx<T>(p.k, t * p.k_ld + (size_t)hd * DK + tid);
+    sq[tid] = qv;
+    sk[tid] = kv;
+    if constexpr (CH) sw[tid] = expf(p.log_w[(t * p.H + hd) * DK + tid]);
+    if constexpr (BONUS) bonus = qv * p.u[hd * DK + tid] * kv;
+  }
+  if constexpr (BONUS) bonus = mb::block_sum(bonus, red);
+  __syncthreads();
+  const float wc = CH ? 0.f : p.decay[hd];
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int r0 = 0; r0 < DK; r0 += kDecRows * RG) {
+    if (r0 > 0) load(r0);
+#pragma unroll
+    for (int i = 0; i < kDecRows; ++i) {
+      const int r = r0 + rg + i * RG;
+      if (r < DK) {
+        const float q = sq[r], k = sk[r], w = CH ? sw[r] : wc;
+        float4 x = s[i];
+        if constexpr (BONUS) { o.x = fmaf(q, x.x, o.x); o.y = fmaf(q, x.y, o.y); o.z = fmaf(q, x.z, o.z); o.w = fmaf(q, x.w, o.w); }
+        x.x = fmaf(w, x.x, k * v.x); x.y = fmaf(w, x.y, k * v.y); x.z = fmaf(w, x.z, k * v.z); x.w = fmaf(w, x.w, k * v.w);
+        if constexpr (!BONUS) { o.x = fmaf(q, x.x, o.x); o.y = fmaf(q, x.y, o.y); o.z = fmaf(q, x.z, o.z); o.w = fmaf(q, x.w, o.w); }
+        if (p.write_state && col_ok) *reinterpret_cast<float4*>(st + (size_t)r * DV) = x;
+      }
+    }
+  }
+  if (!p.write_out) return;
+  *reinterpret_cast<float4*>(so + (rg * QV) * 4 + c4) = o;
+  __syncthreads();
+  float y = 0.f;
+  if (tid < DV) {
+#pragma unroll
+    for (int g = 0; g < RG; ++g) y += so[g * QV * 4 + tid];
+    if constexpr (BONUS) y = fmaf(bonus, ldx<T>(p.v, t * p.v_ld + (size_t)hd * DV + tid), y);
+  }
+  if (!nm.w) {
+    if (tid < DV) p.out[(t * p.H + hd) * DV + tid] = y;
+    return;
+  }
+  const float inv = rsqrtf(mb::block_sum(y * y, red) / (float)DV + nm.eps);
+  if (tid < DV) {
+    const int col = hd * DV + tid;
+    const float z = ldx<T>(nm.gate, t * nm.gate_ld + col);
+    const float a = nm.sigmoid_gate ? mb::sigmoid_exact(z) : mb::silu_exact(z);
+    const float r = y * inv * __bfloat162float(nm.w[col]) * a * nm.scale;
+    if constexpr (sizeof(T) == 2) reinterpret_cast<bf16*>(nm.out)[t * nm.out_ld + col] = __float2bfloat16(r);
+    else reinterpret_cast<float*>(nm.out)[t * nm.out_ld + col] = r;
+  }
+}
+
+template <typename T, bool CH, bool BONUS>
+int launch_decode(const LinParams& p, const DecodeNorm& nm, int num_seqs, cudaStream_t stream) {
+  const dim3 grid(p.H, num_seqs), block(256);
+  const int quads = p.DV / 4;
+  if (quads <= 8) return (int)mb::launch_kernel(linear_decode_kernel<T, 8, CH, BONUS>, grid, block, 0, stream, p, nm);
+  if (quads <= 16) return (int)mb::launch_kernel(linear_decode_kernel<T, 16, CH, BONUS>, grid, block, 0, stream, p, nm);
+  if (quads <= 32) return (int)mb::launch_kernel(linear_decode_kernel<T, 32, CH, BONUS>, grid, block, 0, stream, p, nm);
+  return (int)mb::launch_kernel(linear_decode_kernel<T, 64, CH, BONUS>, grid, block, 0, stream, p, nm);
+}
+template <typename T>
+int decode_mode(const LinParams& p, const DecodeNorm& nm, int num_seqs, cudaStream_t stream) {
+  if (p.log_w) return p.u ? launch_decode<T, true, true>(p, nm, num_seqs, stream) : launch_decode<T, true, false>(p, nm, num_seqs, stream);
+  return p.u ? launch_decode<T, false, true>(p, nm, num_seqs, stream) : launch_decode<T, false, false>(p, nm, num_seqs, stream);
+}
+
 template <typename T, int KG, bool CH, bool BONUS>
 int launch_k(const LinParams& p, int num_seqs, cudaStream_t stream) {
   constexpr size_t smem = lin_smem<KG, CH>();
@@ -314,13 +431,28 @@ struct MbLinearAttnArgs {
   const int* slots;
   int num_seqs, num_slots, write_state, write_out;
   uint32_t* status;
+  int decode;                // every sequence has at most one row: the streaming kernel (DV % 4 == 0, DK and DV <= 256)
+  const void* norm_w;        // decode: finish the head's output (RMS, weight, gate, scale) into norm_out
+  const void* gate;
+  long long gate_ld;
+  int sigmoid_gate;
+  float eps, scale;
+  void* norm_out;
+  long long norm_out_ld;
 };
 
 extern "C" int mb_linear_attn(const MbLinearAttnArgs* a, cudaStream_t stream) {
-  if (!a || !a->q || !a->k || !a->v || !a->state || (a->write_out && !a->out) || (!a->log_w && !a->decay)) return MB_ERR_BAD_ARG;
+  if (!a || !a->q || !a->k || !a->v || !a->state || (a->write_out && !a->out && !a->norm_w) || (!a->log_w && !a->decay)) return MB_ERR_BAD_ARG;
   if (a->H <= 0 || a->DK <= 0 || a->DV <= 0 || a->num_seqs <= 0 || a->num_seqs > 65535 || a->H > 65535) return MB_ERR_BAD_ARG;
   if (reinterpret_cast<uintptr_t>(a->state) % 16) return MB_ERR_BAD_ARG;
   LinParams p{a->q, a->k, a->v, a->q_ld, a->k_ld, a->v_ld, a->H, a->DK, a->DV, a->log_w, a->decay, a->u, a->state, a->out,
               a->q_start, a->q_len, a->positions, a->slots, a->num_slots, a->write_state, a->write_out, a->status};
+  if (a->decode) {
+    if (a->DV % 4 || a->DV > 256 || a->DK > 256) return MB_ERR_UNSUPPORTED;
+    if (a->norm_w && (!a->gate || !a->norm_out)) return MB_ERR_BAD_ARG;
+    const DecodeNorm nm{(const bf16*)a->norm_w, a->gate, a->gate_ld, a->sigmoid_gate, a->eps, a->scale, a->norm_out, a->norm_out_ld};
+    return a->f32 ? decode_mode<float>(p, nm, a->num_seqs, stream) : decode_mode<bf16>(p, nm, a->num_seqs, stream);
+  }
+  if (a->norm_w) return MB_ERR_UNSUPPORTED;
   return a->f32 ? launch_mode<float>(p, a->num_seqs, stream) : launch_mode<bf16>(p, a->num_seqs, stream);
 }

@@ -301,6 +301,19 @@ __global__ void __launch_bounds__(128) side_gate_kernel(const float* z, const in
   stv(out + i, g * e);
 }
 
+// tanh(z) as two bf16 terms side by side: out[t] = [value (R) | remainder (R)], the operand of a GEMM against [W | W]
+__global__ void __launch_bounds__(256) tanh_split_kernel(const float* z, bf16* out, long long total, int R) {
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const long long t = i / R, c = i - t * R;
+  const float v = tanhf(z[i]);
+  const bf16 h = __float2bfloat16(v);
+  out[t * 2 * R + c] = h;
+  out[t * 2 * R + R + c] = __float2bfloat16(v - __bfloat162float(h));
+}
+
 __global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, const bf16* table, float* out, int W, int vocab, float scale,
                                                            uint32_t* status) {
   mb::pdl_wait();
@@ -501,6 +514,12 @@ int mb_side_gate(const float* z, const int* tokens, const void* table, long long
 int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, uint32_t* status, cudaStream_t stream) {
   if (!tokens || !table || !out || M <= 0 || W <= 0) return MB_ERR_BAD_ARG;
   return (int)mb::launch_kernel(embed_scaled_kernel, dim3(M), dim3(256), 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status);
+}
+
+int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) {
+  if (!z || !out || T <= 0 || R <= 0) return MB_ERR_BAD_ARG;
+  const long long total = (long long)T * R;
+  return (int)mb::launch_kernel(tanh_split_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, z, (bf16*)out, total, R);
 }
 
 int mb_rope_dims(const MbRopeDimsArgs* a, cudaStream_t stream) {

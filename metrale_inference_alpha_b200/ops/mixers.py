@@ -409,7 +409,10 @@ class _LinearAttnArgs(C.Structure):
                 ("v_ld", C.c_longlong), ("H", C.c_int), ("DK", C.c_int), ("DV", C.c_int), ("f32", C.c_int), ("log_w", C.c_void_p),
                 ("decay", C.c_void_p), ("u", C.c_void_p), ("state", C.c_void_p), ("out", C.c_void_p), ("q_start", C.c_void_p),
                 ("q_len", C.c_void_p), ("positions", C.c_void_p), ("slots", C.c_void_p), ("num_seqs", C.c_int),
-                ("num_slots", C.c_int), ("write_state", C.c_int), ("write_out", C.c_int), ("status", C.c_void_p)]
+                ("num_slots", C.c_int), ("write_state", C.c_int), ("write_out", C.c_int), ("status", C.c_void_p),
+                ("decode", C.c_int), ("norm_w", C.c_void_p), ("gate", C.c_void_p), ("gate_ld", C.c_longlong),
+                ("sigmoid_gate", C.c_int), ("eps", C.c_float), ("scale", C.c_float), ("norm_out", C.c_void_p),
+                ("norm_out_ld", C.c_longlong)]
 
 
 class _LinearChunkedArgs(C.Structure):
@@ -454,15 +457,29 @@ def _linear_chunked(q, k, v, state, batch, H, dk, dv, log_w, decay, u, write_sta
     return out
 
 
+def _decode_ok(batch, dk: int, dv: int, kernel: str) -> bool:
+    """The streaming decode kernel: one row per sequence, whole 16-byte vectors, heads up to 256 x 256."""
+    return kernel in ("auto", "decode") and int(batch.max_q_len) == 1 and dv % 4 == 0 and max(dk, dv) <= 256
+
+
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, *, heads: int, dk: int, dv: int,
                      fmt: str, log_w: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None,
                      u: Optional[torch.Tensor] = None, write_state: bool = True, write_out: bool = True,
-                     kernel: str = "auto") -> Optional[torch.Tensor]:
+                     kernel: str = "auto", norm: Optional[dict] = None) -> Optional[torch.Tensor]:
     """Per head S_t = diag(w_t) S_(t-1) + k_t v_t^T over a ragged batch; w_t = ``decay`` [H], or exp(``log_w``
     [T, H dk]). Output q_t^T S_t, or with ``u`` [H, dk] q_t^T (S_(t-1) + diag(u) k_t v_t^T). q, k, v [T, *]
     may be column ranges; state [slots, H, dk, dv] fp32. Returns fp32 [T, H dv]. ``kernel``: auto | seq |
-    chunked (tests)."""
+    chunked | decode (tests). ``norm`` (keyword arguments of ``gated_norm`` with group = dv, and ``w``, ``gate``,
+    ``out``): the gated per-head norm of the output goes to norm["out"], inside the decode kernel where that
+    serves the step; nothing is returned then."""
     T, H = q.shape[0], heads
+    if norm is not None:
+        kw = dict(heads=H, dk=dk, dv=dv, fmt=fmt, log_w=log_w, decay=decay, u=u, write_state=write_state, kernel=kernel)
+        if not (q.is_cuda and _decode_ok(batch, dk, dv, kernel)):
+            core = linear_attention(q, k, v, state, batch, **kw)
+            gated_norm(core, norm["w"], norm["gate"], fmt, group=dv, gate_act=norm["gate_act"], eps=norm["eps"], scale=norm["scale"],
+                       out=norm["out"])
+            return None
     if not q.is_cuda:
         out = torch.zeros(T, H * dv, dtype=torch.float32)
         qs, ql, sl = batch.q_start.tolist(), batch.q_len.tolist(), batch.state_slots.tolist()
@@ -489,11 +506,17 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
         if out is not None:
             return out
         assert kernel == "auto", "the chunked kernels do not take this shape"
-    out = torch.empty(T, H * dv, dtype=torch.float32, device=dev) if write_out else None
+    out = torch.empty(T, H * dv, dtype=torch.float32, device=dev) if write_out and norm is None else None
     a = _LinearAttnArgs(_ptr(q), _ptr(k), _ptr(v), q.stride(0), k.stride(0), v.stride(0), H, dk, dv, _f32(fmt), _ptr(log_w),
                         _ptr(decay), _ptr(u), _ptr(state), _ptr(out), _ptr(batch.q_start), _ptr(batch.q_len),
                         _ptr(batch.positions), _ptr(batch.state_slots), batch.q_len.numel(), state.shape[0], int(write_state),
                         int(write_out), _ptr(runtime(dev).status))
+    a.decode = int(_decode_ok(batch, dk, dv, kernel))
+    if norm is not None:
+        g, o = norm["gate"], norm["out"]
+        assert g.stride(1) == 1 and o.stride(1) == 1 and g.dtype == o.dtype == DTYPE[fmt]
+        a.norm_w, a.gate, a.gate_ld, a.sigmoid_gate = _ptr(norm["w"]), _ptr(g), g.stride(0), int(norm["gate_act"] == "sigmoid")
+        a.eps, a.scale, a.norm_out, a.norm_out_ld = float(norm["eps"]), float(norm["scale"]), _ptr(o), o.stride(0)
     _native.check(_native.lib().mb_linear_attn(C.byref(a), _stream()), f"linear_attn[T={T} H={H}]")
     _count()
     return out
@@ -523,8 +546,20 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, tanh_in: b
     return out
 
 
-def log_decay(z: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor) -> torch.Tensor:
-    """-exp(tanh(z) w2^T + w0) in fp32: the logarithm of the decay exp(-exp(.)). z [T, rank] fp32."""
+_native.register_optional("mb_tanh_split", [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p])
+_DECAY_TC_MIN_ROWS = 256         # from here on the tensor cores, below the CUDA-core GEMM
+
+
+def log_decay(z: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, w2_twice=None) -> torch.Tensor:
+    """-exp(tanh(z) w2^T + w0) in fp32: the logarithm of the decay exp(-exp(.)). z [T, rank] fp32. ``w2_twice``
+    (bf16 QuantWeight [w2 | w2]): prefill-sized steps run it on the tensor cores, tanh(z) entering as two bf16 terms."""
+    if z.is_cuda and w2_twice is not None and z.shape[0] >= _DECAY_TC_MIN_ROWS:
+        from . import linear
+        T, R = z.shape
+        zs = torch.empty(T, 2 * R, dtype=torch.bfloat16, device=z.device)
+        _native.check(_native.lib().mb_tanh_split(_ptr(z), _ptr(zs), T, R, _stream()), "tanh_split")
+        _count()
+        return linear(act_of(zs, "bf16"), w2_twice, out_f32=True, neg_exp_bias=w0)
     if not z.is_cuda:
         return -torch.exp((torch.tanh(z).double() @ w2.double().t()).float() + w0)
     out = torch.empty(z.shape[0], w2.shape[0], dtype=torch.float32, device=z.device)

@@ -95,6 +95,8 @@ def load_fabulix(ld) -> ModelW:
         right = TimeMixW(mu=torch.stack([ld.vec(f"{q}.mu.{n}") for n in "rkvgw"]).contiguous(), w1=lin(f"{q}.w1"),
                          w2=ld.vec(f"{q}.w2"), w0=ld.vec(f"{q}.w0", torch.float32), u=ld.vec(f"{q}.u", torch.float32),
                          norm=ld.vec(f"{q}.norm"), heads=r["heads"], dim=r["dim"])
+        if fmt == "bf16" and right.w2.shape[1] % 4 == 0:
+            right.w2_twice = QuantWeight("bf16", right.w2.shape[0], 2 * right.w2.shape[1], torch.cat([right.w2, right.w2], 1).contiguous())
         if ops.mixers.grouped_ok(c.hidden_size, r["heads"] * r["dim"], fmt) and ld.dev.type == "cuda":
             right.rkvg_stack = lin(*(f"{q}.{n}" for n in "rkvg"))
         else:

@@ -215,6 +215,7 @@ class TimeMixW:
     rkvg: List[QuantWeight] = field(default_factory=list)
     w1: QuantWeight = None               # hidden -> rank
     w2: torch.Tensor = None              # [H D, rank], as stored
+    w2_twice: Optional[QuantWeight] = None   # [H D, 2 rank] = [w2 | w2]: the operand of a two-term tanh (bf16 models)
     w0: torch.Tensor = None              # fp32 [H D]
     u: torch.Tensor = None               # fp32 [H, D]
     norm: torch.Tensor = None            # bf16 [H D]

@@ -284,6 +284,34 @@ def test_linear_attention(device, fmt, dims, mode):
         close(state2[[1, 2, 3][s]], S, 2e-4)
 
 
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", DTYPES)
+@pytest.mark.parametrize("dims", [(3, 20, 28), (2, 64, 64), (2, 40, 96), (1, 128, 128), (2, 200, 160), (2, 16, 7)])
+@pytest.mark.parametrize("n", [1, 3])
+def test_linear_attention_with_its_norm(device, fmt, dims, n):
+    """The head norm, gate and scale behind the recurrence (inside the decode kernel for single rows): as separate steps."""
+    H, dk, dv = dims
+    T = 3 * n
+    q, k, v = (gen(T, H * d, seed=s).to(dt(fmt)).to(device) for d, s in ((dk, 1), (dk, 2), (dv, 3)))
+    lw, u = -torch.exp(gen(T, H * dk, seed=4)).to(device), gen(H, dk, seed=5).to(device)
+    gate, w = gen(T, H * dv, seed=6).to(dt(fmt)).to(device), b16(gen(H * dv, seed=7)).to(device)
+    b = fc.batch([n] * 3, [n, n + 4, n + 20], [2, 1, 3], device=device)
+    init = gen(4, H, dk, dv, seed=8).to(device)
+    init[2] = float("nan")                                             # a fresh sequence reads nothing from its slot
+    kw = dict(heads=H, dk=dk, dv=dv, fmt=fmt, log_w=lw, u=u)
+    s1, s2 = init.clone(), init.clone()
+    core = mx.linear_attention(q, k, v, s1, b, kernel="seq", **kw)
+    want = mx.gated_norm(core, w, gate, fmt, group=dv, gate_act="silu", eps=1e-5, scale=0.65)
+    out = torch.full((T, H * dv + 8), 3.0, dtype=dt(fmt), device=device)
+    mx.linear_attention(q, k, v, s2, b, norm=dict(w=w, gate=gate, gate_act="silu", eps=1e-5, scale=0.65, out=out[:, 8:]), **kw)
+    close(out[:, 8:], want.double().cpu(), 1e-5 if fmt == "fp32" else 8e-3)
+    assert bool((out[:, :8] == 3.0).all())
+    close(s2[1:], s1[1:].double().cpu(), 1e-5)
+    kw = dict(heads=H, dk=dk, dv=dv, fmt=fmt, decay=torch.full((H,), 0.9, device=device))      # no norm, read after the update
+    a, b2 = (mx.linear_attention(q, k, v, init.clone(), b, kernel=x, **kw) for x in ("seq", "auto"))
+    close(b2, a.double().cpu(), 1e-5)
+
+
 @pytest.mark.gpu
 @pytest.mark.parametrize("dims", [(2, 64, 64), (3, 64, 128), (2, 128, 64), (5, 128, 128)])
 @pytest.mark.parametrize("mode", ["head", "channel+bonus"])
@@ -357,6 +385,11 @@ def test_small_ops(device, fmt):
     z, w2, w0 = gen(9, 14, seed=1), b16(gen(50, 14, seed=2)), gen(50, seed=3, mean=-1)
     want = -torch.exp(torch.tanh(z.double()) @ w2.double().T + w0.double())
     close(mx.log_decay(z.to(device), w2.to(device), w0.to(device)), want, 1e-5)
+    z, w2 = gen(300, 16, seed=1), b16(gen(136, 16, seed=2))
+    w0 = gen(136, seed=3, mean=-1)
+    want = -torch.exp(torch.tanh(z.double()) @ w2.double().T + w0.double())
+    got = mx.log_decay(z.to(device), w2.to(device), w0.to(device), QuantWeight("bf16", 136, 32, torch.cat([w2, w2], 1).to(device)))
+    assert float(((got.double().cpu() - want) / want).abs().max()) < 1e-4
     tab, ids = b16(gen(20, 36, seed=4)), torch.tensor([3, 19, 0, 7], dtype=torch.int32)
     zz = gen(4, 12, seed=5, std=2.0)
     close(mx.side_gate(zz.to(device), ids.to(device), tab.to(device), 24, fmt), fo.gelu_tanh(zz.double()) * tab[ids.long(), 24:].double(),
