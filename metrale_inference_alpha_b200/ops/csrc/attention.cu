@@ -390,6 +390,7 @@ struct TileLoader {
 //     output columns (undone when O is written).
 template <int ROWB>
 __device__ __forceinline__ uint32_t raw_off(int row, int chunk) {
+  if constexpr (ROWB == 64) return (uint32_t)(row * ROWB + ((chunk ^ ((row >> 1) & 3)) << 4));   // two rows per 128-byte line
   return (uint32_t)(row * ROWB + ((chunk ^ (row & 7)) << 4));
 }
 // two e4m3 bytes -> f16x2 (exact). lo16 / hi16 take the low / high half of a 32-bit word,

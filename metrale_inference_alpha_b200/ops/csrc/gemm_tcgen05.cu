@@ -454,14 +454,21 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = x[i] * wcol[i] * as;
+          // whole vectors at a time: eight independent chains, no branch per element
           if (p.epilogue == EPI_SILU_COLS) {
+            if (n_out0 + 8 <= p.epi_n) {
 #pragma unroll
-            for (int i = 0; i < 8; ++i)
-              if (n_out0 + i < p.epi_n) y[i] = mb::silu(y[i]);
+              for (int i = 0; i < 8; ++i) y[i] = mb::silu(y[i]);
+            } else if (n_out0 < p.epi_n) {
+#pragma unroll
+              for (int i = 0; i < 8; ++i) y[i] = n_out0 + i < p.epi_n ? mb::silu(y[i]) : y[i];
+            }
           } else if (p.epilogue == EPI_NEG_EXP) {
+            float eb[8];
 #pragma unroll
-            for (int i = 0; i < 8; ++i)
-              if (n_out0 + i < n_out_limit) y[i] = -expf(y[i] + p.epi_bias[n_out0 + i]);
+            for (int i = 0; i < 8; ++i) eb[i] = n_out0 + i < n_out_limit ? __ldg(p.epi_bias + n_out0 + i) : 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[i] = -expf(y[i] + eb[i]);
           }
         }
         const size_t o = (size_t)m * p.ldo + n_out0;
@@ -797,6 +804,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
     const bool clamp_glu = p.epilogue == EPI_CLAMP_GLU;
     mb::pdl_wait();
     const int f = q * 32 + lane;                          // weight row of this thread inside a tile
+    const bool pair_ok = !p.out_f32 && !p.residual && !(p.N & 1) && !(p.ldo & 1) && (reinterpret_cast<uintptr_t>(p.out) & 3) == 0;
     const float outq_inv6gs = p.outq ? 1.f / (6.f * p.outq_gs) : 0.f;
     bool ok = true;
     for (int it = 0; it < my_tiles && ok; ++it) {
@@ -884,6 +892,22 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = -expf(v[j] * wsc * asc[c * 16 + j] + bias);
           }
+          if (pair_ok) {
+            // neighbouring lanes hold neighbouring output columns: per pair of tokens the even lane stores both
+            // columns of token j, the odd one of token j + 1, so every store is a full 4-byte word
+            const bool odd = lane & 1;
+            __nv_bfloat16* outp = reinterpret_cast<__nv_bfloat16*>(p.out) + (n & ~1);
+#pragma unroll
+            for (int j = 0; j < 16; j += 2) {
+              const int m0 = c * 16 + j;
+              const float2 as = *reinterpret_cast<const float2*>(&asc[m0]);
+              const float x0 = v[j] * wsc * as.x, x1 = v[j + 1] * wsc * as.y;
+              const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
+              const int ml = m0 + (odd ? 1 : 0);
+              if (ml < m_valid && n < p.N)
+                *reinterpret_cast<__nv_bfloat162*>(outp + (size_t)(m_base + ml) * p.ldo) = __floats2bfloat162_rn(odd ? other : x0, odd ? x1 : other);
+            }
+          } else {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int ml = c * 16 + j;
@@ -894,6 +918,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
               if (p.out_f32) reinterpret_cast<float*>(p.out)[o] = y;
               else reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16(y);
             }
+          }
           }
         }
       }

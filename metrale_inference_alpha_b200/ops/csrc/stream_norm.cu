@@ -281,24 +281,30 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedParams p) {
 }
 
 // ------------------------------------------------------------------ token side input
-template <typename T>
-__global__ void __launch_bounds__(128) side_gate_kernel(const float* z, const int* tokens, const bf16* table, long long table_ld, int off,
+template <int VEC, typename T>
+__global__ void __launch_bounds__(256) side_gate_kernel(const float* z, const int* tokens, const bf16* table, long long table_ld, int off,
                                                         int dim, int rows, int num_rows, T* out, uint32_t* status) {
   mb::pdl_wait();
   mb::pdl_launch_dependents();
-  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= (long long)rows * dim) return;
-  const int t = (int)(i / dim), c = (int)(i - (long long)t * dim);
+  const unsigned i = blockIdx.x * blockDim.x + threadIdx.x;            // one vector of one row
+  const unsigned per = (unsigned)(dim / VEC), t = i / per, c = (i - t * per) * VEC;
+  if (t >= (unsigned)rows) return;
   const int tok = tokens[t];
-  float e = 0.f;
+  float e[VEC], v[VEC], o[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) e[j] = 0.f;
   if (tok < 0 || tok >= num_rows) {
     if (status) atomicCAS(status, 0u, MB_ST_BOUNDS);
   } else {
-    e = __bfloat162float(table[(size_t)tok * table_ld + off + c]);
+    ldn<VEC>(table + (size_t)tok * table_ld + off + c, e);
   }
-  const float v = z[i];
-  const float g = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));   // sqrt(2 / pi)
-  stv(out + i, g * e);
+  ldn<VEC>(z + (size_t)t * dim + c, v);
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    const float x = v[j];
+    o[j] = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x))) * e[j];   // sqrt(2 / pi)
+  }
+  stn<VEC>(out + (size_t)t * dim + c, o);
 }
 
 // tanh(z) as two bf16 terms side by side: out[t] = [value (R) | remainder (R)], the operand of a GEMM against [W | W]
@@ -314,6 +320,7 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float* z, bf16* o
   out[t * 2 * R + R + c] = __float2bfloat16(v - __bfloat162float(h));
 }
 
+template <int VEC>
 __global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, const bf16* table, float* out, int W, int vocab, float scale,
                                                            uint32_t* status) {
   mb::pdl_wait();
@@ -321,8 +328,15 @@ __global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, co
   const int t = blockIdx.x, tok = tokens[t];
   const bool ok = tok >= 0 && tok < vocab;
   if (!ok && status && threadIdx.x == 0) atomicCAS(status, 0u, MB_ST_BOUNDS);
-  for (int k = threadIdx.x; k < W; k += blockDim.x)
-    out[(size_t)t * W + k] = ok ? __bfloat162float(table[(size_t)tok * W + k]) * scale : 0.f;
+  for (int k = threadIdx.x * VEC; k < W; k += blockDim.x * VEC) {
+    float v[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+    if (ok) ldn<VEC>(table + (size_t)tok * W + k, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] *= scale;
+    stn<VEC>(out + (size_t)t * W + k, v);
+  }
 }
 
 // ------------------------------------------------------------------ rotary + cache write, separate head sizes
@@ -506,14 +520,23 @@ int mb_gated_norm(const MbGatedNormArgs* a, cudaStream_t stream) {
 int mb_side_gate(const float* z, const int* tokens, const void* table, long long table_ld, int off, int dim, int rows, int num_rows, void* out,
                  int f32, uint32_t* status, cudaStream_t stream) {
   if (!z || !tokens || !table || !out || rows <= 0 || dim <= 0 || off < 0 || off + dim > table_ld) return MB_ERR_BAD_ARG;
-  const dim3 g((unsigned)(((long long)rows * dim + 127) / 128));
-  if (f32) return (int)mb::launch_kernel(side_gate_kernel<float>, g, dim3(128), 0, stream, z, tokens, (const bf16*)table, table_ld, off, dim, rows, num_rows, (float*)out, status);
-  return (int)mb::launch_kernel(side_gate_kernel<bf16>, g, dim3(128), 0, stream, z, tokens, (const bf16*)table, table_ld, off, dim, rows, num_rows, (bf16*)out, status);
+  if ((long long)rows * dim > (1ll << 31)) return MB_ERR_TOO_LARGE;
+  const bool v4 = dim % 4 == 0 && off % 4 == 0 && table_ld % 4 == 0 && al(table, 8) && al(z, 16) && al(out, 16);
+  const long long n = (long long)rows * dim / (v4 ? 4 : 1);
+  const dim3 g((unsigned)((n + 255) / 256)), b(256);
+  const bf16* tb = (const bf16*)table;
+  if (f32) return (int)(v4 ? mb::launch_kernel(side_gate_kernel<4, float>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (float*)out, status)
+                           : mb::launch_kernel(side_gate_kernel<1, float>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (float*)out, status));
+  return (int)(v4 ? mb::launch_kernel(side_gate_kernel<4, bf16>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (bf16*)out, status)
+                  : mb::launch_kernel(side_gate_kernel<1, bf16>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (bf16*)out, status));
 }
 
 int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, uint32_t* status, cudaStream_t stream) {
   if (!tokens || !table || !out || M <= 0 || W <= 0) return MB_ERR_BAD_ARG;
-  return (int)mb::launch_kernel(embed_scaled_kernel, dim3(M), dim3(256), 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status);
+  const bool v4 = W % 4 == 0 && al(table, 8) && al(out, 16);
+  const dim3 g(M), b(row_threads(W, v4 ? 4 : 1));
+  return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4>, g, b, 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status)
+                  : mb::launch_kernel(embed_scaled_kernel<1>, g, b, 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status));
 }
 
 int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) {

@@ -479,6 +479,12 @@ def test_attention_decode_gqa5_d128(fp8):
 
 
 @pytest.mark.parametrize("fp8", [False, True])
+def test_attention_decode_d64(fp8):
+    """Head dim 64: an e4m3 cache row is 64 bytes, half a shared-memory line."""
+    _attn_case(fp8, 64, 8, 2, [1, 1, 1, 3], [1, 17, 640, 1153])
+
+
+@pytest.mark.parametrize("fp8", [False, True])
 def test_attention_verify_rows(fp8):
     _attn_case(fp8, 128, 40, 8, [5, 5, 3], [133, 700, 64])       # 25 rows: two m16 tiles
     _attn_case(fp8, 64, 4, 2, [1, 4, 2], [33, 100, 2])
