@@ -27,6 +27,8 @@ What is measured (all as the max over ranks; rank 0 prints ONE JSON line):
            the sampled ids (and the kernels' status word) device -> host. `e2e.k_steps` is the
            same K steps as `value`, driven through `step()`.
   config.ladder   the same end-to-end measurement for every rung 1..128 (`--no-ladder` skips it).
+
+`--mixers` runs another workload instead: the Fabulix decoder beside an equal-size hybrid.
 """
 from __future__ import annotations
 
@@ -173,9 +175,20 @@ def main() -> int:
     ap.add_argument("--parallelism", default="tp", choices=["dp", "tp", "ep"],
                     help="N>1: tp = one engine sharded over N GPUs, C requests in total (strong scaling, the "
                          "configuration's TP sweep); dp = one engine replica per GPU, each serving C requests")
+    ap.add_argument("--mixers", default="", choices=["", "all", "kernels", "models"],
+                    help="instead of the headline run: the Fabulix decoder's kernels beside the like kernels of an equal-size "
+                         "attention / Kimi-delta hybrid, and both models' prefill and decode throughput (1 GPU; benchmarks/mixer_bench.py)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.mixers:
+        from benchmarks.mixer_bench import run as mixer_run
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = mixer_run(args.mixers)
+        print(json.dumps({"bench": "mixers", "l2": "flushed before every call", "dtype": "bf16", "data": "random weights and inputs",
+                          **res, "clocks": sampler.stop()}), flush=True)
+        return 0
     if args.warmup < 3:
         args.warmup = 3
 
