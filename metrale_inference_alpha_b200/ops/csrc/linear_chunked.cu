@@ -95,18 +95,25 @@ __device__ __forceinline__ void stage_rows(bf16 (*dst)[D + 8], const bf16* src, 
     cp16(&dst[r][c * 8], src + (ok ? (size_t)r * ld + c * 8 : 0), ok);
   }
 }
-// running sums of log2 decays over the chunk's tokens, one thread per channel; rows past `valid` repeat the last
+// running sums of log2 decays over the chunk's tokens; rows past `valid` repeat the last. All 256 threads: 256 / D
+// groups of rows side by side, joined through each group's last row. Ends with a barrier.
 template <int D>
 __device__ __forceinline__ void running_logs(float (*sL)[D + 4], const float* lw, size_t ld, int valid) {
-  const int d = threadIdx.x;
-  if (d < D) {
-    float acc = 0.f;
-#pragma unroll 8
-    for (int r = 0; r < kC; ++r) {
-      if (r < valid) acc += fmaxf(lw[(size_t)r * ld + d] * kLog2e, kMinLog);
-      sL[r][d] = acc;
-    }
-  }
+  constexpr int kR = kC * D / 256;
+  const int d = threadIdx.x % D, grp = threadIdx.x / D, r0 = grp * kR;
+  float v[kR];
+#pragma unroll
+  for (int i = 0; i < kR; ++i) v[i] = r0 + i < valid ? fmaxf(lw[(size_t)(r0 + i) * ld + d] * kLog2e, kMinLog) : 0.f;
+#pragma unroll
+  for (int i = 1; i < kR; ++i) v[i] += v[i - 1];
+  sL[r0 + kR - 1][d] = v[kR - 1];
+  __syncthreads();
+  float before = 0.f;
+  for (int g = 0; g < grp; ++g) before += sL[g * kR + kR - 1][d];
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < kR; ++i) sL[r0 + i][d] = before + v[i];
+  __syncthreads();
 }
 
 // ------------------------------------------------------------------ a chunk's contribution to the state
@@ -221,12 +228,17 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const ChunkParams p) {
 }
 
 // ------------------------------------------------------------------ outputs of a chunk
+// The scores are built first, from q, k and the logs. Then the decayed queries replace q and k (value and remainder)
+// and the logs' space takes the start state, 64 key rows at a time: 105 KB at 128 x 128, two CTAs per SM, so that one
+// CTA's loads run under the other's products.
 template <int DK, int DV>
 struct OutSmem {
   bf16 q[kC][DK + 8], k[kC][DK + 8], v[kC][DV + 8];
-  bf16 sh[DK][DV + 8], sl[DK][DV + 8];              // start state, value and remainder
-  bf16 ah[kC][kC + 8], al[kC][kC + 8];              // scores
-  float L[kC][DK + 4];                              // per-channel mode: decays of each step, then their running logs
+  bf16 ah[kC][kC + 8], al[kC][kC + 8];              // scores, value and remainder
+  union {
+    float L[kC][DK + 4];                            // per-channel mode: decays of each step, then their running logs
+    struct { bf16 h[64][DV + 8], l[64][DV + 8]; } st;
+  };
 };
 
 // sum over the 32 lanes of each of 16 values; lane l returns value l & 15
@@ -246,7 +258,7 @@ __device__ __forceinline__ float reduce16(float (&v)[16], int lane) {
 }
 
 template <int DK, int DV, bool CH>
-__global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) uint8_t raw[];
   auto& s = *reinterpret_cast<OutSmem<DK, DV>*>(raw);
   const int c = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
@@ -260,13 +272,17 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
   stage_rows<DK>(s.k, p.k + (size_t)t0 * p.k_ld + (size_t)hd * DK, p.k_ld, valid);
   asm volatile("cp.async.commit_group;" ::: "memory");
   stage_rows<DV>(s.v, p.v + (size_t)t0 * p.v_ld + (size_t)hd * DV, p.v_ld, valid);
-  const bf16 *gh = p.ws_hi + ci * (DK * DV), *gl = p.ws_lo + ci * (DK * DV);
-  for (int i = tid; i < DK * (DV / 8); i += 256) {
-    const int r = i / (DV / 8), cc = (i - r * (DV / 8)) * 8;
-    cp16(&s.sh[r][cc], gh + r * DV + cc, true);
-    cp16(&s.sl[r][cc], gl + r * DV + cc, true);
-  }
   asm volatile("cp.async.commit_group;" ::: "memory");
+  const bf16 *gh = p.ws_hi + ci * (DK * DV), *gl = p.ws_lo + ci * (DK * DV);
+  auto stage_state = [&](int row0) {
+    for (int i = tid; i < 64 * (DV / 8); i += 256) {
+      const int r = i / (DV / 8), cc = (i - r * (DV / 8)) * 8;
+      cp16(&s.st.h[r][cc], gh + (row0 + r) * DV + cc, true);
+      cp16(&s.st.l[r][cc], gl + (row0 + r) * DV + cc, true);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if constexpr (!CH) stage_state(0);                                  // nothing else needs that space
   const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int rb = warp & 3, half = warp >> 2, i0 = rb * 16;            // this warp's 16 tokens and column half
   const float ld2 = CH ? 0.f : head_log(p.decay[hd]);
@@ -278,7 +294,7 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
       s.L[r][d] = r < valid ? ex2(lw[(size_t)r * p.H * DK + d] * kLog2e) : 1.f;
     }
   }
-  asm volatile("cp.async.wait_group 1;" ::: "memory");
+  asm volatile("cp.async.wait_group %0;" ::"n"(CH ? 1 : 2) : "memory");
   __syncthreads();
   if constexpr (CH) {
     // ---- diagonal blocks: key j times the decays of the steps between j and i, multiplied up step by step
@@ -315,9 +331,8 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
     }
     __syncthreads();
     running_logs<DK>(s.L, lw, (size_t)p.H * DK, valid);
-    __syncthreads();
   }
-  // decayed query fragments of this warp's rows: q_i 2^(L_(i-1) - ref), value and remainder
+  // query fragments of this warp's rows decayed from the reference on: q_i 2^(L_(i-1) - ref), value and remainder
   auto q_frag = [&](int k0, const float* refL, uint32_t* hi, uint32_t* lo) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -328,10 +343,8 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
         la = s.L[i - 1][d];
         lb = s.L[i - 1][d + 1];
       }
-      if (refL) {
-        la -= refL[d];
-        lb -= refL[d + 1];
-      }
+      la -= refL[d];
+      lb -= refL[d + 1];
       split2(qv.x * ex2(la), qv.y * ex2(lb), hi[e], lo[e]);
     }
   };
@@ -406,8 +419,22 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
         }
       }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  __syncthreads();
+  // ---- per-channel mode: q and k become the queries decayed from the chunk's start, value and remainder
+  if constexpr (CH) {
+    __syncthreads();
+    for (int i = tid; i < kC * (DK / 2); i += 256) {
+      const int r = i / (DK / 2), d = (i - r * (DK / 2)) * 2;
+      const float2 qv = bf2(&s.q[r][d]);
+      float la = 0.f, lb = 0.f;
+      if (r > 0) {
+        la = s.L[r - 1][d];
+        lb = s.L[r - 1][d + 1];
+      }
+      split2(qv.x * ex2(la), qv.y * ex2(lb), *reinterpret_cast<uint32_t*>(&s.q[r][d]), *reinterpret_cast<uint32_t*>(&s.k[r][d]));
+    }
+    __syncthreads();
+    stage_state(0);
+  }
   // ---- o = (decayed q) S + A V for 16 rows and DV / 2 columns
   constexpr int kN = DV / 16;
   const int n0 = half * (DV / 2);
@@ -416,24 +443,33 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkParams p) {
   for (int i = 0; i < kN; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-  for (int k0 = 0; k0 < DK; k0 += 16) {
-    uint32_t hi[4], lo[4];
-    if constexpr (CH) q_frag(k0, nullptr, hi, lo);
-    else ldsm4(hi, &s.q[i0 + (lane & 15)][k0 + (lane >> 4) * 8]);
+  for (int row0 = 0; row0 < DK; row0 += 64) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
 #pragma unroll
-    for (int i = 0; i < kN; i += 2) {
-      uint32_t bh[4], bl[4];
-      const int r = k0 + (lane & 15), cc = n0 + i * 8 + (lane >> 4) * 8;
-      ldsm4t(bh, &s.sh[r][cc]);
-      ldsm4t(bl, &s.sl[r][cc]);
-      mma(o[i], hi, bh[0], bh[1]);
-      mma(o[i], hi, bl[0], bl[1]);
-      mma(o[i + 1], hi, bh[2], bh[3]);
-      mma(o[i + 1], hi, bl[2], bl[3]);
-      if constexpr (CH) {
-        mma(o[i], lo, bh[0], bh[1]);
-        mma(o[i + 1], lo, bh[2], bh[3]);
+    for (int kk = 0; kk < 64; kk += 16) {
+      uint32_t hi[4], lo[4];
+      ldsm4(hi, &s.q[i0 + (lane & 15)][row0 + kk + (lane >> 4) * 8]);
+      if constexpr (CH) ldsm4(lo, &s.k[i0 + (lane & 15)][row0 + kk + (lane >> 4) * 8]);
+#pragma unroll
+      for (int i = 0; i < kN; i += 2) {
+        uint32_t bh[4], bl[4];
+        const int r = kk + (lane & 15), cc = n0 + i * 8 + (lane >> 4) * 8;
+        ldsm4t(bh, &s.st.h[r][cc]);
+        ldsm4t(bl, &s.st.l[r][cc]);
+        mma(o[i], hi, bh[0], bh[1]);
+        mma(o[i + 1], hi, bh[2], bh[3]);
+        mma(o[i], hi, bl[0], bl[1]);
+        mma(o[i + 1], hi, bl[2], bl[3]);
+        if constexpr (CH) {
+          mma(o[i], lo, bh[0], bh[1]);
+          mma(o[i + 1], lo, bh[2], bh[3]);
+        }
       }
+    }
+    if (row0 + 64 < DK) {
+      __syncthreads();
+      stage_state(row0 + 64);
     }
   }
   if constexpr (!CH) {
@@ -469,7 +505,7 @@ template <int DK, int DV, bool CH>
 int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
   using SS = StateSmem<DK, DV>;
   using SO = OutSmem<DK, DV>;
-  const size_t ss = CH ? sizeof(SS) : offsetof(SS, L), so = CH ? sizeof(SO) : offsetof(SO, L);
+  const size_t ss = CH ? sizeof(SS) : offsetof(SS, L), so = sizeof(SO);
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(chunk_state_kernel<DK, DV, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
