@@ -542,6 +542,24 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
     const uint32_t sK = sbase + (it % kStages) * C::kStageB, sV = sK + kTileK;
     const int tok0 = tok_begin + it * kTile;
     const int blk0 = (tok0 - tok_begin) >> bs_shift;
+    if constexpr (kRowK == kRowV) {
+      if (ck.lin) {                                            // one block lookup and one offset for both tiles
+#pragma unroll
+        for (int i = 0; i < TileCopy<kRowK>::kCopies; ++i) {
+          constexpr int kStep = TileCopy<kRowK>::kStep;
+          const bool valid = tok0 + ck.r0 + i * kStep < tok_end;
+          const int blk = valid ? s_blk[blk0 + ck.bsel0 + i * ck.bstep] : 0;
+          const size_t off = (size_t)blk * ck.blk_pitch + ck.gbase;
+          const int sz = valid ? 16 : 0;
+          const uint32_t so = ck.soff0 + (uint32_t)(i * kStep * kRowK);
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + so),
+                       "l"(reinterpret_cast<const uint8_t*>(p.k_cache) + off), "r"(sz) : "memory");
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + so),
+                       "l"(reinterpret_cast<const uint8_t*>(p.v_cache) + off), "r"(sz) : "memory");
+        }
+        return;
+      }
+    }
     if (ck.lin) issue_lin(ck, tok0, blk0, sK, kRowK);
     else issue_any(ck, tok0, blk0, sK, std::integral_constant<int, kRowK>{});
     if (cv.lin) issue_lin(cv, tok0, blk0, sV, kRowV);

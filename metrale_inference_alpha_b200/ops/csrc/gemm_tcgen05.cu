@@ -317,8 +317,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
     float* s_tile = reinterpret_cast<float*>(smem);
     bool ok = true;
-    const bool swiglu = p.epilogue == EPI_SWIGLU || p.epilogue == EPI_CLAMP_GLU;   // paired (gate, up) columns
-    const bool clamp_glu = p.epilogue == EPI_CLAMP_GLU;
+    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU);   // paired (gate, up) columns
+    const bool clamp_glu = KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU;      // bf16 models only
     mb::pdl_wait();                                        // first global access of these warps follows
     // per-token scales of this tile, staged while the main loop runs
     for (int j = et; j < TN; j += 128) {
@@ -455,7 +455,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = x[i] * wcol[i] * as;
           // whole vectors at a time: eight independent chains, no branch per element
-          if (p.epilogue == EPI_SILU_COLS) {
+          if (KIND == KIND_BF16 && p.epilogue == EPI_SILU_COLS) {
             if (n_out0 + 8 <= p.epi_n) {
 #pragma unroll
               for (int i = 0; i < 8; ++i) y[i] = mb::silu(y[i]);
@@ -463,7 +463,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
               for (int i = 0; i < 8; ++i) y[i] = n_out0 + i < p.epi_n ? mb::silu(y[i]) : y[i];
             }
-          } else if (p.epilogue == EPI_NEG_EXP) {
+          } else if (KIND == KIND_BF16 && p.epilogue == EPI_NEG_EXP) {
             float eb[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) eb[i] = n_out0 + i < n_out_limit ? __ldg(p.epi_bias + n_out0 + i) : 0.f;
@@ -800,11 +800,10 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
     const int lane = threadIdx.x & 31;
     const int et = threadIdx.x - 64;
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
-    const bool swiglu = p.epilogue == EPI_SWIGLU || p.epilogue == EPI_CLAMP_GLU;   // paired (gate, up) columns
-    const bool clamp_glu = p.epilogue == EPI_CLAMP_GLU;
+    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU);   // paired (gate, up) columns
+    const bool clamp_glu = KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU;      // bf16 models only
     mb::pdl_wait();
     const int f = q * 32 + lane;                          // weight row of this thread inside a tile
-    const bool pair_ok = !p.out_f32 && !p.residual && !(p.N & 1) && !(p.ldo & 1) && (reinterpret_cast<uintptr_t>(p.out) & 3) == 0;
     const float outq_inv6gs = p.outq ? 1.f / (6.f * p.outq_gs) : 0.f;
     bool ok = true;
     for (int it = 0; it < my_tiles && ok; ++it) {
@@ -882,32 +881,16 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             }
           }
         } else {
-          if (p.epilogue == EPI_SILU_COLS) {
+          if (KIND == KIND_BF16 && p.epilogue == EPI_SILU_COLS) {
             if (n < p.epi_n) {                                 // bf16 operands only: the scales below are 1
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] = mb::silu(v[j] * wsc * asc[c * 16 + j]);
             }
-          } else if (p.epilogue == EPI_NEG_EXP) {
+          } else if (KIND == KIND_BF16 && p.epilogue == EPI_NEG_EXP) {
             const float bias = n < p.N ? p.epi_bias[n] : 0.f;
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = -expf(v[j] * wsc * asc[c * 16 + j] + bias);
           }
-          if (pair_ok) {
-            // neighbouring lanes hold neighbouring output columns: per pair of tokens the even lane stores both
-            // columns of token j, the odd one of token j + 1, so every store is a full 4-byte word
-            const bool odd = lane & 1;
-            __nv_bfloat16* outp = reinterpret_cast<__nv_bfloat16*>(p.out) + (n & ~1);
-#pragma unroll
-            for (int j = 0; j < 16; j += 2) {
-              const int m0 = c * 16 + j;
-              const float2 as = *reinterpret_cast<const float2*>(&asc[m0]);
-              const float x0 = v[j] * wsc * as.x, x1 = v[j + 1] * wsc * as.y;
-              const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
-              const int ml = m0 + (odd ? 1 : 0);
-              if (ml < m_valid && n < p.N)
-                *reinterpret_cast<__nv_bfloat162*>(outp + (size_t)(m_base + ml) * p.ldo) = __floats2bfloat162_rn(odd ? other : x0, odd ? x1 : other);
-            }
-          } else {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int ml = c * 16 + j;
@@ -918,7 +901,6 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
               if (p.out_f32) reinterpret_cast<float*>(p.out)[o] = y;
               else reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16(y);
             }
-          }
           }
         }
       }
@@ -1021,6 +1003,7 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
   if ((a->epilogue == EPI_SILU_COLS || a->epilogue == EPI_NEG_EXP) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
   if (a->epilogue == EPI_NEG_EXP && !a->epi_bias) return MB_ERR_BAD_ARG;
+  if (a->epilogue == EPI_CLAMP_GLU && kind != KIND_BF16) return MB_ERR_UNSUPPORTED;
   const int num_kb = (a->K + kelems - 1) / kelems;
   if (kind == KIND_NVFP4 && a->sf_k64 < num_kb * 4) return MB_ERR_BAD_ARG;
 
