@@ -17,16 +17,16 @@ from typing import List, Optional
 
 WEIGHT_FORMATS = ("bf16", "nvfp4", "fp8_block", "fp8_row", "fp32")
 KV_DTYPES = ("bf16", "fp8", "fp32")
-LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning")
-KV_KINDS = ("attention", "mla", "parallel")                       # kinds that own a KV pool
-STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning")   # kinds that own a recurrent state
+LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning", "latent", "gla")
+KV_KINDS = ("attention", "mla", "parallel", "latent")                    # kinds that own a KV pool
+STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning", "gla")   # kinds that own a recurrent state
 FFN_KINDS = ("dense", "moe", "none")
 
 
 @dataclass
 class ModelConfig:
     name: str = "model"
-    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix
+    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix | finelix
     vocab_size: int = 4096
     hidden_size: int = 256
     num_layers: int = 2
@@ -61,8 +61,9 @@ class ModelConfig:
     residual_multiplier: float = 1.0    # Granite: a block's output is scaled by this before it joins the stream
     logits_divisor: float = 1.0         # Granite: logits are divided by this
     tie_embeddings: bool = False
-    # fabulix: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
+    # fabulix, finelix: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
     layer_specs: List[dict] = field(default_factory=list)
+    loop: Optional[dict] = None         # layers start .. stop - 1 run `times` times with the same weights: {"start", "stop", "times"}
     token_side_dim: int = 0             # width of a layer's slice of the token side embedding (0 = none)
     glu_alpha: float = 1.702            # sigmoid slope of the clamped GLU
     # per-layer structure
@@ -168,19 +169,39 @@ class ModelConfig:
         return [i for i, t in enumerate(self.layer_types) if t in KV_KINDS]
 
     @property
+    def stream32(self) -> bool:
+        """The residual stream is kept in 32-bit, and the layers' sizes are per layer (``layer_specs``)."""
+        return self.arch in ("fabulix", "finelix")
+
+    def layer_runs(self) -> List[tuple]:
+        """(layer, pass) of every layer run in order. A looped layer appears once per pass, and each of its runs
+        has a cache or state of its own; `pass` is given on the first run of a pass only, else None."""
+        lo, hi, times = (self.loop["start"], self.loop["stop"], self.loop["times"]) if self.loop else (0, 0, 0)
+        if times == 0:
+            return [(i, None) for i in range(self.num_layers)]
+        return ([(i, None) for i in range(lo)]
+                + [(i, t if i == lo else None) for t in range(times) for i in range(lo, hi)]
+                + [(i, None) for i in range(hi, self.num_layers)])
+
+    @property
     def act_fmt(self) -> str:
         """Activation type of models with a 32-bit residual stream: bf16, or fp32 when served in 32-bit."""
         return "fp32" if self.weight_format == "fp32" else "bf16"
 
     def kv_layer_dims(self) -> List[tuple]:
-        """(kv heads, K row, V row) of every KV pool of a model whose layers have their own head sizes; the
-        rows are padded to what the attention kernels tile."""
+        """(kv heads, K row, V row) of every KV pool (one per layer run) of a model whose layers have their own head
+        sizes; the rows are padded to what the attention kernels tile. Latent layers cache one row per token
+        that serves as key and value."""
+        from ..ops.latent import latent_row
         from ..ops.mixers import padded_head_dims
         out = []
-        for t, sp in zip(self.layer_types, self.layer_specs):
+        for i, _ in self.layer_runs() if self.layer_specs else ():
+            t, m = self.layer_types[i], self.layer_specs[i]["mixer"]
             if t == "parallel":
-                m = sp["mixer"]["left"]
+                m = m["left"]
                 out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
+            elif t == "latent":
+                out.append((1, latent_row(m["kv_rank"], m["rot_dim"], self.act_fmt).row, 0))
         return out
 
     def kv_bytes_per_token(self) -> int:
@@ -197,9 +218,9 @@ class ModelConfig:
     def param_count(self) -> int:
         """Approximate parameter count (linear layers + embeddings)."""
         h = self.hidden_size
-        if self.arch == "fabulix":
-            from ..weights.fabulix import tensor_shapes
-            return sum(math.prod(s) for s, _ in tensor_shapes(self).values())
+        if self.stream32:
+            from ..weights.source import spec_shapes
+            return sum(math.prod(s) for s, _ in spec_shapes(self).values())
         n = self.vocab_size * h * (1 if self.tie_embeddings else 2)
         for lt, ft in zip(self.layer_types, self.ffn_types):
             if lt == "attention":
@@ -391,8 +412,51 @@ def fabulix_3b(**kw) -> ModelConfig:
     return fabulix(**base)
 
 
+def finelix(num_layers: int = 6, width: int = 256, heads: int = 4, dim: int = 48, rot_dim: int = 16, vdim: int = 40, kv_rank: int = 96,
+            q_rank: int = 80, rot_base: float = 10000.0, lin_heads: int = 4, lin_dim: int = 64, lin_vdim: int = 64, tau: float = 16.0,
+            ff: int = 512, experts: int = 8, top: int = 2, expert_ff: int = 96, shared_ff: int = 160, vocab: int = 1024, period: int = 2,
+            loop: Optional[dict] = None, eps: float = 1e-5, **kw) -> ModelConfig:
+    """Finelix decoder of uniform layers: every `period`-th layer is latent attention beside a mixture of
+    experts, the others gated linear attention beside a dense feed-forward; `loop` repeats a range of layers."""
+    layers = []
+    for i in range(num_layers):
+        if i % period == period - 1:
+            m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank,
+                 "scale": (dim + rot_dim) ** -0.5, "rot": {"base": rot_base, "dims": rot_dim}}
+            mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+            if shared_ff:
+                mlp["shared"] = {"ff": shared_ff}
+            layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+        else:
+            m = {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "tau": tau}
+            layers.append({"type": "gla", "mixer": m, "mlp": {"kind": "dense", "ff": ff}})
+    cfg = {"architecture": "Finelix", "vocab": vocab, "width": width, "embedding": {"scale": float(width) ** 0.5},
+           "norm": {"eps": eps}, "layers": layers}
+    if loop:
+        cfg["loop"] = dict(loop)
+    return from_finelix_config(cfg, name=kw.pop("name", "finelix")).scaled(**kw)
+
+
+def tiny_finelix(**kw) -> ModelConfig:
+    """Six-layer Finelix with a looped range (tests, smoke runs)."""
+    return finelix(**{"name": "tiny-finelix", "loop": {"start": 1, "stop": 3, "times": 2}, **kw})
+
+
+def finelix_3b(**kw) -> ModelConfig:
+    """Finelix with the layer sizes of a ~3B-active model: width 2560, latent attention of 32 heads (128 + 64, value
+    128, latent 512, query latent 1536) beside 64 experts of 1024, top 6, and a shared one; gated linear attention
+    of 20 heads of 128 beside a feed-forward of 6912; 24 layers, the first two run three times."""
+    base = dict(name="finelix-3b", num_layers=24, width=2560, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536,
+                lin_heads=20, lin_dim=128, lin_vdim=128, ff=6912, experts=64, top=6, expert_ff=1024, shared_ff=2048, vocab=65536,
+                loop={"start": 0, "stop": 2, "times": 3})
+    base.update(kw)
+    return finelix(**base)
+
+
 PRESETS = {
     "tiny-dense": tiny_dense,
+    "tiny-finelix": tiny_finelix,
+    "finelix-3b": finelix_3b,
     "tiny-fabulix": tiny_fabulix,
     "fabulix-3b": fabulix_3b,
     "tiny-kimi-linear": tiny_kimi_linear,
@@ -479,10 +543,52 @@ def from_fabulix_config(cfg: dict, name: str = "model") -> ModelConfig:
         token_side_dim=int((cfg.get("token_side") or {}).get("dim", 0)), max_position=131072)
 
 
+_FINELIX_MIXERS = {"latent_attention": "latent", "gla": "gla", "gla_2": "gla"}
+
+
+def from_finelix_config(cfg: dict, name: str = "model") -> ModelConfig:
+    """A Finelix ``config.json``: sizes and constants are given per layer and kept per layer, `loop` names the
+    range of layers that runs several times. Mixer types and feed-forward kinds this engine does not know are
+    refused."""
+    types, ffns, specs = [], [], []
+    for i, L in enumerate(cfg["layers"]):
+        t, m, mlp = L["type"], L["mixer"], L.get("mlp")
+        if t not in _FINELIX_MIXERS:
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+        if mlp is not None and mlp.get("kind") not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        if _FINELIX_MIXERS[t] == "latent":
+            if m["rot_dim"] % 2 or m["rot"]["dims"] != m["rot_dim"]:
+                raise ValueError(f"layer {i}: the rotary size is not the rotated part's")
+        elif not m["tau"] > 0:
+            raise ValueError(f"layer {i}: tau must be positive")
+        if mlp is not None and mlp["kind"] == "moe" and not 0 < mlp["router"]["top"] <= min(32, mlp["router"]["experts"]):
+            raise ValueError(f"layer {i}: {mlp['router']['top']} of {mlp['router']['experts']} experts per token")
+        types.append(_FINELIX_MIXERS[t])
+        ffns.append("none" if mlp is None else mlp["kind"])
+        specs.append({"mixer": m, "mlp": mlp})
+    loop = cfg.get("loop") or None
+    if loop is not None:
+        loop = {k: int(loop[k]) for k in ("start", "stop", "times")}
+        if not (0 <= loop["start"] < loop["stop"] <= len(types) and loop["times"] > 0):
+            raise ValueError(f"loop {loop} does not fit {len(types)} layers")
+    att = next((s["mixer"] for t, s in zip(types, specs) if t == "latent"), {"heads": 1, "dim": 64, "rot_dim": 0})
+    moe = next((s["mlp"] for f, s in zip(ffns, specs) if f == "moe"), None)
+    return ModelConfig(
+        name=name, arch="finelix", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(types), layer_types=types,
+        ffn_types=ffns, layer_specs=specs, loop=loop, num_heads=att["heads"], num_kv_heads=att["heads"], head_dim=att["dim"] + att["rot_dim"],
+        rotary_dim=-1, rms_eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), tie_embeddings=False,
+        intermediate_size=max((s["mlp"]["ff"] for s, f in zip(specs, ffns) if f == "dense"), default=0),
+        num_experts=moe["router"]["experts"] if moe else 0, experts_per_token=moe["router"]["top"] if moe else 0,
+        moe_intermediate_size=moe["expert"]["ff"] if moe else 0, max_position=131072)
+
+
 def from_hf_config(cfg: dict, name: str = "model") -> ModelConfig:
     """Map a HF ``config.json`` dict (text stack) to ModelConfig; refuses unknown model types."""
     if cfg.get("architecture") == "Fabulix":
         return from_fabulix_config(cfg, name)
+    if cfg.get("architecture") == "Finelix":
+        return from_finelix_config(cfg, name)
     outer = cfg
     if "text_config" in cfg:
         inner = dict(cfg["text_config"])

@@ -33,7 +33,7 @@ from .runner import ModelRunner, plan_kv_blocks
 class EngineArgs:
     model: Union[str, ModelConfig] = "tiny-dense"     # preset name, checkpoint dir, or a config
     device: str = "cpu"
-    dtype: str = "auto"                                # auto (the model's) | bf16 | fp32 (true 32-bit: Fabulix models)
+    dtype: str = "auto"                                # auto (the model's) | bf16 | fp32 (true 32-bit: Fabulix and Finelix models)
     seed: int = 0
     max_num_seqs: int = 128
     max_model_len: int = 2048
@@ -120,13 +120,15 @@ class LLMEngine:
         if args.dtype != "auto":
             if args.dtype not in ("bf16", "fp32"):
                 raise ValueError(f"dtype must be auto | bf16 | fp32, not {args.dtype!r}")
-            if cfg.arch == "fabulix":
+            if cfg.stream32:
                 cfg = cfg.scaled(weight_format=args.dtype, kv_dtype=args.dtype)
             elif args.dtype == "fp32" or cfg.weight_format != args.dtype:
                 raise ValueError(f"{cfg.name} is served in {cfg.weight_format}, not {args.dtype}")
-        if cfg.arch == "fabulix":
+        if cfg.stream32:
             if args.speculative in ("mtp", "dflash"):
-                raise NotImplementedError("Fabulix models speculate with n-grams and predicted outputs only")
+                raise NotImplementedError(f"{cfg.arch.capitalize()} models speculate with n-grams and predicted outputs only")
+            if args.expert_arena_slots > 0:
+                raise NotImplementedError(f"the experts of {cfg.arch.capitalize()} models stay on the device")
             if args.kv_cache_dtype not in ("auto", cfg.kv_dtype):
                 raise NotImplementedError(f"this model's KV cache is {cfg.kv_dtype}")
         if args.kv_cache_dtype not in ("auto", cfg.kv_dtype):
@@ -248,8 +250,8 @@ class LLMEngine:
         from ..lora import LoraAdapter, LoraManager
         if self.tp.size > 1:
             raise NotImplementedError("LoRA adapters are served on single-rank engines")
-        if self.cfg.arch == "fabulix":
-            raise NotImplementedError("LoRA adapters are not served on Fabulix models")
+        if self.cfg.stream32:
+            raise NotImplementedError(f"LoRA adapters are not served on {self.cfg.arch.capitalize()} models")
         dec, c = self.runner.decoder, self.cfg
         if dec.lora is None:
             D = c.head_dim

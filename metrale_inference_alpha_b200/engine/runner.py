@@ -30,9 +30,10 @@ from .batch import ForwardBatch
 
 
 def state_shapes(cfg: ModelConfig, w: ModelW):
-    """(conv window, ssm matrix) shapes of every recurrent layer, from the loaded (sharded) weights."""
+    """(conv window, ssm matrix) shapes of every run of a recurrent layer, from the loaded (sharded) weights."""
     out = []
-    for lw in w.layers:
+    for i, _ in cfg.layer_runs():
+        lw = w.layers[i]
         if lw.kind == "gdn":
             m = lw.mixer
             C = 2 * m.k_heads * cfg.gdn_k_dim + m.v_heads * cfg.gdn_v_dim
@@ -47,7 +48,7 @@ def state_shapes(cfg: ModelConfig, w: ModelW):
         elif lw.kind == "parallel":                # the token shift's window is the previous token's mixer input
             m = lw.mixer.right
             out.append(((cfg.hidden_size,), (m.heads, m.dim, m.dim)))
-        elif lw.kind == "lightning":
+        elif lw.kind in ("lightning", "gla"):
             m = lw.mixer
             out.append(((0,), (m.heads, m.dim, m.vdim)))
     return out
@@ -59,9 +60,10 @@ def kv_config(cfg: ModelConfig, w: ModelW, block_size: int, mtp: bool = False) -
         return KvCacheConfig(1 if mtp else len(cfg.attention_layers()), 1, cfg.kv_lora_rank + cfg.qk_rope_dim,
                              block_size, cfg.kv_dtype if cfg.kv_dtype == "bf16" else "bf16",
                              v_head_dim=cfg.index_head_dim if cfg.index_topk > 0 else None, has_v=cfg.index_topk > 0)
-    if cfg.arch == "fabulix":
+    if cfg.stream32:
         dims = tuple(cfg.kv_layer_dims()) or ((1, 16, 16),)      # a model without attention keeps a token-sized pool
-        return KvCacheConfig(len(dims), dims[0][0], dims[0][1], block_size, cfg.kv_dtype, layer_dims=dims)
+        return KvCacheConfig(len(dims), dims[0][0], dims[0][1], block_size, cfg.kv_dtype, layer_dims=dims,
+                             has_v=any(dv for _, _, dv in dims))         # latent rows are keys and values at once
     kvh = cfg.num_kv_heads
     for lw in ([w.mtp.layer] if (mtp and w.mtp) else w.layers):
         if lw.kind == "attention":

@@ -33,12 +33,13 @@ class LayerCaches:
         self.kv, self.state, self.mtp_kv = kv, state, mtp_kv
         self.kv_index, self.state_index = {}, {}
         a = s = 0
-        for i, t in enumerate(cfg.layer_types):
+        for run, (i, _) in enumerate(cfg.layer_runs()):       # keyed by layer run: the layer itself where nothing loops
+            t = cfg.layer_types[i]
             if t in KV_KINDS:
-                self.kv_index[i] = a
+                self.kv_index[run] = a
                 a += 1
             if t in STATE_KINDS:
-                self.state_index[i] = s
+                self.state_index[run] = s
                 s += 1
 
 
@@ -104,7 +105,7 @@ class Decoder:
         the norm kernel performs the sum (+ residual) itself; afterwards ``self.res(x)`` is the
         summed stream. `res_only`: the caller uses that stream only as the residual of the next
         row-parallel projection, so each rank may keep just its own row share."""
-        if isinstance(w, mixers.DytNorm):
+        if isinstance(w, (mixers.DytNorm, mixers.RmsNorm)):
             s = x if isinstance(x, ResidualStream) else ResidualStream(x, self.cfg.act_fmt)
             return mixers.act_of(s.norm(w), s.fmt)
         if hasattr(x, "resolve"):
@@ -283,7 +284,11 @@ class Decoder:
         from .moe import moe_block
         return moe_block(self, x, lw)
 
-    def layer(self, i: int, x, lw: LayerW, batch: ForwardBatch, caches: LayerCaches, kv=None, kv_idx=None):
+    def layer(self, i: int, x, lw: LayerW, batch: ForwardBatch, caches: LayerCaches, kv=None, kv_idx=None, run: Optional[int] = None):
+        """`run`: which cache and state this run of the layer has (the layer's own unless it is looped)."""
+        if lw.out is not None:
+            from .joint import joint_layer
+            return joint_layer(self, x, lw, batch, caches, i if run is None else run)
         if lw.kind == "attention":
             kv = kv or caches.kv
             j = caches.kv_index[i] if kv_idx is None else kv_idx
@@ -328,8 +333,12 @@ class Decoder:
 
     # ------------------------------------------------------------------ full forward
     def embed(self, token_ids: torch.Tensor) -> torch.Tensor:
-        if self.cfg.arch == "fabulix":             # 32-bit residual stream
-            return ResidualStream(mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale), self.cfg.act_fmt)
+        if self.cfg.stream32:
+            fmt, pair, W = self.cfg.act_fmt, None, self.cfg.hidden_size
+            if self.w.loop_in is not None:
+                pair = torch.empty(token_ids.numel(), 2 * W, dtype=mixers.DTYPE[fmt], device=self.w.embed.device)
+            x = mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale, None if pair is None else pair[:, W:])
+            return ResidualStream(x, fmt, pair)
         x = ops.embed(token_ids, self.w.embed)
         if self.cfg.embed_scale != 1.0:
             x = x * torch.tensor(self.cfg.embed_scale, dtype=torch.bfloat16).to(x.dtype)
@@ -346,8 +355,10 @@ class Decoder:
             side.begin(x.shape[0])
         if self.cfg.hc_mult > 1:
             return self._backbone_highway(x, batch, caches)
-        for i, lw in enumerate(self.w.layers):
-            x = self.layer(i, x, lw, batch, caches)
+        for run, (i, step) in enumerate(self.cfg.layer_runs()):
+            if step is not None:
+                x.enter_pass(self.w.loop_in, self.w.loop_step[step])
+            x = self.layer(i, x, self.w.layers[i], batch, caches, run=run)
             if side is not None and i in side.capture_ids:
                 x = self.full(x)
                 side.capture(i, x)

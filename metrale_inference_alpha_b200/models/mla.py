@@ -1,4 +1,4 @@
-"""Multi-head latent attention block (DeepSeek-V3 shape) in absorbed form.
+"""Multi-head latent attention (DeepSeek-V3 shape; and with per-layer sizes, ``latent_mixer``) in absorbed form.
 
 The paged cache stores one row per token: ``[kv_lora latent (RMS-normed) | rope key]``
 (kv_lora + rope dims, a single "kv head"). Queries are projected into latent space with
@@ -19,7 +19,8 @@ import math
 import torch
 
 from .. import ops
-from ..ops import ACT_FOR_WEIGHT, mla_cuda, sparse_attn
+from ..ops import ACT_FOR_WEIGHT, latent, mla_cuda, sparse_attn
+from ..ops.mixers import act_of
 from ..ops import reference as ref
 
 
@@ -89,6 +90,21 @@ def mla_block(dec, x, lw, batch, kv, j: int):
     o = torch.einsum("thl,hvl->thv", o_lat, w.w_uv.float()).reshape(T, H * vd)
     oa = ops.quantize_act(o.to(torch.bfloat16), ACT_FOR_WEIGHT[w.o.fmt])
     return dec.tp.linear_reduce(oa, w.o, residual=x, defer=True)
+
+
+def latent_mixer(dec, a, w, batch, cache, fmt: str, out):
+    """Latent attention of a layer with its own sizes, scale and rotation, on a normed input; the heads' values
+    go to ``out`` [T, H vdim]. Returns the columns of the input projection behind its own (a router's logits)."""
+    q_rank, L, R = w.q_rank, w.kv_rank, w.rot_dim
+    lay = latent.latent_row(L, R, fmt)
+    cos, sin = dec.rotary(R, w.rot_base)
+    x = ops.linear(a, w.in_proj, out_f32=True)                             # [T, q_rank | L | R | ...]
+    cq = latent.norm_and_cache(x, fmt, q_rank=q_rank, L=L, R=R, q_w=w.q_norm, kv_w=w.kv_norm, eps=dec.cfg.rms_eps, cos=cos, sin=sin,
+                               positions=batch.positions, slots=batch.slot_mapping, cache=cache, lay=lay)
+    q = ops.linear(act_of(cq, fmt), w.uq)
+    qq = latent.absorbed_query(q, w.w_uk, fmt, H=w.heads, dim=w.dim, R=R, cos=cos, sin=sin, positions=batch.positions, lay=lay)
+    latent.attention(qq, cache, batch, w.w_uv, w.scale, fmt, lay, out)
+    return x[:, q_rank + L + R:]
 
 
 def _index_select(dec, x, a, qn, w, batch, kv, j: int):

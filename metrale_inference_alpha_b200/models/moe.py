@@ -74,6 +74,17 @@ def moe_block(dec, x, lw):
     return (x.float() + y.float()).to(torch.bfloat16)
 
 
+def routed_rows(dec, a, logits, w):
+    """The routed experts' outputs before their sum (``ops.mixers.Routed``), for a stream that sums them itself."""
+    from ..ops.mixers import Routed
+    weights, idx = moe_ops.route(logits, w.spec, w.bias)
+    if not a.data.is_cuda:
+        return Routed(moe_ops.expert_sum_ref(a, weights, idx, w.grouped, dec.cfg.hidden_size), None, None)
+    from ..ops.moe_cuda import grouped_pairs
+    y, sp = grouped_pairs(w.spec, a, idx, w)
+    return Routed(y, sp.pair_row, weights)
+
+
 def shared_expert(dec, a, w):
     f = w.shared
     fmt_d = ACT_FOR_WEIGHT[f.down.fmt]

@@ -72,7 +72,7 @@ def commit(kind: str, lw, x_in, qkv, log_w, pool, sidx: int, cb) -> None:
     w = lw.mixer.right if kind == "parallel" else lw.mixer
     dv = w.dim if kind == "parallel" else w.vdim
     fmt = "fp32" if qkv[0].dtype == torch.float32 else "bf16"
-    kw = dict(log_w=log_w, u=w.u) if kind == "parallel" else dict(decay=w.decay)
+    kw = dict(log_w=log_w, u=w.u) if kind == "parallel" else dict(log_w=log_w) if kind == "gla" else dict(decay=w.decay)
     mx.linear_attention(*qkv, pool.ssm[sidx], cb, heads=w.heads, dk=w.dim, dv=dv, fmt=fmt, write_out=False, **kw)
     if kind == "parallel":
         mx.shift_commit(x_in, pool.conv[sidx], cb)

@@ -1,4 +1,5 @@
-"""Recurrent mixers: gated-delta-net (Qwen3.5 / 3.6 linear attention) and Mamba2 (Nemotron-H).
+"""Recurrent mixers: gated-delta-net (Qwen3.5 / 3.6 linear attention), Mamba2 (Nemotron-H), Kimi delta attention and
+gated linear attention.
 
 Both keep an fp32 state per sequence in the state pool (a conv window + a matrix) and
 process a batch whose sequences contribute any number of tokens (decode 1, verify k+1,
@@ -13,6 +14,7 @@ import torch
 
 from .. import ops
 from ..ops import ACT_FOR_WEIGHT
+from ..ops import mixers as mx
 from ..ops import recurrent as rops
 
 
@@ -64,6 +66,31 @@ def kda_block(dec, x, lw, batch, pool, sidx: int):
     return dec.tp.linear_reduce(ya, w.out, residual=x, defer=True)
 
 
+def gla_mixer(dec, a, lw, batch, pool, sidx: int, fmt: str, out) -> None:
+    """Gated linear attention on a normed input: q | k | v | g and the low-rank decay from one projection, matrix state
+    read after its update, RMS norm per head, SiLU gate; ``out`` [T, H vdim]. The queries' factor dim^-1/2 stands in
+    front of a norm, where it is the same as an eps of dim times the size."""
+    w = lw.mixer
+    H, dk, dv = w.heads, w.dim, w.vdim
+    y = ops.linear(a, w.in_proj)
+    q, k, v, g, a1 = (y[:, lo:hi] for lo, hi in _bounds(H * dk, H * dk, H * dv, H * dv, w.a2.shape[1]))
+    decay = mx.LowRankDecay(a1, w.a2, w.a2_bias, 1.0 / w.tau, w.a2_lin)
+    stash = getattr(batch, "spec_stash", None)
+    kw = dict(low_rank=decay)
+    if stash is not None:                                            # verify steps commit the state afterwards
+        kw = dict(log_w=decay.log())
+        stash.layers[sidx] = ("gla", lw, None, (q, k, v), kw["log_w"])
+    mx.linear_attention(q, k, v, pool.ssm[sidx], batch, heads=H, dk=dk, dv=dv, fmt=fmt, write_state=stash is None,
+                        norm=dict(w=w.norm, gate=g, gate_act="silu", eps=dec.cfg.rms_eps * dk, scale=1.0, out=out), **kw)
+
+
+def _bounds(*sizes):
+    at = 0
+    for n in sizes:
+        yield at, at + n
+        at += n
+
+
 def _tile(owner, w: torch.Tensor, n: int) -> torch.Tensor:
     """`w` repeated n times (the per-head norm weight laid out for all heads of a row), built once
     and kept on the layer's own weight object: a cache keyed by anything else (a device address,
@@ -103,7 +130,7 @@ def commit_recurrent(cfg, pool, stash, commit_batch) -> None:
     sequence (0 = leave the sequence's state as it was)."""
     for sidx, (kind, lw, x_in, conv_out, gate) in stash.layers.items():
         w = lw.mixer
-        if kind in ("parallel", "lightning"):
+        if kind in ("parallel", "lightning", "gla"):
             from .parallel_mix import commit
             commit(kind, lw, x_in, conv_out, gate, pool, sidx, commit_batch)
         elif kind == "gdn":

@@ -33,7 +33,7 @@ GEMM_ONE_TILE_PER_CTA, GEMM_DECODE_TILE_ORDER, GEMM_PERSISTENT_PREFILL, GEMM_DSM
 # measure 1.5x faster there; METRALE_PERSISTENT_PREFILL=0 keeps one tile per CTA)
 _PERSIST_PREFILL = GEMM_PERSISTENT_PREFILL if os.environ.get("METRALE_PERSISTENT_PREFILL", "1") != "0" else 0
 GEMM_GROUPED_ONE_CTA = 512
-EPI_CLAMP_GLU, EPI_SILU_COLS, EPI_NEG_EXP = 2, 3, 4      # csrc/epilogue.cuh
+EPI_SWIGLU, EPI_CLAMP_GLU, EPI_SILU_COLS, EPI_NEG_EXP, EPI_GEGLU, EPI_BIAS, EPI_LOG_SIGMOID = 1, 2, 3, 4, 5, 6, 7      # csrc/epilogue.cuh
 _GROUPED_CTAS = GEMM_GROUPED_ONE_CTA if os.environ.get("METRALE_GROUPED_CTAS", "2") == "1" else 0
 
 
@@ -424,7 +424,13 @@ def _linear_a16(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool,
     return out
 
 
-def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual):
+def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu=False, bias=None, log_sigmoid=None):
+    if geglu:
+        y = torch.nn.functional.gelu(y[:, 0::2], approximate="tanh") * y[:, 1::2]
+    elif bias is not None:
+        y = y + bias
+    elif log_sigmoid is not None:
+        y = log_sigmoid[1] * torch.nn.functional.logsigmoid(y + log_sigmoid[0])
     if clamp_glu is not None:
         alpha, limit = clamp_glu
         g, u = y[:, 0::2].clamp(max=limit), y[:, 1::2].clamp(-limit, limit)
@@ -436,19 +442,26 @@ def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual):
     return y if residual is None else y + residual.float()
 
 
-def _linear_simt(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool, out, clamp_glu, silu_cols: int):
+def _linear_simt(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool, out, clamp_glu, silu_cols: int, geglu=False, bias=None,
+                 log_sigmoid=None):
     """CUDA-core GEMM (csrc/gemm_simt.cu); on CPU its fp64-accumulated restatement."""
-    assert not swiglu and residual is None, "the CUDA-core GEMM has no SwiGLU or residual epilogue"
+    assert residual is None, "the CUDA-core GEMM has no residual epilogue"
     f32 = out_f32 or w.fmt == "fp32"
     if not act.data.is_cuda:
-        y = _linear_epilogue_ref((act.data.double() @ w.dequant64().t()).float(), False, clamp_glu, silu_cols, None)
+        y = _linear_epilogue_ref((act.data.double() @ w.dequant64().t()).float(), swiglu, clamp_glu, silu_cols, None, geglu, bias, log_sigmoid)
         y = y if f32 else y.to(torch.bfloat16)
         return y if out is None else out.copy_(y)
     from .mixers import gemm_simt
     if out is None:
-        out = torch.empty(act.M, w.N // 2 if clamp_glu else w.N, dtype=torch.float32 if f32 else torch.bfloat16, device=act.data.device)
+        out = torch.empty(act.M, w.N // 2 if clamp_glu or swiglu or geglu else w.N, dtype=torch.float32 if f32 else torch.bfloat16, device=act.data.device)
     if clamp_glu is not None:
         return gemm_simt(act.data, w.data, out, epilogue=EPI_CLAMP_GLU, epi_a=clamp_glu[0], epi_b=clamp_glu[1])
+    if swiglu or geglu:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_SWIGLU if swiglu else EPI_GEGLU)
+    if bias is not None:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_BIAS, bias=bias)
+    if log_sigmoid is not None:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_LOG_SIGMOID, bias=log_sigmoid[0], epi_a=log_sigmoid[1])
     return gemm_simt(act.data, w.data, out, epilogue=EPI_SILU_COLS if silu_cols else 0, epi_n=silu_cols)
 
 
@@ -456,7 +469,8 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
            swiglu: bool = False, out_f32: bool = False, out: Optional[torch.Tensor] = None,
            force_tn: int = 0, force_splits: int = 0, one_tile_per_cta: bool = False, decode_tile_order: bool = False,
            dsmem_splitk: bool = False, grouped=None, no_cluster: bool = False, quant_out: float = 0.0,
-           clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0, neg_exp_bias=None):
+           clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0, neg_exp_bias=None,
+           geglu: bool = False, bias: Optional[torch.Tensor] = None, log_sigmoid=None):
     """out[m, n] = sum_k act[m, k] * w[n, k] (+ residual); with `swiglu`, w holds gate/up rows
     interleaved (2j, 2j+1) and the result is silu(gate) * up of width N/2. `quant_out` > 0 (with
     `swiglu`): return the result as an NVFP4 `Act` quantised with that calibrated global scale --
@@ -466,11 +480,13 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     its partial tiles over distributed shared memory instead of the L2-resident workspace (all
     three for A/B comparisons and tests). `clamp_glu` = (alpha, limit): like `swiglu` with the gate
     g = min(gate, limit) and u = clamp(up, -limit, limit), result g * sigmoid(alpha g) * (u + 1).
-    `silu_cols`: SiLU on the first that many output columns. `neg_exp_bias` (CUDA, bf16): -exp(y + bias). An fp32 weight gives fp32 outputs."""
+    `silu_cols`: SiLU on the first that many output columns. `neg_exp_bias` (CUDA, bf16): -exp(y + bias). `geglu`: like
+    `swiglu` with gelu_tanh(gate) * up. `bias` (fp32 [N]): y + bias. `log_sigmoid` = (bias, c): c * log(sigmoid(y + bias)).
+    An fp32 weight gives fp32 outputs."""
     assert act.K == w.K, (act.K, w.K)
     if w.fmt == "fp32" or (act.data.is_cuda and w.fmt == "bf16" and w.K % 8):
         # true 32-bit, or bf16 rows that are not whole 16-byte vectors (no tensor map can describe them)
-        return _linear_simt(act, w, residual, swiglu, out_f32, out, clamp_glu, silu_cols)
+        return _linear_simt(act, w, residual, swiglu, out_f32, out, clamp_glu, silu_cols, geglu, bias, log_sigmoid)
     a16 = act.fmt == "bf16" and w.fmt != "bf16"
     assert a16 or act.fmt == NATIVE_ACT_FOR_WEIGHT[w.fmt], (act.fmt, w.fmt)
     M, N = act.M, w.N
@@ -491,11 +507,12 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         # (fp32 BLAS picks different blockings for different M, and a random-weight test model has
         # near-ties everywhere), so that batch-invariance tests on the CPU path are exact
         y = (act.data.double() @ w.dequant64().t()).float()
-        y = _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual)
-        return y if out_f32 else y.to(torch.bfloat16)
+        y = _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu, bias, log_sigmoid)
+        y = y if out_f32 else y.to(torch.bfloat16)
+        return y if out is None else out.copy_(y)
     L = _native.lib()
     rt = runtime(act.data.device)
-    n_out = N // 2 if (swiglu or clamp_glu) else N
+    n_out = N // 2 if (swiglu or clamp_glu or geglu) else N
     if grouped is not None:
         n_out = grouped[3] // 2 if swiglu else grouped[3]
     if out is None and quant_out <= 0.0:
@@ -525,6 +542,12 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         a.epilogue, a.epi_n = EPI_SILU_COLS, silu_cols
     elif neg_exp_bias is not None:
         a.epilogue, a.epi_bias = EPI_NEG_EXP, _ptr(neg_exp_bias)
+    elif geglu:
+        a.epilogue = EPI_GEGLU
+    elif bias is not None:
+        a.epilogue, a.epi_bias = EPI_BIAS, _ptr(bias)
+    elif log_sigmoid is not None:
+        a.epilogue, a.epi_bias, a.epi_a = EPI_LOG_SIGMOID, _ptr(log_sigmoid[0]), float(log_sigmoid[1])
     a.ws, a.ws_bytes, a.status = _ptr(rt.ws), rt.ws_bytes, _ptr(rt.status)
     a.force_tn, a.force_splits, a.sm_count = force_tn, force_splits, rt.sm_count
     a.flags = (_PERSIST_PREFILL | _GROUPED_CTAS | (GEMM_ONE_TILE_PER_CTA if one_tile_per_cta else 0)

@@ -1,5 +1,5 @@
 // Paged causal attention on the CUDA cores in fp32 arithmetic: any query/key and value head size (up to
-// 512), bf16 or fp32 cache, optional sink (one added to the softmax denominator). It serves models that
+// 2048 / 1024), bf16 or fp32 cache, optional sink (one added to the softmax denominator). It serves models that
 // run in true 32-bit, and head sizes beyond the tensor-core kernels' tiles.
 //
 // One CTA per (query head, query row), 128 threads. Per tile of 128 cached tokens: thread j scores token j
@@ -34,7 +34,7 @@ __device__ __forceinline__ float lda(const T* p) {
   else return *p;
 }
 
-constexpr int kMaxDv = 512;
+constexpr int kMaxDv = 1024;
 
 template <typename T>
 __global__ void __launch_bounds__(128) attn_simt_kernel(const SimtAttnParams p) {

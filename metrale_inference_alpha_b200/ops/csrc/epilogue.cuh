@@ -4,7 +4,7 @@
 
 namespace mb {
 
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_NEG_EXP = 4 };
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_NEG_EXP = 4, EPI_GEGLU = 5, EPI_BIAS = 6, EPI_LOG_SIGMOID = 7 };
 
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
@@ -19,5 +19,14 @@ __device__ __forceinline__ float clamp_glu_fast(float gate, float up, float alph
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   return __fdividef(g * (u + 1.f), 1.f + __expf(-alpha * g));
 }
+
+
+// gelu_tanh(gate) * up; 0.5 (1 + tanh(a)) = sigmoid(2 a), and 1.5957... = 2 sqrt(2 / pi)
+__device__ __forceinline__ float gelu_tanh(float z) { return z * sigmoid_exact(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
+__device__ __forceinline__ float geglu_fast(float gate, float up) {
+  return __fdividef(gate * up, 1.f + __expf(-1.5957691216057308f * (gate + 0.044715f * gate * gate * gate)));
+}
+// log(sigmoid(z)), without cancellation on either side
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
 }  // namespace mb

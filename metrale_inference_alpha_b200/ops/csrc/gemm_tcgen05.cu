@@ -43,6 +43,9 @@ namespace {
 
 enum { KIND_BF16 = 0, KIND_FP8 = 1, KIND_NVFP4 = 2, KIND_FP8_BLOCK = 3 };
 using mb::EPI_CLAMP_GLU;
+using mb::EPI_BIAS;
+using mb::EPI_GEGLU;
+using mb::EPI_LOG_SIGMOID;
 using mb::EPI_NEG_EXP;
 using mb::EPI_PLAIN;
 using mb::EPI_SILU_COLS;
@@ -63,9 +66,9 @@ struct GemmParams {
   uint32_t* cnt;
   int splits, kb_per_split, num_kb;
   int epilogue, out_f32;
-  float epi_a, epi_b;     // EPI_CLAMP_GLU: sigmoid slope and clamp limit
+  float epi_a, epi_b;     // EPI_CLAMP_GLU: sigmoid slope and clamp limit; EPI_LOG_SIGMOID: epi_a log(sigmoid(y + bias[n]))
   int epi_n;              // EPI_SILU_COLS: SiLU on output columns below this
-  const float* epi_bias;  // EPI_NEG_EXP: -exp(y + bias[n])
+  const float* epi_bias;  // EPI_NEG_EXP, EPI_BIAS, EPI_LOG_SIGMOID (set for those alone)
   uint32_t* status;
   // grouped (MoE) mode: blockIdx.y indexes a tile work-list; W is [experts * n_per_expert, K]
   const int* tile_expert;
@@ -317,8 +320,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
     float* s_tile = reinterpret_cast<float*>(smem);
     bool ok = true;
-    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU);   // paired (gate, up) columns
+    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && (p.epilogue == EPI_CLAMP_GLU || p.epilogue == EPI_GEGLU));   // paired (gate, up) columns
     const bool clamp_glu = KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU;      // bf16 models only
+    const bool geglu = KIND == KIND_BF16 && p.epilogue == EPI_GEGLU;
     mb::pdl_wait();                                        // first global access of these warps follows
     // per-token scales of this tile, staged while the main loop runs
     for (int j = et; j < TN; j += 128) {
@@ -448,6 +452,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
           for (int i = 0; i < 8; ++i)
             y[i] = mb::clamp_glu_fast(x[2 * i] * wcol[2 * i] * as, x[2 * i + 1] * wcol[2 * i + 1] * as, p.epi_a, p.epi_b);
+        } else if (geglu) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[i] = mb::geglu_fast(x[2 * i] * wcol[2 * i] * as, x[2 * i + 1] * wcol[2 * i + 1] * as);
         } else if (swiglu) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) y[i] = mb::silu(x[2 * i] * wcol[2 * i] * as) * (x[2 * i + 1] * wcol[2 * i + 1] * as);
@@ -463,12 +470,19 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
               for (int i = 0; i < 8; ++i) y[i] = n_out0 + i < p.epi_n ? mb::silu(y[i]) : y[i];
             }
-          } else if (KIND == KIND_BF16 && p.epilogue == EPI_NEG_EXP) {
+          } else if (KIND == KIND_BF16 && p.epi_bias) {
             float eb[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) eb[i] = n_out0 + i < n_out_limit ? __ldg(p.epi_bias + n_out0 + i) : 0.f;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) y[i] = -expf(y[i] + eb[i]);
+            for (int i = 0; i < 8; ++i) y[i] += eb[i];
+            if (p.epilogue == EPI_NEG_EXP) {
+#pragma unroll
+              for (int i = 0; i < 8; ++i) y[i] = -expf(y[i]);
+            } else if (p.epilogue == EPI_LOG_SIGMOID) {
+#pragma unroll
+              for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::log_sigmoid(y[i]);
+            }
           }
         }
         const size_t o = (size_t)m * p.ldo + n_out0;
@@ -800,8 +814,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
     const int lane = threadIdx.x & 31;
     const int et = threadIdx.x - 64;
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
-    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU);   // paired (gate, up) columns
+    const bool swiglu = p.epilogue == EPI_SWIGLU || (KIND == KIND_BF16 && (p.epilogue == EPI_CLAMP_GLU || p.epilogue == EPI_GEGLU));   // paired (gate, up) columns
     const bool clamp_glu = KIND == KIND_BF16 && p.epilogue == EPI_CLAMP_GLU;      // bf16 models only
+    const bool geglu = KIND == KIND_BF16 && p.epilogue == EPI_GEGLU;
     mb::pdl_wait();
     const int f = q * 32 + lane;                          // weight row of this thread inside a tile
     const float outq_inv6gs = p.outq ? 1.f / (6.f * p.outq_gs) : 0.f;
@@ -850,7 +865,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             const float x0 = v[j] * (wsc * as.x), x1 = v[j + 1] * (wsc * as.y);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x0 : x1, 1);
             const float gate = odd ? other : x0, up = odd ? x1 : other;
-            const float y = clamp_glu ? mb::clamp_glu_fast(gate, up, p.epi_a, p.epi_b) : mb::silu(gate) * up;
+            const float y = clamp_glu ? mb::clamp_glu_fast(gate, up, p.epi_a, p.epi_b) : geglu ? mb::geglu_fast(gate, up) : mb::silu(gate) * up;
             const int ml = m0 + (odd ? 1 : 0);                 // row inside the tile
             const int m = m_base + ml;
             if (p.outq) {
@@ -886,10 +901,17 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] = mb::silu(v[j] * wsc * asc[c * 16 + j]);
             }
-          } else if (KIND == KIND_BF16 && p.epilogue == EPI_NEG_EXP) {
+          } else if (KIND == KIND_BF16 && p.epi_bias) {        // bf16 operands: the scales below are 1
             const float bias = n < p.N ? p.epi_bias[n] : 0.f;
 #pragma unroll
-            for (int j = 0; j < 16; ++j) v[j] = -expf(v[j] * wsc * asc[c * 16 + j] + bias);
+            for (int j = 0; j < 16; ++j) v[j] = v[j] * wsc * asc[c * 16 + j] + bias;
+            if (p.epilogue == EPI_NEG_EXP) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = -expf(v[j]);
+            } else if (p.epilogue == EPI_LOG_SIGMOID) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::log_sigmoid(v[j]);
+            }
           }
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -1000,10 +1022,11 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   if (row_bytes % 16) return MB_ERR_BAD_ARG;           // TMA global stride rule
   if (kind == KIND_NVFP4 && (!a->sfa || !a->sfb)) return MB_ERR_BAD_ARG;
   if (kind == KIND_FP8_BLOCK && (!a->w_scale || !a->a_scale)) return MB_ERR_BAD_ARG;
-  if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
-  if ((a->epilogue == EPI_SILU_COLS || a->epilogue == EPI_NEG_EXP) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
-  if (a->epilogue == EPI_NEG_EXP && !a->epi_bias) return MB_ERR_BAD_ARG;
-  if (a->epilogue == EPI_CLAMP_GLU && kind != KIND_BF16) return MB_ERR_UNSUPPORTED;
+  if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU || a->epilogue == EPI_GEGLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
+  const bool biased = a->epilogue == EPI_NEG_EXP || a->epilogue == EPI_BIAS || a->epilogue == EPI_LOG_SIGMOID;
+  if ((a->epilogue == EPI_SILU_COLS || biased) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
+  if (biased != (a->epi_bias != nullptr)) return MB_ERR_BAD_ARG;
+  if ((a->epilogue == EPI_CLAMP_GLU || a->epilogue == EPI_GEGLU) && kind != KIND_BF16) return MB_ERR_UNSUPPORTED;
   const int num_kb = (a->K + kelems - 1) / kelems;
   if (kind == KIND_NVFP4 && a->sf_k64 < num_kb * 4) return MB_ERR_BAD_ARG;
 

@@ -16,13 +16,24 @@
 //
 // Steps of one token per sequence take linear_decode_kernel instead: one CTA per (sequence, head) streams the
 // state once, 16 rows of 16-byte vectors in flight per thread, and can finish the head's output itself (RMS over
-// the head, weight, gate, scale), so decode needs no separate norm launch.
+// the head, weight, gate, scale), so decode needs no separate norm launch; decays given as a low-rank projection are
+// computed there too, one channel per thread.
 #include "common.cuh"
 #include "epilogue.cuh"
 
 namespace {
 
 using bf16 = __nv_bfloat16;
+
+// log decays c log(sigmoid(a2 a1 + bias)): a1 [T, rank] of the activation type, a2 [H * DK, rank], bias [H * DK]
+struct LowRank {
+  const void* a1;                  // null: not used
+  long long a1_ld;
+  const bf16* a2;
+  const float* bias;
+  int rank;
+  float c;
+};
 
 struct LinParams {
   const void* q;
@@ -32,6 +43,7 @@ struct LinParams {
   int H, DK, DV;
   const float* log_w;              // [T, H * DK] or null
   const float* decay;              // [H] when log_w is null
+  LowRank lr;                      // decode: the decays from their low-rank projection instead of log_w
   const float* u;                  // [H, DK]: bonus readout before the update; null: readout after it
   float* state;                    // [slots, H, DK, DV]
   float* out;                      // [T, H * DV]
@@ -323,7 +335,17 @@ __global__ void __launch_bounds__(256, 2) linear_decode_kernel(const LinParams p
     const float qv = ldx<T>(p.q, t * p.q_ld + (size_t)hd * DK + tid), kv = ldx<T>(p.k, t * p.k_ld + (size_t)hd * DK + tid);
     sq[tid] = qv;
     sk[tid] = kv;
-    if constexpr (CH) sw[tid] = expf(p.log_w[(t * p.H + hd) * DK + tid]);
+    if constexpr (CH) {
+      if (p.lr.a1) {
+        const size_t n = (size_t)hd * DK + tid;
+        const bf16* a2 = p.lr.a2 + n * p.lr.rank;
+        float z = p.lr.bias[n];
+        for (int r = 0; r < p.lr.rank; ++r) z = fmaf(ldx<T>(p.lr.a1, t * p.lr.a1_ld + r), __bfloat162float(a2[r]), z);
+        sw[tid] = expf(p.lr.c * mb::log_sigmoid(z));
+      } else {
+        sw[tid] = expf(p.log_w[(t * p.H + hd) * DK + tid]);
+      }
+    }
     if constexpr (BONUS) bonus = qv * p.u[hd * DK + tid] * kv;
   }
   if constexpr (BONUS) bonus = mb::block_sum(bonus, red);
@@ -380,7 +402,7 @@ int launch_decode(const LinParams& p, const DecodeNorm& nm, int num_seqs, cudaSt
 }
 template <typename T>
 int decode_mode(const LinParams& p, const DecodeNorm& nm, int num_seqs, cudaStream_t stream) {
-  if (p.log_w) return p.u ? launch_decode<T, true, true>(p, nm, num_seqs, stream) : launch_decode<T, true, false>(p, nm, num_seqs, stream);
+  if (p.log_w || p.lr.a1) return p.u ? launch_decode<T, true, true>(p, nm, num_seqs, stream) : launch_decode<T, true, false>(p, nm, num_seqs, stream);
   return p.u ? launch_decode<T, false, true>(p, nm, num_seqs, stream) : launch_decode<T, false, false>(p, nm, num_seqs, stream);
 }
 
@@ -439,20 +461,27 @@ struct MbLinearAttnArgs {
   float eps, scale;
   void* norm_out;
   long long norm_out_ld;
+  const void* lr_a1;         // decode: low-rank decays (log_w and decay null)
+  long long lr_a1_ld;
+  const void* lr_a2;
+  const float* lr_bias;
+  int lr_rank;
+  float lr_c;
 };
 
 extern "C" int mb_linear_attn(const MbLinearAttnArgs* a, cudaStream_t stream) {
-  if (!a || !a->q || !a->k || !a->v || !a->state || (a->write_out && !a->out && !a->norm_w) || (!a->log_w && !a->decay)) return MB_ERR_BAD_ARG;
+  if (!a || !a->q || !a->k || !a->v || !a->state || (a->write_out && !a->out && !a->norm_w) || (!a->log_w && !a->decay && !a->lr_a1)) return MB_ERR_BAD_ARG;
   if (a->H <= 0 || a->DK <= 0 || a->DV <= 0 || a->num_seqs <= 0 || a->num_seqs > 65535 || a->H > 65535) return MB_ERR_BAD_ARG;
   if (reinterpret_cast<uintptr_t>(a->state) % 16) return MB_ERR_BAD_ARG;
-  LinParams p{a->q, a->k, a->v, a->q_ld, a->k_ld, a->v_ld, a->H, a->DK, a->DV, a->log_w, a->decay, a->u, a->state, a->out,
-              a->q_start, a->q_len, a->positions, a->slots, a->num_slots, a->write_state, a->write_out, a->status};
+  LinParams p{a->q, a->k, a->v, a->q_ld, a->k_ld, a->v_ld, a->H, a->DK, a->DV, a->log_w, a->decay,
+              LowRank{a->lr_a1, a->lr_a1_ld, (const bf16*)a->lr_a2, a->lr_bias, a->lr_rank, a->lr_c}, a->u, a->state, a->out, a->q_start, a->q_len, a->positions, a->slots, a->num_slots, a->write_state, a->write_out, a->status};
+  if (a->lr_a1 && (!a->lr_a2 || !a->lr_bias || a->lr_rank <= 0)) return MB_ERR_BAD_ARG;
   if (a->decode) {
     if (a->DV % 4 || a->DV > 256 || a->DK > 256) return MB_ERR_UNSUPPORTED;
     if (a->norm_w && (!a->gate || !a->norm_out)) return MB_ERR_BAD_ARG;
     const DecodeNorm nm{(const bf16*)a->norm_w, a->gate, a->gate_ld, a->sigmoid_gate, a->eps, a->scale, a->norm_out, a->norm_out_ld};
     return a->f32 ? decode_mode<float>(p, nm, a->num_seqs, stream) : decode_mode<bf16>(p, nm, a->num_seqs, stream);
   }
-  if (a->norm_w) return MB_ERR_UNSUPPORTED;
+  if (a->norm_w || a->lr_a1) return MB_ERR_UNSUPPORTED;
   return a->f32 ? launch_mode<float>(p, a->num_seqs, stream) : launch_mode<bf16>(p, a->num_seqs, stream);
 }

@@ -16,7 +16,8 @@
 // Per-channel decays make a plain factorisation q_i 2^L_i . k_j 2^-L_j overflow. The scores are built in 16 x 16
 // blocks: off the diagonal both factors are taken relative to the end of the block before the query's, so both
 // exponents are <= 0; on the diagonal the decay between j and i is multiplied up step by step, without a logarithm
-// or an exponential. Modes: per-head decay read after the update, per-channel decay with a bonus read before it.
+// or an exponential. Modes: per-head decay read after the update, per-channel decay read after it or, with a bonus,
+// before it.
 // Head sizes 64 and 128. Sequence s keeps its chunks from index q_start[s] / 64 + s on, which never overlaps.
 #include "common.cuh"
 
@@ -33,7 +34,7 @@ struct ChunkParams {
   int H;
   const float* log_w;          // [T, H * DK] or null
   const float* decay;          // [H] when log_w is null
-  const float* u;              // [H, DK] with log_w
+  const float* u;              // [H, DK]: bonus readout (with log_w)
   float* state;                // [slots, H, DK, DV]
   float* out;                  // [T, H * DV]
   float* ws_c;                 // [chunks, H, DK * DV] contributions
@@ -257,7 +258,7 @@ __device__ __forceinline__ float reduce16(float (&v)[16], int lane) {
   return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 16);
 }
 
-template <int DK, int DV, bool CH>
+template <int DK, int DV, bool CH, bool BONUS>
 __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) uint8_t raw[];
   auto& s = *reinterpret_cast<OutSmem<DK, DV>*>(raw);
@@ -301,7 +302,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) 
     constexpr int kCh = DK / 32;
     float uu[kCh];
 #pragma unroll
-    for (int e = 0; e < kCh; ++e) uu[e] = p.u[hd * DK + e * 32 + lane];
+    for (int e = 0; e < kCh; ++e) uu[e] = BONUS ? p.u[hd * DK + e * 32 + lane] : 1.f;
     for (int j = half; j < 16; j += 2) {
       float kk[kCh], val[16];
 #pragma unroll
@@ -315,6 +316,9 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) 
             const float qv = __bfloat162float(s.q[i0 + i][e * 32 + lane]);
             if (i == j) {
               val[i] = fmaf(qv * uu[e], kk[e], val[i]);              // the bonus stands in for the token itself
+            } else if constexpr (!BONUS) {
+              kk[e] *= s.L[i0 + i][e * 32 + lane];                   // read after step i's decay
+              val[i] = fmaf(qv, kk[e], val[i]);
             } else {
               val[i] = fmaf(qv, kk[e], val[i]);
               kk[e] *= s.L[i0 + i][e * 32 + lane];
@@ -332,16 +336,18 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) 
     __syncthreads();
     running_logs<DK>(s.L, lw, (size_t)p.H * DK, valid);
   }
-  // query fragments of this warp's rows decayed from the reference on: q_i 2^(L_(i-1) - ref), value and remainder
+  // query fragments of this warp's rows decayed from the reference on: q_i 2^(L_(i-1) - ref), or L_i when read after
+  // the update; value and remainder
+  constexpr int kBefore = BONUS ? 1 : 0;
   auto q_frag = [&](int k0, const float* refL, uint32_t* hi, uint32_t* lo) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int i = i0 + g + (e & 1) * 8, d = k0 + 2 * t + (e >> 1) * 8;
       const float2 qv = bf2(&s.q[i][d]);
       float la = 0.f, lb = 0.f;
-      if (i > 0) {
-        la = s.L[i - 1][d];
-        lb = s.L[i - 1][d + 1];
+      if (i >= kBefore) {
+        la = s.L[i - kBefore][d];
+        lb = s.L[i - kBefore][d + 1];
       }
       la -= refL[d];
       lb -= refL[d + 1];
@@ -426,9 +432,9 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) 
       const int r = i / (DK / 2), d = (i - r * (DK / 2)) * 2;
       const float2 qv = bf2(&s.q[r][d]);
       float la = 0.f, lb = 0.f;
-      if (r > 0) {
-        la = s.L[r - 1][d];
-        lb = s.L[r - 1][d + 1];
+      if (r >= kBefore) {
+        la = s.L[r - kBefore][d];
+        lb = s.L[r - kBefore][d + 1];
       }
       split2(qv.x * ex2(la), qv.y * ex2(lb), *reinterpret_cast<uint32_t*>(&s.q[r][d]), *reinterpret_cast<uint32_t*>(&s.k[r][d]));
     }
@@ -501,7 +507,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const ChunkParams p) 
   }
 }
 
-template <int DK, int DV, bool CH>
+template <int DK, int DV, bool CH, bool BONUS>
 int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
   using SS = StateSmem<DK, DV>;
   using SO = OutSmem<DK, DV>;
@@ -509,22 +515,22 @@ int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(chunk_state_kernel<DK, DV, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(chunk_out_kernel<DK, DV, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(chunk_out_kernel<DK, DV, CH, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const dim3 grid((max_q_len + kC - 1) / kC, p.H, num_seqs);
   cudaError_t e = mb::launch_kernel(chunk_state_kernel<DK, DV, CH>, grid, dim3(256), ss, stream, p);
   if (e == cudaSuccess) e = mb::launch_kernel(chunk_scan_kernel<DK, DV>, dim3(DK * DV / 1024, p.H, num_seqs), dim3(256), 0, stream, p);
-  if (e == cudaSuccess) e = mb::launch_kernel(chunk_out_kernel<DK, DV, CH>, grid, dim3(256), so, stream, p);
+  if (e == cudaSuccess) e = mb::launch_kernel(chunk_out_kernel<DK, DV, CH, BONUS>, grid, dim3(256), so, stream, p);
   return (int)e;
 }
-template <bool CH>
+template <bool CH, bool BONUS>
 int dispatch_dims(const ChunkParams& p, int DK, int DV, int num_seqs, int max_q_len, cudaStream_t stream) {
-  if (DK == 64 && DV == 64) return launch_chunks<64, 64, CH>(p, num_seqs, max_q_len, stream);
-  if (DK == 64 && DV == 128) return launch_chunks<64, 128, CH>(p, num_seqs, max_q_len, stream);
-  if (DK == 128 && DV == 64) return launch_chunks<128, 64, CH>(p, num_seqs, max_q_len, stream);
-  if (DK == 128 && DV == 128) return launch_chunks<128, 128, CH>(p, num_seqs, max_q_len, stream);
+  if (DK == 64 && DV == 64) return launch_chunks<64, 64, CH, BONUS>(p, num_seqs, max_q_len, stream);
+  if (DK == 64 && DV == 128) return launch_chunks<64, 128, CH, BONUS>(p, num_seqs, max_q_len, stream);
+  if (DK == 128 && DV == 64) return launch_chunks<128, 64, CH, BONUS>(p, num_seqs, max_q_len, stream);
+  if (DK == 128 && DV == 128) return launch_chunks<128, 128, CH, BONUS>(p, num_seqs, max_q_len, stream);
   return MB_ERR_UNSUPPORTED;
 }
 
@@ -558,7 +564,7 @@ extern "C" size_t mb_linear_chunked_ws_bytes(int total_rows, int num_seqs, int H
 extern "C" int mb_linear_chunked(const MbLinearChunkedArgs* a, cudaStream_t stream) {
   if (!a || !a->q || !a->k || !a->v || !a->state || !a->out || !a->ws) return MB_ERR_BAD_ARG;
   if (a->num_seqs <= 0 || a->num_seqs > 65535 || a->H <= 0 || a->H > 65535 || a->max_q_len <= 0 || a->total_rows <= 0) return MB_ERR_BAD_ARG;
-  if ((a->log_w != nullptr) != (a->u != nullptr) || (!a->log_w && !a->decay)) return MB_ERR_UNSUPPORTED;
+  if ((a->u && !a->log_w) || (!a->log_w && !a->decay)) return MB_ERR_UNSUPPORTED;
   const uintptr_t al = reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) | reinterpret_cast<uintptr_t>(a->v) |
                        reinterpret_cast<uintptr_t>(a->state) | reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->ws);
   if ((al & 15) || (a->q_ld | a->k_ld | a->v_ld) % 8) return MB_ERR_UNSUPPORTED;      // 16-byte copies
@@ -574,6 +580,7 @@ extern "C" int mb_linear_chunked(const MbLinearChunkedArgs* a, cudaStream_t stre
   p.ws_d = reinterpret_cast<float*>(p.ws_lo + chunks * per);
   p.q_start = a->q_start; p.q_len = a->q_len; p.positions = a->positions; p.slots = a->slots;
   p.num_slots = a->num_slots; p.write_state = a->write_state; p.status = a->status;
-  return a->log_w ? dispatch_dims<true>(p, a->DK, a->DV, a->num_seqs, a->max_q_len, stream)
-                  : dispatch_dims<false>(p, a->DK, a->DV, a->num_seqs, a->max_q_len, stream);
+  if (a->u) return dispatch_dims<true, true>(p, a->DK, a->DV, a->num_seqs, a->max_q_len, stream);
+  return a->log_w ? dispatch_dims<true, false>(p, a->DK, a->DV, a->num_seqs, a->max_q_len, stream)
+                  : dispatch_dims<false, false>(p, a->DK, a->DV, a->num_seqs, a->max_q_len, stream);
 }

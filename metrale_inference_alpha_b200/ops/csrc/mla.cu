@@ -27,7 +27,8 @@ namespace {
 constexpr int kD = 576, kL = 512, kRowB = kD * 2, kChunks = kRowB / 16, kTile = 64;
 constexpr int kTileB = kTile * kRowB;
 constexpr int kQB = 16 * kRowB;
-constexpr int kSmem = 2 * kTileB + kQB + 16 * 128 /*P*/ + 4 * 16 * 4 /*max*/ + 4 * 16 * 4 /*l*/;
+constexpr int kPB = 16 * 128;                 // P, and as much again for what rounding took off it
+constexpr int kSmem = 2 * kTileB + kQB + 2 * kPB + 4 * 16 * 4 /*max*/ + 4 * 16 * 4 /*l*/;
 
 struct MlaParams {
   const __nv_bfloat16* q;       // [rows, H, 576]
@@ -40,10 +41,11 @@ struct MlaParams {
   int H, block_size;
   long long num_blocks;
   float scale;
-  float* out;                   // [rows, H, 512] fp32
+  void* out;                    // [rows, H, 512] fp32, or bf16 with out_bf16
   float* part_o;                // [rows * H, parts, 512]
   float* part_ml;               // [rows * H, parts, 2]
   int parts, part_tokens;
+  int split_p, out_bf16;
   uint32_t* status;
 };
 
@@ -78,7 +80,7 @@ __global__ void __launch_bounds__(128, 1) mla_decode_kernel(const MlaParams p) {
   extern __shared__ __align__(128) uint8_t smem_mla[];
   const uint32_t sbase = mb::smem_u32(smem_mla);
   const uint32_t sQ = sbase + 2 * kTileB, sP = sQ + kQB;
-  float* s_max = reinterpret_cast<float*>(smem_mla + 2 * kTileB + kQB + 16 * 128);
+  float* s_max = reinterpret_cast<float*>(smem_mla + 2 * kTileB + kQB + 2 * kPB);
   float* s_l = s_max + 64;
   const int rg = blockIdx.x, seq = blockIdx.y, part = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -218,7 +220,12 @@ __global__ void __launch_bounds__(128, 1) mla_decode_kernel(const MlaParams p) {
         const int r = g + hr * 8;
         const int col = warp * 16 + n * 8 + t * 2;                 // token column
         const uint32_t addr = sP + r * 128 + ((((col >> 3) ^ (r & 7)) << 4) | ((col & 7) << 1));
-        asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(pack_bf16(s[n][hr * 2], s[n][hr * 2 + 1])) : "memory");
+        const uint32_t hi = pack_bf16(s[n][hr * 2], s[n][hr * 2 + 1]);
+        asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(hi) : "memory");
+        if (p.split_p) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
+          asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr + kPB), "r"(pack_bf16(s[n][hr * 2] - f.x, s[n][hr * 2 + 1] - f.y)) : "memory");
+        }
       }
     __syncthreads();
     // ---- O[:, 128 warp ..] = alpha * O + P V
@@ -229,11 +236,12 @@ __global__ void __launch_bounds__(128, 1) mla_decode_kernel(const MlaParams p) {
     }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
-      uint32_t a[4];
+      uint32_t a[4], al[4];
       {
         const int r = (lane & 7) + (((lane >> 3) & 1) << 3);
         const int ch = kk * 2 + (lane >> 4);
         ldsm4(a, sP + r * 128 + ((ch ^ (r & 7)) << 4));
+        if (p.split_p) ldsm4(al, sP + kPB + r * 128 + ((ch ^ (r & 7)) << 4));
       }
 #pragma unroll
       for (int n2 = 0; n2 < 8; ++n2) {
@@ -241,6 +249,10 @@ __global__ void __launch_bounds__(128, 1) mla_decode_kernel(const MlaParams p) {
         ldsm4t(b, kT + swz(kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), warp * 16 + n2 * 2 + (lane >> 4)));
         mma_bf16(o_acc[n2 * 2], a, b[0], b[1]);
         mma_bf16(o_acc[n2 * 2 + 1], a, b[2], b[3]);
+        if (p.split_p) {
+          mma_bf16(o_acc[n2 * 2], al, b[0], b[1]);
+          mma_bf16(o_acc[n2 * 2 + 1], al, b[2], b[3]);
+        }
       }
     }
   }
@@ -264,11 +276,14 @@ __global__ void __launch_bounds__(128, 1) mla_decode_kernel(const MlaParams p) {
     const float inv = l > 0.f ? 1.f / l : 0.f;
     const int tq = row / p.H, hh = row - tq * p.H;
     const size_t grow = (size_t)(qs + tq) * p.H + hh;
-    float* dst = nparts == 1 ? p.out + grow * kL : p.part_o + (grow * p.parts + part) * kL;
+    const bool bf = nparts == 1 && p.out_bf16;
+    float* dst = nparts == 1 ? reinterpret_cast<float*>(p.out) + (bf ? 0 : grow * kL) : p.part_o + (grow * p.parts + part) * kL;
 #pragma unroll
     for (int n = 0; n < 16; ++n) {
       const float2 v = make_float2(o_acc[n][hr * 2] * inv, o_acc[n][hr * 2 + 1] * inv);
-      *reinterpret_cast<float2*>(dst + warp * 128 + n * 8 + t * 2) = v;
+      const int c = warp * 128 + n * 8 + t * 2;
+      if (bf) *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + grow * kL + c) = pack_bf16(v.x, v.y);
+      else *reinterpret_cast<float2*>(dst + c) = v;
     }
     if (nparts > 1 && warp == 0 && t == 0) {
       p.part_ml[(grow * p.parts + part) * 2] = m_run[hr];
@@ -300,7 +315,8 @@ __global__ void mla_merge_kernel(const MlaParams p, const int* row_seq) {
       const float w = m == -INFINITY ? 0.f : l * exp2f(m - M) * inv;
       acc += w * p.part_o[((size_t)grow * p.parts + s) * kL + d];
     }
-    p.out[(size_t)grow * kL + d] = acc;
+    if (p.out_bf16) reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)grow * kL + d] = __float2bfloat16(acc);
+    else reinterpret_cast<float*>(p.out)[(size_t)grow * kL + d] = acc;
   }
 }
 
@@ -357,7 +373,7 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
       const uint4 v = src ? src[c] : make_uint4(0, 0, 0, 0);
       *reinterpret_cast<uint4*>(sQ + (c >> 3) * kTcQB + tc_sw(tid, c & 7)) = v;
     }
-    // the upper half of every P row is never written again: the second product only reads 32 tokens
+    // the upper half of every P row holds what rounding took off the weights (split_p), else it is never read
 #pragma unroll
     for (int c = 4; c < 8; ++c) *reinterpret_cast<uint4*>(sP + tc_sw(tid, c)) = make_uint4(0, 0, 0, 0);
   }
@@ -457,16 +473,19 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
       float rs = 0.f;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        uint4 pk;
-        uint32_t* pw = reinterpret_cast<uint32_t*>(&pk);
+        uint4 pk, lo;
+        uint32_t *pw = reinterpret_cast<uint32_t*>(&pk), *lw = reinterpret_cast<uint32_t*>(&lo);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float a = tc_ex2(sv[c * 8 + 2 * i] - m_use), b = tc_ex2(sv[c * 8 + 2 * i + 1] - m_use);
           const __nv_bfloat162 pb = __floats2bfloat162_rn(a, b);
           rs += a + b;
           pw[i] = *reinterpret_cast<const uint32_t*>(&pb);
+          const float2 f = __bfloat1622float2(pb);
+          lw[i] = pack_bf16(a - f.x, b - f.y);
         }
         *reinterpret_cast<uint4*>(sP + tc_sw(tid, c)) = pk;
+        if (p.split_p) *reinterpret_cast<uint4*>(sP + tc_sw(tid, c + 4)) = lo;
       }
       l_run = l_run * alpha + rs;
     }
@@ -480,6 +499,12 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
       for (int s = 0; s < 2; ++s)                         // 16 tokens per step = two 8-row groups of the tile
         mb::umma_f16(tmem + 32, mb::umma_desc_sw128(aP + s * 32),
                      mb::umma_desc_sw128_mn(aK + (4 * hv) * kTcKB + s * 2048, kTcKB, 1024), kIdescO, (j | s) != 0);
+      if (p.split_p) {                                    // the remainders sit 32 tokens further, over the same values
+#pragma unroll
+        for (int s = 0; s < 2; ++s)
+          mb::umma_f16(tmem + 32, mb::umma_desc_sw128(aP + (2 + s) * 32),
+                       mb::umma_desc_sw128_mn(aK + (4 * hv) * kTcKB + s * 2048, kTcKB, 1024), kIdescO, true);
+      }
       mb::tc_commit(&bar_o);
     }
   }
@@ -491,12 +516,23 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
     const bool row_ok = tid < p.H;
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
     const size_t grow = (size_t)row * p.H + (row_ok ? tid : 0);
-    float* dst = (nparts == 1 ? p.out + grow * kL : p.part_o + (grow * p.parts + part) * kL) + hv * 256;
+    const bool bf = nparts == 1 && p.out_bf16;
+    float* dst = (nparts == 1 ? reinterpret_cast<float*>(p.out) + (bf ? 0 : grow * kL) : p.part_o + (grow * p.parts + part) * kL) + hv * 256;
+    __nv_bfloat16* dst16 = reinterpret_cast<__nv_bfloat16*>(p.out) + grow * kL + hv * 256;
 #pragma unroll
     for (int c = 0; c < 16; ++c) {
       float ov[16];
       mb::tmem_ld16(t_row + 32 + c * 16, ov);
-      if (row_ok) {
+      if (row_ok && bf) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          uint4 v;
+          uint32_t* pv = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) pv[e] = pack_bf16(ov[8 * i + 2 * e] * inv, ov[8 * i + 2 * e + 1] * inv);
+          *reinterpret_cast<uint4*>(dst16 + c * 16 + i * 8) = v;
+        }
+      } else if (row_ok) {
 #pragma unroll
         for (int i = 0; i < 4; ++i)
           *reinterpret_cast<float4*>(dst + c * 16 + i * 4) =
@@ -537,6 +573,7 @@ int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream) {
   p.q_start = a->q_start; p.q_len = a->q_len; p.ctx_len = a->ctx_len;
   p.H = a->H; p.block_size = a->block_size; p.num_blocks = a->num_blocks;
   p.scale = a->scale; p.out = a->out; p.status = a->status;
+  p.split_p = a->split_p; p.out_bf16 = a->out_bf16;
   p.part_tokens = a->part_tokens > 0 ? a->part_tokens : 1024;
   p.parts = (a->max_ctx + p.part_tokens - 1) / p.part_tokens;
   if (p.parts < 1) p.parts = 1;
@@ -572,6 +609,7 @@ int mb_mla_attention(const MbMlaArgs* a, cudaStream_t stream) {
   p.q_start = a->q_start; p.q_len = a->q_len; p.ctx_len = a->ctx_len;
   p.H = a->H; p.block_size = a->block_size; p.num_blocks = a->num_blocks;
   p.scale = a->scale; p.out = a->out; p.status = a->status;
+  p.split_p = a->split_p; p.out_bf16 = a->out_bf16;
   p.part_tokens = a->part_tokens > 0 ? a->part_tokens : 1024;
   p.parts = (a->max_ctx + p.part_tokens - 1) / p.part_tokens;
   if (p.parts < 1) p.parts = 1;

@@ -19,12 +19,14 @@ struct MbMlaArgs {
   int H, block_size;
   long long num_blocks;
   float scale;
-  float* out;
+  void* out;                 // [rows, H, 512] fp32 or bf16
   void* ws;
   size_t ws_bytes;
   int part_tokens;           // 0 = default 1024
   uint32_t* status;
   int impl;                  // 0 = choose, 1 = mma.sync kernel, 2 = tcgen05 kernel (decode rows, H <= 128)
+  int split_p;               // softmax weights enter the product with V as two bf16 terms
+  int out_bf16;              // out is bf16 [rows, H, 512]
 };
 
 extern "C" int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream);

@@ -4,8 +4,9 @@
 //   mb_moe_route    one warp per token over <= 512 expert logits: softmax top-k, or sigmoid
 //                   scores + selection bias with group-limited selection (keep the
 //                   `topk_group` groups with the largest sum of their two best biased scores,
-//                   then top-k inside them). Ties resolve to the lower expert id. Weights are
-//                   the un-biased scores, optionally sum-normalised and scaled.
+//                   then top-k inside them), or the softmax over the chosen ones of biased
+//                   logits (mode 2, 32-bit throughout). Ties resolve to the lower expert id.
+//                   Weights are the un-biased scores, optionally sum-normalised and scaled.
 //   mb_moe_sort     counting sort of the (token, slot) pairs by *local* expert: per-expert row
 //                   ranges, the pair -> row map, and a tile work-list of (expert, first row,
 //                   rows) entries for the grouped GEMM. Pairs routed to experts outside
@@ -40,7 +41,18 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
     score[j] = (j < per && e < E) ? x[e] : -INFINITY;
     mx = fmaxf(mx, score[j]);
   }
-  if (mode == 0) {  // softmax
+  if (mode == 2) {  // softmax over the chosen ones of the biased logits (normalised below)
+    mx = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < kMaxPerLane; ++j) {
+      const int e = j * 32 + lane;
+      sel[j] = (j < per && e < E) ? score[j] + (bias ? bias[e] : 0.f) : -INFINITY;
+      mx = fmaxf(mx, sel[j]);
+    }
+    mx = mb::warp_max(mx);
+#pragma unroll
+    for (int j = 0; j < kMaxPerLane; ++j) score[j] = sel[j] == -INFINITY ? 0.f : expf(sel[j] - mx);
+  } else if (mode == 0) {  // softmax
     mx = mb::warp_max(mx);
     float se = 0.f;
 #pragma unroll
@@ -140,7 +152,7 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
   }
   if (lane < K) {
     float w = my_w;
-    if (renorm) w = w / (wsum + (mode == 0 ? 0.f : 1e-20f));
+    if (renorm) w = w / (wsum + (mode == 1 ? 1e-20f : 0.f));
     out_w[(size_t)tok * out_ld + lane] = w * scaling;
     out_id[(size_t)tok * out_ld + lane] = my_id;
   }

@@ -10,11 +10,14 @@
 //                 carried state on the first row of its portion (zero at position 0). The CTA of a
 //                 sequence's first row also advances that state to its last row's h: it is the only
 //                 reader of the old value, so no other CTA can see a half-updated state.
+//   stream_rms    the same step for streams with RMS norms in front of their sublayers and none behind: x + y, plus
+//                 (mixture of experts) the weighted sum of a token's expert rows, gathered where the grouped GEMM
+//                 left them; then RMS norm, or the value as it is, into a row of a possibly wider matrix
 //   shift_commit  state := h of the last accepted row (write-on-accept after speculative verification)
 //   gated_norm    RMS over groups of channels x weight x act(gate) x scale, act = SiLU or sigmoid; the
 //                 output may be a column range of a wider matrix
 //   side_gate     gelu_tanh(z) * e, e gathered from a per-layer slice of a second embedding table
-//   embed_scaled  fp32 embedding rows times a constant
+//   embed_scaled  fp32 embedding rows times a constant, optionally with a copy in the activation type
 //   rope_dims     rotate-half positions on q and k with separate query/key and value head sizes, scattered
 //                 into a paged cache whose rows are padded (with zeros) to the attention kernel's tile
 // T is the activation type: bf16, or fp32 for models served in 32-bit.
@@ -210,6 +213,88 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamParams p) 
   }
 }
 
+// ------------------------------------------------------------------ add, gather experts, RMS norm
+enum { RMS_NONE = 0, RMS_NORM = 1, RMS_RAW = 2 };
+
+struct StreamRmsParams {
+  int W;
+  const float* x;
+  const void* y;             // [T, W] or null
+  const float* ye;           // expert rows, or null
+  long long ye_ld;
+  const int* pair_row;       // [T, K] rows of ye, -1 = none
+  const float* pair_w;       // [T, K]
+  int K, out_mode;
+  const bf16* w;
+  float eps;
+  float* x_out;              // or null
+  void* out;
+  long long out_ld;
+};
+
+// a row is NIT vectors per thread, kept in registers between the sum of squares and the output
+template <int VEC, int NIT, typename T>
+__global__ void __launch_bounds__(256) stream_rms_kernel(const StreamRmsParams p) {
+  __shared__ float red[32];
+  __shared__ int s_row[32];
+  __shared__ float s_w[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, W = p.W;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  if (p.ye) {
+    if (tid < p.K) {
+      s_row[tid] = p.pair_row[(size_t)t * p.K + tid];
+      s_w[tid] = p.pair_w[(size_t)t * p.K + tid];
+    }
+    __syncthreads();
+  }
+  float v[NIT][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NIT; ++i) {
+    const int k = (i * nt + tid) * VEC;
+    if (k >= W) continue;
+    ldn<VEC>(p.x + (size_t)t * W + k, v[i]);
+    if (p.y) {
+      float a[VEC];
+      ldn<VEC>(reinterpret_cast<const T*>(p.y) + (size_t)t * W + k, a);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i][e] += a[e];
+    }
+    if (p.ye) {
+      float s[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s[e] = 0.f;
+      for (int j = 0; j < p.K; ++j) {
+        if (s_row[j] < 0) continue;
+        float a[VEC];
+        ldn<VEC>(p.ye + (size_t)s_row[j] * p.ye_ld + k, a);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[e] = fmaf(s_w[j], a[e], s[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i][e] += s[e];
+    }
+    if (p.x_out) stn<VEC>(p.x_out + (size_t)t * W + k, v[i]);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[i][e], v[i][e], ss);
+  }
+  if (p.out_mode == RMS_NONE) return;
+  const float inv = p.out_mode == RMS_NORM ? rsqrtf(mb::block_sum(ss, red) / (float)W + p.eps) : 1.f;
+#pragma unroll
+  for (int i = 0; i < NIT; ++i) {
+    const int k = (i * nt + tid) * VEC;
+    if (k >= W) continue;
+    if (p.out_mode == RMS_NORM) {
+      float w[VEC];
+      ldn<VEC>(p.w + k, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i][e] *= inv * w[e];
+    }
+    stn<VEC>(reinterpret_cast<T*>(p.out) + (size_t)t * p.out_ld + k, v[i]);
+  }
+}
+
 __global__ void __launch_bounds__(256) shift_commit_kernel(const float* h32, int W, float* state, const int* q_start, const int* q_len,
                                                            const int* slots, int num_slots, uint32_t* status) {
   const int s = blockIdx.x, n = q_len[s];
@@ -320,9 +405,9 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float* z, bf16* o
   out[t * 2 * R + R + c] = __float2bfloat16(v - __bfloat162float(h));
 }
 
-template <int VEC>
+template <int VEC, typename T>
 __global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, const bf16* table, float* out, int W, int vocab, float scale,
-                                                           uint32_t* status) {
+                                                           T* copy, long long copy_ld, uint32_t* status) {
   mb::pdl_wait();
   mb::pdl_launch_dependents();
   const int t = blockIdx.x, tok = tokens[t];
@@ -336,6 +421,7 @@ __global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, co
 #pragma unroll
     for (int i = 0; i < VEC; ++i) v[i] *= scale;
     stn<VEC>(out + (size_t)t * W + k, v);
+    if (copy) stn<VEC>(copy + (size_t)t * copy_ld + k, v);
   }
 }
 
@@ -440,6 +526,22 @@ struct MbStreamNormArgs {
   uint32_t* status;
 };
 
+struct MbStreamRmsArgs {
+  int T, W, f32, out_mode;
+  const float* x;
+  const void* y;
+  const float* ye;
+  long long ye_ld;
+  const int* pair_row;
+  const float* pair_w;
+  int K;
+  const void* w;
+  float eps;
+  float* x_out;
+  void* out;
+  long long out_ld;
+};
+
 struct MbGatedNormArgs {
   int T, K, group, f32;
   const float* x;
@@ -501,6 +603,31 @@ int mb_stream_norm(const MbStreamNormArgs* a, cudaStream_t stream) {
   return (int)(v4 ? mb::launch_kernel(stream_norm_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(stream_norm_kernel<1, bf16>, g, b, 0, stream, p));
 }
 
+int mb_stream_rms(const MbStreamRmsArgs* a, cudaStream_t stream) {
+  if (!a || a->T <= 0 || a->W <= 0 || !a->x || (a->out_mode != RMS_NONE && !a->out) || (a->out_mode == RMS_NORM && !a->w)) return MB_ERR_BAD_ARG;
+  if (a->ye && (!a->pair_row || !a->pair_w || a->K <= 0 || a->K > 32 || a->ye_ld < a->W)) return MB_ERR_BAD_ARG;
+  const StreamRmsParams p{a->W, a->x, a->y, a->ye, a->ye_ld, a->pair_row, a->pair_w, a->K, a->out_mode, (const bf16*)a->w, a->eps, a->x_out, a->out, a->out_ld};
+  const bool v4 = a->W % 4 == 0 && a->out_ld % 4 == 0 && a->ye_ld % 4 == 0 && al(a->x, 16) && al(a->y, 16) && al(a->ye, 16) && al(a->x_out, 16) &&
+                  al(a->out, a->f32 ? 16 : 8) && al(a->w, 8);
+  const int vec = v4 ? 4 : 1, nt = max(row_threads(a->W, vec), 32), nit = (a->W + nt * vec - 1) / (nt * vec);
+  const dim3 g(a->T), b(nt);
+#define MB_RMS(V, N)                                                                                                   \
+  return a->f32 ? (int)mb::launch_kernel(stream_rms_kernel<V, N, float>, g, b, 0, stream, p)                           \
+                : (int)mb::launch_kernel(stream_rms_kernel<V, N, bf16>, g, b, 0, stream, p)
+  if (v4) {
+    if (nit <= 1) MB_RMS(4, 1);
+    if (nit <= 3) MB_RMS(4, 3);
+    if (nit <= 8) MB_RMS(4, 8);
+    if (nit <= 16) MB_RMS(4, 16);
+  } else {
+    if (nit <= 4) MB_RMS(1, 4);
+    if (nit <= 16) MB_RMS(1, 16);
+    if (nit <= 64) MB_RMS(1, 64);
+  }
+#undef MB_RMS
+  return MB_ERR_TOO_LARGE;
+}
+
 int mb_shift_commit(const float* h32, int W, float* state, const int* q_start, const int* q_len, const int* slots, int num_seqs, int num_slots,
                     uint32_t* status, cudaStream_t stream) {
   if (!h32 || !state || W <= 0 || num_seqs <= 0) return MB_ERR_BAD_ARG;
@@ -531,12 +658,18 @@ int mb_side_gate(const float* z, const int* tokens, const void* table, long long
                   : mb::launch_kernel(side_gate_kernel<1, bf16>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (bf16*)out, status));
 }
 
-int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, uint32_t* status, cudaStream_t stream) {
-  if (!tokens || !table || !out || M <= 0 || W <= 0) return MB_ERR_BAD_ARG;
-  const bool v4 = W % 4 == 0 && al(table, 8) && al(out, 16);
+// copy (or null): the same rows in the activation type, copy_ld elements apart
+int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, void* copy, long long copy_ld,
+                    int copy_f32, uint32_t* status, cudaStream_t stream) {
+  if (!tokens || !table || !out || M <= 0 || W <= 0 || (copy && copy_ld < W)) return MB_ERR_BAD_ARG;
+  const bool v4 = W % 4 == 0 && al(table, 8) && al(out, 16) && copy_ld % 4 == 0 && al(copy, 16);
   const dim3 g(M), b(row_threads(W, v4 ? 4 : 1));
-  return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4>, g, b, 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status)
-                  : mb::launch_kernel(embed_scaled_kernel<1>, g, b, 0, stream, tokens, (const bf16*)table, out, W, vocab, scale, status));
+  const bf16* tab = (const bf16*)table;
+  if (copy_f32)
+    return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, float>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (float*)copy, copy_ld, status)
+                    : mb::launch_kernel(embed_scaled_kernel<1, float>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (float*)copy, copy_ld, status));
+  return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, bf16>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (bf16*)copy, copy_ld, status)
+                  : mb::launch_kernel(embed_scaled_kernel<1, bf16>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (bf16*)copy, copy_ld, status));
 }
 
 int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) {

@@ -1,4 +1,4 @@
-"""Ops of models with a 32-bit residual stream: Dynamic-Tanh norms fused around the stream, token-shift
+"""Ops of models with a 32-bit residual stream: Dynamic-Tanh and RMS norms fused around the stream, token-shift
 mixes, attention with separate query/key and value head sizes and a softmax sink, decaying linear
 attention (per-head or per-channel decay), gated group norms and the token side input.
 
@@ -37,6 +37,15 @@ class RmsNorm:
     eps: float
 
 
+@dataclass
+class Routed:
+    """A mixture of experts' output that has not been summed: row pair_row[t K + j] of y, times w[t, j]. With
+    ``pair_row`` None (CPU) y is the sum itself, [T, W]."""
+    y: torch.Tensor                        # fp32 [pairs, >= W]
+    pair_row: Optional[torch.Tensor]       # int32 [T K], -1 = no row
+    w: Optional[torch.Tensor]              # fp32 [T, K]
+
+
 def act_of(t: torch.Tensor, fmt: str) -> Act:
     """`t` (already of the activation type) as a GEMM operand; on CPU operands are kept in fp32."""
     d = t if t.is_cuda else t.float()
@@ -58,12 +67,55 @@ class _StreamNormArgs(C.Structure):
                 ("status", C.c_void_p)]
 
 
+class _StreamRmsArgs(C.Structure):
+    _fields_ = [("T", C.c_int), ("W", C.c_int), ("f32", C.c_int), ("out_mode", C.c_int), ("x", C.c_void_p), ("y", C.c_void_p),
+                ("ye", C.c_void_p), ("ye_ld", C.c_longlong), ("pair_row", C.c_void_p), ("pair_w", C.c_void_p), ("K", C.c_int),
+                ("w", C.c_void_p), ("eps", C.c_float), ("x_out", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_longlong)]
+
+
 _native.register_optional("mb_stream_norm", [C.POINTER(_StreamNormArgs), C.c_void_p])
+_native.register_optional("mb_stream_rms", [C.POINTER(_StreamRmsArgs), C.c_void_p])
 _native.register_optional("mb_shift_commit", [C.c_void_p, C.c_int] + [C.c_void_p] * 4 + [C.c_int, C.c_int, C.c_void_p, C.c_void_p])
 
 
 def dyt_ref(x: torch.Tensor, n: DytNorm) -> torch.Tensor:
     return torch.tanh(n.alpha * x.float()) * n.w.float() + n.b.float()
+
+
+def stream_rms(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, routed: Optional[Routed] = None,
+               pre: Optional[RmsNorm] = None, raw: bool = False, out: Optional[torch.Tensor] = None):
+    """x' = x (+ y) (+ the routed experts' weighted sum), x [T, W] fp32, y of the activation type. Output pre(x'), or x'
+    itself with ``raw``, or none; ``out`` may be a column range of a wider matrix. Returns (x', output); x' is x itself
+    when nothing is added."""
+    T, W = x.shape
+    wanted = pre is not None or raw
+    if wanted and out is None:
+        out = torch.empty(T, W, dtype=DTYPE[fmt], device=x.device)
+    if not x.is_cuda:
+        x1 = x if y is None else x + y.float()
+        x1 = x1 if routed is None else x1 + routed.y
+        if wanted:
+            out.copy_(x1 if raw else x1 * torch.rsqrt(x1.pow(2).mean(-1, keepdim=True) + pre.eps) * pre.w.float())
+        return x1, out
+    a = _StreamRmsArgs()
+    a.T, a.W, a.f32, a.x = T, W, _f32(fmt), _ptr(x)
+    x1 = x
+    if y is not None or routed is not None:
+        x1 = torch.empty_like(x)
+        a.x_out = _ptr(x1)
+    if y is not None:
+        assert y.dtype == DTYPE[fmt] and y.is_contiguous()
+        a.y = _ptr(y)
+    if routed is not None:
+        a.ye, a.ye_ld, a.pair_row, a.pair_w, a.K = _ptr(routed.y), routed.y.stride(0), _ptr(routed.pair_row), _ptr(routed.w), routed.w.shape[1]
+    if wanted:
+        assert out.stride(1) == 1 and out.dtype == DTYPE[fmt]
+        a.out_mode, a.out, a.out_ld = (2 if raw else 1), _ptr(out), out.stride(0)
+        if pre is not None:
+            a.w, a.eps = _ptr(pre.w), pre.eps
+    _native.check(_native.lib().mb_stream_rms(C.byref(a), _stream()), f"stream_rms[T={T} W={W}]")
+    _count()
+    return x1, out
 
 
 def stream_norm(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, post=None, pre: Optional[DytNorm] = None,
@@ -226,18 +278,22 @@ def gated_norm(x: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, fmt: str, *
 
 # ----------------------------------------------------------------------------- embedding, token side input
 _native.register_optional("mb_embed_scaled", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_void_p,
-                                              C.c_void_p])
+                                              C.c_longlong, C.c_int, C.c_void_p, C.c_void_p])
 _native.register_optional("mb_side_gate", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_longlong] + [C.c_int] * 4 +
                           [C.c_void_p, C.c_int, C.c_void_p, C.c_void_p])
 
 
-def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
-    """fp32 [T, W] = table[ids] * scale."""
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 [T, W] = table[ids] * scale; ``copy`` (may be a column range) takes the same in the activation type."""
     if not table.is_cuda:
-        return table[ids.long()].float() * scale
+        x = table[ids.long()].float() * scale
+        if copy is not None:
+            copy.copy_(x)
+        return x
     M, W = ids.numel(), table.shape[1]
     out = torch.empty(M, W, dtype=torch.float32, device=table.device)
-    rc = _native.lib().mb_embed_scaled(_ptr(ids), _ptr(table), _ptr(out), M, W, table.shape[0], float(scale),
+    rc = _native.lib().mb_embed_scaled(_ptr(ids), _ptr(table), _ptr(out), M, W, table.shape[0], float(scale), _ptr(copy),
+                                       copy.stride(0) if copy is not None else 0, int(copy is not None and copy.dtype == torch.float32),
                                        _ptr(runtime(table.device).status), _stream())
     _native.check(rc, "embed_scaled")
     _count()
@@ -412,7 +468,8 @@ class _LinearAttnArgs(C.Structure):
                 ("num_slots", C.c_int), ("write_state", C.c_int), ("write_out", C.c_int), ("status", C.c_void_p),
                 ("decode", C.c_int), ("norm_w", C.c_void_p), ("gate", C.c_void_p), ("gate_ld", C.c_longlong),
                 ("sigmoid_gate", C.c_int), ("eps", C.c_float), ("scale", C.c_float), ("norm_out", C.c_void_p),
-                ("norm_out_ld", C.c_longlong)]
+                ("norm_out_ld", C.c_longlong), ("lr_a1", C.c_void_p), ("lr_a1_ld", C.c_longlong), ("lr_a2", C.c_void_p),
+                ("lr_bias", C.c_void_p), ("lr_rank", C.c_int), ("lr_c", C.c_float)]
 
 
 class _LinearChunkedArgs(C.Structure):
@@ -433,7 +490,7 @@ _chunk_ws: dict = {}
 
 def _linear_chunked(q, k, v, state, batch, H, dk, dv, log_w, decay, u, write_state):
     """Chunked kernels (csrc/linear_chunked.cu); None for shapes, layouts or sizes they do not take."""
-    if dk not in (64, 128) or dv not in (64, 128) or q.dtype != torch.bfloat16 or (log_w is None) != (u is None):
+    if dk not in (64, 128) or dv not in (64, 128) or q.dtype != torch.bfloat16 or (u is not None and log_w is None):
         return None
     if any(t.data_ptr() % 16 or t.stride(0) % 8 for t in (q, k, v)):
         return None
@@ -457,6 +514,27 @@ def _linear_chunked(q, k, v, state, batch, H, dk, dv, log_w, decay, u, write_sta
     return out
 
 
+@dataclass
+class LowRankDecay:
+    """Decays sigmoid(a2 a1 + bias)^c per token and key channel, a1 [T, rank] being their projection's first half."""
+    a1: torch.Tensor                       # activation type, may be a column range
+    a2: torch.Tensor                       # bf16 [H dk, rank]
+    bias: torch.Tensor                     # fp32 [H dk]
+    c: float
+    a2_lin: object = None                  # bf16 QuantWeight of a2: prefill-sized steps run on the tensor cores
+
+    def log(self) -> torch.Tensor:
+        """c log(sigmoid(a2 a1 + bias)), fp32 [T, H dk]."""
+        if not self.a1.is_cuda:
+            z = (self.a1.double() @ self.a2.double().t()).float() + self.bias
+            return self.c * torch.nn.functional.logsigmoid(z)
+        if self.a2_lin is not None and self.a1.shape[0] >= _DECAY_TC_MIN_ROWS:
+            from . import linear
+            return linear(act_of(self.a1.contiguous(), "bf16"), self.a2_lin, out_f32=True, log_sigmoid=(self.bias, self.c))
+        out = torch.empty(self.a1.shape[0], self.a2.shape[0], dtype=torch.float32, device=self.a1.device)
+        return gemm_simt(self.a1, self.a2, out, epilogue=7, bias=self.bias, epi_a=self.c)
+
+
 def _decode_ok(batch, dk: int, dv: int, kernel: str) -> bool:
     """The streaming decode kernel: one row per sequence, whole 16-byte vectors, heads up to 256 x 256."""
     return kernel in ("auto", "decode") and int(batch.max_q_len) == 1 and dv % 4 == 0 and max(dk, dv) <= 256
@@ -465,14 +543,16 @@ def _decode_ok(batch, dk: int, dv: int, kernel: str) -> bool:
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, *, heads: int, dk: int, dv: int,
                      fmt: str, log_w: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None,
                      u: Optional[torch.Tensor] = None, write_state: bool = True, write_out: bool = True,
-                     kernel: str = "auto", norm: Optional[dict] = None) -> Optional[torch.Tensor]:
+                     kernel: str = "auto", norm: Optional[dict] = None, low_rank: Optional[LowRankDecay] = None) -> Optional[torch.Tensor]:
     """Per head S_t = diag(w_t) S_(t-1) + k_t v_t^T over a ragged batch; w_t = ``decay`` [H], or exp(``log_w``
-    [T, H dk]). Output q_t^T S_t, or with ``u`` [H, dk] q_t^T (S_(t-1) + diag(u) k_t v_t^T). q, k, v [T, *]
+    [T, H dk]), or ``low_rank`` (computed inside the decode kernel where that serves the step). Output q_t^T S_t, or with ``u`` [H, dk] q_t^T (S_(t-1) + diag(u) k_t v_t^T). q, k, v [T, *]
     may be column ranges; state [slots, H, dk, dv] fp32. Returns fp32 [T, H dv]. ``kernel``: auto | seq |
     chunked | decode (tests). ``norm`` (keyword arguments of ``gated_norm`` with group = dv, and ``w``, ``gate``,
     ``out``): the gated per-head norm of the output goes to norm["out"], inside the decode kernel where that
     serves the step; nothing is returned then."""
     T, H = q.shape[0], heads
+    if low_rank is not None and not (q.is_cuda and _decode_ok(batch, dk, dv, kernel)):
+        log_w, low_rank = low_rank.log(), None
     if norm is not None:
         kw = dict(heads=H, dk=dk, dv=dv, fmt=fmt, log_w=log_w, decay=decay, u=u, write_state=write_state, kernel=kernel)
         if not (q.is_cuda and _decode_ok(batch, dk, dv, kernel)):
@@ -512,6 +592,11 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
                         _ptr(batch.positions), _ptr(batch.state_slots), batch.q_len.numel(), state.shape[0], int(write_state),
                         int(write_out), _ptr(runtime(dev).status))
     a.decode = int(_decode_ok(batch, dk, dv, kernel))
+    if low_rank is not None:
+        lr = low_rank
+        assert lr.a1.stride(1) == 1 and lr.a1.dtype == DTYPE[fmt] and lr.a2.is_contiguous()
+        a.lr_a1, a.lr_a1_ld, a.lr_a2, a.lr_bias, a.lr_rank, a.lr_c = (_ptr(lr.a1), lr.a1.stride(0), _ptr(lr.a2), _ptr(lr.bias),
+                                                                     lr.a2.shape[1], float(lr.c))
     if norm is not None:
         g, o = norm["gate"], norm["out"]
         assert g.stride(1) == 1 and o.stride(1) == 1 and g.dtype == o.dtype == DTYPE[fmt]
@@ -527,20 +612,30 @@ class _SimtGemmArgs(C.Structure):
     _fields_ = [("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("x_bf16", C.c_int), ("w_bf16", C.c_int), ("out_bf16", C.c_int),
                 ("X", C.c_void_p), ("ldx", C.c_longlong), ("W", C.c_void_p), ("ldw", C.c_longlong), ("out", C.c_void_p),
                 ("ldo", C.c_longlong), ("a_op", C.c_int), ("epilogue", C.c_int), ("bias", C.c_void_p), ("epi_a", C.c_float),
-                ("epi_b", C.c_float), ("epi_n", C.c_int)]
+                ("epi_b", C.c_float), ("epi_n", C.c_int), ("tile_expert", C.c_void_p), ("tile_row0", C.c_void_p), ("tile_nrows", C.c_void_p),
+                ("max_tiles", C.c_int), ("tile_rows", C.c_int), ("row_index", C.c_void_p), ("row_div", C.c_int)]
 
 
 _native.register_optional("mb_gemm_simt", [C.POINTER(_SimtGemmArgs), C.c_void_p])
 
 
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, tanh_in: bool = False, epilogue: int = 0, bias=None,
-              epi_a: float = 0.0, epi_b: float = 0.0, epi_n: int = 0) -> torch.Tensor:
+              epi_a: float = 0.0, epi_b: float = 0.0, epi_n: int = 0, grouped=None, row_index=None, row_div: int = 1) -> torch.Tensor:
+    """out = epilogue(x w^T). ``grouped`` = (tile_expert, tile_row0, tile_nrows, rows of w per expert, max_tiles,
+    tile_rows): x's rows are sorted by expert, or read as x[row_index // row_div]."""
     M, K = x.shape
     N = w.shape[0]
+    if row_index is not None:
+        M = row_index.numel()
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
     bf = torch.bfloat16
     a = _SimtGemmArgs(M, N, K, int(x.dtype == bf), int(w.dtype == bf), int(out.dtype == bf), _ptr(x), x.stride(0), _ptr(w),
                       w.stride(0), _ptr(out), out.stride(0), int(tanh_in), epilogue, _ptr(bias), float(epi_a), float(epi_b), epi_n)
+    if grouped is not None:
+        a.tile_expert, a.tile_row0, a.tile_nrows = _ptr(grouped[0]), _ptr(grouped[1]), _ptr(grouped[2])
+        a.N, a.max_tiles, a.tile_rows = grouped[3], grouped[4], grouped[5]
+    if row_index is not None:
+        a.row_index, a.row_div = _ptr(row_index), row_div
     _native.check(_native.lib().mb_gemm_simt(C.byref(a), _stream()), f"gemm_simt[M={M} N={N} K={K}]")
     _count()
     return out

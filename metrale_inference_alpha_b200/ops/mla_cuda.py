@@ -19,7 +19,7 @@ class MlaArgs(C.Structure):
         ("num_seqs", c_int), ("max_q_len", c_int), ("max_ctx", c_int), ("total_rows", c_int),
         ("H", c_int), ("block_size", c_int), ("num_blocks", c_ll), ("scale", c_float),
         ("out", c_void_p), ("ws", c_void_p), ("ws_bytes", c_size_t), ("part_tokens", c_int), ("status", c_void_p),
-        ("impl", c_int),
+        ("impl", c_int), ("split_p", c_int), ("out_bf16", c_int),
     ]
 
 
@@ -38,8 +38,10 @@ def supported(q: torch.Tensor, cache: torch.Tensor) -> bool:
 
 
 def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_len, ctx_len, *, max_q_len: int,
-                  max_ctx: int, scale: float, row_seq=None, part_tokens: int = 0, impl: int = 0) -> torch.Tensor:
-    """q [T, H, 576] bf16 -> [T, H, 512] fp32. `impl`: 0 = decode steps (one query row per sequence,
+                  max_ctx: int, scale: float, row_seq=None, part_tokens: int = 0, impl: int = 0, split_p: bool = False,
+                  out_bf16: bool = False) -> torch.Tensor:
+    """q [T, H, 576] bf16 -> [T, H, 512] fp32, or bf16 with `out_bf16`. `split_p`: the softmax weights enter the product
+    with the values as two bf16 terms (16 mantissa bits) instead of one. `impl`: 0 = decode steps (one query row per sequence,
     16 <= H <= 128) take the tcgen05 / TMEM kernel, everything else the mma.sync kernel; 1 / 2 force one."""
     from . import _count, _ptr, _stream, runtime
     L = _native.lib()
@@ -54,7 +56,7 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_
         # keep the SMs busy at small batch (a constant, so a sequence's split never depends on the batch)
         part_tokens = TC_PART_TOKENS
     rt = runtime(q.device)
-    out = torch.empty(T, H, LATENT, dtype=torch.float32, device=q.device)
+    out = torch.empty(T, H, LATENT, dtype=torch.bfloat16 if out_bf16 else torch.float32, device=q.device)
     need = L.mb_mla_ws_bytes(T, H, max_ctx, part_tokens)
     if need:
         # the head of the shared attention workspace holds the split-KV kernel's arrival counters,
@@ -70,6 +72,7 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_
     a.num_seqs, a.max_q_len, a.max_ctx, a.total_rows = q_len.numel(), max_q_len, max_ctx, T
     a.H, a.block_size, a.num_blocks, a.scale = H, cache.shape[1], cache.shape[0], scale
     a.out, a.part_tokens, a.status, a.impl = _ptr(out), part_tokens, _ptr(rt.status), impl
+    a.split_p, a.out_bf16 = int(split_p), int(out_bf16)
     a.ws, a.ws_bytes = (_ptr(rt.attn_ws) + _CNT_BYTES, rt.attn_ws.numel() - _CNT_BYTES) if need else (None, 0)
     _native.check(L.mb_mla_attention(C.byref(a), _stream()), "mla_attention")
     _count()

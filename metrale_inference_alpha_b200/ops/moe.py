@@ -30,6 +30,19 @@ class GroupedExperts:
     shared_slot: Optional[int] = None     # local expert index of a folded-in shared expert (every token routes to it)
 
 
+@dataclass
+class RouterSpec:
+    """Routing of one layer, where layers differ; the names are the model configuration's."""
+    num_experts: int
+    experts_per_token: int
+    router: str = "softmax_topk"          # softmax over the chosen ones of the biased logits
+    router_n_group: int = 1
+    router_topk_group: int = 1
+    router_renormalize: bool = True
+    router_scaling: float = 1.0
+    ffn_act: str = "swiglu"
+
+
 def stack_experts(experts) -> Optional[GroupedExperts]:
     if not experts:
         return None
@@ -55,9 +68,28 @@ def route(logits: torch.Tensor, cfg, bias=None):
     if logits.is_cuda and _native.available() and hasattr(_native.lib(), "mb_moe_route"):
         from .moe_cuda import route_cuda
         return route_cuda(logits, cfg, bias)
-    if cfg.router == "softmax":
+    if cfg.router == "softmax_topk":
+        z = logits.float() if bias is None else logits.float() + bias
+        top, idx = ref.topk_stable(z, k)
+        w = torch.softmax(top, -1)
+    elif cfg.router == "softmax":
         w, idx = ref.route_softmax_topk(logits, k, cfg.router_renormalize)
     else:
         w, idx = ref.route_sigmoid_grouped(logits, bias, k, cfg.router_n_group, cfg.router_topk_group,
                                            cfg.router_renormalize, cfg.router_scaling)
     return w.float(), idx.to(torch.int32)
+
+
+def expert_sum_ref(act, weights: torch.Tensor, idx: torch.Tensor, ge: GroupedExperts, width: int) -> torch.Tensor:
+    """CPU: sum_j weights[t, j] * expert idx[t, j] of row t over stacked (padded) SwiGLU experts; fp32 [T, width]."""
+    from . import Act, QuantWeight, linear
+    out = torch.zeros(act.M, width)
+    part = lambda w, e, n: QuantWeight(w.fmt, n, w.K, w.data[e * n:(e + 1) * n])
+    for e in range(ge.num):
+        tok, slot = torch.nonzero(idx == e, as_tuple=True)
+        if tok.numel() == 0:
+            continue
+        h = linear(Act(act.fmt, tok.numel(), act.K, act.data[tok]), part(ge.gate_up, e, ge.n_gate_up), swiglu=True)
+        y = linear(Act(act.fmt, tok.numel(), h.shape[1], h.float()), part(ge.down, e, ge.n_down), out_f32=True)
+        out.index_add_(0, tok, y[:, :width] * weights[tok, slot][:, None])
+    return out

@@ -7,9 +7,10 @@ import ctypes as C
 
 import torch
 
-from . import Act, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
+from . import Act, EPI_SWIGLU, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
 
 c = C
+ROUTER_MODE = {"softmax": 0, "sigmoid": 1, "softmax_topk": 2}
 _native.register_optional("mb_moe_route", [c.c_void_p, c.c_longlong, c.c_int, c.c_int, c.c_int, c.c_int, c.c_void_p,
                                           c.c_int, c.c_int, c.c_int, c.c_float, c.c_void_p, c.c_void_p, c.c_void_p])
 _native.register_optional("mb_moe_sort", [c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_int] + [c.c_void_p] * 6 +
@@ -43,10 +44,10 @@ def route_shared_cuda(logits: torch.Tensor, cfg, bias, shared_id: int, gate_col:
     E, K = cfg.num_experts, cfg.experts_per_token
     w = torch.empty(T, K + 1, dtype=torch.float32, device=logits.device)
     idx = torch.empty(T, K + 1, dtype=torch.int32, device=logits.device)
-    mode = 0 if cfg.router == "softmax" else 1
+    mode = ROUTER_MODE[cfg.router]
     rc = _native.lib().mb_moe_route_shared(_ptr(logits), logits.stride(0), T, E, K, mode, _ptr(bias),
-                                           cfg.router_n_group if mode else 1, cfg.router_topk_group if mode else 1,
-                                           int(cfg.router_renormalize), float(cfg.router_scaling if mode else 1.0),
+                                           cfg.router_n_group if mode == 1 else 1, cfg.router_topk_group if mode == 1 else 1,
+                                           int(cfg.router_renormalize), float(cfg.router_scaling if mode == 1 else 1.0),
                                            _ptr(w), _ptr(idx), shared_id, gate_col, _stream())
     _native.check(rc, "moe_route_shared")
     _count()
@@ -58,10 +59,10 @@ def route_cuda(logits: torch.Tensor, cfg, bias=None):
     K = cfg.experts_per_token
     w = torch.empty(T, K, dtype=torch.float32, device=logits.device)
     idx = torch.empty(T, K, dtype=torch.int32, device=logits.device)
-    mode = 0 if cfg.router == "softmax" else 1
+    mode = ROUTER_MODE[cfg.router]
     rc = _native.lib().mb_moe_route(_ptr(logits), logits.stride(0), T, E, K, mode, _ptr(bias),
-                                    cfg.router_n_group if mode else 1, cfg.router_topk_group if mode else 1,
-                                    int(cfg.router_renormalize), float(cfg.router_scaling if mode else 1.0),
+                                    cfg.router_n_group if mode == 1 else 1, cfg.router_topk_group if mode == 1 else 1,
+                                    int(cfg.router_renormalize), float(cfg.router_scaling if mode == 1 else 1.0),
                                     _ptr(w), _ptr(idx), _stream())
     _native.check(rc, "moe_route")
     _count()
@@ -135,14 +136,22 @@ def gather_act(a: Act, sp: SortedPairs) -> Act:
     return out
 
 
-def grouped_ffn(cfg, a: Act, weights: torch.Tensor, idx: torch.Tensor, w, finish=None) -> torch.Tensor:
-    """Routed experts for all tokens: fp32 [T, hidden] = sum_j weight_j * expert_j(x). With
-    `finish` = (shared bf16 [T, hidden] | None, gate logit fp32 [T, 1] | None, residual bf16 | None)
-    the combine kernel also adds the (sigmoid-gated) shared expert and the residual and returns
-    the bf16 block output."""
+def grouped_pairs(cfg, a: Act, idx: torch.Tensor, w):
+    """Every (token, slot) pair's expert output, in expert order: (fp32 [pairs, hidden], the pairs' places)."""
     ge = w.grouped
     T = a.M
     per_expert = max(1, (T * cfg.experts_per_token) // max(1, ge.num))
+    if ge.gate_up.fmt == "fp32" or ge.gate_up.K % 8:
+        # 32-bit models, and bf16 rows that are not whole 16-byte vectors: the CUDA-core GEMM, which reads the
+        # token rows through the pairs' index itself
+        from .mixers import gemm_simt
+        sp = SortedPairs(idx, w.expert_lo, ge.num, 16 if per_expert <= 16 else 64)
+        g = lambda n: (sp.tile_expert, sp.tile_row0, sp.tile_nrows, n, sp.max_tiles, sp.tile_rows)
+        assert ge.interleaved
+        h = torch.empty(sp.pairs, ge.n_gate_up // 2, dtype=a.data.dtype, device=a.data.device)
+        gemm_simt(a.data, ge.gate_up.data, h, epilogue=EPI_SWIGLU, grouped=g(ge.n_gate_up), row_index=sp.row_pair, row_div=sp.K)
+        y = torch.empty(sp.pairs, ge.n_down, dtype=torch.float32, device=h.device)
+        return gemm_simt(h, ge.down.data, y, grouped=g(ge.n_down)), sp
     nvfp4 = ge.gate_up.fmt == "nvfp4"
     # NVFP4: every token tile starts on a 128-row block of scale factors and takes its first tile_rows rows
     tile_rows = 16 if per_expert <= 16 else (32 if per_expert <= 32 else (64 if per_expert <= 64 or not nvfp4 else 128))
@@ -155,14 +164,24 @@ def grouped_ffn(cfg, a: Act, weights: torch.Tensor, idx: torch.Tensor, w, finish
         h = row_op(linear(xa, ge.gate_up, grouped=g(ge.n_gate_up)), fmt_d, IN_RELU2, row_index=live)[0]
     elif ge.interleaved:
         act = linear(xa, ge.gate_up, swiglu=True, grouped=g(ge.n_gate_up))
-        h = row_op(act, fmt_d, scale_pad=64, row_index=live)[0]
+        h = Act("bf16", act.shape[0], act.shape[1], act, bf16=act) if fmt_d == "bf16" else row_op(act, fmt_d, scale_pad=64, row_index=live)[0]
     else:
         h = row_op(linear(xa, ge.gate_up, grouped=g(ge.n_gate_up)), fmt_d, IN_SILU_MUL, scale_pad=64, row_index=live)[0]
     if cfg.ffn_act == "relu2" and h.fmt == "fp8_g128" and h.scale.shape[1] < h.M + 64:
         pad = torch.empty(h.scale.shape[0], h.M + 64, dtype=torch.float32, device=h.scale.device)
         pad[:, :h.scale.shape[1]] = h.scale
         h.scale = pad
-    y = linear(h, ge.down, out_f32=True, grouped=g(ge.n_down))
+    return linear(h, ge.down, out_f32=True, grouped=g(ge.n_down)), sp
+
+
+def grouped_ffn(cfg, a: Act, weights: torch.Tensor, idx: torch.Tensor, w, finish=None) -> torch.Tensor:
+    """Routed experts for all tokens: fp32 [T, hidden] = sum_j weight_j * expert_j(x). With
+    `finish` = (shared bf16 [T, hidden] | None, gate logit fp32 [T, 1] | None, residual bf16 | None)
+    the combine kernel also adds the (sigmoid-gated) shared expert and the residual and returns
+    the bf16 block output."""
+    ge = w.grouped
+    T = a.M
+    y, sp = grouped_pairs(cfg, a, idx, w)
     if finish is not None:
         shared, gate, residual = finish
         out = torch.empty(T, ge.n_down, dtype=torch.bfloat16, device=y.device)

@@ -363,7 +363,7 @@ def mamba2_step(h, x, dt, A_log, B, Cm, Dp, dt_bias, dt_min: float = 0.0, dt_max
 def route_softmax_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
     """softmax over experts, top-k, ties -> lower index (kernels/gb10/common/moe_topk.cu)."""
     p = torch.softmax(logits.float(), dim=-1)
-    w, idx = _topk_stable(p, k)
+    w, idx = topk_stable(p, k)
     if renormalize:
         w = w / w.sum(-1, keepdim=True)
     return w, idx
@@ -382,19 +382,19 @@ def route_sigmoid_grouped(logits, bias, k: int, n_group: int = 1, topk_group: in
     if n_group > 1:
         gs = sel.view(T, n_group, E // n_group)
         gscore = gs.topk(2, dim=-1).values.sum(-1)
-        _, gidx = _topk_stable(gscore, topk_group)
+        _, gidx = topk_stable(gscore, topk_group)
         gmask = torch.zeros(T, n_group, dtype=torch.bool, device=sel.device)
         gmask.scatter_(1, gidx, True)
         sel = sel.masked_fill(~gmask[:, :, None].expand(T, n_group, E // n_group).reshape(T, E),
                               float("-inf"))
-    _, idx = _topk_stable(sel, k)
+    _, idx = topk_stable(sel, k)
     w = s.gather(1, idx)
     if renormalize:
         w = w / (w.sum(-1, keepdim=True) + 1e-20)
     return w * scaling, idx
 
 
-def _topk_stable(x: torch.Tensor, k: int):
+def topk_stable(x: torch.Tensor, k: int):
     """top-k with ties resolved toward the lower index."""
     order = torch.sort(x, dim=-1, descending=True, stable=True)
     return order.values[..., :k], order.indices[..., :k]

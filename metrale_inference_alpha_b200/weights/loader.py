@@ -132,6 +132,7 @@ class MoeW:
     router_ext: Optional[QuantWeight] = None               # router rows + the shared expert's gate row (shared expert folded into `grouped`)
     paged: Optional[object] = None                         # storage.expert_store.PagedExperts: the experts live in a store and are paged into an arena
     paged_layer: int = 0                                   # this layer's index in that store
+    spec: Optional[object] = None                          # ops.moe.RouterSpec of models whose layers route differently (None: the model configuration's)
 
 
 @dataclass
@@ -193,6 +194,47 @@ class MlaW:
     idx_k: Optional[QuantWeight] = None          # hidden -> Di
     idx_k_norm: Optional[torch.Tensor] = None    # LayerNorm weight | bias, fp32 [2, Di]
     idx_w: Optional[QuantWeight] = None          # hidden -> Hi (head weights), bf16
+
+
+@dataclass
+class LatentW:
+    """Latent attention of a 32-bit-stream model: sizes, scale and rotation are the layer's own."""
+    in_proj: QuantWeight = None          # rows: query latent | key-value latent | rotated key part (| router)
+    q_norm: torch.Tensor = None          # bf16 [q_rank]
+    kv_norm: torch.Tensor = None         # bf16 [kv_rank]
+    uq: QuantWeight = None               # query latent -> heads of [dim unrotated, rot_dim rotated]
+    w_uk: torch.Tensor = None            # [H, dim, kv_rank]
+    w_uv: torch.Tensor = None            # [H, vdim, kv_rank]
+    heads: int = 0
+    dim: int = 0
+    rot_dim: int = 0
+    vdim: int = 0
+    kv_rank: int = 0
+    q_rank: int = 0
+    scale: float = 1.0
+    rot_base: float = 10000.0
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass
+class GlaW:
+    """Gated linear attention: a low-rank, per-channel decay sigmoid(.)^(1 / tau)."""
+    in_proj: QuantWeight = None          # rows: q | k | v | g | first half of the decay projection (| zero rows)
+    a2: torch.Tensor = None              # bf16 [H dim, rank]
+    a2_lin: Optional[QuantWeight] = None # the same as a GEMM operand (rows of whole 16-byte vectors)
+    a2_bias: torch.Tensor = None         # fp32 [H dim]
+    norm: torch.Tensor = None            # bf16 [H vdim]: the head norm's weight, repeated
+    heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    tau: float = 1.0
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
 
 
 @dataclass
@@ -266,6 +308,7 @@ class LayerW:
     hc_attn: Optional[tuple] = None              # hyper-connection site in front of the mixer: (fn bf16, scale fp32 [3], base fp32)
     hc_ffn: Optional[tuple] = None               # ... and in front of the feed-forward block
     side: Optional[TokenSideW] = None            # per-layer token side input, after the feed-forward block
+    out: Optional[QuantWeight] = None            # mixer and feed-forward side by side: both output projections, stacked along their inputs
 
 
 @dataclass
@@ -287,6 +330,8 @@ class ModelW:
     vocab_lo: int = 0
     vocab_hi: int = 0
     side_embed: Optional[torch.Tensor] = None      # bf16 [V, layers * side dim]
+    loop_in: Optional[QuantWeight] = None          # looped layers: [stream | embedding output] -> stream, ahead of every pass
+    loop_step: Optional[torch.Tensor] = None       # fp32 [times, H], added in front of each pass
 
     def nbytes(self) -> int:
         n = 0
@@ -453,6 +498,9 @@ class Loader:
         if c.arch == "fabulix":
             from .fabulix import load_fabulix
             return load_fabulix(self)
+        if c.arch == "finelix":
+            from .finelix import load_finelix
+            return load_finelix(self)
         m = ModelW()
         m.embed = self.vec("model.embed_tokens.weight")
         m.final_norm = self.vec("model.norm.weight")

@@ -102,6 +102,12 @@ def _seed_for(name: str, seed: int) -> int:
     return int.from_bytes(hashlib.sha256(f"{seed}:{name}".encode()).digest()[:7], "little")
 
 
+def spec_shapes(c: ModelConfig) -> dict:
+    """Tensors of a model whose sizes are per layer: name -> (shape, kind of synthetic values)."""
+    from . import fabulix, finelix
+    return {"fabulix": fabulix, "finelix": finelix}[c.arch].tensor_shapes(c)
+
+
 class SyntheticSource(TensorSource):
     """Random N(0, std) weights in HF checkpoint layout for `cfg`. Each tensor is a pure
     function of (seed, name), so every rank of a tensor-parallel job sees the same checkpoint."""
@@ -158,9 +164,8 @@ class SyntheticSource(TensorSource):
         c = self.cfg
         if c.arch == "nemotron_h":
             return self._describe_nemotron()
-        if c.arch == "fabulix":
-            from .fabulix import tensor_shapes
-            for name, (shape, kind) in tensor_shapes(c).items():
+        if c.stream32:
+            for name, (shape, kind) in spec_shapes(c).items():
                 self._vec(name, shape, kind)
             return
         self._lin("model.embed_tokens", c.vocab_size, c.hidden_size, quant=False)
