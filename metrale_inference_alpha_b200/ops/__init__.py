@@ -430,7 +430,7 @@ def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu=False,
     elif bias is not None:
         y = y + bias
     elif log_sigmoid is not None:
-        y = log_sigmoid[1] * torch.nn.functional.logsigmoid(y + log_sigmoid[0])
+        y = log_sigmoid[1] * ref.log_sigmoid(y + log_sigmoid[0])
     if clamp_glu is not None:
         alpha, limit = clamp_glu
         g, u = y[:, 0::2].clamp(max=limit), y[:, 1::2].clamp(-limit, limit)

@@ -527,7 +527,7 @@ class LowRankDecay:
         """c log(sigmoid(a2 a1 + bias)), fp32 [T, H dk]."""
         if not self.a1.is_cuda:
             z = (self.a1.double() @ self.a2.double().t()).float() + self.bias
-            return self.c * torch.nn.functional.logsigmoid(z)
+            return self.c * ref.log_sigmoid(z)
         if self.a2_lin is not None and self.a1.shape[0] >= _DECAY_TC_MIN_ROWS:
             from . import linear
             return linear(act_of(self.a1.contiguous(), "bf16"), self.a2_lin, out_f32=True, log_sigmoid=(self.bias, self.c))

@@ -360,6 +360,11 @@ def mamba2_step(h, x, dt, A_log, B, Cm, Dp, dt_bias, dt_min: float = 0.0, dt_max
 
 
 # ----------------------------------------------------------------------------- MoE routing
+def log_sigmoid(z: torch.Tensor) -> torch.Tensor:
+    """log(sigmoid(z)) without cancellation on either side."""
+    return z.clamp(max=0.0) - torch.log1p(torch.exp(-z.abs()))
+
+
 def route_softmax_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
     """softmax over experts, top-k, ties -> lower index (kernels/gb10/common/moe_topk.cu)."""
     p = torch.softmax(logits.float(), dim=-1)
