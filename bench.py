@@ -28,7 +28,7 @@ What is measured (all as the max over ranks; rank 0 prints ONE JSON line):
            same K steps as `value`, driven through `step()`.
   config.ladder   the same end-to-end measurement for every rung 1..128 (`--no-ladder` skips it).
 
-`--mixers` runs another workload instead: the Fabulix decoder beside an equal-size hybrid.
+`--mixers` runs another workload instead: the Fabulix (or, with `--design finelix`, the Finelix) decoder beside an equal-size hybrid.
 """
 from __future__ import annotations
 
@@ -178,6 +178,8 @@ def main() -> int:
     ap.add_argument("--mixers", default="", choices=["", "all", "kernels", "models"],
                     help="instead of the headline run: the Fabulix decoder's kernels beside the like kernels of an equal-size "
                          "attention / Kimi-delta hybrid, and both models' prefill and decode throughput (1 GPU; benchmarks/mixer_bench.py)")
+    ap.add_argument("--design", default="fabulix", choices=["fabulix", "finelix"],
+                    help="--mixers: the decoder that is measured (finelix: beside an MLA / Kimi-delta hybrid with experts)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
@@ -185,7 +187,7 @@ def main() -> int:
         from benchmarks.mixer_bench import run as mixer_run
         sampler = ClockSampler(0)
         sampler.start()
-        res = mixer_run(args.mixers)
+        res = mixer_run(args.mixers, args.design)
         print(json.dumps({"bench": "mixers", "l2": "flushed before every call", "dtype": "bf16", "data": "random weights and inputs",
                           **res, "clocks": sampler.stop()}), flush=True)
         return 0

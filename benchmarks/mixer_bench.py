@@ -1,8 +1,9 @@
 #!/usr/bin/env python
-"""The kernels of the Fabulix decoder next to the like kernels of the engine's attention / Kimi-delta-attention /
-Mamba2 hybrids at equal size, each with its distance from the roofline (measured copy bandwidth and measured
-bf16 GEMM rate), and the throughput of a whole model next to an equal-size hybrid. CUDA events around one call,
-L2 flushed by a 512 MB write before every call, median of the timed calls. Reached as `bench.py --mixers`.
+"""The kernels of the Fabulix or Finelix decoder next to the like kernels of the engine's attention / MLA /
+Kimi-delta-attention / Mamba2 hybrids at equal size, each with its distance from the roofline (measured copy
+bandwidth and measured bf16 GEMM rate), and the throughput of a whole model next to an equal-size hybrid. CUDA
+events around one call, L2 flushed by a 512 MB write before every call, median of the timed calls. Reached as
+`bench.py --mixers`, `--design` naming the decoder.
 """
 from __future__ import annotations
 
@@ -56,10 +57,9 @@ def rnd(*s, dtype=BF, std=1.0):
     return (torch.randn(*s, device=DEV) * std).to(dtype)
 
 
-def kernels(W=2560, H=20, G=4, D=128, FF=6912, R=64, side=128):
-    """Rows: (shape, mechanism, new us, new bytes, new flops, like name, like us, like bytes, like flops)."""
-    t, rows, bw, fl = Timer(), [], *peaks()
-    HD = H * D
+def pairing(rows):
+    """pair(shape, name, new, bytes, flops, like name, like, bytes, flops): times both and appends one row."""
+    t, bw, fl = Timer(), *peaks()
 
     def pair(shape, name, new, nb, nf, like_name, like, lb, lf):
         a, b = t(new), t(like)
@@ -67,8 +67,17 @@ def kernels(W=2560, H=20, G=4, D=128, FF=6912, R=64, side=128):
         rows.append({"shape": shape, "kernel": name, "us": round(a * 1e6, 1), "x_roofline": round(a / ra, 2), "like": like_name,
                      "like_us": round(b * 1e6, 1), "like_x_roofline": round(b / rb, 2), "ratio": round(a / ra / (b / rb), 2)})
         print(rows[-1], file=sys.stderr, flush=True)
+    return pair
 
-    for shape, lens, start in (("decode 128 seqs, ctx 1024", [1] * 128, 1023), ("prefill 1 x 4096", [4096], 0), ("prefill 8 x 1024", [1024] * 8, 0)):
+
+SHAPES = (("decode 128 seqs, ctx 1024", [1] * 128, 1023), ("prefill 1 x 4096", [4096], 0), ("prefill 8 x 1024", [1024] * 8, 0))
+
+
+def kernels(W=2560, H=20, G=4, D=128, FF=6912, R=64, side=128):
+    """Rows: (shape, mechanism, new us, new bytes, new flops, like name, like us, like bytes, like flops)."""
+    rows = []
+    HD, pair = H * D, pairing(rows)
+    for shape, lens, start in SHAPES:
         b, nblk = batch(lens, start)
         T, S = sum(lens), len(lens)
         ctx = lens[0] + start
@@ -146,6 +155,135 @@ def kernels(W=2560, H=20, G=4, D=128, FF=6912, R=64, side=128):
     return rows
 
 
+def finelix_kernels(W=2560, H=20, D=128, FF=6912, rank=16, Hl=32, dim=128, R=64, dv=128, L=512, QR=1536, E=64, top=6, EF=1024):
+    """The same rows for Finelix: the like kernels are those of MLA + Kimi-delta hybrids with experts."""
+    from metrale_inference_alpha_b200.ops import latent as lt, mla_cuda, moe as moe_ops, moe_cuda
+    from metrale_inference_alpha_b200.weights.loader import MoeW
+    rows = []
+    HD, pair, lay = H * D, pairing(rows), lt.latent_row(L, R, "bf16")
+    f32 = torch.float32
+    for shape, lens, start in SHAPES:
+        b, nblk = batch(lens, start)
+        T, S, ctx = sum(lens), len(lens), lens[0] + start
+        # ---- the stream
+        x, y, xb, wv = rnd(T, W, dtype=f32), rnd(T, W), rnd(T, W), rnd(W)
+        n1 = mx.RmsNorm(wv, 1e-5)
+        pair(shape, "stream_rms (add + norm)", lambda: mx.stream_rms(x, "bf16", y=y, pre=n1), T * W * 12, 0, "residual + RMSNorm",
+             lambda: ops.row_op(xb, "bf16", ops.IN_RMSNORM, w=wv, residual=y, write_residual=True), T * W * 8, 0)
+        # ---- experts
+        gu, dn = QuantWeight("bf16", E * 2 * EF, W, rnd(E * 2 * EF, W, std=0.02)), QuantWeight("bf16", E * W, EF, rnd(E * W, EF, std=0.02))
+        w = MoeW(grouped=moe_ops.GroupedExperts(gu, dn, E, 2 * EF, W, True), bias=rnd(E, dtype=f32), spec=moe_ops.RouterSpec(E, top))
+        act, logits = mx.act_of(rnd(T, W), "bf16"), rnd(T, E, dtype=f32)
+        soft = moe_ops.RouterSpec(E, top, "softmax")
+        pair(shape, "route (biased, over the chosen)", lambda: moe_ops.route(logits, w.spec, w.bias), T * (E + 2 * top) * 4, 0, "route (softmax)",
+             lambda: moe_ops.route(logits, soft), T * (E + 2 * top) * 4, 0)
+        wt, idx = moe_ops.route(logits, w.spec, w.bias)
+        hit = len(set(idx.flatten().tolist()))
+        eb, ef = hit * 3 * EF * W * 2 + T * W * 2 + T * top * (W * 4 + 2 * EF * 2), T * top * 6 * EF * W
+        pair(shape, "experts, unsummed", lambda: moe_cuda.grouped_pairs(w.spec, act, idx, w), eb, ef, "experts + combine + residual",
+             lambda: moe_cuda.grouped_ffn(w.spec, act, wt, idx, w, finish=(y, None, xb)), eb + T * W * 6, ef)
+        ye, sp = moe_cuda.grouped_pairs(w.spec, act, idx, w)
+        routed = mx.Routed(ye, sp.pair_row, wt)
+
+        def combine():
+            out = torch.empty(T, W, dtype=BF, device=DEV)
+            ops._native.lib().mb_moe_finish(ops._ptr(ye), ye.stride(0), ops._ptr(sp.pair_row), ops._ptr(wt), T, top, W, ops._ptr(y), W, None, 0,
+                                            ops._ptr(xb), ops._ptr(out), ops._stream())
+        pair(shape, "stream_rms with the experts' sum", lambda: mx.stream_rms(x, "bf16", y=y, routed=routed, pre=n1), T * W * (12 + 4 * top), 0,
+             "expert combine", combine, T * W * (6 + 4 * top), 0)
+        del gu, dn, w, ye, sp, routed
+        # ---- latent attention
+        cos, sin = ref.rope_tables(8192, R, 1e4, device=DEV)
+        cache, p = rnd(nblk, 16, 1, lay.row), rnd(T, QR + L + R + E, dtype=f32)
+        qn, kn = rnd(QR), rnd(L)
+        kw = dict(q_rank=QR, L=L, R=R, q_w=qn, kv_w=kn, eps=1e-5, cos=cos, sin=sin, positions=b.positions, slots=b.slot_mapping, cache=cache, lay=lay)
+        qa = rnd(T, QR)
+        pair(shape, "latent_norm (+ cache row)", lambda: lt.norm_and_cache(p, "bf16", **kw), T * ((QR + L + R) * 4 + QR * 2 + lay.row * 2), 0,
+             "RMSNorm of the query latent", lambda: ops.row_op(qa, "bf16", ops.IN_RMSNORM, w=qn), T * QR * 4, 0)
+        q, uk, ckv = rnd(T, Hl * (dim + R)), rnd(Hl, dim, L, std=0.05), rnd(T, L + R)
+        q3 = q.view(T, Hl, dim + R)
+
+        def like_query():
+            ql = torch.bmm(q3[..., :dim].transpose(0, 1), uk)
+            return mla_cuda.prepare(q3, ql, ckv, kn, cos, sin, b.positions, b.slot_mapping, cache, dim, 1e-5)
+        nb = T * Hl * (dim + R + lay.row) * 2 + uk.numel() * 2
+        pair(shape, "absorbed queries", lambda: lt.absorbed_query(q, uk, "bf16", H=Hl, dim=dim, R=R, cos=cos, sin=sin, positions=b.positions, lay=lay),
+             nb, 2 * T * Hl * dim * L, "absorbed queries + cache row", like_query, nb + T * (L + R) * 4, 2 * T * Hl * dim * L)
+        qq, uv = rnd(T, Hl, lay.row, std=0.3), rnd(Hl, dv, L, std=0.05)
+        out = torch.empty(T, Hl * dv, dtype=BF, device=DEV)
+        akw = dict(max_q_len=b.max_q_len, max_ctx=b.max_ctx, scale=0.07)
+        pairs_ = sum(n * start + n * (n + 1) / 2 for n in lens)
+        nb, nf = S * ctx * lay.row * 2 + T * Hl * (lay.row * 2 + L * 2), 2 * Hl * (lay.row + L) * pairs_
+
+        def like_att():
+            o = mla_cuda.mla_attention(qq, cache, b.block_table, b.q_start, b.q_len, b.ctx_len, **akw)
+            return torch.bmm(o.to(BF).transpose(0, 1), uv.transpose(1, 2)).transpose(0, 1).reshape(T, Hl * dv)
+        nb, nf = nb + uv.numel() * 2 + T * Hl * (L + dv) * 2, nf + 2 * T * Hl * L * dv
+        pair(shape, "latent attention + value product", lambda: lt.attention(qq, cache, b, uv, 0.07, "bf16", lay, out), nb, nf,
+             "MLA attention + value product", like_att, nb, nf)
+        del qq, q, cache
+        # ---- gated linear attention
+        z = rnd(T, 4 * HD + rank)
+        q, k, v, g, a1 = z[:, :HD], z[:, HD:2 * HD], z[:, 2 * HD:3 * HD], z[:, 3 * HD:4 * HD], z[:, 4 * HD:]
+        a2, bias, gw = rnd(HD, rank, std=0.1), rnd(HD, dtype=f32), rnd(HD)
+        lr = mx.LowRankDecay(a1, a2, bias, 1 / 16, QuantWeight("bf16", HD, rank, a2))
+        ssm, out = torch.zeros(S + 2, H, D, D, device=DEV), torch.empty(T, HD, dtype=BF, device=DEV)
+        sb = 2 * S * H * D * D * 4
+        conv, graw, braw = rnd(T, 3 * HD, dtype=f32), rnd(T, HD, dtype=f32), rnd(T, H, dtype=f32)
+        A, dtb = torch.zeros(H, device=DEV), torch.zeros(HD, device=DEV)
+        nw = rnd(D, dtype=f32)
+        norm = dict(w=gw, gate=g, gate_act="silu", eps=1e-5, scale=1.0, out=out)
+        pair(shape, "gated linear attention (decay, recurrence, norm)",
+             lambda: mx.linear_attention(q, k, v, ssm, b, heads=H, dk=D, dv=D, fmt="bf16", low_rank=lr, norm=norm), T * HD * 10 + T * rank * 2 + sb, 0,
+             "Kimi delta attention (recurrence, norm)",
+             lambda: rops.kda_recurrence(conv, graw, braw, A, dtb, -5.0, ssm, b, heads=H, dim=D, norm=(nw, g, 1e-5)), T * HD * 20 + sb, 0)
+        zb, a2q = mx.act_of(rnd(T, rank), "bf16"), QuantWeight("bf16", HD, rank, a2)
+        pair(shape, "log decay (log sigmoid / tau)", lr.log, T * HD * 4 + T * rank * 2 + HD * rank * 2, 0, "low-rank decay GEMM, bf16",
+             lambda: ops.linear(zb, a2q, out_f32=True), T * HD * 4 + T * rank * 2 + HD * rank * 2, 0)
+        del conv, graw
+        # ---- matrix products with their epilogues
+        gu = QuantWeight("bf16", 2 * FF, W, rnd(2 * FF, W, std=0.02))
+        cat = torch.empty(T, HD + FF, dtype=BF, device=DEV)
+        gb, gf = (2 * FF * W + T * W + T * FF) * 2, 2 * T * 2 * FF * W
+        pair(shape, "GEMM + tanh-GELU GLU", lambda: ops.linear(act, gu, geglu=True, out=cat[:, HD:]), gb, gf, "GEMM + SwiGLU",
+             lambda: ops.linear(act, gu, swiglu=True), gb, gf)
+        wo, wm, wd = (QuantWeight("bf16", W, n, rnd(W, n, std=0.02)) for n in (HD + FF, HD, FF))
+        ca, cm, cd = (mx.act_of(rnd(T, n), "bf16") for n in (HD + FF, HD, FF))
+        gb, gf = ((HD + FF) * (W + T) + T * W) * 2, 2 * T * (HD + FF) * W
+        pair(shape, "joint output GEMM", lambda: ops.linear(ca, wo), gb, gf, "o_proj + down_proj, residual", lambda:
+             ops.linear(cd, wd, residual=ops.linear(cm, wm, residual=xb)), gb + T * W * 6, gf)
+        wi, pa, step = QuantWeight("bf16", W, 2 * W, rnd(W, 2 * W, std=0.02)), mx.act_of(rnd(T, 2 * W), "bf16"), rnd(W, dtype=f32)
+        gb, gf = 2 * W * (W + T) * 2 + T * W * 4, 4 * T * W * W
+        pair(shape, "pass entry GEMM (32-bit out + step)", lambda: ops.linear(pa, wi, out_f32=True, bias=step), gb, gf, "GEMM, 32-bit out",
+             lambda: ops.linear(pa, wi, out_f32=True), gb, gf)
+        ids, et = torch.randint(0, 60000, (T,), dtype=torch.int32, device=DEV), rnd(60000, W)
+        pr = torch.empty(T, 2 * W, dtype=BF, device=DEV)
+        pair(shape, "scaled embedding (+ copy)", lambda: mx.embed_scaled(ids, et, 2.0, pr[:, W:]), T * W * 8, 0, "embedding gather",
+             lambda: ops.embed(ids, et), T * W * 4, 0)
+    return rows
+
+
+def finelix_models():
+    """(label, name -> configuration): Finelix, the same with its first two layers looped three times, and a hybrid of
+    equal size: MLA and experts where Finelix has latent attention, Kimi delta attention and SwiGLU elsewhere; bf16."""
+    from metrale_inference_alpha_b200.config.model_config import ModelConfig, preset
+    for label, kw in (("1B-like layers", dict(width=2048, heads=16, lin_heads=16, ff=5632, experts=32, top=4, expert_ff=768, shared_ff=1536, vocab=32768)),
+                      ("3B-like layers", {})):
+        looped = preset("finelix-3b", num_layers=6, **kw)
+        f = looped.scaled(loop=None)
+        m, mlp = f.layer_specs[1]["mixer"], f.layer_specs[1]["mlp"]
+        g = f.layer_specs[0]["mixer"]
+        h = ModelConfig(name="mla-kda-hybrid", arch="deepseek_mla", vocab_size=f.vocab_size, hidden_size=f.hidden_size, num_layers=6,
+                        num_heads=m["heads"], num_kv_heads=m["heads"], head_dim=m["dim"] + m["rot_dim"], rope_theta=10000.0,
+                        layer_types=["mla" if t == "latent" else "kda" for t in f.layer_types], ffn_types=list(f.ffn_types),
+                        dense_intermediate_size=f.intermediate_size, intermediate_size=f.intermediate_size, q_lora_rank=m["q_rank"],
+                        kv_lora_rank=m["kv_rank"], qk_nope_dim=m["dim"], qk_rope_dim=m["rot_dim"], v_head_dim=m["vdim"],
+                        num_experts=mlp["router"]["experts"], experts_per_token=mlp["router"]["top"], moe_intermediate_size=mlp["expert"]["ff"],
+                        num_shared_experts=mlp["shared"]["ff"] // mlp["expert"]["ff"], router="sigmoid", kda_heads=g["heads"], kda_head_dim=g["dim"],
+                        kda_gate_rank=64, weight_format="bf16", kv_dtype="bf16", max_position=16384)
+        yield label, {"finelix": f, "MLA / Kimi-delta hybrid": h, "finelix, two layers looped three times": looped}
+
+
 def models():
     """(label, Fabulix configuration, hybrid of equal size: attention where Fabulix runs two mixers in parallel,
     Kimi delta attention where it runs lightning attention; SwiGLU; bf16)."""
@@ -160,7 +298,7 @@ def models():
                         layer_types=["kda" if t == "lightning" else "attention" for t in f.layer_types], ffn_types=["dense"] * f.num_layers,
                         intermediate_size=f.intermediate_size, kda_heads=a["heads"], kda_head_dim=128, kda_gate_rank=64, tie_embeddings=True,
                         norm_plus_one=True, weight_format="bf16", kv_dtype="bf16", max_position=16384)
-        yield label, f, h
+        yield label, {"fabulix": f, "attention / Kimi-delta hybrid": h}
 
 
 def throughput(cfg, decode_batches=(1, 32, 128), prefills=((1, 4096), (8, 1024)), ctx=1024):
@@ -198,15 +336,15 @@ def throughput(cfg, decode_batches=(1, 32, 128), prefills=((1, 4096), (8, 1024))
     return out
 
 
-def run(what="all"):
-    res = {}
+def run(what="all", design="fabulix"):
+    res = {"design": design}
     if what in ("all", "kernels"):
-        res["kernels"] = kernels()
+        res["kernels"] = {"fabulix": kernels, "finelix": finelix_kernels}[design]()
     if what in ("all", "models"):
         res["models"] = {}
-        for label, f, h in models():
+        for label, cfgs in {"fabulix": models, "finelix": finelix_models}[design]():
             res["models"][label] = {}
-            for name, cfg in (("fabulix", f), ("attention / Kimi-delta hybrid", h)):
+            for name, cfg in cfgs.items():
                 res["models"][label][name] = throughput(cfg)
                 print(label, name, res["models"][label][name], file=sys.stderr, flush=True)
                 torch.cuda.empty_cache()
@@ -215,4 +353,4 @@ def run(what="all"):
 
 
 if __name__ == "__main__":
-    print(json.dumps(run(sys.argv[1] if len(sys.argv) > 1 else "all")))
+    print(json.dumps(run(*sys.argv[1:3])))

@@ -26,7 +26,19 @@ __device__ __forceinline__ float gelu_tanh(float z) { return z * sigmoid_exact(1
 __device__ __forceinline__ float geglu_fast(float gate, float up) {
   return __fdividef(gate * up, 1.f + __expf(-1.5957691216057308f * (gate + 0.044715f * gate * gate * gate)));
 }
-// log(sigmoid(z)), without cancellation on either side
-__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// log(sigmoid(z)) = min(z, 0) - log(1 + u), u = exp(-|z|), without cancellation on either side: with s = u / (2 + u) <= 1/3,
+// log(1 + u) = 2 atanh(s), its power series to s^15
+__device__ __forceinline__ float log_sigmoid(float z) {
+  const float u = __expf(-fabsf(z)), s = __fdividef(u, 2.f + u), q = s * s;
+  float r = 1.f / 15.f;
+  r = fmaf(r, q, 1.f / 13.f);
+  r = fmaf(r, q, 1.f / 11.f);
+  r = fmaf(r, q, 1.f / 9.f);
+  r = fmaf(r, q, 1.f / 7.f);
+  r = fmaf(r, q, 1.f / 5.f);
+  r = fmaf(r, q, 1.f / 3.f);
+  r = fmaf(r, q, 1.f);
+  return fminf(z, 0.f) - 2.f * s * r;
+}
 
 }  // namespace mb

@@ -43,7 +43,36 @@ struct NormParams {
   uint32_t* status;
 };
 
-template <typename TX, typename T>
+// VEC consecutive elements <-> floats (VEC is 1 or 4; 4 needs the natural vector alignment)
+template <int VEC, typename T>
+__device__ __forceinline__ void ldn(const T* p, float* o) {
+  if constexpr (VEC == 1) {
+    o[0] = ldv(p);
+  } else if constexpr (sizeof(T) == 2) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+  } else {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
+  }
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void stn(T* p, const float* o) {
+  if constexpr (VEC == 1) {
+    stv(p, o[0]);
+  } else if constexpr (sizeof(T) == 2) {
+    uint2 v;
+    *reinterpret_cast<__nv_bfloat162*>(&v.x) = __floats2bfloat162_rn(o[0], o[1]);
+    *reinterpret_cast<__nv_bfloat162*>(&v.y) = __floats2bfloat162_rn(o[2], o[3]);
+    *reinterpret_cast<uint2*>(p) = v;
+  } else {
+    *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]);
+  }
+}
+
+template <int VEC, typename TX, typename T>
 __global__ void __launch_bounds__(256) latent_norm_kernel(const NormParams p) {
   __shared__ float red[32];
   const int t = blockIdx.x, tid = threadIdx.x;
@@ -52,12 +81,26 @@ __global__ void __launch_bounds__(256) latent_norm_kernel(const NormParams p) {
   const TX* x = reinterpret_cast<const TX*>(p.x) + (size_t)t * p.x_ld;
   const TX* kv = x + p.q_rank;
   float sq = 0.f, sk = 0.f;
-  for (int i = tid; i < p.q_rank; i += 256) { const float v = ldv(x + i); sq = fmaf(v, v, sq); }
-  for (int i = tid; i < p.L; i += 256) { const float v = ldv(kv + i); sk = fmaf(v, v, sk); }
+#pragma unroll 2
+  for (int i = tid * VEC; i < p.q_rank + p.L; i += 256 * VEC) {        // a vector lies on one side
+    float v[VEC], s = 0.f;
+    ldn<VEC>(x + i, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s = fmaf(v[e], v[e], s);
+    if (i < p.q_rank) sq += s;
+    else sk += s;
+  }
   const float iq = rsqrtf(mb::block_sum(sq, red) / (float)p.q_rank + p.eps);
   const float ik = rsqrtf(mb::block_sum(sk, red) / (float)p.L + p.eps);
   T* cq = reinterpret_cast<T*>(p.cq) + (size_t)t * p.q_rank;
-  for (int i = tid; i < p.q_rank; i += 256) stv(cq + i, ldv(x + i) * iq * __bfloat162float(p.q_w[i]));
+  for (int i = tid * VEC; i < p.q_rank; i += 256 * VEC) {
+    float v[VEC], w[VEC];
+    ldn<VEC>(x + i, v);
+    ldn<VEC>(p.q_w + i, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] *= iq * w[e];
+    stn<VEC>(cq + i, v);
+  }
   const long long slot = p.slots[t];
   if (slot >= p.num_slots) {
     if (p.status && tid == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
@@ -71,12 +114,18 @@ __global__ void __launch_bounds__(256) latent_norm_kernel(const NormParams p) {
   }
   T* dst = reinterpret_cast<T*>(p.cache) + (size_t)slot * p.row;
   const int half = p.R / 2;
-  for (int i = tid; i < p.row; i += 256) {
-    float v = 0.f;
+  for (int i = tid * VEC; i < p.L; i += 256 * VEC) {
+    float v[VEC], w[VEC];
+    ldn<VEC>(kv + i, v);
+    ldn<VEC>(p.kv_w + i, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] *= ik * w[e];
+    stn<VEC>(dst + i, v);
+  }
+  for (int i = p.L + tid; i < p.row; i += 256) {
     const int r = i - p.rope_at;
-    if (i < p.L) {
-      v = ldv(kv + i) * ik * __bfloat162float(p.kv_w[i]);
-    } else if (r >= 0 && r < p.R) {
+    float v = 0.f;
+    if (r >= 0 && r < p.R) {
       const int a = r < half ? r : r - half;
       const float c = p.cos_tab[(size_t)pos * half + a], s = p.sin_tab[(size_t)pos * half + a];
       const float u = ldv(kv + p.L + a), w = ldv(kv + p.L + half + a);
@@ -161,10 +210,18 @@ extern "C" int mb_latent_norm(const MbLatentNormArgs* a, cudaStream_t stream) {
   if (a->x_ld < (long long)a->q_rank + a->L + a->R) return MB_ERR_BAD_ARG;
   const NormParams p{a->q_rank, a->L, a->R, a->row, a->rope_at, a->x, a->x_ld, (const bf16*)a->q_w, (const bf16*)a->kv_w, a->eps, a->cos_tab,
                      a->sin_tab, a->max_pos, a->positions, a->slots, a->num_slots, a->cache, a->cq, a->status};
+  const auto al = [](const void* q, int n) { return reinterpret_cast<uintptr_t>(q) % n == 0; };
+  const bool v4 = a->q_rank % 4 == 0 && a->L % 4 == 0 && a->row % 4 == 0 && a->x_ld % 4 == 0 && al(a->x, 16) && al(a->cq, 16) && al(a->cache, 16) &&
+                  al(a->q_w, 8) && al(a->kv_w, 8);
   const dim3 grid(a->T), block(256);
-  if (a->f32) return a->in_f32 ? (int)mb::launch_kernel(latent_norm_kernel<float, float>, grid, block, 0, stream, p) : MB_ERR_UNSUPPORTED;
-  if (a->in_f32) return (int)mb::launch_kernel(latent_norm_kernel<float, bf16>, grid, block, 0, stream, p);
-  return (int)mb::launch_kernel(latent_norm_kernel<bf16, bf16>, grid, block, 0, stream, p);
+#define MB_LATENT(TX, T)                                                                                         \
+  return (int)(v4 ? mb::launch_kernel(latent_norm_kernel<4, TX, T>, grid, block, 0, stream, p)                   \
+                  : mb::launch_kernel(latent_norm_kernel<1, TX, T>, grid, block, 0, stream, p))
+  if (a->f32 && !a->in_f32) return MB_ERR_UNSUPPORTED;
+  if (a->f32) MB_LATENT(float, float);
+  if (a->in_f32) MB_LATENT(float, bf16);
+  MB_LATENT(bf16, bf16);
+#undef MB_LATENT
 }
 
 extern "C" int mb_latent_query(const MbLatentQueryArgs* a, cudaStream_t stream) {

@@ -38,7 +38,7 @@ struct MlaParams {
   const int* q_start;
   const int* q_len;
   const int* ctx_len;
-  int H, block_size;
+  int H, block_size, tokens_per_tile;    // query tokens of one 128-row tile (tcgen05 kernel)
   long long num_blocks;
   float scale;
   void* out;                    // [rows, H, 512] fp32, or bf16 with out_bf16
@@ -320,9 +320,10 @@ __global__ void mla_merge_kernel(const MlaParams p, const int* row_seq) {
   }
 }
 
-// ------------------------------------------------------------------ decode on tcgen05 / TMEM
-// One query token per sequence, all heads of it as the 128 rows of one UMMA tile: thread r owns head r.
-// grid (2 halves of the 512 value dims, partitions of the context, sequences), 128 threads. Per tile of
+// ------------------------------------------------------------------ tcgen05 / TMEM
+// All heads of 128 / H consecutive query tokens (one in decode) are the 128 rows of one UMMA tile: thread r owns head
+// r % H of token r / H. grid (row tiles x 2 halves of the 512 value dims, partitions of the context, sequences), 128
+// threads; the row tiles with the longest contexts start first. Rows see the keys up to their own position. Per tile of
 // 32 cached tokens the latent rows [32 x 576] are staged ONCE (nine 64-dim blocks, 128-byte swizzle) and
 // feed both products: S = Q K^T (M 128, N 32, 36 k steps over the 576 dims, K-major) and, for this CTA's
 // half, O += P V (M 128, N 256, 2 k steps) with V = four of the same blocks read as an MN-major operand.
@@ -330,6 +331,7 @@ __global__ void mla_merge_kernel(const MlaParams p, const int* row_seq) {
 // than 2^8; the next tile's rows are fetched into registers while the products run. Both halves compute
 // the same S (the second one's tile reads hit L2). Partitions are merged by mla_merge_kernel.
 constexpr int kTcT = 32;                       // cached tokens per tile
+constexpr int kTcMinRows = 32;                 // from this portion length on; between one row and this, the mma.sync kernel
 constexpr int kTcBlocks = kD / 64;             // 9 blocks of 64 dims
 constexpr int kTcQB = 128 * 128;               // one Q block: 128 rows x 128 B
 constexpr int kTcKB = kTcT * 128;              // one cache block of a tile: 32 rows x 128 B
@@ -342,23 +344,27 @@ __device__ __forceinline__ float tc_ex2(float x) {
   return y;
 }
 
-__global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p) {
+__global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   uint8_t* sQ = smem_raw + ((1024u - (mb::smem_u32(smem_raw) & 1023u)) & 1023u);   // 9 x [128 rows x 128 B]
   uint8_t* sK = sQ + kTcBlocks * kTcQB;                                             // 9 x [32 tokens x 128 B]
   uint8_t* sP = sK + kTcBlocks * kTcKB;                                             // [128 rows x 128 B], 32 tokens used
   __shared__ uint64_t bar_s, bar_o;
   __shared__ uint32_t s_tmem;
-  const int hv = blockIdx.x, part = blockIdx.y, seq = blockIdx.z;
+  const int hv = blockIdx.x & 1, part = blockIdx.y, seq = blockIdx.z;
+  const int q0 = ((int)(gridDim.x >> 1) - 1 - (int)(blockIdx.x >> 1)) * p.tokens_per_tile;    // this tile's first query token
   const int tid = threadIdx.x, warp = tid >> 5;
   mb::pdl_wait();
-  const int ctx = p.ctx_len[seq];
-  if (p.q_len[seq] <= 0) return;
+  const int ctx = p.ctx_len[seq], qlen = p.q_len[seq];
+  if (q0 >= qlen) return;
   const int nparts = max(1, (ctx + p.part_tokens - 1) / p.part_tokens);
   if (part >= nparts) return;
-  const int tok_begin = part * p.part_tokens, tok_end = min(ctx, tok_begin + p.part_tokens);
-  const int tiles = (tok_end - tok_begin + kTcT - 1) / kTcT;
-  const int row = p.q_start[seq];                       // the sequence's single query row
+  const int nq = min(p.tokens_per_tile, qlen - q0), rows = nq * p.H;
+  const int seen = ctx - qlen + q0 + nq;                // keys that the tile's last token sees
+  const int tok_begin = part * p.part_tokens, tok_end = min(seen, tok_begin + p.part_tokens);
+  const int tiles = tok_end > tok_begin ? (tok_end - tok_begin + kTcT - 1) / kTcT : 0;
+  const int row = p.q_start[seq] + q0;                  // the first of the tile's query rows
+  const int lim = tid < rows ? min(tok_end, ctx - qlen + q0 + tid / p.H + 1) : 0;
   const int* bt = p.block_table + (size_t)seq * p.max_blocks;
   if (tid == 0) {
     mb::mbar_init(&bar_s, 1);
@@ -367,7 +373,7 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
   }
   if (warp == 0) mb::tmem_alloc(&s_tmem, 512);
   {
-    const uint4* src = tid < p.H ? reinterpret_cast<const uint4*>(p.q + ((size_t)row * p.H + tid) * kD) : nullptr;
+    const uint4* src = tid < rows ? reinterpret_cast<const uint4*>(p.q + ((size_t)row * p.H + tid) * kD) : nullptr;
 #pragma unroll 8
     for (int c = 0; c < kChunks; ++c) {
       const uint4 v = src ? src[c] : make_uint4(0, 0, 0, 0);
@@ -448,7 +454,7 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
       const int tok0 = tok_begin + j * kTcT;
 #pragma unroll
       for (int i = 0; i < kTcT; ++i) {
-        const float v = (tok0 + i < tok_end) ? sv[i] * sc_log2 : -INFINITY;
+        const float v = (tok0 + i < lim) ? sv[i] * sc_log2 : -INFINITY;
         sv[i] = v;
         mx = fmaxf(mx, v);
       }
@@ -513,7 +519,7 @@ __global__ void __launch_bounds__(128, 1) mla_decode_tc_kernel(const MlaParams p
     mb::tc_fence_after();
   }
   if (ok) {                                               // uniform: tcgen05.ld is a whole-warp instruction
-    const bool row_ok = tid < p.H;
+    const bool row_ok = tid < rows;
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
     const size_t grow = (size_t)row * p.H + (row_ok ? tid : 0);
     const bool bf = nparts == 1 && p.out_bf16;
@@ -561,12 +567,12 @@ size_t mb_mla_ws_bytes(int total_rows, int H, int max_ctx, int part_tokens) {
   return parts <= 1 ? 0 : (size_t)total_rows * H * parts * (kL + 2) * sizeof(float);
 }
 
-// Decode rows (one query token per sequence, H <= 128 heads) on the tcgen05 kernel; same arguments,
-// workspace and results as mb_mla_attention.
-int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream) {
-  if (!a || !a->q || !a->cache || !a->out || a->num_seqs <= 0 || a->H <= 0 || a->H > 128 || a->max_q_len != 1)
+// The tcgen05 kernel (H <= 128 heads); same arguments, workspace and results as mb_mla_attention.
+int mb_mla_tc(const MbMlaArgs* a, cudaStream_t stream) {
+  if (!a || !a->q || !a->cache || !a->out || a->num_seqs <= 0 || a->H <= 0 || a->H > 128 || a->max_q_len <= 0)
     return MB_ERR_BAD_ARG;
   MlaParams p{};
+  p.tokens_per_tile = 128 / a->H;
   p.q = reinterpret_cast<const __nv_bfloat16*>(a->q);
   p.cache = reinterpret_cast<const __nv_bfloat16*>(a->cache);
   p.block_table = a->block_table; p.max_blocks = a->max_blocks;
@@ -583,14 +589,15 @@ int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream) {
     p.part_o = reinterpret_cast<float*>(a->ws);
     p.part_ml = p.part_o + (size_t)a->total_rows * a->H * p.parts * kL;
   }
-  if (p.parts > 65535) return MB_ERR_TOO_LARGE;
+  if (p.parts > 65535 || a->num_seqs > 65535) return MB_ERR_TOO_LARGE;
+  const int row_tiles = (a->max_q_len + p.tokens_per_tile - 1) / p.tokens_per_tile;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(mla_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem);
+    cudaError_t e = cudaFuncSetAttribute(mla_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  cudaError_t e = mb::launch_kernel(mla_decode_tc_kernel, dim3(2, p.parts, a->num_seqs), dim3(128), (size_t)kTcSmem, stream, p);
+  cudaError_t e = mb::launch_kernel(mla_tc_kernel, dim3(2 * row_tiles, p.parts, a->num_seqs), dim3(128), (size_t)kTcSmem, stream, p);
   if (e != cudaSuccess) return (int)e;
   if (p.parts > 1) {
     e = mb::launch_kernel(mla_merge_kernel, dim3(a->total_rows * a->H), dim3(128), (size_t)0, stream, p, a->row_seq);
@@ -601,7 +608,8 @@ int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream) {
 
 int mb_mla_attention(const MbMlaArgs* a, cudaStream_t stream) {
   if (!a || !a->q || !a->cache || !a->out || a->num_seqs <= 0 || a->H <= 0 || a->max_q_len <= 0) return MB_ERR_BAD_ARG;
-  if (a->impl == 2 || (a->impl == 0 && a->max_q_len == 1 && a->H <= 128 && a->H >= 16)) return mb_mla_decode_tc(a, stream);
+  const bool tc = a->H <= 128 && ((a->max_q_len == 1 && a->H >= 16) || a->max_q_len >= kTcMinRows);
+  if (a->impl == 2 || (a->impl == 0 && tc)) return mb_mla_tc(a, stream);
   MlaParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(a->q);
   p.cache = reinterpret_cast<const __nv_bfloat16*>(a->cache);

@@ -1,6 +1,6 @@
-// Arguments of the absorbed-MLA paged attention entry points (mla.cu: mma.sync kernel for any row
-// count; mla_tc.cu: tcgen05 / TMEM kernel for decode rows). Shared so that both launchers and the
-// Python binding agree on one layout.
+// Arguments of the absorbed-MLA paged attention entry points (mla.cu: mma.sync kernel for any head
+// count; tcgen05 / TMEM kernel for up to 128 heads). Shared so that both launchers and the Python
+// binding agree on one layout.
 #pragma once
 #include <cuda_runtime.h>
 #include <stddef.h>
@@ -24,9 +24,9 @@ struct MbMlaArgs {
   size_t ws_bytes;
   int part_tokens;           // 0 = default 1024
   uint32_t* status;
-  int impl;                  // 0 = choose, 1 = mma.sync kernel, 2 = tcgen05 kernel (decode rows, H <= 128)
+  int impl;                  // 0 = choose, 1 = mma.sync kernel, 2 = tcgen05 kernel (H <= 128)
   int split_p;               // softmax weights enter the product with V as two bf16 terms
   int out_bf16;              // out is bf16 [rows, H, 512]
 };
 
-extern "C" int mb_mla_decode_tc(const MbMlaArgs* a, cudaStream_t stream);
+extern "C" int mb_mla_tc(const MbMlaArgs* a, cudaStream_t stream);

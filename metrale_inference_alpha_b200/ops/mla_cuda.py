@@ -29,6 +29,7 @@ _native.register_optional("mb_mla_prepare", [c_void_p] * 10 + [c_int] * 6 + [c_l
 
 LATENT, ROW = 512, 576
 TC_PART_TOKENS = 256
+TC_MIN_ROWS = 32                 # csrc/mla.cu: kTcMinRows
 _CNT_BYTES = 64 * 1024
 
 
@@ -42,7 +43,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_
                   out_bf16: bool = False) -> torch.Tensor:
     """q [T, H, 576] bf16 -> [T, H, 512] fp32, or bf16 with `out_bf16`. `split_p`: the softmax weights enter the product
     with the values as two bf16 terms (16 mantissa bits) instead of one. `impl`: 0 = decode steps (one query row per sequence,
-    16 <= H <= 128) take the tcgen05 / TMEM kernel, everything else the mma.sync kernel; 1 / 2 force one."""
+    16 <= H <= 128) and prefill portions (H <= 128) take the tcgen05 / TMEM kernel, everything else the mma.sync kernel; 1 / 2
+    force one."""
     from . import _count, _ptr, _stream, runtime
     L = _native.lib()
     if not hasattr(L, "mb_mla_attention"):
@@ -55,6 +57,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_
         # the tcgen05 decode kernel runs one CTA per SM: shorter partitions than the mma.sync kernel's 1024
         # keep the SMs busy at small batch (a constant, so a sequence's split never depends on the batch)
         part_tokens = TC_PART_TOKENS
+    elif part_tokens == 0 and H <= 128 and (impl == 2 or (impl == 0 and max_q_len >= TC_MIN_ROWS)):
+        part_tokens = 1 << 30                     # enough row tiles without splitting the context, and no partial rows to merge
     rt = runtime(q.device)
     out = torch.empty(T, H, LATENT, dtype=torch.bfloat16 if out_bf16 else torch.float32, device=q.device)
     need = L.mb_mla_ws_bytes(T, H, max_ctx, part_tokens)

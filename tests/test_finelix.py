@@ -203,8 +203,8 @@ def test_latent_attention_reads_single_keys(device, fmt):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("kernel,name", [("mma", "t64"), ("mma", "t128"), ("auto", "t256"), ("simt", "t256"), ("mma", "mla"), ("mma", "mla full"),
-                                         ("tc", "mla full"), ("auto", "mla full"), ("simt", "mla"), ("auto", "past")])
+@pytest.mark.parametrize("kernel,name", [("mma", "t64"), ("mma", "t128"), ("auto", "t256"), ("simt", "t256"), ("mma", "mla"), ("mma", "mla full"), ("auto", "mla"),
+                                         ("tc", "mla"), ("tc", "mla full"), ("auto", "mla full"), ("simt", "mla"), ("auto", "past")])
 def test_latent_attention_kernels_long(kernel, name):
     """Long contexts: tiles of every kernel, several partitions of the context (decode past 256, 512 and 1024 keys),
     far keys. Queries and cache rows are rounded to bf16 on both sides, so only the attention itself is compared."""
@@ -232,13 +232,9 @@ def test_latent_attention_kernels_long(kernel, name):
     idx = torch.tensor([pages[i // 16] * 16 + i % 16 for i in range(n)])
     cache.view(-1, lay.row)[idx] = row
     cache, qd, uvd = cache.cuda(), q.cuda(), b16(uv).cuda()
-    cuts = [(i, i + 1) for i in range(1190, 1250)] + [(0, 256), (512, 513), (256, 257), (257, 258)]
-    if kernel != "tc":
-        cuts += [(0, 1190), (1000, 1007), (630, 800)]
+    cuts = [(i, i + 1) for i in range(1190, 1250)] + [(0, 256), (512, 513), (256, 257), (257, 258), (0, 1190), (1000, 1007), (630, 800)]
     got, ref_rows = [], []
     for lo, hi in cuts:
-        if kernel == "tc" and hi - lo > 1:
-            continue
         b = fc.batch([hi - lo], [hi], pages=[pages[:(hi + 15) // 16]], device="cuda")
         out = torch.empty(hi - lo, H * dv, dtype=torch.bfloat16, device="cuda")
         lt.attention(qd[lo:hi].contiguous(), cache, b, uvd, scale, fmt, lay, out, kernel=kernel)
