@@ -1,4 +1,5 @@
-"""One recurrence launch sequence on a small case, for a profiler: decode | chunk (time-mix mode)."""
+"""One launch sequence on a small case, for a profiler: decode | chunk (recurrence, time-mix mode), gla (the same
+recurrence read after its update, with low-rank decays and the head norm), latent-decode | latent (latent attention)."""
 import os
 import sys
 
@@ -10,13 +11,28 @@ from metrale_inference_alpha_b200.ops import check_status, mixers as mx  # noqa:
 
 case = sys.argv[1]
 H, D = 20, 128
-lens, start = ([1] * 128, 63) if case == "decode" else ([4096], 0)
-b, _ = batch(lens, start)
-T = sum(lens)
-q, k, v = (rnd(T, H * D) for _ in range(3))
-lw, u = -torch.exp(torch.randn(T, H * D, device="cuda") - 3), torch.rand(H, D, device="cuda")
-ssm = torch.zeros(len(lens) + 2, H, D, D, device="cuda")
+if case.startswith("latent"):
+    from metrale_inference_alpha_b200.ops import latent as lt
+    lens, start = ([1] * 64, 1023) if case == "latent-decode" else ([1024], 0)
+    b, blocks = batch(lens, start)
+    T, heads, lay = sum(lens), 32, lt.latent_row(512, 64, "bf16")
+    cache, q, uv = rnd(blocks, 16, 1, lay.row), rnd(T, heads, lay.row, std=0.3), rnd(heads, 128, 512, std=0.05)
+    out = torch.empty(T, heads * 128, dtype=q.dtype, device="cuda")
+    run = lambda: lt.attention(q, cache, b, uv, 0.07, "bf16", lay, out)
+else:
+    lens, start = ([1] * 128, 63) if case == "decode" else ([4096], 0)
+    b, _ = batch(lens, start)
+    T = sum(lens)
+    q, k, v, g = (rnd(T, H * D) for _ in range(4))
+    ssm = torch.zeros(len(lens) + 2, H, D, D, device="cuda")
+    kw = dict(heads=H, dk=D, dv=D, fmt="bf16")
+    if case == "gla":
+        lr = mx.LowRankDecay(rnd(T, 16), rnd(H * D, 16, std=0.1), rnd(H * D, dtype=torch.float32), 1 / 16)
+        kw.update(low_rank=lr, norm=dict(w=rnd(H * D), gate=g, gate_act="silu", eps=1e-5, scale=1.0, out=torch.empty_like(g)))
+    else:
+        kw.update(log_w=-torch.exp(torch.randn(T, H * D, device="cuda") - 3), u=torch.rand(H, D, device="cuda"))
+    run = lambda: mx.linear_attention(q, k, v, ssm, b, **kw)
 for _ in range(3):
-    mx.linear_attention(q, k, v, ssm, b, heads=H, dk=D, dv=D, fmt="bf16", log_w=lw, u=u)
+    run()
 torch.cuda.synchronize()
 check_status("cuda")

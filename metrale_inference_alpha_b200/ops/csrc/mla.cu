@@ -373,11 +373,13 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
   }
   if (warp == 0) mb::tmem_alloc(&s_tmem, 512);
   {
-    const uint4* src = tid < rows ? reinterpret_cast<const uint4*>(p.q + ((size_t)row * p.H + tid) * kD) : nullptr;
+    // the tile's query rows are consecutive in memory: consecutive threads take consecutive chunks
+    const uint4* src = reinterpret_cast<const uint4*>(p.q + (size_t)row * p.H * kD);
 #pragma unroll 8
-    for (int c = 0; c < kChunks; ++c) {
-      const uint4 v = src ? src[c] : make_uint4(0, 0, 0, 0);
-      *reinterpret_cast<uint4*>(sQ + (c >> 3) * kTcQB + tc_sw(tid, c & 7)) = v;
+    for (int i = 0; i < kChunks; ++i) {
+      const int idx = i * 128 + tid, rq = idx / kChunks, c = idx - rq * kChunks;
+      const uint4 v = rq < rows ? __ldg(src + idx) : make_uint4(0, 0, 0, 0);
+      *reinterpret_cast<uint4*>(sQ + (c >> 3) * kTcQB + tc_sw(rq, c & 7)) = v;
     }
     // the upper half of every P row holds what rounding took off the weights (split_p), else it is never read
 #pragma unroll
@@ -392,14 +394,17 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
   constexpr uint32_t kIdescS = mb::umma_idesc(1, 1, 128, kTcT);
   constexpr uint32_t kIdescO = mb::umma_idesc(1, 1, 128, 256, 0, 1);
   const uint32_t aQ = mb::smem_u32(sQ), aK = mb::smem_u32(sK), aP = mb::smem_u32(sP);
+  const uint64_t dQ = mb::umma_desc_sw128(aQ), dK = mb::umma_desc_sw128(aK);     // the address field counts 16-byte units
   const float sc_log2 = p.scale * 1.44269504088896f;
   float m_run = -INFINITY, l_run = 0.f;
   uint32_t ph_s = 0, ph_o = 0;
   bool ok = true;
-  // staging: thread = (token tid / 4 of the tile, quarter tid % 4 of its row): 18 consecutive 16-byte chunks,
-  // one block-table lookup per tile
+  // staging: four threads per token of the tile, step i takes four consecutive 16-byte chunks of its row. Odd tokens
+  // take the two halves of every 128 bytes in the other order, so that eight threads' stores meet eight bank groups
   constexpr int kPer = kChunks / 4;
-  const int s_tok = tid >> 2, s_c0 = (tid & 3) * kPer;
+  const int s_tok = tid >> 2, s_q = tid & 3, s_par = s_tok & 1;
+  uint8_t* const k_even = sK + tc_sw(s_tok, s_q + 4 * s_par);
+  uint8_t* const k_odd = sK + tc_sw(s_tok, s_q + 4 * (1 - s_par));
   uint4 raw[kPer];
   auto fetch = [&](int jt) {
     const int tok = tok_begin + jt * kTcT + s_tok;
@@ -409,9 +414,10 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
         if (p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
         blk = 0;
       }
-      const uint4* src = reinterpret_cast<const uint4*>(p.cache + ((size_t)blk * p.block_size + (tok % p.block_size)) * kD) + s_c0;
+      const uint4* src = reinterpret_cast<const uint4*>(p.cache + ((size_t)blk * p.block_size + (tok % p.block_size)) * kD) + s_q;
+      const uint4 *even = src + 4 * s_par, *odd = src - 4 * s_par;
 #pragma unroll
-      for (int i = 0; i < kPer; ++i) raw[i] = __ldg(src + i);
+      for (int i = 0; i < kPer; ++i) raw[i] = __ldg((i & 1 ? odd : even) + 4 * i);
     } else {
 #pragma unroll
       for (int i = 0; i < kPer; ++i) raw[i] = make_uint4(0, 0, 0, 0);
@@ -425,10 +431,7 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
       mb::tc_fence_after();
     }
 #pragma unroll
-    for (int i = 0; i < kPer; ++i) {
-      const int c = s_c0 + i;
-      *reinterpret_cast<uint4*>(sK + (c >> 3) * kTcKB + tc_sw(s_tok, c & 7)) = raw[i];
-    }
+    for (int i = 0; i < kPer; ++i) *reinterpret_cast<uint4*>((i & 1 ? k_odd : k_even) + (i >> 1) * kTcKB) = raw[i];
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     mb::tc_fence_before();
     __syncthreads();
@@ -438,8 +441,7 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
       for (int b = 0; b < kTcBlocks; ++b)
 #pragma unroll
         for (int s = 0; s < 4; ++s)
-          mb::umma_f16(tmem, mb::umma_desc_sw128(aQ + b * kTcQB + s * 32), mb::umma_desc_sw128(aK + b * kTcKB + s * 32),
-                       kIdescS, (b | s) != 0);
+          mb::umma_f16(tmem, dQ + ((b * kTcQB + s * 32) >> 4), dK + ((b * kTcKB + s * 32) >> 4), kIdescS, (b | s) != 0);
       mb::tc_commit(&bar_s);
     }
     fetch(j + 1);
@@ -518,36 +520,40 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
     ok = mb::mbar_wait(&bar_o, ph_o, p.status, MB_ST_TIMEOUT_MMA) && ok;
     mb::tc_fence_after();
   }
-  if (ok) {                                               // uniform: tcgen05.ld is a whole-warp instruction
-    const bool row_ok = tid < rows;
+  ok = __syncthreads_and(ok) != 0;
+  if (ok) {
+    // the query tile's space takes the outputs, one padded row per thread, so that rows leave in whole vectors
+    constexpr int kOut = 256 + 4;
+    static_assert(128 * kOut * 4 <= kTcBlocks * kTcQB, "outputs fit into the query tile");
+    float* sO = reinterpret_cast<float*>(sQ);
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-    const size_t grow = (size_t)row * p.H + (row_ok ? tid : 0);
-    const bool bf = nparts == 1 && p.out_bf16;
-    float* dst = (nparts == 1 ? reinterpret_cast<float*>(p.out) + (bf ? 0 : grow * kL) : p.part_o + (grow * p.parts + part) * kL) + hv * 256;
-    __nv_bfloat16* dst16 = reinterpret_cast<__nv_bfloat16*>(p.out) + grow * kL + hv * 256;
 #pragma unroll
     for (int c = 0; c < 16; ++c) {
       float ov[16];
       mb::tmem_ld16(t_row + 32 + c * 16, ov);
-      if (row_ok && bf) {
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          uint4 v;
-          uint32_t* pv = reinterpret_cast<uint32_t*>(&v);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) pv[e] = pack_bf16(ov[8 * i + 2 * e] * inv, ov[8 * i + 2 * e + 1] * inv);
-          *reinterpret_cast<uint4*>(dst16 + c * 16 + i * 8) = v;
-        }
-      } else if (row_ok) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          *reinterpret_cast<float4*>(dst + c * 16 + i * 4) =
-              make_float4(ov[4 * i] * inv, ov[4 * i + 1] * inv, ov[4 * i + 2] * inv, ov[4 * i + 3] * inv);
-      }
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(sO + tid * kOut + c * 16 + i * 4) =
+            make_float4(ov[4 * i] * inv, ov[4 * i + 1] * inv, ov[4 * i + 2] * inv, ov[4 * i + 3] * inv);
     }
-    if (row_ok && nparts > 1 && hv == 0) {
-      p.part_ml[(grow * p.parts + part) * 2] = m_run;
-      p.part_ml[(grow * p.parts + part) * 2 + 1] = l_run;
+    const size_t grow0 = (size_t)row * p.H;
+    if (tid < rows && nparts > 1 && hv == 0) {
+      p.part_ml[((grow0 + tid) * p.parts + part) * 2] = m_run;
+      p.part_ml[((grow0 + tid) * p.parts + part) * 2 + 1] = l_run;
+    }
+    __syncthreads();
+    for (int i = tid; i < rows * 64; i += 128) {
+      const int rr = i >> 6, c4 = (i & 63) * 4;
+      const float4 v = *reinterpret_cast<const float4*>(sO + rr * kOut + c4);
+      const size_t grow = grow0 + rr;
+      if (nparts > 1) {
+        *reinterpret_cast<float4*>(p.part_o + (grow * p.parts + part) * kL + hv * 256 + c4) = v;
+      } else if (p.out_bf16) {
+        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.out) + grow * kL + hv * 256 + c4) =
+            make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      } else {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + grow * kL + hv * 256 + c4) = v;
+      }
     }
   }
   mb::tc_fence_before();

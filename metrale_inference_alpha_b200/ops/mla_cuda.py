@@ -33,6 +33,16 @@ TC_MIN_ROWS = 32                 # csrc/mla.cu: kTcMinRows
 _CNT_BYTES = 64 * 1024
 
 
+_ROWS: dict = {}          # device -> [0, 1, ...]; the older, shorter ones stay alive for graphs that captured them
+
+
+def _row_numbers(n: int, device) -> torch.Tensor:
+    kept = _ROWS.setdefault(str(device), [])
+    if not kept or kept[-1].numel() < n:
+        kept.append(torch.arange(max(1024, 2 * n), dtype=torch.int32, device=device))
+    return kept[-1]
+
+
 def supported(q: torch.Tensor, cache: torch.Tensor) -> bool:
     return (q.is_cuda and q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and q.shape[-1] == ROW
             and cache.shape[-1] == ROW and cache.shape[2] == 1)
@@ -66,6 +76,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_table, q_start, q_
         # the head of the shared attention workspace holds the split-KV kernel's arrival counters,
         # which must stay zero between its launches: the MLA partials live behind them
         rt.ensure_attn_ws(need + _CNT_BYTES)
+        if row_seq is None and max_q_len == 1 and T == q_len.numel():      # one row per sequence
+            row_seq = _row_numbers(T, q.device)
         if row_seq is None:                       # row -> sequence map for the merge pass
             # fixed-shape (capturable): the sequence of row t is the last one whose first row is <= t
             rows = torch.arange(T, device=q.device, dtype=q_start.dtype)

@@ -118,9 +118,10 @@ def load_finelix(ld) -> ModelW:
     def latent(q, m, router) -> LatentW:
         H, dim, R, L, dv = m["heads"], m["dim"], m["rot_dim"], m["kv_rank"], m["vdim"]
         parts = [f"{q}.dq", f"{q}.dkv"] + ([router] if router else [])
-        return LatentW(in_proj=weight(pad_rows(raw(*parts), 4)), q_norm=ld.vec(f"{q}.dq.norm"), kv_norm=ld.vec(f"{q}.dkv.norm"),
+        q_norm = ld.vec(f"{q}.dq.norm")
+        return LatentW(in_proj=weight(pad_rows(raw(*parts), 4)), q_norm=q_norm, kv_norm=ld.vec(f"{q}.dkv.norm"),
                        uq=weight(raw(f"{q}.uq")), w_uk=raw(f"{q}.uk").view(H, dim, L), w_uv=raw(f"{q}.uv").view(H, dv, L), heads=H, dim=dim,
-                       rot_dim=R, vdim=dv, kv_rank=L, q_rank=m["q_rank"], scale=float(m["scale"]), rot_base=float(m["rot"]["base"]))
+                       rot_dim=R, vdim=dv, kv_rank=L, q_rank=q_norm.numel(), scale=float(m["scale"]), rot_base=float(m["rot"]["base"]))
 
     def experts(p, mlp) -> GroupedExperts:
         gu = [pad_rows(gate_up(f"{p}.e{e}"), 128) for e in range(mlp["router"]["experts"])]
