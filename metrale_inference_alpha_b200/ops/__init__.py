@@ -521,6 +521,8 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     a = _native.GemmArgs()
     a.kind, a.M, a.N, a.K, a.ldo = KIND[w.fmt], M, N, w.K, (out.stride(0) if out is not None else n_out)
     a.W, a.X, a.out = _ptr(w.data), _ptr(act.data), _ptr(out)
+    if w.fmt == "bf16" and M > 1 and act.data.stride(0) != w.K:                  # a column range of a wider matrix
+        a.ldx = act.data.stride(0)
     a.residual = _ptr(residual)
     a.alpha = 1.0
     if w.fmt == "fp8_row":

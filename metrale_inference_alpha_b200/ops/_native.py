@@ -29,7 +29,7 @@ class GemmArgs(C.Structure):
         ("outq", c_void_p), ("ldq", c_int), ("outq_sf", c_void_p), ("outq_sf_k64", c_int), ("outq_gs", c_float),
         ("tile_expert", c_void_p), ("tile_row0", c_void_p), ("tile_nrows", c_void_p),
         ("n_per_expert", c_int), ("max_tiles", c_int),
-        ("epi_a", c_float), ("epi_b", c_float), ("epi_n", c_int), ("epi_bias", c_void_p),
+        ("epi_a", c_float), ("epi_b", c_float), ("epi_n", c_int), ("epi_bias", c_void_p), ("ldx", c_ll),
     ]
 
 

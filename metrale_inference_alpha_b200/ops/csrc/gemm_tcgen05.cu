@@ -1020,6 +1020,7 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   }
   const size_t row_bytes = (size_t)a->K * elem_bits / 8;
   if (row_bytes % 16) return MB_ERR_BAD_ARG;           // TMA global stride rule
+  if (a->ldx && (kind != KIND_BF16 || a->ldx < a->K || a->ldx % 8 || reinterpret_cast<uintptr_t>(a->X) % 16)) return MB_ERR_BAD_ARG;
   if (kind == KIND_NVFP4 && (!a->sfa || !a->sfb)) return MB_ERR_BAD_ARG;
   if (kind == KIND_FP8_BLOCK && (!a->w_scale || !a->a_scale)) return MB_ERR_BAD_ARG;
   if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU || a->epilogue == EPI_GEGLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
@@ -1117,7 +1118,7 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   const uint32_t box_inner = (elem_bits == 16) ? 64 : 128;
   int rc = mbh::encode_2d(&tmA, dt, a->W, inner, (uint64_t)a->N, row_bytes, box_inner, kTileN);
   if (rc) return rc;
-  rc = mbh::encode_2d(&tmB, dt, a->X, inner, (uint64_t)a->M, row_bytes, box_inner, (uint32_t)tn);
+  rc = mbh::encode_2d(&tmB, dt, a->X, inner, (uint64_t)a->M, a->ldx > 0 ? (size_t)a->ldx * 2 : row_bytes, box_inner, (uint32_t)tn);
   if (rc) return rc;
 
   // prefill-sized plain GEMMs put the token tiles in x (MB_GEMM_DECODE_TILE_ORDER keeps the decode order)

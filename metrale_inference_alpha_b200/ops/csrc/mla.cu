@@ -406,10 +406,16 @@ __global__ void __launch_bounds__(128, 1) mla_tc_kernel(const MlaParams p) {
   uint8_t* const k_even = sK + tc_sw(s_tok, s_q + 4 * s_par);
   uint8_t* const k_odd = sK + tc_sw(s_tok, s_q + 4 * (1 - s_par));
   uint4 raw[kPer];
+  auto page_of = [&](int jt) {                          // looked up one tile ahead of its use
+    const int tok = tok_begin + jt * kTcT + s_tok;
+    return jt < tiles && tok < tok_end ? bt[tok / p.block_size] : 0;
+  };
+  int page = page_of(0);
   auto fetch = [&](int jt) {
     const int tok = tok_begin + jt * kTcT + s_tok;
+    long long blk = page;
+    page = page_of(jt + 1);
     if (jt < tiles && tok < tok_end) {
-      long long blk = bt[tok / p.block_size];
       if (blk < 0 || blk >= p.num_blocks) {
         if (p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
         blk = 0;

@@ -530,7 +530,8 @@ class LowRankDecay:
             return self.c * ref.log_sigmoid(z)
         if self.a2_lin is not None and self.a1.shape[0] >= _DECAY_TC_MIN_ROWS:
             from . import linear
-            return linear(act_of(self.a1.contiguous(), "bf16"), self.a2_lin, out_f32=True, log_sigmoid=(self.bias, self.c))
+            a1 = self.a1 if self.a1.stride(0) % 8 == 0 and self.a1.data_ptr() % 16 == 0 else self.a1.contiguous()
+            return linear(act_of(a1, "bf16"), self.a2_lin, out_f32=True, log_sigmoid=(self.bias, self.c))
         out = torch.empty(self.a1.shape[0], self.a2.shape[0], dtype=torch.float32, device=self.a1.device)
         return gemm_simt(self.a1, self.a2, out, epilogue=7, bias=self.bias, epi_a=self.c)
 

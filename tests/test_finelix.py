@@ -375,7 +375,8 @@ def test_low_rank_decay(device, fmt, T, rank):
     a1, a2 = gen(T, rank, seed=1, std=2.0).to(dt(fmt)), b16(gen(136, rank, seed=2, std=3.0))
     bias = gen(136, seed=3, std=8.0)
     q = QuantWeight("bf16", 136, rank, a2.to(device)) if rank % 8 == 0 and fmt == "bf16" else None
-    got = mx.LowRankDecay(a1.to(device), a2.to(device), bias.to(device), 1 / 16.0, q).log()
+    wide = torch.cat([torch.full((T, 8), 9.0).to(dt(fmt)), a1, torch.full((T, 32 - rank), 9.0).to(dt(fmt))], 1).to(device)     # a column range
+    got = mx.LowRankDecay(wide[:, 8:8 + rank], a2.to(device), bias.to(device), 1 / 16.0, q).log()
     z = a1.double() @ a2.double().T + bias.double()
     want = (z.clamp(max=0) - torch.log1p(torch.exp(-z.abs()))) / 16.0
     dz = 2e-6 * (a1.double().abs() @ a2.double().T.abs() + bias.double().abs())          # what 32-bit sums may be off by
@@ -428,6 +429,8 @@ def test_linear_epilogues(device, fmt, M, N, K):
     ops.linear(act, W, geglu=True, out=wide[:, 8:])
     close(wide[:, 8:], fo.gelu_tanh(y[:, 0::2]) * y[:, 1::2], tol)
     assert bool((wide[:, :8] == 2.0).all())
+    rows = torch.cat([x, x], 1).to(device)[:, K:] if K % 8 == 0 else x.to(device)        # and operands from one
+    close(ops.linear(mx.act_of(rows, fmt), W), y, tol)
 
 
 @pytest.mark.parametrize("device", DEVICES)
