@@ -264,7 +264,7 @@ def finelix_kernels(W=2560, H=20, D=128, FF=6912, rank=16, Hl=32, dim=128, R=64,
 
 
 def finelix_models():
-    """(label, name -> configuration): Finelix, the same with its first two layers looped three times, and a hybrid of
+    """(label, name -> configuration): Finelix, the same with two layers looped three times, and a hybrid of
     equal size: MLA and experts where Finelix has latent attention, Kimi delta attention and SwiGLU elsewhere; bf16."""
     from metrale_inference_alpha_b200.config.model_config import ModelConfig, preset
     for label, kw in (("1B-like layers", dict(width=2048, heads=16, lin_heads=16, ff=5632, experts=32, top=4, expert_ff=768, shared_ff=1536, vocab=32768)),

@@ -445,10 +445,10 @@ def tiny_finelix(**kw) -> ModelConfig:
 def finelix_3b(**kw) -> ModelConfig:
     """Finelix with the layer sizes of a ~3B-active model: width 2560, latent attention of 32 heads (128 + 64, value
     128, latent 512, query latent 1536) beside 64 experts of 1024, top 6, and a shared one; gated linear attention
-    of 20 heads of 128 beside a feed-forward of 6912; 24 layers, the first two run three times."""
+    of 20 heads of 128 beside a feed-forward of 6912; 24 layers, two of them run three times."""
     base = dict(name="finelix-3b", num_layers=24, width=2560, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536,
                 lin_heads=20, lin_dim=128, lin_vdim=128, ff=6912, experts=64, top=6, expert_ff=1024, shared_ff=2048, vocab=65536,
-                loop={"start": 0, "stop": 2, "times": 3})
+                loop={"start": 2, "stop": 4, "times": 3})
     base.update(kw)
     return finelix(**base)
 
