@@ -17,8 +17,8 @@ from typing import List, Optional
 
 WEIGHT_FORMATS = ("bf16", "nvfp4", "fp8_block", "fp8_row", "fp32")
 KV_DTYPES = ("bf16", "fp8", "fp32")
-LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning", "latent", "gla")
-KV_KINDS = ("attention", "mla", "parallel", "latent")                    # kinds that own a KV pool
+LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning", "latent", "gla", "gated")
+KV_KINDS = ("attention", "mla", "parallel", "latent", "gated")           # kinds that own a KV pool
 STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning", "gla")   # kinds that own a recurrent state
 FFN_KINDS = ("dense", "moe", "none")
 
@@ -26,7 +26,7 @@ FFN_KINDS = ("dense", "moe", "none")
 @dataclass
 class ModelConfig:
     name: str = "model"
-    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix | finelix
+    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix | finelix | pivipel
     vocab_size: int = 4096
     hidden_size: int = 256
     num_layers: int = 2
@@ -61,8 +61,11 @@ class ModelConfig:
     residual_multiplier: float = 1.0    # Granite: a block's output is scaled by this before it joins the stream
     logits_divisor: float = 1.0         # Granite: logits are divided by this
     tie_embeddings: bool = False
-    # fabulix, finelix: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
+    # fabulix, finelix, pivipel: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
     layer_specs: List[dict] = field(default_factory=list)
+    spec_types: List[str] = field(default_factory=list)      # pivipel: the layers' own type names (variants of one layer kind)
+    weights_of: List[int] = field(default_factory=list)      # per layer: the layer whose tensors it uses, -1 = its own; empty = all their own
+    streams: int = 0                    # static hyper-connections: the residual is this many fp32 copies (0 = a single residual)
     loop: Optional[dict] = None         # layers start .. stop - 1 run `times` times with the same weights: {"start", "stop", "times"}
     token_side_dim: int = 0             # width of a layer's slice of the token side embedding (0 = none)
     glu_alpha: float = 1.702            # sigmoid slope of the clamped GLU
@@ -171,7 +174,13 @@ class ModelConfig:
     @property
     def stream32(self) -> bool:
         """The residual stream is kept in 32-bit, and the layers' sizes are per layer (``layer_specs``)."""
-        return self.arch in ("fabulix", "finelix")
+        return self.arch in ("fabulix", "finelix", "pivipel")
+
+    def layer_owner(self, i: int) -> int:
+        """The layer whose tensors layer i uses (its cache or state is its own all the same)."""
+        while self.weights_of and self.weights_of[i] >= 0:
+            i = self.weights_of[i]
+        return i
 
     def layer_runs(self) -> List[tuple]:
         """(layer, pass) of every layer run in order. A looped layer appears once per pass, and each of its runs
@@ -199,6 +208,8 @@ class ModelConfig:
             t, m = self.layer_types[i], self.layer_specs[i]["mixer"]
             if t == "parallel":
                 m = m["left"]
+                out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
+            elif t == "gated":
                 out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
             elif t == "latent":
                 out.append((1, latent_row(m["kv_rank"], m["rot_dim"], self.act_fmt).row, 0))
@@ -453,8 +464,53 @@ def finelix_3b(**kw) -> ModelConfig:
     return finelix(**base)
 
 
+def pivipel(num_layers: int = 4, width: int = 192, heads: int = 4, kv_heads: int = 2, dim: int = 64, vdim: int = 64, rot_dims: int = 32,
+            rot_base: float = 10000.0, window: int = 24, keep: int = 3, ff: int = 512, limit: float = 2.5, experts: int = 8, top: int = 2,
+            expert_ff: int = 80, shared_ff: int = 160, groups: int = 4, keep_groups: int = 2, streams: int = 2, vocab: int = 1024,
+            positions: int = 4096, period: int = 2, dense_layers: int = 1, share: bool = False, eps: float = 1e-5, **kw) -> ModelConfig:
+    """Pivipel decoder of uniform layers: every `period`-th layer has normed attention without positions and a window
+    beside kept first tokens, the others rotated sink attention in a plain window; dense feed-forwards in the first
+    `dense_layers`, mixtures of experts behind them; `share`: the last layer uses the tensors of the one `period` before."""
+    layers = []
+    for i in range(num_layers):
+        m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": window}}
+        t = "attention_2" if i % period == period - 1 else "attention"
+        if t == "attention":
+            m["rot"] = {"base": rot_base, "dims": rot_dims, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}
+        else:
+            m["mask"]["keep_first"] = keep
+        mlp = {"kind": "dense", "ff": ff, "limit": limit}
+        if i >= dense_layers:
+            mlp = {"kind": "moe", "expert": {"ff": expert_ff, "limit": limit},
+                   "router": {"experts": experts, "top": top, "scale": 1.25, "groups": {"count": groups, "keep": keep_groups}}}
+            if shared_ff:
+                mlp["shared"] = {"ff": shared_ff, "limit": limit}
+        layers.append({"type": t, "mixer": m, "mlp": mlp})
+    if share:
+        layers[-1]["weights_of"] = num_layers - 1 - period
+    cfg = {"architecture": "Pivipel", "vocab": vocab, "width": width, "streams": streams, "max_positions": positions, "norm": {"eps": eps},
+           "layers": layers}
+    return from_pivipel_config(cfg, name=kw.pop("name", "pivipel")).scaled(**kw)
+
+
+def tiny_pivipel(**kw) -> ModelConfig:
+    """Four-layer Pivipel whose last layer shares its tensors (tests, smoke runs)."""
+    return pivipel(**{"name": "tiny-pivipel", "share": True, **kw})
+
+
+def pivipel_3b(**kw) -> ModelConfig:
+    """Pivipel with the layer sizes of a ~3B-active model: width 2560, 32 query / 8 key-value heads of 128, windows of
+    1024, 64 experts of 1024, top 6 from half of 8 groups, and a gated shared one of 2048; two streams, 24 layers."""
+    base = dict(name="pivipel-3b", num_layers=24, width=2560, heads=32, kv_heads=8, dim=128, vdim=128, rot_dims=128, window=1024, keep=4,
+                ff=6912, limit=7.0, experts=64, top=6, expert_ff=1024, shared_ff=2048, groups=8, keep_groups=4, vocab=65536, positions=16384)
+    base.update(kw)
+    return pivipel(**base)
+
+
 PRESETS = {
     "tiny-dense": tiny_dense,
+    "tiny-pivipel": tiny_pivipel,
+    "pivipel-3b": pivipel_3b,
     "tiny-finelix": tiny_finelix,
     "finelix-3b": finelix_3b,
     "tiny-fabulix": tiny_fabulix,
@@ -583,8 +639,58 @@ def from_finelix_config(cfg: dict, name: str = "model") -> ModelConfig:
         moe_intermediate_size=moe["expert"]["ff"] if moe else 0, max_position=131072)
 
 
+def from_pivipel_config(cfg: dict, name: str = "model") -> ModelConfig:
+    """A Pivipel ``config.json``: sizes and constants are given per layer and kept per layer; a layer with `weights_of`
+    uses another one's tensors. Mixer types and feed-forward kinds this engine does not know are refused."""
+    types, ffns, specs, owners = [], [], [], []
+    for i, L in enumerate(cfg["layers"]):
+        t, m, mlp = L["type"], L["mixer"], L.get("mlp")
+        if t not in ("attention", "attention_2"):
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+        if mlp is not None and mlp.get("kind") not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        rot, mask, of = m.get("rot") or {"dims": 0}, m.get("mask") or {}, L.get("weights_of")
+        if m["heads"] % m["kv_heads"] or rot["dims"] % 2 or rot["dims"] > m["dim"]:
+            raise ValueError(f"layer {i}: attention heads, key/value heads or rotary size do not fit together")
+        if mask.get("size", 1) < 1 or mask.get("keep_first", 0) < 0:
+            raise ValueError(f"layer {i}: a window of {mask.get('size')} with {mask.get('keep_first')} kept tokens")
+        if mlp is not None and mlp["kind"] == "moe":
+            r = mlp["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            if r["experts"] > 512 or r["experts"] % g["count"] or not 0 < g["keep"] <= g["count"] <= 32 \
+                    or not 0 < r["top"] <= min(32, r["experts"] // g["count"] * g["keep"]):
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts per token from {g['keep']} of {g['count']} groups")
+        if of is not None and not (0 <= of < len(cfg["layers"]) and of != i):
+            raise ValueError(f"layer {i}: no tensors of layer {of}")
+        types.append(t)
+        ffns.append("none" if mlp is None else mlp["kind"])
+        specs.append({"mixer": m, "mlp": mlp})
+        owners.append(-1 if of is None else int(of))
+    for i in range(len(owners)):
+        seen, j = set(), i
+        while owners[j] >= 0:
+            if j in seen:
+                raise ValueError(f"layer {i}: its tensors are its own by way of others")
+            seen.add(j)
+            j = owners[j]
+        if types[j] != types[i] or specs[j] != specs[i]:
+            raise ValueError(f"layer {i}: not like layer {j}, whose tensors it uses")
+    if int(cfg["streams"]) < 1:
+        raise ValueError(f"{cfg['streams']} residual streams")
+    att, moe = specs[0]["mixer"], next((s["mlp"] for f, s in zip(ffns, specs) if f == "moe"), None)
+    return ModelConfig(
+        name=name, arch="pivipel", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(types), layer_types=["gated"] * len(types),
+        ffn_types=ffns, layer_specs=specs, spec_types=types, weights_of=owners, streams=int(cfg["streams"]), num_heads=att["heads"],
+        num_kv_heads=att["kv_heads"], head_dim=att["dim"], rotary_dim=-1, rms_eps=float(cfg["norm"]["eps"]), tie_embeddings=True,
+        intermediate_size=max((s["mlp"]["ff"] for s, f in zip(specs, ffns) if f == "dense"), default=0),
+        num_experts=moe["router"]["experts"] if moe else 0, experts_per_token=moe["router"]["top"] if moe else 0,
+        moe_intermediate_size=moe["expert"]["ff"] if moe else 0, max_position=int(cfg["max_positions"]))
+
+
 def from_hf_config(cfg: dict, name: str = "model") -> ModelConfig:
     """Map a HF ``config.json`` dict (text stack) to ModelConfig; refuses unknown model types."""
+    if cfg.get("architecture") == "Pivipel":
+        return from_pivipel_config(cfg, name)
     if cfg.get("architecture") == "Fabulix":
         return from_fabulix_config(cfg, name)
     if cfg.get("architecture") == "Finelix":

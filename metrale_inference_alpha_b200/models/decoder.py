@@ -23,7 +23,7 @@ from ..ops import ACT_FOR_WEIGHT, Act
 from ..ops import reference as ref
 from ..ops import mixers
 from ..weights.loader import AttnW, FfnW, LayerW, ModelW
-from .stream import ResidualStream
+from .stream import HyperStream, ResidualStream
 
 
 class LayerCaches:
@@ -87,17 +87,17 @@ class Decoder:
         self.kv_cal = None                 # cache.fp8_calibration.Fp8KvCalibration while FP8 KV scales are being calibrated
         self.lora = None                   # lora.LoraManager when adapters are served
         self.calib = None                  # dict while calibrating static activation scales (engine/runner.py)
-        self._rotary = {}                  # (rotated dims, base) -> cos / sin tables of layers with their own rotation
+        self._rotary = {}                  # (rotated dims, base, scaling) -> cos / sin tables of layers with their own rotation
         self.side_head = None              # speculative.dflash.DflashDrafter: sees chosen layers' hidden states of every forward
 
     # ------------------------------------------------------------------ helpers
-    def rotary(self, dims: int, base: float):
-        """cos / sin [max_position, dims / 2] of a layer that names its own rotated size and base."""
+    def rotary(self, dims: int, base: float, scaling: Optional[dict] = None):
+        """cos / sin [max_position, dims / 2] of a layer that names its own rotated size, base and frequency scaling."""
         if dims <= 0:
             return None, None
-        key = (dims, float(base))
+        key = (dims, float(base), tuple(sorted(scaling.items())) if scaling else None)
         if key not in self._rotary:
-            self._rotary[key] = ref.rope_tables(self.cfg.max_position, dims, base, device=self.device)
+            self._rotary[key] = ref.rope_tables(self.cfg.max_position, dims, base, device=self.device, scaling=scaling)
         return self._rotary[key]
 
     def _norm_act(self, x, w, fmt: str, also_bf16: bool = False, res_only: bool = False) -> Act:
@@ -286,6 +286,9 @@ class Decoder:
 
     def layer(self, i: int, x, lw: LayerW, batch: ForwardBatch, caches: LayerCaches, kv=None, kv_idx=None, run: Optional[int] = None):
         """`run`: which cache and state this run of the layer has (the layer's own unless it is looped)."""
+        if isinstance(x, HyperStream):
+            from .hyper import hyper_layer
+            return hyper_layer(self, x, lw, batch, caches, i if run is None else run)
         if lw.out is not None:
             from .joint import joint_layer
             return joint_layer(self, x, lw, batch, caches, i if run is None else run)
@@ -332,7 +335,11 @@ class Decoder:
         return x
 
     # ------------------------------------------------------------------ full forward
-    def embed(self, token_ids: torch.Tensor) -> torch.Tensor:
+    def embed(self, token_ids: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if self.cfg.streams > 0:
+            x = mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale, pos=self.w.pos_embed, positions=positions,
+                                    norm=self.w.embed_norm)
+            return HyperStream(x, self.cfg.streams, self.cfg.act_fmt)
         if self.cfg.stream32:
             fmt, pair, W = self.cfg.act_fmt, None, self.cfg.hidden_size
             if self.w.loop_in is not None:
@@ -346,7 +353,7 @@ class Decoder:
 
     def backbone(self, batch: ForwardBatch, caches: LayerCaches) -> torch.Tensor:
         """Token ids -> final residual stream [T, hidden] (before the final norm)."""
-        x = self.embed(batch.token_ids)
+        x = self.embed(batch.token_ids, batch.positions)
         if getattr(batch, "embed_override", None) is not None:
             rows, emb = batch.embed_override
             x = x.index_copy(0, rows, emb.to(x.dtype))
@@ -411,9 +418,9 @@ class Decoder:
         [R, vocab / size] (greedy selection then merges per-rank maxima instead)."""
         x = self.backbone(batch, caches)
         if batch.logit_rows.numel() != x.shape[0]:
-            rows = self.full(x).index_select(0, batch.logit_rows)
+            rows = x.take(batch.logit_rows) if hasattr(x, "take") and not torch.is_tensor(x) else self.full(x).index_select(0, batch.logit_rows)
         else:
-            rows = x
+            rows = self.full(x) if isinstance(x, HyperStream) else x
         lg = self.logits(rows, out_f32=out_f32, gather=gather_logits)
         return lg, self.res(rows)
 

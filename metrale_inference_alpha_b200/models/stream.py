@@ -58,6 +58,10 @@ class ResidualStream:
         self._step(raw=True, out=self.pair[:, :self.x.shape[1]])
         self.x = ops.linear(mx.act_of(self.pair, self.fmt), w_in, out_f32=True, bias=step)
 
+    def take(self, rows: torch.Tensor) -> torch.Tensor:
+        """Chosen rows of x in fp32."""
+        return self.resolve().index_select(0, rows)
+
     @property
     def value(self) -> torch.Tensor:
         return self.resolve()
@@ -67,3 +71,50 @@ class ResidualStream:
         if self.y is not None:
             self._step()
         return self.x
+
+
+class HyperStream:
+    """The residual of models with static hyper-connections: S fp32 streams per token, read and written by every sublayer
+    with its own weights (``ops.mixers.HyperW``). One kernel joins the pending sublayer output and makes the next input."""
+
+    def __init__(self, x: torch.Tensor, streams: int, fmt: str):
+        self.x, self.S, self.fmt = x, streams, fmt      # [T, W] until the first sublayer has joined, then [T, S, W]
+        self.pending: Optional[mx.SublayerOut] = None
+        self.hc: Optional[mx.HyperW] = None
+        self.ones = None
+
+    @property
+    def shape(self):
+        return torch.Size((self.x.shape[0], self.x.shape[-1]))
+
+    def norm(self, pre: mx.DytNorm, hc: mx.HyperW) -> torch.Tensor:
+        """The next sublayer's input, pre(sum_s w_in[s] x_s)."""
+        return self._step(w_in=hc.w_in, pre=pre)
+
+    def add(self, out: mx.SublayerOut, hc: mx.HyperW) -> "HyperStream":
+        assert self.pending is None
+        self.pending, self.hc = out, hc
+        return self
+
+    def _step(self, **kw):
+        self.x, h = mx.stream_hyper(self.x, self.S, self.fmt, pending=self.pending, hc=self.hc, **kw)
+        if kw.get("rows") is None:
+            self.pending = self.hc = None
+        return h
+
+    def _sum(self, rows=None) -> torch.Tensor:
+        if self.ones is None:
+            self.ones = torch.ones(self.S, dtype=torch.float32, device=self.x.device)
+        return self._step(w_in=self.ones, out_f32=True, rows=rows)
+
+    def take(self, rows: torch.Tensor) -> torch.Tensor:
+        """The sum of the streams at chosen tokens, fp32; the streams themselves are left as they are."""
+        return self._sum(rows)
+
+    def resolve(self) -> torch.Tensor:
+        """The sum of the streams in fp32, nothing pending."""
+        return self._sum()
+
+    @property
+    def value(self) -> torch.Tensor:
+        return self.resolve()

@@ -514,7 +514,7 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     rt = runtime(act.data.device)
     n_out = N // 2 if (swiglu or clamp_glu or geglu) else N
     if grouped is not None:
-        n_out = grouped[3] // 2 if swiglu else grouped[3]
+        n_out = grouped[3] // 2 if (swiglu or clamp_glu) else grouped[3]
     if out is None and quant_out <= 0.0:
         out = torch.empty(M, n_out, dtype=torch.float32 if out_f32 else torch.bfloat16,
                           device=act.data.device)

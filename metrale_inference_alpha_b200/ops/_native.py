@@ -55,6 +55,7 @@ class AttnTcArgs(C.Structure):
         ("max_blocks", c_int), ("num_seqs", c_int), ("max_q_len", c_int), ("Hq", c_int), ("Hkv", c_int), ("D", c_int),
         ("block_size", c_int), ("cache_fp8", c_int), ("scale", c_float), ("v_mn", c_int),
         ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
+        ("sink_w", c_void_p), ("window", c_int), ("keep", c_int), ("gate", c_void_p), ("gate_ld", c_ll), ("gate_mode", c_int),
     ]
 
 
@@ -95,6 +96,7 @@ class AttnArgs(C.Structure):
         ("part_tokens", c_int), ("window", c_int), ("force_mode", c_int), ("status", c_void_p),
         ("outq", c_void_p), ("ldq", c_int), ("outq_sf", c_void_p), ("outq_sf_k64", c_int), ("outq_gs", c_float),
         ("DV", c_int), ("dv", c_int), ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
+        ("sink_w", c_void_p), ("keep", c_int), ("gate", c_void_p), ("gate_ld", c_ll), ("gate_mode", c_int),
     ]
 
 
@@ -153,6 +155,7 @@ def lib():
     L.mb_qk_norm_rope_kvwrite.restype = c_int
     L.mb_paged_attention.argtypes = [P(AttnArgs), c_void_p]
     L.mb_paged_attention.restype = c_int
+    L.mb_attn_visible.argtypes, L.mb_attn_visible.restype = [c_int] * 4, c_int
     L.mb_attn_ws_bytes.argtypes = [c_int, c_int, c_int, c_int, c_int]
     L.mb_attn_ws_bytes.restype = c_size_t
     L.mb_argmax.argtypes = [c_void_p, c_int, c_ll, c_int, c_int, c_void_p, c_void_p, c_int, c_int,

@@ -25,6 +25,7 @@
 // reshape_and_cache.cu, rope.cu, paged_decode_attn{,_fp8,_bf16_gqa,_fp8_gqa}.cu
 // (+ split-K reduce), prefill_paged_compute.cuh and attn_prefill_paged{,_fp8,_batched}.cu.
 #include "common.cuh"
+#include "visible.cuh"
 #include <type_traits>
 
 namespace {
@@ -256,9 +257,15 @@ struct AttnParams {
   long long out_ld;         // elements between consecutive tokens' output rows
   int dv;                   // value columns stored per head (<= the DV tile; the cache rows' padding is dropped)
   float out_scale;          // multiplies the normalised output
-  int sink;                 // one is added to the softmax denominator (a key of score 0 without a value)
+  int sink;                 // exp(sink_w[head]) is added to the softmax denominator (a key without a value), or one
+  const float* sink_w;      // [Hq] or null (score 0)
+  int keep;                 // with a window: the first tokens that every query sees
+  mb::OutputGate<__nv_bfloat16> gate;
   int split_p;              // the weights enter the product with V as two bf16 terms (16 mantissa bits)
 };
+
+// the sink's score in the log2 domain of the kernels' scores
+__device__ __forceinline__ float sink_log2(const AttnParams& p, int head) { return p.sink_w ? p.sink_w[head] * 1.44269504088896f : 0.f; }
 
 // Final store of four consecutive dims (c4 * 4 ..) of output row `orow` = token * Hq + head. In the
 // quantised mode the four lanes that share a 16-dim block agree on its scale with two shuffles;
@@ -283,8 +290,15 @@ __device__ __forceinline__ void store_out4(const AttnParams& p, size_t orow, int
     return;
   }
   const size_t m = orow / p.Hq;
-  __nv_bfloat16* dst = p.out + m * p.out_ld + (orow - m * p.Hq) * p.dv + c4 * 4;
-  const float os = p.out_scale;
+  const int head = (int)(orow - m * p.Hq);
+  __nv_bfloat16* dst = p.out + m * p.out_ld + (size_t)head * p.dv + c4 * 4;
+  const float os = p.gate.mode == mb::GATE_HEAD ? p.out_scale * p.gate(m, head, 0) : p.out_scale;
+  if (p.gate.mode == mb::GATE_ELEMENT) {
+    if (c4 * 4 < p.dv) a *= p.gate(m, head, c4 * 4);
+    if (c4 * 4 + 1 < p.dv) b *= p.gate(m, head, c4 * 4 + 1);
+    if (c4 * 4 + 2 < p.dv) c *= p.gate(m, head, c4 * 4 + 2);
+    if (c4 * 4 + 3 < p.dv) d *= p.gate(m, head, c4 * 4 + 3);
+  }
   if (p.dv == D) {
     *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a * os, b * os);
     *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(c * os, d * os);
@@ -467,15 +481,15 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
   const int qlen = p.q_len[seq], ctx = p.ctx_len[seq], qs = p.q_start[seq];
   const int R = G * qlen;
   if (qlen <= 0) return;
-  // partitions of one sequence: as many as a fixed partition size needs, then balanced
-  // (a function of this sequence's own length only, never of the rest of the batch)
-  const int nparts = max(1, (ctx + p.part_tokens - 1) / p.part_tokens);
+  // partitions of the tokens this sequence's queries see (counted in entries of the list, not in positions): as many as
+  // a fixed partition size needs, then balanced (a function of this sequence's own length only, never of the rest of
+  // the batch)
+  const mb::VisibleTokens vis(ctx - qlen, ctx, p.window, p.keep);
+  const int nparts = max(1, (vis.len + p.part_tokens - 1) / p.part_tokens);
   if (part >= nparts) return;
-  const int part_len = (((ctx + nparts - 1) / nparts) + 63) & ~63;
-  int tok_begin = part * part_len;
-  const int tok_end = min(ctx, tok_begin + part_len);
-  if (p.window > 0) tok_begin = max(tok_begin, (ctx - qlen + 1 - p.window) & ~63);
-  if (tok_begin < 0) tok_begin = 0;
+  const int part_len = (((vis.len + nparts - 1) / nparts) + 63) & ~63;
+  const int tok_begin = part * part_len;
+  const int tok_end = min(vis.len, tok_begin + part_len);
   const bool empty = tok_begin >= tok_end;
   const int* bt = p.block_table + (size_t)seq * p.max_blocks;
   const int ntiles = empty ? 0 : (tok_end - tok_begin + kTile - 1) / kTile;
@@ -486,10 +500,10 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
   const int bs = p.block_size;
   const bool fast_blocks = (bs == 16 || bs == 32 || bs == 64) && (p.part_tokens + 64) / bs <= kMaxBlk;
   const int bs_shift = 31 - __clz(bs);
-  if (!empty) {
-    const int first_blk = tok_begin / bs, nblk = (tok_end - 1) / bs - first_blk + 1;
+  if (!empty && fast_blocks) {
+    const int nblk = (tok_end - tok_begin + bs - 1) >> bs_shift;
     for (int i = tid; i < nblk && i < kMaxBlk; i += 128) {
-      int b = bt[first_blk + i];
+      int b = bt[vis.token(tok_begin + (i << bs_shift)) >> bs_shift];
       if (b < 0 || b >= p.num_blocks) {
         if (p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
         b = 0;
@@ -528,8 +542,9 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
           blk = s_blk[blk0 + (r >> bs_shift)];
           within = r & (bs - 1);                                      // tiles start on a block boundary
         } else {
-          blk = bt[tok / bs];
-          within = tok % bs;
+          const int at = vis.token(tok);
+          blk = bt[at / bs];
+          within = at % bs;
           if (blk < 0 || blk >= p.num_blocks) blk = 0;
         }
         off = ((size_t)blk * bs + within) * cp.row_pitch + (size_t)kvh * kRow + (size_t)c * 16;
@@ -619,7 +634,7 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
   }
   const float kmul = FP8 ? (*p.k_scale) : 1.f;
   const float sc_log2 = p.scale * kmul * 1.44269504088896f;
-  // rows of this thread: (mt, hr) -> causal limit; constant over the whole kernel
+  // rows of this thread: (mt, hr) -> causal limit (a position); constant over the whole kernel
   int lim[MT][2];
   int min_limit = 0x7fffffff;
 #pragma unroll
@@ -682,8 +697,10 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
       }
     }
     // online softmax over this warp's 16 tokens; the mask code only runs for tiles that
-    // touch a causal limit, the end of the range or a sliding window
-    const bool need_mask = (tok0 + 16 > min_limit) || (tok0 + 16 > tok_end) || (p.window > 0);
+    // touch a causal limit, the end of the range or the window's start
+    const int pos0 = vis.token(tok0);                  // the 16 entries are consecutive positions
+    const bool need_mask = (pos0 + 16 > min_limit) || (tok0 + 16 > tok_end) ||
+                           (p.window > 0 && pos0 < ctx - p.window && pos0 + 16 > p.keep);
     uint32_t pa[MT][4], pr[MT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
@@ -691,15 +708,14 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
       for (int hr = 0; hr < 2; ++hr) {
         float mx = -INFINITY;
         if (need_mask) {
-          const int limit = min(lim[mt][hr], tok_end);
-          const int wlo = p.window > 0 ? lim[mt][hr] - p.window : 0;
+          const int limit = lim[mt][hr];
 #pragma unroll
           for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-              const int tok = tok0 + n * 8 + t * 2 + i;
+              const int o = n * 8 + t * 2 + i;
               float v = s[mt][n][hr * 2 + i] * sc_log2;
-              if (tok >= limit || tok < wlo) v = -INFINITY;
+              if (tok0 + o >= tok_end || !mb::sees(pos0 + o, limit, p.window, p.keep)) v = -INFINITY;
               s[mt][n][hr * 2 + i] = v;
               mx = fmaxf(mx, v);
             }
@@ -838,9 +854,11 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
       lw[w] = s_ml[(w * MT * 16 + r) * 2 + 1];
       mx = fmaxf(mx, mw[w]);
     }
+    const int tq = r / G, hh = r - tq * G;
     const bool sink_here = p.sink && nparts == 1;
-    if (sink_here) mx = fmaxf(mx, 0.f);
-    float l = sink_here ? exp2f(-mx) : 0.f;
+    const float sk = sink_here ? sink_log2(p, kvh * G + hh) : 0.f;
+    if (sink_here) mx = fmaxf(mx, sk);
+    float l = sink_here ? exp2f(sk - mx) : 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
@@ -851,7 +869,6 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
     }
     const float inv = l > 0.f ? vmul / l : 0.f;
     acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
-    const int tq = r / G, hh = r - tq * G;
     const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
     if (nparts == 1) {
       store_out4<DV>(p, orow, c4, acc.x, acc.y, acc.z, acc.w);
@@ -883,8 +900,9 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
     const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
     float mx = -INFINITY;
     for (int s2 = 0; s2 < nparts; ++s2) mx = fmaxf(mx, __ldcg(&p.part_ml[(orow * p.parts + s2) * 2]));
-    if (p.sink) mx = fmaxf(mx, 0.f);
-    float denom = p.sink ? exp2f(-mx) : 0.f;
+    const float sk = p.sink ? sink_log2(p, kvh * G + hh) : 0.f;
+    if (p.sink) mx = fmaxf(mx, sk);
+    float denom = p.sink ? exp2f(sk - mx) : 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s2 = 0; s2 < nparts; ++s2) {
       const float m = __ldcg(&p.part_ml[(orow * p.parts + s2) * 2]);
@@ -923,9 +941,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
   const int* bt = p.block_table + (size_t)seq * p.max_blocks;
   const int past = ctx - qlen;                                 // tokens cached before this chunk
   const int tok_end = min(ctx, past + q0 + 64);                // causal upper bound for the tile
-  int tok_begin = 0;
-  if (p.window > 0) tok_begin = max(0, past + q0 + 1 - p.window);
-  tok_begin &= ~63;
+  const mb::VisibleTokens vis(past + q0, tok_end, p.window, p.keep);
 
   for (int idx = tid; idx < 64 * (DK / 8); idx += 128) {
     const int r = idx / (DK / 8), c = idx - r * (DK / 8);
@@ -959,22 +975,21 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
 
   TileLoader<DK, FP8> ldK;
   TileLoader<DV, FP8> ldV;
-  const int ntiles = (tok_end - tok_begin + kTile - 1) / kTile;
-  ldK.fetch(p, p.k_cache, bt, kvh, tok_begin, tok_end, tid, sK);
-  ldV.fetch(p, p.v_cache, bt, kvh, tok_begin, tok_end, tid, sV);
+  const int ntiles = (vis.len + kTile - 1) / kTile;
+  ldK.fetch(p, p.k_cache, bt, kvh, vis.token(0), tok_end, tid, sK);
+  ldV.fetch(p, p.v_cache, bt, kvh, vis.token(0), tok_end, tid, sV);
   for (int it = 0; it < ntiles; ++it) {
     const int buf = it & 1;
     ldK.commit(sK + buf * kTileBytesK, tid);
     ldV.commit(sV + buf * kTileBytesV, tid);
     __syncthreads();
     if (it + 1 < ntiles) {
-      ldK.fetch(p, p.k_cache, bt, kvh, tok_begin + (it + 1) * kTile, tok_end, tid,
-                sK + (buf ^ 1) * kTileBytesK);
-      ldV.fetch(p, p.v_cache, bt, kvh, tok_begin + (it + 1) * kTile, tok_end, tid,
-                sV + (buf ^ 1) * kTileBytesV);
+      const int next = vis.token((it + 1) * kTile);
+      ldK.fetch(p, p.k_cache, bt, kvh, next, tok_end, tid, sK + (buf ^ 1) * kTileBytesK);
+      ldV.fetch(p, p.v_cache, bt, kvh, next, tok_end, tid, sV + (buf ^ 1) * kTileBytesV);
     }
     const uint32_t kT = sK + buf * kTileBytesK, vT = sV + buf * kTileBytesV;
-    const int tile_tok0 = tok_begin + it * kTile;
+    const int tile_tok0 = vis.token(it * kTile);
     // S[16 x 64] for this warp
     float s[8][4];
 #pragma unroll
@@ -999,7 +1014,6 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
     for (int hr = 0; hr < 2; ++hr) {
       const int qr = q0 + warp * 16 + (lane >> 2) + hr * 8;    // query index inside the chunk
       const int limit = past + qr + 1;
-      const int wlo = p.window > 0 ? limit - p.window : 0;
       float mx = -INFINITY;
 #pragma unroll
       for (int n = 0; n < 8; ++n)
@@ -1007,7 +1021,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
         for (int i = 0; i < 2; ++i) {
           const int tok = tile_tok0 + n * 8 + (lane & 3) * 2 + i;
           float v = s[n][hr * 2 + i] * sc_log2;
-          if (tok >= limit || tok >= tok_end || tok < wlo || qr >= qlen) v = -INFINITY;
+          if (tok >= tok_end || qr >= qlen || !mb::sees(tok, limit, p.window, p.keep)) v = -INFINITY;
           s[n][hr * 2 + i] = v;
           mx = fmaxf(mx, v);
         }
@@ -1075,9 +1089,18 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
     const int qr = q0 + warp * 16 + (lane >> 2) + hr * 8;
     if (qr >= qlen) continue;
     // the sink's share of the denominator, at this row's running maximum (every row has seen a key)
-    if (p.sink) l += exp2f(-m_run[hr]);
-    const float inv = (l > 0.f ? vmul / l : 0.f) * p.out_scale;
+    if (p.sink) l += exp2f(sink_log2(p, head) - m_run[hr]);
+    const float inv = (l > 0.f ? vmul / l : 0.f) * p.out_scale * (p.gate.mode == mb::GATE_HEAD ? p.gate(qs + qr, head, 0) : 1.f);
     __nv_bfloat16* dst = p.out + (size_t)(qs + qr) * p.out_ld + (size_t)head * p.dv + (lane & 3) * 2;
+    if (p.gate.mode == mb::GATE_ELEMENT) {
+#pragma unroll
+      for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int d = n * 8 + (lane & 3) * 2 + i;
+          if (d < p.dv) o_acc[n][hr * 2 + i] *= p.gate(qs + qr, head, d);
+        }
+    }
     if (p.dv == DV) {
 #pragma unroll
       for (int n = 0; n < DV / 8; ++n)
@@ -1224,7 +1247,20 @@ struct MbAttnArgs {
   long long out_ld;        // elements between output rows (0 = Hq * dv)
   float out_scale;         // 0 = 1
   int sink, split_p;
+  const float* sink_w;     // [Hq] sink scores (null: 0), with sink
+  int keep;                // with window: first tokens that stay visible
+  const void* gate;        // logits of sigmoid gates on the output (bf16), or null
+  long long gate_ld;
+  int gate_mode;           // 1 one per head, 2 one per element
 };
+
+// most entries of the visible-token list of a sequence: its context, or the kept first tokens and the windows of its
+// queries, each rounded to whole tiles
+int mb_attn_visible(int max_ctx, int max_q_len, int window, int keep) {
+  if (window <= 0) return max_ctx;
+  const long long n = ((long long)keep + 63) / 64 * 64 + window + max_q_len + 63;
+  return n < max_ctx ? (int)n : max_ctx;
+}
 
 // workspace bytes for the split-KV path
 size_t mb_attn_ws_bytes(int total_rows, int Hq, int D, int max_ctx, int part_tokens) {
@@ -1252,9 +1288,12 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
   p.out_ld = a->out_ld > 0 ? a->out_ld : (long long)a->Hq * p.dv;
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.f;
   p.sink = a->sink; p.split_p = a->split_p;
+  p.sink_w = a->sink_w; p.keep = a->window > 0 ? a->keep : 0;
+  p.gate = {reinterpret_cast<const __nv_bfloat16*>(a->gate), a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, p.dv};
+  if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
   if (p.dv > DV || p.out_ld < (long long)a->Hq * p.dv) return MB_ERR_BAD_ARG;
   if (p.dv == DV && (p.out_ld % 2 || (reinterpret_cast<uintptr_t>(a->out) & 3))) return MB_ERR_BAD_ARG;   // paired stores
-  if ((DV != a->D || p.sink || p.split_p || p.dv != DV) && (a->cache_fp8 || a->outq || a->window)) return MB_ERR_UNSUPPORTED;
+  if ((DV != a->D || p.sink || p.split_p || p.dv != DV || p.gate.mode) && (a->cache_fp8 || a->outq)) return MB_ERR_UNSUPPORTED;
   const int G = a->Hq / a->Hkv;
   const int rows = G * a->max_q_len;
   int mode = a->force_mode;
@@ -1271,7 +1310,7 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
     if (rows > 32) return MB_ERR_UNSUPPORTED;
     const int mt = rows <= 16 ? 1 : 2;
     p.part_tokens = a->part_tokens > 0 ? a->part_tokens : 512;
-    p.parts = (a->max_ctx + p.part_tokens - 1) / p.part_tokens;
+    p.parts = (mb_attn_visible(a->max_ctx, a->max_q_len, p.window, p.keep) + p.part_tokens - 1) / p.part_tokens;
     if (p.parts < 1) p.parts = 1;
     if (p.parts > 1) {
       const size_t cnt_bytes = ((size_t)a->num_seqs * a->Hkv * sizeof(uint32_t) + 255) & ~size_t(255);

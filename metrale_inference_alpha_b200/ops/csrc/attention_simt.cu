@@ -1,12 +1,14 @@
 // Paged causal attention on the CUDA cores in fp32 arithmetic: any query/key and value head size (up to
-// 2048 / 1024), bf16 or fp32 cache, optional sink (one added to the softmax denominator). It serves models that
-// run in true 32-bit, and head sizes beyond the tensor-core kernels' tiles.
+// 2048 / 1024), bf16 or fp32 cache, optional sink (a key without a value: score 0, or one per head), window with kept
+// first tokens, sigmoid gates on the output. It serves models that run in true 32-bit, and head sizes beyond the
+// tensor-core kernels' tiles.
 //
 // One CTA per (query head, query row), 128 threads. Per tile of 128 cached tokens: thread j scores token j
 // (dot product over the query held in shared memory), the block agrees on the running maximum and sum, and
 // thread d accumulates value columns d, d + 128, ... over the tile. Cache rows are [slot, kv head, dkp] and
 // [slot, kv head, dvp]; the padding columns are never read.
 #include "common.cuh"
+#include "visible.cuh"
 
 namespace {
 
@@ -23,6 +25,11 @@ struct SimtAttnParams {
   long long num_blocks;
   float scale, out_scale;
   int sink;
+  const float* sink_w;       // [Hq] or null
+  int window, keep;
+  const void* gate;
+  long long gate_ld;
+  int gate_mode;
   void* out;                 // row stride out_ld, head stride dv
   long long out_ld;
   uint32_t* status;
@@ -61,33 +68,37 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const SimtAttnParams p) 
 #pragma unroll
   for (int i = 0; i < kMaxDv / 128; ++i) acc[i] = 0.f;
   // the sink is a key of score 0 without a value: it starts the running maximum and sum
-  float m = p.sink ? 0.f : -INFINITY, l = p.sink ? 1.f : 0.f;
-  for (int j0 = 0; j0 < limit; j0 += 128) {
+  float m = p.sink ? (p.sink_w ? p.sink_w[head] : 0.f) : -INFINITY, l = p.sink ? 1.f : 0.f;
+  // one query: the visible tokens are the kept first ones and the window behind them, exactly
+  const int begin = p.window > 0 ? max(0, limit - p.window) : 0;
+  const int kept = min(p.keep, begin), shift = begin - kept, len = limit - shift;
+  for (int j0 = 0; j0 < len; j0 += 128) {
     __syncthreads();                       // sq ready / the previous tile's sp and sslot consumed
     const int j = j0 + tid;
     float s = -INFINITY;
     long long slot = 0;
-    if (j < limit) {
-      long long blk = bt[j / p.block_size];
+    if (j < len) {
+      const int tok = j < kept ? j : j + shift;
+      long long blk = bt[tok / p.block_size];
       if (blk < 0 || blk >= p.num_blocks) {
         if (p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
         blk = 0;
       }
-      slot = blk * p.block_size + j % p.block_size;
+      slot = blk * p.block_size + tok % p.block_size;
       const T* k = reinterpret_cast<const T*>(p.k_cache) + ((size_t)slot * p.Hkv + kvh) * p.dkp;
       float a = 0.f;
       for (int d = 0; d < p.dk; ++d) a = fmaf(sq[d], lda(k + d), a);
       s = a * p.scale;
     }
     const float m_new = fmaxf(m, mb::block_max(s, red));
-    const float e = j < limit ? expf(s - m_new) : 0.f;
+    const float e = j < len ? expf(s - m_new) : 0.f;
     sp[tid] = e;
     sslot[tid] = slot;
     const float sum = mb::block_sum(e, red);       // its barriers also publish sp and sslot
     const float alpha = expf(m - m_new);
     l = l * alpha + sum;
     m = m_new;
-    const int cnt = min(128, limit - j0);
+    const int cnt = min(128, len - j0);
 #pragma unroll
     for (int i = 0; i < kMaxDv / 128; ++i) {
       const int d = tid + i * 128;
@@ -100,13 +111,15 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const SimtAttnParams p) 
     }
   }
   const float inv = p.out_scale / l;
+  const mb::OutputGate<T> gate{reinterpret_cast<const T*>(p.gate), p.gate_ld, p.gate_mode, p.dv};
   T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.out_ld + (size_t)head * p.dv;
 #pragma unroll
   for (int i = 0; i < kMaxDv / 128; ++i) {
     const int d = tid + i * 128;
     if (d < p.dv) {
-      if constexpr (sizeof(T) == 2) out[d] = __float2bfloat16(acc[i] * inv);
-      else out[d] = acc[i] * inv;
+      const float v = acc[i] * inv * gate((size_t)t, head, d);
+      if constexpr (sizeof(T) == 2) out[d] = __float2bfloat16(v);
+      else out[d] = v;
     }
   }
 }
@@ -129,6 +142,11 @@ struct MbSimtAttnArgs {
   void* out;
   long long out_ld;
   uint32_t* status;
+  const float* sink_w;
+  int window, keep;
+  const void* gate;
+  long long gate_ld;
+  int gate_mode;
 };
 
 extern "C" int mb_attn_simt(const MbSimtAttnArgs* a, cudaStream_t stream) {
@@ -136,7 +154,9 @@ extern "C" int mb_attn_simt(const MbSimtAttnArgs* a, cudaStream_t stream) {
   if (a->Hkv <= 0 || a->Hq % a->Hkv || a->dk <= 0 || a->dv <= 0 || a->dv > kMaxDv || a->dk > 2048 || a->dk > a->dkp || a->dv > a->dvp) return MB_ERR_UNSUPPORTED;
   if (a->total_rows > 65535) return MB_ERR_TOO_LARGE;
   SimtAttnParams p{a->q, a->k_cache, a->v_cache, a->block_table, a->max_blocks, a->q_start, a->q_len, a->ctx_len, a->num_seqs, a->Hq, a->Hkv,
-                   a->dk, a->dv, a->dkp, a->dvp, a->block_size, a->num_blocks, a->scale, a->out_scale, a->sink, a->out, a->out_ld, a->status};
+                   a->dk, a->dv, a->dkp, a->dvp, a->block_size, a->num_blocks, a->scale, a->out_scale, a->sink, a->sink_w, a->window, a->window > 0 ? a->keep : 0,
+                   a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->out, a->out_ld, a->status};
+  if (p.keep < 0 || p.gate_mode < 0 || p.gate_mode > mb::GATE_ELEMENT) return MB_ERR_BAD_ARG;
   const dim3 grid(a->Hq, a->total_rows);
   const size_t smem = (size_t)a->dk * sizeof(float);
   if (a->f32) return (int)mb::launch_kernel(attn_simt_kernel<float>, grid, dim3(128), smem, stream, p);

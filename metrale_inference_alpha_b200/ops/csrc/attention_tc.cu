@@ -20,15 +20,17 @@
 // softmax overlap the other's tensor work. Every wait on an mbarrier is bounded and reports
 // through the status word; TMEM is freed on every path.
 //
-// Softmax variants: a sink (one added to the denominator), and SPLIT, in which the weights enter the
+// Variants: a window with kept first tokens (the tiles of the visible-token list are walked), sigmoid gates on the
+// output, a sink (a key without a value: score 0, or one per head), and SPLIT, in which the weights enter the
 // product with V as two bf16 terms (hi + rest: 16 mantissa bits), for models whose attention weights are
 // 32-bit quantities; the output may be a column range of a wider matrix and takes a constant factor.
 //
-// Serves q_len >= 128 chunks with head_dim 128, bf16 or e4m3 caches, no sliding window; other
+// Serves q_len >= 128 chunks with head_dim 128 or 256, bf16 or e4m3 caches; other
 // shapes stay on the mma.sync kernels in attention.cu, which are also the oracle in the tests.
 // Reference behaviour covered: the prefill paged-attention family
 // (kernels/gb10/common/prefill_paged_compute.cuh:3-7,37-41), re-designed for TMEM accumulators.
 #include "common.cuh"
+#include "visible.cuh"
 
 namespace {
 
@@ -54,6 +56,9 @@ struct TcParams {
   long long out_ld;
   float out_scale;
   int sink;
+  const float* sink_w;           // [Hq] or null (score 0)
+  int window, keep;
+  mb::OutputGate<__nv_bfloat16> gate;
   uint32_t* status;
 };
 
@@ -142,7 +147,9 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   const int limit = row_ok ? ctx - qlen + qi + 1 : 0;                // tokens [0, limit) are visible
   const int first_limit = (qlen - q0 >= kQ) ? ctx - qlen + q0 + 1 : 0;  // smallest limit of the CTA's rows (0: ragged tile, always mask)
   const int last_row = min(qlen, q0 + kQ) - 1;
-  const int tiles = (ctx - qlen + last_row + 1 + kT - 1) / kT;        // up to the last row's limit
+  const int last_limit = ctx - qlen + last_row + 1;
+  const mb::VisibleTokens vis(ctx - qlen + q0, last_limit, p.window, p.keep);
+  const int tiles = (vis.len + kT - 1) / kT;
   const float kmul = FP8 ? (*p.k_scale) * 256.f : 1.f;
   const float sc_log2 = p.scale * kmul * 1.44269504088896f;
   float m_run = -INFINITY, l_run = 0.f;
@@ -155,7 +162,7 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   constexpr int kRaw = FP8 ? 4 : 8;
   uint4 kraw[kNHT][kRaw], vraw[kNHT][kRaw];
   auto fetch = [&](int jt) {
-    const int tok = jt * kT + s_tok;
+    const int tok = vis.token(jt * kT) + s_tok;
     if (jt < tiles && tok < ctx) {
       long long blk = bt[tok / p.block_size];
       if (blk < 0 || blk >= p.num_blocks) {
@@ -247,8 +254,8 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
 #pragma unroll
       for (int c = 0; c < kT / 16; ++c) mb::tmem_ld16(t_row + c * 16, sv + c * 16);
       float mx = -INFINITY;
-      const int tok0 = j * kT;
-      if (tok0 + kT <= first_limit) {                    // the whole tile is visible to every row of this CTA
+      const int tok0 = vis.token(j * kT);
+      if (tok0 + kT <= first_limit && (p.window <= 0 || tok0 >= last_limit - p.window || tok0 + kT <= p.keep)) {   // visible to every row of this CTA
 #pragma unroll
         for (int i = 0; i < kT; ++i) {
           sv[i] *= sc_log2;
@@ -257,7 +264,7 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
       } else {
 #pragma unroll
         for (int i = 0; i < kT; ++i) {
-          const float v = (tok0 + i < limit) ? sv[i] * sc_log2 : -INFINITY;
+          const float v = mb::sees(tok0 + i, limit, p.window, p.keep) ? sv[i] * sc_log2 : -INFINITY;
           sv[i] = v;
           mx = fmaxf(mx, v);
         }
@@ -327,13 +334,29 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
   }
   if (ok) {                                               // uniform: tcgen05.ld is a whole-warp instruction
     const float vmul = FP8 ? (*p.v_scale) * 256.f : 1.f;
-    if (p.sink) l_run += ex2(-m_run);                     // the sink's weight at this row's running maximum
-    const float inv = (l_run > 0.f ? vmul / l_run : 0.f) * p.out_scale;
+    // the sink's weight at this row's running maximum
+    if (p.sink) l_run += ex2((p.sink_w ? p.sink_w[head] * 1.44269504088896f : 0.f) - m_run);
+    const size_t row = (size_t)qs + (row_ok ? qi : 0);
+    const float inv = (l_run > 0.f ? vmul / l_run : 0.f) * p.out_scale * (p.gate.mode == mb::GATE_HEAD ? p.gate(row, head, 0) : 1.f);
     uint4* dst = reinterpret_cast<uint4*>(p.out + (size_t)(qs + (row_ok ? qi : 0)) * p.out_ld + (size_t)head * kD);
 #pragma unroll
     for (int c = 0; c < kD / 16; ++c) {
       float ov[16];
       mb::tmem_ld16(t_row + 64 + c * 16, ov);             // every lane reads; only rows of the sequence store
+      if (p.gate.mode == mb::GATE_ELEMENT) {
+        const uint4* gz = reinterpret_cast<const uint4*>(p.gate.logits + row * p.gate.ld + (size_t)head * kD + c * 16);
+#pragma unroll
+        for (int h2 = 0; h2 < 2; ++h2) {
+          const uint4 g8 = __ldg(gz + h2);
+          const __nv_bfloat162* gb = reinterpret_cast<const __nv_bfloat162*>(&g8);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(gb[i]);
+            ov[h2 * 8 + 2 * i] *= __fdividef(1.f, 1.f + __expf(-f.x));
+            ov[h2 * 8 + 2 * i + 1] *= __fdividef(1.f, 1.f + __expf(-f.y));
+          }
+        }
+      }
 #pragma unroll
       for (int h2 = 0; h2 < 2; ++h2) {
         uint4 w;
@@ -382,6 +405,11 @@ struct MbAttnTcArgs {
   long long out_ld;    // elements between output rows (0 = Hq * D)
   float out_scale;     // 0 = 1
   int sink, split_p;
+  const float* sink_w; // [Hq] sink scores (null: 0), with sink
+  int window, keep;    // 0 = no window; the first `keep` tokens stay visible
+  const void* gate;    // logits of sigmoid gates on the output (bf16), or null
+  long long gate_ld;
+  int gate_mode;       // 1 one per head, 2 one per element
 };
 
 // Causal paged attention for prefill chunks (head dim 128). Returns 0, MB_ERR_* or a CUDA error.
@@ -398,7 +426,11 @@ extern "C" int mb_attn_prefill_tc(const MbAttnTcArgs* a, cudaStream_t stream) {
   p.out = (__nv_bfloat16*)a->out; p.status = a->status;
   p.out_ld = a->out_ld > 0 ? a->out_ld : (long long)a->Hq * a->D;
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.f;
-  p.sink = a->sink;
+  p.sink = a->sink; p.sink_w = a->sink_w;
+  p.window = a->window; p.keep = a->window > 0 ? a->keep : 0;
+  p.gate = {(const __nv_bfloat16*)a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->D};
+  if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
+  if (p.gate.mode == mb::GATE_ELEMENT && (a->gate_ld % 8 || (reinterpret_cast<uintptr_t>(a->gate) & 15))) return MB_ERR_UNSUPPORTED;
   if (p.out_ld % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15)) return MB_ERR_BAD_ARG;      // 16-byte stores
   if (a->split_p && a->cache_fp8) return MB_ERR_UNSUPPORTED;
   const size_t smem = (size_t)(a->D / 64) * (kQ + 2 * kT) * 128 + (a->split_p ? 2 : 1) * kQ * 128 + 1024;

@@ -1,11 +1,12 @@
 // Mixture-of-experts support kernels (the expert FFN itself is the grouped mode of the
 // tcgen05 GEMM in gemm_tcgen05.cu).
 //
-//   mb_moe_route    one warp per token over <= 512 expert logits: softmax top-k, or sigmoid
-//                   scores + selection bias with group-limited selection (keep the
-//                   `topk_group` groups with the largest sum of their two best biased scores,
-//                   then top-k inside them), or the softmax over the chosen ones of biased
-//                   logits (mode 2, 32-bit throughout). Ties resolve to the lower expert id.
+//   mb_moe_route    one warp per token over <= 512 expert logits: softmax top-k (mode 0), or sigmoid
+//                   scores + selection bias (mode 1), both with group-limited selection (keep the
+//                   `topk_group` groups with the largest score, mode 0, or the largest sum of their
+//                   two best biased scores, mode 1; then top-k inside them), or the softmax over the
+//                   chosen ones of biased logits (mode 2, 32-bit throughout). Ties resolve to the
+//                   lower expert id.
 //                   Weights are the un-biased scores, optionally sum-normalised and scaled.
 //   mb_moe_sort     counting sort of the (token, slot) pairs by *local* expert: per-expert row
 //                   ranges, the pair -> row map, and a tile work-list of (expert, first row,
@@ -57,7 +58,7 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
     float se = 0.f;
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
-      score[j] = score[j] == -INFINITY ? 0.f : __expf(score[j] - mx);
+      score[j] = score[j] == -INFINITY ? 0.f : expf(score[j] - mx);
       se += score[j];
     }
     se = mb::warp_sum(se);
@@ -76,48 +77,48 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
       score[j] = ok ? 1.f / (1.f + __expf(-score[j])) : 0.f;
       sel[j] = ok ? score[j] + (bias ? bias[e] : 0.f) : -INFINITY;
     }
-    if (n_group > 1) {
-      // group g owns experts [g * gs, (g + 1) * gs); score = sum of its two best sel values
-      const int gs = E / n_group;
-      float gscore_mine = -INFINITY;  // lane g (< n_group) keeps group g's score
-      for (int g = 0; g < n_group; ++g) {
-        float b1 = -INFINITY, b2 = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < kMaxPerLane; ++j) {
-          const int e = j * 32 + lane;
-          if (j < per && e >= g * gs && e < (g + 1) * gs) {
-            const float v = sel[j];
-            if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
-          }
-        }
-        // merge (b1, b2) pairs across lanes
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float o1 = __shfl_xor_sync(0xffffffffu, b1, o), o2 = __shfl_xor_sync(0xffffffffu, b2, o);
-          const float n1 = fmaxf(b1, o1);
-          const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
-          b1 = n1; b2 = n2;
-        }
-        if (lane == g) gscore_mine = b1 + b2;
-      }
-      // pick topk_group groups (ties -> lower group id); keep-mask as a bit set
-      uint32_t keep = 0;
-      for (int r = 0; r < topk_group; ++r) {
-        float v = (lane < n_group && !((keep >> lane) & 1)) ? gscore_mine : -INFINITY;
-        int idx = lane;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-          const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
-          if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
-        }
-        keep |= 1u << idx;
-      }
+  }
+  if (n_group > 1 && mode != 2) {
+    // group g owns experts [g * gs, (g + 1) * gs); score = its best sel value, or the sum of its two best
+    const int gs = E / n_group;
+    float gscore_mine = -INFINITY;  // lane g (< n_group) keeps group g's score
+    for (int g = 0; g < n_group; ++g) {
+      float b1 = -INFINITY, b2 = -INFINITY;
 #pragma unroll
       for (int j = 0; j < kMaxPerLane; ++j) {
         const int e = j * 32 + lane;
-        if (j < per && e < E && !((keep >> (e / gs)) & 1)) sel[j] = -INFINITY;
+        if (j < per && e >= g * gs && e < (g + 1) * gs) {
+          const float v = sel[j];
+          if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
+        }
       }
+      // merge (b1, b2) pairs across lanes
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float o1 = __shfl_xor_sync(0xffffffffu, b1, o), o2 = __shfl_xor_sync(0xffffffffu, b2, o);
+        const float n1 = fmaxf(b1, o1);
+        const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
+        b1 = n1; b2 = n2;
+      }
+      if (lane == g) gscore_mine = mode == 0 ? b1 : b1 + b2;
+    }
+    // pick topk_group groups (ties -> lower group id); keep-mask as a bit set
+    uint32_t keep = 0;
+    for (int r = 0; r < topk_group; ++r) {
+      float v = (lane < n_group && !((keep >> lane) & 1)) ? gscore_mine : -INFINITY;
+      int idx = lane;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
+        if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
+      }
+      keep |= 1u << idx;
+    }
+#pragma unroll
+    for (int j = 0; j < kMaxPerLane; ++j) {
+      const int e = j * 32 + lane;
+      if (j < per && e < E && !((keep >> (e / gs)) & 1)) sel[j] = -INFINITY;
     }
   }
   // iterative top-k over sel; weights come from score

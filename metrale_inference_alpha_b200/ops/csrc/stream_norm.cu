@@ -17,61 +17,17 @@
 //   gated_norm    RMS over groups of channels x weight x act(gate) x scale, act = SiLU or sigmoid; the
 //                 output may be a column range of a wider matrix
 //   side_gate     gelu_tanh(z) * e, e gathered from a per-layer slice of a second embedding table
-//   embed_scaled  fp32 embedding rows times a constant, optionally with a copy in the activation type
-//   rope_dims     rotate-half positions on q and k with separate query/key and value head sizes, scattered
-//                 into a paged cache whose rows are padded (with zeros) to the attention kernel's tile
+//   embed_scaled  fp32 embedding rows times a constant, optionally plus a learned position row, through a Dynamic
+//                 Tanh, or with a copy in the activation type
+//   rope_dims     per-head RMS norms (optional) and rotate-half positions (optional) on q and k with separate query/key
+//                 and value head sizes, scattered into a paged cache whose rows are padded (with zeros) to the
+//                 attention kernel's tile
 // T is the activation type: bf16, or fp32 for models served in 32-bit.
 #include "common.cuh"
 #include "epilogue.cuh"
+#include "row_io.cuh"
 
 namespace {
-
-using bf16 = __nv_bfloat16;
-
-template <typename T>
-__device__ __forceinline__ float ldv(const T* p) {
-  if constexpr (sizeof(T) == 2) return __bfloat162float(*p);
-  else return *p;
-}
-template <typename T>
-__device__ __forceinline__ void stv(T* p, float v) {
-  if constexpr (sizeof(T) == 2) *p = __float2bfloat16(v);
-  else *p = v;
-}
-// VEC consecutive elements <-> floats (VEC is 1 or 4; 4 needs the natural vector alignment)
-template <int VEC, typename T>
-__device__ __forceinline__ void ldn(const T* p, float* o) {
-  if constexpr (VEC == 1) {
-    o[0] = ldv(p);
-  } else if constexpr (sizeof(T) == 2) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
-    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
-  } else {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
-  }
-}
-template <int VEC, typename T>
-__device__ __forceinline__ void stn(T* p, const float* o) {
-  if constexpr (VEC == 1) {
-    stv(p, o[0]);
-  } else if constexpr (sizeof(T) == 2) {
-    uint2 v;
-    *reinterpret_cast<__nv_bfloat162*>(&v.x) = __floats2bfloat162_rn(o[0], o[1]);
-    *reinterpret_cast<__nv_bfloat162*>(&v.y) = __floats2bfloat162_rn(o[2], o[3]);
-    *reinterpret_cast<uint2*>(p) = v;
-  } else {
-    *reinterpret_cast<float4*>(p) = make_float4(o[0], o[1], o[2], o[3]);
-  }
-}
-
-struct DytW {
-  float alpha;
-  const bf16* w;
-  const bf16* b;
-};
 
 enum { ADD_NONE = 0, ADD_DYT = 1, ADD_RMS = 2 };
 enum { OUT_NONE = 0, OUT_DYT = 1, OUT_RAW = 2 };
@@ -405,23 +361,51 @@ __global__ void __launch_bounds__(256) tanh_split_kernel(const float* z, bf16* o
   out[t * 2 * R + R + c] = __float2bfloat16(v - __bfloat162float(h));
 }
 
+struct EmbedParams {
+  const int* tokens;
+  const bf16* table;
+  float* out;
+  int W, vocab;
+  float scale;
+  void* copy;                // [M, W] of the activation type, rows copy_ld apart, or null
+  long long copy_ld;
+  const int* positions;      // with pos
+  const bf16* pos;           // [max_pos, W] added to the scaled row, or null
+  int max_pos;
+  DytW norm;                 // w null: none
+  uint32_t* status;
+};
+
 template <int VEC, typename T>
-__global__ void __launch_bounds__(256) embed_scaled_kernel(const int* tokens, const bf16* table, float* out, int W, int vocab, float scale,
-                                                           T* copy, long long copy_ld, uint32_t* status) {
+__global__ void __launch_bounds__(256) embed_scaled_kernel(const EmbedParams p) {
   mb::pdl_wait();
   mb::pdl_launch_dependents();
-  const int t = blockIdx.x, tok = tokens[t];
-  const bool ok = tok >= 0 && tok < vocab;
-  if (!ok && status && threadIdx.x == 0) atomicCAS(status, 0u, MB_ST_BOUNDS);
+  const int t = blockIdx.x, tok = p.tokens[t], W = p.W;
+  const int at = p.pos ? p.positions[t] : 0;
+  const bool ok = tok >= 0 && tok < p.vocab, at_ok = p.pos && at >= 0 && at < p.max_pos;
+  if ((!ok || (p.pos && !at_ok)) && p.status && threadIdx.x == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
   for (int k = threadIdx.x * VEC; k < W; k += blockDim.x * VEC) {
     float v[VEC];
 #pragma unroll
     for (int i = 0; i < VEC; ++i) v[i] = 0.f;
-    if (ok) ldn<VEC>(table + (size_t)tok * W + k, v);
+    if (ok) ldn<VEC>(p.table + (size_t)tok * W + k, v);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[i] *= scale;
-    stn<VEC>(out + (size_t)t * W + k, v);
-    if (copy) stn<VEC>(copy + (size_t)t * copy_ld + k, v);
+    for (int i = 0; i < VEC; ++i) v[i] *= p.scale;
+    if (at_ok) {
+      float a[VEC];
+      ldn<VEC>(p.pos + (size_t)at * W + k, a);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] += a[i];
+    }
+    if (p.norm.w) {
+      float w[VEC], b[VEC];
+      ldn<VEC>(p.norm.w + k, w);
+      ldn<VEC>(p.norm.b + k, b);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = dyt(v[i], p.norm.alpha, w[i], b[i]);
+    }
+    stn<VEC>(p.out + (size_t)t * W + k, v);
+    if (p.copy) stn<VEC>(reinterpret_cast<T*>(p.copy) + (size_t)t * p.copy_ld + k, v);
   }
 }
 
@@ -440,6 +424,9 @@ struct RopeDimsParams {
   void* v_cache;
   long long num_slots;
   uint32_t* status;
+  const bf16* q_norm;        // [dk] per-head RMS norm weights, or null
+  const bf16* k_norm;
+  float eps;
 };
 
 // grid (tokens, y): the y CTAs of a token share its q | k | v output elements
@@ -499,6 +486,87 @@ __global__ void __launch_bounds__(256) rope_dims_kernel(const RopeDimsParams p) 
   }
 }
 
+// The same with per-head RMS norms in front of the rotation: a warp per head (q, k or v). The sum of squares and the
+// values run over the row twice; the second time it is in L1.
+template <int VEC, typename T>
+__global__ void __launch_bounds__(256) rope_heads_kernel(const RopeDimsParams p) {
+  const int m = blockIdx.x, head = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (head >= p.Hq + 2 * p.Hkv) return;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const T* src = reinterpret_cast<const T*>(p.qkv) + (size_t)m * p.qkv_ld;
+  long long slot = p.slots[m];
+  int pos = p.positions[m];
+  if (slot >= p.num_slots || pos < 0 || (p.rot > 0 && pos >= p.max_pos)) {
+    if (lane == 0 && p.status) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+    if (slot >= p.num_slots) slot = -1;
+    pos = 0;
+  }
+  if (head >= p.Hq + p.Hkv) {                       // a value row
+    if (slot < 0) return;
+    const int h = head - p.Hq - p.Hkv;
+    const T* row = src + (size_t)(p.Hq + p.Hkv) * p.dk + (size_t)h * p.dv;
+    T* dst = reinterpret_cast<T*>(p.v_cache) + ((size_t)slot * p.Hkv + h) * p.dvp;
+    for (int d = lane * VEC; d < p.dvp; d += 32 * VEC) {
+      float o[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+      if (d < p.dv) ldn<VEC>(row + d, o);
+      stn<VEC>(dst + d, o);
+    }
+    return;
+  }
+  const bool is_q = head < p.Hq;
+  if (!is_q && slot < 0) return;
+  const bf16* nw = is_q ? p.q_norm : p.k_norm;
+  const T* row = src + (size_t)head * p.dk;         // k heads follow the q heads
+  T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + ((size_t)m * p.Hq + head) * p.dkp
+                : reinterpret_cast<T*>(p.k_cache) + ((size_t)slot * p.Hkv + head - p.Hq) * p.dkp;
+  float inv = 1.f;
+  if (nw) {
+    float ss = 0.f;
+    for (int d = lane * VEC; d < p.dk; d += 32 * VEC) {
+      float x[VEC];
+      ldn<VEC>(row + d, x);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss = fmaf(x[j], x[j], ss);
+    }
+    inv = 1.f / sqrtf(mb::warp_sum(ss) / (float)p.dk + p.eps);
+  }
+  const int half = p.rot / 2;
+  const float* cs = p.cos_tab + (size_t)pos * half;
+  const float* sn = p.sin_tab + (size_t)pos * half;
+  auto load = [&](int d, float* o) {
+    ldn<VEC>(row + d, o);
+    if (nw) {
+      float w[VEC];
+      ldn<VEC>(nw + d, w);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] *= inv * w[j];
+    }
+  };
+  for (int d = lane * VEC; d < p.dkp; d += 32 * VEC) {
+    float o[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+    if (d < p.dk) {
+      load(d, o);
+      if (d < p.rot) {                              // VEC divides rot / 2: the whole vector is on one side
+        float q[VEC];
+        const bool first = d < half;
+        load(first ? d + half : d - half, q);
+        const int a = first ? d : d - half;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          const float c = cs[a + j], s = sn[a + j];
+          o[j] = first ? o[j] * c - q[j] * s : o[j] * c + q[j] * s;
+        }
+      }
+    }
+    stn<VEC>(dst + d, o);
+  }
+}
+
 }  // namespace
 
 struct MbStreamNormArgs {
@@ -554,6 +622,23 @@ struct MbGatedNormArgs {
   long long out_ld;
 };
 
+struct MbEmbedArgs {
+  int M, W, vocab, copy_f32;
+  const int* tokens;
+  const void* table;
+  float* out;
+  float scale;
+  void* copy;                // or null: the same rows in the activation type, copy_ld elements apart
+  long long copy_ld;
+  const int* positions;
+  const void* pos;           // [max_pos, W] or null
+  int max_pos;
+  float norm_alpha;
+  const void* norm_w;        // or null
+  const void* norm_b;
+  uint32_t* status;
+};
+
 struct MbRopeDimsArgs {
   int M, Hq, Hkv, dk, dv, rot, dkp, dvp, f32;
   const void* qkv;
@@ -568,16 +653,10 @@ struct MbRopeDimsArgs {
   void* v_cache;
   long long num_slots;
   uint32_t* status;
+  const void* q_norm;        // [dk] per-head RMS norm weights, or null
+  const void* k_norm;
+  float eps;
 };
-
-namespace {
-bool al(const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) % n) == 0; }
-int row_threads(int W, int vec) {
-  int n = 32;
-  while (n < 256 && n * vec < W) n <<= 1;
-  return n;
-}
-}  // namespace
 
 extern "C" {
 
@@ -658,18 +737,16 @@ int mb_side_gate(const float* z, const int* tokens, const void* table, long long
                   : mb::launch_kernel(side_gate_kernel<1, bf16>, g, b, 0, stream, z, tokens, tb, table_ld, off, dim, rows, num_rows, (bf16*)out, status));
 }
 
-// copy (or null): the same rows in the activation type, copy_ld elements apart
-int mb_embed_scaled(const int* tokens, const void* table, float* out, int M, int W, int vocab, float scale, void* copy, long long copy_ld,
-                    int copy_f32, uint32_t* status, cudaStream_t stream) {
-  if (!tokens || !table || !out || M <= 0 || W <= 0 || (copy && copy_ld < W)) return MB_ERR_BAD_ARG;
-  const bool v4 = W % 4 == 0 && al(table, 8) && al(out, 16) && copy_ld % 4 == 0 && al(copy, 16);
-  const dim3 g(M), b(row_threads(W, v4 ? 4 : 1));
-  const bf16* tab = (const bf16*)table;
-  if (copy_f32)
-    return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, float>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (float*)copy, copy_ld, status)
-                    : mb::launch_kernel(embed_scaled_kernel<1, float>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (float*)copy, copy_ld, status));
-  return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, bf16>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (bf16*)copy, copy_ld, status)
-                  : mb::launch_kernel(embed_scaled_kernel<1, bf16>, g, b, 0, stream, tokens, tab, out, W, vocab, scale, (bf16*)copy, copy_ld, status));
+int mb_embed_scaled(const MbEmbedArgs* a, cudaStream_t stream) {
+  if (!a || !a->tokens || !a->table || !a->out || a->M <= 0 || a->W <= 0 || (a->copy && a->copy_ld < a->W)) return MB_ERR_BAD_ARG;
+  if ((a->pos && (!a->positions || a->max_pos <= 0)) || (a->norm_w && !a->norm_b)) return MB_ERR_BAD_ARG;
+  const EmbedParams p{a->tokens, (const bf16*)a->table, a->out, a->W, a->vocab, a->scale, a->copy, a->copy_ld, a->positions, (const bf16*)a->pos,
+                      a->max_pos, DytW{a->norm_alpha, (const bf16*)a->norm_w, (const bf16*)a->norm_b}, a->status};
+  const bool v4 = a->W % 4 == 0 && al(a->table, 8) && al(a->out, 16) && a->copy_ld % 4 == 0 && al(a->copy, 16) && al(a->pos, 8) &&
+                  al(a->norm_w, 8) && al(a->norm_b, 8);
+  const dim3 g(a->M), b(row_threads(a->W, v4 ? 4 : 1));
+  if (a->copy_f32) return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(embed_scaled_kernel<1, float>, g, b, 0, stream, p));
+  return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(embed_scaled_kernel<1, bf16>, g, b, 0, stream, p));
 }
 
 int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) {
@@ -683,9 +760,14 @@ int mb_rope_dims(const MbRopeDimsArgs* a, cudaStream_t stream) {
   if (a->dk <= 0 || a->dv <= 0 || a->dk > a->dkp || a->dv > a->dvp || a->rot < 0 || a->rot > a->dk || a->rot % 2) return MB_ERR_UNSUPPORTED;
   if (a->rot > 0 && (!a->cos_tab || !a->sin_tab)) return MB_ERR_BAD_ARG;
   RopeDimsParams p{a->M, a->Hq, a->Hkv, a->dk, a->dv, a->rot, a->dkp, a->dvp, a->qkv, a->qkv_ld, a->positions, a->slots, a->cos_tab,
-                   a->sin_tab, a->max_pos, a->q_out, a->k_cache, a->v_cache, a->num_slots, a->status};
+                   a->sin_tab, a->max_pos, a->q_out, a->k_cache, a->v_cache, a->num_slots, a->status, (const bf16*)a->q_norm, (const bf16*)a->k_norm, a->eps};
   const bool v4 = a->dk % 4 == 0 && a->dv % 4 == 0 && a->rot % 8 == 0 && a->dkp % 4 == 0 && a->dvp % 4 == 0 && a->qkv_ld % 4 == 0 &&
-                  al(a->qkv, 16) && al(a->q_out, 16) && al(a->k_cache, 16) && al(a->v_cache, 16);
+                  al(a->qkv, 16) && al(a->q_out, 16) && al(a->k_cache, 16) && al(a->v_cache, 16) && al(a->q_norm, 8) && al(a->k_norm, 8);
+  if (a->q_norm || a->k_norm) {
+    const dim3 g(a->M, (a->Hq + 2 * a->Hkv + 7) / 8), b(256);
+    if (a->f32) return (int)(v4 ? mb::launch_kernel(rope_heads_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(rope_heads_kernel<1, float>, g, b, 0, stream, p));
+    return (int)(v4 ? mb::launch_kernel(rope_heads_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(rope_heads_kernel<1, bf16>, g, b, 0, stream, p));
+  }
   const int total = (a->Hq + a->Hkv) * a->dkp + a->Hkv * a->dvp;
   const int vec = v4 ? 4 : 1;
   const int want = (total + 256 * vec - 1) / (256 * vec);

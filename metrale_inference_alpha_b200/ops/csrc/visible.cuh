@@ -1,0 +1,49 @@
+// What the attention kernels share about masks and outputs beyond plain causal attention.
+#pragma once
+#include "common.cuh"
+
+namespace mb {
+
+// Cached tokens that any of a run of consecutive queries may see, as a dense list of whole 64-token tiles: the kept
+// first tokens, then the window. Entry v stands for token v (v < keep64) or v + shift; without a window the list is
+// the context itself. Queries still mask inside the first and last tiles.
+struct VisibleTokens {
+  int keep64;    // entries that stand for the kept first tokens, a multiple of 64
+  int shift;     // token - entry behind them, a multiple of 64
+  int len;       // entries
+
+  // first: position of the run's first query; end: one past the last token that the last query sees
+  __device__ __forceinline__ VisibleTokens(int first, int end, int window, int keep) {
+    const int begin = window > 0 ? max(0, first + 1 - window) & ~63 : 0;
+    keep64 = min((keep + 63) & ~63, begin);
+    shift = begin - keep64;
+    len = end - shift;
+  }
+  __device__ __forceinline__ int token(int v) const { return v < keep64 ? v : v + shift; }
+};
+
+// the query that sees the tokens below `limit`: does it see `tok`?
+__device__ __forceinline__ bool sees(int tok, int limit, int window, int keep) {
+  return tok < limit && (window <= 0 || tok >= limit - window || tok < keep);
+}
+
+enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
+
+// Sigmoid gates on an attention output, read where the projection left their logits: one per head, or one per element
+// (head h's at columns h * dv ...). Row m of the output has its logits gate_ld elements times m on.
+template <typename T>
+struct OutputGate {
+  const T* logits;
+  long long ld;
+  int mode, dv;
+  __device__ __forceinline__ float operator()(size_t row, int head, int d) const {
+    if (mode == GATE_NONE) return 1.f;
+    const T* z = logits + row * ld + (mode == GATE_HEAD ? head : head * dv + d);
+    float v;
+    if constexpr (sizeof(T) == 2) v = __bfloat162float(*z);
+    else v = *z;
+    return 1.f / (1.f + expf(-v));
+  }
+};
+
+}  // namespace mb

@@ -1,8 +1,9 @@
-"""Ops of models with a 32-bit residual stream: Dynamic-Tanh and RMS norms fused around the stream, token-shift
-mixes, attention with separate query/key and value head sizes and a softmax sink, decaying linear
-attention (per-head or per-channel decay), gated group norms and the token side input.
+"""Ops of models with a 32-bit residual stream: Dynamic-Tanh and RMS norms fused around the stream, static
+hyper-connections, token-shift mixes, attention with separate query/key and value head sizes (sinks, windows with kept
+first tokens, output gates), decaying linear attention (per-head or per-channel decay), gated group norms and the
+token side input.
 
-CUDA tensors run the kernels in ``csrc/{stream_norm,attention,attention_tc,attention_simt,linear_attn,
+CUDA tensors run the kernels in ``csrc/{stream_norm,stream_hyper,attention,attention_tc,attention_simt,linear_attn,
 linear_chunked,gemm_simt}.cu``; CPU tensors run the restatements below, which compute the same quantities
 in fp32 and round where the kernels round. The activation type is bf16, or fp32 for models served in
 32-bit (``Act.fmt`` "bf16" / "fp32").
@@ -189,6 +190,91 @@ def stream_norm(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, 
     return x1, h, mixes, h32
 
 
+# ----------------------------------------------------------------------------- several residual streams
+@dataclass
+class HyperW:
+    """Static hyper-connection of one sublayer over S residual streams: it reads sum_s w_in[s] x_s, and every stream becomes
+    sum_s w_mix[s, t] x_s + w_out[t] y."""
+    w_in: torch.Tensor     # fp32 [S]
+    w_out: torch.Tensor    # fp32 [S]
+    w_mix: torch.Tensor    # fp32 [S (from), S (to)]
+
+
+@dataclass
+class SublayerOut:
+    """What a sublayer leaves for the streams: y (activation type), times the sigmoid of ``gate`` [T] (fp32 logits, may be
+    a column), plus the routed experts' sum; any of them may be missing."""
+    y: Optional[torch.Tensor] = None
+    gate: Optional[torch.Tensor] = None
+    routed: Optional[Routed] = None
+
+
+class _StreamHyperArgs(C.Structure):
+    _fields_ = [("T", C.c_int), ("W", C.c_int), ("S", C.c_int), ("f32", C.c_int), ("x_one", C.c_int), ("out_mode", C.c_int), ("K", C.c_int),
+                ("x", C.c_void_p), ("y", C.c_void_p), ("y_gate", C.c_void_p), ("y_gate_ld", C.c_longlong), ("ye", C.c_void_p),
+                ("ye_ld", C.c_longlong), ("pair_row", C.c_void_p), ("pair_w", C.c_void_p), ("w_mix", C.c_void_p), ("w_out", C.c_void_p),
+                ("x_out", C.c_void_p), ("w_in", C.c_void_p), ("alpha", C.c_float), ("norm_w", C.c_void_p), ("norm_b", C.c_void_p),
+                ("out", C.c_void_p), ("rows", C.c_void_p), ("num_rows", C.c_longlong), ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_stream_hyper", [C.POINTER(_StreamHyperArgs), C.c_void_p])
+_HYPER_IN_PLACE = 4              # the kernel holds this many streams in registers
+
+
+def stream_hyper(x: torch.Tensor, S: int, fmt: str, *, pending: Optional[SublayerOut] = None, hc: Optional[HyperW] = None,
+                 w_in: Optional[torch.Tensor] = None, pre: Optional[DytNorm] = None, out_f32: bool = False,
+                 rows: Optional[torch.Tensor] = None):
+    """x [T, S, W] fp32, or [T, W] while all S streams are one row. ``pending`` joins the streams through ``hc``; the
+    output is pre(u), or u itself in fp32 (``out_f32``) or the activation type, u = sum_s w_in[s] x_s of the new streams.
+    ``rows`` (int64): only those tokens, the streams stay. Returns (streams, output); streams that are given whole may be
+    updated in place."""
+    one = x.dim() == 2
+    T, W = x.shape[0], x.shape[-1]
+    n = T if rows is None else rows.numel()
+    out = torch.empty(n, W, dtype=torch.float32 if out_f32 else DTYPE[fmt], device=x.device)
+    if not x.is_cuda:
+        xs = x[:, None, :].expand(T, S, W) if one else x
+        if pending is not None:
+            y = torch.zeros(T, W)
+            if pending.y is not None:
+                y = pending.y.float() * (torch.sigmoid(pending.gate.float())[:, None] if pending.gate is not None else 1.0)
+            if pending.routed is not None:
+                y = y + pending.routed.y
+            xs = torch.einsum("tsw,so->tow", xs, hc.w_mix) + hc.w_out[None, :, None] * y[:, None, :]
+        u = torch.einsum("tsw,s->tw", xs, w_in)
+        u = u if rows is None else u[rows.long()]
+        out.copy_(u if pre is None else dyt_ref(u, pre))
+        return (xs if pending is not None and rows is None else x), out
+    a = _StreamHyperArgs()
+    a.T, a.W, a.S, a.f32, a.x_one = n, W, S, _f32(fmt), int(one)
+    a.x, a.out, a.w_in, a.status = _ptr(x), _ptr(out), _ptr(w_in), _ptr(runtime(x.device).status)
+    a.out_mode = 3 if out_f32 else 1 if pre is not None else 2
+    if pre is not None:
+        assert not out_f32
+        a.alpha, a.norm_w, a.norm_b = pre.alpha, _ptr(pre.w), _ptr(pre.b)
+    x1 = x
+    if rows is not None:
+        assert rows.dtype == torch.int64
+        a.rows, a.num_rows = _ptr(rows), T
+    if pending is not None:
+        a.w_mix, a.w_out = _ptr(hc.w_mix), _ptr(hc.w_out)
+        y, g, r = pending.y, pending.gate, pending.routed
+        if y is not None:
+            assert y.dtype == DTYPE[fmt] and y.is_contiguous() and y.shape == (T, W)
+            a.y = _ptr(y)
+            if g is not None:
+                assert g.dtype == torch.float32 and g.dim() == 1
+                a.y_gate, a.y_gate_ld = _ptr(g), g.stride(0)
+        if r is not None:
+            a.ye, a.ye_ld, a.pair_row, a.pair_w, a.K = _ptr(r.y), r.y.stride(0), _ptr(r.pair_row), _ptr(r.w), r.w.shape[1]
+        if rows is None:
+            x1 = torch.empty(T, S, W, dtype=torch.float32, device=x.device) if one or S > _HYPER_IN_PLACE else x
+            a.x_out = _ptr(x1)
+    _native.check(_native.lib().mb_stream_hyper(C.byref(a), _stream()), f"stream_hyper[T={n} S={S} W={W}]")
+    _count()
+    return x1, out
+
+
 def shift_commit(h32: torch.Tensor, state: torch.Tensor, batch) -> None:
     """state[slot] := h of each sequence's last row in ``batch`` (sequences of zero rows keep theirs)."""
     if not h32.is_cuda:
@@ -277,25 +363,42 @@ def gated_norm(x: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, fmt: str, *
 
 
 # ----------------------------------------------------------------------------- embedding, token side input
-_native.register_optional("mb_embed_scaled", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_void_p,
-                                              C.c_longlong, C.c_int, C.c_void_p, C.c_void_p])
+class _EmbedArgs(C.Structure):
+    _fields_ = [("M", C.c_int), ("W", C.c_int), ("vocab", C.c_int), ("copy_f32", C.c_int), ("tokens", C.c_void_p), ("table", C.c_void_p),
+                ("out", C.c_void_p), ("scale", C.c_float), ("copy", C.c_void_p), ("copy_ld", C.c_longlong), ("positions", C.c_void_p),
+                ("pos", C.c_void_p), ("max_pos", C.c_int), ("norm_alpha", C.c_float), ("norm_w", C.c_void_p), ("norm_b", C.c_void_p),
+                ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_embed_scaled", [C.POINTER(_EmbedArgs), C.c_void_p])
 _native.register_optional("mb_side_gate", [C.c_void_p, C.c_void_p, C.c_void_p, C.c_longlong] + [C.c_int] * 4 +
                           [C.c_void_p, C.c_int, C.c_void_p, C.c_void_p])
 
 
-def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 [T, W] = table[ids] * scale; ``copy`` (may be a column range) takes the same in the activation type."""
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float, copy: Optional[torch.Tensor] = None, *,
+                 pos: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None, norm: Optional[DytNorm] = None) -> torch.Tensor:
+    """fp32 [T, W] = norm(table[ids] * scale + pos[positions]), `pos` and `norm` optional; ``copy`` (may be a column
+    range) takes the same in the activation type."""
     if not table.is_cuda:
         x = table[ids.long()].float() * scale
+        if pos is not None:
+            x = x + pos[positions.long()].float()
+        if norm is not None:
+            x = dyt_ref(x, norm)
         if copy is not None:
             copy.copy_(x)
         return x
     M, W = ids.numel(), table.shape[1]
     out = torch.empty(M, W, dtype=torch.float32, device=table.device)
-    rc = _native.lib().mb_embed_scaled(_ptr(ids), _ptr(table), _ptr(out), M, W, table.shape[0], float(scale), _ptr(copy),
-                                       copy.stride(0) if copy is not None else 0, int(copy is not None and copy.dtype == torch.float32),
-                                       _ptr(runtime(table.device).status), _stream())
-    _native.check(rc, "embed_scaled")
+    a = _EmbedArgs(M=M, W=W, vocab=table.shape[0], copy_f32=int(copy is not None and copy.dtype == torch.float32), tokens=_ptr(ids),
+                   table=_ptr(table), out=_ptr(out), scale=float(scale), status=_ptr(runtime(table.device).status))
+    if copy is not None:
+        a.copy, a.copy_ld = _ptr(copy), copy.stride(0)
+    if pos is not None:
+        a.positions, a.pos, a.max_pos = _ptr(positions), _ptr(pos), pos.shape[0]
+    if norm is not None:
+        a.norm_alpha, a.norm_w, a.norm_b = norm.alpha, _ptr(norm.w), _ptr(norm.b)
+    _native.check(_native.lib().mb_embed_scaled(C.byref(a), _stream()), "embed_scaled")
     _count()
     return out
 
@@ -320,7 +423,7 @@ class _RopeDimsArgs(C.Structure):
                 ("dkp", C.c_int), ("dvp", C.c_int), ("f32", C.c_int), ("qkv", C.c_void_p), ("qkv_ld", C.c_longlong),
                 ("positions", C.c_void_p), ("slots", C.c_void_p), ("cos_tab", C.c_void_p), ("sin_tab", C.c_void_p),
                 ("max_pos", C.c_int), ("q_out", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p),
-                ("num_slots", C.c_longlong), ("status", C.c_void_p)]
+                ("num_slots", C.c_longlong), ("status", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("eps", C.c_float)]
 
 
 class _SimtAttnArgs(C.Structure):
@@ -329,7 +432,8 @@ class _SimtAttnArgs(C.Structure):
                 ("total_rows", C.c_int), ("num_seqs", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("dk", C.c_int),
                 ("dv", C.c_int), ("dkp", C.c_int), ("dvp", C.c_int), ("block_size", C.c_int), ("num_blocks", C.c_longlong),
                 ("scale", C.c_float), ("out_scale", C.c_float), ("sink", C.c_int), ("f32", C.c_int), ("out", C.c_void_p),
-                ("out_ld", C.c_longlong), ("status", C.c_void_p)]
+                ("out_ld", C.c_longlong), ("status", C.c_void_p), ("sink_w", C.c_void_p), ("window", C.c_int), ("keep", C.c_int),
+                ("gate", C.c_void_p), ("gate_ld", C.c_longlong), ("gate_mode", C.c_int)]
 
 
 _native.register_optional("mb_rope_dims", [C.POINTER(_RopeDimsArgs), C.c_void_p])
@@ -348,8 +452,8 @@ def padded_head_dims(dk: int, dv: int, fmt: str) -> Tuple[int, int]:
 
 
 def rope_dims(qkv: torch.Tensor, *, Hq: int, Hkv: int, dk: int, dv: int, positions, slots, k_cache, v_cache, cos, sin,
-              fmt: str) -> torch.Tensor:
-    """qkv [T, Hq dk | Hkv dk | Hkv dv]: rotate the first 2 * cos.shape[1] dimensions of every q and k head
+              fmt: str, q_norm: Optional[RmsNorm] = None, k_norm: Optional[RmsNorm] = None) -> torch.Tensor:
+    """qkv [T, Hq dk | Hkv dk | Hkv dv | ...]: norm every q and k head (``q_norm`` / ``k_norm`` over dk), rotate the first 2 * cos.shape[1] dimensions of every q and k head
     (rotate-half pairing) and scatter k, v into caches [blocks, block, Hkv, padded]. Returns q [T, Hq, padded dk]."""
     M = qkv.shape[0]
     dkp, dvp = k_cache.shape[3], v_cache.shape[3]
@@ -358,7 +462,9 @@ def rope_dims(qkv: torch.Tensor, *, Hq: int, Hkv: int, dk: int, dv: int, positio
         x = qkv.float()
         q = x[:, :Hq * dk].view(M, Hq, dk)
         k = x[:, Hq * dk:(Hq + Hkv) * dk].view(M, Hkv, dk)
-        v = x[:, (Hq + Hkv) * dk:].reshape(M, Hkv, dv)
+        v = x[:, (Hq + Hkv) * dk:(Hq + Hkv) * dk + Hkv * dv].reshape(M, Hkv, dv)
+        rms = lambda t, n: t if n is None else t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + n.eps) * n.w.float()
+        q, k = rms(q, q_norm), rms(k, k_norm)
         if rot:
             q, k = ref.apply_rope_neox(q, positions, cos, sin), ref.apply_rope_neox(k, positions, cos, sin)
         pad = torch.nn.functional.pad
@@ -372,16 +478,40 @@ def rope_dims(qkv: torch.Tensor, *, Hq: int, Hkv: int, dk: int, dv: int, positio
     a = _RopeDimsArgs(M, Hq, Hkv, dk, dv, rot, dkp, dvp, _f32(fmt), _ptr(qkv), qkv.stride(0), _ptr(positions), _ptr(slots),
                       _ptr(cos) if rot else None, _ptr(sin) if rot else None, cos.shape[0] if rot else 0, _ptr(q_out),
                       _ptr(k_cache), _ptr(v_cache), k_cache.shape[0] * k_cache.shape[1], _ptr(runtime(qkv.device).status))
+    if q_norm is not None or k_norm is not None:
+        a.q_norm, a.k_norm = _ptr(q_norm.w if q_norm else None), _ptr(k_norm.w if k_norm else None)
+        a.eps = (q_norm or k_norm).eps
+        assert q_norm is None or k_norm is None or q_norm.eps == k_norm.eps
     _native.check(_native.lib().mb_rope_dims(C.byref(a), _stream()), f"rope_dims[T={M}]")
     _count()
     return q_out
 
 
-def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int, scale: float, sink: bool, fmt: str,
-                   out: torch.Tensor, out_scale: float = 1.0, kernel: str = "auto") -> torch.Tensor:
+@dataclass
+class OutputGate:
+    """Sigmoid gates on an attention output: logits [T, heads] (one per head) or [T, heads * dv], may be a column range."""
+    logits: torch.Tensor
+    per_head: bool
+
+    def values(self, Hq: int, dv: int) -> torch.Tensor:
+        g = torch.sigmoid(self.logits.float())
+        return g[:, :, None] if self.per_head else g.view(-1, Hq, dv)
+
+    def into(self, a) -> None:
+        assert self.logits.stride(1) == 1
+        a.gate, a.gate_ld, a.gate_mode = _ptr(self.logits), self.logits.stride(0), 1 if self.per_head else 2
+
+
+def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int, scale: float, sink, fmt: str,
+                   out: torch.Tensor, out_scale: float = 1.0, kernel: str = "auto", window: int = 0, keep: int = 0,
+                   gate: Optional[OutputGate] = None) -> torch.Tensor:
     """Causal paged attention of q [T, Hq, padded dk] into ``out`` [T, Hq * dv] (may be a column range), times
-    ``out_scale``. ``sink``: one is added to the softmax denominator. The softmax weights keep 32-bit
-    precision: they enter the product with V as two bf16 terms. ``kernel``: auto | simt | mma | tc (tests)."""
+    ``out_scale`` and the ``gate``. ``sink``: True adds one to the softmax denominator, a tensor [Hq] (fp32) exp(sink) per
+    head. ``window`` > 0: a position sees itself, the window - 1 before it and the first ``keep``. The softmax weights keep
+    32-bit precision: they enter the product with V as two bf16 terms. ``kernel``: auto | simt | mma | tc (tests)."""
+    sink_w = sink if isinstance(sink, torch.Tensor) else None
+    sink = sink_w is not None or bool(sink)
+    keep = keep if window > 0 else 0
     T, Hq, dkp = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     dvp = v_cache.shape[3]
@@ -397,13 +527,20 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
             v = v_cache[blocks].reshape(-1, Hkv, dvp)[:ctx, :, :dv].float().repeat_interleave(G, 1)
             sc = torch.einsum("ihd,jhd->hij", q[qs[s]:qs[s] + n, :, :dk].double(), k.double()) * scale
             i = torch.arange(ctx - n, ctx)[:, None]
-            sc.masked_fill_(torch.arange(ctx)[None, :] > i, float("-inf"))
+            j = torch.arange(ctx)[None, :]
+            hide = j > i
+            if window > 0:
+                hide = hide | ((i - j >= window) & (j >= keep))
+            sc.masked_fill_(hide, float("-inf"))
             m = sc.amax(-1, keepdim=True)
+            sk = sink_w.double()[:, None, None] if sink_w is not None else torch.zeros(1, 1, 1, dtype=torch.double)
             if sink:
-                m = m.clamp(min=0.0)
+                m = torch.maximum(m, sk)
             e = torch.exp(sc - m)
-            den = e.sum(-1, keepdim=True) + (torch.exp(-m) if sink else 0.0)
+            den = e.sum(-1, keepdim=True) + (torch.exp(sk - m) if sink else 0.0)
             o = torch.einsum("hij,jhd->ihd", e / den, v.double()) * out_scale
+            if gate is not None:
+                o = o * gate.values(Hq, dv)[qs[s]:qs[s] + n].double()
             out[qs[s]:qs[s] + n] = o.reshape(n, Hq * dv).to(out.dtype)
         return out
     L, rt = _native.lib(), runtime(q.device)
@@ -414,14 +551,17 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
         and (dv != dvp or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0))
     if kernel == "auto":
         kernel = "mma" if tiles_ok else "simt"
-        if tiles_ok and tc_serves(dkp, dvp, dv, out) and mq >= 128:
+        if tiles_ok and tc_serves(dkp, dvp, dv, out, gate) and mq >= 128:
             kernel = "tc"
         elif kernel == "mma" and dkp == 256 and 16 < G * mq <= 32:
             kernel = "simt"                          # between the two row-tile limits of the 256-wide tiles
     if kernel == "simt":
         a = _SimtAttnArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_table), batch.block_table.stride(0),
                           _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len), T, S, Hq, Hkv, dk, dv, dkp, dvp, bs, nb,
-                          float(scale), float(out_scale), int(sink), _f32(fmt), _ptr(out), out.stride(0), _ptr(rt.status))
+                          float(scale), float(out_scale), int(sink), _f32(fmt), _ptr(out), out.stride(0), _ptr(rt.status), _ptr(sink_w),
+                          window, keep)
+        if gate is not None:
+            gate.into(a)
         _native.check(L.mb_attn_simt(C.byref(a), _stream()), f"attn_simt[T={T}]")
         _count()
         return out
@@ -433,6 +573,9 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
             batch.block_table.stride(0), S, mq
         t.Hq, t.Hkv, t.D, t.block_size, t.scale, t.v_mn = Hq, Hkv, dkp, bs, float(scale), 1
         t.out_ld, t.out_scale, t.sink, t.split_p = out.stride(0), float(out_scale), int(sink), 1
+        t.sink_w, t.window, t.keep = _ptr(sink_w), window, keep
+        if gate is not None:
+            gate.into(t)
         _native.check(L.mb_attn_prefill_tc(C.byref(t), _stream()), "attn_prefill_tc")
         _count()
         return out
@@ -445,17 +588,23 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
     a.Hq, a.Hkv, a.D, a.block_size, a.num_blocks, a.scale = Hq, Hkv, dkp, bs, nb, float(scale)
     a.out, a.total_rows, a.part_tokens, a.status = _ptr(out), T, _ATTN_PART_TOKENS, _ptr(rt.status)
     a.DV, a.dv, a.out_ld, a.out_scale, a.sink, a.split_p = dvp, dv, out.stride(0), float(out_scale), int(sink), 1
+    a.sink_w, a.window, a.keep = _ptr(sink_w), window, keep
+    if gate is not None:
+        gate.into(a)
     if G * mq <= 32:
-        rt.ensure_attn_ws(L.mb_attn_ws_bytes(T, Hq, dvp, int(batch.max_ctx), _ATTN_PART_TOKENS))
+        seen = L.mb_attn_visible(int(batch.max_ctx), mq, window, keep)
+        rt.ensure_attn_ws(L.mb_attn_ws_bytes(T, Hq, dvp, seen, _ATTN_PART_TOKENS))
     a.ws, a.ws_bytes = _ptr(rt.attn_ws), rt.attn_ws.numel()
     _native.check(L.mb_paged_attention(C.byref(a), _stream()), f"attention_dims[T={T}]")
     _count()
     return out
 
 
-def tc_serves(dkp: int, dvp: int, dv: int, out: torch.Tensor) -> bool:
-    """Shapes of the tcgen05 prefill kernel: equal 128- or 256-wide tiles stored whole in 16-byte vectors."""
+def tc_serves(dkp: int, dvp: int, dv: int, out: torch.Tensor, gate: Optional[OutputGate] = None) -> bool:
+    """Shapes of the tcgen05 prefill kernel: equal 128- or 256-wide tiles stored (and gated) whole in 16-byte vectors."""
     from . import _ATTN_TC
+    if gate is not None and not gate.per_head and (gate.logits.stride(0) % 8 or gate.logits.data_ptr() % 16):
+        return False
     return _ATTN_TC and dkp == dvp == dv and dkp in (128, 256) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
 
 

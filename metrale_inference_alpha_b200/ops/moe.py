@@ -28,6 +28,7 @@ class GroupedExperts:
     n_down: int
     interleaved: bool
     shared_slot: Optional[int] = None     # local expert index of a folded-in shared expert (every token routes to it)
+    clamp_glu: Optional[tuple] = None     # (alpha, limit): clamped GLU instead of SwiGLU (interleaved rows)
 
 
 @dataclass
@@ -35,7 +36,8 @@ class RouterSpec:
     """Routing of one layer, where layers differ; the names are the model configuration's."""
     num_experts: int
     experts_per_token: int
-    router: str = "softmax_topk"          # softmax over the chosen ones of the biased logits
+    router: str = "softmax_topk"          # softmax over the chosen ones of the biased logits; "softmax_grouped": softmax over
+                                          # all, chosen from the groups with the largest scores, times router_scaling
     router_n_group: int = 1
     router_topk_group: int = 1
     router_renormalize: bool = True
@@ -72,6 +74,8 @@ def route(logits: torch.Tensor, cfg, bias=None):
         z = logits.float() if bias is None else logits.float() + bias
         top, idx = ref.topk_stable(z, k)
         w = torch.softmax(top, -1)
+    elif cfg.router == "softmax_grouped":
+        w, idx = ref.route_softmax_grouped(logits, k, cfg.router_n_group, cfg.router_topk_group, cfg.router_renormalize, cfg.router_scaling)
     elif cfg.router == "softmax":
         w, idx = ref.route_softmax_topk(logits, k, cfg.router_renormalize)
     else:
@@ -81,7 +85,7 @@ def route(logits: torch.Tensor, cfg, bias=None):
 
 
 def expert_sum_ref(act, weights: torch.Tensor, idx: torch.Tensor, ge: GroupedExperts, width: int) -> torch.Tensor:
-    """CPU: sum_j weights[t, j] * expert idx[t, j] of row t over stacked (padded) SwiGLU experts; fp32 [T, width]."""
+    """CPU: sum_j weights[t, j] * expert idx[t, j] of row t over stacked (padded) gated experts; fp32 [T, width]."""
     from . import Act, QuantWeight, linear
     out = torch.zeros(act.M, width)
     part = lambda w, e, n: QuantWeight(w.fmt, n, w.K, w.data[e * n:(e + 1) * n])
@@ -89,7 +93,8 @@ def expert_sum_ref(act, weights: torch.Tensor, idx: torch.Tensor, ge: GroupedExp
         tok, slot = torch.nonzero(idx == e, as_tuple=True)
         if tok.numel() == 0:
             continue
-        h = linear(Act(act.fmt, tok.numel(), act.K, act.data[tok]), part(ge.gate_up, e, ge.n_gate_up), swiglu=True)
+        h = linear(Act(act.fmt, tok.numel(), act.K, act.data[tok]), part(ge.gate_up, e, ge.n_gate_up), swiglu=ge.clamp_glu is None,
+                   clamp_glu=ge.clamp_glu)
         y = linear(Act(act.fmt, tok.numel(), h.shape[1], h.float()), part(ge.down, e, ge.n_down), out_f32=True)
         out.index_add_(0, tok, y[:, :width] * weights[tok, slot][:, None])
     return out

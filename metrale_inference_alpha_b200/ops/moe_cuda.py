@@ -7,10 +7,11 @@ import ctypes as C
 
 import torch
 
-from . import Act, EPI_SWIGLU, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
+from . import Act, EPI_CLAMP_GLU, EPI_SWIGLU, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
 
 c = C
-ROUTER_MODE = {"softmax": 0, "sigmoid": 1, "softmax_topk": 2}
+ROUTER_MODE = {"softmax": 0, "softmax_grouped": 0, "sigmoid": 1, "softmax_topk": 2}
+_GROUPED = ("sigmoid", "softmax_grouped")      # routers with groups of experts and a factor on the weights
 _native.register_optional("mb_moe_route", [c.c_void_p, c.c_longlong, c.c_int, c.c_int, c.c_int, c.c_int, c.c_void_p,
                                           c.c_int, c.c_int, c.c_int, c.c_float, c.c_void_p, c.c_void_p, c.c_void_p])
 _native.register_optional("mb_moe_sort", [c.c_void_p, c.c_int, c.c_int, c.c_int, c.c_int] + [c.c_void_p] * 6 +
@@ -59,10 +60,10 @@ def route_cuda(logits: torch.Tensor, cfg, bias=None):
     K = cfg.experts_per_token
     w = torch.empty(T, K, dtype=torch.float32, device=logits.device)
     idx = torch.empty(T, K, dtype=torch.int32, device=logits.device)
-    mode = ROUTER_MODE[cfg.router]
+    mode, grouped = ROUTER_MODE[cfg.router], cfg.router in _GROUPED
     rc = _native.lib().mb_moe_route(_ptr(logits), logits.stride(0), T, E, K, mode, _ptr(bias),
-                                    cfg.router_n_group if mode == 1 else 1, cfg.router_topk_group if mode == 1 else 1,
-                                    int(cfg.router_renormalize), float(cfg.router_scaling if mode == 1 else 1.0),
+                                    cfg.router_n_group if grouped else 1, cfg.router_topk_group if grouped else 1,
+                                    int(cfg.router_renormalize), float(cfg.router_scaling if grouped else 1.0),
                                     _ptr(w), _ptr(idx), _stream())
     _native.check(rc, "moe_route")
     _count()
@@ -148,8 +149,9 @@ def grouped_pairs(cfg, a: Act, idx: torch.Tensor, w):
         sp = SortedPairs(idx, w.expert_lo, ge.num, 16 if per_expert <= 16 else 64)
         g = lambda n: (sp.tile_expert, sp.tile_row0, sp.tile_nrows, n, sp.max_tiles, sp.tile_rows)
         assert ge.interleaved
+        epi = dict(epilogue=EPI_SWIGLU) if ge.clamp_glu is None else dict(epilogue=EPI_CLAMP_GLU, epi_a=ge.clamp_glu[0], epi_b=ge.clamp_glu[1])
         h = torch.empty(sp.pairs, ge.n_gate_up // 2, dtype=a.data.dtype, device=a.data.device)
-        gemm_simt(a.data, ge.gate_up.data, h, epilogue=EPI_SWIGLU, grouped=g(ge.n_gate_up), row_index=sp.row_pair, row_div=sp.K)
+        gemm_simt(a.data, ge.gate_up.data, h, **epi, grouped=g(ge.n_gate_up), row_index=sp.row_pair, row_div=sp.K)
         y = torch.empty(sp.pairs, ge.n_down, dtype=torch.float32, device=h.device)
         return gemm_simt(h, ge.down.data, y, grouped=g(ge.n_down)), sp
     nvfp4 = ge.gate_up.fmt == "nvfp4"
@@ -163,7 +165,7 @@ def grouped_pairs(cfg, a: Act, idx: torch.Tensor, w):
     if cfg.ffn_act == "relu2":
         h = row_op(linear(xa, ge.gate_up, grouped=g(ge.n_gate_up)), fmt_d, IN_RELU2, row_index=live)[0]
     elif ge.interleaved:
-        act = linear(xa, ge.gate_up, swiglu=True, grouped=g(ge.n_gate_up))
+        act = linear(xa, ge.gate_up, swiglu=ge.clamp_glu is None, clamp_glu=ge.clamp_glu, grouped=g(ge.n_gate_up))
         h = Act("bf16", act.shape[0], act.shape[1], act, bf16=act) if fmt_d == "bf16" else row_op(act, fmt_d, scale_pad=64, row_index=live)[0]
     else:
         h = row_op(linear(xa, ge.gate_up, grouped=g(ge.n_gate_up)), fmt_d, IN_SILU_MUL, scale_pad=64, row_index=live)[0]

@@ -374,6 +374,22 @@ def route_softmax_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
     return w, idx
 
 
+def route_softmax_grouped(logits, k: int, n_group: int = 1, topk_group: int = 1, renormalize: bool = False, scaling: float = 1.0):
+    """softmax over all experts; group-limited: keep the `topk_group` groups of neighbours with the largest score, then
+    top-k inside them; weights are the scores, optionally sum-normalised, times `scaling`."""
+    s = torch.softmax(logits.float(), -1)
+    sel, (T, E) = s, s.shape
+    if n_group > 1:
+        _, gidx = topk_stable(sel.view(T, n_group, E // n_group).amax(-1), topk_group)
+        gmask = torch.zeros(T, n_group, dtype=torch.bool, device=sel.device).scatter_(1, gidx, True)
+        sel = sel.masked_fill(~gmask.repeat_interleave(E // n_group, 1), float("-inf"))
+    _, idx = topk_stable(sel, k)
+    w = s.gather(1, idx)
+    if renormalize:
+        w = w / w.sum(-1, keepdim=True)
+    return w * scaling, idx
+
+
 def route_sigmoid_grouped(logits, bias, k: int, n_group: int = 1, topk_group: int = 1,
                           renormalize: bool = True, scaling: float = 1.0):
     """sigmoid scores; selection uses score + bias; group-limited: keep the `topk_group` groups

@@ -251,6 +251,28 @@ class SinkAttnW:
 
 
 @dataclass
+class GatedAttnW:
+    """Attention with its own head sizes and, each optional: rotation of the leading dimensions, per-head query and key
+    norms, a window with kept first tokens, a learned sink per head, sigmoid gates on the output."""
+    qkvg: QuantWeight = None             # rows: q | k | v | gate logits (| zero rows)
+    o: QuantWeight = None
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    scale: float = 1.0
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    rot_scaling: Optional[dict] = None   # as a HF `rope_scaling`
+    q_norm: object = None                # ops.mixers.RmsNorm over one head
+    k_norm: object = None
+    window: int = 0                      # 0 = none
+    keep: int = 0                        # first tokens that a window leaves visible
+    sink: Optional[torch.Tensor] = None  # fp32 [heads]
+    gate: Optional[str] = None           # "head" | "element"
+
+
+@dataclass
 class TimeMixW:
     """RWKV-style time mixing: token-shift mixes, per-channel data-dependent decay, bonus, gated group norm."""
     mu: torch.Tensor = None              # bf16 [5, W]: r, k, v, g, w
@@ -305,8 +327,9 @@ class LayerW:
     post_ffn: Optional[torch.Tensor] = None
     mixer: object = None
     ffn: object = None
-    hc_attn: Optional[tuple] = None              # hyper-connection site in front of the mixer: (fn bf16, scale fp32 [3], base fp32)
-    hc_ffn: Optional[tuple] = None               # ... and in front of the feed-forward block
+    hc_attn: Optional[object] = None             # hyper-connection site of the mixer: (fn bf16, scale fp32 [3], base fp32), or
+                                                 # ops.mixers.HyperW where it does not depend on the token
+    hc_ffn: Optional[object] = None              # ... and of the feed-forward block
     side: Optional[TokenSideW] = None            # per-layer token side input, after the feed-forward block
     out: Optional[QuantWeight] = None            # mixer and feed-forward side by side: both output projections, stacked along their inputs
 
@@ -323,6 +346,8 @@ class MtpW:
 @dataclass
 class ModelW:
     embed: torch.Tensor = None           # bf16 [V, H]
+    pos_embed: Optional[torch.Tensor] = None     # bf16 [max_position, H]: learned positions added to the embeddings
+    embed_norm: object = None            # ops.mixers.DytNorm of the embedding output
     lm_head: QuantWeight = None          # bf16, vocab-parallel under TP
     final_norm: torch.Tensor = None
     layers: List[LayerW] = field(default_factory=list)
@@ -501,6 +526,9 @@ class Loader:
         if c.arch == "finelix":
             from .finelix import load_finelix
             return load_finelix(self)
+        if c.arch == "pivipel":
+            from .pivipel import load_pivipel
+            return load_pivipel(self)
         m = ModelW()
         m.embed = self.vec("model.embed_tokens.weight")
         m.final_norm = self.vec("model.norm.weight")

@@ -104,8 +104,8 @@ def _seed_for(name: str, seed: int) -> int:
 
 def spec_shapes(c: ModelConfig) -> dict:
     """Tensors of a model whose sizes are per layer: name -> (shape, kind of synthetic values)."""
-    from . import fabulix, finelix
-    return {"fabulix": fabulix, "finelix": finelix}[c.arch].tensor_shapes(c)
+    from . import fabulix, finelix, pivipel
+    return {"fabulix": fabulix, "finelix": finelix, "pivipel": pivipel}[c.arch].tensor_shapes(c)
 
 
 class SyntheticSource(TensorSource):
@@ -374,6 +374,9 @@ class SyntheticSource(TensorSource):
                 return self._rand(name, shape, 0.02).to(torch.bfloat16)
             if kind == "linear":                             # unit-gain rows, for networks without statistics in their norms
                 return self._rand(name, shape, shape[-1] ** -0.5).to(torch.bfloat16)
+            if kind == "hyper":                      # hyper-connections: streams mostly keep to themselves
+                n, r = shape[-1], self._rand(name, shape, 0.05)
+                return (r + (torch.eye(n, device=r.device) * 0.8 + 0.2 / n if len(shape) == 2 else 1.0 / n)).to(torch.bfloat16)
             if kind == "alpha":
                 return (0.5 + self._rand(name, (1,), 0.05).reshape(())).to(torch.bfloat16)
             if kind == "mix":
