@@ -1,6 +1,6 @@
 #!/usr/bin/env python
-"""The kernels of the Fabulix or Finelix decoder next to the like kernels of the engine's attention / MLA /
-Kimi-delta-attention / Mamba2 hybrids at equal size, each with its distance from the roofline (measured copy
+"""The kernels of the Fabulix, Finelix or Pivipel decoder next to the like kernels of the engine's attention / MLA /
+Kimi-delta-attention / Mamba2 hybrids and of its gated-attention MoE models at equal size, each with its distance from the roofline (measured copy
 bandwidth and measured bf16 GEMM rate), and the throughput of a whole model next to an equal-size hybrid. CUDA
 events around one call, L2 flushed by a 512 MB write before every call, median of the timed calls. Reached as
 `bench.py --mixers`, `--design` naming the decoder.
@@ -263,6 +263,109 @@ def finelix_kernels(W=2560, H=20, D=128, FF=6912, rank=16, Hl=32, dim=128, R=64,
     return rows
 
 
+def pivipel_kernels(W=2560, H=32, G=8, D=128, FF=6912, E=64, top=6, EF=1024, S=2, window=512, keep=4, groups=8, keep_groups=4):
+    """The same rows for Pivipel: the like kernels are those of windowed, gated attention models with experts."""
+    from metrale_inference_alpha_b200.ops import moe as moe_ops, moe_cuda
+    from metrale_inference_alpha_b200.weights.loader import MoeW
+    rows = []
+    HD, pair, f32 = H * D, pairing(rows), torch.float32
+    for shape, lens, start in SHAPES:
+        b, nblk = batch(lens, start)
+        T, ctx = sum(lens), lens[0] + start
+        # ---- the streams
+        x, y, xb, wv = rnd(T, S, W, dtype=f32), rnd(T, W), rnd(T, W), rnd(W)
+        hw = mx.HyperW(*(torch.full(s, 0.4, device=DEV) for s in ((S,), (S,), (S, S))))
+        n1 = mx.DytNorm(0.5, rnd(W), rnd(W))
+        one = mx.SublayerOut(y)
+        pair(shape, f"stream_hyper ({S} streams, join + read + norm)", lambda: mx.stream_hyper(x, S, "bf16", pending=one, hc=hw, w_in=hw.w_in, pre=n1),
+             T * W * (8 * S + 4), 0, "residual + RMSNorm", lambda: ops.row_op(xb, "bf16", ops.IN_RMSNORM, w=wv, residual=y, write_residual=True),
+             T * W * 8, 0)
+        ids, et, pt = torch.randint(0, 60000, (T,), dtype=torch.int32, device=DEV), rnd(60000, W), rnd(8192, W)
+        pair(shape, "embedding + position + norm, fp32", lambda: mx.embed_scaled(ids, et, 1.0, pos=pt, positions=b.positions, norm=n1), T * W * 8, 0,
+             "embedding gather", lambda: ops.embed(ids, et), T * W * 4, 0)
+        # ---- experts
+        gu, dn = QuantWeight("bf16", E * 2 * EF, W, rnd(E * 2 * EF, W, std=0.02)), QuantWeight("bf16", E * W, EF, rnd(E * W, EF, std=0.02))
+        soft = moe_ops.RouterSpec(E, top, "softmax")
+        spec = moe_ops.RouterSpec(E, top, "softmax_grouped", router_n_group=groups, router_topk_group=keep_groups, router_renormalize=False)
+        w = MoeW(grouped=moe_ops.GroupedExperts(gu, dn, E, 2 * EF, W, True, clamp_glu=(1.702, 7.0)), spec=spec)
+        lw = MoeW(grouped=moe_ops.GroupedExperts(gu, dn, E, 2 * EF, W, True), spec=soft)
+        act, logits = mx.act_of(rnd(T, W), "bf16"), rnd(T, E, dtype=f32)
+        pair(shape, "route (softmax, groups)", lambda: moe_ops.route(logits, spec), T * (E + 2 * top) * 4, 0, "route (softmax)",
+             lambda: moe_ops.route(logits, soft), T * (E + 2 * top) * 4, 0)
+        rw = QuantWeight("bf16", E + 4, W, rnd(E + 4, W, std=0.02))
+        rl = QuantWeight("bf16", E, W, rw.data[:E])
+        pair(shape, "router + shared gate GEMM", lambda: ops.linear(act, rw, out_f32=True), ((E + 4 + T) * W) * 2 + T * (E + 4) * 4, 2 * T * W * (E + 4),
+             "router GEMM", lambda: ops.linear(act, rl, out_f32=True), ((E + T) * W) * 2 + T * E * 4, 2 * T * W * E)
+        wt, idx = moe_ops.route(logits, soft)
+        hit = len(set(idx.flatten().tolist()))
+        eb, ef = hit * 3 * EF * W * 2 + T * W * 2 + T * top * (W * 4 + 2 * EF * 2), T * top * 6 * EF * W
+        pair(shape, "experts (clamped GLU), unsummed", lambda: moe_cuda.grouped_pairs(spec, act, idx, w), eb, ef, "experts (SwiGLU)",
+             lambda: moe_cuda.grouped_pairs(soft, act, idx, lw), eb, ef)
+        ye, sp = moe_cuda.grouped_pairs(spec, act, idx, w)
+        gate = rnd(T, dtype=f32)
+        full = mx.SublayerOut(y, gate, mx.Routed(ye, sp.pair_row, wt))
+
+        def combine():
+            out = torch.empty(T, W, dtype=BF, device=DEV)
+            ops._native.lib().mb_moe_finish(ops._ptr(ye), ye.stride(0), ops._ptr(sp.pair_row), ops._ptr(wt), T, top, W, ops._ptr(y), W, ops._ptr(gate), 1,
+                                            ops._ptr(xb), ops._ptr(out), ops._stream())
+        pair(shape, "stream_hyper with gated shared expert and experts' sum",
+             lambda: mx.stream_hyper(x, S, "bf16", pending=full, hc=hw, w_in=hw.w_in, pre=n1), T * W * (8 * S + 4 + 4 * top), 0,
+             "expert combine (gated shared)", combine, T * W * (6 + 4 * top), 0)
+        del gu, dn, w, lw, ye, sp, full
+        # ---- attention
+        cos, sin = ref.rope_tables(8192, D, 1e4, device=DEV)
+        kc, vc = rnd(nblk, 16, G, D), rnd(nblk, 16, G, D)
+        qkvg, qn = rnd(T, (H + 2 * G) * D + HD), rnd(D)
+        byt = 2 * T * (H + 2 * G) * D * 2
+        nm = mx.RmsNorm(qn, 1e-5)
+        pos = dict(Hq=H, Hkv=G, positions=b.positions, slots=b.slot_mapping, k_cache=kc, v_cache=vc)
+        plain = qkvg[:, :(H + 2 * G) * D].contiguous()
+        like = lambda c, s, n: (lambda: ops.qk_norm_rope_kvwrite(plain, D=D, cos=c, sin=s, q_norm_w=n, k_norm_w=n, **pos))
+        pair(shape, "rope_dims (rotation)", lambda: mx.rope_dims(qkvg, dk=D, dv=D, cos=cos, sin=sin, fmt="bf16", **pos), byt, 0, "rope + KV write",
+             like(cos, sin, None), byt, 0)
+        pair(shape, "rope_dims (head norms)", lambda: mx.rope_dims(qkvg, dk=D, dv=D, cos=None, sin=None, fmt="bf16", q_norm=nm, k_norm=nm, **pos), byt, 0,
+             "head norms + KV write", like(None, None, qn), byt, 0)
+        q, out, sink = rnd(T, H, D), torch.empty(T, HD, dtype=BF, device=DEV), rnd(H, dtype=f32)
+        seen = sum(min(window, p + 1) for n in lens for p in range(start, start + n))
+        byt = sum(min(ctx, n + window) for n in lens) * G * D * 4 + T * HD * 4
+        ge, gh = qkvg[:, (H + 2 * G) * D:], qkvg[:, (H + 2 * G) * D:(H + 2 * G) * D + H]
+        kw = dict(dk=D, dv=D, scale=0.09, fmt="bf16", out=out, window=window)
+        like = lambda: ops.paged_attention(q, kc, vc, b.block_table, b.q_start, b.q_len, b.ctx_len, max_q_len=b.max_q_len, max_ctx=b.max_ctx, scale=0.09,
+                                           window=window)
+        pair(shape, "windowed attention, sinks, head gates", lambda: mx.attention_dims(q, kc, vc, b, sink=sink, gate=mx.OutputGate(gh, True), **kw),
+             byt + T * H * 2, 4 * HD * seen, "windowed attention", like, byt, 4 * HD * seen)
+        gq = rnd(T, 2 * HD)
+        pair(shape, "windowed attention, kept tokens, element gates",
+             lambda: mx.attention_dims(q, kc, vc, b, sink=False, keep=keep, gate=mx.OutputGate(ge, False), **kw), byt + T * HD * 2, 4 * HD * (seen + T * keep),
+             "windowed attention + gate", lambda: ops.row_op(like().view(T, HD), "bf16", ops.IN_SIGMOID_GATE, gate=gq, head_dim=D, gate_head_stride=2 * D,
+                                                             gate_head_off=D), byt + T * HD * 6, 4 * HD * seen)
+        del q, qkvg, gq, plain
+        # ---- matrix products with their epilogues
+        gu = QuantWeight("bf16", 2 * FF, W, rnd(2 * FF, W, std=0.02))
+        gb, gf = (2 * FF * W + T * W + T * FF) * 2, 2 * T * 2 * FF * W
+        pair(shape, "GEMM + clamped GLU", lambda: ops.linear(act, gu, clamp_glu=(1.702, 7.0)), gb, gf, "GEMM + SwiGLU",
+             lambda: ops.linear(act, gu, swiglu=True), gb, gf)
+    return rows
+
+
+def pivipel_models():
+    """(label, name -> configuration): Pivipel and a model of equal size with the same experts, windows, head norms and
+    output gates on one bf16 residual; bf16."""
+    from metrale_inference_alpha_b200.config.model_config import ModelConfig, preset
+    for label, kw in (("1B-like layers", dict(width=2048, heads=16, kv_heads=4, ff=5632, experts=32, top=4, expert_ff=768, shared_ff=1536, vocab=32768)),
+                      ("3B-like layers", {})):
+        p = preset("pivipel-3b", num_layers=6, window=512, **kw)
+        m, mlp = p.layer_specs[1]["mixer"], p.layer_specs[1]["mlp"]
+        h = ModelConfig(name="gated-attention-moe", arch="qwen_hybrid", vocab_size=p.vocab_size, hidden_size=p.hidden_size, num_layers=6,
+                        num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"], rotary_dim=m["dim"], qk_norm=True, attn_output_gate=True,
+                        norm_plus_one=True, layer_types=["attention"] * 6, ffn_types=list(p.ffn_types), sliding_window=m["mask"]["size"],
+                        intermediate_size=p.intermediate_size, num_experts=mlp["router"]["experts"], experts_per_token=mlp["router"]["top"],
+                        moe_intermediate_size=mlp["expert"]["ff"], num_shared_experts=mlp["shared"]["ff"] // mlp["expert"]["ff"], shared_expert_gate=True,
+                        router="softmax", tie_embeddings=True, weight_format="bf16", kv_dtype="bf16", max_position=16384)
+        yield label, {"pivipel": p, "gated-attention MoE": h}
+
+
 def finelix_models():
     """(label, name -> configuration): Finelix, the same with two layers looped three times, and a hybrid of
     equal size: MLA and experts where Finelix has latent attention, Kimi delta attention and SwiGLU elsewhere; bf16."""
@@ -339,10 +442,10 @@ def throughput(cfg, decode_batches=(1, 32, 128), prefills=((1, 4096), (8, 1024))
 def run(what="all", design="fabulix"):
     res = {"design": design}
     if what in ("all", "kernels"):
-        res["kernels"] = {"fabulix": kernels, "finelix": finelix_kernels}[design]()
+        res["kernels"] = {"fabulix": kernels, "finelix": finelix_kernels, "pivipel": pivipel_kernels}[design]()
     if what in ("all", "models"):
         res["models"] = {}
-        for label, cfgs in {"fabulix": models, "finelix": finelix_models}[design]():
+        for label, cfgs in {"fabulix": models, "finelix": finelix_models, "pivipel": pivipel_models}[design]():
             res["models"][label] = {}
             for name, cfg in cfgs.items():
                 res["models"][label][name] = throughput(cfg)

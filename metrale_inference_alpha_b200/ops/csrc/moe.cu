@@ -53,22 +53,19 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
     mx = mb::warp_max(mx);
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) score[j] = sel[j] == -INFINITY ? 0.f : expf(sel[j] - mx);
-  } else if (mode == 0) {  // softmax
+  } else if (mode == 0) {  // softmax; chosen by the logits, which order experts whose scores underflow
     mx = mb::warp_max(mx);
     float se = 0.f;
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
+      sel[j] = score[j];
       score[j] = score[j] == -INFINITY ? 0.f : expf(score[j] - mx);
       se += score[j];
     }
     se = mb::warp_sum(se);
     const float inv = 1.f / se;
 #pragma unroll
-    for (int j = 0; j < kMaxPerLane; ++j) {
-      const int e = j * 32 + lane;
-      score[j] *= inv;
-      sel[j] = (j < per && e < E) ? score[j] : -INFINITY;
-    }
+    for (int j = 0; j < kMaxPerLane; ++j) score[j] *= inv;
   } else {          // sigmoid + selection bias
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {

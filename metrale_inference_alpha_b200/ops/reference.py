@@ -376,9 +376,10 @@ def route_softmax_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
 
 def route_softmax_grouped(logits, k: int, n_group: int = 1, topk_group: int = 1, renormalize: bool = False, scaling: float = 1.0):
     """softmax over all experts; group-limited: keep the `topk_group` groups of neighbours with the largest score, then
-    top-k inside them; weights are the scores, optionally sum-normalised, times `scaling`."""
-    s = torch.softmax(logits.float(), -1)
-    sel, (T, E) = s, s.shape
+    top-k inside them (by the logits, which order experts whose scores underflow); weights are the scores, optionally
+    sum-normalised, times `scaling`."""
+    s, sel = torch.softmax(logits.float(), -1), logits.float()
+    T, E = s.shape
     if n_group > 1:
         _, gidx = topk_stable(sel.view(T, n_group, E // n_group).amax(-1), topk_group)
         gmask = torch.zeros(T, n_group, dtype=torch.bool, device=sel.device).scatter_(1, gidx, True)
