@@ -1,5 +1,6 @@
 """One launch sequence on a small case, for a profiler: decode | chunk (recurrence, time-mix mode), gla (the same
-recurrence read after its update, with low-rank decays and the head norm), latent-decode | latent (latent attention)."""
+recurrence read after its update, with low-rank decays and the head norm), latent-decode | latent (latent attention),
+hyper (residual streams: join, read, norm), window-decode | window (windowed attention with kept tokens and gates)."""
 import os
 import sys
 
@@ -19,6 +20,19 @@ if case.startswith("latent"):
     cache, q, uv = rnd(blocks, 16, 1, lay.row), rnd(T, heads, lay.row, std=0.3), rnd(heads, 128, 512, std=0.05)
     out = torch.empty(T, heads * 128, dtype=q.dtype, device="cuda")
     run = lambda: lt.attention(q, cache, b, uv, 0.07, "bf16", lay, out)
+elif case == "hyper":
+    T, W, S = 8192, 2560, 2
+    x, pre = rnd(T, S, W, dtype=torch.float32), mx.DytNorm(0.5, rnd(W), rnd(W))
+    hc, out = mx.HyperW(*(torch.full(s, 0.4, device="cuda") for s in ((S,), (S,), (S, S)))), mx.SublayerOut(rnd(T, W))
+    run = lambda: mx.stream_hyper(x, S, "bf16", pending=out, hc=hc, w_in=hc.w_in, pre=pre)
+elif case.startswith("window"):
+    lens, start = ([1] * 128, 1023) if case == "window-decode" else ([4096], 0)
+    b, blocks = batch(lens, start)
+    T, H, G = sum(lens), 32, 8
+    kc, vc, q, z = rnd(blocks, 16, G, D), rnd(blocks, 16, G, D), rnd(T, H, D), rnd(T, H * D)
+    out = torch.empty_like(z)
+    run = lambda: mx.attention_dims(q, kc, vc, b, dk=D, dv=D, scale=0.09, sink=False, fmt="bf16", out=out, window=512, keep=4,
+                                    gate=mx.OutputGate(z, False))
 else:
     lens, start = ([1] * 128, 63) if case == "decode" else ([4096], 0)
     b, _ = batch(lens, start)

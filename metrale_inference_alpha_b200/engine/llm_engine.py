@@ -33,7 +33,7 @@ from .runner import ModelRunner, plan_kv_blocks
 class EngineArgs:
     model: Union[str, ModelConfig] = "tiny-dense"     # preset name, checkpoint dir, or a config
     device: str = "cpu"
-    dtype: str = "auto"                                # auto (the model's) | bf16 | fp32 (true 32-bit: Fabulix and Finelix models)
+    dtype: str = "auto"                                # auto (the model's) | bf16 | fp32 (true 32-bit: Fabulix, Finelix and Pivipel models)
     seed: int = 0
     max_num_seqs: int = 128
     max_model_len: int = 2048

@@ -294,10 +294,9 @@ __device__ __forceinline__ void store_out4(const AttnParams& p, size_t orow, int
   __nv_bfloat16* dst = p.out + m * p.out_ld + (size_t)head * p.dv + c4 * 4;
   const float os = p.gate.mode == mb::GATE_HEAD ? p.out_scale * p.gate(m, head, 0) : p.out_scale;
   if (p.gate.mode == mb::GATE_ELEMENT) {
-    if (c4 * 4 < p.dv) a *= p.gate(m, head, c4 * 4);
-    if (c4 * 4 + 1 < p.dv) b *= p.gate(m, head, c4 * 4 + 1);
-    if (c4 * 4 + 2 < p.dv) c *= p.gate(m, head, c4 * 4 + 2);
-    if (c4 * 4 + 3 < p.dv) d *= p.gate(m, head, c4 * 4 + 3);
+    float v[4] = {a, b, c, d};
+    p.gate.scale4(m, head, c4 * 4, v);
+    a = v[0]; b = v[1]; c = v[2]; d = v[3];
   }
   if (p.dv == D) {
     *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a * os, b * os);

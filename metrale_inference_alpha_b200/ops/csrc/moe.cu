@@ -89,6 +89,11 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
           if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
         }
       }
+      if (mode == 0) {
+        b1 = mb::warp_max(b1);
+        if (lane == g) gscore_mine = b1;
+        continue;
+      }
       // merge (b1, b2) pairs across lanes
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) {
@@ -97,7 +102,7 @@ route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int K
         const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
         b1 = n1; b2 = n2;
       }
-      if (lane == g) gscore_mine = mode == 0 ? b1 : b1 + b2;
+      if (lane == g) gscore_mine = b1 + b2;
     }
     // pick topk_group groups (ties -> lower group id); keep-mask as a bit set
     uint32_t keep = 0;

@@ -44,6 +44,22 @@ struct OutputGate {
     else v = *z;
     return 1.f / (1.f + expf(-v));
   }
+  // elements d .. d + 3 of a bf16 gate times v (d a multiple of 4; those past dv stay)
+  __device__ __forceinline__ void scale4(size_t row, int head, int d, float* v) const {
+    const T* z = logits + row * ld + (size_t)head * dv + d;
+    if (d + 4 <= dv && (reinterpret_cast<uintptr_t>(z) & 7) == 0) {
+      const uint2 w = __ldg(reinterpret_cast<const uint2*>(z));
+      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.x));
+      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.y));
+      const float g[4] = {a.x, a.y, b.x, b.y};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] *= __fdividef(1.f, 1.f + __expf(-g[i]));
+      return;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (d + i < dv) v[i] *= (*this)(row, head, d + i);
+  }
 };
 
 }  // namespace mb
