@@ -17,16 +17,17 @@ from typing import List, Optional
 
 WEIGHT_FORMATS = ("bf16", "nvfp4", "fp8_block", "fp8_row", "fp32")
 KV_DTYPES = ("bf16", "fp8", "fp32")
-LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning", "latent", "gla", "gated")
-KV_KINDS = ("attention", "mla", "parallel", "latent", "gated")           # kinds that own a KV pool
-STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning", "gla")   # kinds that own a recurrent state
+LAYER_KINDS = ("attention", "gdn", "mamba2", "mla", "kda", "parallel", "lightning", "latent", "gla", "gated", "twin",
+               "delta")
+KV_KINDS = ("attention", "mla", "parallel", "latent", "gated", "twin")   # kinds that own a KV pool
+STATE_KINDS = ("gdn", "mamba2", "kda", "parallel", "lightning", "gla", "twin", "delta")   # kinds that own a recurrent state
 FFN_KINDS = ("dense", "moe", "none")
 
 
 @dataclass
 class ModelConfig:
     name: str = "model"
-    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix | finelix | pivipel
+    arch: str = "dense_gqa"            # dense_gqa | qwen_hybrid | nemotron_h | deepseek_mla | fabulix | finelix | pivipel | ledinex
     vocab_size: int = 4096
     hidden_size: int = 256
     num_layers: int = 2
@@ -61,11 +62,13 @@ class ModelConfig:
     residual_multiplier: float = 1.0    # Granite: a block's output is scaled by this before it joins the stream
     logits_divisor: float = 1.0         # Granite: logits are divided by this
     tie_embeddings: bool = False
-    # fabulix, finelix, pivipel: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
+    # fabulix, finelix, pivipel, ledinex: per-layer mixer and feed-forward sizes and constants, [{"mixer": {...}, "mlp": {...} | None}, ...]
     layer_specs: List[dict] = field(default_factory=list)
-    spec_types: List[str] = field(default_factory=list)      # pivipel: the layers' own type names (variants of one layer kind)
+    spec_types: List[str] = field(default_factory=list)      # pivipel, ledinex: the layers' own type names (variants of one layer kind)
     weights_of: List[int] = field(default_factory=list)      # per layer: the layer whose tensors it uses, -1 = its own; empty = all their own
     streams: int = 0                    # static hyper-connections: the residual is this many fp32 copies (0 = a single residual)
+    canon_taps: int = 0                 # every sublayer reads the stream through a causal convolution of this many taps (0 = as it is)
+    logit_scale: float = 1.0            # logits are multiplied by this (folded into the final norm at load)
     loop: Optional[dict] = None         # layers start .. stop - 1 run `times` times with the same weights: {"start", "stop", "times"}
     token_side_dim: int = 0             # width of a layer's slice of the token side embedding (0 = none)
     glu_alpha: float = 1.702            # sigmoid slope of the clamped GLU
@@ -174,7 +177,7 @@ class ModelConfig:
     @property
     def stream32(self) -> bool:
         """The residual stream is kept in 32-bit, and the layers' sizes are per layer (``layer_specs``)."""
-        return self.arch in ("fabulix", "finelix", "pivipel")
+        return self.arch in ("fabulix", "finelix", "pivipel", "ledinex")
 
     def layer_owner(self, i: int) -> int:
         """The layer whose tensors layer i uses (its cache or state is its own all the same)."""
@@ -211,6 +214,9 @@ class ModelConfig:
                 out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
             elif t == "gated":
                 out.append((m["kv_heads"], *padded_head_dims(m["dim"], m["vdim"], self.act_fmt)))
+            elif t == "twin":
+                m = m["left"]
+                out.append((m["kv_heads"], *padded_head_dims(m["dim"], m.get("vdim", m["dim"]), self.act_fmt)))
             elif t == "latent":
                 out.append((1, latent_row(m["kv_rank"], m["rot_dim"], self.act_fmt).row, 0))
         return out
@@ -507,8 +513,55 @@ def pivipel_3b(**kw) -> ModelConfig:
     return pivipel(**base)
 
 
+def ledinex(num_layers: int = 4, width: int = 192, heads: int = 4, kv_heads: int = 2, dim: int = 64, vdim: int = 64, rot_dims: int = 32,
+            window: int = 40, softcap: float = 25.0, right_heads: int = 3, right_dim: int = 64, right_vdim: int = 64, delta_heads: int = 4,
+            delta_kv_heads: int = 2, delta_dim: int = 64, delta_vdim: int = 64, conv: int = 4, taps: int = 3, experts: int = 8, top: int = 2,
+            expert_ff: int = 80, shared_ff: int = 160, vocab: int = 1024, order=("delta", "parallel", "parallel_2"), eps: float = 1e-6,
+            **kw) -> ModelConfig:
+    """Ledinex decoder of uniform layers: the types of `order` in turn, a mixture of experts in each."""
+    layers = []
+    for i in range(num_layers):
+        t = order[i % len(order)]
+        left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "scale": dim ** -0.5}
+        if t == "delta":
+            m = {"heads": delta_heads, "kv_heads": delta_kv_heads, "dim": delta_dim, "vdim": delta_vdim, "conv": conv}
+        elif t == "parallel":
+            left.update(vdim=vdim, softcap=softcap, rot={"base": 500000.0, "dims": dim, "scaling": {"factor": 4.0}})
+            right = {"heads": right_heads, "dim": right_dim, "vdim": right_vdim,
+                     "decay": [1.0 - 2.0 ** -(1.0 + 6.0 * (h + 1) / right_heads) for h in range(right_heads)]}
+            m = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.6}
+        else:
+            left.update(vdim=dim, mask={"size": window},
+                        rot={"base": 10000.0, "dims": rot_dims, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}})
+            m = {"left": left, "right": {"heads": right_heads, "dim": right_dim}, "left_scale": 0.7, "right_scale": 0.6}
+        mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+        if shared_ff:
+            mlp["shared"] = {"ff": shared_ff}
+        layers.append({"type": t, "mixer": m, "mlp": mlp})
+    cfg = {"architecture": "Ledinex", "vocab": vocab, "width": width, "embedding": {"scale": float(width) ** 0.5}, "logit_scale": 1.5,
+           "canon": {"taps": taps}, "norm": {"eps": eps}, "layers": layers}
+    return from_ledinex_config(cfg, name=kw.pop("name", "ledinex")).scaled(**kw)
+
+
+def tiny_ledinex(**kw) -> ModelConfig:
+    """Four-layer Ledinex (tests, smoke runs)."""
+    return ledinex(**{"name": "tiny-ledinex", **kw})
+
+
+def ledinex_3b(**kw) -> ModelConfig:
+    """Ledinex with the layer sizes of a ~3B-active model: width 2560, 32 query / 8 key-value heads of 128, 20 recurrent heads
+    of 128 x 128, windows of 1024, 64 experts of 1024, top 6, and a shared one of 2048; 24 layers."""
+    base = dict(name="ledinex-3b", num_layers=24, width=2560, heads=32, kv_heads=8, dim=128, vdim=128, rot_dims=128, window=1024,
+                right_heads=20, right_dim=128, right_vdim=128, delta_heads=20, delta_kv_heads=20, delta_dim=128, delta_vdim=128, experts=64,
+                top=6, expert_ff=1024, shared_ff=2048, vocab=65536)
+    base.update(kw)
+    return ledinex(**base)
+
+
 PRESETS = {
     "tiny-dense": tiny_dense,
+    "tiny-ledinex": tiny_ledinex,
+    "ledinex-3b": ledinex_3b,
     "tiny-pivipel": tiny_pivipel,
     "pivipel-3b": pivipel_3b,
     "tiny-finelix": tiny_finelix,
@@ -687,8 +740,58 @@ def from_pivipel_config(cfg: dict, name: str = "model") -> ModelConfig:
         moe_intermediate_size=moe["expert"]["ff"] if moe else 0, max_position=int(cfg["max_positions"]))
 
 
+_LEDINEX_MIXERS = {"parallel": "twin", "parallel_2": "twin", "delta": "delta"}
+
+
+def from_ledinex_config(cfg: dict, name: str = "model") -> ModelConfig:
+    """A Ledinex ``config.json``: sizes and constants are given per layer and kept per layer. Mixer types and feed-forward
+    kinds this engine does not know are refused."""
+    types, ffns, specs = [], [], []
+    for i, L in enumerate(cfg["layers"]):
+        t, m, mlp = L["type"], L["mixer"], L.get("mlp")
+        if t not in _LEDINEX_MIXERS:
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+        if mlp is not None and mlp.get("kind") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+        if t == "delta":
+            if m["heads"] % m["kv_heads"] or not 0 < m["conv"] <= 17 or m["dim"] > 256:
+                raise ValueError(f"layer {i}: heads, head sizes or taps this engine does not serve")
+        else:
+            a, r = m["left"], m["right"]
+            rot = a["rot"]["dims"]
+            if a["heads"] % a["kv_heads"] or rot % 2 or rot > a["dim"] or (t == "parallel" and a["vdim"] % 2):
+                raise ValueError(f"layer {i}: attention heads, key/value heads or rotary size do not fit together")
+            if t == "parallel_2" and a.get("vdim", a["dim"]) != a["dim"]:
+                raise ValueError(f"layer {i}: values that are keys have their size")
+            if (a.get("mask") or {}).get("size", 1) < 1:
+                raise ValueError(f"layer {i}: a window of {a['mask']['size']}")
+            if r["dim"] > 256 or (t == "parallel" and len(r["decay"]) != r["heads"]):
+                raise ValueError(f"layer {i}: recurrent heads, head sizes or decays do not fit together")
+        if mlp is not None:
+            r = mlp["router"]
+            if r["experts"] > 512 or not 0 < r["top"] <= min(32, r["experts"]):
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts per token")
+        types.append(t)
+        ffns.append("none" if mlp is None else "moe")
+        specs.append({"mixer": m, "mlp": mlp})
+    taps = int(cfg["canon"]["taps"])
+    if not 0 < taps <= 21:
+        raise ValueError(f"input convolutions of {taps} taps")
+    att = next((s["mixer"]["left"] for t, s in zip(types, specs) if t != "delta"), {"heads": 1, "kv_heads": 1, "dim": 64})
+    moe = next((s["mlp"] for s in specs if s["mlp"]), None)
+    return ModelConfig(
+        name=name, arch="ledinex", vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_layers=len(types),
+        layer_types=[_LEDINEX_MIXERS[t] for t in types], ffn_types=ffns, layer_specs=specs, spec_types=types, canon_taps=taps,
+        num_heads=att["heads"], num_kv_heads=att["kv_heads"], head_dim=att["dim"], rotary_dim=-1, rms_eps=float(cfg["norm"]["eps"]),
+        norm_plus_one=True, embed_scale=float(cfg["embedding"]["scale"]), logit_scale=float(cfg["logit_scale"]), tie_embeddings=True,
+        intermediate_size=0, ffn_act="relu2", num_experts=moe["router"]["experts"] if moe else 0,
+        experts_per_token=moe["router"]["top"] if moe else 0, moe_intermediate_size=moe["expert"]["ff"] if moe else 0, max_position=131072)
+
+
 def from_hf_config(cfg: dict, name: str = "model") -> ModelConfig:
     """Map a HF ``config.json`` dict (text stack) to ModelConfig; refuses unknown model types."""
+    if cfg.get("architecture") == "Ledinex":
+        return from_ledinex_config(cfg, name)
     if cfg.get("architecture") == "Pivipel":
         return from_pivipel_config(cfg, name)
     if cfg.get("architecture") == "Fabulix":

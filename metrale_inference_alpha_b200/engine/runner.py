@@ -51,6 +51,10 @@ def state_shapes(cfg: ModelConfig, w: ModelW):
         elif lw.kind in ("lightning", "gla"):
             m = lw.mixer
             out.append(((0,), (m.heads, m.dim, m.vdim)))
+        elif lw.kind in ("twin", "delta"):         # the windows of the layer's convolutions in one row
+            from ..models.canon import window_floats
+            m = lw.mixer.right if lw.kind == "twin" else lw.mixer
+            out.append(((window_floats(cfg, lw),), (m.heads, m.dim, m.vdim)))
     return out
 
 

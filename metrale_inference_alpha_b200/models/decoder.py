@@ -23,7 +23,7 @@ from ..ops import ACT_FOR_WEIGHT, Act
 from ..ops import reference as ref
 from ..ops import mixers
 from ..weights.loader import AttnW, FfnW, LayerW, ModelW
-from .stream import HyperStream, ResidualStream
+from .stream import CanonStream, HyperStream, ResidualStream
 
 
 class LayerCaches:
@@ -289,6 +289,9 @@ class Decoder:
         if isinstance(x, HyperStream):
             from .hyper import hyper_layer
             return hyper_layer(self, x, lw, batch, caches, i if run is None else run)
+        if isinstance(x, CanonStream):
+            from .canon import canon_layer
+            return canon_layer(self, x, lw, batch, caches, i if run is None else run)
         if lw.out is not None:
             from .joint import joint_layer
             return joint_layer(self, x, lw, batch, caches, i if run is None else run)
@@ -340,6 +343,8 @@ class Decoder:
             x = mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale, pos=self.w.pos_embed, positions=positions,
                                     norm=self.w.embed_norm)
             return HyperStream(x, self.cfg.streams, self.cfg.act_fmt)
+        if self.cfg.canon_taps > 0:
+            return CanonStream(mixers.embed_scaled(token_ids, self.w.embed, self.cfg.embed_scale), self.cfg.act_fmt)
         if self.cfg.stream32:
             fmt, pair, W = self.cfg.act_fmt, None, self.cfg.hidden_size
             if self.w.loop_in is not None:
@@ -420,7 +425,7 @@ class Decoder:
         if batch.logit_rows.numel() != x.shape[0]:
             rows = x.take(batch.logit_rows) if hasattr(x, "take") and not torch.is_tensor(x) else self.full(x).index_select(0, batch.logit_rows)
         else:
-            rows = self.full(x) if isinstance(x, HyperStream) else x
+            rows = self.full(x) if isinstance(x, (CanonStream, HyperStream)) else x
         lg = self.logits(rows, out_f32=out_f32, gather=gather_logits)
         return lg, self.res(rows)
 

@@ -79,7 +79,7 @@ def routed_rows(dec, a, logits, w):
     from ..ops.mixers import Routed
     weights, idx = moe_ops.route(logits, w.spec, w.bias)
     if not a.data.is_cuda:
-        return Routed(moe_ops.expert_sum_ref(a, weights, idx, w.grouped, dec.cfg.hidden_size), None, None)
+        return Routed(moe_ops.expert_sum_ref(a, weights, idx, w.grouped, dec.cfg.hidden_size, w.spec.ffn_act), None, None)
     from ..ops.moe_cuda import grouped_pairs
     y, sp = grouped_pairs(w.spec, a, idx, w)
     return Routed(y, sp.pair_row, weights)

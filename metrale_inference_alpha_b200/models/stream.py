@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from ..ops import mixers as mx
+from ..ops import canon, mixers as mx
 
 
 class ResidualStream:
@@ -114,6 +114,51 @@ class HyperStream:
     def resolve(self) -> torch.Tensor:
         """The sum of the streams in fp32, nothing pending."""
         return self._sum()
+
+    @property
+    def value(self) -> torch.Tensor:
+        return self.resolve()
+
+
+class CanonStream:
+    """The residual of models whose sublayers read x + conv(x), a short causal convolution, and join through an RMS norm of
+    their output: one fp32 stream. One kernel joins the pending output and makes the next input."""
+
+    def __init__(self, x: torch.Tensor, fmt: str):
+        self.x, self.fmt = x, fmt                       # fp32 [T, W]
+        self.pending: Optional[mx.SublayerOut] = None
+        self.post: Optional[mx.RmsNorm] = None
+
+    @property
+    def shape(self):
+        return self.x.shape
+
+    def read(self, filt: torch.Tensor, window: "canon.Window", batch, stash=None) -> torch.Tensor:
+        """The next sublayer's input; the window moves on, or waits for the accepted rows of a verify step."""
+        h = self._step(filt=filt, window=window, batch=batch, write_state=stash is None)
+        if stash is not None:
+            x, taps = self.x, filt.shape[0]
+            stash.later.append(lambda cb: canon.canon_commit(x, taps, window, cb))
+        return h
+
+    def add(self, out: mx.SublayerOut, post: mx.RmsNorm) -> "CanonStream":
+        assert self.pending is None
+        self.pending, self.post = out, post
+        return self
+
+    def _step(self, **kw):
+        self.x, h = canon.stream_canon(self.x, self.fmt, pending=self.pending, norm=self.post, **kw)
+        self.pending = self.post = None
+        return h
+
+    def take(self, rows: torch.Tensor) -> torch.Tensor:
+        """Chosen rows of x in fp32."""
+        return self.resolve().index_select(0, rows)
+
+    def resolve(self) -> torch.Tensor:
+        """x in fp32, nothing pending."""
+        self._step()
+        return self.x
 
     @property
     def value(self) -> torch.Tensor:

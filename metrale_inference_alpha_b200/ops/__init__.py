@@ -33,7 +33,7 @@ GEMM_ONE_TILE_PER_CTA, GEMM_DECODE_TILE_ORDER, GEMM_PERSISTENT_PREFILL, GEMM_DSM
 # measure 1.5x faster there; METRALE_PERSISTENT_PREFILL=0 keeps one tile per CTA)
 _PERSIST_PREFILL = GEMM_PERSISTENT_PREFILL if os.environ.get("METRALE_PERSISTENT_PREFILL", "1") != "0" else 0
 GEMM_GROUPED_ONE_CTA = 512
-EPI_SWIGLU, EPI_CLAMP_GLU, EPI_SILU_COLS, EPI_NEG_EXP, EPI_GEGLU, EPI_BIAS, EPI_LOG_SIGMOID = 1, 2, 3, 4, 5, 6, 7      # csrc/epilogue.cuh
+EPI_SWIGLU, EPI_CLAMP_GLU, EPI_SILU_COLS, EPI_NEG_EXP, EPI_GEGLU, EPI_BIAS, EPI_LOG_SIGMOID, EPI_RELU2, EPI_SIGMOID = 1, 2, 3, 4, 5, 6, 7, 8, 9      # csrc/epilogue.cuh
 _GROUPED_CTAS = GEMM_GROUPED_ONE_CTA if os.environ.get("METRALE_GROUPED_CTAS", "2") == "1" else 0
 
 
@@ -424,13 +424,17 @@ def _linear_a16(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool,
     return out
 
 
-def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu=False, bias=None, log_sigmoid=None):
+def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu=False, bias=None, log_sigmoid=None, relu2=False, sigmoid=None):
     if geglu:
         y = torch.nn.functional.gelu(y[:, 0::2], approximate="tanh") * y[:, 1::2]
     elif bias is not None:
         y = y + bias
     elif log_sigmoid is not None:
         y = log_sigmoid[1] * ref.log_sigmoid(y + log_sigmoid[0])
+    elif sigmoid is not None:
+        y = sigmoid[1] * torch.sigmoid(y + sigmoid[0])
+    elif relu2:
+        y = torch.relu(y).square()
     if clamp_glu is not None:
         alpha, limit = clamp_glu
         g, u = y[:, 0::2].clamp(max=limit), y[:, 1::2].clamp(-limit, limit)
@@ -443,12 +447,12 @@ def _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu=False,
 
 
 def _linear_simt(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool, out, clamp_glu, silu_cols: int, geglu=False, bias=None,
-                 log_sigmoid=None):
+                 log_sigmoid=None, relu2=False, sigmoid=None):
     """CUDA-core GEMM (csrc/gemm_simt.cu); on CPU its fp64-accumulated restatement."""
     assert residual is None, "the CUDA-core GEMM has no residual epilogue"
     f32 = out_f32 or w.fmt == "fp32"
     if not act.data.is_cuda:
-        y = _linear_epilogue_ref((act.data.double() @ w.dequant64().t()).float(), swiglu, clamp_glu, silu_cols, None, geglu, bias, log_sigmoid)
+        y = _linear_epilogue_ref((act.data.double() @ w.dequant64().t()).float(), swiglu, clamp_glu, silu_cols, None, geglu, bias, log_sigmoid, relu2, sigmoid)
         y = y if f32 else y.to(torch.bfloat16)
         return y if out is None else out.copy_(y)
     from .mixers import gemm_simt
@@ -462,6 +466,10 @@ def _linear_simt(act: Act, w: QuantWeight, residual, swiglu: bool, out_f32: bool
         return gemm_simt(act.data, w.data, out, epilogue=EPI_BIAS, bias=bias)
     if log_sigmoid is not None:
         return gemm_simt(act.data, w.data, out, epilogue=EPI_LOG_SIGMOID, bias=log_sigmoid[0], epi_a=log_sigmoid[1])
+    if sigmoid is not None:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_SIGMOID, bias=sigmoid[0], epi_a=sigmoid[1])
+    if relu2:
+        return gemm_simt(act.data, w.data, out, epilogue=EPI_RELU2)
     return gemm_simt(act.data, w.data, out, epilogue=EPI_SILU_COLS if silu_cols else 0, epi_n=silu_cols)
 
 
@@ -470,7 +478,7 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
            force_tn: int = 0, force_splits: int = 0, one_tile_per_cta: bool = False, decode_tile_order: bool = False,
            dsmem_splitk: bool = False, grouped=None, no_cluster: bool = False, quant_out: float = 0.0,
            clamp_glu: Optional[Tuple[float, float]] = None, silu_cols: int = 0, neg_exp_bias=None,
-           geglu: bool = False, bias: Optional[torch.Tensor] = None, log_sigmoid=None):
+           geglu: bool = False, bias: Optional[torch.Tensor] = None, log_sigmoid=None, relu2: bool = False, sigmoid=None):
     """out[m, n] = sum_k act[m, k] * w[n, k] (+ residual); with `swiglu`, w holds gate/up rows
     interleaved (2j, 2j+1) and the result is silu(gate) * up of width N/2. `quant_out` > 0 (with
     `swiglu`): return the result as an NVFP4 `Act` quantised with that calibrated global scale --
@@ -482,11 +490,12 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
     g = min(gate, limit) and u = clamp(up, -limit, limit), result g * sigmoid(alpha g) * (u + 1).
     `silu_cols`: SiLU on the first that many output columns. `neg_exp_bias` (CUDA, bf16): -exp(y + bias). `geglu`: like
     `swiglu` with gelu_tanh(gate) * up. `bias` (fp32 [N]): y + bias. `log_sigmoid` = (bias, c): c * log(sigmoid(y + bias)).
+    `sigmoid` = (bias, c): c * sigmoid(y + bias). `relu2`: relu(y)^2.
     An fp32 weight gives fp32 outputs."""
     assert act.K == w.K, (act.K, w.K)
     if w.fmt == "fp32" or (act.data.is_cuda and w.fmt == "bf16" and w.K % 8):
         # true 32-bit, or bf16 rows that are not whole 16-byte vectors (no tensor map can describe them)
-        return _linear_simt(act, w, residual, swiglu, out_f32, out, clamp_glu, silu_cols, geglu, bias, log_sigmoid)
+        return _linear_simt(act, w, residual, swiglu, out_f32, out, clamp_glu, silu_cols, geglu, bias, log_sigmoid, relu2, sigmoid)
     a16 = act.fmt == "bf16" and w.fmt != "bf16"
     assert a16 or act.fmt == NATIVE_ACT_FOR_WEIGHT[w.fmt], (act.fmt, w.fmt)
     M, N = act.M, w.N
@@ -507,7 +516,7 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         # (fp32 BLAS picks different blockings for different M, and a random-weight test model has
         # near-ties everywhere), so that batch-invariance tests on the CPU path are exact
         y = (act.data.double() @ w.dequant64().t()).float()
-        y = _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu, bias, log_sigmoid)
+        y = _linear_epilogue_ref(y, swiglu, clamp_glu, silu_cols, residual, geglu, bias, log_sigmoid, relu2, sigmoid)
         y = y if out_f32 else y.to(torch.bfloat16)
         return y if out is None else out.copy_(y)
     L = _native.lib()
@@ -550,6 +559,10 @@ def linear(act: Act, w: QuantWeight, *, residual: Optional[torch.Tensor] = None,
         a.epilogue, a.epi_bias = EPI_BIAS, _ptr(bias)
     elif log_sigmoid is not None:
         a.epilogue, a.epi_bias, a.epi_a = EPI_LOG_SIGMOID, _ptr(log_sigmoid[0]), float(log_sigmoid[1])
+    elif sigmoid is not None:
+        a.epilogue, a.epi_bias, a.epi_a = EPI_SIGMOID, _ptr(sigmoid[0]), float(sigmoid[1])
+    elif relu2:
+        a.epilogue = EPI_RELU2
     a.ws, a.ws_bytes, a.status = _ptr(rt.ws), rt.ws_bytes, _ptr(rt.status)
     a.force_tn, a.force_splits, a.sm_count = force_tn, force_splits, rt.sm_count
     a.flags = (_PERSIST_PREFILL | _GROUPED_CTAS | (GEMM_ONE_TILE_PER_CTA if one_tile_per_cta else 0)

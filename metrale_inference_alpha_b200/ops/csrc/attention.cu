@@ -261,6 +261,7 @@ struct AttnParams {
   const float* sink_w;      // [Hq] or null (score 0)
   int keep;                 // with a window: the first tokens that every query sees
   mb::OutputGate<__nv_bfloat16> gate;
+  mb::SoftCap softcap;      // bf16 caches
   int split_p;              // the weights enter the product with V as two bf16 terms (16 mantissa bits)
 };
 
@@ -700,6 +701,16 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
     const int pos0 = vis.token(tok0);                  // the 16 entries are consecutive positions
     const bool need_mask = (pos0 + 16 > min_limit) || (tok0 + 16 > tok_end) ||
                            (p.window > 0 && pos0 < ctx - p.window && pos0 + 16 > p.keep);
+    const bool capped = !FP8 && p.softcap.cap > 0.f;
+    if (capped) {
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) s[mt][n][i] = p.softcap(s[mt][n][i]);
+    }
+    const float mul = capped ? 1.f : sc_log2;
     uint32_t pa[MT][4], pr[MT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
@@ -713,7 +724,7 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
               const int o = n * 8 + t * 2 + i;
-              float v = s[mt][n][hr * 2 + i] * sc_log2;
+              float v = s[mt][n][hr * 2 + i] * mul;
               if (tok0 + o >= tok_end || !mb::sees(pos0 + o, limit, p.window, p.keep)) v = -INFINITY;
               s[mt][n][hr * 2 + i] = v;
               mx = fmaxf(mx, v);
@@ -723,7 +734,7 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
           for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-              const float v = s[mt][n][hr * 2 + i] * sc_log2;
+              const float v = s[mt][n][hr * 2 + i] * mul;
               s[mt][n][hr * 2 + i] = v;
               mx = fmaxf(mx, v);
             }
@@ -1008,6 +1019,14 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
         mma16816<F16>(s[nb * 2 + 1], a, b[2], b[3]);
       }
     }
+    const bool capped = !FP8 && p.softcap.cap > 0.f;
+    if (capped) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[n][i] = p.softcap(s[n][i]);
+    }
+    const float mul = capped ? 1.f : sc_log2;
     float alpha[2];
 #pragma unroll
     for (int hr = 0; hr < 2; ++hr) {
@@ -1019,7 +1038,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int tok = tile_tok0 + n * 8 + (lane & 3) * 2 + i;
-          float v = s[n][hr * 2 + i] * sc_log2;
+          float v = s[n][hr * 2 + i] * mul;
           if (tok >= tok_end || qr >= qlen || !mb::sees(tok, limit, p.window, p.keep)) v = -INFINITY;
           s[n][hr * 2 + i] = v;
           mx = fmaxf(mx, v);
@@ -1251,6 +1270,7 @@ struct MbAttnArgs {
   const void* gate;        // logits of sigmoid gates on the output (bf16), or null
   long long gate_ld;
   int gate_mode;           // 1 one per head, 2 one per element
+  float softcap;           // 0: off; scores become softcap tanh(score / softcap)
 };
 
 // most entries of the visible-token list of a sequence: its context, or the kept first tokens and the windows of its
@@ -1289,10 +1309,11 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
   p.sink = a->sink; p.split_p = a->split_p;
   p.sink_w = a->sink_w; p.keep = a->window > 0 ? a->keep : 0;
   p.gate = {reinterpret_cast<const __nv_bfloat16*>(a->gate), a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, p.dv};
+  p.softcap = mb::SoftCap::make(a->scale, a->softcap);
   if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
   if (p.dv > DV || p.out_ld < (long long)a->Hq * p.dv) return MB_ERR_BAD_ARG;
   if (p.dv == DV && (p.out_ld % 2 || (reinterpret_cast<uintptr_t>(a->out) & 3))) return MB_ERR_BAD_ARG;   // paired stores
-  if ((DV != a->D || p.sink || p.split_p || p.dv != DV || p.gate.mode) && (a->cache_fp8 || a->outq)) return MB_ERR_UNSUPPORTED;
+  if ((DV != a->D || p.sink || p.split_p || p.dv != DV || p.gate.mode || p.softcap.cap > 0.f) && (a->cache_fp8 || a->outq)) return MB_ERR_UNSUPPORTED;
   const int G = a->Hq / a->Hkv;
   const int rows = G * a->max_q_len;
   int mode = a->force_mode;

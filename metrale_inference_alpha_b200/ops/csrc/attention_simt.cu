@@ -30,6 +30,7 @@ struct SimtAttnParams {
   const void* gate;
   long long gate_ld;
   int gate_mode;
+  float softcap;             // 0: off
   void* out;                 // row stride out_ld, head stride dv
   long long out_ld;
   uint32_t* status;
@@ -89,6 +90,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const SimtAttnParams p) 
       float a = 0.f;
       for (int d = 0; d < p.dk; ++d) a = fmaf(sq[d], lda(k + d), a);
       s = a * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     }
     const float m_new = fmaxf(m, mb::block_max(s, red));
     const float e = j < len ? expf(s - m_new) : 0.f;
@@ -147,6 +149,7 @@ struct MbSimtAttnArgs {
   const void* gate;
   long long gate_ld;
   int gate_mode;
+  float softcap;
 };
 
 extern "C" int mb_attn_simt(const MbSimtAttnArgs* a, cudaStream_t stream) {
@@ -155,7 +158,7 @@ extern "C" int mb_attn_simt(const MbSimtAttnArgs* a, cudaStream_t stream) {
   if (a->total_rows > 65535) return MB_ERR_TOO_LARGE;
   SimtAttnParams p{a->q, a->k_cache, a->v_cache, a->block_table, a->max_blocks, a->q_start, a->q_len, a->ctx_len, a->num_seqs, a->Hq, a->Hkv,
                    a->dk, a->dv, a->dkp, a->dvp, a->block_size, a->num_blocks, a->scale, a->out_scale, a->sink, a->sink_w, a->window, a->window > 0 ? a->keep : 0,
-                   a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->out, a->out_ld, a->status};
+                   a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->softcap, a->out, a->out_ld, a->status};
   if (p.keep < 0 || p.gate_mode < 0 || p.gate_mode > mb::GATE_ELEMENT) return MB_ERR_BAD_ARG;
   const dim3 grid(a->Hq, a->total_rows);
   const size_t smem = (size_t)a->dk * sizeof(float);

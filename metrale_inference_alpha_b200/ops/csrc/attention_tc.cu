@@ -59,6 +59,7 @@ struct TcParams {
   const float* sink_w;           // [Hq] or null (score 0)
   int window, keep;
   mb::OutputGate<__nv_bfloat16> gate;
+  mb::SoftCap softcap;           // bf16 caches
   uint32_t* status;
 };
 
@@ -253,18 +254,24 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
       float sv[kT];
 #pragma unroll
       for (int c = 0; c < kT / 16; ++c) mb::tmem_ld16(t_row + c * 16, sv + c * 16);
+      const bool capped = !FP8 && p.softcap.cap > 0.f;
+      if (capped) {
+#pragma unroll
+        for (int i = 0; i < kT; ++i) sv[i] = p.softcap(sv[i]);
+      }
+      const float mul = capped ? 1.f : sc_log2;
       float mx = -INFINITY;
       const int tok0 = vis.token(j * kT);
       if (tok0 + kT <= first_limit && (p.window <= 0 || tok0 >= last_limit - p.window || tok0 + kT <= p.keep)) {   // visible to every row of this CTA
 #pragma unroll
         for (int i = 0; i < kT; ++i) {
-          sv[i] *= sc_log2;
+          sv[i] *= mul;
           mx = fmaxf(mx, sv[i]);
         }
       } else {
 #pragma unroll
         for (int i = 0; i < kT; ++i) {
-          const float v = mb::sees(tok0 + i, limit, p.window, p.keep) ? sv[i] * sc_log2 : -INFINITY;
+          const float v = mb::sees(tok0 + i, limit, p.window, p.keep) ? sv[i] * mul : -INFINITY;
           sv[i] = v;
           mx = fmaxf(mx, v);
         }
@@ -410,6 +417,7 @@ struct MbAttnTcArgs {
   const void* gate;    // logits of sigmoid gates on the output (bf16), or null
   long long gate_ld;
   int gate_mode;       // 1 one per head, 2 one per element
+  float softcap;       // 0: off
 };
 
 // Causal paged attention for prefill chunks (head dim 128). Returns 0, MB_ERR_* or a CUDA error.
@@ -428,6 +436,8 @@ extern "C" int mb_attn_prefill_tc(const MbAttnTcArgs* a, cudaStream_t stream) {
   p.out_scale = a->out_scale != 0.f ? a->out_scale : 1.f;
   p.sink = a->sink; p.sink_w = a->sink_w;
   p.window = a->window; p.keep = a->window > 0 ? a->keep : 0;
+  p.softcap = mb::SoftCap::make(a->scale, a->softcap);
+  if (a->softcap > 0.f && a->cache_fp8) return MB_ERR_UNSUPPORTED;
   p.gate = {(const __nv_bfloat16*)a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->D};
   if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
   if (p.gate.mode == mb::GATE_ELEMENT && (a->gate_ld % 8 || (reinterpret_cast<uintptr_t>(a->gate) & 15))) return MB_ERR_UNSUPPORTED;

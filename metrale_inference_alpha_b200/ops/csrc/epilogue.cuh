@@ -4,8 +4,9 @@
 
 namespace mb {
 
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_NEG_EXP = 4, EPI_GEGLU = 5, EPI_BIAS = 6, EPI_LOG_SIGMOID = 7 };
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_NEG_EXP = 4, EPI_GEGLU = 5, EPI_BIAS = 6, EPI_LOG_SIGMOID = 7, EPI_RELU2 = 8, EPI_SIGMOID = 9 };
 
+__device__ __forceinline__ float relu2(float z) { const float r = fmaxf(z, 0.f); return r * r; }
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
 

@@ -46,7 +46,8 @@ struct MbGemmArgs {
   int n_per_expert, max_tiles;
   // epilogue parameters: 2 = clamped GLU (epi_a sigmoid slope, epi_b limit), 3 = SiLU on columns below epi_n,
   // 4 = -exp(y + epi_bias[n]), 5 = gelu_tanh(gate) * up
-  // on interleaved rows, 6 = y + epi_bias[n], 7 = epi_a * log(sigmoid(y + epi_bias[n])) (3 to 7: bf16 operands)
+  // on interleaved rows, 6 = y + epi_bias[n], 7 = epi_a * log(sigmoid(y + epi_bias[n])), 8 = relu(y)^2,
+  // 9 = epi_a * sigmoid(y + epi_bias[n]) (3 to 9: bf16 operands)
   float epi_a, epi_b;
   int epi_n;
   const float* epi_bias;

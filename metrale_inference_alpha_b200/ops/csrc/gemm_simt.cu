@@ -9,7 +9,7 @@
 // Operand function a(): identity or tanh. Epilogues (shared numbering with the tensor-core GEMM):
 //   plain; SwiGLU, tanh-GELU GLU and clamped GLU on interleaved (gate, up) rows; SiLU on the first epi_n columns;
 //   y + bias; -exp(y + bias), the logarithm of a decay exp(-exp(.)); epi_a log(sigmoid(y + bias)), that of a
-//   decay sigmoid(.)^epi_a.
+//   decay sigmoid(.)^epi_a; epi_a sigmoid(y + bias), that of a decay bounded below; relu(y)^2.
 // Grouped mode: a work list of (expert, first row, rows) tiles over rows sorted by expert, weights stacked
 // [experts * n_per_expert, K]; the rows may be read through an index (row r = X[row_index[r] / row_div]).
 // A CTA owns 64 x 64 outputs (64 x 16 when M <= 16), 256 threads, k steps of 16 through shared memory,
@@ -159,6 +159,10 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const SimtParams p) {
         y += p.bias[n + j];
       } else if (p.epilogue == mb::EPI_LOG_SIGMOID) {
         y = p.epi_a * mb::log_sigmoid(y + p.bias[n + j]);
+      } else if (p.epilogue == mb::EPI_SIGMOID) {
+        y = p.epi_a * mb::sigmoid_exact(y + p.bias[n + j]);
+      } else if (p.epilogue == mb::EPI_RELU2) {
+        y = mb::relu2(y);
       }
       st1(row + n + j, y);
     }
@@ -205,7 +209,7 @@ extern "C" int mb_gemm_simt(const MbSimtGemmArgs* a, cudaStream_t stream) {
   if (!a || !a->X || !a->W || !a->out || a->M <= 0 || a->N <= 0 || a->K <= 0) return MB_ERR_BAD_ARG;
   const bool glu = a->epilogue == mb::EPI_SWIGLU || a->epilogue == mb::EPI_CLAMP_GLU || a->epilogue == mb::EPI_GEGLU;
   if (glu && (a->N & 1)) return MB_ERR_BAD_ARG;
-  if ((a->epilogue == mb::EPI_BIAS || a->epilogue == mb::EPI_LOG_SIGMOID) && !a->bias) return MB_ERR_BAD_ARG;
+  if ((a->epilogue == mb::EPI_BIAS || a->epilogue == mb::EPI_LOG_SIGMOID || a->epilogue == mb::EPI_SIGMOID) && !a->bias) return MB_ERR_BAD_ARG;
   const bool grouped = a->tile_expert != nullptr;
   if (grouped && (!a->tile_row0 || !a->tile_nrows || a->max_tiles <= 0 || (a->tile_rows != 16 && a->tile_rows != 64))) return MB_ERR_BAD_ARG;
   if (a->row_index && a->row_div <= 0) return MB_ERR_BAD_ARG;

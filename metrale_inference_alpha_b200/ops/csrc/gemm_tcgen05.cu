@@ -48,6 +48,8 @@ using mb::EPI_GEGLU;
 using mb::EPI_LOG_SIGMOID;
 using mb::EPI_NEG_EXP;
 using mb::EPI_PLAIN;
+using mb::EPI_RELU2;
+using mb::EPI_SIGMOID;
 using mb::EPI_SILU_COLS;
 using mb::EPI_SWIGLU;
 
@@ -68,7 +70,7 @@ struct GemmParams {
   int epilogue, out_f32;
   float epi_a, epi_b;     // EPI_CLAMP_GLU: sigmoid slope and clamp limit; EPI_LOG_SIGMOID: epi_a log(sigmoid(y + bias[n]))
   int epi_n;              // EPI_SILU_COLS: SiLU on output columns below this
-  const float* epi_bias;  // EPI_NEG_EXP, EPI_BIAS, EPI_LOG_SIGMOID (set for those alone)
+  const float* epi_bias;  // EPI_NEG_EXP, EPI_BIAS, EPI_LOG_SIGMOID, EPI_SIGMOID (set for those alone)
   uint32_t* status;
   // grouped (MoE) mode: blockIdx.y indexes a tile work-list; W is [experts * n_per_expert, K]
   const int* tile_expert;
@@ -470,6 +472,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
 #pragma unroll
               for (int i = 0; i < 8; ++i) y[i] = n_out0 + i < p.epi_n ? mb::silu(y[i]) : y[i];
             }
+          } else if (KIND == KIND_BF16 && p.epilogue == EPI_RELU2) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[i] = mb::relu2(y[i]);
           } else if (KIND == KIND_BF16 && p.epi_bias) {
             float eb[8];
 #pragma unroll
@@ -482,6 +487,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
             } else if (p.epilogue == EPI_LOG_SIGMOID) {
 #pragma unroll
               for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::log_sigmoid(y[i]);
+            } else if (p.epilogue == EPI_SIGMOID) {
+#pragma unroll
+              for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::sigmoid_exact(y[i]);
             }
           }
         }
@@ -901,6 +909,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] = mb::silu(v[j] * wsc * asc[c * 16 + j]);
             }
+          } else if (KIND == KIND_BF16 && p.epilogue == EPI_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = mb::relu2(v[j] * wsc * asc[c * 16 + j]);
           } else if (KIND == KIND_BF16 && p.epi_bias) {        // bf16 operands: the scales below are 1
             const float bias = n < p.N ? p.epi_bias[n] : 0.f;
 #pragma unroll
@@ -911,6 +922,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             } else if (p.epilogue == EPI_LOG_SIGMOID) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::log_sigmoid(v[j]);
+            } else if (p.epilogue == EPI_SIGMOID) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::sigmoid_exact(v[j]);
             }
           }
 #pragma unroll
@@ -1024,8 +1038,8 @@ int mb_gemm(const MbGemmArgs* a, cudaStream_t stream) {
   if (kind == KIND_NVFP4 && (!a->sfa || !a->sfb)) return MB_ERR_BAD_ARG;
   if (kind == KIND_FP8_BLOCK && (!a->w_scale || !a->a_scale)) return MB_ERR_BAD_ARG;
   if ((a->epilogue == EPI_SWIGLU || a->epilogue == EPI_CLAMP_GLU || a->epilogue == EPI_GEGLU) && (a->out_f32 || a->residual)) return MB_ERR_BAD_ARG;
-  const bool biased = a->epilogue == EPI_NEG_EXP || a->epilogue == EPI_BIAS || a->epilogue == EPI_LOG_SIGMOID;
-  if ((a->epilogue == EPI_SILU_COLS || biased) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
+  const bool biased = a->epilogue == EPI_NEG_EXP || a->epilogue == EPI_BIAS || a->epilogue == EPI_LOG_SIGMOID || a->epilogue == EPI_SIGMOID;
+  if ((a->epilogue == EPI_SILU_COLS || a->epilogue == EPI_RELU2 || biased) && (a->residual || kind != KIND_BF16 || a->alpha != 1.f)) return MB_ERR_BAD_ARG;
   if (biased != (a->epi_bias != nullptr)) return MB_ERR_BAD_ARG;
   if ((a->epilogue == EPI_CLAMP_GLU || a->epilogue == EPI_GEGLU) && kind != KIND_BF16) return MB_ERR_UNSUPPORTED;
   const int num_kb = (a->K + kelems - 1) / kelems;

@@ -186,6 +186,7 @@ struct StreamRmsParams {
   float* x_out;              // or null
   void* out;
   long long out_ld;
+  float plus, scale;         // the norm's weight is (plus + w) scale
 };
 
 // a row is NIT vectors per thread, kept in registers between the sum of squares and the output
@@ -245,7 +246,7 @@ __global__ void __launch_bounds__(256) stream_rms_kernel(const StreamRmsParams p
       float w[VEC];
       ldn<VEC>(p.w + k, w);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[i][e] *= inv * w[e];
+      for (int e = 0; e < VEC; ++e) v[i][e] *= inv * (p.plus + w[e]) * p.scale;
     }
     stn<VEC>(reinterpret_cast<T*>(p.out) + (size_t)t * p.out_ld + k, v[i]);
   }
@@ -349,13 +350,14 @@ __global__ void __launch_bounds__(256) side_gate_kernel(const float* z, const in
 }
 
 // tanh(z) as two bf16 terms side by side: out[t] = [value (R) | remainder (R)], the operand of a GEMM against [W | W]
-__global__ void __launch_bounds__(256) tanh_split_kernel(const float* z, bf16* out, long long total, int R) {
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_split_kernel(const T* z, long long ld, bf16* out, long long total, int R) {
   mb::pdl_wait();
   mb::pdl_launch_dependents();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const long long t = i / R, c = i - t * R;
-  const float v = tanhf(z[i]);
+  const float v = tanhf(ldv(z + t * ld + c));
   const bf16 h = __float2bfloat16(v);
   out[t * 2 * R + c] = h;
   out[t * 2 * R + R + c] = __float2bfloat16(v - __bfloat162float(h));
@@ -608,6 +610,8 @@ struct MbStreamRmsArgs {
   float* x_out;
   void* out;
   long long out_ld;
+  int plus_one;              // the norm's weight is 1 + w
+  float scale;               // factor on the normed output
 };
 
 struct MbGatedNormArgs {
@@ -685,7 +689,8 @@ int mb_stream_norm(const MbStreamNormArgs* a, cudaStream_t stream) {
 int mb_stream_rms(const MbStreamRmsArgs* a, cudaStream_t stream) {
   if (!a || a->T <= 0 || a->W <= 0 || !a->x || (a->out_mode != RMS_NONE && !a->out) || (a->out_mode == RMS_NORM && !a->w)) return MB_ERR_BAD_ARG;
   if (a->ye && (!a->pair_row || !a->pair_w || a->K <= 0 || a->K > 32 || a->ye_ld < a->W)) return MB_ERR_BAD_ARG;
-  const StreamRmsParams p{a->W, a->x, a->y, a->ye, a->ye_ld, a->pair_row, a->pair_w, a->K, a->out_mode, (const bf16*)a->w, a->eps, a->x_out, a->out, a->out_ld};
+  const StreamRmsParams p{a->W, a->x, a->y, a->ye, a->ye_ld, a->pair_row, a->pair_w, a->K, a->out_mode, (const bf16*)a->w, a->eps, a->x_out, a->out, a->out_ld,
+                          a->plus_one ? 1.f : 0.f, a->scale};
   const bool v4 = a->W % 4 == 0 && a->out_ld % 4 == 0 && a->ye_ld % 4 == 0 && al(a->x, 16) && al(a->y, 16) && al(a->ye, 16) && al(a->x_out, 16) &&
                   al(a->out, a->f32 ? 16 : 8) && al(a->w, 8);
   const int vec = v4 ? 4 : 1, nt = max(row_threads(a->W, vec), 32), nit = (a->W + nt * vec - 1) / (nt * vec);
@@ -749,11 +754,16 @@ int mb_embed_scaled(const MbEmbedArgs* a, cudaStream_t stream) {
   return (int)(v4 ? mb::launch_kernel(embed_scaled_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(embed_scaled_kernel<1, bf16>, g, b, 0, stream, p));
 }
 
-int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) {
-  if (!z || !out || T <= 0 || R <= 0) return MB_ERR_BAD_ARG;
+// z [T, R] (fp32, or bf16), rows z_ld elements apart
+int mb_tanh_split_cols(const void* z, long long z_ld, int z_bf16, void* out, int T, int R, cudaStream_t stream) {
+  if (!z || !out || T <= 0 || R <= 0 || z_ld < R) return MB_ERR_BAD_ARG;
   const long long total = (long long)T * R;
-  return (int)mb::launch_kernel(tanh_split_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, z, (bf16*)out, total, R);
+  const dim3 g((unsigned)((total + 255) / 256)), b(256);
+  return (int)(z_bf16 ? mb::launch_kernel(tanh_split_kernel<bf16>, g, b, 0, stream, (const bf16*)z, z_ld, (bf16*)out, total, R)
+                      : mb::launch_kernel(tanh_split_kernel<float>, g, b, 0, stream, (const float*)z, z_ld, (bf16*)out, total, R));
 }
+
+int mb_tanh_split(const float* z, void* out, int T, int R, cudaStream_t stream) { return mb_tanh_split_cols(z, R, 0, out, T, R, stream); }
 
 int mb_rope_dims(const MbRopeDimsArgs* a, cudaStream_t stream) {
   if (!a || a->M <= 0 || !a->qkv || !a->positions || !a->slots || !a->q_out || !a->k_cache || !a->v_cache) return MB_ERR_BAD_ARG;

@@ -27,6 +27,21 @@ __device__ __forceinline__ bool sees(int tok, int limit, int window, int keep) {
   return tok < limit && (window <= 0 || tok >= limit - window || tok < keep);
 }
 
+// Scores squashed to (-cap, cap) before the softmax, cap tanh(s / cap), in the log2 domain of the kernels' scores and written
+// with one exponential: cap - 2 cap / (1 + exp(2 s / cap)). `mul` takes a raw dot product into the exponent.
+struct SoftCap {
+  float mul, cap;    // cap 0: off
+  static SoftCap make(float scale, float softcap) {
+    constexpr float kLog2e = 1.44269504088896f;
+    return softcap > 0.f ? SoftCap{2.f * scale * kLog2e / softcap, softcap * kLog2e} : SoftCap{0.f, 0.f};
+  }
+  __device__ __forceinline__ float operator()(float dot) const {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(dot * mul));
+    return cap - __fdividef(2.f * cap, 1.f + e);
+  }
+};
+
 enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 
 // Sigmoid gates on an attention output, read where the projection left their logits: one per head, or one per element

@@ -33,9 +33,15 @@ class DytNorm:
 
 @dataclass
 class RmsNorm:
-    """x / sqrt(mean(x^2) + eps) * w."""
+    """x / sqrt(mean(x^2) + eps) * w * scale, or 1 + w for weights that are stored around zero."""
     w: torch.Tensor        # bf16 [W]
     eps: float
+    plus_one: bool = False
+    scale: float = 1.0
+
+    def ref(self, x: torch.Tensor) -> torch.Tensor:
+        w = self.w.float() + 1.0 if self.plus_one else self.w.float()
+        return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + self.eps) * w * self.scale
 
 
 @dataclass
@@ -71,7 +77,8 @@ class _StreamNormArgs(C.Structure):
 class _StreamRmsArgs(C.Structure):
     _fields_ = [("T", C.c_int), ("W", C.c_int), ("f32", C.c_int), ("out_mode", C.c_int), ("x", C.c_void_p), ("y", C.c_void_p),
                 ("ye", C.c_void_p), ("ye_ld", C.c_longlong), ("pair_row", C.c_void_p), ("pair_w", C.c_void_p), ("K", C.c_int),
-                ("w", C.c_void_p), ("eps", C.c_float), ("x_out", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_longlong)]
+                ("w", C.c_void_p), ("eps", C.c_float), ("x_out", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_longlong),
+                ("plus_one", C.c_int), ("scale", C.c_float)]
 
 
 _native.register_optional("mb_stream_norm", [C.POINTER(_StreamNormArgs), C.c_void_p])
@@ -96,7 +103,7 @@ def stream_rms(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, r
         x1 = x if y is None else x + y.float()
         x1 = x1 if routed is None else x1 + routed.y
         if wanted:
-            out.copy_(x1 if raw else x1 * torch.rsqrt(x1.pow(2).mean(-1, keepdim=True) + pre.eps) * pre.w.float())
+            out.copy_(x1 if raw else pre.ref(x1))
         return x1, out
     a = _StreamRmsArgs()
     a.T, a.W, a.f32, a.x = T, W, _f32(fmt), _ptr(x)
@@ -113,7 +120,7 @@ def stream_rms(x: torch.Tensor, fmt: str, *, y: Optional[torch.Tensor] = None, r
         assert out.stride(1) == 1 and out.dtype == DTYPE[fmt]
         a.out_mode, a.out, a.out_ld = (2 if raw else 1), _ptr(out), out.stride(0)
         if pre is not None:
-            a.w, a.eps = _ptr(pre.w), pre.eps
+            a.w, a.eps, a.plus_one, a.scale = _ptr(pre.w), pre.eps, int(pre.plus_one), pre.scale
     _native.check(_native.lib().mb_stream_rms(C.byref(a), _stream()), f"stream_rms[T={T} W={W}]")
     _count()
     return x1, out
@@ -433,7 +440,7 @@ class _SimtAttnArgs(C.Structure):
                 ("dv", C.c_int), ("dkp", C.c_int), ("dvp", C.c_int), ("block_size", C.c_int), ("num_blocks", C.c_longlong),
                 ("scale", C.c_float), ("out_scale", C.c_float), ("sink", C.c_int), ("f32", C.c_int), ("out", C.c_void_p),
                 ("out_ld", C.c_longlong), ("status", C.c_void_p), ("sink_w", C.c_void_p), ("window", C.c_int), ("keep", C.c_int),
-                ("gate", C.c_void_p), ("gate_ld", C.c_longlong), ("gate_mode", C.c_int)]
+                ("gate", C.c_void_p), ("gate_ld", C.c_longlong), ("gate_mode", C.c_int), ("softcap", C.c_float)]
 
 
 _native.register_optional("mb_rope_dims", [C.POINTER(_RopeDimsArgs), C.c_void_p])
@@ -487,6 +494,76 @@ def rope_dims(qkv: torch.Tensor, *, Hq: int, Hkv: int, dk: int, dv: int, positio
     return q_out
 
 
+class _AttnRowsArgs(C.Structure):
+    _fields_ = [("M", C.c_int), ("Hq", C.c_int), ("Hkv", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("rot", C.c_int), ("dkp", C.c_int),
+                ("dvp", C.c_int), ("f32", C.c_int), ("y", C.c_void_p), ("ld", C.c_longlong), ("q_at", C.c_int), ("k_at", C.c_int),
+                ("v_at", C.c_int), ("positions", C.c_void_p), ("slots", C.c_void_p), ("cos_tab", C.c_void_p), ("sin_tab", C.c_void_p),
+                ("v_cos", C.c_void_p), ("v_sin", C.c_void_p), ("max_pos", C.c_int), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p),
+                ("eps", C.c_float), ("q_out", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("num_slots", C.c_longlong),
+                ("status", C.c_void_p)]
+
+
+_native.register_optional("mb_attention_rows", [C.POINTER(_AttnRowsArgs), C.c_void_p])
+_native.register_optional("mb_turn_rows", [C.c_void_p, C.c_longlong] + [C.c_int] * 4 + [C.c_void_p] * 3 + [C.c_int, C.c_void_p, C.c_void_p])
+
+
+def attention_rows(y: torch.Tensor, *, cols: Tuple[int, int, int], Hq: int, Hkv: int, dk: int, dv: int, positions, slots, k_cache, v_cache, rot,
+                   fmt: str, q_norm: Optional[RmsNorm] = None, k_norm: Optional[RmsNorm] = None, v_rot=None) -> torch.Tensor:
+    """Queries, keys and values at columns ``cols`` of y [T, *] (values may be the keys' own columns): norms over all
+    heads of the projection (weights [Hq dk] and [Hkv dk]), rotation of q and k by ``rot`` = (cos, sin) tables over their leading
+    dimensions and of v by ``v_rot`` over all of dv, k and v into caches [blocks, block, Hkv, padded]. Returns q
+    [T, Hq, padded dk]."""
+    M = y.shape[0]
+    dkp, dvp = k_cache.shape[3], v_cache.shape[3]
+    cos, sin = rot if rot is not None else (None, None)
+    if not y.is_cuda:
+        q, k, v = (y[:, at:at + n].float() for at, n in zip(cols, (Hq * dk, Hkv * dk, Hkv * dv)))
+        q = (q if q_norm is None else q_norm.ref(q)).view(M, Hq, dk)
+        k = (k if k_norm is None else k_norm.ref(k)).view(M, Hkv, dk)
+        v = v.reshape(M, Hkv, dv)
+        if cos is not None:
+            q, k = ref.apply_rope_neox(q, positions, cos, sin), ref.apply_rope_neox(k, positions, cos, sin)
+        if v_rot is not None:
+            v = ref.apply_rope_neox(v, positions, *v_rot)
+        pad = torch.nn.functional.pad
+        ok = slots >= 0
+        idx = slots[ok].long()
+        k_cache.view(-1, Hkv, dkp)[idx] = pad(k, (0, dkp - dk))[ok].to(k_cache.dtype)
+        v_cache.view(-1, Hkv, dvp)[idx] = pad(v, (0, dvp - dv))[ok].to(v_cache.dtype)
+        return pad(q, (0, dkp - dk)).to(DTYPE[fmt])
+    assert y.dtype == k_cache.dtype == v_cache.dtype == DTYPE[fmt] and y.stride(1) == 1
+    for n in (q_norm, k_norm):
+        assert n is None or not n.plus_one and n.scale == 1.0
+    assert q_norm is None or k_norm is None or q_norm.eps == k_norm.eps
+    q_out = torch.empty(M, Hq, dkp, dtype=DTYPE[fmt], device=y.device)
+    a = _AttnRowsArgs(M, Hq, Hkv, dk, dv, 2 * cos.shape[1] if cos is not None else 0, dkp, dvp, _f32(fmt), _ptr(y), y.stride(0), *cols,
+                      _ptr(positions), _ptr(slots), _ptr(cos), _ptr(sin))
+    a.max_pos = (1 << 30) if cos is None and v_rot is None else min(t.shape[0] for t in (cos, v_rot and v_rot[0]) if t is not None)
+    if v_rot is not None:
+        a.v_cos, a.v_sin = _ptr(v_rot[0]), _ptr(v_rot[1])
+    a.q_norm, a.k_norm = _ptr(q_norm.w if q_norm else None), _ptr(k_norm.w if k_norm else None)
+    a.eps = (q_norm or k_norm).eps if q_norm or k_norm else 0.0
+    a.q_out, a.k_cache, a.v_cache, a.num_slots = _ptr(q_out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0] * k_cache.shape[1]
+    a.status = _ptr(runtime(y.device).status)
+    _native.check(_native.lib().mb_attention_rows(C.byref(a), _stream()), f"attention_rows[T={M}]")
+    _count()
+    return q_out
+
+
+def turn_rows(x: torch.Tensor, H: int, dv: int, positions, rot, fmt: str) -> torch.Tensor:
+    """Every head's row of x [T, H dv] (may be a column range) turned by minus its position, in place."""
+    cos, sin = rot
+    if not x.is_cuda:
+        x.copy_(ref.apply_rope_neox(x.reshape(-1, H, dv), positions, cos, -sin).reshape(-1, H * dv))
+        return x
+    assert x.stride(1) == 1 and x.dtype == DTYPE[fmt]
+    rc = _native.lib().mb_turn_rows(_ptr(x), x.stride(0), x.shape[0], H, dv, _f32(fmt), _ptr(positions), _ptr(cos), _ptr(sin), cos.shape[0],
+                                    _ptr(runtime(x.device).status), _stream())
+    _native.check(rc, f"turn_rows[T={x.shape[0]}]")
+    _count()
+    return x
+
+
 @dataclass
 class OutputGate:
     """Sigmoid gates on an attention output: logits [T, heads] (one per head) or [T, heads * dv], may be a column range."""
@@ -504,10 +581,10 @@ class OutputGate:
 
 def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int, scale: float, sink, fmt: str,
                    out: torch.Tensor, out_scale: float = 1.0, kernel: str = "auto", window: int = 0, keep: int = 0,
-                   gate: Optional[OutputGate] = None) -> torch.Tensor:
+                   gate: Optional[OutputGate] = None, softcap: float = 0.0) -> torch.Tensor:
     """Causal paged attention of q [T, Hq, padded dk] into ``out`` [T, Hq * dv] (may be a column range), times
     ``out_scale`` and the ``gate``. ``sink``: True adds one to the softmax denominator, a tensor [Hq] (fp32) exp(sink) per
-    head. ``window`` > 0: a position sees itself, the window - 1 before it and the first ``keep``. The softmax weights keep
+    head. ``softcap`` > 0: scores become softcap tanh(score / softcap). ``window`` > 0: a position sees itself, the window - 1 before it and the first ``keep``. The softmax weights keep
     32-bit precision: they enter the product with V as two bf16 terms. ``kernel``: auto | simt | mma | tc (tests)."""
     sink_w = sink if isinstance(sink, torch.Tensor) else None
     sink = sink_w is not None or bool(sink)
@@ -526,6 +603,8 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
             k = k_cache[blocks].reshape(-1, Hkv, dkp)[:ctx, :, :dk].float().repeat_interleave(G, 1)
             v = v_cache[blocks].reshape(-1, Hkv, dvp)[:ctx, :, :dv].float().repeat_interleave(G, 1)
             sc = torch.einsum("ihd,jhd->hij", q[qs[s]:qs[s] + n, :, :dk].double(), k.double()) * scale
+            if softcap > 0:
+                sc = softcap * torch.tanh(sc / softcap)
             i = torch.arange(ctx - n, ctx)[:, None]
             j = torch.arange(ctx)[None, :]
             hide = j > i
@@ -560,6 +639,7 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
                           _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len), T, S, Hq, Hkv, dk, dv, dkp, dvp, bs, nb,
                           float(scale), float(out_scale), int(sink), _f32(fmt), _ptr(out), out.stride(0), _ptr(rt.status), _ptr(sink_w),
                           window, keep)
+        a.softcap = float(softcap)
         if gate is not None:
             gate.into(a)
         _native.check(L.mb_attn_simt(C.byref(a), _stream()), f"attn_simt[T={T}]")
@@ -573,7 +653,7 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
             batch.block_table.stride(0), S, mq
         t.Hq, t.Hkv, t.D, t.block_size, t.scale, t.v_mn = Hq, Hkv, dkp, bs, float(scale), 1
         t.out_ld, t.out_scale, t.sink, t.split_p = out.stride(0), float(out_scale), int(sink), 1
-        t.sink_w, t.window, t.keep = _ptr(sink_w), window, keep
+        t.sink_w, t.window, t.keep, t.softcap = _ptr(sink_w), window, keep, float(softcap)
         if gate is not None:
             gate.into(t)
         _native.check(L.mb_attn_prefill_tc(C.byref(t), _stream()), "attn_prefill_tc")
@@ -588,7 +668,7 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
     a.Hq, a.Hkv, a.D, a.block_size, a.num_blocks, a.scale = Hq, Hkv, dkp, bs, nb, float(scale)
     a.out, a.total_rows, a.part_tokens, a.status = _ptr(out), T, _ATTN_PART_TOKENS, _ptr(rt.status)
     a.DV, a.dv, a.out_ld, a.out_scale, a.sink, a.split_p = dvp, dv, out.stride(0), float(out_scale), int(sink), 1
-    a.sink_w, a.window, a.keep = _ptr(sink_w), window, keep
+    a.sink_w, a.window, a.keep, a.softcap = _ptr(sink_w), window, keep, float(softcap)
     if gate is not None:
         gate.into(a)
     if G * mq <= 32:

@@ -84,17 +84,17 @@ def route(logits: torch.Tensor, cfg, bias=None):
     return w.float(), idx.to(torch.int32)
 
 
-def expert_sum_ref(act, weights: torch.Tensor, idx: torch.Tensor, ge: GroupedExperts, width: int) -> torch.Tensor:
-    """CPU: sum_j weights[t, j] * expert idx[t, j] of row t over stacked (padded) gated experts; fp32 [T, width]."""
+def expert_sum_ref(act, weights: torch.Tensor, idx: torch.Tensor, ge: GroupedExperts, width: int, ffn_act: str = "swiglu") -> torch.Tensor:
+    """CPU: sum_j weights[t, j] * expert idx[t, j] of row t over stacked (padded) experts; fp32 [T, width]."""
     from . import Act, QuantWeight, linear
     out = torch.zeros(act.M, width)
     part = lambda w, e, n: QuantWeight(w.fmt, n, w.K, w.data[e * n:(e + 1) * n])
+    epi = dict(relu2=True) if ffn_act == "relu2" else dict(swiglu=ge.clamp_glu is None, clamp_glu=ge.clamp_glu)
     for e in range(ge.num):
         tok, slot = torch.nonzero(idx == e, as_tuple=True)
         if tok.numel() == 0:
             continue
-        h = linear(Act(act.fmt, tok.numel(), act.K, act.data[tok]), part(ge.gate_up, e, ge.n_gate_up), swiglu=ge.clamp_glu is None,
-                   clamp_glu=ge.clamp_glu)
+        h = linear(Act(act.fmt, tok.numel(), act.K, act.data[tok]), part(ge.gate_up, e, ge.n_gate_up), **epi)
         y = linear(Act(act.fmt, tok.numel(), h.shape[1], h.float()), part(ge.down, e, ge.n_down), out_f32=True)
         out.index_add_(0, tok, y[:, :width] * weights[tok, slot][:, None])
     return out

@@ -7,7 +7,7 @@ import ctypes as C
 
 import torch
 
-from . import Act, EPI_CLAMP_GLU, EPI_SWIGLU, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
+from . import Act, EPI_CLAMP_GLU, EPI_RELU2, EPI_SWIGLU, NATIVE_ACT_FOR_WEIGHT as ACT_FOR_WEIGHT, IN_RELU2, IN_SILU_MUL, _count, _native, _ptr, _stream, linear, row_op
 
 c = C
 ROUTER_MODE = {"softmax": 0, "softmax_grouped": 0, "sigmoid": 1, "softmax_topk": 2}
@@ -148,9 +148,11 @@ def grouped_pairs(cfg, a: Act, idx: torch.Tensor, w):
         from .mixers import gemm_simt
         sp = SortedPairs(idx, w.expert_lo, ge.num, 16 if per_expert <= 16 else 64)
         g = lambda n: (sp.tile_expert, sp.tile_row0, sp.tile_nrows, n, sp.max_tiles, sp.tile_rows)
-        assert ge.interleaved
-        epi = dict(epilogue=EPI_SWIGLU) if ge.clamp_glu is None else dict(epilogue=EPI_CLAMP_GLU, epi_a=ge.clamp_glu[0], epi_b=ge.clamp_glu[1])
-        h = torch.empty(sp.pairs, ge.n_gate_up // 2, dtype=a.data.dtype, device=a.data.device)
+        relu2 = cfg.ffn_act == "relu2"
+        assert ge.interleaved or relu2
+        epi = dict(epilogue=EPI_RELU2) if relu2 else dict(epilogue=EPI_SWIGLU) if ge.clamp_glu is None else \
+            dict(epilogue=EPI_CLAMP_GLU, epi_a=ge.clamp_glu[0], epi_b=ge.clamp_glu[1])
+        h = torch.empty(sp.pairs, ge.n_gate_up // (1 if relu2 else 2), dtype=a.data.dtype, device=a.data.device)
         gemm_simt(a.data, ge.gate_up.data, h, **epi, grouped=g(ge.n_gate_up), row_index=sp.row_pair, row_div=sp.K)
         y = torch.empty(sp.pairs, ge.n_down, dtype=torch.float32, device=h.device)
         return gemm_simt(h, ge.down.data, y, grouped=g(ge.n_down)), sp
@@ -162,7 +164,10 @@ def grouped_pairs(cfg, a: Act, idx: torch.Tensor, w):
     g = lambda n: (sp.tile_expert, sp.tile_row0, sp.tile_nrows, n, sp.max_tiles, tile_rows)
     live = sp.pair_row if nvfp4 else None       # the aligned layout is mostly padding at decode sizes: one CTA per pair
     fmt_d = ACT_FOR_WEIGHT[ge.down.fmt]
-    if cfg.ffn_act == "relu2":
+    if cfg.ffn_act == "relu2" and ge.gate_up.fmt == ge.down.fmt == "bf16":
+        act = linear(xa, ge.gate_up, relu2=True, grouped=g(ge.n_gate_up))
+        h = Act("bf16", act.shape[0], act.shape[1], act, bf16=act)
+    elif cfg.ffn_act == "relu2":
         h = row_op(linear(xa, ge.gate_up, grouped=g(ge.n_gate_up)), fmt_d, IN_RELU2, row_index=live)[0]
     elif ge.interleaved:
         act = linear(xa, ge.gate_up, swiglu=ge.clamp_glu is None, clamp_glu=ge.clamp_glu, grouped=g(ge.n_gate_up))

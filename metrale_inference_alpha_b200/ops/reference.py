@@ -226,9 +226,7 @@ def rope_inv_freq(rot: int, theta: float, scaling: Optional[dict] = None) -> Tup
         if scaling.get("truncate", True):
             low, high = math.floor(low), math.ceil(high)
         low, high = max(low, 0), min(high, rot - 1)
-        if low == high:
-            high += 0.001
-        ramp = ((torch.arange(rot // 2, dtype=torch.float64) - low) / (high - low)).clamp(0, 1)
+        ramp = ((torch.arange(rot // 2, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0, 1)
         extrap_w = 1 - ramp                                      # 1 = keep the original frequency
         return (inv / factor) * (1 - extrap_w) + inv * extrap_w, float(att)
     raise ValueError(f"unsupported rope_scaling type {kind!r}")

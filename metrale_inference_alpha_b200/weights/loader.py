@@ -310,6 +310,71 @@ class LightningW:
 
 
 @dataclass
+class DeltaW:
+    """Gated delta rule behind a short convolution."""
+    in_proj: QuantWeight = None          # everything the mixer projects; where each part's columns are is in `at`
+    at: Dict[str, tuple] = field(default_factory=dict)   # "qkv", "g", "a", "b" -> (first column, columns)
+    conv: torch.Tensor = None            # fp32 [taps, q | k | v columns]
+    A_log: torch.Tensor = None           # fp32 [heads]
+    dt_bias: torch.Tensor = None         # fp32 [heads]
+    norm: torch.Tensor = None            # bf16 [heads vdim]: the head norm's weight, repeated
+    o: QuantWeight = None
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+
+
+@dataclass
+class TwinAttnW:
+    """Attention whose queries and keys are normed over all heads; each optional: scaled rotation, rotated values, values that
+    are the keys as projected, a window, capped scores."""
+    cols: tuple = (0, 0, 0)              # first columns of q, k and v in the joint projection
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    scale: float = 1.0
+    q_norm: object = None                # ops.mixers.RmsNorm over all heads
+    k_norm: object = None
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    rot_scaling: Optional[dict] = None   # as a HF `rope_scaling`
+    turn_values: bool = False
+    window: int = 0                      # 0 = none
+    softcap: float = 0.0                 # 0 = none
+
+
+@dataclass
+class RecurrenceW:
+    """The recurrent half of a twin mixer: lightning attention, or the general delta rule."""
+    rule: str = "lightning"              # lightning | general
+    at: Dict[str, tuple] = field(default_factory=dict)   # "q", "k", "v", "g" (, "a", "w1") -> (first column, columns)
+    norm: torch.Tensor = None            # bf16 [heads vdim]
+    heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    decay: Optional[torch.Tensor] = None     # lightning: fp32 [heads]
+    w2: Optional[torch.Tensor] = None        # general: bf16 [heads dim, rank]
+    w2_twice: Optional[QuantWeight] = None   # [w2 | w2]: the operand of a two-term tanh (bf16 models)
+    w0: Optional[torch.Tensor] = None        # fp32 [heads dim]
+    decay_scale: float = 0.0                 # log decay = decay_scale * sigmoid(.)
+
+
+@dataclass
+class TwinW:
+    """Attention beside a recurrence: one input projection, one output projection over [left | right]."""
+    left: TwinAttnW = None
+    right: RecurrenceW = None
+    in_proj: QuantWeight = None
+    bias: Optional[torch.Tensor] = None  # fp32, one per row of in_proj
+    silu_cols: int = 0                   # leading columns of the projection that pass through SiLU
+    o: QuantWeight = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass
 class TokenSideW:
     gate: QuantWeight = None             # width -> dim
     proj: QuantWeight = None             # dim -> width
@@ -331,6 +396,7 @@ class LayerW:
                                                  # ops.mixers.HyperW where it does not depend on the token
     hc_ffn: Optional[object] = None              # ... and of the feed-forward block
     side: Optional[TokenSideW] = None            # per-layer token side input, after the feed-forward block
+    canon: Optional[tuple] = None                # bf16 [taps, W] filters on what the mixer and the feed-forward read
     out: Optional[QuantWeight] = None            # mixer and feed-forward side by side: both output projections, stacked along their inputs
 
 
@@ -526,6 +592,9 @@ class Loader:
         if c.arch == "finelix":
             from .finelix import load_finelix
             return load_finelix(self)
+        if c.arch == "ledinex":
+            from .ledinex import load_ledinex
+            return load_ledinex(self)
         if c.arch == "pivipel":
             from .pivipel import load_pivipel
             return load_pivipel(self)

@@ -104,8 +104,8 @@ def _seed_for(name: str, seed: int) -> int:
 
 def spec_shapes(c: ModelConfig) -> dict:
     """Tensors of a model whose sizes are per layer: name -> (shape, kind of synthetic values)."""
-    from . import fabulix, finelix, pivipel
-    return {"fabulix": fabulix, "finelix": finelix, "pivipel": pivipel}[c.arch].tensor_shapes(c)
+    from . import fabulix, finelix, ledinex, pivipel
+    return {"fabulix": fabulix, "finelix": finelix, "ledinex": ledinex, "pivipel": pivipel}[c.arch].tensor_shapes(c)
 
 
 class SyntheticSource(TensorSource):
