@@ -28,7 +28,7 @@ What is measured (all as the max over ranks; rank 0 prints ONE JSON line):
            same K steps as `value`, driven through `step()`.
   config.ladder   the same end-to-end measurement for every rung 1..128 (`--no-ladder` skips it).
 
-`--mixers` runs another workload instead: the Fabulix decoder (`--design finelix`, `--design pivipel`: that one) beside an
+`--mixers` runs another workload instead: the Fabulix decoder (`--design finelix`, `pivipel`, `ledinex`: that one) beside an
 engine model of equal size.
 """
 from __future__ import annotations
@@ -179,9 +179,9 @@ def main() -> int:
     ap.add_argument("--mixers", default="", choices=["", "all", "kernels", "models"],
                     help="instead of the headline run: the Fabulix decoder's kernels beside the like kernels of an equal-size "
                          "attention / Kimi-delta hybrid, and both models' prefill and decode throughput (1 GPU; benchmarks/mixer_bench.py)")
-    ap.add_argument("--design", default="fabulix", choices=["fabulix", "finelix", "pivipel"],
+    ap.add_argument("--design", default="fabulix", choices=["fabulix", "finelix", "pivipel", "ledinex"],
                     help="--mixers: the decoder that is measured (finelix: beside an MLA / Kimi-delta hybrid with experts; pivipel: beside "
-                         "a windowed, gated-attention model with experts)")
+                         "a windowed, gated-attention model with experts; ledinex: beside a gated-delta-net / attention hybrid with experts)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

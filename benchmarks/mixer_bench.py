@@ -1,5 +1,5 @@
 #!/usr/bin/env python
-"""The kernels of the Fabulix, Finelix or Pivipel decoder next to the like kernels of the engine's attention / MLA /
+"""The kernels of the Fabulix, Finelix, Pivipel or Ledinex decoder next to the like kernels of the engine's attention / MLA /
 Kimi-delta-attention / Mamba2 hybrids and of its gated-attention MoE models at equal size, each with its distance from the roofline (measured copy
 bandwidth and measured bf16 GEMM rate), and the throughput of a whole model next to an equal-size hybrid. CUDA
 events around one call, L2 flushed by a 512 MB write before every call, median of the timed calls. Reached as
@@ -349,6 +349,140 @@ def pivipel_kernels(W=2560, H=32, G=8, D=128, FF=6912, E=64, top=6, EF=1024, S=2
     return rows
 
 
+def ledinex_kernels(W=2560, H=32, G=8, D=128, FF=6912, E=64, top=6, EF=1024, SF=2048, HR=20, window=512, rank=64, taps=3, conv=4):
+    """The same rows for Ledinex: the like kernels are those of attention / gated-delta-net / Kimi-delta models with experts."""
+    from metrale_inference_alpha_b200.ops import canon, delta as dl, moe as moe_ops, moe_cuda
+    from metrale_inference_alpha_b200.weights.loader import MoeW
+    rows = []
+    HD, RD, pair, f32 = H * D, HR * D, pairing(rows), torch.float32
+    for shape, lens, start in SHAPES:
+        b, nblk = batch(lens, start)
+        T, S, ctx = sum(lens), len(lens), lens[0] + start
+        # ---- the stream
+        x, y, xb, wv = rnd(T, W, dtype=f32), rnd(T, W), rnd(T, W), rnd(W)
+        nm, filt = mx.RmsNorm(wv, 1e-6, plus_one=True), rnd(taps, W)
+        win = canon.Window(torch.zeros(S + 2, (taps - 1) * W, device=DEV), 0, W)
+        kw = dict(norm=nm, filt=filt, window=win, batch=b)
+        one, wb = mx.SublayerOut(y), 2 * S * (taps - 1) * W * 4
+        pair(shape, "stream_canon (norm + add + convolution)", lambda: canon.stream_canon(x, "bf16", pending=one, **kw), T * W * 12 + wb, 0,
+             "residual + RMSNorm", lambda: ops.row_op(xb, "bf16", ops.IN_RMSNORM, w=wv, residual=y, write_residual=True), T * W * 8, 0)
+        # ---- experts
+        up, gu = QuantWeight("bf16", E * EF, W, rnd(E * EF, W, std=0.02)), QuantWeight("bf16", E * 2 * EF, W, rnd(E * 2 * EF, W, std=0.02))
+        dn = QuantWeight("bf16", E * W, EF, rnd(E * W, EF, std=0.02))
+        soft, spec = moe_ops.RouterSpec(E, top, "softmax"), moe_ops.RouterSpec(E, top, "softmax", ffn_act="relu2")
+        w = MoeW(grouped=moe_ops.GroupedExperts(up, dn, E, EF, W, False), spec=spec)
+        lw = MoeW(grouped=moe_ops.GroupedExperts(gu, dn, E, 2 * EF, W, True), spec=soft)
+        act, logits = mx.act_of(rnd(T, W), "bf16"), rnd(T, E, dtype=f32)
+        wt, idx = moe_ops.route(logits, soft)
+        hit = len(set(idx.flatten().tolist()))
+        eb = lambda n: hit * n * EF * W * 2 + T * W * 2 + T * top * (W * 4 + 2 * EF * 2)
+        pair(shape, "experts (squared ReLU), unsummed", lambda: moe_cuda.grouped_pairs(spec, act, idx, w), eb(2), T * top * 4 * EF * W, "experts (SwiGLU)",
+             lambda: moe_cuda.grouped_pairs(soft, act, idx, lw), eb(3), T * top * 6 * EF * W)
+        ye, sp = moe_cuda.grouped_pairs(spec, act, idx, w)
+        full = mx.SublayerOut(y, None, mx.Routed(ye, sp.pair_row, wt))
+
+        def combine():
+            out = torch.empty(T, W, dtype=BF, device=DEV)
+            ops._native.lib().mb_moe_finish(ops._ptr(ye), ye.stride(0), ops._ptr(sp.pair_row), ops._ptr(wt), T, top, W, ops._ptr(y), W, None, 0,
+                                            ops._ptr(xb), ops._ptr(out), ops._stream())
+        pair(shape, "stream_canon with shared expert and experts' sum", lambda: canon.stream_canon(x, "bf16", pending=full, **kw),
+             T * W * (12 + 4 * top) + wb, 0, "expert combine (shared)", combine, T * W * (6 + 4 * top), 0)
+        del gu, dn, w, lw, ye, sp, full, up
+        su = QuantWeight("bf16", SF, W, rnd(SF, W, std=0.02))
+        gb, gf = (SF * W + T * W + T * SF) * 2, 2 * T * SF * W
+        pair(shape, "GEMM + squared ReLU", lambda: ops.linear(act, su, relu2=True), gb, gf, "GEMM", lambda: ops.linear(act, su), gb, gf)
+        N = (H + G) * D + 5 * RD + rank
+        wi, bias = QuantWeight("bf16", N, W, rnd(N, W, std=0.02)), rnd(N, dtype=f32)
+        gb, gf = (N * W + T * W + T * N) * 2, 2 * T * N * W
+        pair(shape, "twin projection GEMM + bias", lambda: ops.linear(act, wi, bias=bias), gb, gf, "GEMM", lambda: ops.linear(act, wi), gb, gf)
+        # ---- attention
+        cos, sin = ref.rope_tables(8192, D, 1e4, device=DEV)
+        kc, vc = rnd(nblk, 16, G, D), rnd(nblk, 16, G, D)
+        qkv, hn = rnd(T, (H + 2 * G) * D), rnd(D)
+        pos = dict(Hq=H, Hkv=G, positions=b.positions, slots=b.slot_mapping, k_cache=kc, v_cache=vc)
+        qn, kn = mx.RmsNorm(rnd(HD), 1e-6), mx.RmsNorm(rnd(G * D), 1e-6)
+        like = lambda: ops.qk_norm_rope_kvwrite(qkv, D=D, cos=cos, sin=sin, q_norm_w=hn, k_norm_w=hn, **pos)
+        byt, cols = 2 * qkv.numel() * 2, (0, HD, HD + G * D)
+        pair(shape, "attention_rows (norms over all heads, rotated values)",
+             lambda: mx.attention_rows(qkv, cols=cols, dk=D, dv=D, rot=(cos, sin), fmt="bf16", q_norm=qn, k_norm=kn, v_rot=(cos, sin), **pos), byt, 0,
+             "head norms + rope + KV write", like, byt, 0)
+        pair(shape, "attention_rows (values are the keys)",
+             lambda: mx.attention_rows(qkv, cols=(0, HD, HD), dk=D, dv=D, rot=(cos, sin), fmt="bf16", q_norm=qn, k_norm=kn, **pos), byt - T * G * D * 2, 0,
+             "head norms + rope + KV write", like, byt, 0)
+        q, cat = rnd(T, H, D), torch.empty(T, HD + RD, dtype=BF, device=DEV)
+        o2, turn = cat[:, :HD], (cos, sin)
+        flo = sum(4 * HD * (n * start + n * (n + 1) / 2) for n in lens)
+        byt = S * ctx * G * D * 4 + T * HD * 4
+        att = lambda win_: (lambda: ops.paged_attention(q, kc, vc, b.block_table, b.q_start, b.q_len, b.ctx_len, max_q_len=b.max_q_len, max_ctx=b.max_ctx,
+                                                        scale=0.09, window=win_))
+        new = lambda win_, cap, turn_: (lambda: mx.attention_dims(q, kc, vc, b, dk=D, dv=D, scale=0.09, sink=False, fmt="bf16", out=o2, out_scale=0.7,
+                                                                  window=win_, softcap=cap, turn_back=turn_))
+        pair(shape, "capped attention, output turned back", new(0, 30.0, turn), byt, flo, "attention", att(0), byt, flo)
+        seen = sum(min(window, p + 1) for n in lens for p in range(start, start + n))
+        byt = sum(min(ctx, n + window) for n in lens) * G * D * 4 + T * HD * 4
+        pair(shape, "windowed attention", new(window, 0.0, None), byt, 4 * HD * seen, "windowed attention (other models)", att(window), byt, 4 * HD * seen)
+        del q, qkv
+        # ---- recurrences
+        C3, sb = 3 * RD, 2 * S * HR * D * D * 4
+        px, fl = rnd(T, C3 + RD + 64), rnd(conv, C3, dtype=f32)
+        wn = canon.Window(torch.zeros(S + 2, (conv - 1) * C3, device=DEV), 0, C3)
+        cst, cwt = torch.zeros(S + 2, C3, conv - 1, device=DEV), fl.t().contiguous()
+        pair(shape, "short_conv", lambda: canon.short_conv(px[:, :C3], fl, wn, b, "bf16"), T * C3 * 4 + 2 * S * C3 * (conv - 1) * 4, 0, "causal_conv1d",
+             lambda: rops.causal_conv1d(px, C3, cwt, None, cst, b), T * C3 * 6 + 2 * S * C3 * (conv - 1) * 4, 0)
+        ssm = torch.zeros(S + 2, HR, D, D, device=DEV)
+        cv, cf = rnd(T, C3), rnd(T, C3, dtype=f32)
+        q, k, v = cv[:, :RD], cv[:, RD:2 * RD], cv[:, 2 * RD:]
+        A, dtb, ba = torch.zeros(HR, device=DEV), torch.zeros(HR, device=DEV), rnd(T, 2 * HR, dtype=f32)
+        gate, nw, ab = px[:, C3:C3 + RD], rnd(RD), px[:, C3 + RD:]
+        rule = dl.GatedRule(ab[:, :HR], ab[:, 32:32 + HR], A, dtb)
+        nrm = dict(w=nw, gate=gate, gate_act="silu", eps=1e-6, scale=1.0, out=torch.empty(T, RD, dtype=BF, device=DEV))
+        gdn = lambda: ops.row_op(rops.gdn_recurrence(cf, ba, A, dtb, ssm, b, k_heads=HR, v_heads=HR, k_dim=D, v_dim=D), "bf16", ops.IN_GATED_RMSNORM,
+                                 gate=gate, w=nw, group=D)
+        hk = dict(heads=HR, dk=D, dv=D, fmt="bf16")
+        pair(shape, "gated delta rule (recurrence, norm)", lambda: dl.delta_attention(q, k, v, rule, ssm, b, norm=nrm, **hk), T * RD * 10 + sb, 0,
+             "gated delta net (recurrence, norm)", gdn, T * RD * 16 + sb, 0)
+        rw2 = rnd(RD, rank, std=0.1)
+        z, tw = rnd(T, rank), QuantWeight("bf16", RD, 2 * rank, torch.cat([rw2, rw2], 1).contiguous())
+        bd = dl.BoundedDecay(z, rw2, rnd(RD, dtype=f32), -0.6065, tw)
+        lin, za = QuantWeight("bf16", RD, rank, rw2), mx.act_of(z, "bf16")
+        pair(shape, "log decay (bounded, 32-bit low-rank)", bd.log, T * (rank * 2 + RD * 4), 2 * T * rank * RD, "low-rank decay GEMM, bf16",
+             lambda: ops.linear(za, lin, out_f32=True), T * (rank * 2 + RD * 4), 2 * T * rank * RD)
+        aa = rnd(T, RD)
+        gen = dl.GeneralRule(aa, bd)
+        nrm2 = dict(nrm, gate_act="sigmoid")
+        graw, braw, ng, dt2 = rnd(T, RD, dtype=f32), rnd(T, HR, dtype=f32), torch.ones(D, device=DEV), torch.zeros(RD, device=DEV)
+        kda = lambda: rops.kda_recurrence(cf, graw, braw, A, dt2, -5.0, ssm, b, heads=HR, dim=D, norm=(ng, gate, 1e-6))
+        pair(shape, "general delta rule (decay, recurrence, norm)", lambda: dl.delta_attention(q, k, v, gen, ssm, b, norm=nrm2, **hk), T * RD * 12 + sb, 0,
+             "Kimi delta attention (recurrence, norm)", kda, T * RD * 20 + sb, 0)
+        dec = torch.linspace(0.6, 0.999, HR, device=DEV)
+
+        def light():
+            core = mx.linear_attention(q, k, v, ssm, b, decay=dec, **hk)
+            mx.gated_norm(core, nw, gate, "bf16", group=RD, gate_act="sigmoid", eps=1e-6, out=nrm["out"])
+        pair(shape, "lightning attention (recurrence, norm)", light, T * RD * 10 + sb, 0, "gated delta net (recurrence, norm)", gdn, T * RD * 16 + sb, 0)
+        del cv, cf, px, graw, q, k, v
+    return rows
+
+
+def ledinex_models():
+    """(label, name -> configuration): Ledinex and a hybrid of equal size: attention where Ledinex runs two mixers side by
+    side, gated delta net where it runs the gated delta rule, SwiGLU experts with as many rows; bf16."""
+    from metrale_inference_alpha_b200.config.model_config import ModelConfig, preset
+    for label, kw in (("1B-like layers", dict(width=2048, heads=16, kv_heads=4, right_heads=16, delta_heads=16, delta_kv_heads=16, experts=32, top=4,
+                                              expert_ff=768, shared_ff=1536, vocab=32768)),
+                      ("3B-like layers", {})):
+        p = preset("ledinex-3b", num_layers=6, window=512, **kw)
+        m, d, mlp = p.layer_specs[1]["mixer"]["left"], p.layer_specs[0]["mixer"], p.layer_specs[1]["mlp"]
+        h = ModelConfig(name="gdn-attention-moe", arch="qwen_hybrid", vocab_size=p.vocab_size, hidden_size=p.hidden_size, num_layers=6,
+                        num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"], rotary_dim=m["dim"], qk_norm=True, attn_output_gate=True,
+                        norm_plus_one=True, layer_types=["gdn" if t == "delta" else "attention" for t in p.layer_types], ffn_types=list(p.ffn_types),
+                        gdn_k_heads=d["kv_heads"], gdn_v_heads=d["heads"], gdn_k_dim=d["dim"], gdn_v_dim=d["vdim"], conv_kernel=d["conv"],
+                        num_experts=mlp["router"]["experts"], experts_per_token=mlp["router"]["top"], moe_intermediate_size=mlp["expert"]["ff"],
+                        intermediate_size=mlp["expert"]["ff"], num_shared_experts=mlp["shared"]["ff"] // mlp["expert"]["ff"], shared_expert_gate=True,
+                        router="softmax", tie_embeddings=True, weight_format="bf16", kv_dtype="bf16", max_position=16384)
+        yield label, {"ledinex": p, "gated-delta-net / attention MoE": h}
+
+
 def pivipel_models():
     """(label, name -> configuration): Pivipel and a model of equal size with the same experts, windows, head norms and
     output gates on one bf16 residual; bf16."""
@@ -442,10 +576,10 @@ def throughput(cfg, decode_batches=(1, 32, 128), prefills=((1, 4096), (8, 1024))
 def run(what="all", design="fabulix"):
     res = {"design": design}
     if what in ("all", "kernels"):
-        res["kernels"] = {"fabulix": kernels, "finelix": finelix_kernels, "pivipel": pivipel_kernels}[design]()
+        res["kernels"] = {"fabulix": kernels, "finelix": finelix_kernels, "pivipel": pivipel_kernels, "ledinex": ledinex_kernels}[design]()
     if what in ("all", "models"):
         res["models"] = {}
-        for label, cfgs in {"fabulix": models, "finelix": finelix_models, "pivipel": pivipel_models}[design]():
+        for label, cfgs in {"fabulix": models, "finelix": finelix_models, "pivipel": pivipel_models, "ledinex": ledinex_models}[design]():
             res["models"][label] = {}
             for name, cfg in cfgs.items():
                 res["models"][label][name] = throughput(cfg)

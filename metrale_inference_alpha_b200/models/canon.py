@@ -65,9 +65,7 @@ def twin_attention(dec, y, w, batch, kc, vc, fmt: str, out, out_scale: float) ->
     q = mx.attention_rows(y, cols=w.cols, Hq=w.heads, Hkv=w.kv_heads, dk=w.dim, dv=w.vdim, positions=batch.positions, slots=batch.slot_mapping,
                           k_cache=kc, v_cache=vc, rot=rot if rot[0] is not None else None, fmt=fmt, q_norm=w.q_norm, k_norm=w.k_norm, v_rot=turn)
     mx.attention_dims(q, kc, vc, batch, dk=w.dim, dv=w.vdim, scale=w.scale, sink=False, fmt=fmt, out=out, out_scale=out_scale,
-                      window=w.window, softcap=w.softcap)
-    if turn is not None:
-        mx.turn_rows(out, w.heads, w.vdim, batch.positions, turn, fmt)
+                      window=w.window, softcap=w.softcap, turn_back=turn)
 
 
 def twin_mixer(dec, a, lw, batch, kc, vc, state, fmt: str, stash):

@@ -56,6 +56,7 @@ class AttnTcArgs(C.Structure):
         ("block_size", c_int), ("cache_fp8", c_int), ("scale", c_float), ("v_mn", c_int),
         ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
         ("sink_w", c_void_p), ("window", c_int), ("keep", c_int), ("gate", c_void_p), ("gate_ld", c_ll), ("gate_mode", c_int), ("softcap", c_float),
+        ("turn_cos", c_void_p), ("turn_sin", c_void_p), ("turn_max", c_int),
     ]
 
 
@@ -97,6 +98,7 @@ class AttnArgs(C.Structure):
         ("outq", c_void_p), ("ldq", c_int), ("outq_sf", c_void_p), ("outq_sf_k64", c_int), ("outq_gs", c_float),
         ("DV", c_int), ("dv", c_int), ("out_ld", c_ll), ("out_scale", c_float), ("sink", c_int), ("split_p", c_int),
         ("sink_w", c_void_p), ("keep", c_int), ("gate", c_void_p), ("gate_ld", c_ll), ("gate_mode", c_int), ("softcap", c_float),
+        ("turn_cos", c_void_p), ("turn_sin", c_void_p), ("turn_max", c_int),
     ]
 
 

@@ -49,13 +49,16 @@ class _StreamCanonArgs(C.Structure):
 
 
 class _ShortConvArgs(C.Structure):
-    _fields_ = [("C", C.c_int), ("taps", C.c_int), ("f32", C.c_int), ("silu", C.c_int), ("write_out", C.c_int), ("x", C.c_void_p),
+    _fields_ = [("C", C.c_int), ("taps", C.c_int), ("f32", C.c_int), ("write_out", C.c_int), ("x", C.c_void_p),
                 ("x_ld", C.c_longlong), ("filt", C.c_void_p), ("out", C.c_void_p), ("win", _WindowArgs)]
 
 
 _native.register_optional("mb_stream_canon", [C.POINTER(_StreamCanonArgs), C.c_void_p])
 _native.register_optional("mb_canon_commit", [C.c_void_p, C.c_int, C.c_int, C.POINTER(_WindowArgs), C.c_void_p])
 _native.register_optional("mb_short_conv", [C.POINTER(_ShortConvArgs), C.c_void_p])
+
+
+_LONG_PORTION = 96               # portions this long take the join and the convolution as two launches
 
 
 def _sequences(batch):
@@ -111,7 +114,7 @@ def stream_canon(x: torch.Tensor, fmt: str, *, pending: Optional[SublayerOut] = 
     if x1 is None and h is None:
         return x, None
     _native.check(_native.lib().mb_stream_canon(C.byref(a), _stream()), f"stream_canon[T={T} W={W}]")
-    _count()
+    _count(2 if filt is not None and int(batch.max_q_len) >= _LONG_PORTION else 1)
     return (x if x1 is None else x1), h
 
 
@@ -127,7 +130,7 @@ def canon_commit(x: torch.Tensor, taps: int, window: Window, batch) -> None:
     _count()
 
 
-def short_conv(x: torch.Tensor, filt: torch.Tensor, window: Window, batch, fmt: str, *, silu: bool = True, write_state: bool = True,
+def short_conv(x: torch.Tensor, filt: torch.Tensor, window: Window, batch, fmt: str, *, write_state: bool = True,
                write_out: bool = True) -> Optional[torch.Tensor]:
     """Causal convolution of x's columns [T, C] (a column range, activation type) with ``filt`` [taps, C] fp32, through
     SiLU; the window advanced. ``write_out`` off: only that."""
@@ -135,10 +138,10 @@ def short_conv(x: torch.Tensor, filt: torch.Tensor, window: Window, batch, fmt: 
     taps = filt.shape[0]
     if not x.is_cuda:
         y = _convolve_ref(x.float(), filt, window.view(taps), batch, write_state)
-        return (torch.nn.functional.silu(y) if silu else y).to(DTYPE[fmt]) if write_out else None
+        return torch.nn.functional.silu(y).to(DTYPE[fmt]) if write_out else None
     assert x.stride(1) == 1 and x.dtype == DTYPE[fmt] and filt.dtype == torch.float32 and window.width == Cn
     out = torch.empty(T, Cn, dtype=x.dtype, device=x.device) if write_out else None
-    a = _ShortConvArgs(Cn, taps, _f32(fmt), int(silu), int(write_out), _ptr(x), x.stride(0), _ptr(filt), _ptr(out), window.args(batch, write_state))
+    a = _ShortConvArgs(Cn, taps, _f32(fmt), int(write_out), _ptr(x), x.stride(0), _ptr(filt), _ptr(out), window.args(batch, write_state))
     _native.check(_native.lib().mb_short_conv(C.byref(a), _stream()), f"short_conv[T={T} C={Cn}]")
     _count()
     return out

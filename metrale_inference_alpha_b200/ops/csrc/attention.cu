@@ -262,6 +262,7 @@ struct AttnParams {
   int keep;                 // with a window: the first tokens that every query sees
   mb::OutputGate<__nv_bfloat16> gate;
   mb::SoftCap softcap;      // bf16 caches
+  mb::TurnBack turn;        // bf16 caches, no gates
   int split_p;              // the weights enter the product with V as two bf16 terms (16 mantissa bits)
 };
 
@@ -854,21 +855,20 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
       }
     }
   __syncthreads();
-  for (int idx = tid; idx < R * (DV / 4); idx += 128) {
-    const int r = idx / (DV / 4), c4 = idx - r * (DV / 4);
+  // four columns of a row, summed over the warps; also the row's maximum and sum
+  auto merge_warps = [&](int r, int c4, float& mx, float& l) {
     float mw[4], lw[4];
-    float mx = -INFINITY;
+    mx = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       mw[w] = s_ml[(w * MT * 16 + r) * 2];
       lw[w] = s_ml[(w * MT * 16 + r) * 2 + 1];
       mx = fmaxf(mx, mw[w]);
     }
-    const int tq = r / G, hh = r - tq * G;
     const bool sink_here = p.sink && nparts == 1;
-    const float sk = sink_here ? sink_log2(p, kvh * G + hh) : 0.f;
+    const float sk = sink_here ? sink_log2(p, kvh * G + r % G) : 0.f;
     if (sink_here) mx = fmaxf(mx, sk);
-    float l = sink_here ? exp2f(sk - mx) : 0.f;
+    l = sink_here ? exp2f(sk - mx) : 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
@@ -879,8 +879,25 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
     }
     const float inv = l > 0.f ? vmul / l : 0.f;
     acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
-    const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
-    if (nparts == 1) {
+    return acc;
+  };
+  // both groups of four columns that a turn brings together
+  auto store_turned = [&](size_t orow, int pos, int c4, float4 a, float4 b) {
+    float u[4] = {a.x, a.y, a.z, a.w}, v[4] = {b.x, b.y, b.z, b.w};
+    p.turn.operator()<4>(pos, c4 * 4, u, v);
+    store_out4<DV>(p, orow, c4, u[0], u[1], u[2], u[3]);
+    store_out4<DV>(p, orow, c4 + p.dv / 8, v[0], v[1], v[2], v[3]);
+  };
+  const bool turn = p.turn.cos_tab != nullptr;
+  const int per1 = turn && nparts == 1 ? p.dv / 8 : DV / 4;
+  for (int idx = tid; idx < R * per1; idx += 128) {
+    const int r = idx / per1, c4 = idx - r * per1, tq = r / G;
+    float mx, l;
+    const float4 acc = merge_warps(r, c4, mx, l);
+    const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + r - tq * G;
+    if (turn && nparts == 1) {
+      store_turned(orow, ctx - qlen + tq, c4, acc, merge_warps(r, c4 + p.dv / 8, mx, l));
+    } else if (nparts == 1) {
       store_out4<DV>(p, orow, c4, acc.x, acc.y, acc.z, acc.w);
     } else {
       *reinterpret_cast<float4*>(p.part_o + (orow * p.parts + part) * DV + c4 * 4) = acc;
@@ -904,10 +921,7 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  for (int idx = tid; idx < R * (DV / 4); idx += 128) {
-    const int r = idx / (DV / 4), c4 = idx - r * (DV / 4);
-    const int tq = r / G, hh = r - tq * G;
-    const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
+  auto merge_parts = [&](size_t orow, int hh, int c4) {
     float mx = -INFINITY;
     for (int s2 = 0; s2 < nparts; ++s2) mx = fmaxf(mx, __ldcg(&p.part_ml[(orow * p.parts + s2) * 2]));
     const float sk = p.sink ? sink_log2(p, kvh * G + hh) : 0.f;
@@ -924,7 +938,15 @@ __global__ void __launch_bounds__(128, (DK <= 128 && DV <= 128 && MT == 1) ? 4 :
       acc.x += ov.x * wgt; acc.y += ov.y * wgt; acc.z += ov.z * wgt; acc.w += ov.w * wgt;
     }
     const float inv = denom > 0.f ? 1.f / denom : 0.f;
-    store_out4<DV>(p, orow, c4, acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
+    return make_float4(acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
+  };
+  const int per = turn ? p.dv / 8 : DV / 4;
+  for (int idx = tid; idx < R * per; idx += 128) {
+    const int r = idx / per, c4 = idx - r * per, tq = r / G, hh = r - tq * G;
+    const size_t orow = (size_t)(qs + tq) * p.Hq + kvh * G + hh;
+    const float4 a = merge_parts(orow, hh, c4);
+    if (turn) store_turned(orow, ctx - qlen + tq, c4, a, merge_parts(orow, hh, c4 + p.dv / 8));
+    else store_out4<DV>(p, orow, c4, a.x, a.y, a.z, a.w);
   }
 }
 
@@ -1110,6 +1132,10 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const AttnParams p) {
     if (p.sink) l += exp2f(sink_log2(p, head) - m_run[hr]);
     const float inv = (l > 0.f ? vmul / l : 0.f) * p.out_scale * (p.gate.mode == mb::GATE_HEAD ? p.gate(qs + qr, head, 0) : 1.f);
     __nv_bfloat16* dst = p.out + (size_t)(qs + qr) * p.out_ld + (size_t)head * p.dv + (lane & 3) * 2;
+    if (p.turn.cos_tab) {                                      // dv == DV: both halves of a pair are this thread's
+#pragma unroll
+      for (int n = 0; n < DV / 16; ++n) p.turn.operator()<2>(past + qr, n * 8 + (lane & 3) * 2, &o_acc[n][hr * 2], &o_acc[n + DV / 16][hr * 2]);
+    }
     if (p.gate.mode == mb::GATE_ELEMENT) {
 #pragma unroll
       for (int n = 0; n < DV / 8; ++n)
@@ -1271,6 +1297,9 @@ struct MbAttnArgs {
   long long gate_ld;
   int gate_mode;           // 1 one per head, 2 one per element
   float softcap;           // 0: off; scores become softcap tanh(score / softcap)
+  const float* turn_cos;   // [turn_max, dv / 2] or null: every output row is turned back by its position
+  const float* turn_sin;
+  int turn_max;
 };
 
 // most entries of the visible-token list of a sequence: its context, or the kept first tokens and the windows of its
@@ -1310,6 +1339,8 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
   p.sink_w = a->sink_w; p.keep = a->window > 0 ? a->keep : 0;
   p.gate = {reinterpret_cast<const __nv_bfloat16*>(a->gate), a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, p.dv};
   p.softcap = mb::SoftCap::make(a->scale, a->softcap);
+  p.turn = mb::TurnBack{a->turn_cos, a->turn_sin, p.dv / 2, a->turn_max};
+  if (a->turn_cos && (!a->turn_sin || a->turn_max <= 0 || a->gate || p.dv % 8 || a->cache_fp8 || a->outq)) return MB_ERR_UNSUPPORTED;
   if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
   if (p.dv > DV || p.out_ld < (long long)a->Hq * p.dv) return MB_ERR_BAD_ARG;
   if (p.dv == DV && (p.out_ld % 2 || (reinterpret_cast<uintptr_t>(a->out) & 3))) return MB_ERR_BAD_ARG;   // paired stores
@@ -1355,6 +1386,7 @@ int mb_paged_attention(const MbAttnArgs* a, cudaStream_t stream) {
     return rc;                    // partitions are merged inside the kernel by the last arriver
   }
   p.parts = 1;
+  if (a->turn_cos && p.dv != DV) return MB_ERR_UNSUPPORTED;
   if (a->D == 128 && DV == 128) return fp8 ? launch_prefill<128, 128, true>(p, a->num_seqs, a->max_q_len, stream)
                                            : launch_prefill<128, 128, false>(p, a->num_seqs, a->max_q_len, stream);
   if (a->D == 64 && DV == 64) return fp8 ? launch_prefill<64, 64, true>(p, a->num_seqs, a->max_q_len, stream)

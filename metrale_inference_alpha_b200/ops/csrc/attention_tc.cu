@@ -60,6 +60,7 @@ struct TcParams {
   int window, keep;
   mb::OutputGate<__nv_bfloat16> gate;
   mb::SoftCap softcap;           // bf16 caches
+  mb::TurnBack turn;             // bf16 caches, no gates
   uint32_t* status;
 };
 
@@ -346,6 +347,27 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
     const size_t row = (size_t)qs + (row_ok ? qi : 0);
     const float inv = (l_run > 0.f ? vmul / l_run : 0.f) * p.out_scale * (p.gate.mode == mb::GATE_HEAD ? p.gate(row, head, 0) : 1.f);
     uint4* dst = reinterpret_cast<uint4*>(p.out + (size_t)(qs + (row_ok ? qi : 0)) * p.out_ld + (size_t)head * kD);
+    auto store16 = [&](int c, const float* ov) {
+#pragma unroll
+      for (int h2 = 0; h2 < 2; ++h2) {
+        uint4 w;
+        __nv_bfloat162* wb = reinterpret_cast<__nv_bfloat162*>(&w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) wb[i] = __floats2bfloat162_rn(ov[h2 * 8 + 2 * i] * inv, ov[h2 * 8 + 2 * i + 1] * inv);
+        if (row_ok) dst[c * 2 + h2] = w;
+      }
+    };
+    if (!FP8 && p.turn.cos_tab) {                         // columns and their partners half a head on
+#pragma unroll 2
+      for (int c = 0; c < kD / 32; ++c) {
+        float u[16], v[16];
+        mb::tmem_ld16(t_row + 64 + c * 16, u);
+        mb::tmem_ld16(t_row + 64 + kD / 2 + c * 16, v);
+        p.turn.operator()<16>(row_ok ? ctx - qlen + qi : 0, c * 16, u, v);
+        store16(c, u);
+        store16(c + kD / 32, v);
+      }
+    } else
 #pragma unroll
     for (int c = 0; c < kD / 16; ++c) {
       float ov[16];
@@ -364,14 +386,7 @@ __global__ void __launch_bounds__(128, kD == 128 ? 2 : 1) attn_prefill_tc_kernel
           }
         }
       }
-#pragma unroll
-      for (int h2 = 0; h2 < 2; ++h2) {
-        uint4 w;
-        __nv_bfloat162* wb = reinterpret_cast<__nv_bfloat162*>(&w);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) wb[i] = __floats2bfloat162_rn(ov[h2 * 8 + 2 * i] * inv, ov[h2 * 8 + 2 * i + 1] * inv);
-        if (row_ok) dst[c * 2 + h2] = w;
-      }
+      store16(c, ov);
     }
   }
   mb::tc_fence_before();
@@ -418,6 +433,9 @@ struct MbAttnTcArgs {
   long long gate_ld;
   int gate_mode;       // 1 one per head, 2 one per element
   float softcap;       // 0: off
+  const float* turn_cos;   // [turn_max, D / 2] or null: every output row is turned back by its position
+  const float* turn_sin;
+  int turn_max;
 };
 
 // Causal paged attention for prefill chunks (head dim 128). Returns 0, MB_ERR_* or a CUDA error.
@@ -437,7 +455,9 @@ extern "C" int mb_attn_prefill_tc(const MbAttnTcArgs* a, cudaStream_t stream) {
   p.sink = a->sink; p.sink_w = a->sink_w;
   p.window = a->window; p.keep = a->window > 0 ? a->keep : 0;
   p.softcap = mb::SoftCap::make(a->scale, a->softcap);
-  if (a->softcap > 0.f && a->cache_fp8) return MB_ERR_UNSUPPORTED;
+  p.turn = mb::TurnBack{a->turn_cos, a->turn_sin, a->D / 2, a->turn_max};
+  if ((a->softcap > 0.f || a->turn_cos) && a->cache_fp8) return MB_ERR_UNSUPPORTED;
+  if (a->turn_cos && (!a->turn_sin || a->turn_max <= 0 || a->gate)) return MB_ERR_UNSUPPORTED;
   p.gate = {(const __nv_bfloat16*)a->gate, a->gate_ld, a->gate ? a->gate_mode : mb::GATE_NONE, a->D};
   if (p.keep < 0 || (a->gate && a->gate_mode != mb::GATE_HEAD && a->gate_mode != mb::GATE_ELEMENT)) return MB_ERR_BAD_ARG;
   if (p.gate.mode == mb::GATE_ELEMENT && (a->gate_ld % 8 || (reinterpret_cast<uintptr_t>(a->gate) & 15))) return MB_ERR_UNSUPPORTED;

@@ -5,13 +5,14 @@
 //                  through its RMS norm, x' = x + rms(y) w (or 1 + w), and the next sublayer's input is
 //                  h_t = x'_t + sum_j f_j x'_(t - taps + 1 + j), zero in front of the sequence. Without a filter only x'.
 //   canon_commit   state := the last taps - 1 rows of (state | x' of the accepted rows), after speculative verification
-//   short_conv     the same convolution of a projection's columns, through SiLU on request, without the residual
+//   short_conv     the same convolution of a projection's columns, through SiLU instead of the residual
 //
 // A CTA of stream_canon owns up to kRun consecutive tokens of one sequence. It recomputes x' of the taps - 1 rows in front
 // of them, so that no row waits for another CTA; rows in front of the portion come from the carried window. The CTA of a
 // portion's first rows is the only reader of the window, and it alone writes the new one (recomputing the portion's last
 // rows where they are not its own). All rows of a CTA live in shared memory: their sums of squares are taken by whole
 // warps side by side, then every thread walks its own channels over the rows.
+// Long portions take two launches instead, a join of whole rows and the convolution below over x'.
 // short_conv follows the same rule with runs of tokens per thread. Windows are rows of a slot pool, win_ld floats from slot
 // to slot, oldest row first.
 #include "epilogue.cuh"
@@ -21,6 +22,7 @@ namespace {
 
 constexpr int kRun = 8;            // tokens of a run, at most
 constexpr int kMaxRows = 40;       // rows of a CTA: the run and the window
+constexpr int kLongPortion = 96;   // portions this long take the join and the convolution as two launches
 
 struct Window {
   float* base;                     // [slots, win_ld]: taps - 1 rows
@@ -201,19 +203,71 @@ __global__ void __launch_bounds__(256) canon_commit_kernel(const float* x, int W
     }
 }
 
-// ------------------------------------------------------------------ columns of a projection
+// Long portions: x' alone, a CTA per row with the row in registers; the convolution then reads x' from L2.
+template <int VEC, int NIT, typename T>
+__global__ void __launch_bounds__(256) stream_join_kernel(const CanonParams p) {
+  __shared__ float red[32];
+  __shared__ int s_row[32];
+  __shared__ float s_w[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, W = p.W;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  if (p.ye) {
+    if (tid < p.K) {
+      s_row[tid] = p.pair_row[(size_t)t * p.K + tid];
+      s_w[tid] = p.pair_w[(size_t)t * p.K + tid];
+    }
+    __syncthreads();
+  }
+  float v[NIT][VEC], x[NIT][VEC], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NIT; ++i) {
+    const int k = (i * nt + tid) * VEC;
+    if (k >= W) continue;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[i][e] = 0.f;
+    if (p.y) ldn<VEC>(reinterpret_cast<const T*>(p.y) + (size_t)t * W + k, v[i]);
+    ldn<VEC>(p.x + (size_t)t * W + k, x[i]);
+    if (p.ye) {
+      for (int j = 0; j < p.K; ++j) {
+        if (s_row[j] < 0) continue;
+        float a[VEC];
+        ldn<VEC>(p.ye + (size_t)s_row[j] * p.ye_ld + k, a);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[i][e] = fmaf(s_w[j], a[e], v[i][e]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[i][e], v[i][e], ss);
+  }
+  const float inv = 1.f / sqrtf(mb::block_sum(ss, red) / (float)W + p.eps);
+#pragma unroll
+  for (int i = 0; i < NIT; ++i) {
+    const int k = (i * nt + tid) * VEC;
+    if (k >= W) continue;
+    float w[VEC];
+    ldn<VEC>(p.norm_w + k, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[i][e] = fmaf(v[i][e] * inv, p.plus + w[e], x[i][e]);
+    stn<VEC>(p.x_out + (size_t)t * W + k, x[i]);
+  }
+}
+
+// ------------------------------------------------------------------ columns of a matrix
 constexpr int kConvRun = 16;       // tokens of a thread
 
 struct ShortConvParams {
-  int C, taps, silu, write_out;
+  int C, taps, write_out;
   const void* x;
   long long x_ld;
-  const float* filt;               // [taps, C]
+  const void* filt;                // [taps, C]
   void* out;                       // [T, C]
   Window win;                      // rows of C floats
 };
 
-template <int VEC, typename T>
+// TI, TF, TO: inputs, filter, output. TAPS > 0: that many, kept in registers; 0: any number, inputs read again. SILU: through
+// SiLU, else the convolution is added to its input.
+template <int VEC, int TAPS, bool SILU, typename TI, typename TF, typename TO>
 __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p) {
   const int c = (blockIdx.x * 128 + threadIdx.x) * VEC, seq = blockIdx.z, l0 = blockIdx.y * kConvRun;
   mb::pdl_wait();
@@ -227,7 +281,8 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
   }
   float* st = p.win.base + (size_t)slot * p.win.ld + c;
   const bool fresh = p.win.positions[q0] == 0;
-  const T* x = reinterpret_cast<const T*>(p.x) + (size_t)q0 * p.x_ld + c;
+  const TI* x = reinterpret_cast<const TI*>(p.x) + (size_t)q0 * p.x_ld + c;
+  const TF* filt = reinterpret_cast<const TF*>(p.filt) + c;
   auto input = [&](int l, float* v) {
     if (l >= 0) {
       ldn<VEC>(x + (size_t)l * p.x_ld, v);
@@ -238,24 +293,56 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
       for (int i = 0; i < VEC; ++i) v[i] = 0.f;
     }
   };
+  auto emit = [&](int l, const float* conv, const float* in) {
+    float a[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) a[i] = !SILU ? conv[i] + in[i] : sizeof(TO) == 2 ? mb::silu(conv[i]) : mb::silu_exact(conv[i]);
+    stn<VEC>(reinterpret_cast<TO*>(p.out) + (size_t)(q0 + l) * p.C + c, a);
+  };
   if (p.write_out) {
     const int l1 = min(n, l0 + kConvRun);
-    for (int l = l0; l < l1; ++l) {
-      float a[VEC];
+    if constexpr (TAPS > 0) {
+      float f[TAPS][VEC], w[TAPS][VEC];
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) a[i] = 0.f;
-      for (int j = 0; j < p.taps; ++j) {
-        float v[VEC], f[VEC];
-        input(l - halo + j, v);
-        ldn<VEC>(p.filt + (size_t)j * p.C + c, f);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) a[i] = fmaf(f[i], v[i], a[i]);
+      for (int j = 0; j < TAPS; ++j) {
+        ldn<VEC>(filt + (size_t)j * p.C, f[j]);
+        if (j + 1 < TAPS) input(l0 - TAPS + 1 + j, w[j]);
       }
-      if (p.silu) {
+      // four tokens' inputs are on their way at a time
+      for (int lb = l0; lb < l1; lb += 4) {
+        float nx[4][VEC];
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) a[i] = mb::silu_exact(a[i]);
+        for (int u = 0; u < 4; ++u)
+          if (lb + u < l1) ldn<VEC>(x + (size_t)(lb + u) * p.x_ld, nx[u]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          if (lb + u >= l1) break;
+          float a[VEC];
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) {
+            w[TAPS - 1][i] = nx[u][i];
+            a[i] = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) a[i] = fmaf(f[j][i], w[j][i], a[i]);
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) w[j][i] = w[j + 1][i];
+          }
+          emit(lb + u, a, nx[u]);
+        }
       }
-      stn<VEC>(reinterpret_cast<T*>(p.out) + (size_t)(q0 + l) * p.C + c, a);
+    } else {
+      for (int l = l0; l < l1; ++l) {
+        float a[VEC], v[VEC], f[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) a[i] = 0.f;
+        for (int j = 0; j < p.taps; ++j) {                 // ends with the token's own input in v
+          input(l - halo + j, v);
+          ldn<VEC>(filt + (size_t)j * p.C, f);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) a[i] = fmaf(f[i], v[i], a[i]);
+        }
+        emit(l, a, v);
+      }
     }
   }
   if (l0 != 0 || !p.win.write) return;                   // the first run alone reads the window, and writes the new one
@@ -263,6 +350,19 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
     float v[VEC];
     input(n - halo + r, v);
     stn<VEC>(st + (size_t)r * p.C, v);
+  }
+}
+
+template <int VEC, bool SILU, typename TI, typename TF, typename TO>
+int launch_conv(const ShortConvParams& p, int max_q_len, int num_seqs, cudaStream_t stream) {
+  const int runs = p.write_out ? (max_q_len + kConvRun - 1) / kConvRun : 1;
+  if (runs > 65535) return MB_ERR_TOO_LARGE;
+  const dim3 g((p.C + 128 * VEC - 1) / (128 * VEC), runs, num_seqs), b(128);
+  switch (p.taps) {
+    case 2: return (int)mb::launch_kernel(short_conv_kernel<VEC, 2, SILU, TI, TF, TO>, g, b, 0, stream, p);
+    case 3: return (int)mb::launch_kernel(short_conv_kernel<VEC, 3, SILU, TI, TF, TO>, g, b, 0, stream, p);
+    case 4: return (int)mb::launch_kernel(short_conv_kernel<VEC, 4, SILU, TI, TF, TO>, g, b, 0, stream, p);
+    default: return (int)mb::launch_kernel(short_conv_kernel<VEC, 0, SILU, TI, TF, TO>, g, b, 0, stream, p);
   }
 }
 
@@ -296,7 +396,7 @@ struct MbStreamCanonArgs {
 };
 
 struct MbShortConvArgs {
-  int C, taps, f32, silu, write_out;
+  int C, taps, f32, write_out;
   const void* x;
   long long x_ld;
   const float* filt;
@@ -324,6 +424,22 @@ int launch_canon(const CanonParams& p, dim3 grid, int threads, size_t smem, cuda
   }
   return (int)mb::launch_kernel(kern, grid, dim3(threads), smem, stream, p);
 }
+
+template <typename T>
+int join_rows(const CanonParams& p, bool v4, int nit, int threads, cudaStream_t stream) {
+  const dim3 g(p.T), b(threads);
+  if (p.K > 32) return MB_ERR_TOO_LARGE;
+#define MB_JOIN(V, N) return (int)mb::launch_kernel(stream_join_kernel<V, N, T>, g, b, 0, stream, p)
+  if (v4) {
+    if (nit <= 1) MB_JOIN(4, 1);
+    if (nit <= 3) MB_JOIN(4, 3);
+    if (nit <= 8) MB_JOIN(4, 8);
+    MB_JOIN(4, 16);
+  }
+  if (nit <= 4) MB_JOIN(1, 4);
+  MB_JOIN(1, 16);
+#undef MB_JOIN
+}
 }  // namespace
 
 extern "C" {
@@ -348,6 +464,20 @@ int mb_stream_canon(const MbStreamCanonArgs* a, cudaStream_t stream) {
                       a->plus_one ? 1.f : 0.f, a->eps, a->x_out, (const bf16*)a->filt, a->out, window_of(a->win)};
   const bool v4 = a->W % 4 == 0 && a->ye_ld % 4 == 0 && a->win.ld % 4 == 0 && al(a->x, 16) && al(a->y, 16) && al(a->ye, 16) && al(a->norm_w, 8) &&
                   al(a->x_out, 16) && al(a->filt, 8) && al(a->out, 16) && al(a->win.base, 16);
+  // long portions: the join by itself, then the convolution over x' (nothing is recomputed, and rows need no shared memory)
+  if (a->filt && halo <= kConvRun && longest >= kLongPortion) {
+    const int vec = v4 ? 4 : 1, nt = row_threads(a->W, vec), nit = (a->W + nt * vec - 1) / (nt * vec);
+    if (nit <= 16) {
+      if (a->norm_w) {
+        const int rc = a->f32 ? join_rows<float>(p, v4, nit, nt, stream) : join_rows<bf16>(p, v4, nit, nt, stream);
+        if (rc != 0) return rc;
+      }
+      const ShortConvParams c{a->W, a->taps, 1, a->norm_w ? a->x_out : a->x, a->W, a->filt, a->out, p.win};
+      const int S = a->win.num_seqs;
+      if (a->f32) return v4 ? launch_conv<4, false, float, bf16, float>(c, longest, S, stream) : launch_conv<1, false, float, bf16, float>(c, longest, S, stream);
+      return v4 ? launch_conv<4, false, float, bf16, bf16>(c, longest, S, stream) : launch_conv<1, false, float, bf16, bf16>(c, longest, S, stream);
+    }
+  }
   const int threads = a->W >= 1024 ? 512 : 256;
   const dim3 grid((longest + run - 1) / run, a->filt ? a->win.num_seqs : 1);
   if (a->f32) return v4 ? launch_canon<4, float>(p, grid, threads, smem, stream) : launch_canon<1, float>(p, grid, threads, smem, stream);
@@ -365,14 +495,12 @@ int mb_canon_commit(const float* x, int W, int taps, const MbWindowArgs* w, cuda
 int mb_short_conv(const MbShortConvArgs* a, cudaStream_t stream) {
   if (!a || a->C <= 0 || !a->x || !a->filt || (a->write_out && !a->out) || !window_ok(a->win, a->taps, a->C)) return MB_ERR_BAD_ARG;
   if (a->taps - 1 > kConvRun) return MB_ERR_TOO_LARGE;
-  const ShortConvParams p{a->C, a->taps, a->silu, a->write_out, a->x, a->x_ld, a->filt, a->out, window_of(a->win)};
+  const ShortConvParams p{a->C, a->taps, a->write_out, a->x, a->x_ld, a->filt, a->out, window_of(a->win)};
   const size_t es = a->f32 ? 16 : 8;
   const bool v4 = a->C % 4 == 0 && a->x_ld % 4 == 0 && a->win.ld % 4 == 0 && al(a->x, es) && al(a->filt, 16) && al(a->out, es) && al(a->win.base, 16);
-  const int vec = v4 ? 4 : 1, runs = a->write_out ? (a->win.max_q_len + kConvRun - 1) / kConvRun : 1;
-  if (runs > 65535) return MB_ERR_TOO_LARGE;
-  const dim3 g((a->C + 128 * vec - 1) / (128 * vec), runs, a->win.num_seqs), b(128);
-  if (a->f32) return (int)(v4 ? mb::launch_kernel(short_conv_kernel<4, float>, g, b, 0, stream, p) : mb::launch_kernel(short_conv_kernel<1, float>, g, b, 0, stream, p));
-  return (int)(v4 ? mb::launch_kernel(short_conv_kernel<4, bf16>, g, b, 0, stream, p) : mb::launch_kernel(short_conv_kernel<1, bf16>, g, b, 0, stream, p));
+  const int mq = a->win.max_q_len, S = a->win.num_seqs;
+  if (a->f32) return v4 ? launch_conv<4, true, float, float, float>(p, mq, S, stream) : launch_conv<1, true, float, float, float>(p, mq, S, stream);
+  return v4 ? launch_conv<4, true, bf16, float, bf16>(p, mq, S, stream) : launch_conv<1, true, bf16, float, bf16>(p, mq, S, stream);
 }
 
 }  // extern "C"

@@ -49,7 +49,7 @@ struct DeltaParams {
 
 constexpr int kTB = 16;            // tokens per buffer
 constexpr int kNW = 4;             // compute warps
-constexpr int kPW = 4;             // producer warps
+constexpr int kPW = 8;             // producer warps
 
 using f2 = unsigned long long;     // two packed fp32
 __device__ __forceinline__ f2 pk(float a, float b) {
@@ -103,49 +103,77 @@ __global__ void __launch_bounds__(32 * (kNW + kPW)) delta_attn_kernel(const Delt
   const DeltaInputs& in = p.in;
   const int DK = in.DK, DV = in.DV, col0 = blockIdx.x * VB;
 
+  // two tokens per producer warp and tile; everything they read is on its way before the first reduction
+  const float neg_a = GENERAL ? 0.f : -expf(in.A_log[hd]), dtb = GENERAL ? 0.f : in.dt_bias[hd];
   auto produce = [&](int tile, int pw) {
+    constexpr int kE = (DKP + 31) / 32, kV = (VB + 31) / 32, kN = kTB / kPW;
     const int buf = tile & 1, cnt = min(kTB, n - tile * kTB);
-    for (int tt = pw; tt < cnt; tt += kPW) {
-      const size_t t = (size_t)(t0 + tile * kTB + tt);
-      const int at = (buf * kTB + tt) * DKP;
-      constexpr int kE = (DKP + 31) / 32;
-      float q[kE], k[kE], sq = 0.f, sk = 0.f;
+    float q[kN][kE], k[kN][kE], w[kN][kE], a[kN][kE], v[kN][kV], ga[kN], gb[kN];
+#pragma unroll
+    for (int i = 0; i < kN; ++i) {
+      const int tt = pw + i * kPW;
+      const bool ok = tt < cnt;
+      const size_t t = (size_t)(t0 + tile * kTB + (ok ? tt : 0));
 #pragma unroll
       for (int j = 0; j < kE; ++j) {
         const int d = lane + 32 * j;
-        q[j] = d < DK ? in.query<T>(t, hd, d) : 0.f;
-        k[j] = d < DK ? in.key<T>(t, hd, d) : 0.f;
-        sq = fmaf(q[j], q[j], sq);
-        sk = fmaf(k[j], k[j], sk);
+        const bool in_row = ok && d < DK;
+        q[i][j] = in_row ? in.query<T>(t, hd, d) : 0.f;
+        k[i][j] = in_row ? in.key<T>(t, hd, d) : 0.f;
+        if constexpr (GENERAL) {
+          w[i][j] = in_row ? in.log_w[(t * in.H + hd) * DK + d] : 0.f;
+          a[i][j] = in_row ? mb::load1<T>(in.removal, t * in.removal_ld + (size_t)hd * DK + d) : 0.f;
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kV; ++j) {
+        const int c = lane + 32 * j;
+        v[i][j] = ok && c < VB && col0 + c < DV ? in.value<T>(t, hd, col0 + c) : 0.f;
+      }
+      if constexpr (!GENERAL) {
+        ga[i] = mb::load1<T>(in.decay, t * in.gate_ld + hd);
+        gb[i] = mb::load1<T>(in.step, t * in.gate_ld + hd);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kN; ++i) {
+      const int tt = pw + i * kPW;
+      if (tt >= cnt) break;
+      const int at = (buf * kTB + tt) * DKP;
+      float sq = 0.f, sk = 0.f;
+#pragma unroll
+      for (int j = 0; j < kE; ++j) {
+        sq = fmaf(q[i][j], q[i][j], sq);
+        sk = fmaf(k[i][j], k[i][j], sk);
       }
       sk = mb::warp_sum(sk);
-      if constexpr (GENERAL) {
+      float nq = 1.f, nk = 1.f;
+      if constexpr (!GENERAL) {
+        nq = rsqrtf(mb::warp_sum(sq) + mb::kUnitEps) * rsqrtf((float)DK);
+        nk = rsqrtf(sk + mb::kUnitEps);
+      }
 #pragma unroll
-        for (int j = 0; j < kE; ++j) {
-          const int d = lane + 32 * j;
-          if (d >= DKP) continue;
-          sQ[at + d] = q[j];
-          sK[at + d] = k[j];
-          sW[at + d] = d < DK ? expf(in.log_w[(t * in.H + hd) * DK + d]) : 0.f;
-          sA[at + d] = d < DK ? -in.rate<T>(t, hd, d) * k[j] : 0.f;
-        }
-        if (lane == 0) sS[(buf * kTB + tt) * 4] = 1.f / (sk + mb::kUnitEps);
-      } else {
-        sq = mb::warp_sum(sq);
-        const float nq = rsqrtf(sq + mb::kUnitEps) * rsqrtf((float)DK), nk = rsqrtf(sk + mb::kUnitEps);
-#pragma unroll
-        for (int j = 0; j < kE; ++j) {
-          const int d = lane + 32 * j;
-          if (d >= DKP) continue;
-          sQ[at + d] = q[j] * nq;
-          sK[at + d] = k[j] * nk;
-        }
-        if (lane == 0) {
-          sS[(buf * kTB + tt) * 4] = expf(in.log_gate<T>(t, hd));
-          sS[(buf * kTB + tt) * 4 + 1] = in.step_size<T>(t, hd);
+      for (int j = 0; j < kE; ++j) {
+        const int d = lane + 32 * j;
+        if (d >= DKP) continue;
+        sQ[at + d] = q[i][j] * nq;
+        sK[at + d] = k[i][j] * nk;
+        if constexpr (GENERAL) {
+          sW[at + d] = expf(w[i][j]);
+          sA[at + d] = -mb::sigmoid_exact(a[i][j]) * k[i][j];
         }
       }
-      for (int c = lane; c < VB; c += 32) sV[(buf * kTB + tt) * VB + c] = col0 + c < DV ? in.value<T>(t, hd, col0 + c) : 0.f;
+      if (lane == 0) {
+        if constexpr (GENERAL) {
+          sS[(buf * kTB + tt) * 4] = 1.f / (sk + mb::kUnitEps);
+        } else {
+          sS[(buf * kTB + tt) * 4] = expf(neg_a * mb::softplus(ga[i] + dtb));
+          sS[(buf * kTB + tt) * 4 + 1] = mb::sigmoid_exact(gb[i]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kV; ++j)
+        if (lane + 32 * j < VB) sV[(buf * kTB + tt) * VB + lane + 32 * j] = v[i][j];
     }
   };
 
@@ -336,8 +364,20 @@ __global__ void __launch_bounds__(256, 2) delta_decode_kernel(const DeltaParams 
       if (p.lr_z) {
         const bf16* w2 = p.lr_w2 + ch * p.lr_rank;
         float z = p.lr_bias[ch];
-#pragma unroll 4
-        for (int r = 0; r < p.lr_rank; ++r) z = fmaf(sz[r], __bfloat162float(w2[r]), z);
+        int r = 0;
+        if ((p.lr_rank & 7) == 0 && (reinterpret_cast<uintptr_t>(p.lr_w2) & 15) == 0) {      // rows of whole 16-byte vectors
+#pragma unroll 8
+          for (; r < p.lr_rank; r += 8) {
+            const uint4 w8 = __ldg(reinterpret_cast<const uint4*>(w2 + r));
+            const __nv_bfloat162* wb = reinterpret_cast<const __nv_bfloat162*>(&w8);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 f = __bfloat1622float2(wb[i]);
+              z = fmaf(sz[r + 2 * i], f.x, fmaf(sz[r + 2 * i + 1], f.y, z));
+            }
+          }
+        }
+        for (; r < p.lr_rank; ++r) z = fmaf(sz[r], __bfloat162float(w2[r]), z);
         lw = p.lr_c * mb::sigmoid_exact(z);
       } else {
         lw = in.log_w[t * in.H * DK + ch];

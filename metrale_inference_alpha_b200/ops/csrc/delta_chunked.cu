@@ -1,0 +1,802 @@
+// Chunked prefill of the delta rules of delta_attn.cu, 64 tokens per chunk, all large products on the tensor cores
+// (mma.sync m16n8k16, fp32 accumulation).
+//
+// Over a chunk with start state S0, the rows X_j that the rule adds to the state (besides k v^T in the general rule) solve
+// a unit lower-triangular system, so with M = (I + A)^-1
+//     X = Xw S0 + Xu        o = R' S0 + O'        S' = diag(d) S0 + T S0 + E
+// and everything but S0 is known without the state:
+//   general  (L the running sums of log2 decays per key channel, L_-1 = 0; d = 2^L_last)
+//     U_i = u_i 2^L_(i-1)   R_i = r_i 2^L_i   B_j = a_j u_j 2^-L_j   K_j = k_j 2^-L_j
+//     A = tril(U B^T, -1)   Xw = -M U   Xu = -M tril(U K^T, -1) V
+//     Q = tril(R B^T)       R' = R + Q Xw   O' = tril(R K^T) V + Q Xu
+//     T = diag(d) B^T Xw    E = diag(d) (K^T V + B^T Xu)
+//     The decays are bounded below (at most 100 octaves in a chunk), so no factor overflows.
+//   gated    (G the running sums of one log2 decay per token; d = 2^G_last)
+//     A_ij = beta_i 2^(G_i - G_j) k_i.k_j (j < i)   Xw = -M diag(beta 2^G) K   Xu = M diag(beta) V
+//     Q_ij = 2^(G_i - G_j) q_i.k_j (j <= i)         R' = diag(2^G) q + Q Xw    O' = Q Xu
+//     T = (2^(G_last - G) k)^T Xw                   E = (2^(G_last - G) k)^T Xu
+//     Every exponent is <= 0 however strong the decay.
+// Three launches for the whole ragged batch:
+//   delta_prep  per (chunk, head, sequence): all of the above into a workspace
+//   delta_scan  per (32 value columns, head, sequence): the recurrence over chunks, S in registers; leaves every chunk's
+//               start state as two bf16 planes (value and remainder), the final state in the pool
+//   delta_out   per (chunk, head, sequence): o, optionally finished by the head's gated RMS norm
+// Values are exact bf16 operands; every other one is 32-bit and enters as value + remainder (16 mantissa bits), so a product
+// costs two or three passes and keeps 32-bit quantities 32-bit to a few 1e-6. The triangular inverse is fp32, by 16 x 16
+// blocks. Head sizes 64 and 128. Sequence s keeps its chunks from index q_start[s] / 64 + s on, which never overlaps.
+#include "common.cuh"
+#include "delta_attn.cuh"
+#include "epilogue.cuh"
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+using mb::DeltaInputs;
+constexpr int kC = 64;
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct ChunkParams {
+  DeltaInputs in;
+  float* state;                // [slots, H, DK, DV]
+  float* out;                  // [T, H DV], or null with a norm
+  bf16* ws_t;                  // [chunks, H, 2 planes, DK, DK]
+  float* ws_e;                 // [chunks, H, DK, DV]
+  bf16* ws_s;                  // [chunks, H, 2 planes, DK, DV] start states
+  bf16* ws_r;                  // [chunks, H, 2 planes, 64, DK]
+  float* ws_o;                 // [chunks, H, 64, DV]
+  float* ws_d;                 // [chunks, H, DK]
+  const int* q_start;
+  const int* q_len;
+  const int* positions;
+  const int* slots;
+  int num_slots, write_state;
+  uint32_t* status;
+  const bf16* norm_w;          // [H DV] or null
+  const bf16* gate;
+  long long gate_ld;
+  int sigmoid_gate;
+  float eps, scale;
+  bf16* norm_out;
+  long long norm_out_ld;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(mb::smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(mb::smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void cp16(void* dst, const void* src, bool ok) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mb::smem_u32(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+// (a, b) -> packed bf16 pair, and the packed pair of what rounding took off
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+// two planes of a matrix in shared or global memory, ld elements per row
+struct Planes {
+  bf16* hi;
+  bf16* lo;
+  int ld;
+  __device__ __forceinline__ void put(int r, int c, float a, float b) const {
+    uint32_t h, l;
+    split2(a, b, h, l);
+    *reinterpret_cast<uint32_t*>(hi + (size_t)r * ld + c) = h;
+    *reinterpret_cast<uint32_t*>(lo + (size_t)r * ld + c) = l;
+  }
+  __device__ __forceinline__ float2 get(int r, int c) const {
+    const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(hi + (size_t)r * ld + c));
+    const float2 l = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(lo + (size_t)r * ld + c));
+    return make_float2(h.x + l.x, h.y + l.y);
+  }
+};
+
+// acc (16 rows m0 .., 8 N8 columns n0 ..) += A B over k in [k0, k1): A is [row][k], or [k][row] with AT; B is [k][column],
+// exact (one plane) without BL
+template <int N8, bool AT, bool BL>
+__device__ __forceinline__ void mm(float (*acc)[4], const Planes& A, int m0, const Planes& B, int n0, int k0, int k1) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll 2
+  for (int k = k0; k < k1; k += 16) {
+    uint32_t ah[4], al[4];
+    if constexpr (AT) {
+      const size_t o = (size_t)(k + (lane >> 4) * 8 + (lane & 7)) * A.ld + m0 + ((lane >> 3) & 1) * 8;
+      ldsm4t(ah, A.hi + o);
+      ldsm4t(al, A.lo + o);
+    } else {
+      const size_t o = (size_t)(m0 + (lane & 15)) * A.ld + k + (lane >> 4) * 8;
+      ldsm4(ah, A.hi + o);
+      ldsm4(al, A.lo + o);
+    }
+#pragma unroll
+    for (int i = 0; i < N8; i += 2) {
+      uint32_t b[4];
+      const size_t o = (size_t)(k + (lane & 15)) * B.ld + n0 + i * 8 + (lane >> 4) * 8;
+      ldsm4t(b, B.hi + o);
+      mma(acc[i], ah, b[0], b[1]);
+      mma(acc[i + 1], ah, b[2], b[3]);
+      mma(acc[i], al, b[0], b[1]);
+      mma(acc[i + 1], al, b[2], b[3]);
+      if constexpr (BL) {
+        ldsm4t(b, B.lo + o);
+        mma(acc[i], ah, b[0], b[1]);
+        mma(acc[i + 1], ah, b[2], b[3]);
+      }
+    }
+  }
+}
+template <int N8>
+__device__ __forceinline__ void zero(float (*acc)[4]) {
+#pragma unroll
+  for (int i = 0; i < N8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+}
+// the accumulators (times f) into planes
+template <int N8>
+__device__ __forceinline__ void put_acc(const Planes& P, int m0, int n0, const float (*acc)[4], float f) {
+  const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+#pragma unroll
+  for (int i = 0; i < N8; ++i) {
+    P.put(m0 + g, n0 + i * 8 + 2 * t, acc[i][0] * f, acc[i][1] * f);
+    P.put(m0 + g + 8, n0 + i * 8 + 2 * t, acc[i][2] * f, acc[i][3] * f);
+  }
+}
+
+// ------------------------------------------------------------------ per-chunk preparation
+constexpr int kLdF = kC + 4;       // fp32 rows of the inverse
+constexpr int kLdC = kC + 8;       // bf16 rows of 64 x 64 matrices
+
+template <int DK, int DV>
+struct PrepLayout {
+  static constexpr int ldk = DK + 8, ldv = DV + 8, ldx = (DK > DV ? DK : DV) + 8;
+  static constexpr size_t plane_k = (size_t)kC * ldk * 2, plane_x = (size_t)kC * ldx * 2;
+  static constexpr size_t u = 0, r = 2 * plane_k, b = 4 * plane_k, k = 6 * plane_k, v = k + 2 * plane_x, z0 = v + (size_t)kC * ldv * 2;
+  static constexpr size_t zsize = 2 * (size_t)kC * kLdC * 2;                   // two planes of a 64 x 64 matrix, or one in fp32
+  static constexpr size_t z1 = z0 + zsize, tmp = z1 + zsize, vec = tmp + 3 * 16 * 17 * 4, bytes = vec + (DK + 4 * kC) * 4;
+  static_assert(2 * zsize >= (size_t)kC * (DK + 4) * 4, "the running logs live where the 64 x 64 matrices come later");
+  static_assert(zsize >= (size_t)kC * kLdF * 4, "");
+};
+
+template <int DK, int DV, bool GEN>
+__global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p) {
+  using Lay = PrepLayout<DK, DV>;
+  extern __shared__ __align__(16) uint8_t sm[];
+  const DeltaInputs& in = p.in;
+  const int c = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const int n = p.q_len[seq];
+  if (c * kC >= n) return;
+  const int t0 = p.q_start[seq] + c * kC, valid = min(kC, n - c * kC), H = in.H;
+  const size_t ci = ((size_t)(p.q_start[seq] / kC + seq + c)) * H + hd;
+  auto planes = [&](size_t at, int ld) { return Planes{reinterpret_cast<bf16*>(sm + at), reinterpret_cast<bf16*>(sm + at) + kC * ld, ld}; };
+  const Planes U = planes(Lay::u, Lay::ldk), R = planes(Lay::r, Lay::ldk), B = planes(Lay::b, Lay::ldk), K = planes(Lay::k, Lay::ldx);
+  const Planes V{reinterpret_cast<bf16*>(sm + Lay::v), nullptr, Lay::ldv};
+  const Planes Z0 = planes(Lay::z0, kLdC), Z1 = planes(Lay::z1, kLdC);
+  float* sA = reinterpret_cast<float*>(sm + Lay::z0);                         // [64][kLdF]
+  float* sM = reinterpret_cast<float*>(sm + Lay::z1);
+  float* sT = reinterpret_cast<float*>(sm + Lay::tmp);
+  float* sD = reinterpret_cast<float*>(sm + Lay::vec);                         // decay of the whole chunk, [DK]
+  float* sG = sD + DK;                                                         // gated: running log2 decays, step sizes
+  float* sBeta = sG + kC;
+  float* sL = sA;                                                              // general: running logs [64][DK + 4]
+  constexpr int ldl = DK + 4;
+
+  // values, exact
+  for (int i = tid; i < kC * (DV / 8); i += 256) {
+    const int r = i / (DV / 8), cc = (i - r * (DV / 8)) * 8;
+    const bool ok = r < valid;
+    cp16(V.hi + r * Lay::ldv + cc, reinterpret_cast<const bf16*>(in.v) + (ok ? (size_t)(t0 + r) * in.v_ld + (size_t)hd * DV + cc : 0), ok);
+  }
+  cp_commit();
+  if constexpr (GEN) {
+    // running sums of log2 decays; rows past `valid` repeat the last
+    constexpr int kR = kC * DK / 256;
+    const int d = tid % DK, grp = tid / DK, r0 = grp * kR;
+    const float* lw = in.log_w + ((size_t)t0 * H + hd) * DK + d;
+    float v[kR];
+#pragma unroll
+    for (int i = 0; i < kR; ++i) v[i] = r0 + i < valid ? lw[(size_t)(r0 + i) * H * DK] * kLog2e : 0.f;
+#pragma unroll
+    for (int i = 1; i < kR; ++i) v[i] += v[i - 1];
+    sL[(r0 + kR - 1) * ldl + d] = v[kR - 1];
+    __syncthreads();
+    float before = 0.f;
+    for (int i = 0; i < grp; ++i) before += sL[(i * kR + kR - 1) * ldl + d];
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kR; ++i) sL[(r0 + i) * ldl + d] = before + v[i];
+    __syncthreads();
+    if (tid < DK) {
+      sD[tid] = ex2(sL[(kC - 1) * ldl + tid]);
+      p.ws_d[ci * DK + tid] = sD[tid];
+    }
+  } else {
+    if (tid < kC) {
+      float lg = 0.f, beta = 0.f;
+      if (tid < valid) {
+        lg = in.log_gate<bf16>(t0 + tid, hd) * kLog2e;
+        beta = in.step_size<bf16>(t0 + tid, hd);
+      }
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, lg, o);
+        if (lane >= o) lg += up;
+      }
+      sG[tid] = lg;
+      sBeta[tid] = beta;
+    }
+    __syncthreads();
+    if (tid >= 32 && tid < kC) sG[tid] += sG[31];
+    __syncthreads();
+    if (tid < DK) p.ws_d[ci * DK + tid] = ex2(sG[kC - 1]);
+  }
+  // ---- operands, a warp per row
+  {
+    constexpr int E = DK / 32;
+    const int d0 = lane * E, hk = hd / (H / in.HK);
+    auto load = [&](const void* base, long long ld, int head, int row, float* o) {
+      const bf16* src = reinterpret_cast<const bf16*>(base) + (size_t)(t0 + row) * ld + (size_t)head * DK + d0;
+      if constexpr (E == 4) {
+        const uint2 w = *reinterpret_cast<const uint2*>(src);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.y));
+        o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+      } else {
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
+        o[0] = a.x; o[1] = a.y;
+      }
+    };
+#pragma unroll 2
+    for (int i = warp; i < kC; i += 8) {
+      float q[E], k[E], a[E];
+#pragma unroll
+      for (int e = 0; e < E; ++e) q[e] = k[e] = a[e] = 0.f;
+      if (i < valid) {
+        load(in.q, in.q_ld, hk, i, q);
+        load(in.k, in.k_ld, hk, i, k);
+        if constexpr (GEN) load(in.removal, in.removal_ld, hd, i, a);
+      }
+      float sq = 0.f, sk = 0.f;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        sq = fmaf(q[e], q[e], sq);
+        sk = fmaf(k[e], k[e], sk);
+      }
+      const float nk = rsqrtf(mb::warp_sum(sk) + mb::kUnitEps);
+      if constexpr (GEN) {
+        float u[E], rr[E], bb[E], kk[E];
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+          const float l = sL[i * ldl + d0 + e], l1 = i > 0 ? sL[(i - 1) * ldl + d0 + e] : 0.f, up = ex2(-l), un = k[e] * nk;
+          u[e] = un * ex2(l1);
+          rr[e] = q[e] * ex2(l);
+          bb[e] = mb::sigmoid_fast(a[e]) * un * up;
+          kk[e] = k[e] * up;
+        }
+#pragma unroll
+        for (int e = 0; e < E; e += 2) {
+          U.put(i, d0 + e, u[e], u[e + 1]);
+          R.put(i, d0 + e, rr[e], rr[e + 1]);
+          B.put(i, d0 + e, bb[e], bb[e + 1]);
+          K.put(i, d0 + e, kk[e], kk[e + 1]);
+        }
+      } else {
+        const float nq = rsqrtf(mb::warp_sum(sq) + mb::kUnitEps) * rsqrtf((float)DK);
+#pragma unroll
+        for (int e = 0; e < E; e += 2) {
+          U.put(i, d0 + e, k[e] * nk, k[e + 1] * nk);
+          R.put(i, d0 + e, q[e] * nq, q[e + 1] * nq);
+        }
+      }
+    }
+  }
+  __syncthreads();
+  // ---- scores of this warp's 16 rows and 32 columns, blocks up to the diagonal: rows U and R against columns B (and K)
+  const int rb = warp & 3, half = warp >> 2, i0 = rb * 16, j0 = half * 32;
+  float sa[4][4], sb[GEN ? 4 : 1][4], sp[GEN ? 4 : 1][4], sq[4][4];
+  zero<4>(sa);
+  zero<4>(sq);
+  if constexpr (GEN) {
+    zero<4>(sb);
+    zero<4>(sp);
+  }
+  const Planes& CB = GEN ? B : U;
+  if (j0 <= i0) {
+#pragma unroll 1
+    for (int k0 = 0; k0 < DK; k0 += 16) {
+      uint32_t uh[4], ul[4], rh[4], rl[4];
+      const size_t o = (size_t)(i0 + (lane & 15)) * Lay::ldk + k0 + (lane >> 4) * 8;
+      ldsm4(uh, U.hi + o);
+      ldsm4(ul, U.lo + o);
+      ldsm4(rh, R.hi + o);
+      ldsm4(rl, R.lo + o);
+#pragma unroll
+      for (int jb = 0; jb < 2; ++jb) {
+        if (j0 + jb * 16 > i0) continue;
+        const int row = j0 + jb * 16 + (lane & 7) + ((lane >> 4) << 3), col = k0 + ((lane >> 3) & 1) * 8;
+        uint32_t bh[4], bl[4];
+        ldsm4(bh, CB.hi + (size_t)row * CB.ld + col);
+        ldsm4(bl, CB.lo + (size_t)row * CB.ld + col);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mma(sa[jb * 2 + e], uh, bh[2 * e], bh[2 * e + 1]);
+          mma(sq[jb * 2 + e], rh, bh[2 * e], bh[2 * e + 1]);
+          mma(sa[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
+          mma(sq[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
+          mma(sa[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
+          mma(sq[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+        }
+        if constexpr (GEN) {
+          ldsm4(bh, K.hi + (size_t)row * K.ld + col);
+          ldsm4(bl, K.lo + (size_t)row * K.ld + col);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            mma(sb[jb * 2 + e], uh, bh[2 * e], bh[2 * e + 1]);
+            mma(sp[jb * 2 + e], rh, bh[2 * e], bh[2 * e + 1]);
+            mma(sb[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
+            mma(sp[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
+            mma(sb[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
+            mma(sp[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+          }
+        }
+      }
+    }
+  }
+  __syncthreads();                                        // the logs are consumed: their space takes A
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const int i = i0 + g + (x >> 1) * 8, j = j0 + e * 8 + 2 * t + (x & 1);
+      float dec = 1.f, beta = 1.f;
+      if constexpr (!GEN) {
+        dec = j <= i ? ex2(sG[i] - sG[j]) : 0.f;
+        beta = sBeta[i];
+      }
+      sa[e][x] = j < i ? sa[e][x] * dec * beta : 0.f;
+      sq[e][x] = j <= i ? sq[e][x] * dec : 0.f;
+      if constexpr (GEN) {
+        sb[e][x] = j < i ? sb[e][x] : 0.f;
+        sp[e][x] = j <= i ? sp[e][x] : 0.f;
+      }
+      sA[i * kLdF + j] = sa[e][x];
+    }
+  __syncthreads();
+  // ---- M = (I + A)^-1: 16 x 16 diagonal blocks by substitution, a column per thread, then block by block below
+  for (int e = tid; e < kC * kC; e += 256) {
+    const int i = e >> 6, j = e & 63;
+    if ((j >> 4) > (i >> 4)) sM[i * kLdF + j] = 0.f;
+  }
+  if (tid < kC) {
+    const int b0 = tid & ~15, cc = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float s = i == cc ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < 16; ++j)
+        if (j < i) s = fmaf(-sA[(b0 + i) * kLdF + b0 + j], x[j], s);
+      x[i] = s;
+      sM[(b0 + i) * kLdF + b0 + cc] = s;
+    }
+  }
+  __syncthreads();
+  {
+    const int r = tid >> 4, cc = tid & 15;
+    for (int lev = 1; lev < 4; ++lev) {
+      for (int jb = 0; jb + lev < 4; ++jb) {
+        const int ib = jb + lev;
+        float s = 0.f;
+        for (int k = jb * 16; k < ib * 16; ++k) s = fmaf(sA[(ib * 16 + r) * kLdF + k], sM[k * kLdF + jb * 16 + cc], s);
+        sT[(jb * 16 + r) * 17 + cc] = s;
+      }
+      __syncthreads();
+      for (int jb = 0; jb + lev < 4; ++jb) {
+        const int ib = jb + lev;
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) s = fmaf(sM[(ib * 16 + r) * kLdF + ib * 16 + k], sT[(jb * 16 + k) * 17 + cc], s);
+        sM[(ib * 16 + r) * kLdF + jb * 16 + cc] = -s;
+      }
+      __syncthreads();
+    }
+  }
+  // M as planes; gated: times diag(beta 2^G) for Xw, diag(beta) for Xu
+  auto put_m = [&](bool decayed) {
+    for (int e = tid; e < kC * kC / 2; e += 256) {
+      const int i = e >> 5, j = (e & 31) * 2;
+      float a = sM[i * kLdF + j], b = sM[i * kLdF + j + 1];
+      if constexpr (!GEN) {
+        a *= sBeta[j] * (decayed ? ex2(sG[j]) : 1.f);
+        b *= sBeta[j + 1] * (decayed ? ex2(sG[j + 1]) : 1.f);
+      }
+      Z0.put(i, j, a, b);
+    }
+  };
+  put_m(true);
+  cp_wait<0>();
+  __syncthreads();
+  // ---- Xw = -M U and Xu; this warp's 16 rows and one half of the columns
+  constexpr int NK = DK / 16, NV = DV / 16;
+  const int nk0 = half * (DK / 2), nv0 = half * (DV / 2), kend = i0 + 16;
+  float xw[NK][4], xu[NV][4];
+  zero<NK>(xw);
+  zero<NV>(xu);
+  mm<NK, false, true>(xw, Z0, i0, U, nk0, 0, kend);
+  const Planes& XW = GEN ? U : B;
+  float po[NV][4];                                        // O'
+  zero<NV>(po);
+  if constexpr (GEN) {
+    put_acc<4>(Z1, i0, j0, sb, 1.f);
+    __syncthreads();
+    float mbv[4][4];
+    zero<4>(mbv);
+    mm<4, false, true>(mbv, Z0, i0, Z1, j0, 0, kend);
+    __syncthreads();
+    put_acc<4>(Z0, i0, j0, mbv, -1.f);
+    put_acc<4>(Z1, i0, j0, sp, 1.f);
+    put_acc<NK>(XW, i0, nk0, xw, -1.f);
+    __syncthreads();
+    mm<NV, false, false>(xu, Z0, i0, V, nv0, 0, kend);
+    mm<NV, false, false>(po, Z1, i0, V, nv0, 0, kend);
+    __syncthreads();
+    put_acc<4>(Z0, i0, j0, sq, 1.f);
+  } else {
+    __syncthreads();
+    put_m(false);
+    put_acc<NK>(XW, i0, nk0, xw, -1.f);
+    const float gl = sG[kC - 1];
+    for (int e = tid; e < kC * DK / 2; e += 256) {        // the keys decayed to the chunk's end
+      const int i = e / (DK / 2), d = (e - i * (DK / 2)) * 2;
+      const float2 u = U.get(i, d);
+      const float f = i < valid ? ex2(gl - sG[i]) : 0.f;
+      U.put(i, d, u.x * f, u.y * f);
+    }
+    __syncthreads();
+    mm<NV, false, false>(xu, Z0, i0, V, nv0, 0, kend);
+    __syncthreads();
+    put_acc<4>(Z0, i0, j0, sq, 1.f);
+    put_acc<NV>(K, i0, nv0, xu, 1.f);
+  }
+  __syncthreads();
+  // ---- R' = R (gated: decayed) + Q Xw
+  {
+    float acc[NK][4];
+#pragma unroll
+    for (int i = 0; i < NK; ++i)
+#pragma unroll
+      for (int h2 = 0; h2 < 2; ++h2) {
+        const int row = i0 + g + 8 * h2;
+        const float2 r = R.get(row, nk0 + i * 8 + 2 * t);
+        const float f = GEN ? 1.f : ex2(sG[row]);
+        acc[i][2 * h2] = r.x * f;
+        acc[i][2 * h2 + 1] = r.y * f;
+      }
+    mm<NK, false, true>(acc, Z0, i0, XW, nk0, 0, kend);
+    bf16* gr = p.ws_r + ci * 2 * kC * DK;
+    put_acc<NK>(Planes{gr, gr + kC * DK, DK}, i0, nk0, acc, 1.f);
+  }
+  // ---- the state's side: 16 key rows per warp (and, for 64 of them, half of the columns)
+  constexpr int kMB = DK / 16, kCW = 8 / kMB, NE = DV / 8 / kCW, NT = DK / 8 / kCW;
+  const int m0 = (warp % kMB) * 16, e0 = (warp / kMB) * NE * 8, x0 = (warp / kMB) * NT * 8;
+  float acc_e[NE][4];
+  zero<NE>(acc_e);
+  if constexpr (GEN) {
+    mm<NE, true, false>(acc_e, K, m0, V, e0, 0, kC);
+    __syncthreads();                                      // K is consumed: its space takes Xu
+    put_acc<NV>(K, i0, nv0, xu, 1.f);
+    __syncthreads();
+  }
+  mm<NV, false, true>(po, Z0, i0, K, nv0, 0, kend);        // O' += Q Xu
+  {
+    float* go = p.ws_o + ci * kC * DV;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      *reinterpret_cast<float2*>(go + (size_t)(i0 + g) * DV + nv0 + i * 8 + 2 * t) = make_float2(po[i][0], po[i][1]);
+      *reinterpret_cast<float2*>(go + (size_t)(i0 + g + 8) * DV + nv0 + i * 8 + 2 * t) = make_float2(po[i][2], po[i][3]);
+    }
+  }
+  mm<NE, true, true>(acc_e, GEN ? B : U, m0, K, e0, 0, kC);
+  const float d0 = GEN ? sD[m0 + g] : 1.f, d1 = GEN ? sD[m0 + g + 8] : 1.f;
+  {
+    float* ge = p.ws_e + ci * DK * DV;
+#pragma unroll
+    for (int i = 0; i < NE; ++i) {
+      *reinterpret_cast<float2*>(ge + (size_t)(m0 + g) * DV + e0 + i * 8 + 2 * t) = make_float2(acc_e[i][0] * d0, acc_e[i][1] * d0);
+      *reinterpret_cast<float2*>(ge + (size_t)(m0 + g + 8) * DV + e0 + i * 8 + 2 * t) = make_float2(acc_e[i][2] * d1, acc_e[i][3] * d1);
+    }
+  }
+  float acc_t[NT][4];
+  zero<NT>(acc_t);
+  mm<NT, true, true>(acc_t, GEN ? B : U, m0, XW, x0, 0, kC);
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    acc_t[i][0] *= d0; acc_t[i][1] *= d0; acc_t[i][2] *= d1; acc_t[i][3] *= d1;
+  }
+  bf16* gt = p.ws_t + ci * 2 * DK * DK;
+  put_acc<NT>(Planes{gt, gt + DK * DK, DK}, m0, x0, acc_t, 1.f);
+}
+
+// ------------------------------------------------------------------ recurrence over chunks
+constexpr int kSlice = 32;         // value columns per CTA
+
+template <int DK>
+struct ScanLayout {
+  static constexpr int ldt = DK + 8, lds = kSlice + 8;
+  static constexpr size_t t_stage = 2 * (size_t)DK * ldt * 2, s = 2 * t_stage, bytes = s + 2 * (size_t)DK * lds * 2;
+};
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p) {
+  using Lay = ScanLayout<DK>;
+  extern __shared__ __align__(16) uint8_t sm[];
+  const int slice = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const int n = p.q_len[seq];
+  if (n <= 0) return;
+  const int slot = p.slots[seq], H = p.in.H;
+  if (slot < 0 || slot >= p.num_slots) {
+    if (p.status && tid == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
+    return;
+  }
+  const int chunks = (n + kC - 1) / kC, c0 = slice * kSlice;
+  const size_t first = (size_t)(p.q_start[seq] / kC + seq);
+  constexpr int kMB = DK / 16, kCW = 8 / kMB, N8 = kSlice / 8 / kCW;
+  const int m0 = (warp % kMB) * 16, n0 = (warp / kMB) * N8 * 8;
+  const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
+  auto stage = [&](int c) {
+    bf16* base = reinterpret_cast<bf16*>(sm + (c & 1) * Lay::t_stage);
+    return Planes{base, base + DK * Lay::ldt, Lay::ldt};
+  };
+  auto issue = [&](int c) {
+    if (c < chunks) {
+      const Planes d = stage(c);
+      const bf16* src = p.ws_t + ((first + c) * H + hd) * 2 * DK * DK;
+      for (int i = tid; i < 2 * DK * (DK / 8); i += 256) {
+        const int pl = i / (DK * (DK / 8)), e = i - pl * (DK * (DK / 8)), r = e / (DK / 8), cc = (e - r * (DK / 8)) * 8;
+        cp16((pl ? d.lo : d.hi) + r * Lay::ldt + cc, src + (size_t)i * 8, true);
+      }
+    }
+    cp_commit();
+  };
+  float* st = p.state + ((size_t)slot * H + hd) * DK * DV + c0;
+  const bool fresh = p.positions[p.q_start[seq]] == 0;
+  float s[N8][4];
+#pragma unroll
+  for (int i = 0; i < N8; ++i)
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) {
+      float2 v = make_float2(0.f, 0.f);
+      if (!fresh) v = *reinterpret_cast<const float2*>(st + (size_t)(m0 + g + 8 * h2) * DV + n0 + i * 8 + 2 * t);
+      s[i][2 * h2] = v.x;
+      s[i][2 * h2 + 1] = v.y;
+    }
+  issue(0);
+  for (int c = 0; c < chunks; ++c) {
+    const size_t ci = (first + c) * H + hd;
+    issue(c + 1);
+    // this chunk's additions, on their way while the start state is laid out
+    float e[N8][4];
+    const float* ge = p.ws_e + ci * DK * DV + c0;
+    const float d0 = p.ws_d[ci * DK + m0 + g], d1 = p.ws_d[ci * DK + m0 + g + 8];
+#pragma unroll
+    for (int i = 0; i < N8; ++i)
+#pragma unroll
+      for (int h2 = 0; h2 < 2; ++h2) {
+        const float2 v = *reinterpret_cast<const float2*>(ge + (size_t)(m0 + g + 8 * h2) * DV + n0 + i * 8 + 2 * t);
+        e[i][2 * h2] = v.x;
+        e[i][2 * h2 + 1] = v.y;
+      }
+    put_acc<N8>(S, m0, n0, s, 1.f);
+    bf16* gs = p.ws_s + ci * 2 * DK * DV + c0;
+    put_acc<N8>(Planes{gs, gs + DK * DV, DV}, m0, n0, s, 1.f);
+    cp_wait<1>();
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < N8; ++i) {
+      s[i][0] = fmaf(d0, s[i][0], e[i][0]); s[i][1] = fmaf(d0, s[i][1], e[i][1]);
+      s[i][2] = fmaf(d1, s[i][2], e[i][2]); s[i][3] = fmaf(d1, s[i][3], e[i][3]);
+    }
+    mm<N8, false, true>(s, stage(c), m0, S, n0, 0, DK);
+    __syncthreads();                                      // S and this stage are consumed
+  }
+  cp_wait<0>();
+  if (p.write_state) {
+#pragma unroll
+    for (int i = 0; i < N8; ++i)
+#pragma unroll
+      for (int h2 = 0; h2 < 2; ++h2)
+        *reinterpret_cast<float2*>(st + (size_t)(m0 + g + 8 * h2) * DV + n0 + i * 8 + 2 * t) = make_float2(s[i][2 * h2], s[i][2 * h2 + 1]);
+  }
+}
+
+// ------------------------------------------------------------------ outputs of a chunk
+template <int DK, int DV>
+struct OutLayout {
+  static constexpr int ldr = DK + 8, lds = DV + 8;
+  static constexpr size_t r = 0, s = 2 * (size_t)kC * ldr * 2, bytes = s + 2 * (size_t)DK * lds * 2;
+};
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(256, 2) delta_out_kernel(const ChunkParams p) {
+  using Lay = OutLayout<DK, DV>;
+  extern __shared__ __align__(16) uint8_t sm[];
+  __shared__ float s_ss[kC][2];
+  const int c = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  mb::pdl_wait();
+  mb::pdl_launch_dependents();
+  const int n = p.q_len[seq];
+  if (c * kC >= n) return;
+  const int t0 = p.q_start[seq] + c * kC, valid = min(kC, n - c * kC), H = p.in.H;
+  const size_t ci = ((size_t)(p.q_start[seq] / kC + seq + c)) * H + hd;
+  const Planes R{reinterpret_cast<bf16*>(sm + Lay::r), reinterpret_cast<bf16*>(sm + Lay::r) + kC * Lay::ldr, Lay::ldr};
+  const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
+  const bf16 *gr = p.ws_r + ci * 2 * kC * DK, *gs = p.ws_s + ci * 2 * DK * DV;
+  for (int i = tid; i < 2 * kC * (DK / 8); i += 256) {
+    const int pl = i / (kC * (DK / 8)), e = i - pl * (kC * (DK / 8)), r = e / (DK / 8), cc = (e - r * (DK / 8)) * 8;
+    cp16((pl ? R.lo : R.hi) + r * Lay::ldr + cc, gr + (size_t)i * 8, true);
+  }
+  for (int i = tid; i < 2 * DK * (DV / 8); i += 256) {
+    const int pl = i / (DK * (DV / 8)), e = i - pl * (DK * (DV / 8)), r = e / (DV / 8), cc = (e - r * (DV / 8)) * 8;
+    cp16((pl ? S.lo : S.hi) + r * Lay::lds + cc, gs + (size_t)i * 8, true);
+  }
+  cp_commit();
+  constexpr int NV = DV / 16;
+  const int i0 = (warp & 3) * 16, half = warp >> 2, nv0 = half * (DV / 2);
+  float o[NV][4];
+  const float* go = p.ws_o + ci * kC * DV;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) {
+      const float2 v = *reinterpret_cast<const float2*>(go + (size_t)(i0 + g + 8 * h2) * DV + nv0 + i * 8 + 2 * t);
+      o[i][2 * h2] = v.x;
+      o[i][2 * h2 + 1] = v.y;
+    }
+  cp_wait<0>();
+  __syncthreads();
+  mm<NV, false, true>(o, R, i0, S, nv0, 0, DK);
+  if (!p.norm_w) {
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) {
+      const int row = i0 + g + 8 * h2;
+      if (row >= valid) continue;
+      float* dst = p.out + ((size_t)(t0 + row) * H + hd) * DV + nv0 + 2 * t;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][2 * h2], o[i][2 * h2 + 1]);
+    }
+    return;
+  }
+#pragma unroll
+  for (int h2 = 0; h2 < 2; ++h2) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss = fmaf(o[i][2 * h2], o[i][2 * h2], fmaf(o[i][2 * h2 + 1], o[i][2 * h2 + 1], ss));
+    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+    if (t == 0) s_ss[i0 + g + 8 * h2][half] = ss;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int h2 = 0; h2 < 2; ++h2) {
+    const int row = i0 + g + 8 * h2;
+    if (row >= valid) continue;
+    const float inv = rsqrtf((s_ss[row][0] + s_ss[row][1]) / (float)DV + p.eps) * p.scale;
+    const int col = hd * DV + nv0 + 2 * t;
+    const bf16* gz = p.gate + (size_t)(t0 + row) * p.gate_ld + col;
+    bf16* dst = p.norm_out + (size_t)(t0 + row) * p.norm_out_ld + col;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gz + i * 8));
+      const float2 w = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.norm_w + col + i * 8));
+      const float a = p.sigmoid_gate ? mb::sigmoid_fast(z.x) : mb::silu(z.x), b = p.sigmoid_gate ? mb::sigmoid_fast(z.y) : mb::silu(z.y);
+      *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(o[i][2 * h2] * inv * w.x * a, o[i][2 * h2 + 1] * inv * w.y * b);
+    }
+  }
+}
+
+template <int DK, int DV, bool GEN>
+int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
+  constexpr size_t sp = PrepLayout<DK, DV>::bytes, ss = ScanLayout<DK>::bytes, so = OutLayout<DK, DV>::bytes;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<DK, DV, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sp);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_scan_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_out_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const dim3 grid((max_q_len + kC - 1) / kC, p.in.H, num_seqs);
+  cudaError_t e = mb::launch_kernel(delta_prep_kernel<DK, DV, GEN>, grid, dim3(256), sp, stream, p);
+  if (e == cudaSuccess) e = mb::launch_kernel(delta_scan_kernel<DK, DV>, dim3(DV / kSlice, p.in.H, num_seqs), dim3(256), ss, stream, p);
+  if (e == cudaSuccess) e = mb::launch_kernel(delta_out_kernel<DK, DV>, grid, dim3(256), so, stream, p);
+  return (int)e;
+}
+template <int DK, int DV>
+int launch_rule(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
+  return p.in.general ? launch_chunks<DK, DV, true>(p, num_seqs, max_q_len, stream) : launch_chunks<DK, DV, false>(p, num_seqs, max_q_len, stream);
+}
+
+size_t per_chunk(int DK, int DV) { return (size_t)DK * DK * 4 + (size_t)DK * DV * 8 + (size_t)kC * DK * 4 + (size_t)kC * DV * 4 + (size_t)DK * 4; }
+
+}  // namespace
+
+struct MbDeltaChunkedArgs {
+  mb::DeltaInputs in;
+  float* state;
+  float* out;
+  void* ws;
+  size_t ws_bytes;
+  const int* q_start;
+  const int* q_len;
+  const int* positions;
+  const int* slots;
+  int total_rows, num_seqs, num_slots, max_q_len, write_state;
+  uint32_t* status;
+  const void* norm_w;        // or null: fp32 rows to `out`
+  const void* gate;
+  long long gate_ld;
+  int sigmoid_gate;
+  float eps, scale;
+  void* norm_out;
+  long long norm_out_ld;
+};
+
+extern "C" size_t mb_delta_chunked_ws_bytes(int total_rows, int num_seqs, int H, int DK, int DV) {
+  return ((size_t)total_rows / kC + num_seqs) * H * per_chunk(DK, DV) + 1024;
+}
+
+extern "C" int mb_delta_chunked(const MbDeltaChunkedArgs* a, cudaStream_t stream) {
+  if (!a || !mb::delta_inputs_ok(a->in, false) || !a->state || (!a->out && !a->norm_w) || !a->ws || a->in.f32) return MB_ERR_BAD_ARG;
+  if (a->num_seqs <= 0 || a->num_seqs > 65535 || a->in.H > 65535 || a->max_q_len <= 0 || a->total_rows <= 0) return MB_ERR_BAD_ARG;
+  const DeltaInputs& in = a->in;
+  const auto bad = [](const void* ptr, long long ld) { return (reinterpret_cast<uintptr_t>(ptr) & 15) || ld % 8; };
+  if (bad(in.q, in.q_ld) || bad(in.k, in.k_ld) || bad(in.v, in.v_ld) || (in.general && bad(in.removal, in.removal_ld)) || bad(a->state, 0) ||
+      bad(a->out, 0) || bad(a->ws, 0))
+    return MB_ERR_UNSUPPORTED;                             // 16-byte copies
+  if (a->norm_w && (!a->gate || !a->norm_out || a->gate_ld % 2 || a->norm_out_ld % 2 || (reinterpret_cast<uintptr_t>(a->gate) & 3) ||
+                    (reinterpret_cast<uintptr_t>(a->norm_out) & 3) || (reinterpret_cast<uintptr_t>(a->norm_w) & 3)))
+    return MB_ERR_UNSUPPORTED;
+  if (a->ws_bytes < mb_delta_chunked_ws_bytes(a->total_rows, a->num_seqs, in.H, in.DK, in.DV)) return MB_ERR_TOO_LARGE;
+  ChunkParams p{};
+  p.in = in; p.state = a->state; p.out = a->out;
+  const size_t chunks = ((size_t)a->total_rows / kC + a->num_seqs) * in.H, kk = (size_t)in.DK * in.DK, kv = (size_t)in.DK * in.DV;
+  p.ws_t = reinterpret_cast<bf16*>(a->ws);
+  p.ws_e = reinterpret_cast<float*>(p.ws_t + chunks * 2 * kk);
+  p.ws_s = reinterpret_cast<bf16*>(p.ws_e + chunks * kv);
+  p.ws_r = p.ws_s + chunks * 2 * kv;
+  p.ws_o = reinterpret_cast<float*>(p.ws_r + chunks * 2 * kC * in.DK);
+  p.ws_d = p.ws_o + chunks * kC * in.DV;
+  p.q_start = a->q_start; p.q_len = a->q_len; p.positions = a->positions; p.slots = a->slots;
+  p.num_slots = a->num_slots; p.write_state = a->write_state; p.status = a->status;
+  p.norm_w = (const bf16*)a->norm_w; p.gate = (const bf16*)a->gate; p.gate_ld = a->gate_ld; p.sigmoid_gate = a->sigmoid_gate;
+  p.eps = a->eps; p.scale = a->scale; p.norm_out = (bf16*)a->norm_out; p.norm_out_ld = a->norm_out_ld;
+  if (in.DK == 64 && in.DV == 64) return launch_rule<64, 64>(p, a->num_seqs, a->max_q_len, stream);
+  if (in.DK == 64 && in.DV == 128) return launch_rule<64, 128>(p, a->num_seqs, a->max_q_len, stream);
+  if (in.DK == 128 && in.DV == 64) return launch_rule<128, 64>(p, a->num_seqs, a->max_q_len, stream);
+  if (in.DK == 128 && in.DV == 128) return launch_rule<128, 128>(p, a->num_seqs, a->max_q_len, stream);
+  return MB_ERR_UNSUPPORTED;
+}

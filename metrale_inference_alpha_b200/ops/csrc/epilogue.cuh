@@ -8,6 +8,8 @@ enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_CLAMP_GLU = 2, EPI_SILU_COLS = 3, EPI_
 
 __device__ __forceinline__ float relu2(float z) { const float r = fmaxf(z, 0.f); return r * r; }
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
+// the same with the approximate exponential and divide (a few ulp)
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
 
 // g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(alpha g) (u + 1)

@@ -489,7 +489,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
               for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::log_sigmoid(y[i]);
             } else if (p.epilogue == EPI_SIGMOID) {
 #pragma unroll
-              for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::sigmoid_exact(y[i]);
+              for (int i = 0; i < 8; ++i) y[i] = p.epi_a * mb::sigmoid_fast(y[i]);
             }
           }
         }
@@ -924,7 +924,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
               for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::log_sigmoid(v[j]);
             } else if (p.epilogue == EPI_SIGMOID) {
 #pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::sigmoid_exact(v[j]);
+              for (int j = 0; j < 16; ++j) v[j] = p.epi_a * mb::sigmoid_fast(v[j]);
             }
           }
 #pragma unroll

@@ -42,6 +42,25 @@ struct SoftCap {
   }
 };
 
+// An output row turned back by its own position (values that are cached turned by theirs): pair (m, m + dv / 2) by minus
+// the angle in the tables' row of that position.
+struct TurnBack {
+  const float* cos_tab;   // [max_pos, dv / 2], or null: off
+  const float* sin_tab;
+  int half, max_pos;
+  // N consecutive elements of the first half and their partners, element d on
+  template <int N>
+  __device__ __forceinline__ void operator()(int pos, int d, float* u, float* v) const {
+    const size_t at = (size_t)(pos < max_pos ? pos : 0) * half + d;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float c = __ldg(cos_tab + at + i), s = __ldg(sin_tab + at + i), a = u[i], b = v[i];
+      u[i] = a * c + b * s;
+      v[i] = b * c - a * s;
+    }
+  }
+};
+
 enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 
 // Sigmoid gates on an attention output, read where the projection left their logits: one per head, or one per element

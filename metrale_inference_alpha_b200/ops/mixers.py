@@ -581,11 +581,16 @@ class OutputGate:
 
 def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int, scale: float, sink, fmt: str,
                    out: torch.Tensor, out_scale: float = 1.0, kernel: str = "auto", window: int = 0, keep: int = 0,
-                   gate: Optional[OutputGate] = None, softcap: float = 0.0) -> torch.Tensor:
+                   gate: Optional[OutputGate] = None, softcap: float = 0.0, turn_back=None) -> torch.Tensor:
     """Causal paged attention of q [T, Hq, padded dk] into ``out`` [T, Hq * dv] (may be a column range), times
     ``out_scale`` and the ``gate``. ``sink``: True adds one to the softmax denominator, a tensor [Hq] (fp32) exp(sink) per
-    head. ``softcap`` > 0: scores become softcap tanh(score / softcap). ``window`` > 0: a position sees itself, the window - 1 before it and the first ``keep``. The softmax weights keep
+    head. ``softcap`` > 0: scores become softcap tanh(score / softcap). ``turn_back`` = (cos, sin) tables over dv / 2: every
+    output row is turned by minus its position, in the kernel's own store where that has both halves. ``window`` > 0: a position sees itself, the window - 1 before it and the first ``keep``. The softmax weights keep
     32-bit precision: they enter the product with V as two bf16 terms. ``kernel``: auto | simt | mma | tc (tests)."""
+    if turn_back is not None and not (q.is_cuda and gate is None and _turns(q, k_cache, v_cache, batch, dv, fmt, kernel, out)):
+        kw = dict(dk=dk, dv=dv, scale=scale, sink=sink, fmt=fmt, out=out, out_scale=out_scale, window=window, keep=keep, softcap=softcap)
+        assert gate is None
+        return turn_rows(attention_dims(q, k_cache, v_cache, batch, kernel=kernel, **kw), q.shape[1], dv, batch.positions, turn_back, fmt)
     sink_w = sink if isinstance(sink, torch.Tensor) else None
     sink = sink_w is not None or bool(sink)
     keep = keep if window > 0 else 0
@@ -626,14 +631,8 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
     S, mq = batch.q_len.numel(), int(batch.max_q_len)
     assert out.stride(1) == 1 and out.dtype == DTYPE[fmt]
     G = Hq // Hkv
-    tiles_ok = fmt == "bf16" and dkp in (64, 128, 256) and dvp in (64, 128, 256) and (dkp == dvp or max(dkp, dvp) <= 128) \
-        and (dv != dvp or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0))
     if kernel == "auto":
-        kernel = "mma" if tiles_ok else "simt"
-        if tiles_ok and tc_serves(dkp, dvp, dv, out, gate) and mq >= 128:
-            kernel = "tc"
-        elif kernel == "mma" and dkp == 256 and 16 < G * mq <= 32:
-            kernel = "simt"                          # between the two row-tile limits of the 256-wide tiles
+        kernel = _attention_kernel(dkp, dvp, dv, G, mq, fmt, out, gate)
     if kernel == "simt":
         a = _SimtAttnArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_table), batch.block_table.stride(0),
                           _ptr(batch.q_start), _ptr(batch.q_len), _ptr(batch.ctx_len), T, S, Hq, Hkv, dk, dv, dkp, dvp, bs, nb,
@@ -653,6 +652,8 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
             batch.block_table.stride(0), S, mq
         t.Hq, t.Hkv, t.D, t.block_size, t.scale, t.v_mn = Hq, Hkv, dkp, bs, float(scale), 1
         t.out_ld, t.out_scale, t.sink, t.split_p = out.stride(0), float(out_scale), int(sink), 1
+        if turn_back is not None:
+            t.turn_cos, t.turn_sin, t.turn_max = _ptr(turn_back[0]), _ptr(turn_back[1]), turn_back[0].shape[0]
         t.sink_w, t.window, t.keep, t.softcap = _ptr(sink_w), window, keep, float(softcap)
         if gate is not None:
             gate.into(t)
@@ -668,6 +669,8 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
     a.Hq, a.Hkv, a.D, a.block_size, a.num_blocks, a.scale = Hq, Hkv, dkp, bs, nb, float(scale)
     a.out, a.total_rows, a.part_tokens, a.status = _ptr(out), T, _ATTN_PART_TOKENS, _ptr(rt.status)
     a.DV, a.dv, a.out_ld, a.out_scale, a.sink, a.split_p = dvp, dv, out.stride(0), float(out_scale), int(sink), 1
+    if turn_back is not None:
+        a.turn_cos, a.turn_sin, a.turn_max = _ptr(turn_back[0]), _ptr(turn_back[1]), turn_back[0].shape[0]
     a.sink_w, a.window, a.keep, a.softcap = _ptr(sink_w), window, keep, float(softcap)
     if gate is not None:
         gate.into(a)
@@ -678,6 +681,24 @@ def attention_dims(q: torch.Tensor, k_cache, v_cache, batch, *, dk: int, dv: int
     _native.check(L.mb_paged_attention(C.byref(a), _stream()), f"attention_dims[T={T}]")
     _count()
     return out
+
+
+def _attention_kernel(dkp: int, dvp: int, dv: int, G: int, mq: int, fmt: str, out: torch.Tensor, gate) -> str:
+    """Which kernel serves a step: simt (fp32, or sizes without tiles), tc (long portions on tcgen05) or mma."""
+    if not (fmt == "bf16" and dkp in (64, 128, 256) and dvp in (64, 128, 256) and (dkp == dvp or max(dkp, dvp) <= 128)
+            and (dv != dvp or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0))):
+        return "simt"
+    if tc_serves(dkp, dvp, dv, out, gate) and mq >= 128:
+        return "tc"
+    return "simt" if dkp == 256 and 16 < G * mq <= 32 else "mma"    # between the two row-tile limits of the 256-wide tiles
+
+
+def _turns(q, k_cache, v_cache, batch, dv: int, fmt: str, kernel: str, out: torch.Tensor) -> bool:
+    """Whether the kernel that serves a step turns its output rows back itself."""
+    G, mq, dvp = q.shape[1] // k_cache.shape[2], int(batch.max_q_len), v_cache.shape[3]
+    if kernel == "auto":
+        kernel = _attention_kernel(q.shape[2], dvp, dv, G, mq, fmt, out, None)
+    return kernel == "tc" or (kernel == "mma" and dv % 8 == 0 and (G * mq <= 32 or dv == dvp))
 
 
 def tc_serves(dkp: int, dvp: int, dv: int, out: torch.Tensor, gate: Optional[OutputGate] = None) -> bool:

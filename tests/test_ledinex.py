@@ -94,7 +94,7 @@ def run_stream(device, fmt, x, y, routed_of, norm, filt, cuts, slots=4, verify=(
 def test_stream_joins_and_convolves(device, fmt, W, taps, plus):
     """Pending output (alone, with expert rows, only expert rows, none), portions of many lengths beside another sequence,
     windows carried from portion to portion, verify steps that keep part of their rows."""
-    n, K, eps = 45, 3, 1e-3
+    n, K, eps = 130 if W <= 100 else 100, 3, 1e-3
     x, y, e = gen(2, n, W, seed=1, std=2.0), gen(2, n, W, seed=2).to(dt(fmt)).float(), gen(2, n, W, seed=3)
     w, filt = b16(gen(W, seed=4, std=0.4)), b16(gen(W, taps, seed=5, std=0.5))
     norm, f = mx.RmsNorm(w.to(device), eps, plus_one=plus), filt.t().contiguous().to(device)
@@ -115,7 +115,7 @@ def test_stream_joins_and_convolves(device, fmt, W, taps, plus):
     for what, Y in (("y", y.double()), ("both", y.double() + e.double()), ("none", None)):
         X = x.double() if Y is None else x.double() + lo.unit_rms(Y, eps) * wd
         H = torch.stack([X[s] + lo.short_conv(X[s], filt.double()) for s in range(2)])
-        for cuts in ([n], [2], [1], [17, 1, 9, 8, 4]):
+        for cuts in ([n], [2], [17, 1, 9, 8, 4], [3, 97, 1]):
             x1, h = run_stream(device, fmt, x, None if Y is None else y, routed if what == "both" else None, norm, f, cuts,
                                verify=(0, 2) if cuts[0] == 17 else ())
             close(x1, X, 3e-6)                                       # the stream is 32-bit in both formats
@@ -219,8 +219,9 @@ ATT = {"t64": (4, 2, 64, 64), "t64/128": (4, 4, 40, 128), "t128": (6, 2, 128, 12
        "t256": (2, 1, 200, 72), "t256 full": (4, 2, 256, 256), "past": (2, 1, 264, 20), "odd": (3, 1, 22, 30)}
 
 
-def run_attention(device, fmt, q, k, v, dims, cuts, scale, window, softcap, kernel="auto", block=16):
-    """One sequence fed in portions through the paged cache (pages not in order, unwritten slots NaN); [n, H, dv]."""
+def run_attention(device, fmt, q, k, v, dims, cuts, scale, window, softcap, kernel="auto", block=16, turn=None):
+    """One sequence fed in portions through the paged cache (pages not in order, unwritten slots NaN); [n, H, dv]. `turn`:
+    values are cached turned by their position, outputs turned back."""
     H, G, dk, dv = dims
     n = q.shape[0]
     dkp, dvp = mx.padded_head_dims(dk, dv, fmt)
@@ -232,10 +233,11 @@ def run_attention(device, fmt, q, k, v, dims, cuts, scale, window, softcap, kern
     for at, m in portions(n, cuts):
         b = lc.batch([m], [at + m], device=device, block=block, pages=[pages[:(at + m + block - 1) // block]])
         qq = mx.attention_rows(rows[at:at + m].to(device), cols=(0, H * dk, (H + G) * dk), Hq=H, Hkv=G, dk=dk, dv=dv, positions=b.positions,
-                               slots=b.slot_mapping, k_cache=kc, v_cache=vc, rot=None, fmt=fmt)
+                               slots=b.slot_mapping, k_cache=kc, v_cache=vc, rot=None, fmt=fmt, v_rot=turn)
         out = torch.empty(m, H * dv, dtype=dt(fmt), device=device)
         kern = kernel if kernel != "tc" or m >= 2 else "auto"
-        outs.append(mx.attention_dims(qq, kc, vc, b, dk=dk, dv=dv, scale=scale, sink=False, fmt=fmt, out=out, window=window, softcap=softcap, kernel=kern))
+        outs.append(mx.attention_dims(qq, kc, vc, b, dk=dk, dv=dv, scale=scale, sink=False, fmt=fmt, out=out, window=window, softcap=softcap, kernel=kern,
+                                      turn_back=turn))
     return torch.cat(outs).view(n, H, dv)
 
 
@@ -255,6 +257,23 @@ def test_capped_and_windowed_attention(device, fmt, name, window, softcap):
     want = lo.attend(q.double(), k.double(), v.double(), scale, window or None, softcap or None)
     for cuts in ([n], [2], [33, 1], [1]):
         close(run_attention(device, fmt, q, k, v, dims, cuts, scale, window, softcap), want, 2e-5 if fmt == "fp32" else 8e-3)
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", DTYPES)
+@pytest.mark.parametrize("name", list(ATT))
+def test_rotated_values(device, fmt, name):
+    """Values turned by their position and outputs turned back: what reaches a query is turned by the distance alone."""
+    dims, n, scale, base = ATT[name], 150, 0.2, 50.0
+    H, G, dk, dv = dims
+    q, k, v = (gen(n, h, d, seed=s).to(dt(fmt)) for h, d, s in ((H, dk, 1), (G, dk, 2), (G, dv, 3)))
+    turn = ref.rope_tables(200, dv, base, device=device)
+    vt = lo.turn_values(v.double(), base, 1)
+    s = torch.einsum("ihd,jhd->hij", q.double(), k.double().repeat_interleave(H // G, 1)) * scale
+    p = torch.softmax(s.masked_fill(torch.arange(n)[None] > torch.arange(n)[:, None], float("-inf")), -1)
+    want = lo.turn_values(torch.einsum("hij,jhd->ihd", p, vt.repeat_interleave(H // G, 1)), base, -1)
+    for cuts in ([n], [7], [130, 1], [1]):
+        close(run_attention(device, fmt, q, k, v, dims, cuts, scale, 0, 0.0, turn=turn), want, 2e-5 if fmt == "fp32" else 1e-2)
 
 
 @pytest.mark.parametrize("device", DEVICES)
