@@ -1,6 +1,7 @@
 """One launch sequence on a small case, for a profiler: decode | chunk (recurrence, time-mix mode), gla (the same
 recurrence read after its update, with low-rank decays and the head norm), latent-decode | latent (latent attention),
-hyper (residual streams: join, read, norm), window-decode | window (windowed attention with kept tokens and gates)."""
+hyper (residual streams: join, read, norm), window-decode | window (windowed attention with kept tokens and gates),
+gated-delta | general-delta (delta rules with their head norm; -decode: one token each), canon (join and convolution)."""
 import os
 import sys
 
@@ -25,6 +26,24 @@ elif case == "hyper":
     x, pre = rnd(T, S, W, dtype=torch.float32), mx.DytNorm(0.5, rnd(W), rnd(W))
     hc, out = mx.HyperW(*(torch.full(s, 0.4, device="cuda") for s in ((S,), (S,), (S, S)))), mx.SublayerOut(rnd(T, W))
     run = lambda: mx.stream_hyper(x, S, "bf16", pending=out, hc=hc, w_in=hc.w_in, pre=pre)
+elif "delta" in case:
+    from metrale_inference_alpha_b200.ops import delta as dl
+    lens, start = ([1] * 128, 63) if case.endswith("-decode") else ([4096], 0)
+    b, _ = batch(lens, start)
+    T = sum(lens)
+    q, k, v, g, a = (rnd(T, H * D) for _ in range(5))
+    ssm, A = torch.zeros(len(lens) + 2, H, D, D, device="cuda"), torch.zeros(H, device="cuda")
+    low = dl.BoundedDecay(rnd(T, 64), rnd(H * D, 64, std=0.1), rnd(H * D, dtype=torch.float32), -0.6065)
+    rule = dl.GatedRule(a[:, :H], a[:, 64:64 + H], A, A) if case.startswith("gated") else dl.GeneralRule(a, low)
+    norm = dict(w=rnd(H * D), gate=g, gate_act="silu", eps=1e-6, scale=1.0, out=torch.empty_like(g))
+    run = lambda: dl.delta_attention(q, k, v, rule, ssm, b, heads=H, dk=D, dv=D, fmt="bf16", norm=norm)
+elif case == "canon":
+    from metrale_inference_alpha_b200.ops import canon
+    T, W = 8192, 2560
+    b, _ = batch([T], 0)
+    x, y, win = rnd(T, W, dtype=torch.float32), mx.SublayerOut(rnd(T, W)), canon.Window(torch.zeros(4, 2 * W, device="cuda"), 0, W)
+    nm, filt = mx.RmsNorm(rnd(W), 1e-6, plus_one=True), rnd(3, W)
+    run = lambda: canon.stream_canon(x, "bf16", pending=y, norm=nm, filt=filt, window=win, batch=b)
 elif case.startswith("window"):
     lens, start = ([1] * 128, 1023) if case == "window-decode" else ([4096], 0)
     b, blocks = batch(lens, start)

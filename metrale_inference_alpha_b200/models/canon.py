@@ -82,7 +82,8 @@ def twin_mixer(dec, a, lw, batch, kc, vc, state, fmt: str, stash):
     norm = dict(w=R.norm, gate=g, gate_act="sigmoid", eps=dec.cfg.rms_eps, scale=w.right_scale, out=cat[:, nl:])
     if general:
         decay = BoundedDecay(_cols(y, R.at["w1"]), R.w2, R.w0, R.decay_scale, R.w2_twice)
-        rule = GeneralRule(_cols(y, R.at["a"]), decay if ws else decay.log())
+        rule = GeneralRule(_cols(y, R.at["a"]), decay)
+        rule = rule if ws else rule.logs()
         delta_attention(q, k, v, rule, state, batch, heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt, write_state=ws, norm=norm)
         if stash is not None:
             stash.later.append(lambda cb: delta_attention(q, k, v, rule, state, cb, heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt,

@@ -198,8 +198,9 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   float* sM = reinterpret_cast<float*>(sm + Lay::z1);
   float* sT = reinterpret_cast<float*>(sm + Lay::tmp);
   float* sD = reinterpret_cast<float*>(sm + Lay::vec);                         // decay of the whole chunk, [DK]
-  float* sG = sD + DK;                                                         // gated: running log2 decays, step sizes
-  float* sBeta = sG + kC;
+  // gated: running log2 decays (sums of strong decays grow; their differences must not lose the mild ones), step sizes
+  double* sG = reinterpret_cast<double*>(sD + DK);
+  float* sBeta = reinterpret_cast<float*>(sG + kC);
   float* sL = sA;                                                              // general: running logs [64][DK + 4]
   constexpr int ldl = DK + 4;
 
@@ -234,14 +235,15 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     }
   } else {
     if (tid < kC) {
-      float lg = 0.f, beta = 0.f;
+      double lg = 0.0;
+      float beta = 0.f;
       if (tid < valid) {
-        lg = in.log_gate<bf16>(t0 + tid, hd) * kLog2e;
+        lg = (double)in.log_gate<bf16>(t0 + tid, hd) * 1.4426950408889634;
         beta = in.step_size<bf16>(t0 + tid, hd);
       }
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, lg, o);
+        const double up = __shfl_up_sync(0xffffffffu, lg, o);
         if (lane >= o) lg += up;
       }
       sG[tid] = lg;
@@ -250,7 +252,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     __syncthreads();
     if (tid >= 32 && tid < kC) sG[tid] += sG[31];
     __syncthreads();
-    if (tid < DK) p.ws_d[ci * DK + tid] = ex2(sG[kC - 1]);
+    if (tid < DK) p.ws_d[ci * DK + tid] = ex2((float)sG[kC - 1]);
   }
   // ---- operands, a warp per row
   {
@@ -372,7 +374,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       const int i = i0 + g + (x >> 1) * 8, j = j0 + e * 8 + 2 * t + (x & 1);
       float dec = 1.f, beta = 1.f;
       if constexpr (!GEN) {
-        dec = j <= i ? ex2(sG[i] - sG[j]) : 0.f;
+        dec = j <= i ? ex2((float)(sG[i] - sG[j])) : 0.f;
         beta = sBeta[i];
       }
       sa[e][x] = j < i ? sa[e][x] * dec * beta : 0.f;
@@ -429,8 +431,8 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       const int i = e >> 5, j = (e & 31) * 2;
       float a = sM[i * kLdF + j], b = sM[i * kLdF + j + 1];
       if constexpr (!GEN) {
-        a *= sBeta[j] * (decayed ? ex2(sG[j]) : 1.f);
-        b *= sBeta[j + 1] * (decayed ? ex2(sG[j + 1]) : 1.f);
+        a *= sBeta[j] * (decayed ? ex2((float)sG[j]) : 1.f);
+        b *= sBeta[j + 1] * (decayed ? ex2((float)sG[j + 1]) : 1.f);
       }
       Z0.put(i, j, a, b);
     }
@@ -467,11 +469,11 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     __syncthreads();
     put_m(false);
     put_acc<NK>(XW, i0, nk0, xw, -1.f);
-    const float gl = sG[kC - 1];
+    const double gl = sG[kC - 1];
     for (int e = tid; e < kC * DK / 2; e += 256) {        // the keys decayed to the chunk's end
       const int i = e / (DK / 2), d = (e - i * (DK / 2)) * 2;
       const float2 u = U.get(i, d);
-      const float f = i < valid ? ex2(gl - sG[i]) : 0.f;
+      const float f = i < valid ? ex2((float)(gl - sG[i])) : 0.f;
       U.put(i, d, u.x * f, u.y * f);
     }
     __syncthreads();
@@ -490,7 +492,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       for (int h2 = 0; h2 < 2; ++h2) {
         const int row = i0 + g + 8 * h2;
         const float2 r = R.get(row, nk0 + i * 8 + 2 * t);
-        const float f = GEN ? 1.f : ex2(sG[row]);
+        const float f = GEN ? 1.f : ex2((float)sG[row]);
         acc[i][2 * h2] = r.x * f;
         acc[i][2 * h2 + 1] = r.y * f;
       }

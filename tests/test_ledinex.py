@@ -324,6 +324,7 @@ def rule_case(general, H, HK, dk, dv, n, fmt, strong=False):
     x = {"q": gen(n, nk, seed=1), "k": gen(n, nk, seed=2, std=1.5), "v": gen(n, H * dv, seed=3)}
     if general:
         x["a"], lw = gen(n, H * dk, seed=4, std=2.0), -0.6 * torch.sigmoid(gen(n, H * dk, seed=5, std=3.0, mean=-1.0))
+        bound = -math.inf if strong else -0.6
         if strong:
             lw = lw * 40
     else:
@@ -335,7 +336,7 @@ def rule_case(general, H, HK, dk, dv, n, fmt, strong=False):
     if general:
         want = lo.general_delta_recurrence(heads(d["q"], H, dk), heads(d["k"], H, dk), heads(d["v"], H, dv), heads(torch.exp(lw.double()), H, dk),
                                            heads(lo.sigmoid(d["a"]), H, dk))
-        return x, dict(lw=lw), want.reshape(n, -1)
+        return x, dict(lw=lw, bound=bound), want.reshape(n, -1)
     g = torch.exp(-torch.exp(A.double()) * lo.softplus(d["a"] + bias.double()))
     want = lo.gated_delta_recurrence(heads(d["q"], HK, dk), heads(d["k"], HK, dk), heads(d["v"], H, dv), g, lo.sigmoid(d["b"]))
     return x, dict(A=A, bias=bias), want.reshape(n, -1)
@@ -358,7 +359,7 @@ def run_rule(device, fmt, case, general, H, HK, dk, dv, cuts, kernel="auto", ver
         z = torch.cat([wide[lo_:lo_ + m], wide[:1]]).to(device)
         q, k, v, a, bb = (z[:, s:s + w] for s, w in spans)
         rows = torch.cat([torch.arange(lo_, lo_ + m), torch.zeros(1, dtype=torch.long)])
-        rule = dl.GeneralRule(a, c["lw"][rows].to(device).contiguous()) if general else dl.GatedRule(a, bb, c["A"].to(device), c["bias"].to(device))
+        rule = dl.GeneralRule(a, c["lw"][rows].to(device).contiguous(), c["bound"]) if general else dl.GatedRule(a, bb, c["A"].to(device), c["bias"].to(device))
         kw = dict(heads=H, key_heads=HK, dk=dk, dv=dv, fmt=fmt)
         if norm is not None:
             gate = torch.cat([norm["gate"][lo_:lo_ + m], norm["gate"][:1]]).to(device)
@@ -388,7 +389,7 @@ def test_delta_rules(device, fmt, general, H, HK, dk, dv, strong):
     n = 70
     case = rule_case(general, H, HK, dk, dv, n, fmt, strong)
     for cuts, verify in (([n], ()), ([1], ()), ([33, 1, 2, 17], ()), ([16, 5, 5, 40], (1, 2))):
-        close(run_rule(device, fmt, case, general, H, HK, dk, dv, cuts, verify=verify), case[2], 1e-5)
+        close(run_rule(device, fmt, case, general, H, HK, dk, dv, cuts, verify=verify), case[2], 1e-5 if fmt == "fp32" else 3e-5)
 
 
 @pytest.mark.parametrize("device", DEVICES)
@@ -403,6 +404,50 @@ def test_delta_rules_with_head_norm(device, fmt, general, H, HK, dk, dv):
     want = 0.8 * (lo.unit_rms(case[2].view(n, H, dv), 1e-3).reshape(n, -1) * norm["w"].double() * (lo.sigmoid(z) if general else lo.silu(z)))
     for cuts in ([n], [1], [20, 1]):
         close(run_rule(device, fmt, case, general, H, HK, dk, dv, cuts, norm=norm), want, 1e-4 if fmt == "fp32" else 8e-3)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("general,H,HK,dk,dv", [(False, 4, 2, 64, 64), (False, 2, 1, 64, 128), (False, 2, 2, 128, 64), (False, 3, 1, 128, 128),
+                                                (True, 3, 3, 64, 64), (True, 2, 2, 128, 128)])
+@pytest.mark.parametrize("norm", [False, True])
+@pytest.mark.parametrize("strong", [False, True])
+def test_chunked_delta_rules(general, H, HK, dk, dv, norm, strong):
+    """Several chunks, ragged ends, a carried state, a second sequence of one token beside it; the head norm inside."""
+    if general and strong:
+        pytest.skip("decays past the chunked kernels' range are served token by token")
+    n = 250
+    case = rule_case(general, H, HK, dk, dv, n, "bf16", strong)
+    nm, want, tol = None, case[2], 4e-5
+    if norm:
+        nm = dict(w=b16(gen(H * dv, seed=9, mean=1.0)), gate=b16(gen(n, H * dv, seed=10)), act="sigmoid" if general else "silu")
+        z = nm["gate"].double()
+        want = 0.8 * (lo.unit_rms(want.view(n, H, dv), 1e-3).reshape(n, -1) * nm["w"].double() * (lo.sigmoid(z) if general else lo.silu(z)))
+        tol = 8e-3
+    for cuts in ([n], [64, 186], [1, 65, 63, 100], [130, 1]):
+        got = run_rule("cuda", "bf16", case, general, H, HK, dk, dv, cuts, kernel="chunked", norm=nm)
+        close(got, want, tol)
+    ops.check_status("cuda")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("general", [False, True])
+def test_chunked_rule_with_repeated_keys(general):
+    """The hardest systems of a chunk: the same key in every row, full step sizes and removal rates, hardly any decay."""
+    n, H, d = 200, 2, 64
+    x, c, _ = rule_case(general, H, H, d, d, n, "bf16")
+    x["k"][:] = x["k"][:1] * 0.5
+    x["a"][:] = 6.0 if general else -9.0
+    dbl = {k: t.double().view(n, H, -1) for k, t in x.items()}
+    if general:
+        c["lw"][:] = -1e-3
+        want = lo.general_delta_recurrence(dbl["q"], dbl["k"], dbl["v"], torch.exp(c["lw"].double()).view(n, H, d), lo.sigmoid(dbl["a"]))
+    else:
+        x["b"][:] = 6.0
+        g = torch.exp(-torch.exp(c["A"].double()) * lo.softplus(x["a"].double() + c["bias"].double()))
+        want = lo.gated_delta_recurrence(dbl["q"], dbl["k"], dbl["v"], g, lo.sigmoid(x["b"].double()))
+    case = x, c, want.reshape(n, -1)
+    for kernel in ("chunked", "seq"):
+        close(run_rule("cuda", "bf16", case, general, H, H, d, d, [n], kernel=kernel), case[2], 5e-4 if kernel == "chunked" else 1e-5)
 
 
 def test_the_general_rule_reads_the_old_state_and_writes_the_key_itself():
