@@ -14,14 +14,15 @@
 //   gated    (G the running sums of one log2 decay per token; d = 2^G_last)
 //     A_ij = beta_i 2^(G_i - G_j) k_i.k_j (j < i)   Xw = -M diag(beta 2^G) K   Xu = M diag(beta) V
 //     Q_ij = 2^(G_i - G_j) q_i.k_j (j <= i)         R' = diag(2^G) q + Q Xw    O' = Q Xu
-//     T = (2^(G_last - G) k)^T Xw                   E = (2^(G_last - G) k)^T Xu
+//     T = k^T diag(2^(G_last - G)) Xw               E = k^T diag(2^(G_last - G)) Xu
 //     Every exponent is <= 0 however strong the decay.
 // Three launches for the whole ragged batch:
 //   delta_prep  per (chunk, head, sequence): all of the above into a workspace
-//   delta_scan  per (32 value columns, head, sequence): the recurrence over chunks, S in registers; leaves every chunk's
+//   delta_scan  per (16 or 32 value columns, head, sequence): the recurrence over chunks, S in registers; leaves every chunk's
 //               start state as two bf16 planes (value and remainder), the final state in the pool
 //   delta_out   per (chunk, head, sequence): o, optionally finished by the head's gated RMS norm
-// Values are exact bf16 operands; every other one is 32-bit and enters as value + remainder (16 mantissa bits), so a product
+// Values are exact bf16 operands, and so are the gated rule's queries and keys (their lengths enter as factors, above
+// written into k and q); every other one is 32-bit and enters as value + remainder (16 mantissa bits), so a product
 // costs two or three passes and keeps 32-bit quantities 32-bit to a few 1e-6. The triangular inverse is fp32, by 16 x 16
 // blocks. Head sizes 64 and 128. Sequence s keeps its chunks from index q_start[s] / 64 + s on, which never overlaps.
 #include "common.cuh"
@@ -111,9 +112,9 @@ struct Planes {
   }
 };
 
-// acc (16 rows m0 .., 8 N8 columns n0 ..) += A B over k in [k0, k1): A is [row][k], or [k][row] with AT; B is [k][column],
-// exact (one plane) without BL
-template <int N8, bool AT, bool BL>
+// acc (16 rows m0 .., 8 N8 columns n0 ..) += A B over k in [k0, k1): A is [row][k], or [k][row] with AT; B is [k][column];
+// exact (one plane) without AL, BL
+template <int N8, bool AT, bool BL, bool AL = true>
 __device__ __forceinline__ void mm(float (*acc)[4], const Planes& A, int m0, const Planes& B, int n0, int k0, int k1) {
   const int lane = threadIdx.x & 31;
 #pragma unroll 2
@@ -122,11 +123,11 @@ __device__ __forceinline__ void mm(float (*acc)[4], const Planes& A, int m0, con
     if constexpr (AT) {
       const size_t o = (size_t)(k + (lane >> 4) * 8 + (lane & 7)) * A.ld + m0 + ((lane >> 3) & 1) * 8;
       ldsm4t(ah, A.hi + o);
-      ldsm4t(al, A.lo + o);
+      if constexpr (AL) ldsm4t(al, A.lo + o);
     } else {
       const size_t o = (size_t)(m0 + (lane & 15)) * A.ld + k + (lane >> 4) * 8;
       ldsm4(ah, A.hi + o);
-      ldsm4(al, A.lo + o);
+      if constexpr (AL) ldsm4(al, A.lo + o);
     }
 #pragma unroll
     for (int i = 0; i < N8; i += 2) {
@@ -135,8 +136,10 @@ __device__ __forceinline__ void mm(float (*acc)[4], const Planes& A, int m0, con
       ldsm4t(b, B.hi + o);
       mma(acc[i], ah, b[0], b[1]);
       mma(acc[i + 1], ah, b[2], b[3]);
-      mma(acc[i], al, b[0], b[1]);
-      mma(acc[i + 1], al, b[2], b[3]);
+      if constexpr (AL) {
+        mma(acc[i], al, b[0], b[1]);
+        mma(acc[i + 1], al, b[2], b[3]);
+      }
       if constexpr (BL) {
         ldsm4t(b, B.lo + o);
         mma(acc[i], ah, b[0], b[1]);
@@ -173,7 +176,7 @@ struct PrepLayout {
   static constexpr size_t plane_k = (size_t)kC * ldk * 2, plane_x = (size_t)kC * ldx * 2;
   static constexpr size_t u = 0, r = 2 * plane_k, b = 4 * plane_k, k = 6 * plane_k, v = k + 2 * plane_x, z0 = v + (size_t)kC * ldv * 2;
   static constexpr size_t zsize = 2 * (size_t)kC * kLdC * 2;                   // two planes of a 64 x 64 matrix, or one in fp32
-  static constexpr size_t z1 = z0 + zsize, tmp = z1 + zsize, vec = tmp + 3 * 16 * 17 * 4, bytes = vec + (DK + 4 * kC) * 4;
+  static constexpr size_t z1 = z0 + zsize, tmp = z1 + zsize, vec = tmp + 3 * 16 * 17 * 4, bytes = vec + (DK + 5 * kC) * 4;
   static_assert(2 * zsize >= (size_t)kC * (DK + 4) * 4, "the running logs live where the 64 x 64 matrices come later");
   static_assert(zsize >= (size_t)kC * kLdF * 4, "");
 };
@@ -201,6 +204,8 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   // gated: running log2 decays (sums of strong decays grow; their differences must not lose the mild ones), step sizes
   double* sG = reinterpret_cast<double*>(sD + DK);
   float* sBeta = reinterpret_cast<float*>(sG + kC);
+  float* sNk = sBeta + kC;                                                     // gated: one over the lengths of keys and queries
+  float* sNq = sNk + kC;
   float* sL = sA;                                                              // general: running logs [64][DK + 4]
   constexpr int ldl = DK + 4;
 
@@ -307,16 +312,21 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       } else {
         const float nq = rsqrtf(mb::warp_sum(sq) + mb::kUnitEps) * rsqrtf((float)DK);
 #pragma unroll
-        for (int e = 0; e < E; e += 2) {
-          U.put(i, d0 + e, k[e] * nk, k[e + 1] * nk);
-          R.put(i, d0 + e, q[e] * nq, q[e + 1] * nq);
+        for (int e = 0; e < E; e += 2) {                  // as they are, exact; their lengths enter the scores
+          *reinterpret_cast<__nv_bfloat162*>(U.hi + i * Lay::ldk + d0 + e) = __floats2bfloat162_rn(k[e], k[e + 1]);
+          *reinterpret_cast<__nv_bfloat162*>(R.hi + i * Lay::ldk + d0 + e) = __floats2bfloat162_rn(q[e], q[e + 1]);
+        }
+        if (lane == 0) {
+          sNk[i] = nk;
+          sNq[i] = nq;
         }
       }
     }
   }
   __syncthreads();
   // ---- scores of this warp's 16 rows and 32 columns, blocks up to the diagonal: rows U and R against columns B (and K)
-  const int rb = warp & 3, half = warp >> 2, i0 = rb * 16, j0 = half * 32;
+  // (warps w and w + 4 share a scheduler: a long row block of a triangle goes with a short one)
+  const int half = warp >> 2, rb = half ? 3 - (warp & 3) : warp & 3, i0 = rb * 16, j0 = half * 32;
   float sa[4][4], sb[GEN ? 4 : 1][4], sp[GEN ? 4 : 1][4], sq[4][4];
   zero<4>(sa);
   zero<4>(sq);
@@ -331,24 +341,28 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       uint32_t uh[4], ul[4], rh[4], rl[4];
       const size_t o = (size_t)(i0 + (lane & 15)) * Lay::ldk + k0 + (lane >> 4) * 8;
       ldsm4(uh, U.hi + o);
-      ldsm4(ul, U.lo + o);
       ldsm4(rh, R.hi + o);
-      ldsm4(rl, R.lo + o);
+      if constexpr (GEN) {
+        ldsm4(ul, U.lo + o);
+        ldsm4(rl, R.lo + o);
+      }
 #pragma unroll
       for (int jb = 0; jb < 2; ++jb) {
         if (j0 + jb * 16 > i0) continue;
         const int row = j0 + jb * 16 + (lane & 7) + ((lane >> 4) << 3), col = k0 + ((lane >> 3) & 1) * 8;
         uint32_t bh[4], bl[4];
         ldsm4(bh, CB.hi + (size_t)row * CB.ld + col);
-        ldsm4(bl, CB.lo + (size_t)row * CB.ld + col);
+        if constexpr (GEN) ldsm4(bl, CB.lo + (size_t)row * CB.ld + col);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           mma(sa[jb * 2 + e], uh, bh[2 * e], bh[2 * e + 1]);
           mma(sq[jb * 2 + e], rh, bh[2 * e], bh[2 * e + 1]);
-          mma(sa[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
-          mma(sq[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
-          mma(sa[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
-          mma(sq[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+          if constexpr (GEN) {
+            mma(sa[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
+            mma(sq[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
+            mma(sa[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
+            mma(sq[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+          }
         }
         if constexpr (GEN) {
           ldsm4(bh, K.hi + (size_t)row * K.ld + col);
@@ -372,13 +386,14 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
       const int i = i0 + g + (x >> 1) * 8, j = j0 + e * 8 + 2 * t + (x & 1);
-      float dec = 1.f, beta = 1.f;
+      float fa = 1.f, fq = 1.f;
       if constexpr (!GEN) {
-        dec = j <= i ? ex2((float)(sG[i] - sG[j])) : 0.f;
-        beta = sBeta[i];
+        const float dec = j <= i ? ex2((float)(sG[i] - sG[j])) * sNk[j] : 0.f;
+        fa = dec * sBeta[i] * sNk[i];
+        fq = dec * sNq[i];
       }
-      sa[e][x] = j < i ? sa[e][x] * dec * beta : 0.f;
-      sq[e][x] = j <= i ? sq[e][x] * dec : 0.f;
+      sa[e][x] = j < i ? sa[e][x] * fa : 0.f;
+      sq[e][x] = j <= i ? sq[e][x] * fq : 0.f;
       if constexpr (GEN) {
         sb[e][x] = j < i ? sb[e][x] : 0.f;
         sp[e][x] = j <= i ? sp[e][x] : 0.f;
@@ -425,14 +440,14 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       __syncthreads();
     }
   }
-  // M as planes; gated: times diag(beta 2^G) for Xw, diag(beta) for Xu
+  // M as planes; gated: times diag(beta 2^G / |k|) for Xw, diag(beta) for Xu
   auto put_m = [&](bool decayed) {
     for (int e = tid; e < kC * kC / 2; e += 256) {
       const int i = e >> 5, j = (e & 31) * 2;
       float a = sM[i * kLdF + j], b = sM[i * kLdF + j + 1];
       if constexpr (!GEN) {
-        a *= sBeta[j] * (decayed ? ex2((float)sG[j]) : 1.f);
-        b *= sBeta[j + 1] * (decayed ? ex2((float)sG[j + 1]) : 1.f);
+        a *= sBeta[j] * (decayed ? ex2((float)sG[j]) * sNk[j] : 1.f);
+        b *= sBeta[j + 1] * (decayed ? ex2((float)sG[j + 1]) * sNk[j + 1] : 1.f);
       }
       Z0.put(i, j, a, b);
     }
@@ -446,7 +461,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   float xw[NK][4], xu[NV][4];
   zero<NK>(xw);
   zero<NV>(xu);
-  mm<NK, false, true>(xw, Z0, i0, U, nk0, 0, kend);
+  mm<NK, false, GEN>(xw, Z0, i0, U, nk0, 0, kend);
   const Planes& XW = GEN ? U : B;
   float po[NV][4];                                        // O'
   zero<NV>(po);
@@ -469,13 +484,6 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     __syncthreads();
     put_m(false);
     put_acc<NK>(XW, i0, nk0, xw, -1.f);
-    const double gl = sG[kC - 1];
-    for (int e = tid; e < kC * DK / 2; e += 256) {        // the keys decayed to the chunk's end
-      const int i = e / (DK / 2), d = (e - i * (DK / 2)) * 2;
-      const float2 u = U.get(i, d);
-      const float f = i < valid ? ex2((float)(gl - sG[i])) : 0.f;
-      U.put(i, d, u.x * f, u.y * f);
-    }
     __syncthreads();
     mm<NV, false, false>(xu, Z0, i0, V, nv0, 0, kend);
     __syncthreads();
@@ -491,8 +499,14 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
 #pragma unroll
       for (int h2 = 0; h2 < 2; ++h2) {
         const int row = i0 + g + 8 * h2;
-        const float2 r = R.get(row, nk0 + i * 8 + 2 * t);
-        const float f = GEN ? 1.f : ex2((float)sG[row]);
+        float2 r;
+        float f = 1.f;
+        if constexpr (GEN) {
+          r = R.get(row, nk0 + i * 8 + 2 * t);
+        } else {
+          r = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(R.hi + row * Lay::ldk + nk0 + i * 8 + 2 * t));
+          f = ex2((float)sG[row]) * sNq[row];
+        }
         acc[i][2 * h2] = r.x * f;
         acc[i][2 * h2 + 1] = r.y * f;
       }
@@ -520,7 +534,20 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       *reinterpret_cast<float2*>(go + (size_t)(i0 + g + 8) * DV + nv0 + i * 8 + 2 * t) = make_float2(po[i][2], po[i][3]);
     }
   }
-  mm<NE, true, true>(acc_e, GEN ? B : U, m0, K, e0, 0, kC);
+  if constexpr (!GEN) {                                   // rows of X decayed to the chunk's end and over the keys' lengths, in place
+    __syncthreads();
+    const double gl = sG[kC - 1];
+    for (int e = tid; e < kC * (DK + DV) / 2; e += 256) {
+      const int i = e / ((DK + DV) / 2), d = (e - i * ((DK + DV) / 2)) * 2;
+      const float f = i < valid ? ex2((float)(gl - sG[i])) * sNk[i] : 0.f;
+      const Planes& X = d < DK ? XW : K;
+      const int cc = d < DK ? d : d - DK;
+      const float2 x = X.get(i, cc);
+      X.put(i, cc, x.x * f, x.y * f);
+    }
+    __syncthreads();
+  }
+  mm<NE, true, true, GEN>(acc_e, GEN ? B : U, m0, K, e0, 0, kC);
   const float d0 = GEN ? sD[m0 + g] : 1.f, d1 = GEN ? sD[m0 + g + 8] : 1.f;
   {
     float* ge = p.ws_e + ci * DK * DV;
@@ -532,7 +559,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   }
   float acc_t[NT][4];
   zero<NT>(acc_t);
-  mm<NT, true, true>(acc_t, GEN ? B : U, m0, XW, x0, 0, kC);
+  mm<NT, true, true, GEN>(acc_t, GEN ? B : U, m0, XW, x0, 0, kC);
 #pragma unroll
   for (int i = 0; i < NT; ++i) {
     acc_t[i][0] *= d0; acc_t[i][1] *= d0; acc_t[i][2] *= d1; acc_t[i][3] *= d1;
@@ -542,17 +569,16 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
 }
 
 // ------------------------------------------------------------------ recurrence over chunks
-constexpr int kSlice = 32;         // value columns per CTA
-
-template <int DK>
+// SLICE value columns per CTA: 32, or 16 where those CTAs, too, have an SM each
+template <int DK, int SLICE>
 struct ScanLayout {
-  static constexpr int ldt = DK + 8, lds = kSlice + 8;
+  static constexpr int ldt = DK + 8, lds = SLICE + 8;
   static constexpr size_t t_stage = 2 * (size_t)DK * ldt * 2, s = 2 * t_stage, bytes = s + 2 * (size_t)DK * lds * 2;
 };
 
-template <int DK, int DV>
+template <int DK, int DV, int SLICE>
 __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p) {
-  using Lay = ScanLayout<DK>;
+  using Lay = ScanLayout<DK, SLICE>;
   extern __shared__ __align__(16) uint8_t sm[];
   const int slice = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   mb::pdl_wait();
@@ -564,9 +590,9 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
     if (p.status && tid == 0) atomicCAS(p.status, 0u, MB_ST_BOUNDS);
     return;
   }
-  const int chunks = (n + kC - 1) / kC, c0 = slice * kSlice;
+  const int chunks = (n + kC - 1) / kC, c0 = slice * SLICE;
   const size_t first = (size_t)(p.q_start[seq] / kC + seq);
-  constexpr int kMB = DK / 16, kCW = 8 / kMB, N8 = kSlice / 8 / kCW;
+  constexpr int kMB = DK / 16, kThreads = SLICE == 32 || DK == 128 ? 256 : 128, kCW = kThreads / 32 / kMB, N8 = SLICE / 8 / kCW;
   const int m0 = (warp % kMB) * 16, n0 = (warp / kMB) * N8 * 8;
   const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
   auto stage = [&](int c) {
@@ -577,7 +603,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
     if (c < chunks) {
       const Planes d = stage(c);
       const bf16* src = p.ws_t + ((first + c) * H + hd) * 2 * DK * DK;
-      for (int i = tid; i < 2 * DK * (DK / 8); i += 256) {
+      for (int i = tid; i < 2 * DK * (DK / 8); i += kThreads) {
         const int pl = i / (DK * (DK / 8)), e = i - pl * (DK * (DK / 8)), r = e / (DK / 8), cc = (e - r * (DK / 8)) * 8;
         cp16((pl ? d.lo : d.hi) + r * Lay::ldt + cc, src + (size_t)i * 8, true);
       }
@@ -722,18 +748,27 @@ __global__ void __launch_bounds__(256, 2) delta_out_kernel(const ChunkParams p) 
 
 template <int DK, int DV, bool GEN>
 int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_t stream) {
-  constexpr size_t sp = PrepLayout<DK, DV>::bytes, ss = ScanLayout<DK>::bytes, so = OutLayout<DK, DV>::bytes;
+  constexpr size_t sp = PrepLayout<DK, DV>::bytes, so = OutLayout<DK, DV>::bytes;
   static bool configured = false;
+  static int sms = 0;
   if (!configured) {
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) sms = 148;
     cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<DK, DV, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sp);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_scan_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ss);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_scan_kernel<DK, DV, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ScanLayout<DK, 32>::bytes);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_scan_kernel<DK, DV, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ScanLayout<DK, 16>::bytes);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_out_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)so);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   const dim3 grid((max_q_len + kC - 1) / kC, p.in.H, num_seqs);
   cudaError_t e = mb::launch_kernel(delta_prep_kernel<DK, DV, GEN>, grid, dim3(256), sp, stream, p);
-  if (e == cudaSuccess) e = mb::launch_kernel(delta_scan_kernel<DK, DV>, dim3(DV / kSlice, p.in.H, num_seqs), dim3(256), ss, stream, p);
+  if (e == cudaSuccess) {
+    if ((long long)DV / 16 * p.in.H * num_seqs <= sms)
+      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 16>, dim3(DV / 16, p.in.H, num_seqs), dim3(DK == 128 ? 256 : 128), ScanLayout<DK, 16>::bytes, stream, p);
+    else
+      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 32>, dim3(DV / 32, p.in.H, num_seqs), dim3(256), ScanLayout<DK, 32>::bytes, stream, p);
+  }
   if (e == cudaSuccess) e = mb::launch_kernel(delta_out_kernel<DK, DV>, grid, dim3(256), so, stream, p);
   return (int)e;
 }
