@@ -40,11 +40,12 @@ struct ChunkParams {
   DeltaInputs in;
   float* state;                // [slots, H, DK, DV]
   float* out;                  // [T, H DV], or null with a norm
-  bf16* ws_t;                  // [chunks, H, 2 planes, DK, DK]
-  float* ws_e;                 // [chunks, H, DK, DV]
+  // T, R', E and O' are kept as the tensor cores' fragments, a warp's accumulators one vector per lane: see put_frag, put_c
+  uint4* ws_t;                 // [chunks, H] of DK x DK, two planes
+  float4* ws_e;                // [chunks, H] of DK x DV
   bf16* ws_s;                  // [chunks, H, 2 planes, DK, DV] start states
-  bf16* ws_r;                  // [chunks, H, 2 planes, 64, DK]
-  float* ws_o;                 // [chunks, H, 64, DV]
+  uint4* ws_r;                 // [chunks, H] of 64 x DK, two planes
+  float4* ws_o;                // [chunks, H] of 64 x DV
   float* ws_d;                 // [chunks, H, DK]
   const int* q_start;
   const int* q_len;
@@ -166,6 +167,63 @@ __device__ __forceinline__ void put_acc(const Planes& P, int m0, int n0, const f
   }
 }
 
+// Fragments: a 16 x 16 block of an A operand is four registers per lane, which are the accumulators of two neighbouring
+// 8-column tiles. Block (row block, column block) of a matrix of `blocks` column blocks: value plane, then remainder, a
+// 16-byte vector per lane.
+template <int N8>
+__device__ __forceinline__ void put_frag(uint4* dst, int blocks, int m0, int n0, const float (*acc)[4]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < N8; i += 2) {
+    uint4 h, l;
+    split2(acc[i][0], acc[i][1], h.x, l.x);
+    split2(acc[i][2], acc[i][3], h.y, l.y);
+    split2(acc[i + 1][0], acc[i + 1][1], h.z, l.z);
+    split2(acc[i + 1][2], acc[i + 1][3], h.w, l.w);
+    uint4* d = dst + ((size_t)((m0 >> 4) * blocks + (n0 >> 4) + (i >> 1)) * 2) * 32 + lane;
+    d[0] = h;
+    d[32] = l;
+  }
+}
+// acc += A B with A's blocks as above, `frag` at this warp's row of blocks
+template <int N8>
+__device__ __forceinline__ void mm_frag(float (*acc)[4], const uint4* frag, const Planes& B, int n0, int blocks) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll 2
+  for (int kb = 0; kb < blocks; ++kb) {
+    const uint4 h = frag[kb * 64 + lane], l = frag[kb * 64 + 32 + lane];
+    const uint32_t ah[4] = {h.x, h.y, h.z, h.w}, al[4] = {l.x, l.y, l.z, l.w};
+#pragma unroll
+    for (int i = 0; i < N8; i += 2) {
+      uint32_t b[4];
+      const size_t o = (size_t)(kb * 16 + (lane & 15)) * B.ld + n0 + i * 8 + (lane >> 4) * 8;
+      ldsm4t(b, B.hi + o);
+      mma(acc[i], ah, b[0], b[1]);
+      mma(acc[i + 1], ah, b[2], b[3]);
+      mma(acc[i], al, b[0], b[1]);
+      mma(acc[i + 1], al, b[2], b[3]);
+      ldsm4t(b, B.lo + o);
+      mma(acc[i], ah, b[0], b[1]);
+      mma(acc[i + 1], ah, b[2], b[3]);
+    }
+  }
+}
+// accumulators of 8-column tiles, tile (row block, column tile) of a matrix of `tiles` column tiles a vector per lane
+template <int N8>
+__device__ __forceinline__ void put_c(float4* dst, int tiles, int m0, int n0, const float (*acc)[4]) {
+#pragma unroll
+  for (int i = 0; i < N8; ++i)
+    dst[(size_t)((m0 >> 4) * tiles + (n0 >> 3) + i) * 32 + (threadIdx.x & 31)] = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+template <int N8>
+__device__ __forceinline__ void get_c(const float4* src, int tiles, int m0, int n0, float (*acc)[4]) {
+#pragma unroll
+  for (int i = 0; i < N8; ++i) {
+    const float4 v = src[(size_t)((m0 >> 4) * tiles + (n0 >> 3) + i) * 32 + (threadIdx.x & 31)];
+    acc[i][0] = v.x; acc[i][1] = v.y; acc[i][2] = v.z; acc[i][3] = v.w;
+  }
+}
+
 // ------------------------------------------------------------------ per-chunk preparation
 constexpr int kLdF = kC + 4;       // fp32 rows of the inverse
 constexpr int kLdC = kC + 8;       // bf16 rows of 64 x 64 matrices
@@ -209,21 +267,37 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   float* sL = sA;                                                              // general: running logs [64][DK + 4]
   constexpr int ldl = DK + 4;
 
-  // values, exact
-  for (int i = tid; i < kC * (DV / 8); i += 256) {
-    const int r = i / (DV / 8), cc = (i - r * (DV / 8)) * 8;
-    const bool ok = r < valid;
-    cp16(V.hi + r * Lay::ldv + cc, reinterpret_cast<const bf16*>(in.v) + (ok ? (size_t)(t0 + r) * in.v_ld + (size_t)hd * DV + cc : 0), ok);
+  // everything the chunk reads, at once: values and the raw rows of keys, queries and removal logits (a row's owner makes
+  // its operands of them in place), log decays
+  auto rows_in = [&](const void* base, long long ld, int head, int D, bf16* dst, int dst_ld) {
+    for (int i = tid; i < kC * (D / 8); i += 256) {
+      const int r = i / (D / 8), cc = (i - r * (D / 8)) * 8;
+      const bool ok = r < valid;
+      cp16(dst + r * dst_ld + cc, reinterpret_cast<const bf16*>(base) + (ok ? (size_t)(t0 + r) * ld + (size_t)head * D + cc : 0), ok);
+    }
+  };
+  const int hk = hd / (H / in.HK);
+  rows_in(in.k, in.k_ld, hk, DK, U.hi, Lay::ldk);
+  rows_in(in.q, in.q_ld, hk, DK, R.hi, Lay::ldk);
+  rows_in(in.v, in.v_ld, hd, DV, V.hi, Lay::ldv);
+  if constexpr (GEN) {
+    rows_in(in.removal, in.removal_ld, hd, DK, B.hi, Lay::ldk);
+    for (int i = tid; i < kC * (DK / 4); i += 256) {
+      const int r = i / (DK / 4), cc = (i - r * (DK / 4)) * 4;
+      const bool ok = r < valid;
+      cp16(sL + r * ldl + cc, in.log_w + (ok ? ((size_t)(t0 + r) * H + hd) * DK + cc : 0), ok);
+    }
   }
   cp_commit();
   if constexpr (GEN) {
     // running sums of log2 decays; rows past `valid` repeat the last
     constexpr int kR = kC * DK / 256;
     const int d = tid % DK, grp = tid / DK, r0 = grp * kR;
-    const float* lw = in.log_w + ((size_t)t0 * H + hd) * DK + d;
+    cp_wait<0>();
+    __syncthreads();
     float v[kR];
 #pragma unroll
-    for (int i = 0; i < kR; ++i) v[i] = r0 + i < valid ? lw[(size_t)(r0 + i) * H * DK] * kLog2e : 0.f;
+    for (int i = 0; i < kR; ++i) v[i] = sL[(r0 + i) * ldl + d] * kLog2e;
 #pragma unroll
     for (int i = 1; i < kR; ++i) v[i] += v[i - 1];
     sL[(r0 + kR - 1) * ldl + d] = v[kR - 1];
@@ -258,13 +332,14 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     if (tid >= 32 && tid < kC) sG[tid] += sG[31];
     __syncthreads();
     if (tid < DK) p.ws_d[ci * DK + tid] = ex2((float)sG[kC - 1]);
+    cp_wait<0>();
+    __syncthreads();
   }
   // ---- operands, a warp per row
   {
     constexpr int E = DK / 32;
-    const int d0 = lane * E, hk = hd / (H / in.HK);
-    auto load = [&](const void* base, long long ld, int head, int row, float* o) {
-      const bf16* src = reinterpret_cast<const bf16*>(base) + (size_t)(t0 + row) * ld + (size_t)head * DK + d0;
+    const int d0 = lane * E;
+    auto load = [&](const bf16* src, float* o) {
       if constexpr (E == 4) {
         const uint2 w = *reinterpret_cast<const uint2*>(src);
         const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.x));
@@ -278,13 +353,9 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
 #pragma unroll 2
     for (int i = warp; i < kC; i += 8) {
       float q[E], k[E], a[E];
-#pragma unroll
-      for (int e = 0; e < E; ++e) q[e] = k[e] = a[e] = 0.f;
-      if (i < valid) {
-        load(in.q, in.q_ld, hk, i, q);
-        load(in.k, in.k_ld, hk, i, k);
-        if constexpr (GEN) load(in.removal, in.removal_ld, hd, i, a);
-      }
+      load(R.hi + i * Lay::ldk + d0, q);
+      load(U.hi + i * Lay::ldk + d0, k);
+      if constexpr (GEN) load(B.hi + i * Lay::ldk + d0, a);
       float sq = 0.f, sk = 0.f;
 #pragma unroll
       for (int e = 0; e < E; ++e) {
@@ -311,12 +382,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
         }
       } else {
         const float nq = rsqrtf(mb::warp_sum(sq) + mb::kUnitEps) * rsqrtf((float)DK);
-#pragma unroll
-        for (int e = 0; e < E; e += 2) {                  // as they are, exact; their lengths enter the scores
-          *reinterpret_cast<__nv_bfloat162*>(U.hi + i * Lay::ldk + d0 + e) = __floats2bfloat162_rn(k[e], k[e + 1]);
-          *reinterpret_cast<__nv_bfloat162*>(R.hi + i * Lay::ldk + d0 + e) = __floats2bfloat162_rn(q[e], q[e + 1]);
-        }
-        if (lane == 0) {
+        if (lane == 0) {                                  // the rows stay as they are, exact; their lengths enter the scores
           sNk[i] = nk;
           sNq[i] = nq;
         }
@@ -453,7 +519,6 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     }
   };
   put_m(true);
-  cp_wait<0>();
   __syncthreads();
   // ---- Xw = -M U and Xu; this warp's 16 rows and one half of the columns
   constexpr int NK = DK / 16, NV = DV / 16;
@@ -511,8 +576,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
         acc[i][2 * h2 + 1] = r.y * f;
       }
     mm<NK, false, true>(acc, Z0, i0, XW, nk0, 0, kend);
-    bf16* gr = p.ws_r + ci * 2 * kC * DK;
-    put_acc<NK>(Planes{gr, gr + kC * DK, DK}, i0, nk0, acc, 1.f);
+    put_frag<NK>(p.ws_r + ci * (kC * DK / 4), DK / 16, i0, nk0, acc);
   }
   // ---- the state's side: 16 key rows per warp (and, for 64 of them, half of the columns)
   constexpr int kMB = DK / 16, kCW = 8 / kMB, NE = DV / 8 / kCW, NT = DK / 8 / kCW;
@@ -526,14 +590,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     __syncthreads();
   }
   mm<NV, false, true>(po, Z0, i0, K, nv0, 0, kend);        // O' += Q Xu
-  {
-    float* go = p.ws_o + ci * kC * DV;
-#pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      *reinterpret_cast<float2*>(go + (size_t)(i0 + g) * DV + nv0 + i * 8 + 2 * t) = make_float2(po[i][0], po[i][1]);
-      *reinterpret_cast<float2*>(go + (size_t)(i0 + g + 8) * DV + nv0 + i * 8 + 2 * t) = make_float2(po[i][2], po[i][3]);
-    }
-  }
+  put_c<NV>(p.ws_o + ci * (kC * DV / 4), DV / 8, i0, nv0, po);
   if constexpr (!GEN) {                                   // rows of X decayed to the chunk's end and over the keys' lengths, in place
     __syncthreads();
     const double gl = sG[kC - 1];
@@ -549,14 +606,11 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   }
   mm<NE, true, true, GEN>(acc_e, GEN ? B : U, m0, K, e0, 0, kC);
   const float d0 = GEN ? sD[m0 + g] : 1.f, d1 = GEN ? sD[m0 + g + 8] : 1.f;
-  {
-    float* ge = p.ws_e + ci * DK * DV;
 #pragma unroll
-    for (int i = 0; i < NE; ++i) {
-      *reinterpret_cast<float2*>(ge + (size_t)(m0 + g) * DV + e0 + i * 8 + 2 * t) = make_float2(acc_e[i][0] * d0, acc_e[i][1] * d0);
-      *reinterpret_cast<float2*>(ge + (size_t)(m0 + g + 8) * DV + e0 + i * 8 + 2 * t) = make_float2(acc_e[i][2] * d1, acc_e[i][3] * d1);
-    }
+  for (int i = 0; i < NE; ++i) {
+    acc_e[i][0] *= d0; acc_e[i][1] *= d0; acc_e[i][2] *= d1; acc_e[i][3] *= d1;
   }
+  put_c<NE>(p.ws_e + ci * (DK * DV / 4), DV / 8, m0, e0, acc_e);
   float acc_t[NT][4];
   zero<NT>(acc_t);
   mm<NT, true, true, GEN>(acc_t, GEN ? B : U, m0, XW, x0, 0, kC);
@@ -564,16 +618,15 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   for (int i = 0; i < NT; ++i) {
     acc_t[i][0] *= d0; acc_t[i][1] *= d0; acc_t[i][2] *= d1; acc_t[i][3] *= d1;
   }
-  bf16* gt = p.ws_t + ci * 2 * DK * DK;
-  put_acc<NT>(Planes{gt, gt + DK * DK, DK}, m0, x0, acc_t, 1.f);
+  put_frag<NT>(p.ws_t + ci * (DK * DK / 4), DK / 16, m0, x0, acc_t);
 }
 
 // ------------------------------------------------------------------ recurrence over chunks
 // SLICE value columns per CTA: 32, or 16 where those CTAs, too, have an SM each
 template <int DK, int SLICE>
 struct ScanLayout {
-  static constexpr int ldt = DK + 8, lds = SLICE + 8;
-  static constexpr size_t t_stage = 2 * (size_t)DK * ldt * 2, s = 2 * t_stage, bytes = s + 2 * (size_t)DK * lds * 2;
+  static constexpr int lds = SLICE + 8;
+  static constexpr size_t t_stage = (size_t)DK * DK * 4, s = 2 * t_stage, bytes = s + 2 * (size_t)DK * lds * 2;
 };
 
 template <int DK, int DV, int SLICE>
@@ -595,18 +648,11 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
   constexpr int kMB = DK / 16, kThreads = SLICE == 32 || DK == 128 ? 256 : 128, kCW = kThreads / 32 / kMB, N8 = SLICE / 8 / kCW;
   const int m0 = (warp % kMB) * 16, n0 = (warp / kMB) * N8 * 8;
   const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
-  auto stage = [&](int c) {
-    bf16* base = reinterpret_cast<bf16*>(sm + (c & 1) * Lay::t_stage);
-    return Planes{base, base + DK * Lay::ldt, Lay::ldt};
-  };
   auto issue = [&](int c) {
     if (c < chunks) {
-      const Planes d = stage(c);
-      const bf16* src = p.ws_t + ((first + c) * H + hd) * 2 * DK * DK;
-      for (int i = tid; i < 2 * DK * (DK / 8); i += kThreads) {
-        const int pl = i / (DK * (DK / 8)), e = i - pl * (DK * (DK / 8)), r = e / (DK / 8), cc = (e - r * (DK / 8)) * 8;
-        cp16((pl ? d.lo : d.hi) + r * Lay::ldt + cc, src + (size_t)i * 8, true);
-      }
+      const uint4* src = p.ws_t + ((first + c) * H + hd) * (DK * DK / 4);
+      uint4* dst = reinterpret_cast<uint4*>(sm + (c & 1) * Lay::t_stage);
+      for (int i = tid; i < DK * DK / 4; i += kThreads) cp16(dst + i, src + i, true);
     }
     cp_commit();
   };
@@ -628,16 +674,8 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
     issue(c + 1);
     // this chunk's additions, on their way while the start state is laid out
     float e[N8][4];
-    const float* ge = p.ws_e + ci * DK * DV + c0;
     const float d0 = p.ws_d[ci * DK + m0 + g], d1 = p.ws_d[ci * DK + m0 + g + 8];
-#pragma unroll
-    for (int i = 0; i < N8; ++i)
-#pragma unroll
-      for (int h2 = 0; h2 < 2; ++h2) {
-        const float2 v = *reinterpret_cast<const float2*>(ge + (size_t)(m0 + g + 8 * h2) * DV + n0 + i * 8 + 2 * t);
-        e[i][2 * h2] = v.x;
-        e[i][2 * h2 + 1] = v.y;
-      }
+    get_c<N8>(p.ws_e + ci * (DK * DV / 4), DV / 8, m0, c0 + n0, e);
     put_acc<N8>(S, m0, n0, s, 1.f);
     bf16* gs = p.ws_s + ci * 2 * DK * DV + c0;
     put_acc<N8>(Planes{gs, gs + DK * DV, DV}, m0, n0, s, 1.f);
@@ -648,7 +686,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
       s[i][0] = fmaf(d0, s[i][0], e[i][0]); s[i][1] = fmaf(d0, s[i][1], e[i][1]);
       s[i][2] = fmaf(d1, s[i][2], e[i][2]); s[i][3] = fmaf(d1, s[i][3], e[i][3]);
     }
-    mm<N8, false, true>(s, stage(c), m0, S, n0, 0, DK);
+    mm_frag<N8>(s, reinterpret_cast<const uint4*>(sm + (c & 1) * Lay::t_stage) + (m0 >> 4) * (DK / 16) * 64, S, n0, DK / 16);
     __syncthreads();                                      // S and this stage are consumed
   }
   cp_wait<0>();
@@ -664,8 +702,8 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
 // ------------------------------------------------------------------ outputs of a chunk
 template <int DK, int DV>
 struct OutLayout {
-  static constexpr int ldr = DK + 8, lds = DV + 8;
-  static constexpr size_t r = 0, s = 2 * (size_t)kC * ldr * 2, bytes = s + 2 * (size_t)DK * lds * 2;
+  static constexpr int lds = DV + 8;
+  static constexpr size_t r = 0, s = (size_t)kC * DK * 4, bytes = s + 2 * (size_t)DK * lds * 2;
 };
 
 template <int DK, int DV>
@@ -680,13 +718,10 @@ __global__ void __launch_bounds__(256, 2) delta_out_kernel(const ChunkParams p) 
   if (c * kC >= n) return;
   const int t0 = p.q_start[seq] + c * kC, valid = min(kC, n - c * kC), H = p.in.H;
   const size_t ci = ((size_t)(p.q_start[seq] / kC + seq + c)) * H + hd;
-  const Planes R{reinterpret_cast<bf16*>(sm + Lay::r), reinterpret_cast<bf16*>(sm + Lay::r) + kC * Lay::ldr, Lay::ldr};
   const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
-  const bf16 *gr = p.ws_r + ci * 2 * kC * DK, *gs = p.ws_s + ci * 2 * DK * DV;
-  for (int i = tid; i < 2 * kC * (DK / 8); i += 256) {
-    const int pl = i / (kC * (DK / 8)), e = i - pl * (kC * (DK / 8)), r = e / (DK / 8), cc = (e - r * (DK / 8)) * 8;
-    cp16((pl ? R.lo : R.hi) + r * Lay::ldr + cc, gr + (size_t)i * 8, true);
-  }
+  const uint4* gr = p.ws_r + ci * (kC * DK / 4);
+  const bf16* gs = p.ws_s + ci * 2 * DK * DV;
+  for (int i = tid; i < kC * DK / 4; i += 256) cp16(sm + Lay::r + (size_t)i * 16, gr + i, true);
   for (int i = tid; i < 2 * DK * (DV / 8); i += 256) {
     const int pl = i / (DK * (DV / 8)), e = i - pl * (DK * (DV / 8)), r = e / (DV / 8), cc = (e - r * (DV / 8)) * 8;
     cp16((pl ? S.lo : S.hi) + r * Lay::lds + cc, gs + (size_t)i * 8, true);
@@ -695,18 +730,10 @@ __global__ void __launch_bounds__(256, 2) delta_out_kernel(const ChunkParams p) 
   constexpr int NV = DV / 16;
   const int i0 = (warp & 3) * 16, half = warp >> 2, nv0 = half * (DV / 2);
   float o[NV][4];
-  const float* go = p.ws_o + ci * kC * DV;
-#pragma unroll
-  for (int i = 0; i < NV; ++i)
-#pragma unroll
-    for (int h2 = 0; h2 < 2; ++h2) {
-      const float2 v = *reinterpret_cast<const float2*>(go + (size_t)(i0 + g + 8 * h2) * DV + nv0 + i * 8 + 2 * t);
-      o[i][2 * h2] = v.x;
-      o[i][2 * h2 + 1] = v.y;
-    }
+  get_c<NV>(p.ws_o + ci * (kC * DV / 4), DV / 8, i0, nv0, o);
   cp_wait<0>();
   __syncthreads();
-  mm<NV, false, true>(o, R, i0, S, nv0, 0, DK);
+  mm_frag<NV>(o, reinterpret_cast<const uint4*>(sm + Lay::r) + (i0 >> 4) * (DK / 16) * 64, S, nv0, DK / 16);
   if (!p.norm_w) {
 #pragma unroll
     for (int h2 = 0; h2 < 2; ++h2) {
@@ -811,7 +838,7 @@ extern "C" int mb_delta_chunked(const MbDeltaChunkedArgs* a, cudaStream_t stream
   if (a->num_seqs <= 0 || a->num_seqs > 65535 || a->in.H > 65535 || a->max_q_len <= 0 || a->total_rows <= 0) return MB_ERR_BAD_ARG;
   const DeltaInputs& in = a->in;
   const auto bad = [](const void* ptr, long long ld) { return (reinterpret_cast<uintptr_t>(ptr) & 15) || ld % 8; };
-  if (bad(in.q, in.q_ld) || bad(in.k, in.k_ld) || bad(in.v, in.v_ld) || (in.general && bad(in.removal, in.removal_ld)) || bad(a->state, 0) ||
+  if (bad(in.q, in.q_ld) || bad(in.k, in.k_ld) || bad(in.v, in.v_ld) || (in.general && (bad(in.removal, in.removal_ld) || bad(in.log_w, 0))) || bad(a->state, 0) ||
       bad(a->out, 0) || bad(a->ws, 0))
     return MB_ERR_UNSUPPORTED;                             // 16-byte copies
   if (a->norm_w && (!a->gate || !a->norm_out || a->gate_ld % 2 || a->norm_out_ld % 2 || (reinterpret_cast<uintptr_t>(a->gate) & 3) ||
@@ -821,12 +848,12 @@ extern "C" int mb_delta_chunked(const MbDeltaChunkedArgs* a, cudaStream_t stream
   ChunkParams p{};
   p.in = in; p.state = a->state; p.out = a->out;
   const size_t chunks = ((size_t)a->total_rows / kC + a->num_seqs) * in.H, kk = (size_t)in.DK * in.DK, kv = (size_t)in.DK * in.DV;
-  p.ws_t = reinterpret_cast<bf16*>(a->ws);
-  p.ws_e = reinterpret_cast<float*>(p.ws_t + chunks * 2 * kk);
-  p.ws_s = reinterpret_cast<bf16*>(p.ws_e + chunks * kv);
-  p.ws_r = p.ws_s + chunks * 2 * kv;
-  p.ws_o = reinterpret_cast<float*>(p.ws_r + chunks * 2 * kC * in.DK);
-  p.ws_d = p.ws_o + chunks * kC * in.DV;
+  p.ws_t = reinterpret_cast<uint4*>(a->ws);
+  p.ws_e = reinterpret_cast<float4*>(p.ws_t + chunks * (kk / 4));
+  p.ws_s = reinterpret_cast<bf16*>(p.ws_e + chunks * (kv / 4));
+  p.ws_r = reinterpret_cast<uint4*>(p.ws_s + chunks * 2 * kv);
+  p.ws_o = reinterpret_cast<float4*>(p.ws_r + chunks * (kC * in.DK / 4));
+  p.ws_d = reinterpret_cast<float*>(p.ws_o + chunks * (kC * in.DV / 4));
   p.q_start = a->q_start; p.q_len = a->q_len; p.positions = a->positions; p.slots = a->slots;
   p.num_slots = a->num_slots; p.write_state = a->write_state; p.status = a->status;
   p.norm_w = (const bf16*)a->norm_w; p.gate = (const bf16*)a->gate; p.gate_ld = a->gate_ld; p.sigmoid_gate = a->sigmoid_gate;
