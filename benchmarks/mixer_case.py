@@ -1,7 +1,8 @@
 """One launch sequence on a small case, for a profiler: decode | chunk (recurrence, time-mix mode), gla (the same
 recurrence read after its update, with low-rank decays and the head norm), latent-decode | latent (latent attention),
 hyper (residual streams: join, read, norm), window-decode | window (windowed attention with kept tokens and gates),
-gated-delta | general-delta (delta rules with their head norm; -decode: one token each), canon (join and convolution)."""
+gated-delta | general-delta (delta rules with their head norm; -decode: one token each), canon (join and convolution), capped-decode | capped
+(attention with capped scores whose outputs are turned back)."""
 import os
 import sys
 
@@ -44,6 +45,14 @@ elif case == "canon":
     x, y, win = rnd(T, W, dtype=torch.float32), mx.SublayerOut(rnd(T, W)), canon.Window(torch.zeros(4, 2 * W, device="cuda"), 0, W)
     nm, filt = mx.RmsNorm(rnd(W), 1e-6, plus_one=True), rnd(3, W)
     run = lambda: canon.stream_canon(x, "bf16", pending=y, norm=nm, filt=filt, window=win, batch=b)
+elif case.startswith("capped"):
+    from metrale_inference_alpha_b200.ops import reference as ref
+    lens, start = ([1] * 128, 1023) if case == "capped-decode" else ([4096], 0)
+    b, blocks = batch(lens, start)
+    T, H, G = sum(lens), 32, 8
+    kc, vc, q = rnd(blocks, 16, G, D), rnd(blocks, 16, G, D), rnd(T, H, D)
+    out, turn = torch.empty(T, H * D, dtype=q.dtype, device="cuda"), ref.rope_tables(8192, D, 1e4, device="cuda")
+    run = lambda: mx.attention_dims(q, kc, vc, b, dk=D, dv=D, scale=0.09, sink=False, fmt="bf16", out=out, softcap=30.0, turn_back=turn)
 elif case.startswith("window"):
     lens, start = ([1] * 128, 1023) if case == "window-decode" else ([4096], 0)
     b, blocks = batch(lens, start)

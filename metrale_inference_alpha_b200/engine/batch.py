@@ -27,7 +27,7 @@ class SpecStash:
     def __init__(self, batch: "ForwardBatch"):
         self.batch = batch
         self.layers = {}                 # recurrent layer index -> tuple of retained tensors
-        self.later = []                  # or the commit itself, a function of the batch of accepted rows
+        self.later = {}                  # or the commit itself, by what it advances: a function of the batch of accepted rows
 
 
 @dataclass

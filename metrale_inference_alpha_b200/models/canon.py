@@ -53,8 +53,8 @@ def delta_mixer(dec, a, lw, batch, window: Window, state, fmt: str, stash):
                     norm=dict(w=w.norm, gate=_cols(y, at["g"]), gate_act="silu", eps=dec.cfg.rms_eps, scale=1.0, out=out))
     if stash is not None:
         x = _cols(y, at["qkv"])
-        stash.later.append(lambda cb: short_conv(x, w.conv, window, cb, fmt, write_out=False))
-        stash.later.append(lambda cb: delta_attention(q, k, v, rule, state, cb, write_out=False, kernel="seq", **kw))
+        stash.later[window.rows.data_ptr(), window.at] = lambda cb: short_conv(x, w.conv, window, cb, fmt, write_out=False)
+        stash.later[state.data_ptr()] = lambda cb: delta_attention(q, k, v, rule, state, cb, write_out=False, kernel="seq", **kw)
     return ops.linear(mx.act_of(out, fmt), w.o)
 
 
@@ -86,14 +86,14 @@ def twin_mixer(dec, a, lw, batch, kc, vc, state, fmt: str, stash):
         rule = rule if ws else rule.logs()
         delta_attention(q, k, v, rule, state, batch, heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt, write_state=ws, norm=norm)
         if stash is not None:
-            stash.later.append(lambda cb: delta_attention(q, k, v, rule, state, cb, heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt,
-                                                          write_out=False, kernel="seq"))
+            stash.later[state.data_ptr()] = lambda cb: delta_attention(q, k, v, rule, state, cb, heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt,
+                                                                       write_out=False, kernel="seq")
     else:
         kw = dict(heads=R.heads, dk=R.dim, dv=R.vdim, fmt=fmt, decay=R.decay)
         core = mx.linear_attention(q, k, v, state, batch, write_state=ws, **kw)
         mx.gated_norm(core, norm.pop("w"), norm.pop("gate"), fmt, group=nr, **norm)
         if stash is not None:
-            stash.later.append(lambda cb: mx.linear_attention(q, k, v, state, cb, write_out=False, **kw))
+            stash.later[state.data_ptr()] = lambda cb: mx.linear_attention(q, k, v, state, cb, write_out=False, **kw)
     return ops.linear(mx.act_of(cat, fmt), w.o)
 
 

@@ -128,7 +128,7 @@ def commit_recurrent(cfg, pool, stash, commit_batch) -> None:
     """Advance the state of every recurrent layer by the accepted rows of a verify step:
     `commit_batch` is that step's batch with q_len replaced by the number of rows to commit per
     sequence (0 = leave the sequence's state as it was)."""
-    for commit_rows in stash.later:
+    for commit_rows in stash.later.values():
         commit_rows(commit_batch)
     for sidx, (kind, lw, x_in, conv_out, gate) in stash.layers.items():
         w = lw.mixer

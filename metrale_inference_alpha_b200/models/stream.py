@@ -136,9 +136,9 @@ class CanonStream:
     def read(self, filt: torch.Tensor, window: "canon.Window", batch, stash=None) -> torch.Tensor:
         """The next sublayer's input; the window moves on, or waits for the accepted rows of a verify step."""
         h = self._step(filt=filt, window=window, batch=batch, write_state=stash is None)
-        if stash is not None:
+        if stash is not None and filt.shape[0] > 1:
             x, taps = self.x, filt.shape[0]
-            stash.later.append(lambda cb: canon.canon_commit(x, taps, window, cb))
+            stash.later[window.rows.data_ptr(), window.at] = lambda cb: canon.canon_commit(x, taps, window, cb)
         return h
 
     def add(self, out: mx.SublayerOut, post: mx.RmsNorm) -> "CanonStream":

@@ -44,7 +44,7 @@ def config(layers, width, taps=3, vocab=150, eps=1e-5, embed=2.0, logit=0.7):
 # ragged: rows that are not whole 16-byte vectors, head sizes away from every tile, a layer without feed-forward, a mixture
 #   without shared expert, several value heads to a key head, a large eps
 # tiles: aligned sizes, the chunked kernels' head sizes, unequal key and value sizes
-# ones: single heads, experts and taps, a window of one, factors of one
+# ones: single heads, experts and taps (and a short convolution of three beside inputs without one), a window of one, factors of one
 # wide: heads past 128 (and past 256 values), filters longer than a run of tokens is short, a rank past what decode computes
 CONFIGS = {
     "ragged": config([delta(6, 3, 18, 22, 2, moe(6, 2, 18, 26)), capped((3, 1, 22, 30, 10), (3, 20, 26), moe(5, 3, 22)),
@@ -54,7 +54,7 @@ CONFIGS = {
                      capped((4, 4, 128, 64, 64), (2, 128, 64), moe(4, 2, 40, 128)), delta(2, 2, 128, 64, 3, moe(3, 1, 32, 32))], 128, taps=2, vocab=128),
     "ones": config([capped((1, 1, 16, 16, 2), (1, 16, 16), moe(1, 1, 32, 32), softcap=1.0, factor=1.0, scales=(1.0, 1.0), scale=1.0),
                     windowed((1, 1, 16, 2, 1), (1, 16), moe(2, 1, 32), scaling=(1.0, 1, 1.0, 1.0), scales=(1.0, 1.0), scale=1.0),
-                    delta(1, 1, 16, 16, 1, moe(1, 1, 16, 16))], 64, taps=1, embed=1.0, logit=1.0),
+                    delta(1, 1, 16, 16, 1, moe(1, 1, 16, 16)), delta(1, 1, 16, 16, 3)], 64, taps=1, embed=1.0, logit=1.0),
     "wide": config([delta(2, 1, 136, 264, 7, moe(4, 2, 96, 160)), capped((2, 1, 200, 72, 96), (2, 130, 12), moe(5, 2, 64)),
                     windowed((3, 1, 264, 40, 70), (1, 200), moe(3, 3, 40, 8)), capped((4, 2, 128, 128, 128), (3, 64, 128))], 256, taps=12),
 }

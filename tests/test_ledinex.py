@@ -678,6 +678,22 @@ def test_greedy_generation_scheduler_and_speculation(tmp_path, device):
 
 
 @pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("name", ["ragged", "ones"])
+def test_verify_steps_of_one_request(tmp_path, device, name):
+    """A request alone whose predicted output is right, wrong, right again: every verify step has as many drafts (on the GPU
+    they replay one graph), and accepts all, some or none of them."""
+    path = lc.checkpoint(lc.CONFIGS[name], lc.weights(lc.CONFIGS[name]), tmp_path / "m")
+    prompt = lc.tokens(lc.CONFIGS[name], 7, 3)
+    want = greedy_reference(name, prompt, 24)
+    guess = [(w + 1) % 150 if i in (5, 6, 13) else w for i, w in enumerate(want)]
+    eng = LLMEngine(EngineArgs(model=path, device=device, dtype="fp32", max_num_seqs=2, max_model_len=96, num_kv_blocks=24))
+    for _ in range(2):
+        out = eng.generate([prompt], SamplingParams(max_tokens=24, temperature=0.0, prediction_ids=guess))[0]
+        assert out.output_ids == want and out.accepted_draft_tokens > 8
+    assert device == "cpu" or any(k[0] == "verify" for k in eng.runner.graphs)
+
+
+@pytest.mark.parametrize("device", DEVICES)
 def test_prefix_cache(tmp_path, device):
     path = lc.checkpoint(lc.CONFIGS["ragged"], lc.weights(lc.CONFIGS["ragged"]), tmp_path / "m")
     eng = LLMEngine(EngineArgs(model=path, device=device, dtype="fp32", max_num_seqs=2, max_model_len=400, num_kv_blocks=80))
