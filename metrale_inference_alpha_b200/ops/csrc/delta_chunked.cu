@@ -225,6 +225,7 @@ __device__ __forceinline__ void get_c(const float4* src, int tiles, int m0, int 
 }
 
 // ------------------------------------------------------------------ per-chunk preparation
+constexpr int kPrep = 512;         // threads
 constexpr int kLdF = kC + 4;       // fp32 rows of the inverse
 constexpr int kLdC = kC + 8;       // bf16 rows of 64 x 64 matrices
 
@@ -240,7 +241,7 @@ struct PrepLayout {
 };
 
 template <int DK, int DV, bool GEN>
-__global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(kPrep, 1) delta_prep_kernel(const ChunkParams p) {
   using Lay = PrepLayout<DK, DV>;
   extern __shared__ __align__(16) uint8_t sm[];
   const DeltaInputs& in = p.in;
@@ -270,7 +271,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   // everything the chunk reads, at once: values and the raw rows of keys, queries and removal logits (a row's owner makes
   // its operands of them in place), log decays
   auto rows_in = [&](const void* base, long long ld, int head, int D, bf16* dst, int dst_ld) {
-    for (int i = tid; i < kC * (D / 8); i += 256) {
+    for (int i = tid; i < kC * (D / 8); i += kPrep) {
       const int r = i / (D / 8), cc = (i - r * (D / 8)) * 8;
       const bool ok = r < valid;
       cp16(dst + r * dst_ld + cc, reinterpret_cast<const bf16*>(base) + (ok ? (size_t)(t0 + r) * ld + (size_t)head * D + cc : 0), ok);
@@ -282,7 +283,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   rows_in(in.v, in.v_ld, hd, DV, V.hi, Lay::ldv);
   if constexpr (GEN) {
     rows_in(in.removal, in.removal_ld, hd, DK, B.hi, Lay::ldk);
-    for (int i = tid; i < kC * (DK / 4); i += 256) {
+    for (int i = tid; i < kC * (DK / 4); i += kPrep) {
       const int r = i / (DK / 4), cc = (i - r * (DK / 4)) * 4;
       const bool ok = r < valid;
       cp16(sL + r * ldl + cc, in.log_w + (ok ? ((size_t)(t0 + r) * H + hd) * DK + cc : 0), ok);
@@ -291,7 +292,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   cp_commit();
   if constexpr (GEN) {
     // running sums of log2 decays; rows past `valid` repeat the last
-    constexpr int kR = kC * DK / 256;
+    constexpr int kR = kC * DK / kPrep;
     const int d = tid % DK, grp = tid / DK, r0 = grp * kR;
     cp_wait<0>();
     __syncthreads();
@@ -351,7 +352,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
       }
     };
 #pragma unroll 2
-    for (int i = warp; i < kC; i += 8) {
+    for (int i = warp; i < kC; i += kPrep / 32) {
       float q[E], k[E], a[E];
       load(R.hi + i * Lay::ldk + d0, q);
       load(U.hi + i * Lay::ldk + d0, k);
@@ -390,15 +391,15 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     }
   }
   __syncthreads();
-  // ---- scores of this warp's 16 rows and 32 columns, blocks up to the diagonal: rows U and R against columns B (and K)
-  // (warps w and w + 4 share a scheduler: a long row block of a triangle goes with a short one)
-  const int half = warp >> 2, rb = half ? 3 - (warp & 3) : warp & 3, i0 = rb * 16, j0 = half * 32;
-  float sa[4][4], sb[GEN ? 4 : 1][4], sp[GEN ? 4 : 1][4], sq[4][4];
-  zero<4>(sa);
-  zero<4>(sq);
+  // ---- scores of this warp's 16 rows and 16 columns, blocks up to the diagonal: rows U and R against columns B (and K)
+  // (warps w, w + 4 ... share a scheduler: a long row block of a triangle goes with a short one)
+  const int quarter = warp >> 2, rb = quarter & 1 ? 3 - (warp & 3) : warp & 3, i0 = rb * 16, j0 = quarter * 16;
+  float sa[2][4], sb[GEN ? 2 : 1][4], sp[GEN ? 2 : 1][4], sq[2][4];
+  zero<2>(sa);
+  zero<2>(sq);
   if constexpr (GEN) {
-    zero<4>(sb);
-    zero<4>(sp);
+    zero<2>(sb);
+    zero<2>(sp);
   }
   const Planes& CB = GEN ? B : U;
   if (j0 <= i0) {
@@ -412,22 +413,20 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
         ldsm4(ul, U.lo + o);
         ldsm4(rl, R.lo + o);
       }
-#pragma unroll
-      for (int jb = 0; jb < 2; ++jb) {
-        if (j0 + jb * 16 > i0) continue;
-        const int row = j0 + jb * 16 + (lane & 7) + ((lane >> 4) << 3), col = k0 + ((lane >> 3) & 1) * 8;
+      {
+        const int row = j0 + (lane & 7) + ((lane >> 4) << 3), col = k0 + ((lane >> 3) & 1) * 8;
         uint32_t bh[4], bl[4];
         ldsm4(bh, CB.hi + (size_t)row * CB.ld + col);
         if constexpr (GEN) ldsm4(bl, CB.lo + (size_t)row * CB.ld + col);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          mma(sa[jb * 2 + e], uh, bh[2 * e], bh[2 * e + 1]);
-          mma(sq[jb * 2 + e], rh, bh[2 * e], bh[2 * e + 1]);
+          mma(sa[e], uh, bh[2 * e], bh[2 * e + 1]);
+          mma(sq[e], rh, bh[2 * e], bh[2 * e + 1]);
           if constexpr (GEN) {
-            mma(sa[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
-            mma(sq[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
-            mma(sa[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
-            mma(sq[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+            mma(sa[e], uh, bl[2 * e], bl[2 * e + 1]);
+            mma(sq[e], rh, bl[2 * e], bl[2 * e + 1]);
+            mma(sa[e], ul, bh[2 * e], bh[2 * e + 1]);
+            mma(sq[e], rl, bh[2 * e], bh[2 * e + 1]);
           }
         }
         if constexpr (GEN) {
@@ -435,12 +434,12 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
           ldsm4(bl, K.lo + (size_t)row * K.ld + col);
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            mma(sb[jb * 2 + e], uh, bh[2 * e], bh[2 * e + 1]);
-            mma(sp[jb * 2 + e], rh, bh[2 * e], bh[2 * e + 1]);
-            mma(sb[jb * 2 + e], uh, bl[2 * e], bl[2 * e + 1]);
-            mma(sp[jb * 2 + e], rh, bl[2 * e], bl[2 * e + 1]);
-            mma(sb[jb * 2 + e], ul, bh[2 * e], bh[2 * e + 1]);
-            mma(sp[jb * 2 + e], rl, bh[2 * e], bh[2 * e + 1]);
+            mma(sb[e], uh, bh[2 * e], bh[2 * e + 1]);
+            mma(sp[e], rh, bh[2 * e], bh[2 * e + 1]);
+            mma(sb[e], uh, bl[2 * e], bl[2 * e + 1]);
+            mma(sp[e], rh, bl[2 * e], bl[2 * e + 1]);
+            mma(sb[e], ul, bh[2 * e], bh[2 * e + 1]);
+            mma(sp[e], rl, bh[2 * e], bh[2 * e + 1]);
           }
         }
       }
@@ -448,7 +447,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   }
   __syncthreads();                                        // the logs are consumed: their space takes A
 #pragma unroll
-  for (int e = 0; e < 4; ++e)
+  for (int e = 0; e < 2; ++e)
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
       const int i = i0 + g + (x >> 1) * 8, j = j0 + e * 8 + 2 * t + (x & 1);
@@ -468,7 +467,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     }
   __syncthreads();
   // ---- M = (I + A)^-1: 16 x 16 diagonal blocks by substitution, a column per thread, then block by block below
-  for (int e = tid; e < kC * kC; e += 256) {
+  for (int e = tid; e < kC * kC; e += kPrep) {
     const int i = e >> 6, j = e & 63;
     if ((j >> 4) > (i >> 4)) sM[i * kLdF + j] = 0.f;
   }
@@ -487,16 +486,16 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   }
   __syncthreads();
   {
-    const int r = tid >> 4, cc = tid & 15;
+    const int r = (tid >> 4) & 15, cc = tid & 15, side = tid >> 8;
     for (int lev = 1; lev < 4; ++lev) {
-      for (int jb = 0; jb + lev < 4; ++jb) {
+      for (int jb = side; jb + lev < 4; jb += kPrep / 256) {
         const int ib = jb + lev;
         float s = 0.f;
         for (int k = jb * 16; k < ib * 16; ++k) s = fmaf(sA[(ib * 16 + r) * kLdF + k], sM[k * kLdF + jb * 16 + cc], s);
         sT[(jb * 16 + r) * 17 + cc] = s;
       }
       __syncthreads();
-      for (int jb = 0; jb + lev < 4; ++jb) {
+      for (int jb = side; jb + lev < 4; jb += kPrep / 256) {
         const int ib = jb + lev;
         float s = 0.f;
 #pragma unroll
@@ -508,7 +507,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   }
   // M as planes; gated: times diag(beta 2^G / |k|) for Xw, diag(beta) for Xu
   auto put_m = [&](bool decayed) {
-    for (int e = tid; e < kC * kC / 2; e += 256) {
+    for (int e = tid; e < kC * kC / 2; e += kPrep) {
       const int i = e >> 5, j = (e & 31) * 2;
       float a = sM[i * kLdF + j], b = sM[i * kLdF + j + 1];
       if constexpr (!GEN) {
@@ -520,9 +519,9 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   };
   put_m(true);
   __syncthreads();
-  // ---- Xw = -M U and Xu; this warp's 16 rows and one half of the columns
-  constexpr int NK = DK / 16, NV = DV / 16;
-  const int nk0 = half * (DK / 2), nv0 = half * (DV / 2), kend = i0 + 16;
+  // ---- Xw = -M U and Xu; this warp's 16 rows and a quarter of the columns
+  constexpr int NK = DK / 32, NV = DV / 32;
+  const int nk0 = quarter * (DK / 4), nv0 = quarter * (DV / 4), kend = i0 + 16;
   float xw[NK][4], xu[NV][4];
   zero<NK>(xw);
   zero<NV>(xu);
@@ -531,20 +530,20 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   float po[NV][4];                                        // O'
   zero<NV>(po);
   if constexpr (GEN) {
-    put_acc<4>(Z1, i0, j0, sb, 1.f);
+    put_acc<2>(Z1, i0, j0, sb, 1.f);
     __syncthreads();
-    float mbv[4][4];
-    zero<4>(mbv);
-    mm<4, false, true>(mbv, Z0, i0, Z1, j0, 0, kend);
+    float mbv[2][4];
+    zero<2>(mbv);
+    mm<2, false, true>(mbv, Z0, i0, Z1, j0, 0, kend);
     __syncthreads();
-    put_acc<4>(Z0, i0, j0, mbv, -1.f);
-    put_acc<4>(Z1, i0, j0, sp, 1.f);
+    put_acc<2>(Z0, i0, j0, mbv, -1.f);
+    put_acc<2>(Z1, i0, j0, sp, 1.f);
     put_acc<NK>(XW, i0, nk0, xw, -1.f);
     __syncthreads();
     mm<NV, false, false>(xu, Z0, i0, V, nv0, 0, kend);
     mm<NV, false, false>(po, Z1, i0, V, nv0, 0, kend);
     __syncthreads();
-    put_acc<4>(Z0, i0, j0, sq, 1.f);
+    put_acc<2>(Z0, i0, j0, sq, 1.f);
   } else {
     __syncthreads();
     put_m(false);
@@ -552,7 +551,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     __syncthreads();
     mm<NV, false, false>(xu, Z0, i0, V, nv0, 0, kend);
     __syncthreads();
-    put_acc<4>(Z0, i0, j0, sq, 1.f);
+    put_acc<2>(Z0, i0, j0, sq, 1.f);
     put_acc<NV>(K, i0, nv0, xu, 1.f);
   }
   __syncthreads();
@@ -578,8 +577,8 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
     mm<NK, false, true>(acc, Z0, i0, XW, nk0, 0, kend);
     put_frag<NK>(p.ws_r + ci * (kC * DK / 4), DK / 16, i0, nk0, acc);
   }
-  // ---- the state's side: 16 key rows per warp (and, for 64 of them, half of the columns)
-  constexpr int kMB = DK / 16, kCW = 8 / kMB, NE = DV / 8 / kCW, NT = DK / 8 / kCW;
+  // ---- the state's side: 16 key rows and a part of the columns per warp
+  constexpr int kMB = DK / 16, kCW = kPrep / 32 / kMB, NE = DV / 8 / kCW, NT = DK / 8 / kCW;
   const int m0 = (warp % kMB) * 16, e0 = (warp / kMB) * NE * 8, x0 = (warp / kMB) * NT * 8;
   float acc_e[NE][4];
   zero<NE>(acc_e);
@@ -594,7 +593,7 @@ __global__ void __launch_bounds__(256, 1) delta_prep_kernel(const ChunkParams p)
   if constexpr (!GEN) {                                   // rows of X decayed to the chunk's end and over the keys' lengths, in place
     __syncthreads();
     const double gl = sG[kC - 1];
-    for (int e = tid; e < kC * (DK + DV) / 2; e += 256) {
+    for (int e = tid; e < kC * (DK + DV) / 2; e += kPrep) {
       const int i = e / ((DK + DV) / 2), d = (e - i * ((DK + DV) / 2)) * 2;
       const float f = i < valid ? ex2((float)(gl - sG[i])) * sNk[i] : 0.f;
       const Planes& X = d < DK ? XW : K;
@@ -629,8 +628,11 @@ struct ScanLayout {
   static constexpr size_t t_stage = (size_t)DK * DK * 4, s = 2 * t_stage, bytes = s + 2 * (size_t)DK * lds * 2;
 };
 
+template <int DK, int SLICE>
+constexpr int scan_threads() { return DK / 16 * (SLICE / 16) * 32; }    // a warp per 16 x 16 block of the slice
+
 template <int DK, int DV, int SLICE>
-__global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(scan_threads<DK, SLICE>(), 1) delta_scan_kernel(const ChunkParams p) {
   using Lay = ScanLayout<DK, SLICE>;
   extern __shared__ __align__(16) uint8_t sm[];
   const int slice = blockIdx.x, hd = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -645,7 +647,7 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkParams p)
   }
   const int chunks = (n + kC - 1) / kC, c0 = slice * SLICE;
   const size_t first = (size_t)(p.q_start[seq] / kC + seq);
-  constexpr int kMB = DK / 16, kThreads = SLICE == 32 || DK == 128 ? 256 : 128, kCW = kThreads / 32 / kMB, N8 = SLICE / 8 / kCW;
+  constexpr int kMB = DK / 16, kThreads = scan_threads<DK, SLICE>(), N8 = 2;
   const int m0 = (warp % kMB) * 16, n0 = (warp / kMB) * N8 * 8;
   const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
   auto issue = [&](int c) {
@@ -789,12 +791,12 @@ int launch_chunks(const ChunkParams& p, int num_seqs, int max_q_len, cudaStream_
     configured = true;
   }
   const dim3 grid((max_q_len + kC - 1) / kC, p.in.H, num_seqs);
-  cudaError_t e = mb::launch_kernel(delta_prep_kernel<DK, DV, GEN>, grid, dim3(256), sp, stream, p);
+  cudaError_t e = mb::launch_kernel(delta_prep_kernel<DK, DV, GEN>, grid, dim3(kPrep), sp, stream, p);
   if (e == cudaSuccess) {
     if ((long long)DV / 16 * p.in.H * num_seqs <= sms)
-      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 16>, dim3(DV / 16, p.in.H, num_seqs), dim3(DK == 128 ? 256 : 128), ScanLayout<DK, 16>::bytes, stream, p);
+      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 16>, dim3(DV / 16, p.in.H, num_seqs), dim3(scan_threads<DK, 16>()), ScanLayout<DK, 16>::bytes, stream, p);
     else
-      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 32>, dim3(DV / 32, p.in.H, num_seqs), dim3(256), ScanLayout<DK, 32>::bytes, stream, p);
+      e = mb::launch_kernel(delta_scan_kernel<DK, DV, 32>, dim3(DV / 32, p.in.H, num_seqs), dim3(scan_threads<DK, 32>()), ScanLayout<DK, 32>::bytes, stream, p);
   }
   if (e == cudaSuccess) e = mb::launch_kernel(delta_out_kernel<DK, DV>, grid, dim3(256), so, stream, p);
   return (int)e;
