@@ -629,7 +629,7 @@ struct ScanLayout {
 };
 
 template <int DK, int SLICE>
-constexpr int scan_threads() { return DK / 16 * (SLICE / 16) * 32; }    // a warp per 16 x 16 block of the slice
+constexpr int scan_threads() { return SLICE == 32 || DK == 128 ? 256 : 128; }
 
 template <int DK, int DV, int SLICE>
 __global__ void __launch_bounds__(scan_threads<DK, SLICE>(), 1) delta_scan_kernel(const ChunkParams p) {
@@ -647,7 +647,7 @@ __global__ void __launch_bounds__(scan_threads<DK, SLICE>(), 1) delta_scan_kerne
   }
   const int chunks = (n + kC - 1) / kC, c0 = slice * SLICE;
   const size_t first = (size_t)(p.q_start[seq] / kC + seq);
-  constexpr int kMB = DK / 16, kThreads = scan_threads<DK, SLICE>(), N8 = 2;
+  constexpr int kMB = DK / 16, kThreads = scan_threads<DK, SLICE>(), kCW = kThreads / 32 / kMB, N8 = SLICE / 8 / kCW;
   const int m0 = (warp % kMB) * 16, n0 = (warp / kMB) * N8 * 8;
   const Planes S{reinterpret_cast<bf16*>(sm + Lay::s), reinterpret_cast<bf16*>(sm + Lay::s) + DK * Lay::lds, Lay::lds};
   auto issue = [&](int c) {
